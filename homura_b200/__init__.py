@@ -93,6 +93,10 @@ class _KernelStat(C.Structure):
     _fields_ = [("name", C.c_char * 32), ("launches_per_step", C.c_int32), ("ms_per_step", C.c_float), ("bytes_per_step", C.c_uint64)]
 
 
+class _StepEntry(C.Structure):
+    _fields_ = [("seq", C.c_int32), ("n_tokens", C.c_int32), ("tokens", C.c_void_p), ("n_want", C.c_int32), ("want", C.c_void_p)]
+
+
 _vp, _i32, _u32p, _i32p, _f32p, _i64p = C.c_void_p, C.c_int, C.POINTER(C.c_uint32), C.POINTER(C.c_int32), C.POINTER(C.c_float), C.POINTER(C.c_int64)
 
 # name -> (restype, argtypes); every symbol include/homura_b200.h declares
@@ -103,6 +107,8 @@ SIGNATURES = {
     "hm_model_load": (_i32, [C.c_char_p, _i32, _i32, C.POINTER(_vp)]),
     "hm_model_load_gguf": (_i32, [C.c_char_p, _i32, C.POINTER(_vp)]),
     "hm_engine_create": (_i32, [C.POINTER(_Config), _i32, C.POINTER(_vp)]),
+    "hm_engine_create_json": (_i32, [C.c_char_p, _i32, _i32, C.POINTER(_vp)]),
+    "hm_get_arch": (C.c_char_p, [_vp]),
     "hm_load_tensor": (_i32, [_vp, C.c_char_p, _i32, _i64p, _i32, _vp, C.c_size_t]),
     "hm_finalize_weights": (_i32, [_vp]),
     "hm_engine_destroy": (None, [_vp]),
@@ -111,11 +117,15 @@ SIGNATURES = {
     "hm_weight_bytes": (_i32, [_vp, C.POINTER(C.c_uint64)]),
     "hm_checkpoint_info": (_i32, [C.c_char_p, C.c_char_p, C.c_size_t, C.POINTER(C.c_size_t)]),
     "hm_kv_alloc": (_i32, [_vp, _i32, _i32, _i32, _i32]),
+    "hm_kv_alloc_pool": (_i32, [_vp, _i32, _i32, C.c_long, _i32, _i32]),
+    "hm_kv_free_tokens": (_i32, [_vp, C.POINTER(C.c_long)]),
     "hm_kv_free": (_i32, [_vp]),
     "hm_kv_reset": (_i32, [_vp, _i32]),
     "hm_kv_len": (_i32, [_vp, _i32, _i32p]),
     "hm_kv_append": (_i32, [_vp, _i32, _i32, _vp, _vp, _i32, _i32]),
     "hm_kv_view": (_i32, [_vp, _i32, _i32, _vp, _vp]),
+    "hm_latent_view": (_i32, [_vp, _i32, _i32, _vp]),
+    "hm_step": (_i32, [_vp, C.POINTER(_StepEntry), _i32, _vp, _vp, _vp]),
     "hm_prefill": (_i32, [_vp, _i32, _vp, _i32, _vp, _u32p]),
     "hm_decode_step": (_i32, [_vp, _vp, _vp, _vp]),
     "hm_decode_step_sampled": (_i32, [_vp, _vp, C.POINTER(_Sampling), _vp, _vp, _vp]),
@@ -311,7 +321,7 @@ def sample_token_device(logits, config: SamplingConfig, generated_ids: Sequence[
 
 
 class HfModel:
-    """A decoder-only RoPE transformer resident on one B200 (src/hf/model.rs:17-267)."""
+    """A decoder-only transformer resident on one B200 (src/hf/model.rs:17-267)."""
 
     def __init__(self, handle: int):
         self._h = C.c_void_p(handle)
@@ -359,6 +369,23 @@ class HfModel:
             raise
         return cls(h.value)
 
+    @classmethod
+    def from_config_json(cls, config_json: str, tensors, weight_dtype: DType = DType.BF16, device: int = 0) -> "HfModel":
+        """Like from_tensors, from the text of a config.json (every design the library knows)."""
+        lib = load_library()
+        h = C.c_void_p()
+        _check(lib.hm_engine_create_json(config_json.encode(), int(weight_dtype), device, C.byref(h)))
+        try:
+            for name, dt, shape, arr in tensors:
+                arr = np.ascontiguousarray(arr)
+                shp = (C.c_int64 * len(shape))(*shape)
+                _check(lib.hm_load_tensor(h, name.encode(), int(dt), shp, len(shape), _ptr(arr), arr.nbytes), h)
+            _check(lib.hm_finalize_weights(h), h)
+        except Exception:
+            lib.hm_engine_destroy(h)
+            raise
+        return cls(h.value)
+
     def close(self):
         if self._h:
             self._lib.hm_engine_destroy(self._h)
@@ -374,6 +401,10 @@ class HfModel:
     def config(self) -> TransformerConfig:
         return self._config
 
+    def architecture(self) -> str:
+        """Name of the design; "" for the uniform Qwen2 / Qwen3 / Llama stacks."""
+        return (self._lib.hm_get_arch(self._h) or b"").decode()
+
     def weight_bytes(self) -> int:
         v = C.c_uint64(0)
         _check(self._lib.hm_weight_bytes(self._h, C.byref(v)), self._h)
@@ -385,12 +416,16 @@ class HfModel:
         return v.value
 
     # -- KV cache --
-    def init_kv_cache(self, max_seq_len: int, batch: int = 1, kv_dtype: DType = DType.F32, page_tokens: int = 16):
-        """init_kv_cache (src/hf/model.rs:221-229).  Calling it again replaces the cache."""
+    def init_kv_cache(self, max_seq_len: int, batch: int = 1, kv_dtype: DType = DType.F32, page_tokens: int = 0, pool_tokens: Optional[int] = None):
+        """init_kv_cache (src/hf/model.rs:221-229).  Calling it again replaces the cache.  page_tokens 0: the design's
+        own page size.  With pool_tokens the sequences share a pool of that many tokens and take pages as they grow."""
         if self.batch:
             _check(self._lib.hm_kv_free(self._h), self._h)
             self.batch = 0
-        _check(self._lib.hm_kv_alloc(self._h, batch, max_seq_len, page_tokens, int(kv_dtype)), self._h)
+        if pool_tokens is None:
+            _check(self._lib.hm_kv_alloc(self._h, batch, max_seq_len, page_tokens, int(kv_dtype)), self._h)
+        else:
+            _check(self._lib.hm_kv_alloc_pool(self._h, batch, max_seq_len, pool_tokens, page_tokens, int(kv_dtype)), self._h)
         self.batch, self.max_seq_len = batch, max_seq_len
 
     def reset_kv_cache(self, seq: int = -1):
@@ -418,6 +453,39 @@ class HfModel:
         v = np.zeros_like(k)
         _check(self._lib.hm_kv_view(self._h, seq, layer, _ptr(k), _ptr(v)), self._h)
         return k, v
+
+    def latent_view(self, layer: int, rank: int, seq: int = 0) -> np.ndarray:
+        """[len, rank] latents that `layer` of a latent-attention design reads."""
+        out = np.zeros((self.kv_cache_len(seq), rank), np.float32)
+        _check(self._lib.hm_latent_view(self._h, seq, layer, _ptr(out)), self._h)
+        return out
+
+    def free_tokens(self) -> int:
+        """Tokens that fit the free pages of a shared pool."""
+        v = C.c_long(0)
+        _check(self._lib.hm_kv_free_tokens(self._h, C.byref(v)), self._h)
+        return int(v.value)
+
+    # -- one batch over several sequences --
+    def step(self, entries, want_logits: bool = True, want_greedy: bool = False, want_hidden: bool = False):
+        """entries: [(seq, tokens, wanted places)].  Returns (logits [wanted, vocab] or None, greedy ids or None,
+        residual stream after every layer [layers, tokens, width] or None)."""
+        arr = (_StepEntry * len(entries))()
+        keep = []
+        rows = wants = 0
+        for e, (seq, tokens, want) in zip(arr, entries):
+            t = np.ascontiguousarray(tokens, dtype=np.uint32)
+            w = np.ascontiguousarray(want, dtype=np.int32)
+            keep += [t, w]
+            e.seq, e.n_tokens, e.tokens, e.n_want, e.want = seq, t.size, t.ctypes.data, w.size, w.ctypes.data
+            rows += t.size
+            wants += w.size
+        c = self._config
+        logits = np.empty((wants, c.vocab_size), np.float32) if want_logits else None
+        greedy = np.empty(wants, np.uint32) if want_greedy else None
+        hidden = np.empty((c.num_hidden_layers, rows, c.hidden_size), np.float32) if want_hidden else None
+        _check(self._lib.hm_step(self._h, arr, len(entries), _ptr(logits), _ptr(greedy), _ptr(hidden)), self._h)
+        return logits, greedy, hidden
 
     # -- GenerativeModel --
     def prefill(self, token_ids, seq: int = 0, want_logits: bool = False):

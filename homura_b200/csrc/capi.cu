@@ -291,15 +291,32 @@ int hm_device_count(void) {
 
 const char* hm_last_error_global(void) { return g_err.c_str(); }
 
-int hm_engine_create(const hm_config* cfg, int device, hm_engine** out) {
-    if (!cfg || !out) return gfail(HM_ERR_INVALID, "hm_engine_create: null argument");
+static int create_engine(const ModelSpec& spec, int device, bool strict_f32, hm_engine** out) {
     Engine* e = nullptr;
     std::string err;
-    int rc = Engine::create(*cfg, device, &e, &err);
+    int rc = Engine::create(spec, device, strict_f32, &e, &err);
     if (rc) return gfail(rc, err);
     *out = new hm_engine{e};
     return HM_OK;
 }
+
+int hm_engine_create(const hm_config* cfg, int device, hm_engine** out) {
+    if (!cfg || !out) return gfail(HM_ERR_INVALID, "hm_engine_create: null argument");
+    ModelSpec spec;
+    spec.cfg = *cfg;
+    return create_engine(spec, device, false, out);
+}
+
+int hm_engine_create_json(const char* config_json, int weight_dtype, int device, hm_engine** out) {
+    if (!config_json || !out) return gfail(HM_ERR_INVALID, "hm_engine_create_json: null argument");
+    if (weight_dtype != HM_BF16 && weight_dtype != HM_F32) return gfail(HM_ERR_UNSUPPORTED, "hm_engine_create_json: weight_dtype must be HM_BF16 or HM_F32");
+    ModelSpec spec;
+    std::string err;
+    if (!parse_model_spec(config_json, std::strlen(config_json), &spec, &err)) return gfail(HM_ERR_IO, err);
+    return create_engine(spec, device, weight_dtype == HM_F32, out);
+}
+
+const char* hm_get_arch(hm_engine* e) { return e ? e->impl->spec().arch.c_str() : ""; }
 
 void hm_engine_destroy(hm_engine* e) {
     if (!e) return;
@@ -393,9 +410,9 @@ int hm_model_load(const char* model_dir, int weight_dtype, int device, hm_engine
     if (weight_dtype != HM_BF16 && weight_dtype != HM_F32)
         return gfail(HM_ERR_UNSUPPORTED, "hm_model_load: weight_dtype must be HM_BF16 or HM_F32 (Homura's --dtype bf16 / f32)");
     const std::string dir(model_dir);
-    hm_config cfg;
+    ModelSpec spec;
     std::string err;
-    if (!parse_config_json(dir + "/config.json", &cfg, &err)) return gfail(HM_ERR_IO, err);
+    if (!parse_model_spec_file(dir + "/config.json", &spec, &err)) return gfail(HM_ERR_IO, err);
     NEED_DEVICE();
     std::vector<std::string> files;
     {
@@ -403,7 +420,7 @@ int hm_model_load(const char* model_dir, int weight_dtype, int device, hm_engine
         if (frc) return gfail(frc, err);
     }
     Engine* eng = nullptr;
-    int rc = Engine::create(cfg, device, &eng, &err);
+    int rc = Engine::create(spec, device, weight_dtype == HM_F32, &eng, &err);
     if (rc) return gfail(rc, err);
     for (auto& f : files) {
         MappedFile mf;
@@ -439,11 +456,11 @@ int hm_model_load_gguf(const char* gguf_path, int device, hm_engine** out) {
     if (!mf.open(gguf_path, &err)) return gfail(HM_ERR_IO, err);
     GgufFile g;
     if (!parse_gguf(mf, &g, &err)) return gfail(HM_ERR_IO, err);
-    hm_config cfg;
-    if (!gguf_config(g, &cfg, &err)) return gfail(HM_ERR_IO, err);
+    ModelSpec spec;
+    if (!gguf_config(g, &spec.cfg, &err)) return gfail(HM_ERR_IO, err);
     NEED_DEVICE();
     Engine* eng = nullptr;
-    int rc = Engine::create(cfg, device, &eng, &err);
+    int rc = Engine::create(spec, device, false, &eng, &err);
     if (rc) return gfail(rc, err);
     rc = load_views(eng, g.tensors, &err);
     if (!rc) {
@@ -478,7 +495,8 @@ int hm_checkpoint_info(const char* path, char* buf, size_t cap, size_t* needed) 
     if (!path) return gfail(HM_ERR_INVALID, "hm_checkpoint_info: null path");
     const std::string p(path);
     std::string err, fmt;
-    hm_config cfg;
+    ModelSpec spec;
+    hm_config& cfg = spec.cfg;
     std::vector<TensorView> views;
     MappedFile mf;
     std::vector<std::unique_ptr<MappedFile>> shards;  // the views point into these
@@ -492,7 +510,7 @@ int hm_checkpoint_info(const char* path, char* buf, size_t cap, size_t* needed) 
         views = g.tensors;
     } else {
         fmt = "safetensors";
-        if (!parse_config_json(p + "/config.json", &cfg, &err)) return gfail(HM_ERR_IO, err);
+        if (!parse_model_spec_file(p + "/config.json", &spec, &err)) return gfail(HM_ERR_IO, err);
         std::vector<std::string> files;
         const int frc = safetensors_files(p, &files, &err);
         if (frc) return gfail(frc, err);
@@ -515,6 +533,11 @@ int hm_checkpoint_info(const char* path, char* buf, size_t cap, size_t* needed) 
                   cfg.max_position_embeddings, cfg.head_dim, cfg.tie_word_embeddings ? "true" : "false", cfg.rms_norm_eps, cfg.rope_theta,
                   cfg.eos_token_id == UINT32_MAX ? -1ll : (long long)cfg.eos_token_id, cfg.bos_token_id == UINT32_MAX ? -1ll : (long long)cfg.bos_token_id);
     o += tmp;
+    if (spec.listed()) {
+        std::snprintf(tmp, sizeof(tmp), ",\"architecture\":\"%s\",\"norm_groups\":%d,\"layers\":", spec.arch.c_str(), spec.norm_groups);
+        o += tmp;
+        o += layers_json(spec);
+    }
     o += "},\"tensors\":[";
     bool first = true;
     for (const TensorView& t : views) {
@@ -540,6 +563,19 @@ int hm_checkpoint_info(const char* path, char* buf, size_t cap, size_t* needed) 
 }
 
 int hm_kv_alloc(hm_engine* e, int batch, int max_seq_len, int page_tokens, int kv_dtype) { return e ? e->impl->kv_alloc(batch, max_seq_len, page_tokens, kv_dtype) : gfail(HM_ERR_INVALID, "null engine"); }
+int hm_kv_alloc_pool(hm_engine* e, int batch, int max_seq_len, long pool_tokens, int page_tokens, int kv_dtype) {
+    if (!e) return gfail(HM_ERR_INVALID, "null engine");
+    if (pool_tokens < 1) {
+        e->impl->err = "hm_kv_alloc_pool: the pool must hold at least one token";
+        return HM_ERR_INVALID;
+    }
+    return e->impl->kv_alloc(batch, max_seq_len, page_tokens, kv_dtype, pool_tokens);
+}
+int hm_kv_free_tokens(hm_engine* e, long* out) { return e ? e->impl->kv_free_tokens(out) : gfail(HM_ERR_INVALID, "null engine"); }
+int hm_latent_view(hm_engine* e, int seq, int layer, float* out) { return e ? e->impl->latent_view(seq, layer, out) : gfail(HM_ERR_INVALID, "null engine"); }
+int hm_step(hm_engine* e, const hm_step_entry* entries, int n_entries, float* logits_or_null, uint32_t* greedy_or_null, float* hidden_or_null) {
+    return e ? e->impl->step(entries, n_entries, logits_or_null, greedy_or_null, hidden_or_null) : gfail(HM_ERR_INVALID, "null engine");
+}
 int hm_kv_free(hm_engine* e) { return e ? e->impl->kv_free() : gfail(HM_ERR_INVALID, "null engine"); }
 int hm_kv_reset(hm_engine* e, int seq) { return e ? e->impl->kv_reset(seq) : gfail(HM_ERR_INVALID, "null engine"); }
 int hm_kv_len(hm_engine* e, int seq, int* out) { return e ? e->impl->kv_len(seq, out) : gfail(HM_ERR_INVALID, "null engine"); }

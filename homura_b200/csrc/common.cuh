@@ -226,8 +226,25 @@ __device__ __forceinline__ float warp_max(float v) {
 }
 
 // ---- GEMV argument block ---------------------------------------------------------------
-enum Prologue { PRO_PLAIN = 0, PRO_RMSNORM = 1 };
-enum Epilogue { EPI_STORE = 0, EPI_QKV_ROPE = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3 };
+// PRO_GNORM: RMSNorm in equal groups, optionally followed by the token shift (see RowNorm)
+enum Prologue { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_GNORM = 2 };
+// EPI_GATE: y = acc * sigmoid(gate); EPI_SQRELU: y = max(acc, 0)^2
+enum Epilogue { EPI_STORE = 0, EPI_QKV_ROPE = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3, EPI_GATE = 4, EPI_SQRELU = 5 };
+
+// Normalisation of a projection's input rows in `groups` equal runs, each divided by its own root mean square, and the
+// token shift h + (h' - h) * shift, where h' is the normalised row of the sequence's previous token before its own shift
+// (zeros for position 0).  h' comes from the row in front when that row is the previous token of the same sequence, else
+// from `state`: [sequence][SHIFT_RING][K] f32, the row of position p in slot p % SHIFT_RING.  Only a run's last row has to
+// be kept; the ring is longer than the rows of one streaming launch, so that a launch whose CTAs read the row in front of
+// its first token never writes that slot.
+constexpr int SHIFT_RING = 16;
+struct RowNorm {
+    int groups;              // >= 1
+    const float* shift;      // [K] or null: no token shift
+    float* state;            // with shift
+    const int32_t* row_pos;  // with shift: position and sequence of every row
+    const int32_t* row_seq;
+};
 
 // Element offsets inside one [16 tokens][hd] page tile.  Chunk-major means: the chunk c of every token is stored
 // together, so that the 16 tokens' copies of one chunk are one contiguous run; either way the tile is one
@@ -376,12 +393,19 @@ struct GemvArgs {
     int pro;
     const float* norm_w;
     float eps;
+    RowNorm gn;          // PRO_GNORM
+    // Grouped projection (block-diagonal weights, e.g. one matrix per attention head): group g owns group_slabs slabs,
+    // reads its own K inputs at x + g * group_x and writes outputs [g * group_n, (g + 1) * group_n).  0: one group.
+    int group_slabs, group_x, group_n;
     // epilogue
     int epi;
     float* y;
     int ldy;
     const float* bias;   // [N] or null
     const float* resid;  // [M][ldy] or null (EPI_STORE: y = resid + acc)
+    const float* out_scale;  // [N] or null (EPI_STORE: the result is multiplied element by element before the residual is added)
+    const float* gate;   // EPI_GATE: [M][ld_gate]
+    int ld_gate;
     // EPI_QKV_ROPE
     int q_dim, kv_dim, hd, has_qk_norm;
     const float* q_norm_w;
@@ -478,6 +502,8 @@ int attn_pick_cluster(int max_pages, int max_cluster);
 
 cudaError_t launch_pack_slabs_from_nk(const uint16_t* src_nk, int N, int K, uint16_t* dst, int n_off, int interleave_which, cudaStream_t st);
 cudaError_t launch_pack_slabs_from_kn(const uint16_t* src_kn, int K, int N, uint16_t* dst, cudaStream_t st);
+// dst[i] = src[rows[i]] for n rows of W floats
+cudaError_t launch_gather_rows(const float* src, const int32_t* rows, int n, int W, float* dst, cudaStream_t st, bool pdl);
 cudaError_t launch_embed_gather(const void* table, int table_dtype, const uint32_t* tokens, int M, int H, int V, float* out, int* err_flag, cudaStream_t st, bool pdl);
 cudaError_t launch_argmax_finish(const float* amax_val, const int32_t* amax_idx, int nslabs, int M, uint32_t* next_tok, uint32_t* feed_tok, int32_t* pos, uint32_t* hist, int hist_stride, cudaStream_t st, bool pdl);
 cudaError_t launch_argmax_rows(const float* logits, int rows, int n, uint32_t* out, cudaStream_t st);

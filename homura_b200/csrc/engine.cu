@@ -1,5 +1,6 @@
 // Engine implementation.  See engine.h.
 #include "engine.h"
+#include "engine_util.h"
 #include "gemm_tc.h"
 #include "kquant.h"
 #include "sampler.h"
@@ -14,14 +15,8 @@
 
 namespace hm {
 
-#define HM_CUDA(call)                                      \
-    do {                                                   \
-        cudaError_t _e = (call);                           \
-        if (_e != cudaSuccess) return cuda_fail(_e, #call); \
-    } while (0)
-
 size_t LinearW::bytes() const {
-    if (kind == HM_BF16) return (size_t)((N + SLAB - 1) / SLAB) * K * SLAB * 2;
+    if (kind == HM_BF16) return (size_t)((columns() + SLAB - 1) / SLAB) * K * SLAB * 2;
     if (kind == HM_Q8_0) return (size_t)N * (K / 32) * 34;
     if (kind == HM_Q4_0) return (size_t)N * (K / 32) * 18;
     if (kind == HM_Q4_K) return kq_bytes;
@@ -38,7 +33,8 @@ int Engine::cuda_fail(cudaError_t e, const char* what) {
 }
 bool Engine::set_device() { return cudaSetDevice(device_) == cudaSuccess; }
 
-int Engine::create(const hm_config& cfg, int device, Engine** out, std::string* err) {
+int Engine::create(const ModelSpec& spec, int device, bool strict_f32, Engine** out, std::string* err) {
+    const hm_config& cfg = spec.cfg;
     int ndev = 0;
     if (cudaGetDeviceCount(&ndev) != cudaSuccess || ndev == 0) {
         *err = "no CUDA device available (this engine has no CPU fallback)";
@@ -53,6 +49,7 @@ int Engine::create(const hm_config& cfg, int device, Engine** out, std::string* 
         return HM_ERR_INVALID;
     }
     Engine* e = new Engine();
+    e->spec_ = spec;
     e->cfg_ = cfg;
     e->device_ = device;
     e->H_ = cfg.hidden_size;
@@ -74,9 +71,18 @@ int Engine::create(const hm_config& cfg, int device, Engine** out, std::string* 
         delete e;
         return HM_ERR_UNSUPPORTED;
     };
-    if (e->hd_ != 64 && e->hd_ != 128) return bad("head_dim must be 64 or 128");
-    if (e->heads_ % e->kvh_ != 0 || e->heads_ / e->kvh_ > 8) return bad("heads / kv_heads must be an integer <= 8");
-    if (e->H_ % 32 != 0 || e->I_ % 64 != 0) return bad("hidden_size must be a multiple of 32 and intermediate_size of 64");
+    if (spec.listed()) {
+        e->kvdim_ = 0;
+        e->qdim_ = 0;
+        for (const LayerSpec& l : spec.layers) {
+            e->qdim_ = std::max(e->qdim_, l.heads * l.vdim);
+            if (l.kv_rank > 1024) return bad("kv_rank must be at most 1024");
+        }
+    } else {
+        if (e->hd_ != 64 && e->hd_ != 128) return bad("head_dim must be 64 or 128");
+        if (e->heads_ % e->kvh_ != 0 || e->heads_ / e->kvh_ > 8) return bad("heads / kv_heads must be an integer <= 8");
+        if (e->H_ % 32 != 0 || e->I_ % 64 != 0) return bad("hidden_size must be a multiple of 32 and intermediate_size of 64");
+    }
     if (cudaSetDevice(device) != cudaSuccess) return bad("cudaSetDevice failed");
     cudaDeviceProp prop;
     if (cudaGetDeviceProperties(&prop, device) == cudaSuccess) e->sm_count_ = prop.multiProcessorCount;
@@ -88,7 +94,7 @@ int Engine::create(const hm_config& cfg, int device, Engine** out, std::string* 
     e->use_clusters_ = !(nocl && nocl[0] == '1');
     e->max_cluster_ = gemv_max_cluster();
     const char* notc = std::getenv("HM_NO_TC");
-    e->use_tc_ = !(notc && notc[0] == '1');
+    e->use_tc_ = !(notc && notc[0] == '1') && !(spec.listed() && strict_f32);
     *out = e;
     return HM_OK;
 }
@@ -103,11 +109,13 @@ Engine::~Engine() {
         if (p) cudaFree(p);
     };
     fr(embed_); fr(final_norm_); fr(rope_cos_); fr(rope_sin_);
-    for (auto& l : layers_) {
-        fr(l.in_ln); fr(l.post_ln); fr(l.qkv_bias); fr(l.q_norm); fr(l.k_norm);
-        for (LinearW* w : {&l.qkv, &l.o, &l.gu, &l.down}) { fr(w->slabs); fr(w->tc); fr(w->scales); fr(w->codes); fr(w->kq_data); fr(w->kq_tile_type); }
-    }
-    fr(lm_head_.slabs); fr(lm_head_.tc); fr(lm_head_.scales); fr(lm_head_.codes); fr(lm_head_.kq_data); fr(lm_head_.kq_tile_type);
+    for (auto& l : layers_)
+        for (float* p : {l.in_ln, l.post_ln, l.qkv_bias, l.q_norm, l.k_norm, l.shift, l.ls1, l.ls2, l.latent_norm}) fr(p);
+    each_linear([&](LinearW& w) { fr(w.slabs); fr(w.tc); fr(w.scales); fr(w.codes); fr(w.kq_data); fr(w.kq_tile_type); });
+    free_listed();
+    free_listed_cache();
+    fr(hsel_); fr(st_tokens_); fr(st_pos_); fr(st_seq_); fr(st_want_); fr(st_next_); fr(seq_iota_);
+    if (st_pin_) cudaFreeHost(st_pin_);
     fr(xpack_); fr(xpack_attn_); fr(xpack_act_); fr(xpack_h_); fr(xpack_h2_); fr(ss_h_); fr(ss_h2_); fr(h_); fr(q_); fr(attn_); fr(act_); fr(qkv_raw_); fr(gu_raw_); fr(logits_); fr(amax_val_); fr(amax_idx_);
     fr(partial_); fr(tickets_); fr(att_acc_); fr(att_ml_); fr(att_tickets_); fr(err_flag_); fr(fin_ticket_);
     for (void* p : k_pool_) fr(p);
@@ -268,6 +276,7 @@ int Engine::load_tensor(const char* cname, int dtype, const int64_t* shape, int 
     auto shape1 = [&](int64_t a) { return ndim == 1 && shape[0] == a; };
     auto bad_shape = [&]() { return fail(HM_ERR_INVALID, "unexpected shape for tensor " + name); };
 
+    if (spec_.listed()) return load_listed_tensor(name, dtype, shape, ndim, host, nbytes);
     if (name == "model.embed_tokens.weight" || name == "token_embd.weight") {
         if (!shape2(V_, H_)) return bad_shape();
         if (embed_) return fail(HM_ERR_STATE, "embedding loaded twice");
@@ -368,7 +377,11 @@ int Engine::finalize() {
     if (!embed_) return fail(HM_ERR_STATE, "missing weight: model.embed_tokens.weight");
     if (!final_norm_) return fail(HM_ERR_STATE, "missing weight: model.norm.weight");
     if (lm_head_.kind < 0) return fail(HM_ERR_STATE, "missing weight: lm_head.weight");
-    for (int i = 0; i < L_; ++i) {
+    if (spec_.listed()) {
+        const int rc = finalize_listed();
+        if (rc) return rc;
+    }
+    for (int i = 0; i < L_ && !spec_.listed(); ++i) {
         const LayerW& l = layers_[i];
         const std::string p = "missing weight in layer " + std::to_string(i) + ": ";
         if (!l.in_ln) return fail(HM_ERR_STATE, p + "input_layernorm");
@@ -379,12 +392,14 @@ int Engine::finalize() {
         if (l.down.loaded_parts != 1) return fail(HM_ERR_STATE, p + "down projection");
         if (cfg_.has_qk_norm && (!l.q_norm || !l.k_norm)) return fail(HM_ERR_STATE, p + "q_norm/k_norm");
     }
-    std::vector<float> c, s;
-    build_rope_table(hd_, cfg_.max_position_embeddings, cfg_.rope_theta, &c, &s);
-    HM_CUDA(cudaMalloc(&rope_cos_, c.size() * 4));
-    HM_CUDA(cudaMalloc(&rope_sin_, s.size() * 4));
-    HM_CUDA(cudaMemcpy(rope_cos_, c.data(), c.size() * 4, cudaMemcpyHostToDevice));
-    HM_CUDA(cudaMemcpy(rope_sin_, s.data(), s.size() * 4, cudaMemcpyHostToDevice));
+    if (!spec_.listed()) {
+        std::vector<float> c, s;
+        build_rope_table(hd_, cfg_.max_position_embeddings, cfg_.rope_theta, &c, &s);
+        HM_CUDA(cudaMalloc(&rope_cos_, c.size() * 4));
+        HM_CUDA(cudaMalloc(&rope_sin_, s.size() * 4));
+        HM_CUDA(cudaMemcpy(rope_cos_, c.data(), c.size() * 4, cudaMemcpyHostToDevice));
+        HM_CUDA(cudaMemcpy(rope_sin_, s.data(), s.size() * 4, cudaMemcpyHostToDevice));
+    }
     HM_CUDA(cudaMalloc(&err_flag_, 4));
     HM_CUDA(cudaMemset(err_flag_, 0, 4));
     HM_CUDA(cudaMalloc(&fin_ticket_, 4));
@@ -394,8 +409,8 @@ int Engine::finalize() {
 }
 
 uint64_t Engine::weight_bytes() const {
-    uint64_t b = lm_head_.bytes();
-    for (auto& l : layers_) b += l.qkv.bytes() + l.o.bytes() + l.gu.bytes() + l.down.bytes();
+    uint64_t b = 0;
+    const_cast<Engine*>(this)->each_linear([&](LinearW& w) { b += w.bytes(); });
     return b;
 }
 
@@ -403,7 +418,7 @@ uint64_t Engine::weight_bytes() const {
 
 int Engine::ensure_scratch(int rows) {
     const bool tall = use_tc_ && !quant_;  // prefill chunks of TC_ROWS rows on the tensor-core GEMM
-    if (tall || quant_) rows = std::max(rows, TC_ROWS);
+    if (tall || quant_ || spec_.listed()) rows = std::max(rows, TC_ROWS);
     const int cap = (rows + MAX_M - 1) / MAX_M * MAX_M;
     if (cap <= scratch_rows_) return HM_OK;
     auto re = [&](auto** p, size_t count) -> cudaError_t {
@@ -415,6 +430,7 @@ int Engine::ensure_scratch(int rows) {
     };
     const int nslabs_v = (V_ + SLAB - 1) / SLAB;
     HM_CUDA(re(&h_, (size_t)cap * H_));
+    HM_CUDA(re(&hsel_, (size_t)std::max(cap, TC_ROWS) * H_));
     HM_CUDA(re(&q_, (size_t)cap * qdim_));
     HM_CUDA(re(&attn_, (size_t)cap * qdim_));
     HM_CUDA(re(&act_, (size_t)cap * I_));
@@ -436,7 +452,10 @@ int Engine::ensure_scratch(int rows) {
         HM_CUDA(re(&qrows_img_, quant_rows_image_words(qrows_k_)));
         HM_CUDA(re(&qrows_bs_, quant_rows_scale_floats(qrows_k_)));
     }
-    if (quant_ || tall) {
+    if (spec_.listed()) {
+        const int rc = alloc_listed_scratch(cap);
+        if (rc) return rc;
+    } else if (quant_ || tall) {
         HM_CUDA(re(&qkv_raw_, (size_t)cap * (qdim_ + 2 * kvdim_)));
         HM_CUDA(re(&gu_raw_, (size_t)cap * 2 * I_));
         if (tall) {
@@ -457,13 +476,12 @@ int Engine::ensure_scratch(int rows) {
         if (w.kind != HM_BF16) return;
         for (int M : {1, 2, 4, 8}) {
             int ks, rps;
-            gemv_pick_split(w.K, w.N, M, sm_count_, &ks, &rps);
-            pf = std::max(pf, gemv_partial_floats(w.N, ks, M));
+            gemv_pick_split(w.K, w.columns(), M, sm_count_, &ks, &rps);
+            pf = std::max(pf, gemv_partial_floats(w.columns(), ks, M));
         }
-        max_slabs = std::max(max_slabs, (w.N + SLAB - 1) / SLAB);
+        max_slabs = std::max(max_slabs, (w.columns() + SLAB - 1) / SLAB);
     };
-    for (auto& l : layers_) { acc(l.qkv); acc(l.o); acc(l.gu); acc(l.down); }
-    acc(lm_head_);
+    each_linear(acc);
     partial_floats_ = std::max<size_t>(pf, 1);
     HM_CUDA(re(&partial_, partial_floats_));
     HM_CUDA(re(&tickets_, (size_t)max_slabs));
@@ -473,30 +491,38 @@ int Engine::ensure_scratch(int rows) {
 
 // ---- KV cache --------------------------------------------------------------------------------
 
-int Engine::kv_alloc(int batch, int max_seq_len, int page_tokens, int kv_dtype) {
+int Engine::kv_alloc(int batch, int max_seq_len, int page_tokens, int kv_dtype, long pool_tokens) {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (!finalized_) return fail(HM_ERR_STATE, "kv_alloc before weights are finalised");
     if (batch_ > 0) return fail(HM_ERR_STATE, "KV cache already allocated");
     if (batch < 1 || max_seq_len < 1) return fail(HM_ERR_INVALID, "kv_alloc: batch and max_seq_len must be positive");
-    if (page_tokens != 16) return fail(HM_ERR_UNSUPPORTED, "kv_alloc: page size must be 16 tokens");
+    const int native = spec_.listed() ? LATENT_PAGE : 16;
+    if (page_tokens == 0) page_tokens = native;
+    if (page_tokens != native) return fail(HM_ERR_UNSUPPORTED, "kv_alloc: page size must be " + std::to_string(native) + " tokens");
+    if (pool_tokens < 0) return fail(HM_ERR_INVALID, "kv_alloc: negative pool size");
     if (kv_dtype != HM_F32 && kv_dtype != HM_BF16) return fail(HM_ERR_UNSUPPORTED, "kv_alloc: cache dtype must be f32 or bf16");
     if (max_seq_len > cfg_.max_position_embeddings) return fail(HM_ERR_INVALID, "kv_alloc: max_seq_len exceeds max_position_embeddings (RoPE table)");
     kv_bf16_ = kv_dtype == HM_BF16;
     page_tokens_ = page_tokens;
     max_pages_ = (max_seq_len + page_tokens - 1) / page_tokens;
-    const size_t n_pages = (size_t)batch * max_pages_;
+    const size_t table_len = (size_t)batch * max_pages_;
+    const size_t n_pages = pool_tokens > 0 ? (size_t)(pool_tokens + page_tokens - 1) / page_tokens : table_len;
     const size_t page_elems = (size_t)kvh_ * page_tokens * hd_;
     const size_t pool_bytes = n_pages * page_elems * (kv_bf16_ ? 2 : 4);
     k_pool_.assign(L_, nullptr);
     v_pool_.assign(L_, nullptr);
-    for (int l = 0; l < L_; ++l) {
+    if (spec_.listed()) {
+        const int rc = alloc_listed_cache(batch, n_pages);
+        if (rc) return rc;
+    }
+    for (int l = 0; l < L_ && !spec_.listed(); ++l) {
         HM_CUDA(cudaMalloc(&k_pool_[l], pool_bytes));
         HM_CUDA(cudaMalloc(&v_pool_[l], pool_bytes));
         HM_CUDA(cudaMemset(k_pool_[l], 0, pool_bytes));
         HM_CUDA(cudaMemset(v_pool_[l], 0, pool_bytes));
     }
-    // Every sequence owns max_pages pages; the mapping is a fixed pseudo-random permutation of
-    // the pool so that consecutive logical pages are not physically adjacent.
+    // Without a shared pool every sequence owns max_pages pages; the mapping is a fixed pseudo-random permutation of
+    // the pool so that consecutive logical pages are not physically adjacent.  With one the permutation is the free list.
     std::vector<int32_t> perm(n_pages);
     for (size_t i = 0; i < n_pages; ++i) perm[i] = (int32_t)i;
     uint64_t st = 0x9E3779B97F4A7C15ull;
@@ -504,8 +530,20 @@ int Engine::kv_alloc(int batch, int max_seq_len, int page_tokens, int kv_dtype) 
         st ^= st << 13; st ^= st >> 7; st ^= st << 17;
         std::swap(perm[i - 1], perm[st % i]);
     }
-    HM_CUDA(cudaMalloc(&page_table_, n_pages * 4));
-    HM_CUDA(cudaMemcpy(page_table_, perm.data(), n_pages * 4, cudaMemcpyHostToDevice));
+    HM_CUDA(cudaMalloc(&page_table_, table_len * 4));
+    pooled_ = pool_tokens > 0;
+    free_pages_.clear();
+    seq_pages_.assign(batch, {});
+    if (pooled_) {
+        free_pages_ = perm;
+        HM_CUDA(cudaMemset(page_table_, 0, table_len * 4));
+    } else {
+        HM_CUDA(cudaMemcpy(page_table_, perm.data(), table_len * 4, cudaMemcpyHostToDevice));
+    }
+    std::vector<int32_t> iota(std::max(batch, TC_ROWS));
+    for (size_t i = 0; i < iota.size(); ++i) iota[i] = (int32_t)i;
+    HM_CUDA(cudaMalloc(&seq_iota_, iota.size() * 4));
+    HM_CUDA(cudaMemcpy(seq_iota_, iota.data(), iota.size() * 4, cudaMemcpyHostToDevice));
     HM_CUDA(cudaMalloc(&pos_dev_, batch * 4));
     HM_CUDA(cudaMemset(pos_dev_, 0, batch * 4));
     HM_CUDA(cudaMalloc(&tokens_dev_, batch * 4));
@@ -543,10 +581,12 @@ int Engine::kv_alloc(int batch, int max_seq_len, int page_tokens, int kv_dtype) 
     // of attn_pick_nsplit answers with few splits of many pages each, i.e. the bulk-copy ring kernel
     att_cluster_ = use_clusters_ && max_pages_ <= 64 && (long)batch * kvh_ < sm_count_ / 2;
     att_nsplit_ = att_cluster_ ? attn_pick_cluster(max_pages_, std::min(max_cluster_, 16)) : attn_pick_nsplit(batch, kvh_, max_pages_, sm_count_, kv_bf16_);
-    HM_CUDA(cudaMalloc(&att_acc_, (size_t)scratch_rows_ * heads_ * att_nsplit_ * hd_ * 4));
-    HM_CUDA(cudaMalloc(&att_ml_, (size_t)scratch_rows_ * heads_ * att_nsplit_ * 2 * 4));
-    HM_CUDA(cudaMalloc(&att_tickets_, (size_t)scratch_rows_ * kvh_ * 4));
-    HM_CUDA(cudaMemset(att_tickets_, 0, (size_t)scratch_rows_ * kvh_ * 4));
+    if (!spec_.listed()) {
+        HM_CUDA(cudaMalloc(&att_acc_, (size_t)scratch_rows_ * heads_ * att_nsplit_ * hd_ * 4));
+        HM_CUDA(cudaMalloc(&att_ml_, (size_t)scratch_rows_ * heads_ * att_nsplit_ * 2 * 4));
+        HM_CUDA(cudaMalloc(&att_tickets_, (size_t)scratch_rows_ * kvh_ * 4));
+        HM_CUDA(cudaMemset(att_tickets_, 0, (size_t)scratch_rows_ * kvh_ * 4));
+    }
 #ifdef HM_PHASE_TRACE
     if (const char* gt = std::getenv("HM_GEMV_TRACE")) {
         if (gt[0] == '1' && !gemv_trace_) {
@@ -577,6 +617,11 @@ int Engine::kv_free() {
     for (void*& p : v_pool_) fr(p);
     k_pool_.clear();
     v_pool_.clear();
+    free_listed_cache();
+    free_pages_.clear();
+    seq_pages_.clear();
+    pooled_ = false;
+    fr(seq_iota_);
     fr(page_table_); fr(pos_dev_); fr(tokens_dev_); fr(next_dev_); fr(hist_dev_); fr(pf_tokens_); fr(pf_pos_); fr(pf_seq_);
     fr(att_acc_); fr(att_ml_); fr(att_tickets_);
     fr(smp_scaled_); fr(smp_count_); fr(smp_rng_); fr(smp_gen_start_); fr(smp_overflow_);
@@ -603,9 +648,11 @@ int Engine::kv_reset(int seq) {
     HM_CUDA(cudaStreamSynchronize(stream_));
     if (seq < 0) {
         std::fill(len_.begin(), len_.end(), 0);
+        for (int b = 0; b < batch_; ++b) release_pages(b);
         HM_CUDA(cudaMemset(pos_dev_, 0, batch_ * 4));
     } else {
         len_[seq] = 0;
+        release_pages(seq);
         HM_CUDA(cudaMemset(pos_dev_ + seq, 0, 4));
     }
     return HM_OK;
@@ -628,6 +675,11 @@ int Engine::kv_append(int seq, int layer, const float* k_rows, const float* v_ro
     if (seq < 0 || seq >= batch_ || layer < 0 || layer >= L_ || n_new < 0) return fail(HM_ERR_INVALID, "kv_append: index out of range");
     if (len_[seq] + n_new > max_seq_)
         return fail(HM_ERR_KV_FULL, "KV cache full (" + std::to_string(len_[seq]) + " + " + std::to_string(n_new) + " > " + std::to_string(max_seq_) + ")");
+    if (spec_.listed() && n_new > 0) return fail(HM_ERR_UNSUPPORTED, "kv_append: this design caches latents, not keys and values");
+    {
+        const int prc = ensure_pages({{seq, (long)len_[seq] + n_new}});
+        if (prc) return prc;
+    }
     if (n_new > 0 && (k_rows || v_rows)) {
         const size_t bytes = (size_t)kvh_ * n_new * hd_ * 4;
         float *dk = nullptr, *dv = nullptr;
@@ -657,6 +709,7 @@ int Engine::kv_view(int seq, int layer, float* k_out, float* v_out) {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (batch_ == 0) return fail(HM_ERR_STATE, "kv_view before kv_alloc");
     if (seq < 0 || seq >= batch_ || layer < 0 || layer >= L_ || !k_out || !v_out) return fail(HM_ERR_INVALID, "kv_view: bad arguments");
+    if (spec_.listed()) return fail(HM_ERR_UNSUPPORTED, "kv_view: this design caches latents, not keys and values (hm_latent_view)");
     const int len = len_[seq];
     if (len == 0) return HM_OK;
     const size_t bytes = (size_t)kvh_ * len * hd_ * 4;
@@ -676,8 +729,8 @@ int Engine::kv_view(int seq, int layer, float* k_out, float* v_out) {
 
 // ---- the pass ----------------------------------------------------------------------------------
 
-enum ProfClass { PC_EMBED = 0, PC_QKV, PC_ATTN, PC_O, PC_GATE_UP, PC_DOWN, PC_LM_HEAD, PC_SAMPLE, PC_COUNT };
 static const char* kProfNames[PC_COUNT] = {"embed", "qkv_rope_kvwrite", "attention", "o_proj_residual", "gate_up_swiglu", "down_residual", "lm_head", "argmax"};
+static const char* kProfNamesListed[PC_COUNT_LISTED] = {"embed", "in_proj", "attention", "o_proj_residual", "up_sqrelu", "down_residual", "lm_head", "argmax", "latent_write", "key_up", "value_up_gate"};
 
 void Engine::prof_mark(int) {}
 
@@ -769,7 +822,7 @@ RopeEpi Engine::rope_epi(int layer, const int32_t* row_pos, const int32_t* row_s
 }
 
 int Engine::enqueue_linear(const LinearW& L, int M, const float* x, int ldx, int pro, const float* norm_w, int epi, float* y, int ldy, const float* bias, const float* resid, int layer,
-                           const int32_t* row_pos, const int32_t* row_seq, float* amax_val, int32_t* amax_idx, int* launches, const ArgmaxFold* fold) {
+                           const int32_t* row_pos, const int32_t* row_seq, float* amax_val, int32_t* amax_idx, int* launches, const ArgmaxFold* fold, const LinOpt* opt) {
     // Q8_0 / Q4_0 projections over more than eight rows (prefill chunks, larger batches): the rows become digit planes once
     // and 64-row launches multiply them, instead of every CTA of an 8-row launch packing its own
     if ((L.kind == HM_Q8_0 || L.kind == HM_Q4_0) && M > MAX_M && qrows_img_ && L.K <= qrows_k_ && (epi == EPI_STORE || epi == EPI_SWIGLU || epi == EPI_QKV_ROPE)) {
@@ -875,12 +928,25 @@ int Engine::enqueue_linear(const LinearW& L, int M, const float* x, int ldx, int
             a.N = L.N;
             a.m_valid = mv;
             if (use_clusters_) {
-                gemv_pick_cluster(L.K, L.N, mp, sm_count_, max_cluster_, &a.ksplit, &a.rows_per_split);
+                gemv_pick_cluster(L.K, L.columns(), mp, sm_count_, max_cluster_, &a.ksplit, &a.rows_per_split);
                 a.cluster = a.ksplit > 1 && a.ksplit <= max_cluster_ ? a.ksplit : 0;
             }
             if (!use_clusters_ || (a.ksplit > 1 && a.cluster == 0)) {
                 a.cluster = 0;
-                gemv_pick_split(L.K, L.N, mp, sm_count_, &a.ksplit, &a.rows_per_split);
+                gemv_pick_split(L.K, L.columns(), mp, sm_count_, &a.ksplit, &a.rows_per_split);
+            }
+            if (opt) {
+                a.gn = opt->gn;
+                if (a.gn.row_pos) a.gn.row_pos += m0;
+                if (a.gn.row_seq) a.gn.row_seq += m0;
+                a.out_scale = opt->out_scale;
+                a.gate = opt->gate ? opt->gate + (size_t)m0 * opt->ld_gate : nullptr;
+                a.ld_gate = opt->ld_gate;
+            }
+            if (L.groups) {
+                a.group_slabs = L.group_slabs;
+                a.group_n = L.group_n;
+                a.group_x = opt ? opt->group_x : 0;
             }
             a.x = x + (size_t)m0 * ldx;
             a.ldx = ldx;
@@ -896,7 +962,7 @@ int Engine::enqueue_linear(const LinearW& L, int M, const float* x, int ldx, int
             a.kv_dim = kvdim_;
             a.hd = hd_;
             a.has_qk_norm = cfg_.has_qk_norm;
-            if (layer >= 0) {
+            if (layer >= 0 && !spec_.listed()) {
                 a.q_norm_w = layers_[layer].q_norm;
                 a.k_norm_w = layers_[layer].k_norm;
                 a.kv = KvDesc{k_pool_[layer], v_pool_[layer], page_table_, max_pages_, page_tokens_, kvh_, hd_, kv_bf16_ ? 1 : 0};
@@ -919,7 +985,7 @@ int Engine::enqueue_linear(const LinearW& L, int M, const float* x, int ldx, int
                 a.hist = fold->hist ? fold->hist + (size_t)m0 * fold->hist_stride : nullptr;
                 a.hist_stride = fold->hist_stride;
             }
-            if (a.cluster == 0 && gemv_partial_floats(L.N, a.ksplit, mp) > partial_floats_) return fail(HM_ERR_STATE, "split-K scratch too small");
+            if (a.cluster == 0 && gemv_partial_floats(L.columns(), a.ksplit, mp) > partial_floats_) return fail(HM_ERR_STATE, "split-K scratch too small");
             ce = launch_gemv_bf16(a, mp, stream_, pdl_);
         } else if (L.kind == HM_Q4_K) {
             KQuantArgs a{};
@@ -985,6 +1051,21 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
                          int32_t* pos_dev, uint32_t* hist_dev, int* launches) {
     (void)advance;
     cudaError_t ce = cudaSuccess;
+    if (spec_.listed()) {
+        if (!row_seq) row_seq = seq_iota_;
+        if (M > TC_ROWS) {  // a decode step over more sequences than one tensor-core launch takes: one pass after the other
+            if (lm_row0 != 0 || lm_rows != M || lm_pick_) return fail(HM_ERR_STATE, "a pass over more than 64 rows takes the logits of every row");
+            int rc = HM_OK;
+            for (int c0 = 0; c0 < M && rc == HM_OK; c0 += TC_ROWS) {
+                const int mc = std::min(TC_ROWS, M - c0);
+                lm_dst_row_ = c0;
+                rc = enqueue_pass(mc, tokens_dev + c0, row_pos + c0, row_seq + c0, 0, mc, advance, next_dev + c0, feed_dev ? feed_dev + c0 : nullptr, pos_dev ? pos_dev + c0 : nullptr,
+                                  hist_dev ? hist_dev + (size_t)c0 * (max_seq_ + 1) : nullptr, launches);
+            }
+            lm_dst_row_ = 0;
+            return rc;
+        }
+    }
     auto want = [&](int cls) { return only_class_ < 0 || only_class_ == cls; };
     if (want(PC_EMBED)) {
         ce = launch_embed_gather(embed_, embed_dtype_ == HM_BF16 ? 1 : 0, tokens_dev, M, H_, V_, h_, err_flag_, stream_, pdl_);
@@ -1014,6 +1095,13 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
     // producer's epilogue (weight multiply, sums of squares) and the consumer's (row factor)
     const bool fused = direct_pack && H_ % 128 == 0;
     for (int l = 0; l < L_; ++l) {
+        if (spec_.listed()) {
+            rc = enqueue_listed_layer(l, M, row_pos, row_seq, lm_rows, launches);
+            if (rc) return rc;
+            rc = tap(l, M);
+            if (rc) return rc;
+            continue;
+        }
         const LayerW& w = layers_[l];
         KvDesc kv{k_pool_[l], v_pool_[l], page_table_, max_pages_, page_tokens_, kvh_, hd_, kv_bf16_ ? 1 : 0};
         if (!want(PC_QKV)) {
@@ -1129,15 +1217,29 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
             rc = enqueue_linear(w.down, M, act_, I_, PRO_PLAIN, nullptr, EPI_STORE, h_, H_, nullptr, h_, l, row_pos, row_seq, nullptr, nullptr, launches);
             if (rc) return rc;
         }
+        rc = tap(l, M);
+        if (rc) return rc;
     }
     if (lm_rows > 0) {
         const int nslabs = (V_ + SLAB - 1) / SLAB;
         const float* x = h_ + (size_t)lm_row0 * H_;
+        if (lm_pick_) {  // rows of a mixed batch whose logits are wanted
+            ce = launch_gather_rows(h_, lm_pick_, lm_rows, H_, hsel_, stream_, pdl_);
+            if (ce != cudaSuccess) return cuda_fail(ce, "gather_rows");
+            ++*launches;
+            x = hsel_;
+        }
+        float* const lg = logits_ + lm_dst_row_ * V_;
         const bool lm_tall = use_tc_ && lm_head_.kind == HM_BF16 && lm_head_.tc && lm_rows > MAX_M;
         const bool slab_argmax = lm_head_.kind == HM_BF16;  // per-block argmax partials from the projection's epilogue
         const bool fold_argmax = slab_argmax && !lm_tall;    // the streaming kernel's last epilogue also produces the greedy token
         lm_folds_argmax_ = fold_argmax;
-        if (want(PC_LM_HEAD) && lm_tall && fused && lm_row0 == 0 && lm_rows == M) {
+        if (spec_.listed()) {
+            if (want(PC_LM_HEAD)) {
+                rc = enqueue_listed_logits(x, lm_rows, (lm_out_ && fold_argmax) ? lm_out_ : lg, ArgmaxFold{next_dev, feed_dev, pos_dev, hist_dev, max_seq_ + 1}, launches);
+                if (rc) return rc;
+            }
+        } else if (want(PC_LM_HEAD) && lm_tall && fused && lm_row0 == 0 && lm_rows == M && !lm_pick_) {
             TcFuse f;
             f.ss_in = ss_h_;
             f.ss_parts = H_ / 128;
@@ -1155,7 +1257,7 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
         }
         if (want(PC_SAMPLE) && !fold_argmax) {
             ce = slab_argmax ? launch_argmax_finish(amax_val_, amax_idx_, nslabs, lm_rows, next_dev, feed_dev, pos_dev, hist_dev, max_seq_ + 1, stream_, pdl_)
-                             : launch_argmax_finish(logits_, nullptr, V_, lm_rows, next_dev, feed_dev, pos_dev, hist_dev, max_seq_ + 1, stream_, pdl_);
+                             : launch_argmax_finish(lg, nullptr, V_, lm_rows, next_dev, feed_dev, pos_dev, hist_dev, max_seq_ + 1, stream_, pdl_);
             if (ce != cudaSuccess) return cuda_fail(ce, "argmax_finish");
             ++*launches;
         }
@@ -1165,6 +1267,7 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
 
 int Engine::capture_decode_graph() {
     int launches = 0;
+    pass_longest_ = max_seq_;
     HM_CUDA(cudaStreamBeginCapture(stream_, cudaStreamCaptureModeThreadLocal));
     int rc = enqueue_pass(batch_, tokens_dev_, pos_dev_, nullptr, 0, batch_, true, next_dev_, tokens_dev_, pos_dev_, hist_dev_, &launches);
     cudaGraph_t g = nullptr;
@@ -1206,7 +1309,7 @@ int Engine::selftest_expire_wait() {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (batch_ == 0) return fail(HM_ERR_STATE, "selftest_expire_wait before kv_alloc");
     // any 16 aligned device bytes serve as the source of the probe's real copy
-    HM_CUDA(launch_bounded_wait_probe(rope_cos_, err_flag_, 20000ull, nullptr, stream_));
+    HM_CUDA(launch_bounded_wait_probe(pf_pos_, err_flag_, 20000ull, nullptr, stream_));
     return HM_OK;
 }
 
@@ -1259,6 +1362,7 @@ int Engine::ensure_host_logits_graph() {
     if (lm_head_.kind != HM_BF16 || batch_ > MAX_M || !graph_exec_) return HM_OK;
     if (!alloc_pin_logits((size_t)batch_ * V_ * 4)) return HM_OK;
     host_graph_tried_ = true;  // alloc_pin_logits may have cleared it
+    pass_longest_ = max_seq_;
     HM_CUDA(cudaStreamSynchronize(stream_));
     int launches = 0;
     HM_CUDA(cudaStreamBeginCapture(stream_, cudaStreamCaptureModeThreadLocal));
@@ -1286,6 +1390,7 @@ int Engine::prefill(int seq, const int64_t* ids, int n, float* logits, uint32_t*
     if (len0 + n > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full (" + std::to_string(len0) + " + " + std::to_string(n) + " > " + std::to_string(max_seq_) + ")");
     for (int i = 0; i < n; ++i)
         if (ids[i] < 0 || ids[i] >= V_) return fail(HM_ERR_INVALID, "prefill: token id out of range");
+    if (const int prc = ensure_pages({{seq, (long)len0 + n}})) return prc;
     HM_CUDA(cudaStreamSynchronize(stream_));
     uint32_t* st = pin_u32_;
     for (int i = 0; i < n; ++i) {
@@ -1308,6 +1413,7 @@ int Engine::prefill(int seq, const int64_t* ids, int n, float* logits, uint32_t*
     for (int c0 = 0; c0 < n; c0 += chunk) {
         const int mc = std::min(chunk, n - c0);
         const bool last = c0 + mc >= n;
+        pass_longest_ = len0 + c0 + mc;
         int rc = enqueue_pass(mc, pf_tokens_ + c0, pf_pos_ + c0, pf_seq_ + c0, mc - 1, last ? 1 : 0, false, next_dev_ + seq, tokens_dev_ + seq, pos_dev_ + seq, hist_dev_ + (size_t)seq * (max_seq_ + 1),
                               &launches);
         if (rc) return rc;
@@ -1335,6 +1441,7 @@ int Engine::decode_step(const uint32_t* tokens, float* logits, uint32_t* next_to
         if (len_[b] + 1 > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full (" + std::to_string(len_[b]) + " + 1 > " + std::to_string(max_seq_) + ")");
         if (tokens[b] >= (uint32_t)V_) return fail(HM_ERR_INVALID, "decode_step: token id out of range");
     }
+    if (const int prc = ensure_pages_all(1)) return prc;
     std::memcpy(pin_u32_, tokens, (size_t)batch_ * 4);
     HM_CUDA(cudaMemcpyAsync(tokens_dev_, pin_u32_, (size_t)batch_ * 4, cudaMemcpyHostToDevice, stream_));
     float* land = nullptr;
@@ -1369,6 +1476,7 @@ int Engine::decode_greedy_n(const uint32_t* first_tokens, int steps, uint32_t* o
     if (steps < 0 || (steps > 0 && !out_ids)) return fail(HM_ERR_INVALID, "decode_greedy_n: bad arguments");
     for (int b = 0; b < batch_; ++b)
         if (len_[b] + steps > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full (" + std::to_string(len_[b]) + " + " + std::to_string(steps) + " > " + std::to_string(max_seq_) + ")");
+    if (const int prc = ensure_pages_all(steps)) return prc;
     if (first_tokens) {
         for (int b = 0; b < batch_; ++b)
             if (first_tokens[b] >= (uint32_t)V_) return fail(HM_ERR_INVALID, "decode_greedy_n: token id out of range");
@@ -1399,6 +1507,7 @@ int Engine::time_decode(int warmup, int steps, float* ms_total) {
     if (warmup < 0 || steps < 1 || !ms_total) return fail(HM_ERR_INVALID, "time_decode: bad arguments");
     for (int b = 0; b < batch_; ++b)
         if (len_[b] + warmup + steps > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full: not enough room for the timed steps");
+    if (const int prc = ensure_pages_all(warmup + steps)) return prc;
     cudaEvent_t e0, e1;
     HM_CUDA(cudaEventCreate(&e0));
     HM_CUDA(cudaEventCreate(&e1));
@@ -1505,19 +1614,22 @@ int Engine::time_decode(int warmup, int steps, float* ms_total) {
 int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (batch_ == 0) return fail(HM_ERR_STATE, "profile_decode before kv_alloc");
-    if (steps < 1 || !out || !n_out || cap < PC_COUNT) return fail(HM_ERR_INVALID, "profile_decode: bad arguments (cap >= 8)");
+    if (steps < 1 || !out || !n_out || cap < (spec_.listed() ? PC_COUNT_LISTED : PC_COUNT)) return fail(HM_ERR_INVALID, "profile_decode: bad arguments (cap >= 8; 11 for listed designs)");
     for (int b = 0; b < batch_; ++b)
         if (len_[b] + steps > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full: not enough room for the profiled steps");
+    if (const int prc = ensure_pages_all(steps)) return prc;
+    const int classes = spec_.listed() ? PC_COUNT_LISTED : PC_COUNT;
+    pass_longest_ = max_seq_;
     HM_CUDA(cudaStreamSynchronize(stream_));
     double kv_tokens = 0.0;
     for (int b = 0; b < batch_; ++b) kv_tokens += len_[b] + 1;
     cudaEvent_t e0, e1;
     HM_CUDA(cudaEventCreate(&e0));
     HM_CUDA(cudaEventCreate(&e1));
-    float ms[PC_COUNT] = {0};
-    int count[PC_COUNT] = {0};
+    float ms[PC_COUNT_LISTED] = {0};
+    int count[PC_COUNT_LISTED] = {0};
     int rc = HM_OK;
-    for (int c = 0; c < PC_COUNT && rc == HM_OK; ++c) {
+    for (int c = 0; c < classes && rc == HM_OK; ++c) {
         int launches = 0;
         only_class_ = c;
         cudaError_t ce = cudaStreamBeginCapture(stream_, cudaStreamCaptureModeThreadLocal);
@@ -1552,24 +1664,30 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
     cudaEventDestroy(e1);
     if (rc) return rc;
     for (int b = 0; b < batch_; ++b) len_[b] += steps;
-    uint64_t bytes[PC_COUNT] = {0};
+    uint64_t bytes[PC_COUNT_LISTED] = {0};
     bytes[PC_EMBED] = (uint64_t)batch_ * H_ * (embed_dtype_ == HM_BF16 ? 2 : 4);
     for (auto& l : layers_) {
-        bytes[PC_QKV] += l.qkv.bytes();
+        bytes[PC_QKV] += l.qkv.bytes() + l.in.bytes();
+        bytes[PC_KUP] += l.kup.bytes();
+        bytes[PC_VUP] += l.vup.bytes();
         bytes[PC_O] += l.o.bytes();
         bytes[PC_GATE_UP] += l.gu.bytes();
         bytes[PC_DOWN] += l.down.bytes();
     }
     bytes[PC_LM_HEAD] = lm_head_.bytes();
-    bytes[PC_ATTN] = (uint64_t)(kv_tokens * L_ * 2.0 * kvh_ * hd_ * (kv_bf16_ ? 2 : 4));
-    for (int c = 0; c < PC_COUNT; ++c) {
+    if (spec_.listed()) {
+        for (const LayerSpec& l : spec_.layers) bytes[PC_ATTN] += (uint64_t)(kv_tokens * l.kv_rank * (kv_bf16_ ? 2 : 4));
+    } else {
+        bytes[PC_ATTN] = (uint64_t)(kv_tokens * L_ * 2.0 * kvh_ * hd_ * (kv_bf16_ ? 2 : 4));
+    }
+    for (int c = 0; c < classes; ++c) {
         std::memset(&out[c], 0, sizeof(out[c]));
-        std::strncpy(out[c].name, kProfNames[c], sizeof(out[c].name) - 1);
+        std::strncpy(out[c].name, spec_.listed() ? kProfNamesListed[c] : kProfNames[c], sizeof(out[c].name) - 1);
         out[c].launches_per_step = count[c];
         out[c].ms_per_step = ms[c] / steps;
         out[c].bytes_per_step = bytes[c];
     }
-    *n_out = PC_COUNT;
+    *n_out = classes;
     return HM_OK;
 }
 
@@ -1620,6 +1738,7 @@ int Engine::decode_step_sampled(const uint32_t* tokens, const hm_sampling* sp, u
         if (len_[b] + 1 > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full (" + std::to_string(len_[b]) + " + 1 > " + std::to_string(max_seq_) + ")");
         if (tokens[b] >= (uint32_t)V_) return fail(HM_ERR_INVALID, "decode_step_sampled: token id out of range");
     }
+    if (const int prc = ensure_pages_all(1)) return prc;
     int rc = ensure_sampler_scratch();
     if (rc) return rc;
     // staging: [0, B) tokens in, [B, 2B) tokens out, [2B, 3B) overflow words, then B RNG words (8-byte aligned)
@@ -1691,13 +1810,17 @@ int Engine::generate(int seq, const int64_t* prompt, int n_prompt, int max_new, 
         std::vector<uint32_t> blk(32);
         while (!stop && (int)gen.size() < max_new && real_pos < max_seq_) {
             const int want = std::min({32, max_new - (int)gen.size(), max_seq_ - real_pos});
+            rc = save_state(seq);
+            if (rc) return rc;
             rc = decode_greedy_n(&cur, want, blk.data());
             if (rc) return rc;
             for (int i = 0; i < want; ++i) {
                 if (blk[i] == eos) {
-                    // tokens after EOS were speculative: roll the cache length back
-                    len_[seq] = real_pos + i + 1;
-                    HM_CUDA(cudaMemcpy(pos_dev_ + seq, &len_[seq], 4, cudaMemcpyHostToDevice));
+                    // tokens after EOS were speculative: roll the sequence back
+                    std::vector<uint32_t> fed(1, cur);
+                    fed.insert(fed.end(), blk.begin(), blk.begin() + i);
+                    rc = rewind(seq, real_pos, fed);
+                    if (rc) return rc;
                     stop = true;
                     break;
                 }
@@ -1732,6 +1855,11 @@ int Engine::generate(int seq, const int64_t* prompt, int n_prompt, int max_new, 
             std::vector<float> logits;
             while (!stop && (int)gen.size() < max_new && real_pos < max_seq_) {
                 const int want = exact ? std::min({32, max_new - (int)gen.size(), max_seq_ - real_pos}) : 1;
+                rc = ensure_pages({{seq, (long)real_pos + want}});
+                if (rc) return rc;
+                rc = save_state(seq);
+                if (rc) return rc;
+                const uint32_t cur = gen.back();
                 for (int i = 0; i < want; ++i) {
                     rc = launch_step();
                     if (rc) return rc;
@@ -1761,8 +1889,11 @@ int Engine::generate(int seq, const int64_t* prompt, int n_prompt, int max_new, 
                 }
                 for (int i = 0; i < want; ++i) {
                     if (blk[i] == eos) {
-                        len_[seq] = real_pos + i + 1;  // tokens after EOS were speculative: roll the cache length back
-                        HM_CUDA(cudaMemcpy(pos_dev_ + seq, &len_[seq], 4, cudaMemcpyHostToDevice));
+                        // tokens after EOS were speculative: roll the sequence back
+                        std::vector<uint32_t> fed(1, cur);
+                        fed.insert(fed.end(), blk.begin(), blk.begin() + i);
+                        rc = rewind(seq, real_pos, fed);
+                        if (rc) return rc;
                         stop = true;
                         break;
                     }

@@ -12,9 +12,13 @@
 
 #include "../../include/homura_b200.h"
 #include "common.cuh"
+#include "latent_attn.h"
+#include "model_spec.h"
 #include "sampler.h"
 
 namespace hm {
+
+struct TcArgs;
 
 struct LinearW {
     int K = 0, N = 0;        // N = output count of the (possibly fused) projection
@@ -29,6 +33,9 @@ struct LinearW {
     int kq_part_type = -1;            // type of the part loaded last (gate and up must agree: they share tiles)
     bool kq_has_q6 = false;           // some tile is Q6_K: passes over more than 8 rows keep the 8-row launches (the row-block kernel is Q4_K only)
     int loaded_parts = 0;
+    // grouped (block-diagonal) projection: K inputs and group_n outputs per group, every group in group_slabs 128-column slabs of its own
+    int groups = 0, group_n = 0, group_slabs = 0;
+    int columns() const { return groups ? groups * group_slabs * SLAB : N; }  // output columns counting the padding between groups
     bool rope_rows = false;  // quantised fused QKV: q and k rows stored in rotation-pair tiles (rope_tile_row), the projection's epilogue rotates
     size_t bytes() const;
 };
@@ -39,7 +46,22 @@ struct LayerW {
     float* qkv_bias = nullptr;  // fused [q_dim + 2 kv_dim]
     float* q_norm = nullptr;
     float* k_norm = nullptr;
-    LinearW qkv, o, gu, down;
+    LinearW qkv, o, gu, down;  // listed designs: gu is the up projection alone, qkv is empty
+    // listed designs (ModelSpec::layers)
+    float* shift = nullptr;              // token shift [H]
+    float *ls1 = nullptr, *ls2 = nullptr;  // layer scales [H]
+    float* latent_norm = nullptr;        // [kv_rank]
+    LinearW in;                          // queries, output gate and (unless another layer's latents are used) latents, parts padded to 128 columns
+    LinearW kup, vup;                    // per head: query -> latent space, latent space -> values
+};
+
+// What a projection launch needs beyond the common arguments (enqueue_linear)
+struct LinOpt {
+    RowNorm gn{};                        // with PRO_GNORM
+    const float* out_scale = nullptr;
+    const float* gate = nullptr;
+    int ld_gate = 0;
+    int group_x = 0;                     // grouped projections: inputs of one group to the next
 };
 
 // final argmax folded into the LM-head launch (see GemvArgs::fin_ticket)
@@ -52,13 +74,20 @@ struct ArgmaxFold {
 
 class Engine {
    public:
-    static int create(const hm_config& cfg, int device, Engine** out, std::string* err);
+    // strict_f32: projections on the f32 streaming kernels only (no tensor-core copies of the weights)
+    static int create(const ModelSpec& spec, int device, bool strict_f32, Engine** out, std::string* err);
     ~Engine();
 
     int load_tensor(const char* name, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
     int finalize();
 
-    int kv_alloc(int batch, int max_seq_len, int page_tokens, int kv_dtype);
+    // pool_tokens 0: every sequence owns pages for max_seq_len tokens; else the sequences share a pool of that many tokens and
+    // take pages from it as they grow
+    int kv_alloc(int batch, int max_seq_len, int page_tokens, int kv_dtype, long pool_tokens = 0);
+    int kv_free_tokens(long* out);
+    int latent_view(int seq, int layer, float* out);
+    // One batch over several sequences, each bringing any number of tokens
+    int step(const hm_step_entry* entries, int n, float* logits, uint32_t* greedy, float* hidden);
     int kv_free();
     int kv_reset(int seq);
     int kv_len(int seq, int* out);
@@ -75,6 +104,7 @@ class Engine {
     int selftest_expire_wait();
 
     const hm_config& config() const { return cfg_; }
+    const ModelSpec& spec() const { return spec_; }
     uint64_t weight_bytes() const;
     cudaStream_t stream() const { return stream_; }
     int launches_per_step() const { return launches_per_step_; }
@@ -93,7 +123,33 @@ class Engine {
     // Enqueue one pass over M rows (decode: one row per sequence; prefill: a chunk of one
     // sequence).  lm_row0/lm_rows select the rows that go through the LM head.
     int enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_pos, const int32_t* row_seq, int lm_row0, int lm_rows, bool advance, uint32_t* next_dev, uint32_t* feed_dev, int32_t* pos_dev, uint32_t* hist_dev, int* launches);
-    int enqueue_linear(const LinearW& L, int M, const float* x, int ldx, int pro, const float* norm_w, int epi, float* y, int ldy, const float* bias, const float* resid, int layer, const int32_t* row_pos, const int32_t* row_seq, float* amax_val, int32_t* amax_idx, int* launches, const struct ArgmaxFold* fold = nullptr);
+    int enqueue_linear(const LinearW& L, int M, const float* x, int ldx, int pro, const float* norm_w, int epi, float* y, int ldy, const float* bias, const float* resid, int layer, const int32_t* row_pos, const int32_t* row_seq, float* amax_val, int32_t* amax_idx, int* launches, const struct ArgmaxFold* fold = nullptr, const LinOpt* opt = nullptr);
+    // listed designs (engine_listed.cu)
+    int load_listed_tensor(const std::string& name, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
+    int load_grouped(LinearW& L, int groups, int K, int group_n, bool src_is_kn, int dtype, const void* host, size_t nbytes);
+    int finalize_listed();
+    int alloc_listed_scratch(int cap);
+    int alloc_listed_cache(int batch, size_t n_pages);
+    void free_listed_cache();
+    void free_listed();
+    int enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int next_lm_rows, int* launches);
+    int enqueue_listed_logits(const float* x, int rows, float* dst, const struct ArgmaxFold& fold, int* launches);
+    int enqueue_tc(const LinearW& L, int M, const unsigned char* xp, int epi, float* y, int ldy, TcArgs& a, int* launches);
+    LatentPool latent_pool(int layer) const;
+    // The per-sequence state that is not addressed by position (token shift): copies of one sequence's, for generation loops
+    // that run ahead of the host, and the way back from a run that went too far.
+    int save_state(int seq);
+    int rewind(int seq, int len, const std::vector<uint32_t>& fed);
+    // pages
+    int ensure_pages(const std::vector<std::pair<int, long>>& need);  // (sequence, tokens it will hold)
+    int ensure_pages_all(int more);
+    void release_pages(int seq);
+    template <typename F>
+    void each_linear(F f) {
+        for (auto& l : layers_)
+            for (LinearW* w : {&l.qkv, &l.o, &l.gu, &l.down, &l.in, &l.kup, &l.vup}) f(*w);
+        f(lm_head_);
+    }
     // RMSNorm handed from one tensor-core GEMM to the next without a packing launch (see TcArgs)
     struct TcFuse {
         const float* ss_in = nullptr;   // consumer: partial sums of squares of the rows of `prepacked`
@@ -113,6 +169,7 @@ class Engine {
     int check_device_error();  // after the synchronisation that follows queue_error_copy()
     void prof_mark(int cls);
 
+    ModelSpec spec_;
     hm_config cfg_{};
     int device_ = 0, sm_count_ = 148;
     int H_ = 0, I_ = 0, heads_ = 0, kvh_ = 0, hd_ = 0, qdim_ = 0, kvdim_ = 0, L_ = 0, V_ = 0;
@@ -157,6 +214,32 @@ class Engine {
     bool att_cluster_ = true;
     int* err_flag_ = nullptr;
     unsigned int* fin_ticket_ = nullptr;  // ticket of the LM head's folded argmax
+
+    // listed designs
+    float *mix_raw_ = nullptr, *qlat_ = nullptr, *ctx_ = nullptr;  // input projection, queries in latent space, attention result in latent space
+    unsigned char *xpack_q_ = nullptr, *xpack_ctx_ = nullptr;      // their tensor-core images, one per head
+    float *lat_acc_ = nullptr, *lat_ml_ = nullptr;                 // split attention
+    size_t lat_acc_floats_ = 0, lat_ml_floats_ = 0;
+    std::vector<void*> lat_pool_;  // per layer, null for layers that read another's
+    float *shift_state_ = nullptr, *shift_saved_ = nullptr;  // [layers][sequences][SHIFT_RING][H]; [layers][SHIFT_RING][H]
+    int32_t* seq_iota_ = nullptr;    // 0, 1, 2, ...: the sequence of every row of a decode step
+    int pass_longest_ = 0;           // longest context of the pass being enqueued (splits of the attention)
+    // portions (step)
+    float* hsel_ = nullptr;              // rows whose logits are wanted
+    const int32_t* lm_pick_ = nullptr;   // their indices within the pass being enqueued (null: lm_row0 ..)
+    size_t lm_dst_row_ = 0;              // first row of logits_ the pass writes
+    uint32_t *st_tokens_ = nullptr, *st_next_ = nullptr;
+    int32_t *st_pos_ = nullptr, *st_seq_ = nullptr, *st_want_ = nullptr;
+    uint32_t* st_pin_ = nullptr;
+    size_t st_rows_ = 0;
+    float* tap_ = nullptr;               // host: residual stream after every layer, [layers][tap_rows_][H]
+    size_t tap_rows_ = 0, tap_row0_ = 0;
+    int tap(int layer, int M);
+
+    // pages
+    bool pooled_ = false;
+    std::vector<int32_t> free_pages_;
+    std::vector<std::vector<int32_t>> seq_pages_;
 
     // KV cache
     int batch_ = 0, max_seq_ = 0, page_tokens_ = 16, max_pages_ = 0;

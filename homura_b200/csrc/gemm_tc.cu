@@ -78,7 +78,7 @@ struct TcShared {
 // out: [k-block][term][mpad][64] bf16, rows of 128 B, 16-byte chunks XOR-swizzled by (row & 7) where
 // row = term * mpad + m.  One block per padded row; an RMSNorm is folded in when norm_w is given
 // (x' = (x * inv_rms) * w, src/graph_builder/emit_linalg.rs:7-26).
-__global__ void __launch_bounds__(256) tc_pack_x_kernel(const float* __restrict__ x, int ldx, int M, int mpad, int K, int Kp, const float* __restrict__ norm_w, float eps, unsigned char* __restrict__ out, unsigned long long* trace) {
+__global__ void __launch_bounds__(256) tc_pack_x_kernel(const float* __restrict__ x, int ldx, int M, int mpad, int K, int Kp, const float* __restrict__ norm_w, float eps, unsigned char* __restrict__ out, unsigned long long* trace, int group_x, size_t group_bytes) {
     HM_TRACE(const bool tr = trace != nullptr && blockIdx.x == 0 && threadIdx.x == 0;)
     HM_TRACE(if (tr) trace[0] = global_timer();)
     pdl_launch_dependents();
@@ -86,7 +86,8 @@ __global__ void __launch_bounds__(256) tc_pack_x_kernel(const float* __restrict_
     HM_TRACE(if (tr) trace[2] = global_timer();)
     const int m = blockIdx.x, tid = threadIdx.x;
     const bool row_ok = m < M;
-    const float* xr = x + (size_t)m * ldx;
+    const float* xr = x + (size_t)m * ldx + (size_t)blockIdx.y * group_x;
+    out += (size_t)blockIdx.y * group_bytes;
     __shared__ float sw[8];
     __shared__ float s_inv;
     float inv = 1.0f;
@@ -136,16 +137,86 @@ __global__ void __launch_bounds__(256) tc_pack_x_kernel(const float* __restrict_
     HM_TRACE(if (trace && threadIdx.x == 0) atomicMax(trace + 12, global_timer());)
 }
 
+// ---- the same image of rows normalised in groups and token-shifted (RowNorm) ----
+// One block per padded row.  A row whose predecessor is the row in front normalises that row a second time instead of
+// waiting for its block.  The block of a run's FIRST row also keeps the run's last row in the state: it has read the
+// slot in front of the run by then, and it is the only block that touches this sequence's state.
+__device__ __forceinline__ void gnorm_row(const float* __restrict__ src, float* __restrict__ row, float* __restrict__ fac, int K, int groups, float eps, int tid) {
+    stage_row<256, false>(src, row, K, tid);
+    __syncthreads();
+    const int gs = K / groups, lane = tid & 31;
+    for (int g = tid >> 5; g < groups; g += 8) {
+        float s = 0.f;
+        for (int i = lane; i < gs; i += 32) s = fmaf(row[g * gs + i], row[g * gs + i], s);
+        s = warp_sum(s);
+        if (lane == 0) fac[g] = 1.0f / sqrtf(s / (float)gs + eps);
+    }
+    __syncthreads();
+}
+__global__ void __launch_bounds__(256) tc_pack_gnorm_kernel(const float* __restrict__ x, int ldx, int M, int mpad, int K, int Kp, const float* __restrict__ norm_w, float eps, const RowNorm gn, unsigned char* __restrict__ out) {
+    extern __shared__ __align__(16) float rows[];
+    float *cur = rows, *nb = rows + Kp, *fac = nb + (gn.shift ? Kp : 0), *nfac = fac + gn.groups;
+    __shared__ int s_last;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int m = blockIdx.x, tid = threadIdx.x;
+    const bool row_ok = m < M;
+    const int gs = K / gn.groups;
+    if (row_ok) {
+        gnorm_row(x + (size_t)m * ldx, cur, fac, K, gn.groups, eps, tid);
+        for (int k = tid; k < K; k += 256) cur[k] = (cur[k] * fac[k / gs]) * __ldg(norm_w + k);
+        if (gn.shift) {
+            const int pos = gn.row_pos[m], seq = gn.row_seq[m];
+            const bool follows = m > 0 && gn.row_seq[m - 1] == seq && gn.row_pos[m - 1] + 1 == pos;
+            float* st = gn.state + (size_t)seq * SHIFT_RING * K;
+            if (follows) {
+                gnorm_row(x + (size_t)(m - 1) * ldx, nb, nfac, K, gn.groups, eps, tid);
+                for (int k = tid; k < K; k += 256) {
+                    const float p = (nb[k] * nfac[k / gs]) * __ldg(norm_w + k), h = cur[k];
+                    cur[k] = fmaf(p - h, __ldg(gn.shift + k), h);
+                }
+            } else {
+                if (tid == 0) {
+                    int e = m;
+                    while (e + 1 < M && gn.row_seq[e + 1] == seq && gn.row_pos[e + 1] == gn.row_pos[e] + 1) ++e;
+                    s_last = e;
+                }
+                __syncthreads();
+                const int e = s_last;
+                if (e != m) gnorm_row(x + (size_t)e * ldx, nb, nfac, K, gn.groups, eps, tid);
+                float* keep = st + (size_t)((pos + e - m) % SHIFT_RING) * K;
+                const float* prev = st + (size_t)((pos + SHIFT_RING - 1) % SHIFT_RING) * K;
+                for (int k = tid; k < K; k += 256) {
+                    const float h = cur[k], p = pos > 0 ? prev[k] : 0.f;  // a plain load: it must stay in front of the store, which may be to the same slot
+                    keep[k] = e != m ? (nb[k] * nfac[k / gs]) * __ldg(norm_w + k) : h;
+                    cur[k] = fmaf(p - h, __ldg(gn.shift + k), h);
+                }
+            }
+        }
+        for (int k = K + tid; k < Kp; k += 256) cur[k] = 0.f;
+        __syncthreads();
+    }
+    for (int c = tid; c < Kp / 8; c += 256) {
+        float v[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = row_ok ? cur[c * 8 + e] : 0.f;
+        tc_xpack_store8(out, mpad, m, c * 8, v);
+    }
+}
+
 // ---- epilogues on rows [m_lo, m_hi) of the f32 tile [m][128] (output features n0 .. n0+127) ----
 // The same four epilogues as the streaming projection kernel (gemv_bf16.cu), for up to 64 rows.
 __device__ __forceinline__ bool tc_better(float v, int i, float bv, int bi) { return v > bv || (v == bv && i > bi); }
 
 __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, int nblk, int tid, const int* s_pos, const int* s_page) {
-    const int n0 = nblk * BM, rows = m_hi - m_lo;
+    // grouped projections: this block's output columns [n0, n_end)
+    const int grp = a.group_blocks ? nblk / a.group_blocks : 0;
+    const int n0 = a.group_blocks ? grp * a.group_n + (nblk - grp * a.group_blocks) * BM : nblk * BM, rows = m_hi - m_lo;
+    const int n_end = a.group_blocks ? (grp + 1) * a.group_n : a.N;
     const int lane = tid & 31, warp = tid >> 5;
     constexpr int NW = TC_THREADS / 32;
     if (a.epi == EPI_STORE) {
-        const bool vec = (a.ldy & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.resid) | reinterpret_cast<uintptr_t>(a.bias)) & 15) == 0 && n0 + BM <= a.N;
+        const bool vec = (a.ldy & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.resid) | reinterpret_cast<uintptr_t>(a.bias) | reinterpret_cast<uintptr_t>(a.out_scale)) & 15) == 0 && n0 + BM <= n_end && (n0 & 3) == 0;
         if (vec) {
             // eight consecutive features per thread (one 16-byte chunk of the next GEMM's activation image); the 16
             // threads of a row are half a warp, which is where the row's sum of squares is reduced
@@ -158,6 +229,14 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                 {
                     const float4 t0 = *reinterpret_cast<const float4*>(tile + m * BM + c), t1 = *reinterpret_cast<const float4*>(tile + m * BM + c + 4);
                     v[0] = t0.x; v[1] = t0.y; v[2] = t0.z; v[3] = t0.w; v[4] = t1.x; v[5] = t1.y; v[6] = t1.z; v[7] = t1.w;
+                }
+                if (a.out_scale) {
+                    const float4 s0 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c)), s1 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c + 4));
+                    v[0] *= s0.x; v[1] *= s0.y; v[2] *= s0.z; v[3] *= s0.w; v[4] *= s1.x; v[5] *= s1.y; v[6] *= s1.z; v[7] *= s1.w;
+                }
+                if (a.split_xp && n0 + c < a.split_n) {  // 8-element pieces never straddle split_n or an image: both are multiples of 8
+                    if (ok) tc_xpack_store8(a.split_xp + (size_t)((n0 + c) / a.split_k) * a.split_bytes, a.xp_mpad, m, (n0 + c) % a.split_k, v);
+                    continue;
                 }
                 if (ok && a.resid) {
                     const float4 r0 = ld_cg_f32x4(a.resid + (size_t)m * a.ldy + n0 + c), r1 = ld_cg_f32x4(a.resid + (size_t)m * a.ldy + n0 + c + 4);
@@ -190,9 +269,14 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
         } else {
             for (int idx = tid; idx < rows * BM; idx += TC_THREADS) {
                 const int m = m_lo + idx / BM, c = idx % BM, n = n0 + c;
-                if (n < a.N) {
+                if (n < n_end) {
                     float v = tile[m * BM + c];
                     if (a.bias) v += __ldg(a.bias + n);
+                    if (a.out_scale) v *= __ldg(a.out_scale + n);
+                    if (a.split_xp && n < a.split_n) {
+                        tc_xpack_store(a.split_xp + (size_t)(n / a.split_k) * a.split_bytes, a.xp_mpad, m, n % a.split_k, v);
+                        continue;
+                    }
                     if (a.resid) v = a.resid[(size_t)m * a.ldy + n] + v;
                     a.y[(size_t)m * a.ldy + n] = v;
                 }
@@ -221,6 +305,29 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                     if (a.xp_out) tc_xpack_store(a.xp_out, a.xp_mpad, m, j, act);
                     else a.y[(size_t)m * a.ldy + j] = act;
                 }
+            }
+        }
+    } else if (a.epi == EPI_GATE || a.epi == EPI_SQRELU) {
+        auto act = [&](int m, int n, float v) {
+            if (a.epi == EPI_GATE) return v / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + n)));
+            v = fmaxf(v, 0.f);
+            return v * v;
+        };
+        if (a.xp_out && (n0 & 7) == 0 && n0 + BM <= n_end) {
+            for (int idx = tid; idx < rows * (BM / 8); idx += TC_THREADS) {
+                const int m = m_lo + idx / (BM / 8), c = (idx % (BM / 8)) * 8;
+                float v[8];
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] = act(m, n0 + c + e, tile[m * BM + c + e]);
+                tc_xpack_store8(a.xp_out, a.xp_mpad, m, n0 + c, v);
+            }
+        } else {
+            for (int idx = tid; idx < rows * BM; idx += TC_THREADS) {
+                const int m = m_lo + idx / BM, c = idx % BM, n = n0 + c;
+                if (n >= n_end) continue;
+                const float v = act(m, n, tile[m * BM + c]);
+                if (a.xp_out) tc_xpack_store(a.xp_out, a.xp_mpad, m, n, v);
+                else a.y[(size_t)m * a.ldy + n] = v;
             }
         }
     } else if (a.epi == EPI_LOGITS) {
@@ -386,7 +493,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) 
     if (warp == 0) {
         if (lane == 0) {
             const unsigned char* wsrc = reinterpret_cast<const unsigned char*>(a.W) + ((size_t)nblk * kb_total + kb0) * W_TILE;
-            const unsigned char* xsrc = a.xp + (size_t)kb0 * x_tile;
+            const unsigned char* xsrc = a.xp + (a.group_blocks ? (size_t)(nblk / a.group_blocks) * a.group_xp : 0) + (size_t)kb0 * x_tile;
             // weights never depend on the previous kernel: fill the ring with them first, then wait for
             // the packed activations
             const int pre = min(nkb, nst);
@@ -553,10 +660,10 @@ int tc_pick_split(int K, int N, int sm_count) {
     return s < 1 ? 1 : s;
 }
 
-cudaError_t launch_tc_pack_x(const float* x, int ldx, int M, int K, const float* norm_w, float eps, void* xp, cudaStream_t st, bool pdl, unsigned long long* trace) {
-    if (M < 1 || M > MR) return cudaErrorInvalidValue;
+cudaError_t launch_tc_pack_x(const float* x, int ldx, int M, int K, const float* norm_w, float eps, void* xp, cudaStream_t st, bool pdl, unsigned long long* trace, int groups, int group_x, size_t group_bytes) {
+    if (M < 1 || M > MR || groups < 1) return cudaErrorInvalidValue;
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3((unsigned)tc_mpad(M));
+    cfg.gridDim = dim3((unsigned)tc_mpad(M), (unsigned)groups);
     cfg.blockDim = dim3(256);
     cfg.stream = st;
     cudaLaunchAttribute at[1];
@@ -564,7 +671,26 @@ cudaError_t launch_tc_pack_x(const float* x, int ldx, int M, int K, const float*
     at[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = at;
     cfg.numAttrs = pdl ? 1 : 0;
-    return cudaLaunchKernelEx(&cfg, tc_pack_x_kernel, x, ldx, M, tc_mpad(M), K, tc_padded_k(K), norm_w, eps, (unsigned char*)xp, trace);
+    return cudaLaunchKernelEx(&cfg, tc_pack_x_kernel, x, ldx, M, tc_mpad(M), K, tc_padded_k(K), norm_w, eps, (unsigned char*)xp, trace, group_x, group_bytes);
+}
+
+cudaError_t launch_tc_pack_gnorm(const float* x, int ldx, int M, int K, const float* norm_w, float eps, const RowNorm& gn, void* xp, cudaStream_t st, bool pdl) {
+    if (M < 1 || M > MR || gn.groups < 1 || K % gn.groups != 0) return cudaErrorInvalidValue;
+    const int Kp = tc_padded_k(K);
+    const size_t smem = ((size_t)Kp * (gn.shift ? 2 : 1) + 2 * (size_t)gn.groups) * sizeof(float);
+    const cudaError_t e = ensure_dyn_smem(tc_pack_gnorm_kernel, smem);
+    if (e != cudaSuccess) return e;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3((unsigned)tc_mpad(M));
+    cfg.blockDim = dim3(256);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute at[1];
+    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = at;
+    cfg.numAttrs = pdl ? 1 : 0;
+    return cudaLaunchKernelEx(&cfg, tc_pack_gnorm_kernel, x, ldx, M, tc_mpad(M), K, Kp, norm_w, eps, gn, (unsigned char*)xp);
 }
 
 cudaError_t launch_gemm_tc(const TcArgs& a_in, cudaStream_t st, bool pdl) {
@@ -573,10 +699,10 @@ cudaError_t launch_gemm_tc(const TcArgs& a_in, cudaStream_t st, bool pdl) {
     a.mpad = tc_mpad(a.M);
     int dev = 0, sms = 148;
     if (cudaGetDevice(&dev) == cudaSuccess) cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    const bool multi_wave = (long)((a.N + BM - 1) / BM) * (a.ksplit > 1 ? a.ksplit : 1) >= 2L * sms;
+    const int nblk = a.group_blocks ? a.N / a.group_n * a.group_blocks : (a.N + BM - 1) / BM;
+    const bool multi_wave = (long)nblk * (a.ksplit > 1 ? a.ksplit : 1) >= 2L * sms;
     a.nstage = tc_nstage(a.mpad, multi_wave);
     a.tmem_cols = a.mpad == 16 ? 64 : a.mpad == 32 ? 128 : 256;  // power of two >= 3 * mpad
-    const int nblk = (a.N + BM - 1) / BM;
     const bool cl = a.ksplit > 1;
     const size_t smem = tc_smem_for(a.mpad, multi_wave) + (cl ? tc_recv_bytes(a.M, a.ksplit) : 0);
     {

@@ -21,7 +21,19 @@ struct TcArgs {
     const float* resid;      // optional [M][ldy], added as resid + y
     float* y;                // [M][ldy]
     int ldy;
-    unsigned char* xp_out;   // EPI_SWIGLU only, optional: write the result as packed activations for the next GEMM instead of y
+    const float* out_scale;  // EPI_STORE, optional [N]: y = resid + out_scale * (acc + bias)
+    const float* gate;       // EPI_GATE: [M][ld_gate]
+    int ld_gate;
+    // Grouped projection (block-diagonal weights, e.g. one matrix per attention head): group g owns group_blocks blocks
+    // of 128 features, reads the activation image at xp + g * group_xp and writes outputs [g * group_n, (g + 1) * group_n).
+    int group_blocks, group_n;
+    size_t group_xp;
+    // EPI_STORE, optional: outputs below split_n go to the activation images of a grouped projection instead of y
+    // (image n / split_k, element n % split_k, images split_bytes apart); split_k a multiple of 8
+    unsigned char* split_xp;
+    int split_n, split_k;
+    size_t split_bytes;
+    unsigned char* xp_out;   // EPI_SWIGLU, EPI_GATE and EPI_SQRELU, optional: write the result as packed activations for the next GEMM instead of y
     int xp_mpad;
     // RMSNorm across two GEMMs without a packing launch in between.  Producer side (EPI_STORE): besides y, the
     // epilogue writes (y * next_norm_w) as the packed activations of the next GEMM and, per 128-feature block,
@@ -53,7 +65,10 @@ int tc_mpad(int M);  // rows padded to 16 / 32 / 64
 int tc_pick_split(int K, int N, int sm_count);  // cluster size that fills the SMs once
 // f32 rows -> three bf16 terms per element in the tile layout the GEMM copies in bulk; folds an
 // RMSNorm (weight norm_w, epsilon eps) when norm_w is not NULL.
-cudaError_t launch_tc_pack_x(const float* x, int ldx, int M, int K, const float* norm_w, float eps, void* xp, cudaStream_t st, bool pdl, unsigned long long* trace = nullptr);
+// groups > 1: the images of a grouped projection, group g from x + g * group_x to xp + g * group_bytes.
+cudaError_t launch_tc_pack_x(const float* x, int ldx, int M, int K, const float* norm_w, float eps, void* xp, cudaStream_t st, bool pdl, unsigned long long* trace = nullptr, int groups = 1, int group_x = 0, size_t group_bytes = 0);
+// The same image of rows normalised in groups and token-shifted (RowNorm; runs of any length up to M).
+cudaError_t launch_tc_pack_gnorm(const float* x, int ldx, int M, int K, const float* norm_w, float eps, const RowNorm& gn, void* xp, cudaStream_t st, bool pdl);
 cudaError_t launch_gemm_tc(const TcArgs& a, cudaStream_t st, bool pdl);
 // src is [N][K] (src_is_kn = false) or [K][N]; rows land at n_off + n, or interleaved 64/64 per
 // 128-row block when interleave_which is 0 (gate) or 1 (up).

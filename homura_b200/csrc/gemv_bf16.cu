@@ -85,6 +85,100 @@ __device__ __forceinline__ float sum_slots_any(const float* s, int stride, int n
 
 __device__ __forceinline__ bool better(float v, int i, float bv, int bi) { return v > bv || (v == bv && i > bi); }
 
+// Most groups of the norm that a K range of rps rows can meet.
+__host__ __device__ __forceinline__ int gnorm_span(int K, int groups, int rps) {
+    const int n = rps / (K / groups) + 2;
+    return n < groups ? n : groups;
+}
+
+// PRO_GNORM: rows [k0, k0 + nrows) of every activation row, normalised in groups and shifted, into xs[M][rps].  Every CTA
+// forms the factors of the groups its range meets from the whole groups; the element a thread stages first and
+// everything that goes with it is requested before the factors are known.  The first slab's CTAs keep the last
+// row of every run in the state.
+template <int M>
+__device__ __forceinline__ void gnorm_stage(const GemvArgs& a, float* __restrict__ xs, float* __restrict__ gfac, int rps, int k0, int nrows, int slab, int tid) {
+    if (nrows <= 0) return;  // uniform over the CTA
+    const int lane = tid & 31, warp = tid >> 5;
+    const int gs = a.K / a.gn.groups, g_lo = k0 / gs, ng = (k0 + nrows - 1) / gs - g_lo + 1;
+    __shared__ float s_part[8];
+    int pos[M], seq[M];
+#pragma unroll
+    for (int m = 0; m < M; ++m) {
+        pos[m] = 0;
+        seq[m] = -1;
+        if (a.gn.shift && m < a.m_valid) {
+            pos[m] = a.gn.row_pos[m];
+            seq[m] = a.gn.row_seq[m];
+        }
+    }
+    auto follows = [&](int m) { return m > 0 && m < a.m_valid && seq[m] == seq[m - 1] && pos[m] == pos[m - 1] + 1; };
+    float x0[M], p0[M], w0 = 0.f, sh0 = 0.f;
+    auto fetch = [&](int k, float (&xv)[M], float (&pv)[M], float& wv, float& shv) {
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+            xv[m] = ld_cg_f32(a.x + (size_t)m * a.ldx + k);
+            pv[m] = 0.f;
+            if (a.gn.shift && m < a.m_valid && !follows(m) && pos[m] > 0) pv[m] = ld_cg_f32(a.gn.state + ((size_t)seq[m] * SHIFT_RING + (pos[m] - 1) % SHIFT_RING) * a.K + k);
+        }
+        wv = __ldg(a.norm_w + k);
+        shv = a.gn.shift ? __ldg(a.gn.shift + k) : 0.f;
+    };
+    if (tid < nrows) fetch(k0 + tid, x0, p0, w0, sh0);
+    // factors: the eight warps share the (row, group) pairs, several warps to a pair when there are fewer pairs than warps
+    const int pairs = M * ng, wpp = pairs >= 8 ? 1 : 8 / pairs;
+    for (int pb = 0; pb < pairs; pb += 8 / wpp) {
+        const int pr = pb + warp / wpp, sub = warp % wpp;
+        float s = 0.f;
+        if (pr < pairs && warp / wpp < 8 / wpp) {
+            const float* g = a.x + (size_t)(pr / ng) * a.ldx + (size_t)(g_lo + pr % ng) * gs;
+            if ((gs & 3) == 0 && (reinterpret_cast<uintptr_t>(g) & 15) == 0) {
+#pragma unroll 4
+                for (int i = sub * 32 + lane; i < gs / 4; i += 32 * wpp) {
+                    const float4 v = ld_cg_f32x4(g + 4 * (size_t)i);
+                    s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+                }
+            } else {
+#pragma unroll 4
+                for (int i = sub * 32 + lane; i < gs; i += 32 * wpp) {
+                    const float v = ld_cg_f32(g + i);
+                    s = fmaf(v, v, s);
+                }
+            }
+        }
+        s = warp_sum(s);
+        if (wpp == 1) {
+            if (lane == 0 && pr < pairs) gfac[pr] = 1.0f / sqrtf(s / (float)gs + a.eps);
+        } else {
+            if (lane == 0) s_part[warp] = s;
+            __syncthreads();
+            if (tid < 8 / wpp && tid < pairs) {
+                float t = 0.f;
+                for (int i = 0; i < wpp; ++i) t += s_part[tid * wpp + i];
+                gfac[tid] = 1.0f / sqrtf(t / (float)gs + a.eps);
+            }
+        }
+    }
+    __syncthreads();
+    for (int r = tid; r < nrows; r += GEMV_THREADS) {
+        if (r != tid) fetch(k0 + r, x0, p0, w0, sh0);
+        const int g = (k0 + r) / gs - g_lo;
+        float h[M];
+#pragma unroll
+        for (int m = 0; m < M; ++m) h[m] = (x0[m] * gfac[m * ng + g]) * w0;
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+            float v = h[m];
+            if (a.gn.shift) {
+                const float prev = m > 0 && follows(m) ? h[m > 0 ? m - 1 : 0] : p0[m];
+                v = fmaf(prev - v, sh0, v);
+                const bool last = m < a.m_valid && !(m + 1 < M && follows(m + 1 < M ? m + 1 : m));
+                if (slab == 0 && last) a.gn.state[((size_t)seq[m] * SHIFT_RING + pos[m] % SHIFT_RING) * a.K + k0 + r] = h[m];
+            }
+            xs[m * rps + r] = v;
+        }
+    }
+}
+
 // The unsplit M = 1 variant (LM head: one long stream per CTA) runs three CTAs per SM (<= 85
 // registers) to keep ~96 KB of weight loads in flight per SM; measured 5.0 -> 5.3 TB/s.  The
 // clustered one-row variants are latency chains and were slower under a tighter register budget.  The
@@ -111,6 +205,7 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
     float* cs_s = nws + rps;                        // [M][128] RoPE cos, [M][128] sin of this slab's columns (QKV epilogue)
     float* sn_s = cs_s + M * SLAB;
     float* bias_s = sn_s + M * SLAB;                // [128] bias of this slab's columns (QKV epilogue with bias)
+    float* gfac = cs_s;                             // [M][groups that meet this CTA's K range] (grouped norm; no rotation then)
     __shared__ int s_page[MAX_M], s_pos[MAX_M];     // page and position of every row's new token
     __shared__ float s_inv[MAX_M];
     __shared__ float s_warp[8][MAX_M];
@@ -124,7 +219,12 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
     const int nrows = max(0, min(a.K, k0 + rps) - k0);
     const int cg = tid & 15, rl = tid >> 4;
     const int niter = (nrows + ROWS_PER_PASS - 1) / ROWS_PER_PASS;
-    const bool col_ok = (slab * SLAB + cg * 8) < a.N;
+    // grouped projections: this slab's group, its inputs and its output columns [n0, n_end)
+    const int grp = a.group_slabs ? slab / a.group_slabs : 0;
+    const int n0 = a.group_slabs ? grp * a.group_n + (slab - grp * a.group_slabs) * SLAB : slab * SLAB;
+    const int n_end = a.group_slabs ? (grp + 1) * a.group_n : a.N;
+    const float* xin = a.x + (size_t)grp * a.group_x;
+    const bool col_ok = (n0 + cg * 8) < n_end;
     const char* wbase = (const char*)a.W + (long long)slab * a.slab_stride + (long long)(k0 + rl) * a.row_stride + cg * 16;
     const long long pass_stride = (long long)ROWS_PER_PASS * a.row_stride;
 
@@ -203,8 +303,8 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
     float resid_v = 0.f;
     const bool resid_early = a.epi == EPI_STORE && a.resid && tid < M * SLAB && (CL ? cluster_ctarank() == 0 : a.ksplit == 1);
     if (resid_early) {
-        const int m = tid / SLAB, n = slab * SLAB + (tid % SLAB);
-        if (n < a.N && m < a.m_valid) resid_v = ld_cg_f32(a.resid + (size_t)m * a.ldy + n);
+        const int m = tid / SLAB, n = n0 + (tid % SLAB);
+        if (n < n_end && m < a.m_valid) resid_v = ld_cg_f32(a.resid + (size_t)m * a.ldy + n);
     }
 
     // ---- prologue: activation slice [k0, k0+nrows) of every row into shared memory ----
@@ -228,6 +328,8 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
                     rowv[m][i] = idx < (a.K >> 2) ? ld_cg_f32x4(a.x + (size_t)m * a.ldx + 4 * (size_t)idx) : make_float4(0.f, 0.f, 0.f, 0.f);
                 }
         }
+    } else if (a.pro == PRO_GNORM) {
+        gnorm_stage<M>(a, xs, gfac, rps, k0, nrows, slab, tid);
     } else if (a.pro == PRO_RMSNORM) {
         float ss[M];
 #pragma unroll
@@ -260,7 +362,7 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
             for (int r = tid; r < nrows; r += GEMV_THREADS) xs[m * rps + r] = (__ldg(xr + r) * inv) * nws[r];
         }
     } else {
-        stage_rows<GEMV_THREADS, M>(a.x + k0, a.ldx, xs, rps, nrows, tid);
+        stage_rows<GEMV_THREADS, M>(xin + k0, a.ldx, xs, rps, nrows, tid);
     }
     __syncthreads();
     __syncthreads();
@@ -413,13 +515,13 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
 
     HM_TRACE(if (tr) a.trace[5] = global_timer();)  // split-K reduced
     // ---- epilogues on vals[M][128] (columns n0 .. n0+127 of the output) ----
-    const int n0 = slab * SLAB;
     if (a.epi == EPI_STORE) {
         for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) {
             const int m = idx / SLAB, n = n0 + (idx % SLAB);
-            if (n < a.N && m < a.m_valid) {
+            if (n < n_end && m < a.m_valid) {
                 float v = vals[idx];
                 if (a.bias) v += __ldg(a.bias + n);
+                if (a.out_scale) v *= __ldg(a.out_scale + n);
                 if (a.resid) v = (resid_early && idx == tid ? resid_v : a.resid[(size_t)m * a.ldy + n]) + v;
                 a.y[(size_t)m * a.ldy + n] = v;
             }
@@ -433,6 +535,19 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
                 const float g = vals[m * SLAB + c], u = vals[m * SLAB + 64 + c];
                 const float act = g / (1.0f + expf(-g));
                 a.y[(size_t)m * a.ldy + j] = act * u;
+            }
+        }
+    } else if (a.epi == EPI_GATE) {
+        for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) {
+            const int m = idx / SLAB, n = n0 + (idx % SLAB);
+            if (n < n_end && m < a.m_valid) a.y[(size_t)m * a.ldy + n] = vals[idx] / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + n)));
+        }
+    } else if (a.epi == EPI_SQRELU) {
+        for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) {
+            const int m = idx / SLAB, n = n0 + (idx % SLAB);
+            if (n < n_end && m < a.m_valid) {
+                const float v = fmaxf(vals[idx], 0.f);
+                a.y[(size_t)m * a.ldy + n] = v * v;
             }
         }
     } else if (a.epi == EPI_LOGITS) {
@@ -612,10 +727,14 @@ cudaError_t launch_mcs(const GemvArgs& a, size_t smem, int nslabs, cudaStream_t 
 template <int M, bool CL>
 cudaError_t launch_mc(const GemvArgs& a_in, cudaStream_t st, bool pdl) {
     GemvArgs a = a_in;
-    const int nslabs = (a.N + SLAB - 1) / SLAB;
+    const int nslabs = a.group_slabs ? a.N / a.group_n * a.group_slabs : (a.N + SLAB - 1) / SLAB;
     size_t floats = (size_t)M * a.rows_per_split + 8 * (size_t)M * SLAB + (CL ? (size_t)a.ksplit * M * SLAB : 0);
     floats += (size_t)a.rows_per_split;                            // pre-fetched RMSNorm weights
     if (a.epi == EPI_QKV_ROPE) floats += 2 * (size_t)M * SLAB + SLAB;  // pre-fetched RoPE rows and bias
+    if (a.pro == PRO_GNORM) {
+        if (a.gn.groups < 1 || a.K % a.gn.groups != 0) return cudaErrorInvalidValue;
+        floats += (size_t)M * gnorm_span(a.K, a.gn.groups, a.rows_per_split);
+    }
     size_t smem = sizeof(float) * floats;
     // cluster launches over the slab layout whose slice fits: weights staged in shared memory before the dependency wait
     const size_t slice = (size_t)a.rows_per_split * SLAB * 2;

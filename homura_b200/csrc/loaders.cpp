@@ -208,15 +208,7 @@ bool json_parse(const char* text, size_t len, Json* out, std::string* err) {
 }
 
 // ---- config.json ----------------------------------------------------------------------------
-bool parse_config_json(const std::string& path, hm_config* cfg, std::string* err) {
-    MappedFile f;
-    if (!f.open(path, err)) return false;
-    Json j;
-    if (!json_parse(reinterpret_cast<const char*>(f.data()), f.size(), &j, err)) return false;
-    if (j.kind != Json::Obj) {
-        *err = "config.json: top level is not an object";
-        return false;
-    }
+bool config_from_json(const Json& j, hm_config* cfg, std::string* err) {
     auto need = [&](const char* k, int32_t* dst) {
         const Json* v = j.get(k);
         if (!v || v->kind != Json::Num) {

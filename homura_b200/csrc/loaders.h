@@ -52,7 +52,7 @@ struct Json {
 bool json_parse(const char* text, size_t len, Json* out, std::string* err);
 
 // config.json -> hm_config (defaults: eps 1e-6, theta 1e4, max_pos 2048, src/hf/config.rs:39-47).
-bool parse_config_json(const std::string& path, hm_config* cfg, std::string* err);
+bool config_from_json(const Json& j, hm_config* cfg, std::string* err);
 
 // safetensors: 8-byte LE header length + JSON header + data.  Views point into `file`.
 bool parse_safetensors(const MappedFile& file, std::vector<TensorView>* out, std::string* err);

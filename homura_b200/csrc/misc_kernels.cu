@@ -65,6 +65,14 @@ __global__ void embed_gather_kernel(const void* table, int dtype, const uint32_t
     }
 }
 
+// rows whose logits are wanted, out of a pass over portions of several sequences
+__global__ void gather_rows_kernel(const float* src, const int32_t* rows, int W, float* dst) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const float* s = src + (size_t)rows[blockIdx.x] * W;
+    for (int i = threadIdx.x; i < W; i += blockDim.x) dst[(size_t)blockIdx.x * W + i] = s[i];
+}
+
 __device__ __forceinline__ bool better(float v, int i, float bv, int bi) { return v > bv || (v == bv && i > bi); }
 
 // ---- argmax finish: merge per-slab (value, index) pairs; ties go to the highest index ----
@@ -408,6 +416,9 @@ cudaError_t launch_pack_slabs_from_kn(const uint16_t* src_kn, int K, int N, uint
 }
 cudaError_t launch_embed_gather(const void* table, int table_dtype, const uint32_t* tokens, int M, int H, int V, float* out, int* err_flag, cudaStream_t st, bool pdl) {
     return launch_pdl(embed_gather_kernel, dim3(M), dim3(256), st, pdl, table, table_dtype, tokens, H, V, out, err_flag);
+}
+cudaError_t launch_gather_rows(const float* src, const int32_t* rows, int n, int W, float* dst, cudaStream_t st, bool pdl) {
+    return launch_pdl(gather_rows_kernel, dim3(n), dim3(256), st, pdl, src, rows, W, dst);
 }
 cudaError_t launch_argmax_finish(const float* amax_val, const int32_t* amax_idx, int nslabs, int M, uint32_t* next_tok, uint32_t* feed_tok, int32_t* pos, uint32_t* hist, int hist_stride, cudaStream_t st, bool pdl) {
     return launch_pdl(argmax_finish_kernel, dim3(M), dim3(nslabs > 4096 ? 1024 : 256), st, pdl, amax_val, amax_idx, nslabs, next_tok, feed_tok, pos, hist, hist_stride);

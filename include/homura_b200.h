@@ -98,7 +98,8 @@ HM_API const char* hm_last_error_global(void);
  * sharded index) from `model_dir`.  weight_dtype HM_BF16 keeps bf16 projections; HM_F32 (what
  * HfModel::load asks for, src/hf/model.rs:37-39) is accepted for checkpoints stored in bf16, where
  * widening to f32 changes no value; a checkpoint whose projections are stored as f32 / f16 is
- * HM_ERR_UNSUPPORTED (no f32-weight kernel). */
+ * HM_ERR_UNSUPPORTED (no f32-weight kernel).  Designs with a layer list of their own (hm_get_arch) run every projection on
+ * the f32 streaming kernels when HM_F32 is asked for, and take tensor-core copies of the weights otherwise. */
 HM_API int hm_model_load(const char* model_dir, int weight_dtype, int device, hm_engine** out);
 /* HfModel::load_gguf, src/hf/model.rs:46-75: config from `<arch>.*` metadata, blk.N.* tensors. */
 HM_API int hm_model_load_gguf(const char* gguf_path, int device, hm_engine** out);
@@ -107,6 +108,11 @@ HM_API int hm_model_load_gguf(const char* gguf_path, int device, hm_engine** out
  * QK-norm is inferred from its tensors and decides how quantised q / k / v projections are stored: hand over the
  * q_norm / k_norm weights before those projections (HM_ERR_STATE otherwise; hm_model_load* do so). */
 HM_API int hm_engine_create(const hm_config* cfg, int device, hm_engine** out);
+/* The same from the text of a config.json, for every design the library knows (its "architecture" key, e.g. "Tunitar", or
+ * the Qwen2 / Qwen3 / Llama keys).  weight_dtype as in hm_model_load. */
+HM_API int hm_engine_create_json(const char* config_json, int weight_dtype, int device, hm_engine** out);
+/* Name of the design, "" for the uniform Qwen2 / Qwen3 / Llama stacks.  Valid until the engine is destroyed. */
+HM_API const char* hm_get_arch(hm_engine* e);
 HM_API int hm_load_tensor(hm_engine* e, const char* name, int dtype, const int64_t* shape, int ndim, const void* host_data, size_t nbytes);
 HM_API int hm_finalize_weights(hm_engine* e);
 HM_API void hm_engine_destroy(hm_engine* e);
@@ -128,6 +134,13 @@ HM_API int hm_checkpoint_info(const char* path, char* buf, size_t cap, size_t* n
  * `batch` independent sequences of up to max_seq_len tokens in pages of page_tokens (16);
  * kv_dtype HM_F32 (Homura's cache dtype) or HM_BF16. */
 HM_API int hm_kv_alloc(hm_engine* e, int batch, int max_seq_len, int page_tokens, int kv_dtype);
+/* The same with one pool of pool_tokens tokens (rounded up to pages) that all sequences share: a sequence takes pages as it
+ * grows and hm_kv_reset gives them back; a call that needs more pages than are free is HM_ERR_KV_FULL and changes nothing.
+ * page_tokens 0: the design's own page size (16; 64 for latent caches), here and in hm_kv_alloc.  No counterpart in the
+ * reference, whose cache holds one sequence. */
+HM_API int hm_kv_alloc_pool(hm_engine* e, int batch, int max_seq_len, long pool_tokens, int page_tokens, int kv_dtype);
+/* Tokens that fit the free pages of the pool. */
+HM_API int hm_kv_free_tokens(hm_engine* e, long* out);
 /* Drops the cache (weights stay resident) so that hm_kv_alloc can be called again with another batch,
  * length or dtype: what init_kv_cache does when called on a model that already has a cache,
  * src/runtime.rs:1898-1938. */
@@ -141,6 +154,24 @@ HM_API int hm_kv_len(hm_engine* e, int seq, int* out);
 HM_API int hm_kv_append(hm_engine* e, int seq, int layer, const float* k_rows, const float* v_rows, int n_new, int advance);
 /* KvCache::view, src/runtime.rs:463-507: contiguous f32 [kv_heads, len, head_dim] copies. */
 HM_API int hm_kv_view(hm_engine* e, int seq, int layer, float* k_out, float* v_out);
+
+/* Latent caches: f32 [len, kv_rank] copies of the layer's latents (of the layer it shares them with). */
+HM_API int hm_latent_view(hm_engine* e, int seq, int layer, float* out);
+
+/* ---- one batch over several sequences --------------------------------------------------- */
+/* The next n_tokens tokens of sequence `seq`, after what its cache holds; want[] are the places among them whose logits are
+ * asked for (ascending). */
+typedef struct hm_step_entry {
+    int32_t seq;
+    int32_t n_tokens;
+    const uint32_t* tokens;
+    int32_t n_want;
+    const int32_t* want;
+} hm_step_entry;
+/* Runs the entries (different sequences, any mix of lengths) as one batch: the step function of a continuous-batching loop.  logits_or_null [sum of n_want, vocab], greedy_or_null [sum of n_want] argmax ids, in the
+ * order of the entries and of want; hidden_or_null [layers, sum of n_tokens, hidden] receives the residual stream after
+ * every layer (a debugging aid).  Extends the sequences; nothing changes when a status is returned. */
+HM_API int hm_step(hm_engine* e, const hm_step_entry* entries, int n_entries, float* logits_or_null, uint32_t* greedy_or_null, float* hidden_or_null);
 
 /* ---- generation (trait GenerativeModel, src/generate.rs:19-30) ---------------------- */
 /* HfGenerationContext::prefill, src/hf/model.rs:314-357: runs n prompt ids of sequence `seq`
