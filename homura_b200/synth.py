@@ -173,19 +173,6 @@ def write_hf_model(model_dir: str, cfg: DecoderConfig, seed: int, norm_jitter: f
     ``norm_jitter`` > 0 perturbs the norm weights around 1 so tests can tell a missing
     norm multiply from a present one; the benchmark models use exactly 1.
     """
-    os.makedirs(model_dir, exist_ok=True)
-    with open(os.path.join(model_dir, "config.json"), "w") as f:
-        json.dump(config_json(cfg), f, indent=1)
-    specs = hf_tensor_specs(cfg)
-    header: Dict[str, dict] = {}
-    off = 0
-    for name, shape, _ in specs:
-        nbytes = int(np.prod(shape)) * 2
-        header[name] = {"dtype": "BF16", "shape": list(shape), "data_offsets": [off, off + nbytes]}
-        off += nbytes
-    hjson = json.dumps(header, separators=(",", ":")).encode()
-    hjson += b" " * ((8 - len(hjson) % 8) % 8)
-    path = os.path.join(model_dir, "model.safetensors")
 
     def make(spec):
         name, shape, kind = spec
@@ -195,6 +182,24 @@ def write_hf_model(model_dir: str, cfg: DecoderConfig, seed: int, norm_jitter: f
             v = 1.0 + norm_jitter * _rng(seed, name).standard_normal(shape, dtype=np.float32)
             return f32_to_bf16_rne(v)
         return ones_bf16(shape)
+
+    return _write_model(model_dir, config_json(cfg), hf_tensor_specs(cfg), make)
+
+
+def _write_model(model_dir: str, config: dict, specs, make) -> str:
+    """config.json + model.safetensors with every tensor in bf16; make(spec) returns the bits of one."""
+    os.makedirs(model_dir, exist_ok=True)
+    with open(os.path.join(model_dir, "config.json"), "w") as f:
+        json.dump(config, f, indent=1)
+    header: Dict[str, dict] = {}
+    off = 0
+    for name, shape, _ in specs:
+        nbytes = int(np.prod(shape)) * 2
+        header[name] = {"dtype": "BF16", "shape": list(shape), "data_offsets": [off, off + nbytes]}
+        off += nbytes
+    hjson = json.dumps(header, separators=(",", ":")).encode()
+    hjson += b" " * ((8 - len(hjson) % 8) % 8)
+    path = os.path.join(model_dir, "model.safetensors")
 
     # every tensor has its own generator (seed, name), so they can be drawn by several threads (numpy's
     # generators release the GIL) and still be written in file order
@@ -212,6 +217,64 @@ def write_hf_model(model_dir: str, cfg: DecoderConfig, seed: int, norm_jitter: f
                 futs.append(pool.submit(make, specs[i + window]))
             f.write(arr.tobytes())
     return model_dir
+
+
+# ---- Tunitar ----------------------------------------------------------------------------------
+
+
+def tunitar_layer(heads: int, dim: int, vdim: int, kv_rank: int, ff: Optional[int], kv_from: Optional[int] = None, scale: Optional[float] = None) -> dict:
+    mixer = {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": kv_rank, "scale": dim**-0.5 if scale is None else scale}
+    if kv_from is not None:
+        mixer["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": mixer, "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+def tunitar_config(width: int, vocab: int, layers: List[dict], groups: int = 1, eps: float = 1e-6, **extra) -> dict:
+    return {"architecture": "Tunitar", "width": width, "vocab": vocab, "norm": {"groups": groups, "eps": eps}, "layers": layers, **extra}
+
+
+def tunitar_uniform(width: int, vocab: int, n_layers: int, heads: int, dim: int, kv_rank: int, ff: int, groups: int, share: bool = True) -> dict:
+    """A stack of equal layers; with `share` every second layer reads the latents of the one in front of it."""
+    return tunitar_config(width, vocab, [tunitar_layer(heads, dim, dim, kv_rank, ff, i - 1 if share and i % 2 else None) for i in range(n_layers)], groups)
+
+
+def tunitar_tensor_specs(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
+    """(name, shape, kind); kind in {'embed', 'w', 'one', 'blend'}."""
+    W, V = cfg["width"], cfg["vocab"]
+    specs: List[Tuple[str, Tuple[int, ...], str]] = [("embed", (V, W), "embed")]
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        q, v, r = m["heads"] * m["dim"], m["heads"] * m["vdim"], m["kv_rank"]
+        specs += [(p + "norm1", (W,), "one"), (p + "mix.q", (q, W), "w")]
+        if m.get("kv_from") is None:
+            specs += [(p + "mix.dkv", (r, W), "w"), (p + "mix.dkv.norm", (r,), "one")]
+        specs += [(p + "mix.uk", (q, r), "w"), (p + "mix.uv", (v, r), "w"), (p + "mix.g", (v, W), "w"), (p + "mix.o", (W, v), "w"), (p + "ls1", (W,), "one"), (p + "shift", (W,), "blend")]
+        if layer.get("mlp") is not None:
+            ff = layer["mlp"]["ff"]
+            specs += [(p + "norm2", (W,), "one"), (p + "mlp.up", (ff, W), "w"), (p + "mlp.down", (W, ff), "w"), (p + "ls2", (W,), "one")]
+    return specs + [("final.norm", (W,), "one"), ("head", (V, W), "w")]
+
+
+def tunitar_tensor(seed: int, spec) -> np.ndarray:
+    """bf16 bits of one tensor: linears N(0, 1/in), vectors around 1, blends uniform in [0, 1)."""
+    name, shape, kind = spec
+    if kind == "w":
+        return normal_bf16(seed, name, shape, float(shape[1]) ** -0.5)
+    if kind == "embed":
+        return normal_bf16(seed, name, shape, 1.0)
+    g = _rng(seed, name)
+    v = g.random(shape, dtype=np.float32) if kind == "blend" else 1.0 + 0.25 * g.standard_normal(shape, dtype=np.float32)
+    return f32_to_bf16_rne(v)
+
+
+def tunitar_weights(cfg: dict, seed: int) -> Dict[str, np.ndarray]:
+    """name -> bf16 bits of every tensor."""
+    return {s[0]: tunitar_tensor(seed, s) for s in tunitar_tensor_specs(cfg)}
+
+
+def write_tunitar_model(model_dir: str, cfg: dict, seed: int, weights: Optional[Dict[str, np.ndarray]] = None) -> str:
+    """config.json + model.safetensors of a Tunitar model (weights: bits to write instead of the seeded ones)."""
+    return _write_model(model_dir, cfg, tunitar_tensor_specs(cfg), lambda s: tunitar_tensor(seed, s) if weights is None else weights[s[0]])
 
 
 def shard_hf_model(src_dir: str, dst_dir: str, n_shards: int = 2) -> str:

@@ -62,7 +62,9 @@ def squared_relu_mlp(h, w_up, w_down):
 class Oracle:
     """config: the dict of config.json; weights: name -> array (any float dtype, widened to `dtype`)."""
 
-    def __init__(self, config: dict, weights: Dict[str, np.ndarray], dtype=np.float64):
+    def __init__(self, config: dict, weights: Dict[str, np.ndarray], dtype=np.float64, cache_round=None):
+        """cache_round: applied to the latents as a cache of fewer bits would (None: kept as they are)."""
+        self.cache_round = cache_round or (lambda c: c)
         self.cfg = config
         self.w = {k: np.asarray(v, dtype=dtype) for k, v in weights.items()}
         self.groups = int(config["norm"]["groups"])
@@ -92,7 +94,7 @@ class Oracle:
         m, p, w = self.cfg["layers"][i]["mixer"], f"l{i}.mix.", self.w
         src: Optional[int] = m.get("kv_from")
         if src is None:
-            cached[i] = latents(h, w[p + "dkv"], w[p + "dkv.norm"], self.eps)
+            cached[i] = self.cache_round(latents(h, w[p + "dkv"], w[p + "dkv.norm"], self.eps))
             src = i
         return latent_attention(h, cached[src], w[p + "q"], w[p + "uk"], w[p + "uv"], w[p + "g"], w[p + "o"], m["heads"], m["dim"], m["vdim"], m["scale"])
 
