@@ -149,6 +149,9 @@ SIGNATURES = {
     "hm_rms_norm": (_i32, [_vp, _vp, C.c_float, _i32, _i32, _vp, _vp]),
     "hm_qknorm_rope": (_i32, [_vp, _i32, _i32, _i32, _vp, C.c_float, _vp, _vp, _vp]),
     "hm_attn_decode_paged": (_i32, [_vp, _vp, _vp, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _vp]),
+    "hm_latent_pool_bytes": (C.c_size_t, [_i32, _i32, _i32]),
+    "hm_latent_write": (_i32, [_vp, _vp, C.c_float, _i32, _i32, _vp, _i32, _vp, _i32, _i32, _vp, _vp, _vp]),
+    "hm_latent_attn_paged": (_i32, [_vp, _vp, _i32, _vp, _i32, _i32, _vp, _vp, _i32, _i32, _i32, C.c_float, _i32, _vp, _vp]),
     "hm_argmax": (_i32, [_vp, _i32, _i32, _vp, _vp]),
     "hm_dev_alloc": (_i32, [C.c_size_t, C.POINTER(_vp)]),
     "hm_dev_free": (_i32, [_vp]),
@@ -737,6 +740,32 @@ def attn_decode_paged(q, k_pages: DeviceBuffer, v_pages: DeviceBuffer, kv_dtype:
     out = np.empty((B, heads * hd), np.float32)
     _check(lib.hm_attn_decode_paged(_ptr(q), C.c_void_p(k_pages.ptr), C.c_void_p(v_pages.ptr), int(kv_dtype), _ptr(pt), _ptr(kl), B, heads, kv_heads, hd, page_tokens, max_pages, _ptr(out), None))
     return out
+
+
+class LatentCache:
+    """A paged cache of latents outside an engine: normalised writes and attention over it (hm_latent_*)."""
+
+    def __init__(self, rank: int, kv_dtype: DType, page_table):
+        self._lib = load_library()
+        self.rank, self.kv_dtype = rank, kv_dtype
+        self.table = np.ascontiguousarray(page_table, dtype=np.int32)  # [sequences, pages]
+        n = int(self._lib.hm_latent_pool_bytes(rank, int(kv_dtype), int(self.table.max()) + 1))
+        self.pages = DeviceBuffer(n)
+        self.pages.upload(np.zeros(n, np.uint8))
+
+    def write(self, c, w, eps: float, row_seq, row_pos):
+        c = np.ascontiguousarray(c, dtype=np.float32)
+        w = np.ascontiguousarray(w, dtype=np.float32)
+        s, p = np.ascontiguousarray(row_seq, dtype=np.int32), np.ascontiguousarray(row_pos, dtype=np.int32)
+        _check(self._lib.hm_latent_write(_ptr(c), _ptr(w), eps, c.shape[0], self.rank, _ptr(self.pages.ptr), int(self.kv_dtype), _ptr(self.table), self.table.shape[0], self.table.shape[1], _ptr(s), _ptr(p), None))
+
+    def attend(self, q, scale: float, row_seq, row_pos, nsplit: int = 0) -> np.ndarray:
+        """q [rows, heads, rank] -> softmax(scale * q . latents) latents, row m up to position row_pos[m]."""
+        q = np.ascontiguousarray(q, dtype=np.float32)
+        s, p = np.ascontiguousarray(row_seq, dtype=np.int32), np.ascontiguousarray(row_pos, dtype=np.int32)
+        out = np.empty_like(q)
+        _check(self._lib.hm_latent_attn_paged(_ptr(q), _ptr(self.pages.ptr), int(self.kv_dtype), _ptr(self.table), self.table.shape[0], self.table.shape[1], _ptr(s), _ptr(p), q.shape[0], q.shape[1], self.rank, scale, nsplit, _ptr(out), None))
+        return out
 
 
 def dev_sync():

@@ -12,6 +12,7 @@
 #include "engine.h"
 #include "gemm_tc.h"
 #include "kquant.h"
+#include "latent_attn.h"
 #include "sampler.h"
 #include "loaders.h"
 
@@ -978,6 +979,78 @@ int hm_attn_decode_paged(const float* q, const void* k_pages, const void* v_page
     const int rc = sg.finish(le);
     if (rc != HM_OK) return rc;
     if (synced && take_wait_err()) return gfail(HM_ERR_TIMEOUT, "hm_attn_decode_paged: a bounded device-side wait ran out");
+    return HM_OK;
+}
+
+size_t hm_latent_pool_bytes(int rank, int kv_dtype, int n_pages) {
+    if (rank < 1 || n_pages < 1 || (kv_dtype != HM_F32 && kv_dtype != HM_BF16)) return 0;
+    return (size_t)n_pages * latent_page_elems(rank, kv_dtype == HM_BF16) * (kv_dtype == HM_BF16 ? 2 : 4);
+}
+
+static int check_latent_rows(const int32_t* row_seq, const int32_t* row_pos, int M, int n_seq, int max_pages) {
+    for (int m = 0; m < M; ++m)
+        if (row_seq[m] < 0 || row_seq[m] >= n_seq || row_pos[m] < 0 || row_pos[m] >= max_pages * LATENT_PAGE) return gfail(HM_ERR_INVALID, "latent cache: row outside the page table");
+    return HM_OK;
+}
+
+int hm_latent_write(const float* c, const float* w, float eps, int M, int rank, void* pages, int kv_dtype, const int32_t* page_table, int n_seq, int max_pages, const int32_t* row_seq, const int32_t* row_pos, void* stream) {
+    if (!c || !w || !pages || !page_table || !row_seq || !row_pos || M < 1 || rank < 1 || rank > 1024 || n_seq < 1 || max_pages < 1) return gfail(HM_ERR_INVALID, "hm_latent_write: bad arguments");
+    if (kv_dtype != HM_F32 && kv_dtype != HM_BF16) return gfail(HM_ERR_UNSUPPORTED, "hm_latent_write: cache dtype must be f32 or bf16");
+    NEED_DEVICE();
+    if (!is_device_ptr(pages)) return gfail(HM_ERR_INVALID, "hm_latent_write: the pages must live in device memory");
+    if (is_device_ptr(row_seq) || is_device_ptr(row_pos)) return gfail(HM_ERR_INVALID, "hm_latent_write: row_seq and row_pos are host arrays");
+    if (const int rc = check_latent_rows(row_seq, row_pos, M, n_seq, max_pages)) return rc;
+    cudaStream_t st = (cudaStream_t)stream;
+    Staging sg(st);
+    const LatentPool pool{pages, sg.in(page_table, (size_t)n_seq * max_pages), max_pages, rank, kv_dtype == HM_BF16};
+    const float *cd = sg.in(c, (size_t)M * rank), *wd = sg.in(w, (size_t)rank);
+    const int32_t *sd = sg.in(row_seq, (size_t)M), *pd = sg.in(row_pos, (size_t)M);
+    if (!pool.page_table || !cd || !wd || !sd || !pd) return sg.finish(cudaErrorMemoryAllocation);
+    return sg.finish(launch_latent_write(pool, cd, rank, M, wd, eps, pd, sd, st, false));
+}
+
+int hm_latent_attn_paged(const float* q, const void* pages, int kv_dtype, const int32_t* page_table, int n_seq, int max_pages, const int32_t* row_seq, const int32_t* row_pos, int M, int heads, int rank, float scale,
+                         int nsplit, float* out, void* stream) {
+    if (!q || !pages || !page_table || !row_seq || !row_pos || !out || M < 1 || M > 64 || heads < 1 || rank < 1 || rank > 1024 || n_seq < 1 || max_pages < 1 || nsplit < 0 || nsplit > 256)
+        return gfail(HM_ERR_INVALID, "hm_latent_attn_paged: bad arguments (M <= 64, rank <= 1024)");
+    if (kv_dtype != HM_F32 && kv_dtype != HM_BF16) return gfail(HM_ERR_UNSUPPORTED, "hm_latent_attn_paged: cache dtype must be f32 or bf16");
+    NEED_DEVICE();
+    if (!is_device_ptr(pages)) return gfail(HM_ERR_INVALID, "hm_latent_attn_paged: the pages must live in device memory");
+    if (is_device_ptr(row_seq) || is_device_ptr(row_pos)) return gfail(HM_ERR_INVALID, "hm_latent_attn_paged: row_seq and row_pos are host arrays");
+    if (const int rc = check_latent_rows(row_seq, row_pos, M, n_seq, max_pages)) return rc;
+    const int bf16 = kv_dtype == HM_BF16;
+    int longest = 0, tiles = 0;
+    const int rpt = latent_rows_per_tile(M, heads, rank, bf16);
+    for (int m = 0; m < M; ++m) {
+        longest = std::max(longest, row_pos[m] + 1);
+        if (m % rpt == 0 || row_seq[m - 1] != row_seq[m] || row_pos[m - 1] + 1 != row_pos[m]) ++tiles;
+    }
+    cudaStream_t st = (cudaStream_t)stream;
+    Staging sg(st);
+    LatentAttnArgs a{};
+    a.pool = LatentPool{const_cast<void*>(pages), sg.in(page_table, (size_t)n_seq * max_pages), max_pages, rank, bf16};
+    a.q = sg.in(q, (size_t)M * heads * rank);
+    a.ldq = a.ldo = heads * rank;
+    a.M = M;
+    a.heads = heads;
+    a.row_pos = sg.in(row_pos, (size_t)M);
+    a.row_seq = sg.in(row_seq, (size_t)M);
+    a.scale = scale;
+    a.tiles = rpt > 1 ? tiles : 0;
+    a.nsplit = nsplit ? nsplit : latent_pick_nsplit(tiles, heads, rank, bf16, longest, sm_count_of_current_device(), 256);
+    a.out = sg.out(out, (size_t)M * heads * rank);
+    if (!a.pool.page_table || !a.q || !a.row_pos || !a.row_seq || !a.out) return sg.finish(cudaErrorMemoryAllocation);
+    if (!sg.ok(get_wait_err(&a.err_flag))) return sg.finish(cudaSuccess);
+    if (a.nsplit > 1) {
+        const size_t acc = (size_t)M * heads * a.nsplit * rank;
+        unsigned int* unused = nullptr;
+        if (!sg.ok(get_scratch(acc + (size_t)M * heads * a.nsplit * 2, 1, &a.part_acc, &unused))) return sg.finish(cudaSuccess);
+        a.part_ml = a.part_acc + acc;
+    }
+    int launches = 0;
+    const int rc = sg.finish(launch_latent_attn(a, st, false, &launches));  // the row arrays are always staged, so this call synchronised
+    if (rc != HM_OK) return rc;
+    if (take_wait_err()) return gfail(HM_ERR_TIMEOUT, "hm_latent_attn_paged: a bounded device-side wait ran out");
     return HM_OK;
 }
 

@@ -1414,8 +1414,10 @@ int Engine::prefill(int seq, const int64_t* ids, int n, float* logits, uint32_t*
         const int mc = std::min(chunk, n - c0);
         const bool last = c0 + mc >= n;
         pass_longest_ = len0 + c0 + mc;
+        pass_runs_.assign(1, {0, mc});
         int rc = enqueue_pass(mc, pf_tokens_ + c0, pf_pos_ + c0, pf_seq_ + c0, mc - 1, last ? 1 : 0, false, next_dev_ + seq, tokens_dev_ + seq, pos_dev_ + seq, hist_dev_ + (size_t)seq * (max_seq_ + 1),
                               &launches);
+        pass_runs_.clear();
         if (rc) return rc;
     }
     uint32_t* tok_pin = st + 3 * n + 1;

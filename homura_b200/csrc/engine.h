@@ -224,6 +224,7 @@ class Engine {
     float *shift_state_ = nullptr, *shift_saved_ = nullptr;  // [layers][sequences][SHIFT_RING][H]; [layers][SHIFT_RING][H]
     int32_t* seq_iota_ = nullptr;    // 0, 1, 2, ...: the sequence of every row of a decode step
     int pass_longest_ = 0;           // longest context of the pass being enqueued (splits of the attention)
+    std::vector<std::pair<int, int>> pass_runs_;  // that pass's runs: first row, rows; empty: a run per row
     // portions (step)
     float* hsel_ = nullptr;              // rows whose logits are wanted
     const int32_t* lm_pick_ = nullptr;   // their indices within the pass being enqueued (null: lm_row0 ..)

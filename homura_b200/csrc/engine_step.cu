@@ -143,6 +143,11 @@ int Engine::step(const hm_step_entry* entries, int n, float* logits, uint32_t* g
         const int mc = (int)std::min<size_t>(chunk, rows - c0), nw = logits || greedy ? pass_wants[pass] : 0;
         tap_row0_ = c0;
         pass_longest_ = pass_longest[pass];
+        pass_runs_.clear();
+        for (int m = 0; m < mc; ++m) {  // a sequence's tokens are consecutive, so its rows within the pass are one run
+            if (m > 0 && p_seq[c0 + m] == p_seq[c0 + m - 1]) pass_runs_.back().second++;
+            else pass_runs_.push_back({m, 1});
+        }
         lm_pick_ = nw ? st_want_ + done : nullptr;
         rc = enqueue_pass(mc, st_tokens_ + c0, st_pos_ + c0, st_seq_ + c0, 0, nw, false, st_next_ + done, nullptr, nullptr, nullptr, &launches);
         if (rc == HM_OK && nw && logits) {
@@ -151,6 +156,7 @@ int Engine::step(const hm_step_entry* entries, int n, float* logits, uint32_t* g
         }
         done += nw;
     }
+    pass_runs_.clear();
     tap_ = nullptr;
     lm_pick_ = nullptr;
     if (rc) return rc;

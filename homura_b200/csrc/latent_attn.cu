@@ -288,13 +288,23 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
     float* sc = reinterpret_cast<float*>(pb + g.p_bytes);     // [np][132]
     constexpr int SLD = TCL_TOK + 4;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int m0 = blockIdx.x, h0 = blockIdx.y * heads_per_cta, split = blockIdx.z;
+    const int h0 = blockIdx.y * heads_per_cta, split = blockIdx.z;
     const int nh = min(heads_per_cta, a.heads - h0), R = a.pool.rank;
-    // rows of the pass never change within it: the run that starts here, and nothing to do when the row belongs to the CTA in front
+    // The pass's rows cut into tiles: a tile starts at every multiple of rows_per_tile and wherever a run starts.  Every warp
+    // finds this CTA's tile, the blockIdx.x-th, on its own (the rows of a pass never change within it).
+    uint64_t starts = 0;
+    for (int i = 0; i < a.M; i += 32) {
+        const int m = i + lane;
+        const bool st = m < a.M && (m % a.rows_per_tile == 0 || a.row_seq[m - 1] != a.row_seq[m] || a.row_pos[m - 1] + 1 != a.row_pos[m]);
+        starts |= (uint64_t)__ballot_sync(0xffffffffu, st) << i;
+    }
+    if (a.M < 64) starts |= (uint64_t)1 << a.M;  // end mark
+    for (int i = 0; i < (int)blockIdx.x && starts; ++i) starts &= starts - 1;
+    const int m0 = starts ? __ffsll((long long)starts) - 1 : a.M;
+    if (m0 >= a.M) return;  // fewer tiles than CTAs
+    const uint64_t after = starts & (starts - 1);
+    const int rows = (after ? __ffsll((long long)after) - 1 : a.M) - m0;
     const int seq = a.row_seq[m0], pos0 = a.row_pos[m0];
-    if (m0 % a.rows_per_tile != 0 && a.row_seq[m0 - 1] == seq && a.row_pos[m0 - 1] + 1 == pos0) return;
-    int rows = 1;
-    while ((m0 + rows) % a.rows_per_tile != 0 && m0 + rows < a.M && a.row_seq[m0 + rows] == seq && a.row_pos[m0 + rows] == pos0 + rows) ++rows;
     const int pairs = rows * nh;  // pair p: row p / nh, head p % nh
     const int len = pos0 + rows, tiles = (len + TCL_TOK - 1) / TCL_TOK, per = (tiles + a.nsplit - 1) / a.nsplit;
     const int t0 = split * per, nt = min(tiles, t0 + per) - t0;
@@ -582,11 +592,10 @@ int latent_rows_per_tile(int M, int heads, int rank, int bf16) {
     return r < 1 ? 1 : r;
 }
 
-int latent_pick_nsplit(int M, int heads, int rank, int bf16, int longest, int sm_count, int max_split) {
+int latent_pick_nsplit(int tiles, int heads, int rank, int bf16, int longest, int sm_count, int max_split) {
     const int mp = latent_tc_pairs(rank, bf16);
-    const int rpt = latent_rows_per_tile(M, heads, rank, bf16);
     const int hg = mp ? (heads + tcl_heads(heads, mp) - 1) / tcl_heads(heads, mp) : (heads + CC_HEADS - 1) / CC_HEADS;
-    const int ctas = (M + rpt - 1) / rpt * hg;
+    const int ctas = tiles * hg;
     const int tok = mp ? TCL_TOK : CC_TOK;
     int s = sm_count / (ctas > 0 ? ctas : 1);
     const int most = (longest + tok - 1) / tok;
@@ -609,7 +618,7 @@ cudaError_t launch_latent_read(const LatentPool& pool, int seq, int len, float* 
 cudaError_t launch_latent_attn(const LatentAttnArgs& a_in, cudaStream_t st, bool pdl, int* launches) {
     LatentAttnArgs a = a_in;
     const int R = a.pool.rank, mp = latent_tc_pairs(R, a.pool.bf16);
-    if (R < 1 || a.M < 1 || a.heads < 1 || a.nsplit < 1 || a.nsplit > 256) return cudaErrorInvalidValue;
+    if (R < 1 || a.M < 1 || (mp > 0 && a.M > 64) || a.tiles < 0 || a.tiles > a.M || a.heads < 1 || a.nsplit < 1 || a.nsplit > 256) return cudaErrorInvalidValue;
     cudaError_t e;
     if (mp > 0) {
         const int hpc = tcl_heads(a.heads, mp);
@@ -617,7 +626,7 @@ cudaError_t launch_latent_attn(const LatentAttnArgs& a_in, cudaStream_t st, bool
         TclGeom g;
         const int rows = a.rows_per_tile < a.M ? a.rows_per_tile : a.M;
         if (!tcl_geom(R, rows * hpc, &g)) return cudaErrorInvalidValue;
-        e = launch(latent_attn_tc_kernel, dim3(a.M, (a.heads + hpc - 1) / hpc, a.nsplit), dim3(TCL_THREADS), g.smem, st, pdl, a, g, hpc);
+        e = launch(latent_attn_tc_kernel, dim3(a.tiles > 0 ? a.tiles : a.M, (a.heads + hpc - 1) / hpc, a.nsplit), dim3(TCL_THREADS), g.smem, st, pdl, a, g, hpc);
     } else {
         const size_t smem = (size_t)(CC_HEADS + CC_TOK) * cc_stride(R) * 4;
         const dim3 grid(a.M, (a.heads + CC_HEADS - 1) / CC_HEADS, a.nsplit);

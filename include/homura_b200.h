@@ -298,6 +298,15 @@ HM_API int hm_qknorm_rope(float* x, int rows, int heads, int hd, const float* no
  * memory is trusted (entries must lie in [1, max_pages*page_tokens]) and the call stays asynchronous
  * when every pointer is a device pointer. */
 HM_API int hm_attn_decode_paged(const float* q, const void* k_pages, const void* v_pages, int kv_dtype, const int32_t* page_table, const int32_t* kv_len, int B, int heads, int kv_heads, int hd, int page_tokens, int max_pages, float* out, void* stream);
+/* RMSNorm over rank (weight w) of M latent rows [M, rank] f32 and their write into a paged latent cache: `pages` is device
+ * memory of hm_latent_pool_bytes, page_table [n_seq, max_pages] int32 over 64-token pages, row m belongs at position
+ * row_pos[m] of sequence row_seq[m].  No counterpart in the reference. */
+HM_API size_t hm_latent_pool_bytes(int rank, int kv_dtype, int n_pages);
+HM_API int hm_latent_write(const float* c, const float* w, float eps, int M, int rank, void* pages, int kv_dtype, const int32_t* page_table, int n_seq, int max_pages, const int32_t* row_seq, const int32_t* row_pos, void* stream);
+/* Softmax attention whose keys and values are the cached latents themselves: q [M, heads, rank], out [M, heads, rank] f32, row m
+ * sees positions 0 .. row_pos[m] of sequence row_seq[m] (M <= 64).  row_seq and row_pos are HOST arrays (range-checked);
+ * nsplit CTAs share a context (0 = choose). */
+HM_API int hm_latent_attn_paged(const float* q, const void* pages, int kv_dtype, const int32_t* page_table, int n_seq, int max_pages, const int32_t* row_seq, const int32_t* row_pos, int M, int heads, int rank, float scale, int nsplit, float* out, void* stream);
 /* argmax with ties to the highest index (src/generate.rs:457-468): logits [rows, n]. */
 HM_API int hm_argmax(const float* logits, int rows, int n, uint32_t* out, void* stream);
 
