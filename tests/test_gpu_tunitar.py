@@ -169,3 +169,161 @@ def test_latents_in_the_cache(hm, engines):
         close(m.latent_view(layer, c.shape[1], seq=1), c, "F32", "cached latents")
     with pytest.raises(hm.HomuraError):
         m.kv_view(0)
+
+
+# ---- generation through the engine's own loops and the scheduler ---------------------------------
+
+
+@functools.lru_cache(maxsize=None)
+def greedy(name, seed, n_prompt, n_new):
+    ids = tuple(int(t) for t in synth.prompt_ids(seed, n_prompt, model(name)["vocab"]))
+    return ids, tuple(oracle_of(name, "F32").greedy(ids, n_new))
+
+
+def test_greedy_generation(hm, engines):
+    ids, want = greedy("mixed", 70, 37, 60)
+    m = engines("mixed", "F32")
+    m.init_kv_cache(128, batch=1, kv_dtype=hm.DType.F32)
+    assert tuple(m.generate_ids(ids, 60, hm.SamplingConfig.greedy())) == want
+
+
+def test_batched_decode_graph(hm, engines):
+    """Three, twelve (tensor-core projections) and seventy sequences decode together what each decodes alone."""
+    for batch in (3, 12, 70):
+        m = engines("mixed", "F32" if batch == 3 else "BF16")
+        m.init_kv_cache(64, batch=batch, kv_dtype=hm.DType.F32)
+        refs = [greedy("mixed", 80 + b % 6, 5 + b % 6, 12) for b in range(batch)]
+        first = [m.prefill(ids, seq=b) for b, (ids, _) in enumerate(refs)]
+        rest = m.decode_greedy_n(first, 11)
+        for b, (_, want) in enumerate(refs):
+            assert (first[b], *rest[b].tolist()) == want
+
+
+def test_scheduler_generates_what_each_prompt_generates_alone(hm, engines):
+    refs = [greedy("mixed", 90 + i, n, 20) for i, n in enumerate((70, 1, 33, 150, 2, 64))]
+    m = engines("mixed", "F32")
+    sched = Scheduler(Session(m, 3, 5 * 64, kv_dtype=hm.DType.F32), portion=24, batch_tokens=40)
+    assert [tuple(o) for o in sched.run([ids for ids, _ in refs], 20)] == [want for _, want in refs]
+    assert m.free_tokens() == 5 * 64
+    with pytest.raises(hm.KvCacheFull):
+        sched.run([[1] * 400], 4)
+
+
+def test_sampled_generation_matches_the_host_sampler(hm, engines):
+    cfg = hm.SamplingConfig(temperature=0.8, top_k=12, top_p=0.9, repetition_penalty=1.2, seed=5)
+    ids, _ = greedy("mixed", 70, 37, 60)
+    m = engines("mixed", "F32")
+    m.init_kv_cache(128, batch=1, kv_dtype=hm.DType.F32)
+    got = m.generate_ids(ids, 25, cfg)
+    m.reset_kv_cache()
+    cur, rng, out = m.prefill(ids), 5 | 1, []
+    out.append(cur)
+    for _ in range(24):
+        lg, _ = m.decode_step([cur])
+        cur, rng = hm.sample_token(lg[0], cfg, out, rng)
+        out.append(cur)
+    assert got == out
+
+
+@pytest.mark.parametrize("sampling", ["greedy", "sampled"])
+def test_a_conversation_goes_on_after_the_end_token(hm, tmp_path, sampling):
+    """Generation runs ahead of the host in blocks; what the end token cut off must leave no trace in the next turn."""
+    cfg = model("mixed")
+    ids, out = greedy("mixed", 70, 37, 60)
+    sc = hm.SamplingConfig.greedy() if sampling == "greedy" else hm.SamplingConfig(temperature=0.7, top_k=4, repetition_penalty=1.0, seed=3)
+    if sampling == "sampled":
+        m = hm.HfModel.load_with_dtype(synth.write_tunitar_model(str(tmp_path / "a"), cfg, 21, weights("mixed")), hm.DType.F32)
+        m.init_kv_cache(128, batch=1, kv_dtype=hm.DType.F32)
+        out = tuple(m.generate_ids(ids, 60, sc))
+        m.close()
+    k = next(i for i in range(5, 31) if out[i] not in out[:i])
+    cfg["eos_token_id"] = int(out[k])
+    m = hm.HfModel.load_with_dtype(synth.write_tunitar_model(str(tmp_path / "b"), cfg, 21, weights("mixed")), hm.DType.F32)
+    m.init_kv_cache(128, batch=1, kv_dtype=hm.DType.F32)
+    got = m.generate_ids(ids, 60, sc)
+    assert tuple(got) == out[:k] and m.kv_cache_len() == len(ids) + k
+    more = [3, 1, 4, 1, 5]
+    _, lg = m.prefill(more, want_logits=True)
+    close(lg, oracle_of("mixed", "F32").forward([*ids, *out[:k], *more])[-1], "F32", "second turn")
+    m.close()
+
+
+def test_tensors_one_by_one_and_missing_ones(hm):
+    import json
+
+    cfg = model("odd")
+    tensors = [(n, hm.DType.BF16, s, weights("odd")[n]) for n, s, _ in synth.tunitar_tensor_specs(cfg)]
+    ids, want, _ = expected("odd", "F32", 1, 150)
+    m = hm.HfModel.from_config_json(json.dumps(cfg), tensors, hm.DType.F32)
+    m.init_kv_cache(64, batch=1, kv_dtype=hm.DType.F32)
+    close(run_portions(m, ids[:30], [30]), want[:30], "F32", "logits of a prompt")
+    m.close()
+    for drop in ("l0.shift", "l1.ls2", "l0.mix.dkv.norm", "l1.mix.uk", "l0.mix.g", "final.norm", "head"):
+        with pytest.raises(hm.HomuraError) as e:
+            hm.HfModel.from_config_json(json.dumps(cfg), [t for t in tensors if t[0] != drop])
+        assert "missing weight" in e.value.message
+    with pytest.raises(hm.HomuraError):
+        hm.HfModel.from_config_json(json.dumps(cfg), [("l1.mix.dkv", hm.DType.BF16, (65, 130), np.zeros((65, 130), np.uint16))])
+
+
+def test_step_refuses_bad_entries_and_keeps_its_state(hm, engines):
+    ids, want, _ = expected("mixed", "F32", 1, 150)
+    m = engines("mixed", "F32")
+    m.init_kv_cache(128, batch=2, kv_dtype=hm.DType.F32, pool_tokens=128)
+    close(run_portions(m, ids[:40], [40]), want[:40], "F32", "logits of a prompt")
+    for bad in ([(0, [1], [0]), (0, [2], [])], [(2, [1], [])], [(0, [], [])], [(0, [100], [])], [(0, [1, 2], [1, 0])], [(0, [1], [1])]):
+        with pytest.raises(hm.HomuraError):
+            m.step(bad)
+    with pytest.raises(hm.KvCacheFull):
+        m.step([(0, [1] * 60, []), (1, [1] * 10, [])])
+    assert (m.kv_cache_len(0), m.kv_cache_len(1), m.free_tokens()) == (40, 0, 64)
+    close(run_portions(m, ids[40:90], [50]), want[40:90], "F32", "logits after a refusal")
+
+
+def test_uniform_models_take_mixed_batches_too(hm, oracle, tmp_path):
+    """The page pool and hm_step serve the Qwen2-shaped stack as well."""
+    cfg = synth.tiny_config()
+    d = synth.write_hf_model(str(tmp_path), cfg, 7, norm_jitter=0.1)
+    m = hm.HfModel.load(d)
+    session = Session(m, 2, 10 * 16, kv_dtype=hm.DType.F32)
+    for _ in range(2):  # the second round runs on pages that were given back
+        prompts = {k: synth.prompt_ids(s, n, cfg.vocab_size) for k, s, n in (("x", 1, 40), ("y", 2, 90))}
+        want = {}
+        for k, p in prompts.items():
+            om = oracle.OracleModel.from_hf_dir(d, max_seq_len=128)
+            want[k] = om.forward_all(p)
+        session.step([("x", prompts["x"][:3], [])], want_logits=False)
+        lg, ids = session.step([("y", prompts["y"][:70], [0, 69]), ("x", prompts["x"][3:39], [35])], want_greedy=True)
+        ref = np.stack([want["y"][0], want["y"][69], want["x"][38]])
+        assert np.abs(lg - ref).max() < 1e-4 * max(1.0, np.abs(ref).max())
+        assert ids.tolist() == [oracle.argmax(r) for r in ref]
+        lg, _ = session.step([("x", prompts["x"][39:], [0]), ("y", prompts["y"][70:], [19])])
+        ref = np.stack([want["x"][39], want["y"][89]])
+        assert np.abs(lg - ref).max() < 1e-4 * max(1.0, np.abs(ref).max())
+        session.end("x")
+        session.end("y")
+    m.close()
+
+
+def test_the_trace_runner_replays_steps(hm, tmp_path):
+    import json
+    import os
+    import subprocess
+    import sys
+
+    ids, want, _ = expected("odd", "F32", 1, 150)
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    d = synth.write_tunitar_model(str(tmp_path / "model"), model("odd"), 21, weights("odd"))
+    out = tmp_path / "out"
+    out.mkdir()
+    steps = [{"step": 0, "entries": [{"id": "p", "tokens": ids[:50], "want": [2, 49]}], "end": []},
+             {"step": 1, "entries": [{"id": "q", "tokens": ids[:9], "want": []}, {"id": "p", "tokens": ids[50:51], "want": []}], "end": ["p"]},
+             {"step": 2, "entries": [{"id": "q", "tokens": ids[9:11], "want": [1]}, {"id": "r", "tokens": ids[:64], "want": [63]}], "end": ["q", "r"]}]
+    r = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", d, "--dtype", "float32", "--out", str(out), "--max-tokens", "128"],
+                       input="\n".join(map(json.dumps, steps)), capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stderr
+    assert [ln for ln in r.stdout.splitlines() if ln.startswith("done")] == ["done 0", "done 1", "done 2"]
+    read = lambda n: np.fromfile(out / f"{n}.f32", "<f4").reshape(-1, 77)
+    close(read(0), want[[2, 49]], "F32", "replayed logits")
+    assert not (out / "1.f32").exists()
+    close(read(2), want[[10, 63]], "F32", "replayed logits")
