@@ -238,6 +238,11 @@ def tunitar_uniform(width: int, vocab: int, n_layers: int, heads: int, dim: int,
     return tunitar_config(width, vocab, [tunitar_layer(heads, dim, dim, kv_rank, ff, i - 1 if share and i % 2 else None) for i in range(n_layers)], groups)
 
 
+# Tunitar stacks with the width, depth, heads, cache bytes per token and MLP parameters of the Qwen2.5 architectures above.
+TUNITAR_05B = tunitar_uniform(896, 151936, 24, 14, 64, 256, 7296, 7)
+TUNITAR_15B = tunitar_uniform(1536, 151936, 28, 12, 128, 512, 13440, 12)
+
+
 def tunitar_tensor_specs(cfg: dict) -> List[Tuple[str, Tuple[int, ...], str]]:
     """(name, shape, kind); kind in {'embed', 'w', 'one', 'blend'}."""
     W, V = cfg["width"], cfg["vocab"]
