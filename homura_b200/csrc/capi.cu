@@ -1019,8 +1019,12 @@ int hm_latent_attn_paged(const float* q, const void* pages, int kv_dtype, const 
     if (is_device_ptr(row_seq) || is_device_ptr(row_pos)) return gfail(HM_ERR_INVALID, "hm_latent_attn_paged: row_seq and row_pos are host arrays");
     if (const int rc = check_latent_rows(row_seq, row_pos, M, n_seq, max_pages)) return rc;
     const int bf16 = kv_dtype == HM_BF16;
-    int longest = 0, tiles = 0;
-    const int rpt = latent_rows_per_tile(M, heads, rank, bf16);
+    int longest = 0, tiles = 0, longest_run = 1;
+    for (int m = 1, run = 1; m < M; ++m) {
+        run = row_seq[m - 1] == row_seq[m] && row_pos[m - 1] + 1 == row_pos[m] ? run + 1 : 1;
+        longest_run = std::max(longest_run, run);
+    }
+    const int rpt = latent_rows_per_tile(longest_run, heads, rank, bf16);
     for (int m = 0; m < M; ++m) {
         longest = std::max(longest, row_pos[m] + 1);
         if (m % rpt == 0 || row_seq[m - 1] != row_seq[m] || row_pos[m - 1] + 1 != row_pos[m]) ++tiles;
@@ -1036,7 +1040,8 @@ int hm_latent_attn_paged(const float* q, const void* pages, int kv_dtype, const 
     a.row_pos = sg.in(row_pos, (size_t)M);
     a.row_seq = sg.in(row_seq, (size_t)M);
     a.scale = scale;
-    a.tiles = rpt > 1 ? tiles : 0;
+    a.rows_per_tile = rpt;
+    a.tiles = tiles;
     a.nsplit = nsplit ? nsplit : latent_pick_nsplit(tiles, heads, rank, bf16, longest, sm_count_of_current_device(), 256);
     a.out = sg.out(out, (size_t)M * heads * rank);
     if (!a.pool.page_table || !a.q || !a.row_pos || !a.row_seq || !a.out) return sg.finish(cudaErrorMemoryAllocation);

@@ -208,6 +208,19 @@ __device__ __forceinline__ uint16_t f32_to_bf16_rne(float f) {
     u += 0x7FFFu + ((u >> 16) & 1u);
     return (uint16_t)(u >> 16);
 }
+// Two values as one word of bf16 (lo in the lower half), and as three words whose sum they are (exact to 2^-24 relative).
+__device__ __forceinline__ uint32_t bf16x2_rne(float lo, float hi) {
+    uint32_t r;
+    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r) : "f"(hi), "f"(lo));
+    return r;
+}
+__device__ __forceinline__ void bf16x2_split3(float lo, float hi, uint32_t& a, uint32_t& b, uint32_t& c) {
+    a = bf16x2_rne(lo, hi);
+    lo -= bf16_lo(a);
+    hi -= bf16_hi(a);
+    b = bf16x2_rne(lo, hi);
+    c = bf16x2_rne(lo - bf16_lo(b), hi - bf16_hi(b));
+}
 __device__ __forceinline__ float f16_bits_to_f32(uint16_t h) {
     float f;
     asm("{ .reg .b16 t; mov.b16 t, %1; cvt.f32.f16 %0, t; }" : "=f"(f) : "h"(h));
@@ -279,20 +292,7 @@ __device__ __forceinline__ void tc_xpack_store(unsigned char* xp, int mpad, int 
 __device__ __forceinline__ void tc_xpack_store8(unsigned char* xp, int mpad, int m, int k0, const float (&v)[8]) {
     uint32_t w[3][4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-        uint16_t h[2], md[2], lo[2];
-#pragma unroll
-        for (int u = 0; u < 2; ++u) {
-            const float x = v[2 * e + u];
-            h[u] = f32_to_bf16_rne(x);
-            const float r1 = x - bf16_bits_to_f32(h[u]);
-            md[u] = f32_to_bf16_rne(r1);
-            lo[u] = f32_to_bf16_rne(r1 - bf16_bits_to_f32(md[u]));
-        }
-        w[0][e] = (uint32_t)h[0] | ((uint32_t)h[1] << 16);
-        w[1][e] = (uint32_t)md[0] | ((uint32_t)md[1] << 16);
-        w[2][e] = (uint32_t)lo[0] | ((uint32_t)lo[1] << 16);
-    }
+    for (int e = 0; e < 4; ++e) bf16x2_split3(v[2 * e], v[2 * e + 1], w[0][e], w[1][e], w[2][e]);
     const int kb = k0 >> 6, chunk = (k0 & 63) >> 3;
     unsigned char* tile = xp + (size_t)kb * (3 * mpad * 128);
 #pragma unroll

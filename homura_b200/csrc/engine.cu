@@ -675,7 +675,7 @@ int Engine::kv_append(int seq, int layer, const float* k_rows, const float* v_ro
     if (seq < 0 || seq >= batch_ || layer < 0 || layer >= L_ || n_new < 0) return fail(HM_ERR_INVALID, "kv_append: index out of range");
     if (len_[seq] + n_new > max_seq_)
         return fail(HM_ERR_KV_FULL, "KV cache full (" + std::to_string(len_[seq]) + " + " + std::to_string(n_new) + " > " + std::to_string(max_seq_) + ")");
-    if (spec_.listed() && n_new > 0) return fail(HM_ERR_UNSUPPORTED, "kv_append: this design caches latents, not keys and values");
+    if (spec_.listed() && (k_rows || v_rows)) return fail(HM_ERR_UNSUPPORTED, "kv_append: this design caches latents, not keys and values");
     {
         const int prc = ensure_pages({{seq, (long)len_[seq] + n_new}});
         if (prc) return prc;

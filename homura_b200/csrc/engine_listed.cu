@@ -387,11 +387,13 @@ int Engine::enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int
         const size_t per = (size_t)M * s.heads;
         const int most = (int)std::min<size_t>(std::min(lat_acc_floats_ / (per * s.kv_rank), lat_ml_floats_ / (per * 2)), 256);
         // tiles: every run is cut at the multiples of the rows that share a CTA
-        const int rpt = latent_rows_per_tile(M, s.heads, s.kv_rank, kv_bf16_);
-        int tiles = pass_runs_.empty() || rpt == 1 ? M : 0;
-        if (tiles == 0)
-            for (auto& r : pass_runs_) tiles += (r.first + r.second - 1) / rpt - r.first / rpt + 1;
-        a.tiles = rpt == 1 ? 0 : tiles;
+        int longest_run = 1, tiles = 0;
+        for (auto& r : pass_runs_) longest_run = std::max(longest_run, r.second);
+        a.rows_per_tile = latent_rows_per_tile(longest_run, s.heads, s.kv_rank, kv_bf16_);
+        for (auto& r : pass_runs_) tiles += (r.first + r.second - 1) / a.rows_per_tile - r.first / a.rows_per_tile + 1;
+        if (a.rows_per_tile == 1) tiles = M;
+        a.tiles = tiles;
+        a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
         a.nsplit = latent_pick_nsplit(tiles, s.heads, s.kv_rank, kv_bf16_, pass_longest_, sm_count_, most);
         a.part_acc = lat_acc_;
         a.part_ml = lat_ml_;

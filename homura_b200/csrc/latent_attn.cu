@@ -192,8 +192,8 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnArgs 
 }
 
 // ---- tensor cores -----------------------------------------------------------------------------
-constexpr int TCL_THREADS = 192, TCL_TOK = 128, TCL_TERMS = 3, TCL_SLICE = 2 * TCL_TOK * 128;  // a slice: 128 elements of 128 tokens, two K-major halves of 16 KB
-constexpr int TCL_MAXSTG = 8, TCL_MAXPAIRS = 64;
+constexpr int TCL_THREADS = 192, TCL_TERMS = 3;
+constexpr int TCL_MAXSTG = 12, TCL_MAXPAIRS = 64;
 constexpr float TCL_SLACK = 8.f;  // base-2 exponent by which a score may exceed the reference maximum
 
 // Shared-memory operand descriptors, 128-byte swizzle, version 1.  K-major: groups of 8 rows 1024 B apart.  MN-major: pieces of
@@ -201,8 +201,8 @@ constexpr float TCL_SLACK = 8.f;  // base-2 exponent by which a score may exceed
 __device__ __forceinline__ uint64_t desc_sw128(uint32_t addr, uint32_t lbo) {
     return (uint64_t)((addr >> 4) & 0x3FFF) | ((uint64_t)(lbo >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | ((uint64_t)1 << 46) | ((uint64_t)2 << 61);
 }
-// f32 accumulator, bf16 operands, M = 128; A transposed (MN-major) on request
-__device__ __forceinline__ uint32_t idesc_bf16(int n, int a_mn) { return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)a_mn << 15) | ((uint32_t)(n >> 3) << 17) | (8u << 24); }
+// f32 accumulator, bf16 operands; A transposed (MN-major) on request
+__device__ __forceinline__ uint32_t idesc_bf16(int m, int n, int a_mn) { return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)a_mn << 15) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24); }
 __device__ __forceinline__ void mma_bf16(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
     asm volatile("{ .reg .pred p; setp.ne.b32 p, %4, 0;\n"
                  "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p; }" ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate) : "memory");
@@ -230,14 +230,8 @@ __device__ __forceinline__ bool wbar_or(bool v) {
     asm volatile("{ .reg .pred p, q; setp.ne.u32 p, %1, 0; bar.red.or.pred q, 1, 128, p; selp.u32 %0, 1, 0, q; }" : "=r"(r) : "r"((uint32_t)v) : "memory");
     return r != 0;
 }
-__device__ __forceinline__ void split3(float x, uint16_t& h, uint16_t& m, uint16_t& l) {
-    h = f32_to_bf16_rne(x);
-    const float r = x - bf16_bits_to_f32(h);
-    m = f32_to_bf16_rne(r);
-    l = f32_to_bf16_rne(r - bf16_bits_to_f32(m));
-}
-
 struct TclGeom {
+    int tok;       // tokens per tile: 128, or 64 for latents so wide that two tiles of 128 do not fit the ring
     int np;        // pairs, padded to 16
     int n;         // MMA N = 3 * np
     int nb;        // 128-element slices of a latent
@@ -247,19 +241,21 @@ struct TclGeom {
     int cols;      // TMEM columns, a power of two
     int q_bytes, p_bytes, s_bytes;
     size_t smem;
+    __host__ __device__ int slice() const { return 2 * tok * 128; }  // bytes of 128 elements of a tile's tokens: two K-major halves
 };
 
-bool tcl_geom(int rank, int pairs, TclGeom* g) {
+bool tcl_geom_tok(int tok, int rank, int pairs, TclGeom* g) {
+    g->tok = tok;
     g->np = (pairs + 15) / 16 * 16;
     if (g->np < 16 || g->np > TCL_MAXPAIRS) return false;
     g->n = TCL_TERMS * g->np;
     g->kbs = latent_rank_pad(rank) / 64;
     g->nb = (g->kbs + 1) / 2;
     g->q_bytes = g->kbs * g->n * 128;
-    g->p_bytes = 2 * g->n * 128;
-    g->s_bytes = g->np * (TCL_TOK + 4) * 4;
-    const int room = 224 * 1024 - (g->q_bytes + g->p_bytes + g->s_bytes + 1024);
-    g->stages = room / TCL_SLICE;
+    g->p_bytes = tok / 64 * g->n * 128;
+    g->s_bytes = g->np * (tok + 4 + 32) * 4;
+    const int fixed = g->q_bytes + g->p_bytes + g->s_bytes + 1024;
+    g->stages = (222 * 1024 - fixed) / g->slice();
     if (g->stages > TCL_MAXSTG) g->stages = TCL_MAXSTG;
     if (g->stages < (g->nb > 2 ? g->nb : 2)) return false;  // the values of a tile are needed after its scores: the ring holds a whole tile
     g->look = g->stages >= 2 * g->nb && (g->nb + 2) * g->n <= 512 ? 1 : 0;
@@ -267,8 +263,16 @@ bool tcl_geom(int rank, int pairs, TclGeom* g) {
     if (need > 512) return false;
     g->cols = 32;
     while (g->cols < need) g->cols *= 2;
-    g->smem = (size_t)g->q_bytes + g->p_bytes + g->s_bytes + (size_t)g->stages * TCL_SLICE + 1024;
+    // two CTAs per SM where their tensor memory and a ring of two tiles and a slice allow it
+    const int pair = (112 * 1024 - fixed) / g->slice();
+    if (g->look && g->cols <= 256 && pair >= 2 * g->nb) g->stages = pair < TCL_MAXSTG ? pair : TCL_MAXSTG;
+    g->smem = (size_t)fixed + (size_t)g->stages * g->slice();
     return true;
+}
+bool tcl_geom(int rank, int pairs, TclGeom* g) {
+    if (tcl_geom_tok(128, rank, pairs, g) && g->look) return true;
+    if (tcl_geom_tok(64, rank, pairs, g) && g->look) return true;
+    return tcl_geom_tok(128, rank, pairs, g) || tcl_geom_tok(64, rank, pairs, g);
 }
 
 struct TclShared {
@@ -277,36 +281,41 @@ struct TclShared {
     volatile int abort_flag;
     float ref[TCL_MAXPAIRS], sum[TCL_MAXPAIRS], alpha[TCL_MAXPAIRS];
     int pos[TCL_MAXPAIRS];  // last visible position of the pair's row; -1: padding
+    int row[TCL_MAXPAIRS], head[TCL_MAXPAIRS];
 };
 
-__global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const LatentAttnArgs a, const TclGeom g, int heads_per_cta) {
+template <int TOK>
+__global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const LatentAttnArgs a, const TclGeom g, int heads_per_cta) {
     extern __shared__ __align__(1024) unsigned char tcl_smem[];
     __shared__ TclShared sh;
+    constexpr int SLICE = 2 * TOK * 128, PAGES = TOK / LATENT_PAGE, SLD = TOK + 4, TPL = TOK / 32;  // bytes, pages per tile, score row, tokens per lane
     unsigned char* ring = tcl_smem + ((1024u - (s32(tcl_smem) & 1023u)) & 1023u);
-    unsigned char* qs = ring + (size_t)g.stages * TCL_SLICE;  // [kbs][n][128 B]
-    unsigned char* pb = qs + g.q_bytes;                       // [2][n][128 B]
-    float* sc = reinterpret_cast<float*>(pb + g.p_bytes);     // [np][132]
-    constexpr int SLD = TCL_TOK + 4;
+    unsigned char* qs = ring + (size_t)g.stages * SLICE;   // [kbs][n][128 B]
+    unsigned char* pb = qs + g.q_bytes;                    // [TOK / 64][n][128 B]
+    float* sc = reinterpret_cast<float*>(pb + g.p_bytes);  // [np][SLD]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h0 = blockIdx.y * heads_per_cta, split = blockIdx.z;
     const int nh = min(heads_per_cta, a.heads - h0), R = a.pool.rank;
     // The pass's rows cut into tiles: a tile starts at every multiple of rows_per_tile and wherever a run starts.  Every warp
     // finds this CTA's tile, the blockIdx.x-th, on its own (the rows of a pass never change within it).
-    uint64_t starts = 0;
-    for (int i = 0; i < a.M; i += 32) {
-        const int m = i + lane;
-        const bool st = m < a.M && (m % a.rows_per_tile == 0 || a.row_seq[m - 1] != a.row_seq[m] || a.row_pos[m - 1] + 1 != a.row_pos[m]);
-        starts |= (uint64_t)__ballot_sync(0xffffffffu, st) << i;
+    int m0 = blockIdx.x, rows = 1;
+    if (a.rows_per_tile > 1) {
+        uint64_t starts = 0;
+        for (int i = 0; i < a.M; i += 32) {
+            const int m = i + lane;
+            const bool st = m < a.M && (m % a.rows_per_tile == 0 || a.row_seq[m - 1] != a.row_seq[m] || a.row_pos[m - 1] + 1 != a.row_pos[m]);
+            starts |= (uint64_t)__ballot_sync(0xffffffffu, st) << i;
+        }
+        if (a.M < 64) starts |= (uint64_t)1 << a.M;  // end mark
+        for (int i = 0; i < (int)blockIdx.x && starts; ++i) starts &= starts - 1;
+        m0 = starts ? __ffsll((long long)starts) - 1 : a.M;
+        if (m0 >= a.M) return;  // fewer tiles than CTAs
+        const uint64_t after = starts & (starts - 1);
+        rows = (after ? __ffsll((long long)after) - 1 : a.M) - m0;
     }
-    if (a.M < 64) starts |= (uint64_t)1 << a.M;  // end mark
-    for (int i = 0; i < (int)blockIdx.x && starts; ++i) starts &= starts - 1;
-    const int m0 = starts ? __ffsll((long long)starts) - 1 : a.M;
-    if (m0 >= a.M) return;  // fewer tiles than CTAs
-    const uint64_t after = starts & (starts - 1);
-    const int rows = (after ? __ffsll((long long)after) - 1 : a.M) - m0;
     const int seq = a.row_seq[m0], pos0 = a.row_pos[m0];
     const int pairs = rows * nh;  // pair p: row p / nh, head p % nh
-    const int len = pos0 + rows, tiles = (len + TCL_TOK - 1) / TCL_TOK, per = (tiles + a.nsplit - 1) / a.nsplit;
+    const int len = pos0 + rows, tiles = (len + TOK - 1) / TOK, per = (tiles + a.nsplit - 1) / a.nsplit;
     const int t0 = split * per, nt = min(tiles, t0 + per) - t0;
     if (nt <= 0) {  // only with nsplit > 1
         pdl_launch_dependents();
@@ -333,8 +342,9 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
     }
     for (int p = tid; p < g.np; p += TCL_THREADS) {
         sh.pos[p] = p < pairs ? pos0 + p / nh : -1;
+        sh.row[p] = m0 + p / nh;
+        sh.head[p] = h0 + p % nh;
         sh.ref[p] = -INFINITY;
-        sh.sum[p] = 0.f;
     }
     __syncthreads();
     if (warp == 1) {
@@ -346,42 +356,48 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
     tc_fence_after();
     const uint32_t tmem = sh.tmem, tmem_o = tmem + (uint32_t)((1 + g.look) * g.n);
     pdl_launch_dependents();
-    pdl_wait();
 
     if (warp == 0) {
         if (lane == 0) {
             const int32_t* table = a.pool.page_table + (size_t)seq * a.pool.max_pages;
             const int npages = (len + LATENT_PAGE - 1) / LATENT_PAGE;
-            const uint32_t piece = LATENT_PAGE * 128;
+            const int settled = a.early ? pos0 / LATENT_PAGE : 0;  // pages in front of the one that gets this step's latent
+            constexpr uint32_t piece = LATENT_PAGE * 128;
             const unsigned char* pool = reinterpret_cast<const unsigned char*>(a.pool.pages);
-            // a tile's second page may lie behind the context: its first page stands in (masked, but finite)
-            auto page_of = [&](int t, int i) { return table[min(2 * t + i, npages - 1)]; };
-            int pg0 = page_of(t0, 0), pg1 = page_of(t0, 1);
+            // a tile's last page may lie behind the context: the last one of the context stands in (masked, but finite)
+            auto page_of = [&](int t, int i) { return table[min(PAGES * t + i, npages - 1)]; };
+            int next[PAGES];
+#pragma unroll
+            for (int i = 0; i < PAGES; ++i) next[i] = page_of(t0, i);
             int it = 0;
-            bool ok = true;
+            bool ok = true, waited = false;
             for (int t = 0; t < nt && ok; ++t) {
-                const int c0 = pg0, c1 = pg1;
-                if (t + 1 < nt) {
-                    pg0 = page_of(t0 + t + 1, 0);
-                    pg1 = page_of(t0 + t + 1, 1);
+                int cur[PAGES];
+#pragma unroll
+                for (int i = 0; i < PAGES; ++i) cur[i] = next[i];
+                if (t + 1 < nt)
+#pragma unroll
+                    for (int i = 0; i < PAGES; ++i) next[i] = page_of(t0 + t + 1, i);
+                if (!waited && PAGES * (t0 + t + 1) > settled) {
+                    pdl_wait();
+                    waited = true;
                 }
                 for (int b = 0; b < g.nb; ++b, ++it) {
                     const int s = it % g.stages;
                     if (it >= g.stages && !mb_wait(&sh.empty[s], ((it / g.stages) & 1) ^ 1, a.err_flag, &sh.abort_flag)) { ok = false; break; }
                     const int halves = min(2, g.kbs - 2 * b);
-                    mb_expect_tx(&sh.full[s], (uint32_t)halves * 2 * piece);
-                    for (int hf = 0; hf < halves; ++hf) {
-                        unsigned char* dst = ring + (size_t)s * TCL_SLICE + hf * (TCL_SLICE / 2);
-                        const size_t kb = (size_t)(2 * b + hf);
-                        bulk_copy(dst, pool + ((size_t)c0 * g.kbs + kb) * piece, piece, &sh.full[s]);
-                        bulk_copy(dst + piece, pool + ((size_t)c1 * g.kbs + kb) * piece, piece, &sh.full[s]);
-                    }
+                    mb_expect_tx(&sh.full[s], (uint32_t)halves * PAGES * piece);
+                    for (int hf = 0; hf < halves; ++hf)
+#pragma unroll
+                        for (int i = 0; i < PAGES; ++i)
+                            bulk_copy(ring + (size_t)s * SLICE + hf * (SLICE / 2) + i * piece, pool + ((size_t)cur[i] * g.kbs + 2 * b + hf) * piece, piece, &sh.full[s]);
                 }
             }
+            if (!waited) pdl_wait();
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            const uint32_t id_s = idesc_bf16(g.n, 0), id_o = idesc_bf16(g.n, 1);
+            const uint32_t id_s = idesc_bf16(TOK, g.n, 0), id_o = idesc_bf16(128, g.n, 1);
             const uint32_t q0 = s32(qs), p0 = s32(pb), r0 = s32(ring);
             bool ok = mb_wait(&sh.q_full, 0, a.err_flag, &sh.abort_flag);
             tc_fence_after();
@@ -395,7 +411,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
                     for (int hf = 0; hf < halves; ++hf)
 #pragma unroll
                         for (int ks = 0; ks < 4; ++ks)
-                            mma_bf16(d, desc_sw128(r0 + s * TCL_SLICE + hf * (TCL_SLICE / 2) + ks * 32, 16), desc_sw128(q0 + (2 * b + hf) * g.n * 128 + ks * 32, 16), id_s, (b | hf | ks) ? 1u : 0u);
+                            mma_bf16(d, desc_sw128(r0 + s * SLICE + hf * (SLICE / 2) + ks * 32, 16), desc_sw128(q0 + (2 * b + hf) * g.n * 128 + ks * 32, 16), id_s, (b | hf | ks) ? 1u : 0u);
                 }
                 mma_commit(&sh.s_full[t & 1]);
                 return true;
@@ -409,8 +425,8 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
                 for (int b = 0; b < g.nb; ++b) {
                     const int s = (t * g.nb + b) % g.stages;
 #pragma unroll
-                    for (int ks = 0; ks < 8; ++ks)
-                        mma_bf16(tmem_o + b * g.n, desc_sw128(r0 + s * TCL_SLICE + ks * 2048, TCL_SLICE / 2), desc_sw128(p0 + (ks >> 2) * g.n * 128 + (ks & 3) * 32, 16), id_o, (t | ks) ? 1u : 0u);
+                    for (int ks = 0; ks < TOK / 16; ++ks)
+                        mma_bf16(tmem_o + b * g.n, desc_sw128(r0 + s * SLICE + ks * 2048, SLICE / 2), desc_sw128(p0 + (ks >> 2) * g.n * 128 + (ks & 3) * 32, 16), id_o, (t | ks) ? 1u : 0u);
                     mma_commit(&sh.empty[s]);
                 }
                 mma_commit(&sh.pv_done);
@@ -420,20 +436,37 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
         const int wt = tid - 64, ww = wt >> 5;
         const int lane_base = (warp & 3) * 32;  // the quarter of the TMEM lanes this warp may touch
         const uint32_t lane_addr = (uint32_t)lane_base << 16;
-        // queries: f32 rows -> three bf16 terms, K-major rows term * np + pair, 16-byte pieces XOR-ed by row & 7
-        for (int i = wt; i < g.np * g.kbs * 8; i += 128) {
-            const int p = i / (g.kbs * 8), c = i % (g.kbs * 8), r = c * 8;
-            float v[8];
-            const float* src = a.q + (size_t)(m0 + p / nh) * a.ldq + (size_t)(h0 + p % nh) * R + r;
-            const bool vec = p < pairs && r + 8 <= R && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
-            if (vec) {
-                const float4 x = ld_cg_f32x4(src), y = ld_cg_f32x4(src + 4);
-                v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
-            } else {
+        // the token of a score accumulator's lane: M = 128 fills all lanes, M = 64 the first 16 of every quarter
+        const bool has_tok = TOK == 128 || lane < 16;
+        const int my_tok = TOK == 128 ? lane_base + lane : (warp & 3) * 16 + lane;
+        float* ls = sc + (size_t)g.np * SLD;  // [np][32]: every lane's share of the pairs' sums
+        for (int i = wt; i < g.np * 32; i += 128) ls[i] = 0.f;
+        pdl_wait();
+        // queries: f32 rows -> three bf16 terms, K-major rows term * np + pair, 16-byte pieces XOR-ed by row & 7; four pieces of a
+        // thread are requested before the first is used
+        const int pieces = g.kbs * 8, items = g.np * pieces;
+        const bool vec = ((R | a.ldq) & 3) == 0 && (reinterpret_cast<uintptr_t>(a.q) & 15) == 0;
+        for (int base = wt; base < items; base += 4 * 128) {
+            float v[4][8];
 #pragma unroll
-                for (int e = 0; e < 8; ++e) v[e] = p < pairs && r + e < R ? ld_cg_f32(src + e) : 0.f;
+            for (int u = 0; u < 4; ++u) {
+                const int i = base + u * 128, p = i / pieces, r = (i % pieces) * 8;
+                const bool ok = i < items && p < pairs;
+                const float* src = a.q + (ok ? (size_t)sh.row[p] * a.ldq + (size_t)sh.head[p] * R + r : 0);
+                if (vec) {
+                    const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+                    const float4 x = ok && r + 4 <= R ? ld_cg_f32x4(src) : z, y = ok && r + 8 <= R ? ld_cg_f32x4(src + 4) : z;
+                    v[u][0] = x.x; v[u][1] = x.y; v[u][2] = x.z; v[u][3] = x.w; v[u][4] = y.x; v[u][5] = y.y; v[u][6] = y.z; v[u][7] = y.w;
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) v[u][e] = ok && r + e < R ? ld_cg_f32(src + e) : 0.f;
+                }
             }
-            tc_xpack_store8(qs, g.np, p, r, v);  // the image layout of the projections' activations: [block][term][np][64]
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int i = base + u * 128;
+                if (i < items) tc_xpack_store8(qs, g.np, i / pieces, (i % pieces) * 8, v[u]);  // the image layout of the projections' activations: [block][term][np][64]
+            }
         }
         fence_async_smem();
         mb_arrive(&sh.q_full);
@@ -441,7 +474,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
         bool bad = false;
         for (int t = 0; t < nt; ++t) {
             bad = !mb_wait(&sh.s_full[t & 1], (t >> 1) & 1, a.err_flag, &sh.abort_flag);
-            if (wbar_or(bad)) { bad = true; break; }
+            __syncwarp();
             tc_fence_after();
             const uint32_t s_addr = tmem + lane_addr + (g.look ? (uint32_t)((t & 1) * g.n) : 0u);
             for (int c0 = 0; c0 < g.np; c0 += 16) {
@@ -449,55 +482,100 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
 #pragma unroll
                 for (int k = 0; k < TCL_TERMS; ++k) tmem_ld16(s_addr + k * g.np + c0, r[k]);
                 tmem_ld_wait();
+                if (has_tok)
 #pragma unroll
-                for (int j = 0; j < 16; ++j) sc[(c0 + j) * SLD + lane_base + lane] = (__uint_as_float(r[2][j]) + __uint_as_float(r[1][j])) + __uint_as_float(r[0][j]);
+                    for (int j = 0; j < 16; ++j) sc[(c0 + j) * SLD + my_tok] = ((__uint_as_float(r[2][j]) + __uint_as_float(r[1][j])) + __uint_as_float(r[0][j])) * scale2;
+                __syncwarp();
             }
             tc_fence_before();
             // the weights of the tile in front must have been consumed before theirs are overwritten (and before O is rescaled)
-            bad = t > 0 && !mb_wait(&sh.pv_done, (t - 1) & 1, a.err_flag, &sh.abort_flag);
+            bad |= t > 0 && !mb_wait(&sh.pv_done, (t - 1) & 1, a.err_flag, &sh.abort_flag);
             if (wbar_or(bad)) { bad = true; break; }
             tc_fence_after();
-            const int tok = (t0 + t) * TCL_TOK + lane * 4;
+            const int tok = (t0 + t) * TOK + lane * TPL;
+            const bool whole = (t0 + t + 1) * TOK - 1 <= pos0;  // every row sees every token of the tile
             bool moved = false;
-            for (int p = ww; p < g.np; p += 4) {
-                const float4 s4 = *reinterpret_cast<const float4*>(sc + p * SLD + lane * 4);
-                const int last = sh.pos[p];
-                float s[4] = {s4.x, s4.y, s4.z, s4.w}, mx = -INFINITY;
+            for (int c0 = 0; c0 < g.np; c0 += 16) {
+                // four pairs per warp side by side
+                float s[4][TPL], ref[4];
+                bool grow = t == 0;
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    s[e] = tok + e <= last ? s[e] * scale2 : -INFINITY;
-                    mx = fmaxf(mx, s[e]);
-                }
-                mx = warp_max(mx);
-                float ref = sh.ref[p], al = 1.f;
-                if (mx > (t == 0 ? ref : ref + TCL_SLACK)) {
-                    al = t == 0 ? 1.f : exp2f(ref - mx);
-                    ref = mx;
-                }
-                float sum = 0.f;
-                uint16_t w[TCL_TERMS][4];
+                for (int j = 0; j < 4; ++j) {
+                    const int p = c0 + ww + 4 * j;
+                    if (TPL == 4) {
+                        const float4 v = *reinterpret_cast<const float4*>(sc + p * SLD + lane * 4);
+                        s[j][0] = v.x; s[j][1] = v.y; s[j][TPL - 2] = v.z; s[j][TPL - 1] = v.w;
+                    } else {
+                        const float2 v = *reinterpret_cast<const float2*>(sc + p * SLD + lane * 2);
+                        s[j][0] = v.x; s[j][1] = v.y;
+                    }
+                    ref[j] = sh.ref[p];
+                    if (!whole) {
+                        const int last = sh.pos[p];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const float v = s[e] == -INFINITY ? 0.f : exp2f(s[e] - ref);
-                    sum += v;
-                    split3(v, w[0][e], w[1][e], w[2][e]);
+                        for (int e = 0; e < TPL; ++e)
+                            if (tok + e > last) s[j][e] = -INFINITY;
+                    }
+#pragma unroll
+                    for (int e = 0; e < TPL; ++e) grow |= s[j][e] > ref[j] + TCL_SLACK;
                 }
-                sum = warp_sum(sum);
+                float al[4] = {1.f, 1.f, 1.f, 1.f};
+                const bool any = __any_sync(0xffffffffu, grow);
+                if (any) {
+                    float mx[4];
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        mx[j] = s[j][0];
+#pragma unroll
+                        for (int e = 1; e < TPL; ++e) mx[j] = fmaxf(mx[j], s[j][e]);
+                    }
+#pragma unroll
+                    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) mx[j] = fmaxf(mx[j], __shfl_xor_sync(0xffffffffu, mx[j], o));
+#pragma unroll
+                    for (int j = 0; j < 4; ++j)
+                        if (mx[j] > (t == 0 ? ref[j] : ref[j] + TCL_SLACK)) {
+                            if (t > 0) al[j] = exp2f(ref[j] - mx[j]);
+                            ref[j] = mx[j];
+                            moved |= t > 0;
+                        }
+                }
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const int p = c0 + ww + 4 * j;
+                    float w[TPL], sum = 0.f;
+#pragma unroll
+                    for (int e = 0; e < TPL; ++e) {
+                        w[e] = s[j][e] == -INFINITY ? 0.f : exp2f(s[j][e] - ref[j]);
+                        sum += w[e];
+                    }
+                    ls[p * 32 + lane] = ls[p * 32 + lane] * al[j] + sum;
+                    uint32_t q[TCL_TERMS][TPL / 2];
+#pragma unroll
+                    for (int e = 0; e < TPL / 2; ++e) bf16x2_split3(w[2 * e], w[2 * e + 1], q[0][e], q[1][e], q[2][e]);
+                    // this lane's tokens of row term * np + p: 64-token block, 16-byte piece XOR-ed by row & 7, place in the piece
+                    const int tk = lane * TPL;
+                    unsigned char* blk = pb + (size_t)(tk >> 6) * g.n * 128 + (tk & 7) * 2;
+#pragma unroll
+                    for (int k = 0; k < TCL_TERMS; ++k) {
+                        const int row = k * g.np + p;
+                        unsigned char* dst = blk + (size_t)row * 128 + ((((tk & 63) >> 3) ^ (row & 7)) << 4);
+                        if (TPL == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(q[k][0], q[k][TPL / 2 - 1]);
+                        else *reinterpret_cast<uint32_t*>(dst) = q[k][0];
+                    }
+                }
                 __syncwarp();
-                if (lane == 0) {
-                    sh.ref[p] = ref;
-                    sh.sum[p] = sh.sum[p] * al + sum;
-                    sh.alpha[p] = al;
-                }
-                moved |= al != 1.f;
-                // tokens lane*4 .. +3 of row term * np + p: block lane / 16, 16-byte piece (lane % 16) / 2, half of it
-                unsigned char* blk = pb + (size_t)(lane >> 4) * g.n * 128;
+                if (any && lane == 0)
 #pragma unroll
-                for (int k = 0; k < TCL_TERMS; ++k) {
-                    const int row = k * g.np + p;
-                    *reinterpret_cast<uint2*>(blk + (size_t)row * 128 + ((((lane & 15) >> 1) ^ (row & 7)) << 4) + (lane & 1) * 8) =
-                        make_uint2((uint32_t)w[k][0] | ((uint32_t)w[k][1] << 16), (uint32_t)w[k][2] | ((uint32_t)w[k][3] << 16));
-                }
+                    for (int j = 0; j < 4; ++j) {
+                        sh.ref[c0 + ww + 4 * j] = ref[j];
+                        sh.alpha[c0 + ww + 4 * j] = al[j];
+                    }
+                else if (lane == 0)
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) sh.alpha[c0 + ww + 4 * j] = 1.f;
+                __syncwarp();
             }
             if (wbar_or(moved)) {
                 for (int b = 0; b < g.nb; ++b)
@@ -516,12 +594,18 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
             fence_async_smem();
             mb_arrive(&sh.p_full);
         }
-        if (!bad) bad = !mb_wait(&sh.pv_done, (nt - 1) & 1, a.err_flag, &sh.abort_flag);
+        if (!bad) {
+            for (int p = ww; p < g.np; p += 4) {
+                const float sum = warp_sum(ls[p * 32 + lane]);
+                if (lane == 0) sh.sum[p] = a.nsplit == 1 ? 1.0f / sum : sum;
+            }
+            bad = !mb_wait(&sh.pv_done, (nt - 1) & 1, a.err_flag, &sh.abort_flag);
+        }
         if (!wbar_or(bad)) {
             tc_fence_after();
             if (a.nsplit > 1)
                 for (int p = wt; p < pairs; p += 128) {
-                    float* ml = a.part_ml + (((size_t)(m0 + p / nh) * a.heads + h0 + p % nh) * a.nsplit + split) * 2;
+                    float* ml = a.part_ml + (((size_t)sh.row[p] * a.heads + sh.head[p]) * a.nsplit + split) * 2;
                     ml[0] = sh.ref[p];
                     ml[1] = sh.sum[p];
                 }
@@ -537,9 +621,8 @@ __global__ void __launch_bounds__(TCL_THREADS, 1) latent_attn_tc_kernel(const La
                         const int p = c0 + j;
                         if (p < pairs && r0 < R) {
                             const float v = (__uint_as_float(r[2][j]) + __uint_as_float(r[1][j])) + __uint_as_float(r[0][j]);
-                            const int m = m0 + p / nh, h = h0 + p % nh;
-                            if (a.nsplit == 1) put_result(a, m, h, r0, v / sh.sum[p]);
-                            else a.part_acc[(((size_t)m * a.heads + h) * a.nsplit + split) * R + r0] = v;
+                            if (a.nsplit == 1) put_result(a, sh.row[p], sh.head[p], r0, v * sh.sum[p]);
+                            else a.part_acc[(((size_t)sh.row[p] * a.heads + sh.head[p]) * a.nsplit + split) * R + r0] = v;
                         }
                     }
                     __syncwarp();
@@ -585,10 +668,11 @@ int latent_tc_pairs(int rank, int bf16) {
     return 0;
 }
 
-int latent_rows_per_tile(int M, int heads, int rank, int bf16) {
+int latent_rows_per_tile(int longest_run, int heads, int rank, int bf16) {
     const int mp = latent_tc_pairs(rank, bf16);
-    if (mp == 0 || M < 2) return 1;
-    const int r = mp / tcl_heads(heads, mp);
+    if (mp == 0 || longest_run < 2) return 1;
+    int r = mp / tcl_heads(heads, mp);
+    if (r > longest_run) r = longest_run;
     return r < 1 ? 1 : r;
 }
 
@@ -596,10 +680,11 @@ int latent_pick_nsplit(int tiles, int heads, int rank, int bf16, int longest, in
     const int mp = latent_tc_pairs(rank, bf16);
     const int hg = mp ? (heads + tcl_heads(heads, mp) - 1) / tcl_heads(heads, mp) : (heads + CC_HEADS - 1) / CC_HEADS;
     const int ctas = tiles * hg;
-    const int tok = mp ? TCL_TOK : CC_TOK;
+    const int tok = mp ? 128 : CC_TOK;
     int s = sm_count / (ctas > 0 ? ctas : 1);
     const int most = (longest + tok - 1) / tok;
     if (s > most) s = most;
+    if (mp && most < 4) s = 1;  // the merge costs as much as three tiles
     if (s > max_split) s = max_split;
     if (s > 256) s = 256;
     return s < 1 ? 1 : s;
@@ -618,15 +703,16 @@ cudaError_t launch_latent_read(const LatentPool& pool, int seq, int len, float* 
 cudaError_t launch_latent_attn(const LatentAttnArgs& a_in, cudaStream_t st, bool pdl, int* launches) {
     LatentAttnArgs a = a_in;
     const int R = a.pool.rank, mp = latent_tc_pairs(R, a.pool.bf16);
-    if (R < 1 || a.M < 1 || (mp > 0 && a.M > 64) || a.tiles < 0 || a.tiles > a.M || a.heads < 1 || a.nsplit < 1 || a.nsplit > 256) return cudaErrorInvalidValue;
+    if (R < 1 || a.M < 1 || (mp > 0 && a.rows_per_tile > 1 && a.M > 64) || a.tiles < 0 || a.tiles > a.M || a.heads < 1 || a.nsplit < 1 || a.nsplit > 256) return cudaErrorInvalidValue;
     cudaError_t e;
     if (mp > 0) {
         const int hpc = tcl_heads(a.heads, mp);
-        a.rows_per_tile = latent_rows_per_tile(a.M, a.heads, R, a.pool.bf16);
         TclGeom g;
-        const int rows = a.rows_per_tile < a.M ? a.rows_per_tile : a.M;
-        if (!tcl_geom(R, rows * hpc, &g)) return cudaErrorInvalidValue;
-        e = launch(latent_attn_tc_kernel, dim3(a.tiles > 0 ? a.tiles : a.M, (a.heads + hpc - 1) / hpc, a.nsplit), dim3(TCL_THREADS), g.smem, st, pdl, a, g, hpc);
+        if (a.rows_per_tile < 1) a.rows_per_tile = 1;
+        if (a.rows_per_tile == 1) a.tiles = a.M;
+        if (!tcl_geom(R, a.rows_per_tile * hpc, &g)) return cudaErrorInvalidValue;
+        const dim3 grid(a.tiles > 0 ? a.tiles : a.M, (a.heads + hpc - 1) / hpc, a.nsplit);
+        e = g.tok == 128 ? launch(latent_attn_tc_kernel<128>, grid, dim3(TCL_THREADS), g.smem, st, pdl, a, g, hpc) : launch(latent_attn_tc_kernel<64>, grid, dim3(TCL_THREADS), g.smem, st, pdl, a, g, hpc);
     } else {
         const size_t smem = (size_t)(CC_HEADS + CC_TOK) * cc_stride(R) * 4;
         const dim3 grid(a.M, (a.heads + CC_HEADS - 1) / CC_HEADS, a.nsplit);

@@ -35,8 +35,9 @@ struct LatentAttnArgs {
     const int32_t* row_pos;  // a row sees positions <= its own
     const int32_t* row_seq;
     float scale;
-    int rows_per_tile;       // filled in by launch_latent_attn: rows of one run (consecutive positions of a sequence) that may share a CTA
-    int tiles;               // tensor-core kernel (at most 64 rows): tiles the rows fall into, 0: take every row for one
+    int rows_per_tile;       // latent_rows_per_tile: rows of one run (consecutive positions of a sequence) that may share a CTA
+    int tiles;               // with rows_per_tile > 1 (at most 64 rows then): tiles the rows fall into, 0: not known
+    int early;               // every row is its own sequence and the pages in front of its newest token were complete before the launch in front began
     int nsplit;
     float* part_acc;         // [M][heads][nsplit][rank], with nsplit > 1
     float* part_ml;          // [M][heads][nsplit][2]: running maximum (of base-2 exponents) and sum
@@ -55,8 +56,8 @@ cudaError_t launch_latent_read(const LatentPool& pool, int seq, int len, float* 
 
 // Largest (row, head) pair count a tensor-core CTA takes for this rank; 0: the kernel does not cover it (or the pages are f32).
 int latent_tc_pairs(int rank, int bf16);
-// Rows of a run that share a CTA.
-int latent_rows_per_tile(int M, int heads, int rank, int bf16);
+// Rows of a run that share a CTA, in a pass whose longest run has so many rows.
+int latent_rows_per_tile(int longest_run, int heads, int rank, int bf16);
 // Splits of the longest context (in tokens) so that a pass of so many tiles fills the SMs; at most max_split.
 int latent_pick_nsplit(int tiles, int heads, int rank, int bf16, int longest, int sm_count, int max_split);
 cudaError_t launch_latent_attn(const LatentAttnArgs& a, cudaStream_t st, bool pdl, int* launches);
