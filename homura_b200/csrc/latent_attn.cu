@@ -197,15 +197,15 @@ constexpr int TCL_MAXSTG = 12, TCL_MAXPAIRS = 64;
 constexpr float TCL_SLACK = 8.f;  // base-2 exponent by which a score may exceed the reference maximum
 
 // Shared-memory operand descriptors, 128-byte swizzle, version 1.  K-major: groups of 8 rows 1024 B apart.  MN-major: pieces of
-// 64 elements along MN `lbo` bytes apart, groups of 8 along K 1024 B apart.
-__device__ __forceinline__ uint64_t desc_sw128(uint32_t addr, uint32_t lbo) {
-    return (uint64_t)((addr >> 4) & 0x3FFF) | ((uint64_t)(lbo >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | ((uint64_t)1 << 46) | ((uint64_t)2 << 61);
-}
+// 64 elements along MN `lbo` bytes apart, groups of 8 along K 1024 B apart.  Only the lower word depends on the address: the
+// issuing thread steps through a tile by adding to it.
+__device__ __forceinline__ uint32_t desc_lo(uint32_t addr, uint32_t lbo) { return ((addr >> 4) & 0x3FFF) | ((lbo >> 4) << 16); }
+constexpr uint32_t DESC_HI = (1024u >> 4) | (1u << 14) | (2u << 29);
 // f32 accumulator, bf16 operands; A transposed (MN-major) on request
 __device__ __forceinline__ uint32_t idesc_bf16(int m, int n, int a_mn) { return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)a_mn << 15) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24); }
-__device__ __forceinline__ void mma_bf16(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
-    asm volatile("{ .reg .pred p; setp.ne.b32 p, %4, 0;\n"
-                 "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p; }" ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate) : "memory");
+__device__ __forceinline__ void mma_bf16(uint32_t d, uint32_t a_lo, uint32_t b_lo, uint32_t idesc, bool accumulate) {
+    asm volatile("{ .reg .pred p; .reg .b64 da, db; setp.ne.b32 p, %5, 0; mov.b64 da, {%1, %4}; mov.b64 db, {%2, %4};\n"
+                 "tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %3, p; }" ::"r"(d), "r"(a_lo), "r"(b_lo), "r"(idesc), "n"(DESC_HI), "r"((uint32_t)accumulate) : "memory");
 }
 __device__ __forceinline__ void mma_commit(uint64_t* bar) { asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(s32(bar)) : "memory"); }
 __device__ __forceinline__ void tmem_ld16(uint32_t addr, uint32_t (&r)[16]) {
@@ -369,7 +369,8 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
             int next[PAGES];
 #pragma unroll
             for (int i = 0; i < PAGES; ++i) next[i] = page_of(t0, i);
-            int it = 0;
+            int s = 0, it = 0;
+            uint32_t phase = 1;  // of the stage's empty barrier; its first round needs no wait
             bool ok = true, waited = false;
             for (int t = 0; t < nt && ok; ++t) {
                 int cur[PAGES];
@@ -383,14 +384,17 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                     waited = true;
                 }
                 for (int b = 0; b < g.nb; ++b, ++it) {
-                    const int s = it % g.stages;
-                    if (it >= g.stages && !mb_wait(&sh.empty[s], ((it / g.stages) & 1) ^ 1, a.err_flag, &sh.abort_flag)) { ok = false; break; }
+                    if (it >= g.stages && !mb_wait(&sh.empty[s], phase, a.err_flag, &sh.abort_flag)) { ok = false; break; }
                     const int halves = min(2, g.kbs - 2 * b);
                     mb_expect_tx(&sh.full[s], (uint32_t)halves * PAGES * piece);
                     for (int hf = 0; hf < halves; ++hf)
 #pragma unroll
                         for (int i = 0; i < PAGES; ++i)
                             bulk_copy(ring + (size_t)s * SLICE + hf * (SLICE / 2) + i * piece, pool + ((size_t)cur[i] * g.kbs + 2 * b + hf) * piece, piece, &sh.full[s]);
+                    if (++s == g.stages) {
+                        s = 0;
+                        phase ^= 1;
+                    }
                 }
             }
             if (!waited) pdl_wait();
@@ -398,20 +402,32 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
     } else if (warp == 1) {
         if (lane == 0) {
             const uint32_t id_s = idesc_bf16(TOK, g.n, 0), id_o = idesc_bf16(128, g.n, 1);
-            const uint32_t q0 = s32(qs), p0 = s32(pb), r0 = s32(ring);
+            const uint32_t qlo = desc_lo(s32(qs), 16), plo = desc_lo(s32(pb), 16), klo = desc_lo(s32(ring), 16), vlo = desc_lo(s32(ring), SLICE / 2);
+            const uint32_t row_block = (uint32_t)g.n * 128 / 16;  // one 64-element block of Q or P, in descriptor units
             bool ok = mb_wait(&sh.q_full, 0, a.err_flag, &sh.abort_flag);
             tc_fence_after();
+            int ks_stage = 0, pv_stage = 0;
+            uint32_t ks_phase = 0;
             auto scores = [&](int t) {
                 const uint32_t d = tmem + (g.look ? (uint32_t)((t & 1) * g.n) : 0u);
+                uint32_t q = qlo;
                 for (int b = 0; b < g.nb; ++b) {
-                    const int it = t * g.nb + b, s = it % g.stages;
-                    if (!mb_wait(&sh.full[s], (it / g.stages) & 1, a.err_flag, &sh.abort_flag)) return false;
+                    if (!mb_wait(&sh.full[ks_stage], ks_phase, a.err_flag, &sh.abort_flag)) return false;
                     tc_fence_after();
-                    const int halves = min(2, g.kbs - 2 * b);
-                    for (int hf = 0; hf < halves; ++hf)
+                    uint32_t k = klo + (uint32_t)ks_stage * (SLICE / 16);
 #pragma unroll
-                        for (int ks = 0; ks < 4; ++ks)
-                            mma_bf16(d, desc_sw128(r0 + s * SLICE + hf * (SLICE / 2) + ks * 32, 16), desc_sw128(q0 + (2 * b + hf) * g.n * 128 + ks * 32, 16), id_s, (b | hf | ks) ? 1u : 0u);
+                    for (int ks = 0; ks < 4; ++ks) mma_bf16(d, k + ks * 2, q + ks * 2, id_s, b > 0 || ks > 0);
+                    q += row_block;
+                    if (2 * b + 1 < g.kbs) {
+                        k += SLICE / 2 / 16;
+#pragma unroll
+                        for (int ks = 0; ks < 4; ++ks) mma_bf16(d, k + ks * 2, q + ks * 2, id_s, true);
+                        q += row_block;
+                    }
+                    if (++ks_stage == g.stages) {
+                        ks_stage = 0;
+                        ks_phase ^= 1;
+                    }
                 }
                 mma_commit(&sh.s_full[t & 1]);
                 return true;
@@ -422,12 +438,13 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                 else if (t + 1 < nt) ok = scores(t + 1);
                 if (!ok || !mb_wait(&sh.p_full, t & 1, a.err_flag, &sh.abort_flag)) break;
                 tc_fence_after();
-                for (int b = 0; b < g.nb; ++b) {
-                    const int s = (t * g.nb + b) % g.stages;
+                uint32_t d = tmem_o;
+                for (int b = 0; b < g.nb; ++b, d += g.n) {
+                    const uint32_t v = vlo + (uint32_t)pv_stage * (SLICE / 16);
 #pragma unroll
-                    for (int ks = 0; ks < TOK / 16; ++ks)
-                        mma_bf16(tmem_o + b * g.n, desc_sw128(r0 + s * SLICE + ks * 2048, SLICE / 2), desc_sw128(p0 + (ks >> 2) * g.n * 128 + (ks & 3) * 32, 16), id_o, (t | ks) ? 1u : 0u);
-                    mma_commit(&sh.empty[s]);
+                    for (int ks = 0; ks < TOK / 16; ++ks) mma_bf16(d, v + ks * 128, plo + (ks >> 2) * row_block + (ks & 3) * 2, id_o, t > 0 || ks > 0);
+                    mma_commit(&sh.empty[pv_stage]);
+                    if (++pv_stage == g.stages) pv_stage = 0;
                 }
                 mma_commit(&sh.pv_done);
             }
