@@ -160,7 +160,7 @@ int Engine::alloc_listed_scratch(int cap) {
         kmax = std::max(kmax, std::max(std::max(s.heads * s.vdim, s.ff), std::max(s.dim, s.kv_rank)));
         // splits times rows never exceed the SMs times the rows that share a CTA (latent_pick_nsplit)
         for (int bf16 = 0; bf16 < 2; ++bf16) {
-            const size_t rows = (size_t)sm_count_ * latent_rows_per_tile(TC_ROWS, s.heads, s.kv_rank, bf16);
+            const size_t rows = 2 * (size_t)sm_count_ * latent_rows_per_tile(TC_ROWS, s.heads, s.kv_rank, bf16);
             acc = std::max(acc, rows * s.heads * s.kv_rank);
             ml = std::max(ml, rows * s.heads * 2);
         }
@@ -394,7 +394,7 @@ int Engine::enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int
         if (a.rows_per_tile == 1) tiles = M;
         a.tiles = tiles;
         a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
-        a.nsplit = latent_pick_nsplit(tiles, s.heads, s.kv_rank, kv_bf16_, pass_longest_, sm_count_, most);
+        a.nsplit = latent_pick_nsplit(tiles, a.rows_per_tile, s.heads, s.kv_rank, kv_bf16_, pass_longest_, sm_count_, most);
         a.part_acc = lat_acc_;
         a.part_ml = lat_ml_;
         a.out = ctx_;

@@ -223,6 +223,11 @@ __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.
 __device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
 __device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
 __device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
+__device__ __forceinline__ uint32_t elect_lane() {
+    uint32_t p;
+    asm volatile("{ .reg .pred P; .reg .b32 r; elect.sync r|P, 0xffffffff; selp.u32 %0, 1, 0, P; }" : "=r"(p));
+    return p;
+}
 // barrier of the four weight warps with an OR over their predicates
 __device__ __forceinline__ bool wbar_or(bool v) {
     __syncwarp();
@@ -252,7 +257,7 @@ bool tcl_geom_tok(int tok, int rank, int pairs, TclGeom* g) {
     g->kbs = latent_rank_pad(rank) / 64;
     g->nb = (g->kbs + 1) / 2;
     g->q_bytes = g->kbs * g->n * 128;
-    g->p_bytes = tok / 64 * g->n * 128;
+    g->p_bytes = 2 * (tok / 64) * g->n * 128;  // the weights of two tiles
     g->s_bytes = g->np * (tok + 4 + 32) * 4;
     const int fixed = g->q_bytes + g->p_bytes + g->s_bytes + 1024;
     g->stages = (222 * 1024 - fixed) / g->slice();
@@ -276,7 +281,7 @@ bool tcl_geom(int rank, int pairs, TclGeom* g) {
 }
 
 struct TclShared {
-    uint64_t full[TCL_MAXSTG], empty[TCL_MAXSTG], s_full[2], p_full, pv_done, q_full;
+    uint64_t full[TCL_MAXSTG], empty[TCL_MAXSTG], s_full[2], p_full, pv_done[2], q_full;
     uint32_t tmem;
     volatile int abort_flag;
     float ref[TCL_MAXPAIRS], sum[TCL_MAXPAIRS], alpha[TCL_MAXPAIRS];
@@ -291,7 +296,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
     constexpr int SLICE = 2 * TOK * 128, PAGES = TOK / LATENT_PAGE, SLD = TOK + 4, TPL = TOK / 32;  // bytes, pages per tile, score row, tokens per lane
     unsigned char* ring = tcl_smem + ((1024u - (s32(tcl_smem) & 1023u)) & 1023u);
     unsigned char* qs = ring + (size_t)g.stages * SLICE;   // [kbs][n][128 B]
-    unsigned char* pb = qs + g.q_bytes;                    // [TOK / 64][n][128 B]
+    unsigned char* pb = qs + g.q_bytes;                    // [2][TOK / 64][n][128 B]
     float* sc = reinterpret_cast<float*>(pb + g.p_bytes);  // [np][SLD]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h0 = blockIdx.y * heads_per_cta, split = blockIdx.z;
@@ -335,7 +340,8 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
         mb_init(&sh.s_full[0], 1);
         mb_init(&sh.s_full[1], 1);
         mb_init(&sh.p_full, 128);
-        mb_init(&sh.pv_done, 1);
+        mb_init(&sh.pv_done[0], 1);
+        mb_init(&sh.pv_done[1], 1);
         mb_init(&sh.q_full, 128);
         sh.abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -400,53 +406,73 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
             if (!waited) pdl_wait();
         }
     } else if (warp == 1) {
-        if (lane == 0) {
-            const uint32_t id_s = idesc_bf16(TOK, g.n, 0), id_o = idesc_bf16(128, g.n, 1);
-            const uint32_t qlo = desc_lo(s32(qs), 16), plo = desc_lo(s32(pb), 16), klo = desc_lo(s32(ring), 16), vlo = desc_lo(s32(ring), SLICE / 2);
-            const uint32_t row_block = (uint32_t)g.n * 128 / 16;  // one 64-element block of Q or P, in descriptor units
-            bool ok = mb_wait(&sh.q_full, 0, a.err_flag, &sh.abort_flag);
-            tc_fence_after();
-            int ks_stage = 0, pv_stage = 0;
-            uint32_t ks_phase = 0;
-            auto scores = [&](int t) {
-                const uint32_t d = tmem + (g.look ? (uint32_t)((t & 1) * g.n) : 0u);
-                uint32_t q = qlo;
-                for (int b = 0; b < g.nb; ++b) {
-                    if (!mb_wait(&sh.full[ks_stage], ks_phase, a.err_flag, &sh.abort_flag)) return false;
+        // The whole warp runs this in step, so that the addresses and stage counters live in uniform registers; one elected lane
+        // issues (a lane that runs alone takes twice as long per MMA).
+        const uint32_t lead = elect_lane();
+        const uint32_t base = __shfl_sync(0xffffffffu, tmem, 0), base_o = base + (uint32_t)((1 + g.look) * g.n);
+        const uint32_t id_s = idesc_bf16(TOK, g.n, 0), id_o = idesc_bf16(128, g.n, 1);
+        const uint32_t qlo = desc_lo(s32(qs), 16), plo = desc_lo(s32(pb), 16), klo = desc_lo(s32(ring), 16), vlo = desc_lo(s32(ring), SLICE / 2);
+        const uint32_t row_block = (uint32_t)g.n * 128 / 16;  // one 64-element block of Q or P, in descriptor units
+        auto ready = [&](uint64_t* bar, uint32_t parity) { return __any_sync(0xffffffffu, mb_test(bar, parity)) != 0; };
+        bool ok = __any_sync(0xffffffffu, mb_wait(&sh.q_full, 0, a.err_flag, &sh.abort_flag)) != 0;
+        int ks_stage = 0, pv_stage = 0, ks_slice = 0, ks_tile = 0;
+        uint32_t ks_phase = 0, q = qlo;
+        for (int t = 0; t < nt && ok; ++t) {
+            // Whatever is ready first: a slice of this tile (of the next one too, with two score accumulators) or this tile's
+            // weights, whose product frees the ring for the tile after next.
+            const int upto = g.look ? min(nt, t + 2) : t + 1;
+            bool pv = false;
+            unsigned long long spins = 0;
+            while (!pv) {
+                if (ks_tile > t && ready(&sh.p_full, t & 1)) {
                     tc_fence_after();
-                    uint32_t k = klo + (uint32_t)ks_stage * (SLICE / 16);
+                    uint32_t d = base_o;
+                    const uint32_t p = plo + (uint32_t)(t & 1) * (TOK / 64) * row_block;
+                    for (int b = 0; b < g.nb; ++b, d += g.n) {
+                        const uint32_t v = vlo + (uint32_t)pv_stage * (SLICE / 16);
+                        if (lead) {
 #pragma unroll
-                    for (int ks = 0; ks < 4; ++ks) mma_bf16(d, k + ks * 2, q + ks * 2, id_s, b > 0 || ks > 0);
-                    q += row_block;
-                    if (2 * b + 1 < g.kbs) {
-                        k += SLICE / 2 / 16;
-#pragma unroll
-                        for (int ks = 0; ks < 4; ++ks) mma_bf16(d, k + ks * 2, q + ks * 2, id_s, true);
-                        q += row_block;
+                            for (int ks = 0; ks < TOK / 16; ++ks) mma_bf16(d, v + ks * 128, p + (ks >> 2) * row_block + (ks & 3) * 2, id_o, t > 0 || ks > 0);
+                            mma_commit(&sh.empty[pv_stage]);
+                        }
+                        __syncwarp();
+                        if (++pv_stage == g.stages) pv_stage = 0;
                     }
+                    if (lead) mma_commit(&sh.pv_done[t & 1]);
+                    __syncwarp();
+                    pv = true;
+                } else if (ks_tile < upto && ready(&sh.full[ks_stage], ks_phase)) {
+                    // scores of one slice; the last slice of a tile publishes the tile's scores
+                    tc_fence_after();
+                    const uint32_t d = base + (g.look ? (uint32_t)((ks_tile & 1) * g.n) : 0u), k = klo + (uint32_t)ks_stage * (SLICE / 16);
+                    const bool two = 2 * ks_slice + 1 < g.kbs;
+                    if (lead) {
+#pragma unroll
+                        for (int ks = 0; ks < 4; ++ks) mma_bf16(d, k + ks * 2, q + ks * 2, id_s, ks_slice > 0 || ks > 0);
+                        if (two)
+#pragma unroll
+                            for (int ks = 0; ks < 4; ++ks) mma_bf16(d, k + SLICE / 2 / 16 + ks * 2, q + row_block + ks * 2, id_s, true);
+                    }
+                    __syncwarp();
+                    q += two ? 2 * row_block : row_block;
                     if (++ks_stage == g.stages) {
                         ks_stage = 0;
                         ks_phase ^= 1;
                     }
+                    if (++ks_slice == g.nb) {
+                        if (lead) mma_commit(&sh.s_full[ks_tile & 1]);
+                        __syncwarp();
+                        ks_slice = 0;
+                        ++ks_tile;
+                        q = qlo;
+                    }
+                    spins = 0;
+                } else if (__any_sync(0xffffffffu, sh.abort_flag != 0) || ++spins > MB_SPIN_LIMIT) {
+                    if (lane == 0 && !sh.abort_flag && a.err_flag) atomicExch(a.err_flag, 2);
+                    sh.abort_flag = 1;
+                    ok = false;
+                    break;
                 }
-                mma_commit(&sh.s_full[t & 1]);
-                return true;
-            };
-            if (ok && g.look) ok = scores(0);
-            for (int t = 0; t < nt && ok; ++t) {
-                if (!g.look) ok = scores(t);
-                else if (t + 1 < nt) ok = scores(t + 1);
-                if (!ok || !mb_wait(&sh.p_full, t & 1, a.err_flag, &sh.abort_flag)) break;
-                tc_fence_after();
-                uint32_t d = tmem_o;
-                for (int b = 0; b < g.nb; ++b, d += g.n) {
-                    const uint32_t v = vlo + (uint32_t)pv_stage * (SLICE / 16);
-#pragma unroll
-                    for (int ks = 0; ks < TOK / 16; ++ks) mma_bf16(d, v + ks * 128, plo + (ks >> 2) * row_block + (ks & 3) * 2, id_o, t > 0 || ks > 0);
-                    mma_commit(&sh.empty[pv_stage]);
-                    if (++pv_stage == g.stages) pv_stage = 0;
-                }
-                mma_commit(&sh.pv_done);
             }
         }
     } else {
@@ -505,10 +531,10 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                 __syncwarp();
             }
             tc_fence_before();
-            // the weights of the tile in front must have been consumed before theirs are overwritten (and before O is rescaled)
-            bad |= t > 0 && !mb_wait(&sh.pv_done, (t - 1) & 1, a.err_flag, &sh.abort_flag);
+            // this tile's weights go where those of two tiles ago were: their product must be done
+            bad |= t > 1 && !mb_wait(&sh.pv_done[t & 1], ((t >> 1) - 1) & 1, a.err_flag, &sh.abort_flag);
             if (wbar_or(bad)) { bad = true; break; }
-            tc_fence_after();
+            unsigned char* pt = pb + (size_t)(t & 1) * (TOK / 64) * g.n * 128;
             const int tok = (t0 + t) * TOK + lane * TPL;
             const bool whole = (t0 + t + 1) * TOK - 1 <= pos0;  // every row sees every token of the tile
             bool moved = false;
@@ -573,7 +599,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                     for (int e = 0; e < TPL / 2; ++e) bf16x2_split3(w[2 * e], w[2 * e + 1], q[0][e], q[1][e], q[2][e]);
                     // this lane's tokens of row term * np + p: 64-token block, 16-byte piece XOR-ed by row & 7, place in the piece
                     const int tk = lane * TPL;
-                    unsigned char* blk = pb + (size_t)(tk >> 6) * g.n * 128 + (tk & 7) * 2;
+                    unsigned char* blk = pt + (size_t)(tk >> 6) * g.n * 128 + (tk & 7) * 2;
 #pragma unroll
                     for (int k = 0; k < TCL_TERMS; ++k) {
                         const int row = k * g.np + p;
@@ -595,6 +621,10 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                 __syncwarp();
             }
             if (wbar_or(moved)) {
+                // the accumulators are rescaled once the tile in front has been added
+                bad = !mb_wait(&sh.pv_done[(t - 1) & 1], ((t - 1) >> 1) & 1, a.err_flag, &sh.abort_flag);
+                if (wbar_or(bad)) { bad = true; break; }
+                tc_fence_after();
                 for (int b = 0; b < g.nb; ++b)
                     for (int c0 = 0; c0 < g.n; c0 += 16) {
                         uint32_t r[16];
@@ -616,7 +646,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                 const float sum = warp_sum(ls[p * 32 + lane]);
                 if (lane == 0) sh.sum[p] = a.nsplit == 1 ? 1.0f / sum : sum;
             }
-            bad = !mb_wait(&sh.pv_done, (nt - 1) & 1, a.err_flag, &sh.abort_flag);
+            bad = !mb_wait(&sh.pv_done[(nt - 1) & 1], ((nt - 1) >> 1) & 1, a.err_flag, &sh.abort_flag);
         }
         if (!wbar_or(bad)) {
             tc_fence_after();
@@ -693,17 +723,18 @@ int latent_rows_per_tile(int longest_run, int heads, int rank, int bf16) {
     return r < 1 ? 1 : r;
 }
 
-int latent_pick_nsplit(int tiles, int heads, int rank, int bf16, int longest, int sm_count, int max_split) {
+int latent_pick_nsplit(int tiles, int rows_per_tile, int heads, int rank, int bf16, int longest, int sm_count, int max_split) {
     const int mp = latent_tc_pairs(rank, bf16);
-    const int hg = mp ? (heads + tcl_heads(heads, mp) - 1) / tcl_heads(heads, mp) : (heads + CC_HEADS - 1) / CC_HEADS;
-    const int ctas = tiles * hg;
-    const int tok = mp ? 128 : CC_TOK;
-    int s = sm_count / (ctas > 0 ? ctas : 1);
-    const int most = (longest + tok - 1) / tok;
+    const int hpc = mp ? tcl_heads(heads, mp) : CC_HEADS, ctas = tiles * ((heads + hpc - 1) / hpc);
+    TclGeom g;
+    const bool tc = mp > 0 && tcl_geom(rank, rows_per_tile * hpc, &g);
+    const int tok = tc ? 128 : CC_TOK, most = (longest + tok - 1) / tok;
+    const int slots = tc && g.smem <= 112 * 1024 && g.cols <= 256 ? 2 * sm_count : sm_count;  // CTAs resident at once
+    int s = slots / (ctas > 0 ? ctas : 1);
     if (s > most) s = most;
-    if (mp && most < 4) s = 1;  // the merge costs as much as three tiles
     if (s > max_split) s = max_split;
     if (s > 256) s = 256;
+    if (tc && most < 4) s = 1;  // the merge costs as much as three tiles
     return s < 1 ? 1 : s;
 }
 

@@ -19,7 +19,13 @@ __device__ __forceinline__ bool mb_try(uint64_t* b, uint32_t parity) {
     asm volatile("{ .reg .pred p; mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2; selp.u32 %0, 1, 0, p; }" : "=r"(ok) : "r"(s32(b)), "r"(parity) : "memory");
     return ok != 0;
 }
-// The same poll with acquire semantics at cluster scope: for barriers completed by other CTAs' st.async stores.
+// A poll that returns at once (try_wait may suspend the thread for a while): for a thread that watches several barriers.
+__device__ __forceinline__ bool mb_test(uint64_t* b, uint32_t parity) {
+    uint32_t ok;
+    asm volatile("{ .reg .pred p; mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2; selp.u32 %0, 1, 0, p; }" : "=r"(ok) : "r"(s32(b)), "r"(parity) : "memory");
+    return ok != 0;
+}
+// mb_try with acquire semantics at cluster scope: for barriers completed by other CTAs' st.async stores.
 __device__ __forceinline__ bool mb_try_cluster(uint64_t* b, uint32_t parity) {
     uint32_t ok;
     asm volatile("{ .reg .pred p; mbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2; selp.u32 %0, 1, 0, p; }" : "=r"(ok) : "r"(s32(b)), "r"(parity) : "memory");
