@@ -12,7 +12,7 @@
 // The MMA's N holds the (row, head) pairs of the CTA three times: queries and weights stay f32 in effect, split into three
 // bf16 terms (exact to 2^-24), and the three column groups are added when an accumulator is read back.  Rows of a prompt
 // that follow one another share a CTA (each masks the tokens behind its own position); a decoded token is a tile of one row.
-// Warp 0 copies pages into a ring of 128-element slices, warp 1 issues the MMAs, warps 2-5 turn scores into weights.  The
+// Warp 0 copies pages into a ring of 128-element slices, warp 1 issues the MMAs, warps 2-9 turn scores into weights.  The
 // reference maximum of a pair moves only when a score exceeds it by more than 2^8 (the weights then still fit), so the
 // accumulators are almost never rescaled.
 #include "latent_attn.h"
@@ -192,7 +192,8 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnArgs 
 }
 
 // ---- tensor cores -----------------------------------------------------------------------------
-constexpr int TCL_THREADS = 192, TCL_TERMS = 3;
+constexpr int TCL_SWARPS = 8, TCL_STHREADS = 32 * TCL_SWARPS, TCL_THREADS = 64 + TCL_STHREADS, TCL_TERMS = 3;  // SWARPS: score warps, two per quarter of the tensor memory's lanes
+constexpr int TCL_PAIR_SMEM = 113 * 1024 - 2048;  // dynamic shared memory with which two CTAs share an SM (2 KB static and 1 KB of the system's each)
 constexpr int TCL_MAXSTG = 12, TCL_MAXPAIRS = 64;
 constexpr float TCL_SLACK = 8.f;  // base-2 exponent by which a score may exceed the reference maximum
 
@@ -213,6 +214,11 @@ __device__ __forceinline__ void tmem_ld16(uint32_t addr, uint32_t (&r)[16]) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
                  : "r"(addr));
 }
+__device__ __forceinline__ void tmem_ld8(uint32_t addr, uint32_t (&r)[8]) {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+                 : "r"(addr));
+}
 __device__ __forceinline__ void tmem_st16(uint32_t addr, const uint32_t (&r)[16]) {
     asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(addr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]),
                  "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
@@ -228,11 +234,11 @@ __device__ __forceinline__ uint32_t elect_lane() {
     asm volatile("{ .reg .pred P; .reg .b32 r; elect.sync r|P, 0xffffffff; selp.u32 %0, 1, 0, P; }" : "=r"(p));
     return p;
 }
-// barrier of the four weight warps with an OR over their predicates
+// barrier of the score warps with an OR over their predicates
 __device__ __forceinline__ bool wbar_or(bool v) {
     __syncwarp();
     uint32_t r;
-    asm volatile("{ .reg .pred p, q; setp.ne.u32 p, %1, 0; bar.red.or.pred q, 1, 128, p; selp.u32 %0, 1, 0, q; }" : "=r"(r) : "r"((uint32_t)v) : "memory");
+    asm volatile("{ .reg .pred p, q; setp.ne.u32 p, %1, 0; bar.red.or.pred q, 1, 256, p; selp.u32 %0, 1, 0, q; }" : "=r"(r) : "r"((uint32_t)v) : "memory");
     return r != 0;
 }
 struct TclGeom {
@@ -258,7 +264,7 @@ bool tcl_geom_tok(int tok, int rank, int pairs, TclGeom* g) {
     g->nb = (g->kbs + 1) / 2;
     g->q_bytes = g->kbs * g->n * 128;
     g->p_bytes = 2 * (tok / 64) * g->n * 128;  // the weights of two tiles
-    g->s_bytes = g->np * (tok + 4 + 32) * 4;
+    g->s_bytes = g->np * (tok + 32) * 4;  // scores, and every lane's share of the sums
     const int fixed = g->q_bytes + g->p_bytes + g->s_bytes + 1024;
     g->stages = (222 * 1024 - fixed) / g->slice();
     if (g->stages > TCL_MAXSTG) g->stages = TCL_MAXSTG;
@@ -269,7 +275,7 @@ bool tcl_geom_tok(int tok, int rank, int pairs, TclGeom* g) {
     g->cols = 32;
     while (g->cols < need) g->cols *= 2;
     // two CTAs per SM where their tensor memory and a ring of two tiles and a slice allow it
-    const int pair = (112 * 1024 - fixed) / g->slice();
+    const int pair = (TCL_PAIR_SMEM - fixed) / g->slice();
     if (g->look && g->cols <= 256 && pair >= 2 * g->nb) g->stages = pair < TCL_MAXSTG ? pair : TCL_MAXSTG;
     g->smem = (size_t)fixed + (size_t)g->stages * g->slice();
     return true;
@@ -293,7 +299,7 @@ template <int TOK>
 __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const LatentAttnArgs a, const TclGeom g, int heads_per_cta) {
     extern __shared__ __align__(1024) unsigned char tcl_smem[];
     __shared__ TclShared sh;
-    constexpr int SLICE = 2 * TOK * 128, PAGES = TOK / LATENT_PAGE, SLD = TOK + 4, TPL = TOK / 32;  // bytes, pages per tile, score row, tokens per lane
+    constexpr int SLICE = 2 * TOK * 128, PAGES = TOK / LATENT_PAGE, SLD = TOK, TPL = TOK / 32;  // bytes, pages per tile, score row, tokens per lane
     unsigned char* ring = tcl_smem + ((1024u - (s32(tcl_smem) & 1023u)) & 1023u);
     unsigned char* qs = ring + (size_t)g.stages * SLICE;   // [kbs][n][128 B]
     unsigned char* pb = qs + g.q_bytes;                    // [2][TOK / 64][n][128 B]
@@ -339,10 +345,10 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
         }
         mb_init(&sh.s_full[0], 1);
         mb_init(&sh.s_full[1], 1);
-        mb_init(&sh.p_full, 128);
+        mb_init(&sh.p_full, TCL_STHREADS);
         mb_init(&sh.pv_done[0], 1);
         mb_init(&sh.pv_done[1], 1);
-        mb_init(&sh.q_full, 128);
+        mb_init(&sh.q_full, TCL_STHREADS);
         sh.abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -476,24 +482,24 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
             }
         }
     } else {
-        const int wt = tid - 64, ww = wt >> 5;
+        const int wt = tid - 64, ww = wt >> 5, half = ww >> 2;  // half: which eight of every 16 accumulator columns this warp reads
         const int lane_base = (warp & 3) * 32;  // the quarter of the TMEM lanes this warp may touch
         const uint32_t lane_addr = (uint32_t)lane_base << 16;
         // the token of a score accumulator's lane: M = 128 fills all lanes, M = 64 the first 16 of every quarter
         const bool has_tok = TOK == 128 || lane < 16;
         const int my_tok = TOK == 128 ? lane_base + lane : (warp & 3) * 16 + lane;
         float* ls = sc + (size_t)g.np * SLD;  // [np][32]: every lane's share of the pairs' sums
-        for (int i = wt; i < g.np * 32; i += 128) ls[i] = 0.f;
+        for (int i = wt; i < g.np * 32; i += TCL_STHREADS) ls[i] = 0.f;
         pdl_wait();
         // queries: f32 rows -> three bf16 terms, K-major rows term * np + pair, 16-byte pieces XOR-ed by row & 7; four pieces of a
         // thread are requested before the first is used
         const int pieces = g.kbs * 8, items = g.np * pieces;
         const bool vec = ((R | a.ldq) & 3) == 0 && (reinterpret_cast<uintptr_t>(a.q) & 15) == 0;
-        for (int base = wt; base < items; base += 4 * 128) {
+        for (int base = wt; base < items; base += 4 * TCL_STHREADS) {
             float v[4][8];
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-                const int i = base + u * 128, p = i / pieces, r = (i % pieces) * 8;
+                const int i = base + u * TCL_STHREADS, p = i / pieces, r = (i % pieces) * 8;
                 const bool ok = i < items && p < pairs;
                 const float* src = a.q + (ok ? (size_t)sh.row[p] * a.ldq + (size_t)sh.head[p] * R + r : 0);
                 if (vec) {
@@ -507,7 +513,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
             }
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-                const int i = base + u * 128;
+                const int i = base + u * TCL_STHREADS;
                 if (i < items) tc_xpack_store8(qs, g.np, i / pieces, (i % pieces) * 8, v[u]);  // the image layout of the projections' activations: [block][term][np][64]
             }
         }
@@ -520,14 +526,14 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
             __syncwarp();
             tc_fence_after();
             const uint32_t s_addr = tmem + lane_addr + (g.look ? (uint32_t)((t & 1) * g.n) : 0u);
-            for (int c0 = 0; c0 < g.np; c0 += 16) {
-                uint32_t r[TCL_TERMS][16];
+            for (int c0 = half * 8; c0 < g.np; c0 += 16) {
+                uint32_t r[TCL_TERMS][8];
 #pragma unroll
-                for (int k = 0; k < TCL_TERMS; ++k) tmem_ld16(s_addr + k * g.np + c0, r[k]);
+                for (int k = 0; k < TCL_TERMS; ++k) tmem_ld8(s_addr + k * g.np + c0, r[k]);
                 tmem_ld_wait();
                 if (has_tok)
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) sc[(c0 + j) * SLD + my_tok] = ((__uint_as_float(r[2][j]) + __uint_as_float(r[1][j])) + __uint_as_float(r[0][j])) * scale2;
+                    for (int j = 0; j < 8; ++j) sc[(c0 + j) * SLD + my_tok] = ((__uint_as_float(r[2][j]) + __uint_as_float(r[1][j])) + __uint_as_float(r[0][j])) * scale2;
                 __syncwarp();
             }
             tc_fence_before();
@@ -539,12 +545,12 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
             const bool whole = (t0 + t + 1) * TOK - 1 <= pos0;  // every row sees every token of the tile
             bool moved = false;
             for (int c0 = 0; c0 < g.np; c0 += 16) {
-                // four pairs per warp side by side
-                float s[4][TPL], ref[4];
+                // two pairs per warp side by side
+                float s[2][TPL], ref[2];
                 bool grow = t == 0;
 #pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    const int p = c0 + ww + 4 * j;
+                for (int j = 0; j < 2; ++j) {
+                    const int p = c0 + ww + 8 * j;
                     if (TPL == 4) {
                         const float4 v = *reinterpret_cast<const float4*>(sc + p * SLD + lane * 4);
                         s[j][0] = v.x; s[j][1] = v.y; s[j][TPL - 2] = v.z; s[j][TPL - 1] = v.w;
@@ -562,12 +568,12 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
 #pragma unroll
                     for (int e = 0; e < TPL; ++e) grow |= s[j][e] > ref[j] + TCL_SLACK;
                 }
-                float al[4] = {1.f, 1.f, 1.f, 1.f};
+                float al[2] = {1.f, 1.f};
                 const bool any = __any_sync(0xffffffffu, grow);
                 if (any) {
-                    float mx[4];
+                    float mx[2];
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) {
+                    for (int j = 0; j < 2; ++j) {
                         mx[j] = s[j][0];
 #pragma unroll
                         for (int e = 1; e < TPL; ++e) mx[j] = fmaxf(mx[j], s[j][e]);
@@ -575,9 +581,9 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
 #pragma unroll
                     for (int o = 16; o > 0; o >>= 1)
 #pragma unroll
-                        for (int j = 0; j < 4; ++j) mx[j] = fmaxf(mx[j], __shfl_xor_sync(0xffffffffu, mx[j], o));
+                        for (int j = 0; j < 2; ++j) mx[j] = fmaxf(mx[j], __shfl_xor_sync(0xffffffffu, mx[j], o));
 #pragma unroll
-                    for (int j = 0; j < 4; ++j)
+                    for (int j = 0; j < 2; ++j)
                         if (mx[j] > (t == 0 ? ref[j] : ref[j] + TCL_SLACK)) {
                             if (t > 0) al[j] = exp2f(ref[j] - mx[j]);
                             ref[j] = mx[j];
@@ -585,8 +591,8 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                         }
                 }
 #pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    const int p = c0 + ww + 4 * j;
+                for (int j = 0; j < 2; ++j) {
+                    const int p = c0 + ww + 8 * j;
                     float w[TPL], sum = 0.f;
 #pragma unroll
                     for (int e = 0; e < TPL; ++e) {
@@ -611,13 +617,13 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                 __syncwarp();
                 if (any && lane == 0)
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) {
-                        sh.ref[c0 + ww + 4 * j] = ref[j];
-                        sh.alpha[c0 + ww + 4 * j] = al[j];
+                    for (int j = 0; j < 2; ++j) {
+                        sh.ref[c0 + ww + 8 * j] = ref[j];
+                        sh.alpha[c0 + ww + 8 * j] = al[j];
                     }
                 else if (lane == 0)
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) sh.alpha[c0 + ww + 4 * j] = 1.f;
+                    for (int j = 0; j < 2; ++j) sh.alpha[c0 + ww + 8 * j] = 1.f;
                 __syncwarp();
             }
             if (wbar_or(moved)) {
@@ -625,7 +631,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                 bad = !mb_wait(&sh.pv_done[(t - 1) & 1], ((t - 1) >> 1) & 1, a.err_flag, &sh.abort_flag);
                 if (wbar_or(bad)) { bad = true; break; }
                 tc_fence_after();
-                for (int b = 0; b < g.nb; ++b)
+                for (int b = half; b < g.nb; b += 2)
                     for (int c0 = 0; c0 < g.n; c0 += 16) {
                         uint32_t r[16];
                         const uint32_t addr = tmem_o + lane_addr + (uint32_t)(b * g.n + c0);
@@ -642,7 +648,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
             mb_arrive(&sh.p_full);
         }
         if (!bad) {
-            for (int p = ww; p < g.np; p += 4) {
+            for (int p = ww; p < g.np; p += TCL_SWARPS) {
                 const float sum = warp_sum(ls[p * 32 + lane]);
                 if (lane == 0) sh.sum[p] = a.nsplit == 1 ? 1.0f / sum : sum;
             }
@@ -651,20 +657,20 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
         if (!wbar_or(bad)) {
             tc_fence_after();
             if (a.nsplit > 1)
-                for (int p = wt; p < pairs; p += 128) {
+                for (int p = wt; p < pairs; p += TCL_STHREADS) {
                     float* ml = a.part_ml + (((size_t)sh.row[p] * a.heads + sh.head[p]) * a.nsplit + split) * 2;
                     ml[0] = sh.ref[p];
                     ml[1] = sh.sum[p];
                 }
             for (int b = 0; b < g.nb; ++b) {
                 const int r0 = b * 128 + lane_base + lane;
-                for (int c0 = 0; c0 < g.np; c0 += 16) {
-                    uint32_t r[TCL_TERMS][16];
+                for (int c0 = half * 8; c0 < g.np; c0 += 16) {
+                    uint32_t r[TCL_TERMS][8];
 #pragma unroll
-                    for (int k = 0; k < TCL_TERMS; ++k) tmem_ld16(tmem_o + lane_addr + (uint32_t)(b * g.n + k * g.np + c0), r[k]);
+                    for (int k = 0; k < TCL_TERMS; ++k) tmem_ld8(tmem_o + lane_addr + (uint32_t)(b * g.n + k * g.np + c0), r[k]);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) {
+                    for (int j = 0; j < 8; ++j) {
                         const int p = c0 + j;
                         if (p < pairs && r0 < R) {
                             const float v = (__uint_as_float(r[2][j]) + __uint_as_float(r[1][j])) + __uint_as_float(r[0][j]);
@@ -729,7 +735,7 @@ int latent_pick_nsplit(int tiles, int rows_per_tile, int heads, int rank, int bf
     TclGeom g;
     const bool tc = mp > 0 && tcl_geom(rank, rows_per_tile * hpc, &g);
     const int tok = tc ? 128 : CC_TOK, most = (longest + tok - 1) / tok;
-    const int slots = tc && g.smem <= 112 * 1024 && g.cols <= 256 ? 2 * sm_count : sm_count;  // CTAs resident at once
+    const int slots = tc && g.smem <= TCL_PAIR_SMEM && g.cols <= 256 ? 2 * sm_count : sm_count;  // CTAs resident at once
     int s = slots / (ctas > 0 ? ctas : 1);
     if (s > most) s = most;
     if (s > max_split) s = max_split;
