@@ -1042,7 +1042,7 @@ int hm_latent_attn_paged(const float* q, const void* pages, int kv_dtype, const 
     a.scale = scale;
     a.rows_per_tile = rpt;
     a.tiles = tiles;
-    a.nsplit = nsplit ? nsplit : latent_pick_nsplit(tiles, rpt, heads, rank, bf16, longest, sm_count_of_current_device(), 256);
+    a.nsplit = nsplit ? nsplit : latent_pick_nsplit(tiles, rpt, heads, rank, bf16, longest, sm_count_of_current_device(), 256, false);
     a.out = sg.out(out, (size_t)M * heads * rank);
     if (!a.pool.page_table || !a.q || !a.row_pos || !a.row_seq || !a.out) return sg.finish(cudaErrorMemoryAllocation);
     if (!sg.ok(get_wait_err(&a.err_flag))) return sg.finish(cudaSuccess);

@@ -240,7 +240,8 @@ __device__ __forceinline__ float warp_max(float v) {
 
 // ---- GEMV argument block ---------------------------------------------------------------
 // PRO_GNORM: RMSNorm in equal groups, optionally followed by the token shift (see RowNorm)
-enum Prologue { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_GNORM = 2 };
+// PRO_MERGE: the input rows are the splits of an attention over latents, still to be combined (SplitRows)
+enum Prologue { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_GNORM = 2, PRO_MERGE = 3 };
 // EPI_GATE: y = acc * sigmoid(gate); EPI_SQRELU: y = max(acc, 0)^2
 enum Epilogue { EPI_STORE = 0, EPI_QKV_ROPE = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3, EPI_GATE = 4, EPI_SQRELU = 5 };
 
@@ -301,6 +302,13 @@ __device__ __forceinline__ void tc_xpack_store8(unsigned char* xp, int mpad, int
         *reinterpret_cast<uint4*>(tile + (size_t)row * 128 + ((chunk ^ (row & 7)) << 4)) = make_uint4(w[t][0], w[t][1], w[t][2], w[t][3]);
     }
 }
+
+// Splits of attention results: row m of group (head) g is sum_s 2^(max_s - max) acc_s / sum_s 2^(max_s - max) sum_s over its n splits.
+struct SplitRows {
+    const float* acc;  // [rows][groups][n][K], K a multiple of 4
+    const float* ml;   // [rows][groups][n][2]: maximum (base-2 exponent; -inf: an empty split, whose acc is not written), sum
+    int n, groups;
+};
 
 struct KvDesc {
     void* k_pool;            // this layer's K pages [n_pages][kv_heads][page_tokens][hd]
@@ -394,6 +402,7 @@ struct GemvArgs {
     const float* norm_w;
     float eps;
     RowNorm gn;          // PRO_GNORM
+    SplitRows split;     // PRO_MERGE
     // Grouped projection (block-diagonal weights, e.g. one matrix per attention head): group g owns group_slabs slabs,
     // reads its own K inputs at x + g * group_x and writes outputs [g * group_n, (g + 1) * group_n).  0: one group.
     int group_slabs, group_x, group_n;

@@ -939,6 +939,11 @@ int Engine::enqueue_linear(const LinearW& L, int M, const float* x, int ldx, int
                 a.gn = opt->gn;
                 if (a.gn.row_pos) a.gn.row_pos += m0;
                 if (a.gn.row_seq) a.gn.row_seq += m0;
+                a.split = opt->split;
+                if (a.split.n) {
+                    a.split.acc += (size_t)m0 * a.split.groups * a.split.n * L.K;
+                    a.split.ml += (size_t)m0 * a.split.groups * a.split.n * 2;
+                }
                 a.out_scale = opt->out_scale;
                 a.gate = opt->gate ? opt->gate + (size_t)m0 * opt->ld_gate : nullptr;
                 a.ld_gate = opt->ld_gate;
@@ -1230,7 +1235,7 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
             x = hsel_;
         }
         float* const lg = logits_ + lm_dst_row_ * V_;
-        const bool lm_tall = use_tc_ && lm_head_.kind == HM_BF16 && lm_head_.tc && lm_rows > MAX_M;
+        const bool lm_tall = use_tc_ && lm_head_.kind == HM_BF16 && lm_head_.tc && tall_rows(lm_rows);
         const bool slab_argmax = lm_head_.kind == HM_BF16;  // per-block argmax partials from the projection's epilogue
         const bool fold_argmax = slab_argmax && !lm_tall;    // the streaming kernel's last epilogue also produces the greedy token
         lm_folds_argmax_ = fold_argmax;

@@ -58,6 +58,7 @@ struct LayerW {
 // What a projection launch needs beyond the common arguments (enqueue_linear)
 struct LinOpt {
     RowNorm gn{};                        // with PRO_GNORM
+    SplitRows split{};                   // with PRO_MERGE
     const float* out_scale = nullptr;
     const float* gate = nullptr;
     int ld_gate = 0;
@@ -132,6 +133,9 @@ class Engine {
     int alloc_listed_cache(int batch, size_t n_pages);
     void free_listed_cache();
     void free_listed();
+    // Rows from which a pass's projections run on the tensor cores.  The grouped norms of listed designs cost the streaming kernel
+    // more per row, so theirs move over earlier.
+    bool tall_rows(int rows) const { return use_tc_ && rows > (spec_.listed() ? 4 : MAX_M); }
     int enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int next_lm_rows, int* launches);
     int enqueue_listed_logits(const float* x, int rows, float* dst, const struct ArgmaxFold& fold, int* launches);
     int enqueue_tc(const LinearW& L, int M, const unsigned char* xp, int epi, float* y, int ldy, TcArgs& a, int* launches);
@@ -223,6 +227,7 @@ class Engine {
     std::vector<void*> lat_pool_;  // per layer, null for layers that read another's
     float *shift_state_ = nullptr, *shift_saved_ = nullptr;  // [layers][sequences][SHIFT_RING][H]; [layers][SHIFT_RING][H]
     int32_t* seq_iota_ = nullptr;    // 0, 1, 2, ...: the sequence of every row of a decode step
+    int pass_nsplit_ = 1;            // splits the attention of the layer being enqueued left for the next projection to combine
     int pass_longest_ = 0;           // longest context of the pass being enqueued (splits of the attention)
     std::vector<std::pair<int, int>> pass_runs_;  // that pass's runs: first row, rows; empty: a run per row
     // portions (step)

@@ -10,7 +10,7 @@
 //   vup     per head: result -> values, times sigmoid(gate)
 //   o       output projection, layer scale, residual
 //   up      grouped norm, projection, squared ReLU;   down  projection, layer scale, residual
-// Passes of up to eight rows run the streaming kernel with the norm in its prologue; larger passes run the tensor-core GEMM on
+// Passes of a few rows run the streaming kernel with the norm in its prologue; larger passes run the tensor-core GEMM on
 // packed activations, which the producers write themselves wherever the sizes allow.
 #include <algorithm>
 
@@ -304,7 +304,7 @@ int Engine::enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int
     const LayerW& w = layers_[l];
     const LayerSpec& s = spec_.layers[l];
     const float eps = (float)cfg_.rms_norm_eps;
-    const bool tall = use_tc_ && M > MAX_M;
+    const bool tall = tall_rows(M);
     auto want = [&](int cls) { return only_class_ < 0 || only_class_ == cls; };
     auto prefetch = [&](const LinearW* n) {  // weights of the kernel two launches ahead (streaming passes)
         pf_ptr_ = nullptr;
@@ -393,8 +393,10 @@ int Engine::enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int
         for (auto& r : pass_runs_) tiles += (r.first + r.second - 1) / a.rows_per_tile - r.first / a.rows_per_tile + 1;
         if (a.rows_per_tile == 1) tiles = M;
         a.tiles = tiles;
+        a.unmerged = !tall && s.kv_rank % 4 == 0 ? 1 : 0;
         a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
-        a.nsplit = latent_pick_nsplit(tiles, a.rows_per_tile, s.heads, s.kv_rank, kv_bf16_, pass_longest_, sm_count_, most);
+        a.nsplit = latent_pick_nsplit(tiles, a.rows_per_tile, s.heads, s.kv_rank, kv_bf16_, pass_longest_, sm_count_, most, a.unmerged != 0);
+        pass_nsplit_ = a.unmerged ? a.nsplit : 1;
         a.part_acc = lat_acc_;
         a.part_ml = lat_ml_;
         a.out = ctx_;
@@ -420,8 +422,10 @@ int Engine::enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int
             o.group_x = s.kv_rank;
             o.gate = gate;
             o.ld_gate = ld;
+            const bool merge = pass_nsplit_ > 1;
+            if (merge) o.split = SplitRows{lat_acc_, lat_ml_, pass_nsplit_, s.heads};
             prefetch(s.mlp == MLP_NONE ? nullptr : &w.gu);
-            rc = enqueue_linear(w.vup, M, ctx_, lat, PRO_PLAIN, nullptr, EPI_GATE, attn_, vals, nullptr, nullptr, l, row_pos, row_seq, nullptr, nullptr, launches, nullptr, &o);
+            rc = enqueue_linear(w.vup, M, ctx_, lat, merge ? PRO_MERGE : PRO_PLAIN, nullptr, EPI_GATE, attn_, vals, nullptr, nullptr, l, row_pos, row_seq, nullptr, nullptr, launches, nullptr, &o);
         }
         if (rc) return rc;
     }
@@ -479,7 +483,7 @@ int Engine::enqueue_listed_logits(const float* x, int rows, float* dst, const Ar
     RowNorm gn{};
     gn.groups = spec_.norm_groups;
     const float eps = (float)cfg_.rms_norm_eps;
-    if (use_tc_ && rows > MAX_M) {
+    if (tall_rows(rows)) {
         const cudaError_t ce = launch_tc_pack_gnorm(x, H_, rows, H_, final_norm_, eps, gn, xpack_, stream_, pdl_);
         if (ce != cudaSuccess) return cuda_fail(ce, "norm and pack launch");
         ++*launches;

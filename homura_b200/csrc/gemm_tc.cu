@@ -313,12 +313,20 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
             v = fmaxf(v, 0.f);
             return v * v;
         };
-        if (a.xp_out && (n0 & 7) == 0 && n0 + BM <= n_end) {
-            for (int idx = tid; idx < rows * (BM / 8); idx += TC_THREADS) {
-                const int m = m_lo + idx / (BM / 8), c = (idx % (BM / 8)) * 8;
+        if (a.xp_out && ((n0 | n_end) & 7) == 0) {
+            const int nc = min(BM, n_end - n0) / 8;  // pieces of eight outputs
+            for (int idx = tid; idx < rows * nc; idx += TC_THREADS) {
+                const int m = m_lo + idx / nc, c = (idx % nc) * 8;
                 float v[8];
+                if (a.epi == EPI_GATE && (a.ld_gate & 3) == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 15) == 0) {
+                    const float4 g0 = ld_cg_f32x4(a.gate + (size_t)m * a.ld_gate + n0 + c), g1 = ld_cg_f32x4(a.gate + (size_t)m * a.ld_gate + n0 + c + 4);
+                    const float g[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
 #pragma unroll
-                for (int e = 0; e < 8; ++e) v[e] = act(m, n0 + c + e, tile[m * BM + c + e]);
+                    for (int e = 0; e < 8; ++e) v[e] = tile[m * BM + c + e] / (1.0f + expf(-g[e]));
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) v[e] = act(m, n0 + c + e, tile[m * BM + c + e]);
+                }
                 tc_xpack_store8(a.xp_out, a.xp_mpad, m, n0 + c, v);
             }
         } else {

@@ -96,7 +96,7 @@ __host__ __device__ __forceinline__ int gnorm_span(int K, int groups, int rps) {
 // everything that goes with it is requested before the factors are known.  The first slab's CTAs keep the last
 // row of every run in the state.
 template <int M>
-__device__ __forceinline__ void gnorm_stage(const GemvArgs& a, float* __restrict__ xs, float* __restrict__ gfac, int rps, int k0, int nrows, int slab, int tid) {
+__device__ __forceinline__ void gnorm_stage(const GemvArgs& a, float* __restrict__ xs, float* __restrict__ gfac, const int* s_pos, const int* s_seq, int rps, int k0, int nrows, int slab, int tid) {
     if (nrows <= 0) return;  // uniform over the CTA
     const int lane = tid & 31, warp = tid >> 5;
     const int gs = a.K / a.gn.groups, g_lo = k0 / gs, ng = (k0 + nrows - 1) / gs - g_lo + 1;
@@ -107,8 +107,8 @@ __device__ __forceinline__ void gnorm_stage(const GemvArgs& a, float* __restrict
         pos[m] = 0;
         seq[m] = -1;
         if (a.gn.shift && m < a.m_valid) {
-            pos[m] = a.gn.row_pos[m];
-            seq[m] = a.gn.row_seq[m];
+            pos[m] = s_pos[m];
+            seq[m] = s_seq[m];
         }
     }
     auto follows = [&](int m) { return m > 0 && m < a.m_valid && seq[m] == seq[m - 1] && pos[m] == pos[m - 1] + 1; };
@@ -177,6 +177,60 @@ __device__ __forceinline__ void gnorm_stage(const GemvArgs& a, float* __restrict
             xs[m * rps + r] = v;
         }
     }
+}
+
+// PRO_MERGE: elements [k0, k0 + nrows) of the combined rows of group `grp` into xs[M][rps]; wts holds M * n floats, part
+// M * 1024 (the slots of the reduction behind the multiply, not yet in use).
+template <int M>
+__device__ __forceinline__ void merge_stage(const GemvArgs& a, float* __restrict__ xs, float* __restrict__ wts, float* __restrict__ part, int rps, int k0, int nrows, int grp, int tid) {
+    const int lane = tid & 31, warp = tid >> 5, n = a.split.n;
+    if (warp < M && warp < a.m_valid) {
+        const float* ml = a.split.ml + ((size_t)warp * a.split.groups + grp) * n * 2;
+        float mx = -INFINITY, l = 0.f;
+        for (int s = lane; s < n; s += 32) {
+            const float v = ld_cg_f32(ml + 2 * s);
+            wts[warp * n + s] = v;
+            mx = fmaxf(mx, v);
+        }
+        mx = warp_max(mx);
+        for (int s = lane; s < n; s += 32) {
+            const float f = exp2f(wts[warp * n + s] - mx);
+            wts[warp * n + s] = f;
+            l = fmaf(f, ld_cg_f32(ml + 2 * s + 1), l);
+        }
+        const float inv = 1.0f / warp_sum(l);
+        for (int s = lane; s < n; s += 32) wts[warp * n + s] *= inv;
+    }
+    __syncthreads();
+    if (nrows <= 0) return;
+    const int n4 = nrows >> 2, sg_n = GEMV_THREADS / n4, i4 = tid % n4, sg = tid / n4;  // at most 1024 rows (K <= 1024)
+    if (sg < sg_n) {
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+            float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (m < a.m_valid) {
+                const float* src = a.split.acc + ((size_t)m * a.split.groups + grp) * n * a.K + k0 + 4 * i4;
+#pragma unroll 4
+                for (int s = sg; s < n; s += sg_n) {
+                    const float f = wts[m * n + s];
+                    if (f > 0.f) {
+                        const float4 v = ld_cg_f32x4(src + (size_t)s * a.K);
+                        t.x = fmaf(f, v.x, t.x); t.y = fmaf(f, v.y, t.y); t.z = fmaf(f, v.z, t.z); t.w = fmaf(f, v.w, t.w);
+                    }
+                }
+            }
+            *reinterpret_cast<float4*>(part + m * 1024 + (sg * n4 + i4) * 4) = t;
+        }
+    }
+    __syncthreads();
+    for (int r = tid; r < nrows; r += GEMV_THREADS)
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+            float v = 0.f;
+            for (int g = 0; g < sg_n; ++g) v += part[m * 1024 + g * nrows + r];
+            xs[m * rps + r] = v;
+        }
+    __syncthreads();  // part is written again behind the multiply
 }
 
 // The unsplit M = 1 variant (LM head: one long stream per CTA) runs three CTAs per SM (<= 85
@@ -293,6 +347,12 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
         if (a.bias && tid < SLAB) bias_s[tid] = n0e + tid < a.N ? __ldg(a.bias + n0e + tid) : 0.f;
     }
 
+    if (a.pro == PRO_GNORM && a.gn.shift && tid < M && tid < a.m_valid) {
+        s_pos[tid] = a.gn.row_pos[tid];
+        s_page[tid] = a.gn.row_seq[tid];
+    }
+    if (a.pro == PRO_GNORM) __syncthreads();
+
     pdl_wait();
     // the RMSNorm weights fetched above are read below by other threads than those that stored them (a CTA that
     // became resident just before its dependency resolved may still have those loads in flight)
@@ -328,8 +388,10 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
                     rowv[m][i] = idx < (a.K >> 2) ? ld_cg_f32x4(a.x + (size_t)m * a.ldx + 4 * (size_t)idx) : make_float4(0.f, 0.f, 0.f, 0.f);
                 }
         }
+    } else if (a.pro == PRO_MERGE) {
+        merge_stage<M>(a, xs, gfac, red, rps, k0, nrows, grp, tid);
     } else if (a.pro == PRO_GNORM) {
-        gnorm_stage<M>(a, xs, gfac, rps, k0, nrows, slab, tid);
+        gnorm_stage<M>(a, xs, gfac, s_pos, s_page, rps, k0, nrows, slab, tid);
     } else if (a.pro == PRO_RMSNORM) {
         float ss[M];
 #pragma unroll
@@ -734,6 +796,10 @@ cudaError_t launch_mc(const GemvArgs& a_in, cudaStream_t st, bool pdl) {
     if (a.pro == PRO_GNORM) {
         if (a.gn.groups < 1 || a.K % a.gn.groups != 0) return cudaErrorInvalidValue;
         floats += (size_t)M * gnorm_span(a.K, a.gn.groups, a.rows_per_split);
+    }
+    if (a.pro == PRO_MERGE) {
+        if (a.K > 1024 || a.K % 4 != 0 || a.split.n < 1) return cudaErrorInvalidValue;
+        floats += (size_t)M * a.split.n;
     }
     size_t smem = sizeof(float) * floats;
     // cluster launches over the slab layout whose slice fits: weights staged in shared memory before the dependency wait

@@ -729,7 +729,7 @@ int latent_rows_per_tile(int longest_run, int heads, int rank, int bf16) {
     return r < 1 ? 1 : r;
 }
 
-int latent_pick_nsplit(int tiles, int rows_per_tile, int heads, int rank, int bf16, int longest, int sm_count, int max_split) {
+int latent_pick_nsplit(int tiles, int rows_per_tile, int heads, int rank, int bf16, int longest, int sm_count, int max_split, bool free_merge) {
     const int mp = latent_tc_pairs(rank, bf16);
     const int hpc = mp ? tcl_heads(heads, mp) : CC_HEADS, ctas = tiles * ((heads + hpc - 1) / hpc);
     TclGeom g;
@@ -740,7 +740,7 @@ int latent_pick_nsplit(int tiles, int rows_per_tile, int heads, int rank, int bf
     if (s > most) s = most;
     if (s > max_split) s = max_split;
     if (s > 256) s = 256;
-    if (tc && most < 4) s = 1;  // the merge costs as much as three tiles
+    if (tc && most < 4 && !free_merge) s = 1;  // the merge launch costs as much as three tiles
     return s < 1 ? 1 : s;
 }
 
@@ -777,7 +777,7 @@ cudaError_t launch_latent_attn(const LatentAttnArgs& a_in, cudaStream_t st, bool
     }
     if (e != cudaSuccess) return e;
     ++*launches;
-    if (a.nsplit > 1) {
+    if (a.nsplit > 1 && !a.unmerged) {
         e = launch(latent_merge_kernel, dim3(a.M, a.heads, (R + 127) / 128), dim3(128), 0, st, pdl, a);
         if (e == cudaSuccess) ++*launches;
     }

@@ -37,6 +37,7 @@ struct LatentAttnArgs {
     float scale;
     int rows_per_tile;       // latent_rows_per_tile: rows of one run (consecutive positions of a sequence) that may share a CTA
     int tiles;               // with rows_per_tile > 1 (at most 64 rows then): tiles the rows fall into, 0: not known
+    int unmerged;            // leave the splits in part_acc / part_ml (the caller's next kernel combines them)
     int early;               // every row is its own sequence and the pages in front of its newest token were complete before the launch in front began
     int nsplit;
     float* part_acc;         // [M][heads][nsplit][rank], with nsplit > 1
@@ -59,7 +60,7 @@ int latent_tc_pairs(int rank, int bf16);
 // Rows of a run that share a CTA, in a pass whose longest run has so many rows.
 int latent_rows_per_tile(int longest_run, int heads, int rank, int bf16);
 // Splits of the longest context (in tokens) so that a pass of so many tiles fills the SMs; at most max_split.
-int latent_pick_nsplit(int tiles, int rows_per_tile, int heads, int rank, int bf16, int longest, int sm_count, int max_split);
+int latent_pick_nsplit(int tiles, int rows_per_tile, int heads, int rank, int bf16, int longest, int sm_count, int max_split, bool free_merge);
 cudaError_t launch_latent_attn(const LatentAttnArgs& a, cudaStream_t st, bool pdl, int* launches);
 
 }  // namespace hm
