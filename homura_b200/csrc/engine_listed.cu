@@ -283,6 +283,8 @@ int Engine::enqueue_tc(const LinearW& L, int M, const unsigned char* xp, int epi
     a.N = L.N;
     a.M = M;
     a.ksplit = tc_pick_split(L.K, L.columns(), sm_count_);
+    if (L.groups)  // short contractions over few blocks: half as many k-blocks per CTA as the wide projections keep
+        while (a.ksplit < 4 && a.Kp / 64 / (a.ksplit * 2) >= 2 && L.columns() / SLAB * a.ksplit * 2 <= sm_count_) a.ksplit *= 2;
     a.xp = xp;
     a.xp_mpad = tc_mpad(M);
     a.epi = epi;

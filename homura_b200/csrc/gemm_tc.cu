@@ -141,65 +141,105 @@ __global__ void __launch_bounds__(256) tc_pack_x_kernel(const float* __restrict_
 // One block per padded row.  A row whose predecessor is the row in front normalises that row a second time instead of
 // waiting for its block.  The block of a run's FIRST row also keeps the run's last row in the state: it has read the
 // slot in front of the run by then, and it is the only block that touches this sequence's state.
-__device__ __forceinline__ void gnorm_row(const float* __restrict__ src, float* __restrict__ row, float* __restrict__ fac, int K, int groups, float eps, int tid) {
-    stage_row<256, false>(src, row, K, tid);
-    __syncthreads();
+// Two rows at once (src1 null: zeros), both requested before the first is stored.
+__device__ __forceinline__ void gnorm_stage2(const float* src0, const float* src1, float* __restrict__ dst0, float* __restrict__ dst1, int K, int tid) {
+    if (((reinterpret_cast<uintptr_t>(src0) | reinterpret_cast<uintptr_t>(src1)) & 15) == 0 && (K & 3) == 0) {
+        const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int i = tid; i < K / 4; i += 512) {
+            const bool more = i + 256 < K / 4;
+            const float4 v0 = ld_cg_f32x4(src0 + 4 * (size_t)i), v1 = more ? ld_cg_f32x4(src0 + 4 * (size_t)(i + 256)) : z;
+            const float4 u0 = src1 ? ld_cg_f32x4(src1 + 4 * (size_t)i) : z, u1 = src1 && more ? ld_cg_f32x4(src1 + 4 * (size_t)(i + 256)) : z;
+            reinterpret_cast<float4*>(dst0)[i] = v0;
+            if (dst1) reinterpret_cast<float4*>(dst1)[i] = u0;
+            if (more) {
+                reinterpret_cast<float4*>(dst0)[i + 256] = v1;
+                if (dst1) reinterpret_cast<float4*>(dst1)[i + 256] = u1;
+            }
+        }
+    } else {
+        for (int i = tid; i < K; i += 256) {
+            const float v = ld_cg_f32(src0 + i), u = src1 ? ld_cg_f32(src1 + i) : 0.f;
+            dst0[i] = v;
+            if (dst1) dst1[i] = u;
+        }
+    }
+}
+// 1 / root mean square of every group of a staged row; the eight warps take the groups in turn.
+__device__ __forceinline__ void gnorm_factors(const float* __restrict__ row, float* __restrict__ fac, int K, int groups, float eps, int tid) {
     const int gs = K / groups, lane = tid & 31;
     for (int g = tid >> 5; g < groups; g += 8) {
         float s = 0.f;
+#pragma unroll 4
         for (int i = lane; i < gs; i += 32) s = fmaf(row[g * gs + i], row[g * gs + i], s);
         s = warp_sum(s);
         if (lane == 0) fac[g] = 1.0f / sqrtf(s / (float)gs + eps);
     }
-    __syncthreads();
 }
 __global__ void __launch_bounds__(256) tc_pack_gnorm_kernel(const float* __restrict__ x, int ldx, int M, int mpad, int K, int Kp, const float* __restrict__ norm_w, float eps, const RowNorm gn, unsigned char* __restrict__ out) {
     extern __shared__ __align__(16) float rows[];
-    float *cur = rows, *nb = rows + Kp, *fac = nb + (gn.shift ? Kp : 0), *nfac = fac + gn.groups;
+    // the row, the one in front (its raw values, or the kept row), and, in the block of a run's first row, the run's last row
+    float *cur = rows, *nb = rows + Kp, *end = nb + Kp, *fac = rows + (gn.shift ? 3 : 1) * (size_t)Kp, *nfac = fac + gn.groups, *efac = nfac + gn.groups;
     __shared__ int s_last;
-    pdl_launch_dependents();
-    pdl_wait();
     const int m = blockIdx.x, tid = threadIdx.x;
-    const bool row_ok = m < M;
+    const bool row_ok = m < M, shift = gn.shift != nullptr;
     const int gs = K / gn.groups;
-    if (row_ok) {
-        gnorm_row(x + (size_t)m * ldx, cur, fac, K, gn.groups, eps, tid);
-        for (int k = tid; k < K; k += 256) cur[k] = (cur[k] * fac[k / gs]) * __ldg(norm_w + k);
-        if (gn.shift) {
-            const int pos = gn.row_pos[m], seq = gn.row_seq[m];
-            const bool follows = m > 0 && gn.row_seq[m - 1] == seq && gn.row_pos[m - 1] + 1 == pos;
-            float* st = gn.state + (size_t)seq * SHIFT_RING * K;
-            if (follows) {
-                gnorm_row(x + (size_t)(m - 1) * ldx, nb, nfac, K, gn.groups, eps, tid);
-                for (int k = tid; k < K; k += 256) {
-                    const float p = (nb[k] * nfac[k / gs]) * __ldg(norm_w + k), h = cur[k];
-                    cur[k] = fmaf(p - h, __ldg(gn.shift + k), h);
-                }
-            } else {
-                if (tid == 0) {
-                    int e = m;
-                    while (e + 1 < M && gn.row_seq[e + 1] == seq && gn.row_pos[e + 1] == gn.row_pos[e] + 1) ++e;
-                    s_last = e;
-                }
-                __syncthreads();
-                const int e = s_last;
-                if (e != m) gnorm_row(x + (size_t)e * ldx, nb, nfac, K, gn.groups, eps, tid);
-                float* keep = st + (size_t)((pos + e - m) % SHIFT_RING) * K;
-                const float* prev = st + (size_t)((pos + SHIFT_RING - 1) % SHIFT_RING) * K;
-                for (int k = tid; k < K; k += 256) {
-                    const float h = cur[k], p = pos > 0 ? prev[k] : 0.f;  // a plain load: it must stay in front of the store, which may be to the same slot
-                    keep[k] = e != m ? (nb[k] * nfac[k / gs]) * __ldg(norm_w + k) : h;
-                    cur[k] = fmaf(p - h, __ldg(gn.shift + k), h);
-                }
-            }
+    pdl_launch_dependents();
+    // positions, sequences and weights do not depend on the launch in front
+    int pos = 0, seq = 0;
+    bool follows = false;
+    if (shift && row_ok) {
+        pos = gn.row_pos[m];
+        seq = gn.row_seq[m];
+        follows = m > 0 && gn.row_seq[m - 1] == seq && gn.row_pos[m - 1] + 1 == pos;
+        if (!follows && tid == 0) {
+            int e = m;
+            while (e + 1 < M && gn.row_seq[e + 1] == seq && gn.row_pos[e + 1] == gn.row_pos[e] + 1) ++e;
+            s_last = e;
         }
-        for (int k = K + tid; k < Kp; k += 256) cur[k] = 0.f;
+    }
+    float w[8], sh[8];
+    auto weights = [&](int k0) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            w[e] = k0 + e < K ? __ldg(norm_w + k0 + e) : 0.f;
+            sh[e] = shift && k0 + e < K ? __ldg(gn.shift + k0 + e) : 0.f;
+        }
+    };
+    weights(tid * 8);
+    pdl_wait();
+    float* st = shift ? gn.state + (size_t)seq * SHIFT_RING * K : nullptr;
+    int e = m;
+    if (row_ok) {
+        const float* xr = x + (size_t)m * ldx;
+        gnorm_stage2(xr, !shift ? nullptr : follows ? xr - ldx : pos > 0 ? st + (size_t)((pos + SHIFT_RING - 1) % SHIFT_RING) * K : nullptr, cur, shift ? nb : nullptr, K, tid);
+        __syncthreads();  // the kept row has been read: its slot may be written
+        e = shift && !follows ? s_last : m;
+        if (e != m) {
+            gnorm_stage2(x + (size_t)e * ldx, nullptr, end, nullptr, K, tid);
+            __syncthreads();
+            gnorm_factors(end, efac, K, gn.groups, eps, tid);
+        }
+        gnorm_factors(cur, fac, K, gn.groups, eps, tid);
+        if (follows) gnorm_factors(nb, nfac, K, gn.groups, eps, tid);
         __syncthreads();
     }
     for (int c = tid; c < Kp / 8; c += 256) {
+        if (c != tid) weights(c * 8);
         float v[8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = row_ok ? cur[c * 8 + e] : 0.f;
+        for (int i = 0; i < 8; ++i) {
+            const int k = c * 8 + i;
+            v[i] = 0.f;
+            if (!row_ok || k >= K) continue;
+            const int g = k / gs;
+            const float h = (cur[k] * fac[g]) * w[i];
+            v[i] = h;
+            if (shift) {
+                const float p = follows ? (nb[k] * nfac[g]) * w[i] : nb[k];
+                v[i] = fmaf(p - h, sh[i], h);
+                if (!follows) st[(size_t)((pos + e - m) % SHIFT_RING) * K + k] = e != m ? (end[k] * efac[g]) * w[i] : h;
+            }
+        }
         tc_xpack_store8(out, mpad, m, c * 8, v);
     }
 }
@@ -685,7 +725,7 @@ cudaError_t launch_tc_pack_x(const float* x, int ldx, int M, int K, const float*
 cudaError_t launch_tc_pack_gnorm(const float* x, int ldx, int M, int K, const float* norm_w, float eps, const RowNorm& gn, void* xp, cudaStream_t st, bool pdl) {
     if (M < 1 || M > MR || gn.groups < 1 || K % gn.groups != 0) return cudaErrorInvalidValue;
     const int Kp = tc_padded_k(K);
-    const size_t smem = ((size_t)Kp * (gn.shift ? 2 : 1) + 2 * (size_t)gn.groups) * sizeof(float);
+    const size_t smem = ((size_t)Kp + 3 * (size_t)gn.groups + (gn.shift ? 2 * (size_t)Kp : 0)) * sizeof(float);
     const cudaError_t e = ensure_dyn_smem(tc_pack_gnorm_kernel, smem);
     if (e != cudaSuccess) return e;
     cudaLaunchConfig_t cfg = {};
