@@ -327,3 +327,15 @@ def test_the_trace_runner_replays_steps(hm, tmp_path):
     close(read(0), want[[2, 49]], "F32", "replayed logits")
     assert not (out / "1.f32").exists()
     close(read(2), want[[10, 63]], "F32", "replayed logits")
+
+
+def test_generation_on_the_command_line(hm, tmp_path, capsys):
+    from homura_b200.__main__ import main
+
+    d = synth.write_tunitar_model(str(tmp_path), model("mixed"), 21, weights("mixed"))
+    refs = [greedy("mixed", 70, 37, 60), greedy("mixed", 90, 70, 20)]
+    args = ["generate", d, "--max-new", "20", "--dtype", "f32"]
+    for ids, _ in refs:
+        args += ["--ids", ",".join(map(str, ids))]
+    assert main(args) == 0
+    assert capsys.readouterr().out.split() == [",".join(map(str, want[:20])) for _, want in refs]

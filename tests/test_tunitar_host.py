@@ -126,3 +126,11 @@ def test_shared_latents_are_the_named_layers():
     for k in ("uk", "uv"):
         w[f"l3.mix.{k}"] = np.pad(w[f"l3.mix.{k}"], ((0, 0), (0, 24)))
     assert np.abs(Oracle(swapped, w).forward(ids) - want).max() > 0.05 * np.abs(want).max()
+
+
+def test_info_on_the_command_line(hm, tmp_path, capsys):
+    from homura_b200.__main__ import main
+
+    assert main(["info", synth.write_tunitar_model(str(tmp_path), model("mixed"), 1)]) == 0
+    out = capsys.readouterr().out
+    assert "architecture: Tunitar" in out and "layer 2:" in out and "l1.mix.dkv.norm  BF16  [48]" in out
