@@ -1020,13 +1020,13 @@ int hm_latent_attn_paged(const float* q, const void* pages, int kv_dtype, const 
     if (const int rc = check_latent_rows(row_seq, row_pos, M, n_seq, max_pages)) return rc;
     const int bf16 = kv_dtype == HM_BF16;
     int longest = 0, tiles = 0, longest_run = 1;
+    for (int m = 0; m < M; ++m) longest = std::max(longest, row_pos[m] + 1);
     for (int m = 1, run = 1; m < M; ++m) {
         run = row_seq[m - 1] == row_seq[m] && row_pos[m - 1] + 1 == row_pos[m] ? run + 1 : 1;
         longest_run = std::max(longest_run, run);
     }
-    const int rpt = latent_rows_per_tile(longest_run, heads, rank, bf16);
+    const int rpt = latent_rows_per_tile(longest_run, longest, heads, rank, bf16);
     for (int m = 0; m < M; ++m) {
-        longest = std::max(longest, row_pos[m] + 1);
         if (m % rpt == 0 || row_seq[m - 1] != row_seq[m] || row_pos[m - 1] + 1 != row_pos[m]) ++tiles;
     }
     cudaStream_t st = (cudaStream_t)stream;

@@ -160,7 +160,7 @@ int Engine::alloc_listed_scratch(int cap) {
         kmax = std::max(kmax, std::max(std::max(s.heads * s.vdim, s.ff), std::max(s.dim, s.kv_rank)));
         // splits times rows never exceed the SMs times the rows that share a CTA (latent_pick_nsplit)
         for (int bf16 = 0; bf16 < 2; ++bf16) {
-            const size_t rows = 2 * (size_t)sm_count_ * latent_rows_per_tile(TC_ROWS, s.heads, s.kv_rank, bf16);
+            const size_t rows = 2 * (size_t)sm_count_ * latent_rows_per_tile(TC_ROWS, 1 << 30, s.heads, s.kv_rank, bf16);
             acc = std::max(acc, rows * s.heads * s.kv_rank);
             ml = std::max(ml, rows * s.heads * 2);
         }
@@ -391,7 +391,7 @@ int Engine::enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int
         // tiles: every run is cut at the multiples of the rows that share a CTA
         int longest_run = 1, tiles = 0;
         for (auto& r : pass_runs_) longest_run = std::max(longest_run, r.second);
-        a.rows_per_tile = latent_rows_per_tile(longest_run, s.heads, s.kv_rank, kv_bf16_);
+        a.rows_per_tile = latent_rows_per_tile(longest_run, pass_longest_, s.heads, s.kv_rank, kv_bf16_);
         for (auto& r : pass_runs_) tiles += (r.first + r.second - 1) / a.rows_per_tile - r.first / a.rows_per_tile + 1;
         if (a.rows_per_tile == 1) tiles = M;
         a.tiles = tiles;

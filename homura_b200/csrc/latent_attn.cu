@@ -721,10 +721,14 @@ int latent_tc_pairs(int rank, int bf16) {
     return 0;
 }
 
-int latent_rows_per_tile(int longest_run, int heads, int rank, int bf16) {
-    const int mp = latent_tc_pairs(rank, bf16);
+// Rows share a CTA where that costs no MMA columns (16 pairs), and up to 32 pairs where the contexts are long enough for the
+// re-read latents to matter more than the CTAs that are lost (measured: 64 pairs are slower at every length).
+int latent_rows_per_tile(int longest_run, int longest, int heads, int rank, int bf16) {
+    int mp = latent_tc_pairs(rank, bf16);
     if (mp == 0 || longest_run < 2) return 1;
-    int r = mp / tcl_heads(heads, mp);
+    const int hpc = tcl_heads(heads, mp), fill = longest >= 4096 ? 32 : 16;
+    if (mp > fill) mp = fill;
+    int r = mp / hpc;
     if (r > longest_run) r = longest_run;
     return r < 1 ? 1 : r;
 }

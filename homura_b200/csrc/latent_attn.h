@@ -57,8 +57,8 @@ cudaError_t launch_latent_read(const LatentPool& pool, int seq, int len, float* 
 
 // Largest (row, head) pair count a tensor-core CTA takes for this rank; 0: the kernel does not cover it (or the pages are f32).
 int latent_tc_pairs(int rank, int bf16);
-// Rows of a run that share a CTA, in a pass whose longest run has so many rows.
-int latent_rows_per_tile(int longest_run, int heads, int rank, int bf16);
+// Rows of a run that share a CTA, in a pass whose longest run has so many rows and whose longest context so many tokens.
+int latent_rows_per_tile(int longest_run, int longest, int heads, int rank, int bf16);
 // Splits of the longest context (in tokens) so that a pass of so many tiles fills the SMs; at most max_split.
 int latent_pick_nsplit(int tiles, int rows_per_tile, int heads, int rank, int bf16, int longest, int sm_count, int max_split, bool free_merge);
 cudaError_t launch_latent_attn(const LatentAttnArgs& a, cudaStream_t st, bool pdl, int* launches);

@@ -143,3 +143,18 @@ def test_bad_rows_are_errors(hm):
     for seq, pos in ((1, 0), (-1, 0), (0, 64), (0, -1)):
         with pytest.raises(hm.HomuraError):
             cache.attend(q, 1.0, [seq], [pos])
+
+
+@pytest.mark.parametrize("heads", [1, 3, 12])
+def test_portions_behind_a_long_context(hm, heads):
+    """Rows that share a CTA, in passes whose contexts are long enough for the wider tiles, with a key that stands out far away."""
+    rank, length = 64, 4300
+    cache, stored = make_cache(hm, rank, hm.DType.BF16, [length, 30], 17)
+    rows = [(0, p) for p in range(4200, 4233)] + [(1, p) for p in range(5, 25)] + [(0, 1)]
+    rs, rp = np.array([r[0] for r in rows]), np.array([r[1] for r in rows])
+    g = np.random.default_rng(heads)
+    q = g.standard_normal((len(rows), heads, rank)).astype(np.float32) * 0.3
+    q[3, 0], q[20, heads - 1] = stored[0][2], stored[0][4095]
+    want = reference(q, stored, 1.0, rs, rp)
+    for nsplit in (0, 1, 5):
+        check(cache.attend(q, 1.0, rs, rp, nsplit), want, 5e-3)
