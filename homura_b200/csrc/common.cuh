@@ -381,7 +381,7 @@ __device__ __forceinline__ void rope_tile_epilogue(const RopeEpi& r, const float
     }
 }
 
-struct GemvArgs {
+struct GemvBase {
     int* err_flag;                 // optional: raised to 2 when the bounded wait for the staged weights runs out
     unsigned long long* trace;     // optional (HM_GEMV_TRACE=1): 8 %globaltimer stamps of CTA 0 of this launch
     const void* pf_ptr;            // optional: weights of a later kernel to pull into the L2 (see l2_prefetch_slice)
@@ -401,20 +401,12 @@ struct GemvArgs {
     int pro;
     const float* norm_w;
     float eps;
-    RowNorm gn;          // PRO_GNORM
-    SplitRows split;     // PRO_MERGE
-    // Grouped projection (block-diagonal weights, e.g. one matrix per attention head): group g owns group_slabs slabs,
-    // reads its own K inputs at x + g * group_x and writes outputs [g * group_n, (g + 1) * group_n).  0: one group.
-    int group_slabs, group_x, group_n;
     // epilogue
     int epi;
     float* y;
     int ldy;
     const float* bias;   // [N] or null
     const float* resid;  // [M][ldy] or null (EPI_STORE: y = resid + acc)
-    const float* out_scale;  // [N] or null (EPI_STORE: the result is multiplied element by element before the residual is added)
-    const float* gate;   // EPI_GATE: [M][ld_gate]
-    int ld_gate;
     // EPI_QKV_ROPE
     int q_dim, kv_dim, hd, has_qk_norm;
     const float* q_norm_w;
@@ -440,6 +432,20 @@ struct GemvArgs {
     // split-K scratch
     float* partial;      // [nslabs*ksplit][M][128]
     unsigned int* tickets;  // [nslabs], zero between launches
+};
+
+// The arguments of the kernel's extended variant (gemv_ext.cu): what only some designs need is compiled apart, so that the
+// plain projections, which are latency chains, carry none of it.
+struct GemvArgs : GemvBase {
+    RowNorm gn;          // PRO_GNORM
+    SplitRows split;     // PRO_MERGE
+    // Grouped projection (block-diagonal weights, e.g. one matrix per attention head): group g owns group_slabs slabs,
+    // reads its own K inputs at x + g * group_x and writes outputs [g * group_n, (g + 1) * group_n).  0: one group.
+    int group_slabs, group_x, group_n;
+    const float* out_scale;  // [N] or null (EPI_STORE: the result is multiplied element by element before the residual is added)
+    const float* gate;   // EPI_GATE: [M][ld_gate]
+    int ld_gate;
+    bool extended() const { return pro == PRO_GNORM || pro == PRO_MERGE || epi == EPI_GATE || epi == EPI_SQRELU || group_slabs != 0 || out_scale != nullptr; }
 };
 
 struct AttnArgs {
@@ -499,6 +505,7 @@ struct QuantArgs {
 
 // ---- launchers (defined in the .cu files) ----------------------------------------------
 cudaError_t launch_gemv_bf16(const GemvArgs& a, int M, cudaStream_t st, bool pdl);
+cudaError_t launch_gemv_bf16_ext(const GemvArgs& a, int M, cudaStream_t st, bool pdl);  // what launch_gemv_bf16 calls for extended() arguments
 
 size_t gemv_partial_floats(int N, int ksplit, int M);
 void gemv_pick_split(int K, int N, int M, int sm_count, int* ksplit, int* rows_per_split);

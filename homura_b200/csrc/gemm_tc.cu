@@ -248,15 +248,24 @@ __global__ void __launch_bounds__(256) tc_pack_gnorm_kernel(const float* __restr
 // The same four epilogues as the streaming projection kernel (gemv_bf16.cu), for up to 64 rows.
 __device__ __forceinline__ bool tc_better(float v, int i, float bv, int bi) { return v > bv || (v == bv && i > bi); }
 
+// X: the extended variant (grouped weights, output scale, gate, squared ReLU, queries split into images), compiled apart so that the
+// plain projections carry none of it.
+template <bool X>
 __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, int nblk, int tid, const int* s_pos, const int* s_page) {
     // grouped projections: this block's output columns [n0, n_end)
-    const int grp = a.group_blocks ? nblk / a.group_blocks : 0;
-    const int n0 = a.group_blocks ? grp * a.group_n + (nblk - grp * a.group_blocks) * BM : nblk * BM, rows = m_hi - m_lo;
-    const int n_end = a.group_blocks ? (grp + 1) * a.group_n : a.N;
+    const int rows = m_hi - m_lo;
+    int n0 = nblk * BM, n_end = a.N;
+    if constexpr (X) {
+        if (a.group_blocks) {
+            const int grp = nblk / a.group_blocks;
+            n0 = grp * a.group_n + (nblk - grp * a.group_blocks) * BM;
+            n_end = (grp + 1) * a.group_n;
+        }
+    }
     const int lane = tid & 31, warp = tid >> 5;
     constexpr int NW = TC_THREADS / 32;
     if (a.epi == EPI_STORE) {
-        const bool vec = (a.ldy & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.resid) | reinterpret_cast<uintptr_t>(a.bias) | reinterpret_cast<uintptr_t>(a.out_scale)) & 15) == 0 && n0 + BM <= n_end && (n0 & 3) == 0;
+        const bool vec = (a.ldy & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.resid) | reinterpret_cast<uintptr_t>(a.bias)) & 15) == 0 && n0 + BM <= n_end && (!X || ((n0 & 3) == 0 && (reinterpret_cast<uintptr_t>(a.out_scale) & 15) == 0));
         if (vec) {
             // eight consecutive features per thread (one 16-byte chunk of the next GEMM's activation image); the 16
             // threads of a row are half a warp, which is where the row's sum of squares is reduced
@@ -270,13 +279,15 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                     const float4 t0 = *reinterpret_cast<const float4*>(tile + m * BM + c), t1 = *reinterpret_cast<const float4*>(tile + m * BM + c + 4);
                     v[0] = t0.x; v[1] = t0.y; v[2] = t0.z; v[3] = t0.w; v[4] = t1.x; v[5] = t1.y; v[6] = t1.z; v[7] = t1.w;
                 }
-                if (a.out_scale) {
-                    const float4 s0 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c)), s1 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c + 4));
-                    v[0] *= s0.x; v[1] *= s0.y; v[2] *= s0.z; v[3] *= s0.w; v[4] *= s1.x; v[5] *= s1.y; v[6] *= s1.z; v[7] *= s1.w;
-                }
-                if (a.split_xp && n0 + c < a.split_n) {  // 8-element pieces never straddle split_n or an image: both are multiples of 8
-                    if (ok) tc_xpack_store8(a.split_xp + (size_t)((n0 + c) / a.split_k) * a.split_bytes, a.xp_mpad, m, (n0 + c) % a.split_k, v);
-                    continue;
+                if constexpr (X) {
+                    if (a.out_scale) {
+                        const float4 s0 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c)), s1 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c + 4));
+                        v[0] *= s0.x; v[1] *= s0.y; v[2] *= s0.z; v[3] *= s0.w; v[4] *= s1.x; v[5] *= s1.y; v[6] *= s1.z; v[7] *= s1.w;
+                    }
+                    if (a.split_xp && n0 + c < a.split_n) {  // 8-element pieces never straddle split_n or an image: both are multiples of 8
+                        if (ok) tc_xpack_store8(a.split_xp + (size_t)((n0 + c) / a.split_k) * a.split_bytes, a.xp_mpad, m, (n0 + c) % a.split_k, v);
+                        continue;
+                    }
                 }
                 if (ok && a.resid) {
                     const float4 r0 = ld_cg_f32x4(a.resid + (size_t)m * a.ldy + n0 + c), r1 = ld_cg_f32x4(a.resid + (size_t)m * a.ldy + n0 + c + 4);
@@ -312,10 +323,12 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                 if (n < n_end) {
                     float v = tile[m * BM + c];
                     if (a.bias) v += __ldg(a.bias + n);
-                    if (a.out_scale) v *= __ldg(a.out_scale + n);
-                    if (a.split_xp && n < a.split_n) {
-                        tc_xpack_store(a.split_xp + (size_t)(n / a.split_k) * a.split_bytes, a.xp_mpad, m, n % a.split_k, v);
-                        continue;
+                    if constexpr (X) {
+                        if (a.out_scale) v *= __ldg(a.out_scale + n);
+                        if (a.split_xp && n < a.split_n) {
+                            tc_xpack_store(a.split_xp + (size_t)(n / a.split_k) * a.split_bytes, a.xp_mpad, m, n % a.split_k, v);
+                            continue;
+                        }
                     }
                     if (a.resid) v = a.resid[(size_t)m * a.ldy + n] + v;
                     a.y[(size_t)m * a.ldy + n] = v;
@@ -347,7 +360,7 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                 }
             }
         }
-    } else if (a.epi == EPI_GATE || a.epi == EPI_SQRELU) {
+    } else if (X && (a.epi == EPI_GATE || a.epi == EPI_SQRELU)) {
         auto act = [&](int m, int n, float v) {
             if (a.epi == EPI_GATE) return v / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + n)));
             v = fmaxf(v, 0.f);
@@ -477,7 +490,7 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
 }
 
 // ---- the GEMM: warp 0 = bulk-copy producer, warp 1 = TMEM owner + MMA issuer, warps 2-5 = epilogue ----
-template <bool CL>
+template <bool CL, bool X>
 __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) {
     extern __shared__ __align__(1024) unsigned char dsm[];
     __shared__ TcShared sh;
@@ -541,7 +554,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) 
     if (warp == 0) {
         if (lane == 0) {
             const unsigned char* wsrc = reinterpret_cast<const unsigned char*>(a.W) + ((size_t)nblk * kb_total + kb0) * W_TILE;
-            const unsigned char* xsrc = a.xp + (a.group_blocks ? (size_t)(nblk / a.group_blocks) * a.group_xp : 0) + (size_t)kb0 * x_tile;
+            const unsigned char* xsrc = a.xp + (X && a.group_blocks ? (size_t)(nblk / a.group_blocks) * a.group_xp : 0) + (size_t)kb0 * x_tile;
             // weights never depend on the previous kernel: fill the ring with them first, then wait for
             // the packed activations
             const int pre = min(nkb, nst);
@@ -675,7 +688,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) 
         __syncthreads();
     }
     HM_TRACE(if (tr && tid == 0) a.trace[8] = global_timer();)
-    tc_epilogue(a, out_tile, m_lo, m_hi, nblk, tid, sh.pos, sh.page);
+    tc_epilogue<X>(a, out_tile, m_lo, m_hi, nblk, tid, sh.pos, sh.page);
     HM_TRACE(if (tr && tid == 0) a.trace[9] = global_timer();)
     HM_TRACE(if (tr && tid == 0) a.trace[10] = global_timer();)
     HM_TRACE(if (a.trace && tid == 0) atomicMax(a.trace + 12, global_timer());)
@@ -741,7 +754,8 @@ cudaError_t launch_tc_pack_gnorm(const float* x, int ldx, int M, int K, const fl
     return cudaLaunchKernelEx(&cfg, tc_pack_gnorm_kernel, x, ldx, M, tc_mpad(M), K, Kp, norm_w, eps, gn, (unsigned char*)xp);
 }
 
-cudaError_t launch_gemm_tc(const TcArgs& a_in, cudaStream_t st, bool pdl) {
+template <bool X>
+static cudaError_t launch_gemm_tc_x(const TcArgs& a_in, cudaStream_t st, bool pdl) {
     TcArgs a = a_in;
     if (a.M < 1 || a.M > MR || a.Kp % BK != 0 || !a.xp) return cudaErrorInvalidValue;
     a.mpad = tc_mpad(a.M);
@@ -755,7 +769,7 @@ cudaError_t launch_gemm_tc(const TcArgs& a_in, cudaStream_t st, bool pdl) {
     const size_t smem = tc_smem_for(a.mpad, multi_wave) + (cl ? tc_recv_bytes(a.M, a.ksplit) : 0);
     {
         const size_t mx = (tc_smem_for(64, false) > tc_smem_for(32, false) ? tc_smem_for(64, false) : tc_smem_for(32, false)) + (cl ? (size_t)(MR + 16) * BM * 4 : 0);
-        cudaError_t e = cl ? ensure_dyn_smem(gemm_tc_kernel<true>, mx) : ensure_dyn_smem(gemm_tc_kernel<false>, mx);
+        cudaError_t e = cl ? ensure_dyn_smem(gemm_tc_kernel<true, X>, mx) : ensure_dyn_smem(gemm_tc_kernel<false, X>, mx);
         if (e != cudaSuccess) return e;
     }
     cudaLaunchConfig_t cfg = {};
@@ -773,7 +787,7 @@ cudaError_t launch_gemm_tc(const TcArgs& a_in, cudaStream_t st, bool pdl) {
     if (cl) {
         if (a.ksplit > 16) return cudaErrorInvalidValue;
         if (a.ksplit > 8) {  // clusters of 9..16 CTAs are allowed on request
-            cudaError_t e = ensure_nonportable_clusters(gemm_tc_kernel<true>);
+            cudaError_t e = ensure_nonportable_clusters(gemm_tc_kernel<true, X>);
             if (e != cudaSuccess) return e;
         }
         at[n].id = cudaLaunchAttributeClusterDimension;
@@ -784,7 +798,12 @@ cudaError_t launch_gemm_tc(const TcArgs& a_in, cudaStream_t st, bool pdl) {
     }
     cfg.attrs = at;
     cfg.numAttrs = n;
-    return cl ? cudaLaunchKernelEx(&cfg, gemm_tc_kernel<true>, a) : cudaLaunchKernelEx(&cfg, gemm_tc_kernel<false>, a);
+    return cl ? cudaLaunchKernelEx(&cfg, gemm_tc_kernel<true, X>, a) : cudaLaunchKernelEx(&cfg, gemm_tc_kernel<false, X>, a);
+}
+
+cudaError_t launch_gemm_tc(const TcArgs& a, cudaStream_t st, bool pdl) {
+    const bool x = a.group_blocks || a.out_scale || a.split_xp || a.epi == EPI_GATE || a.epi == EPI_SQRELU;
+    return x ? launch_gemm_tc_x<true>(a, st, pdl) : launch_gemm_tc_x<false>(a, st, pdl);
 }
 
 // ---- weight packing: [N][K] (HF [out,in]) or [K][N] bf16 -> swizzled K-major tiles ----------
