@@ -75,7 +75,7 @@ int Engine::create(const ModelSpec& spec, int device, bool strict_f32, Engine** 
         e->kvdim_ = 0;
         e->qdim_ = 0;
         for (const LayerSpec& l : spec.layers) {
-            e->qdim_ = std::max(e->qdim_, l.heads * l.vdim);
+            e->qdim_ = std::max(e->qdim_, l.heads * std::max(l.vdim, l.mixer == MIX_GQA ? l.dim : 0));
             if (l.kv_rank > 1024) return bad("kv_rank must be at most 1024");
         }
     } else {
@@ -110,7 +110,9 @@ Engine::~Engine() {
     };
     fr(embed_); fr(final_norm_); fr(rope_cos_); fr(rope_sin_);
     for (auto& l : layers_)
-        for (float* p : {l.in_ln, l.post_ln, l.qkv_bias, l.q_norm, l.k_norm, l.shift, l.ls1, l.ls2, l.latent_norm}) fr(p);
+        for (float* p : {l.in_ln, l.post_ln, l.qkv_bias, l.q_norm, l.k_norm, l.shift, l.ls1, l.ls2, l.latent_norm, l.v_mix, l.rel, l.correction}) fr(p);
+    for (auto& l : layers_) { fr(l.router); fr(l.exp_gu); fr(l.exp_down); }
+    fr(turns_);
     each_linear([&](LinearW& w) { fr(w.slabs); fr(w.tc); fr(w.scales); fr(w.codes); fr(w.kq_data); fr(w.kq_tile_type); });
     free_listed();
     free_listed_cache();
@@ -265,7 +267,7 @@ static bool parse_layer_name(const std::string& name, const char* prefix, int* l
 int Engine::load_tensor(const char* cname, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes) {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (finalized_) return fail(HM_ERR_STATE, "weights already finalised");
-    if (!cname || !shape || !host || ndim < 1 || ndim > 2) return fail(HM_ERR_INVALID, "load_tensor: bad arguments");
+    if (!cname || (!shape && ndim > 0) || !host || ndim < 0 || ndim > 2) return fail(HM_ERR_INVALID, "load_tensor: bad arguments");
     const std::string name(cname);
     size_t n = 1;
     for (int i = 0; i < ndim; ++i) {
@@ -400,6 +402,13 @@ int Engine::finalize() {
         HM_CUDA(cudaMemcpy(rope_cos_, c.data(), c.size() * 4, cudaMemcpyHostToDevice));
         HM_CUDA(cudaMemcpy(rope_sin_, s.data(), s.size() * 4, cudaMemcpyHostToDevice));
     }
+    if (spec_.sin_pos) {
+        // pair i of the position vector turns by 10000^(-2 i / width) radians per position
+        std::vector<double> t((H_ + 1) / 2);
+        for (size_t i = 0; i < t.size(); ++i) t[i] = std::pow(10000.0, -2.0 * (double)i / H_) / 6.283185307179586;
+        HM_CUDA(cudaMalloc(&turns_, t.size() * 8));
+        HM_CUDA(cudaMemcpy(turns_, t.data(), t.size() * 8, cudaMemcpyHostToDevice));
+    }
     HM_CUDA(cudaMalloc(&err_flag_, 4));
     HM_CUDA(cudaMemset(err_flag_, 0, 4));
     HM_CUDA(cudaMalloc(&fin_ticket_, 4));
@@ -496,6 +505,7 @@ int Engine::kv_alloc(int batch, int max_seq_len, int page_tokens, int kv_dtype, 
     if (!finalized_) return fail(HM_ERR_STATE, "kv_alloc before weights are finalised");
     if (batch_ > 0) return fail(HM_ERR_STATE, "KV cache already allocated");
     if (batch < 1 || max_seq_len < 1) return fail(HM_ERR_INVALID, "kv_alloc: batch and max_seq_len must be positive");
+    static_assert(LATENT_PAGE == GQA_PAGE, "listed designs share one page size");
     const int native = spec_.listed() ? LATENT_PAGE : 16;
     if (page_tokens == 0) page_tokens = native;
     if (page_tokens != native) return fail(HM_ERR_UNSUPPORTED, "kv_alloc: page size must be " + std::to_string(native) + " tokens");
@@ -675,7 +685,7 @@ int Engine::kv_append(int seq, int layer, const float* k_rows, const float* v_ro
     if (seq < 0 || seq >= batch_ || layer < 0 || layer >= L_ || n_new < 0) return fail(HM_ERR_INVALID, "kv_append: index out of range");
     if (len_[seq] + n_new > max_seq_)
         return fail(HM_ERR_KV_FULL, "KV cache full (" + std::to_string(len_[seq]) + " + " + std::to_string(n_new) + " > " + std::to_string(max_seq_) + ")");
-    if (spec_.listed() && (k_rows || v_rows)) return fail(HM_ERR_UNSUPPORTED, "kv_append: this design caches latents, not keys and values");
+    if (spec_.listed() && (k_rows || v_rows)) return fail(HM_ERR_UNSUPPORTED, "kv_append: rows of keys and values belong to the uniform stacks");
     {
         const int prc = ensure_pages({{seq, (long)len_[seq] + n_new}});
         if (prc) return prc;
@@ -709,17 +719,18 @@ int Engine::kv_view(int seq, int layer, float* k_out, float* v_out) {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (batch_ == 0) return fail(HM_ERR_STATE, "kv_view before kv_alloc");
     if (seq < 0 || seq >= batch_ || layer < 0 || layer >= L_ || !k_out || !v_out) return fail(HM_ERR_INVALID, "kv_view: bad arguments");
-    if (spec_.listed()) return fail(HM_ERR_UNSUPPORTED, "kv_view: this design caches latents, not keys and values (hm_latent_view)");
+    const LayerSpec* ls = spec_.listed() ? &spec_.layers[layer] : nullptr;
+    if (ls && ls->mixer == MIX_LATENT) return fail(HM_ERR_UNSUPPORTED, "kv_view: this design caches latents, not keys and values (hm_latent_view)");
     const int len = len_[seq];
     if (len == 0) return HM_OK;
-    const size_t bytes = (size_t)kvh_ * len * hd_ * 4;
+    const size_t k_bytes = (size_t)(ls ? ls->kv_heads * ls->dim : kvh_ * hd_) * len * 4, v_bytes = (size_t)(ls ? ls->kv_heads * ls->vdim : kvh_ * hd_) * len * 4;
     float *dk = nullptr, *dv = nullptr;
-    HM_CUDA(cudaMalloc(&dk, bytes));
-    HM_CUDA(cudaMalloc(&dv, bytes));
+    HM_CUDA(cudaMalloc(&dk, k_bytes));
+    HM_CUDA(cudaMalloc(&dv, v_bytes));
     KvDesc kv{k_pool_[layer], v_pool_[layer], page_table_, max_pages_, page_tokens_, kvh_, hd_, kv_bf16_ ? 1 : 0};
-    cudaError_t ce = launch_kv_read_rows(kv, seq, len, dk, dv, stream_);
-    if (ce == cudaSuccess) ce = cudaMemcpyAsync(k_out, dk, bytes, cudaMemcpyDeviceToHost, stream_);
-    if (ce == cudaSuccess) ce = cudaMemcpyAsync(v_out, dv, bytes, cudaMemcpyDeviceToHost, stream_);
+    cudaError_t ce = ls ? launch_gqa_read(gqa_pool(layer), seq, len, dk, dv, stream_) : launch_kv_read_rows(kv, seq, len, dk, dv, stream_);
+    if (ce == cudaSuccess) ce = cudaMemcpyAsync(k_out, dk, k_bytes, cudaMemcpyDeviceToHost, stream_);
+    if (ce == cudaSuccess) ce = cudaMemcpyAsync(v_out, dv, v_bytes, cudaMemcpyDeviceToHost, stream_);
     if (ce == cudaSuccess) ce = cudaStreamSynchronize(stream_);
     cudaFree(dk);
     cudaFree(dv);
@@ -731,6 +742,7 @@ int Engine::kv_view(int seq, int layer, float* k_out, float* v_out) {
 
 static const char* kProfNames[PC_COUNT] = {"embed", "qkv_rope_kvwrite", "attention", "o_proj_residual", "gate_up_swiglu", "down_residual", "lm_head", "argmax"};
 static const char* kProfNamesListed[PC_COUNT_LISTED] = {"embed", "in_proj", "attention", "o_proj_residual", "up_sqrelu", "down_residual", "lm_head", "argmax", "latent_write", "key_up", "value_up_gate"};
+static const char* kProfNamesGqa[PC_COUNT_LISTED] = {"embed", "qkv_proj", "attention", "o_proj", "experts_gate_up", "experts_down", "lm_head", "argmax", nullptr, nullptr, nullptr, "qk_norm_kv_write", "post_norm_router", "post_norm"};
 
 void Engine::prof_mark(int) {}
 
@@ -1073,7 +1085,7 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
     }
     auto want = [&](int cls) { return only_class_ < 0 || only_class_ == cls; };
     if (want(PC_EMBED)) {
-        ce = launch_embed_gather(embed_, embed_dtype_ == HM_BF16 ? 1 : 0, tokens_dev, M, H_, V_, h_, err_flag_, stream_, pdl_);
+        ce = launch_embed_gather(embed_, embed_dtype_ == HM_BF16 ? 1 : 0, tokens_dev, M, H_, V_, h_, err_flag_, stream_, pdl_, turns_, row_pos);
         if (ce != cudaSuccess) return cuda_fail(ce, "embed_gather");
         ++*launches;
     }
@@ -1101,7 +1113,7 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
     const bool fused = direct_pack && H_ % 128 == 0;
     for (int l = 0; l < L_; ++l) {
         if (spec_.listed()) {
-            rc = enqueue_listed_layer(l, M, row_pos, row_seq, lm_rows, launches);
+            rc = spec_.layers[l].mixer == MIX_GQA ? enqueue_gqa_layer(l, M, row_pos, row_seq, lm_rows, launches) : enqueue_listed_layer(l, M, row_pos, row_seq, lm_rows, launches);
             if (rc) return rc;
             rc = tap(l, M);
             if (rc) return rc;
@@ -1621,7 +1633,7 @@ int Engine::time_decode(int warmup, int steps, float* ms_total) {
 int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (batch_ == 0) return fail(HM_ERR_STATE, "profile_decode before kv_alloc");
-    if (steps < 1 || !out || !n_out || cap < (spec_.listed() ? PC_COUNT_LISTED : PC_COUNT)) return fail(HM_ERR_INVALID, "profile_decode: bad arguments (cap >= 8; 11 for listed designs)");
+    if (steps < 1 || !out || !n_out || cap < (spec_.listed() ? PC_COUNT_LISTED : PC_COUNT)) return fail(HM_ERR_INVALID, "profile_decode: bad arguments (cap >= 8; 14 for listed designs)");
     for (int b = 0; b < batch_; ++b)
         if (len_[b] + steps > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full: not enough room for the profiled steps");
     if (const int prc = ensure_pages_all(steps)) return prc;
@@ -1675,6 +1687,10 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
     bytes[PC_EMBED] = (uint64_t)batch_ * H_ * (embed_dtype_ == HM_BF16 ? 2 : 4);
     for (auto& l : layers_) {
         bytes[PC_QKV] += l.qkv.bytes() + l.in.bytes();
+        const int li = (int)(&l - layers_.data());
+        bytes[PC_ROUTE] += l.router ? (uint64_t)(spec_.layers[li].experts + spec_.layers[li].identity) * H_ * 2 : 0;
+        bytes[PC_GATE_UP] += expert_bytes(li, batch_, true);
+        bytes[PC_DOWN] += expert_bytes(li, batch_, false);
         bytes[PC_KUP] += l.kup.bytes();
         bytes[PC_VUP] += l.vup.bytes();
         bytes[PC_O] += l.o.bytes();
@@ -1683,18 +1699,22 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
     }
     bytes[PC_LM_HEAD] = lm_head_.bytes();
     if (spec_.listed()) {
-        for (const LayerSpec& l : spec_.layers) bytes[PC_ATTN] += (uint64_t)(kv_tokens * l.kv_rank * (kv_bf16_ ? 2 : 4));
+        for (const LayerSpec& l : spec_.layers) bytes[PC_ATTN] += (uint64_t)(kv_tokens * (l.mixer == MIX_LATENT ? l.kv_rank : l.kv_heads * (l.dim + l.vdim)) * (kv_bf16_ ? 2 : 4));
     } else {
         bytes[PC_ATTN] = (uint64_t)(kv_tokens * L_ * 2.0 * kvh_ * hd_ * (kv_bf16_ ? 2 : 4));
     }
+    const char* const* names = !spec_.listed() ? kProfNames : spec_.post_norm ? kProfNamesGqa : kProfNamesListed;
+    int n = 0;
     for (int c = 0; c < classes; ++c) {
-        std::memset(&out[c], 0, sizeof(out[c]));
-        std::strncpy(out[c].name, spec_.listed() ? kProfNamesListed[c] : kProfNames[c], sizeof(out[c].name) - 1);
-        out[c].launches_per_step = count[c];
-        out[c].ms_per_step = ms[c] / steps;
-        out[c].bytes_per_step = bytes[c];
+        if (!names[c]) continue;
+        std::memset(&out[n], 0, sizeof(out[n]));
+        std::strncpy(out[n].name, names[c], sizeof(out[n].name) - 1);
+        out[n].launches_per_step = count[c];
+        out[n].ms_per_step = ms[c] / steps;
+        out[n].bytes_per_step = bytes[c];
+        ++n;
     }
-    *n_out = classes;
+    *n_out = n;
     return HM_OK;
 }
 

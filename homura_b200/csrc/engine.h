@@ -12,7 +12,9 @@
 
 #include "../../include/homura_b200.h"
 #include "common.cuh"
+#include "gqa_attn.h"
 #include "latent_attn.h"
+#include "moe.h"
 #include "model_spec.h"
 #include "sampler.h"
 
@@ -53,6 +55,15 @@ struct LayerW {
     float* latent_norm = nullptr;        // [kv_rank]
     LinearW in;                          // queries, output gate and (unless another layer's latents are used) latents, parts padded to 128 columns
     LinearW kup, vup;                    // per head: query -> latent space, latent space -> values
+    // listed grouped-query attention: `in` is queries, keys and values without padding
+    float* v_mix = nullptr;              // share of the first such layer's values
+    float* rel = nullptr;                // distance bias [heads][reach + 1]
+    int reach = 0;
+    // mixture of experts
+    uint16_t* router = nullptr;          // [experts + identity][H] bf16
+    float* correction = nullptr;
+    uint16_t *exp_gu = nullptr, *exp_down = nullptr;  // all experts' tile images (moe.h)
+    std::vector<uint8_t> exp_seen;       // per expert: bits of the parts loaded
 };
 
 // What a projection launch needs beyond the common arguments (enqueue_linear)
@@ -137,6 +148,18 @@ class Engine {
     // more per row, so theirs move over earlier.
     bool tall_rows(int rows) const { return use_tc_ && rows > (spec_.listed() ? 4 : MAX_M); }
     int enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int next_lm_rows, int* launches);
+    // listed grouped-query attention, post-norms, mixtures of experts (engine_gqa.cu)
+    int load_gqa_tensor(LayerW& w, const LayerSpec& s, const std::string& name, const std::string& rest, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
+    int load_bias_table(LayerW& w, const LayerSpec& s, int dtype, const int64_t* shape, const void* host, size_t nbytes);
+    int load_expert(LayerW& w, const LayerSpec& s, int expert, int part, int dtype, const void* host, size_t nbytes);
+    int finalize_gqa(const LayerW& w, const LayerSpec& s, const std::string& at);
+    int alloc_gqa_scratch();
+    void free_gqa_scratch();
+    GqaPool gqa_pool(int layer) const;
+    RouteOut route_out(const LayerSpec& s) const;
+    ExpertWeights expert_weights(int layer) const;
+    uint64_t expert_bytes(int layer, int rows, bool gate_up) const;
+    int enqueue_gqa_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int next_lm_rows, int* launches);
     int enqueue_listed_logits(const float* x, int rows, float* dst, const struct ArgmaxFold& fold, int* launches);
     int enqueue_tc(const LinearW& L, int M, const unsigned char* xp, int epi, float* y, int ldy, TcArgs& a, int* launches);
     LatentPool latent_pool(int layer) const;
@@ -226,6 +249,13 @@ class Engine {
     size_t lat_acc_floats_ = 0, lat_ml_floats_ = 0;
     std::vector<void*> lat_pool_;  // per layer, null for layers that read another's
     float *shift_state_ = nullptr, *shift_saved_ = nullptr;  // [layers][sequences][SHIFT_RING][H]; [layers][SHIFT_RING][H]
+    double* turns_ = nullptr;        // sinusoidal positions: turns per position of every pair of elements
+    float* sub_ = nullptr;           // what a sublayer gave back, before its norm
+    float* v_first_ = nullptr;       // values of the layer that the others blend in
+    int32_t* rt_ids_ = nullptr;      // router's choice (RouteOut)
+    float *rt_weights_ = nullptr, *rt_identity_ = nullptr, *rt_dense_ = nullptr;
+    uint32_t* rt_mask_ = nullptr;
+    float* exp_act_ = nullptr;       // activations of the chosen experts
     int32_t* seq_iota_ = nullptr;    // 0, 1, 2, ...: the sequence of every row of a decode step
     int pass_nsplit_ = 1;            // splits the attention of the layer being enqueued left for the next projection to combine
     int pass_longest_ = 0;           // longest context of the pass being enqueued (splits of the attention)

@@ -1,0 +1,353 @@
+// Engine parts for listed designs with grouped-query attention whose sublayers read the residual itself and normalise what they
+// give back: weights, scratch, and the launches of one layer.  Beside engine_listed.cu, which holds what all listed designs share.
+//
+// A layer with a mixture of experts is, per pass,
+//   in      [queries | keys | values]  <- residual
+//   post    query and key norms, temperature, blended values; page slots            (gqa_attn.cu)
+//   attn    softmax attention with distance biases                                  (gqa_attn.cu)
+//   o       output projection
+//   norm    residual += mult * norm(o); router over the new residual                (moe.cu)
+//   experts gate and up, down
+//   norm    residual += mult * norm(experts + identity)
+#include <algorithm>
+#include <cmath>
+#include <cstdlib>
+#include <cstring>
+
+#include "engine.h"
+#include "engine_util.h"
+#include "gemm_tc.h"
+
+namespace hm {
+
+namespace {
+int qkv_cols(const LayerSpec& s) { return s.heads * s.dim + s.kv_heads * (s.dim + s.vdim); }
+int qkv_ld(const LayerSpec& s) { return (qkv_cols(s) + 3) / 4 * 4; }
+
+// Row of the bias table for a key n tokens back: a row per distance below half the table, then logarithmic steps up to `reach`.
+int distance_row(int n, int rows, double reach) {
+    const int half = rows / 2;
+    if (n < half) return n;
+    if (n >= reach || reach <= half || half == 0) return rows - 1;
+    // (a distance that lies exactly on a step belongs to the step's upper side)
+    const int r = half + (int)std::floor(std::log((double)n / half) / std::log(reach / half) * (rows - half) + 1e-9);
+    return std::min(rows - 1, r);
+}
+}  // namespace
+
+// ---- weights -------------------------------------------------------------------------------------
+
+// [rows, heads] by bucket -> [heads][reach + 1] by distance, in units of the base-2 exponent.
+int Engine::load_bias_table(LayerW& w, const LayerSpec& s, int dtype, const int64_t* shape, const void* host, size_t nbytes) {
+    const int rows = (int)shape[0];
+    const size_t n = (size_t)rows * s.heads;
+    if ((dtype != HM_BF16 && dtype != HM_F32) || nbytes != n * (dtype == HM_BF16 ? 2 : 4)) return fail(HM_ERR_UNSUPPORTED, "distance biases must be stored as bf16 or f32");
+    auto at = [&](int r, int h) {
+        const size_t i = (size_t)r * s.heads + h;
+        if (dtype == HM_F32) return static_cast<const float*>(host)[i];
+        const uint32_t u = (uint32_t)static_cast<const uint16_t*>(host)[i] << 16;
+        float f;
+        std::memcpy(&f, &u, 4);
+        return f;
+    };
+    w.reach = std::max((int)std::ceil(s.bias_reach), rows / 2);
+    std::vector<float> t((size_t)s.heads * (w.reach + 1));
+    for (int d = 0; d <= w.reach; ++d) {
+        const int r = distance_row(d, rows, s.bias_reach);
+        for (int h = 0; h < s.heads; ++h) t[(size_t)h * (w.reach + 1) + d] = (float)(at(r, h) * 1.4426950408889634);
+    }
+    HM_CUDA(cudaMalloc(&w.rel, t.size() * 4));
+    HM_CUDA(cudaMemcpy(w.rel, t.data(), t.size() * 4, cudaMemcpyHostToDevice));
+    return HM_OK;
+}
+
+// part 0 = gate, 1 = up, 2 = down
+int Engine::load_expert(LayerW& w, const LayerSpec& s, int expert, int part, int dtype, const void* host, size_t nbytes) {
+    if (dtype != HM_BF16) return fail(HM_ERR_UNSUPPORTED, "experts of this design must be stored as bf16");
+    if (nbytes != (size_t)s.ff * H_ * 2) return fail(HM_ERR_INVALID, "tensor byte size does not match its shape");
+    const size_t gu = expert_gu_elems(H_, s.ff), down = expert_down_elems(H_, s.ff);
+    auto room = [&](uint16_t** p, size_t elems) -> cudaError_t {
+        if (*p) return cudaSuccess;
+        const cudaError_t e = cudaMalloc(p, elems * 2);
+        return e == cudaSuccess ? cudaMemsetAsync(*p, 0, elems * 2, stream_) : e;
+    };
+    cudaError_t ce = part < 2 ? room(&w.exp_gu, s.experts * gu) : room(&w.exp_down, s.experts * down);
+    if (ce != cudaSuccess) return cuda_fail(ce, "experts");
+    void* tmp = nullptr;
+    const int rc = stage(host, nbytes, &tmp);
+    if (rc) return rc;
+    const uint16_t* src = static_cast<const uint16_t*>(tmp);
+    ce = part < 2 ? launch_pack_tc(src, s.ff, H_, false, w.exp_gu + expert * gu, 0, part, stream_) : launch_pack_tc(src, H_, s.ff, false, w.exp_down + expert * down, 0, -1, stream_);
+    if (ce == cudaSuccess) ce = cudaStreamSynchronize(stream_);
+    cudaFree(tmp);
+    if (ce != cudaSuccess) return cuda_fail(ce, "load_expert");
+    w.exp_seen.resize(s.experts, 0);
+    w.exp_seen[expert] |= (uint8_t)(1 << part);
+    cfg_.weight_dtype = HM_BF16;
+    return HM_OK;
+}
+
+int Engine::load_gqa_tensor(LayerW& w, const LayerSpec& s, const std::string& name, const std::string& rest, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes) {
+    size_t n = 1;
+    for (int i = 0; i < ndim; ++i) n *= (size_t)shape[i];
+    auto is2 = [&](int64_t a, int64_t b) { return ndim == 2 && shape[0] == a && shape[1] == b; };
+    auto bad_shape = [&]() { return fail(HM_ERR_INVALID, "unexpected shape for tensor " + name); };
+    auto twice = [&]() { return fail(HM_ERR_STATE, "tensor loaded twice: " + name); };
+    auto vec = [&](float** dst, int len) {
+        if (n != (size_t)len || ndim > 1) return bad_shape();
+        return *dst ? twice() : load_vec_f32(dst, len, 0, dtype, host, n, nbytes);
+    };
+    auto lin = [&](LinearW& L, int K, int total, int off, int part) { return is2(part, K) ? load_linear(L, K, total, off, part, -1, dtype, host, nbytes) : bad_shape(); };
+    const int nq = s.heads * s.dim, nk = s.kv_heads * s.dim, nv = s.kv_heads * s.vdim;
+    if (rest == "mix.q") return lin(w.in, H_, qkv_cols(s), 0, nq);
+    if (rest == "mix.k") return lin(w.in, H_, qkv_cols(s), nq, nk);
+    if (rest == "mix.v") return lin(w.in, H_, qkv_cols(s), nq + nk, nv);
+    if (rest == "mix.o") return lin(w.o, s.heads * s.vdim, H_, 0, H_);
+    if (rest == "mix.q.norm" && s.qk_norm != QKN_NONE) return vec(&w.q_norm, s.qk_norm == QKN_ALL ? nq : s.dim);
+    if (rest == "mix.k.norm" && s.qk_norm != QKN_NONE) return vec(&w.k_norm, s.qk_norm == QKN_ALL ? nk : s.dim);
+    if (rest == "mix.vmix") return vec(&w.v_mix, 1);
+    if (rest == "mix.rel" && s.bias_reach > 0) {
+        if (ndim != 2 || shape[1] != s.heads) return bad_shape();
+        return w.rel ? twice() : load_bias_table(w, s, dtype, shape, host, nbytes);
+    }
+    if (s.mlp == MLP_MOE) {
+        const int outs = s.experts + s.identity;
+        if (rest == "mlp.correction") return vec(&w.correction, outs);
+        if (rest == "mlp.router") {
+            if (!is2(outs, H_)) return bad_shape();
+            if (dtype != HM_BF16 || nbytes != n * 2) return fail(HM_ERR_UNSUPPORTED, "the router of this design must be stored as bf16");
+            if (w.router) return twice();
+            const int rc = stage(host, nbytes, reinterpret_cast<void**>(&w.router));
+            if (rc) return rc;
+            HM_CUDA(cudaStreamSynchronize(stream_));
+            return HM_OK;
+        }
+        const size_t dot = rest.find('.', 5);
+        if (rest.compare(0, 5, "mlp.e") == 0 && dot != std::string::npos && dot > 5 && rest.find_first_not_of("0123456789", 5) == dot) {
+            const long e = std::atol(rest.c_str() + 5);
+            const std::string what = rest.substr(dot + 1);
+            const int part = what == "gate" ? 0 : what == "up" ? 1 : what == "down" ? 2 : -1;
+            if (part >= 0) {
+                if (e >= s.experts) return fail(HM_ERR_INVALID, "expert index out of range in " + name);
+                if (!(part < 2 ? is2(s.ff, H_) : is2(H_, s.ff))) return bad_shape();
+                if ((size_t)e < w.exp_seen.size() && (w.exp_seen[e] >> part & 1)) return twice();
+                return load_expert(w, s, (int)e, part, dtype, host, nbytes);
+            }
+        }
+    }
+    return fail(HM_ERR_INVALID, "unknown tensor name: " + name);
+}
+
+int Engine::finalize_gqa(const LayerW& w, const LayerSpec& s, const std::string& at) {
+    if (w.in.loaded_parts != 3) return fail(HM_ERR_STATE, at + "mix.q / mix.k / mix.v");
+    if (w.o.loaded_parts != 1) return fail(HM_ERR_STATE, at + "mix.o");
+    if (s.qk_norm != QKN_NONE && (!w.q_norm || !w.k_norm)) return fail(HM_ERR_STATE, at + "mix.q.norm / mix.k.norm");
+    if (s.bias_reach > 0 && !w.rel) return fail(HM_ERR_STATE, at + "mix.rel");
+    if (s.v_first >= 0 && &w != &layers_[s.v_first] && !w.v_mix) return fail(HM_ERR_STATE, at + "mix.vmix");
+    if (s.mlp != MLP_MOE) return HM_OK;
+    if (!w.post_ln) return fail(HM_ERR_STATE, at + "norm2");
+    if (!w.router || !w.correction) return fail(HM_ERR_STATE, at + "mlp.router / mlp.correction");
+    for (int e = 0; e < s.experts; ++e)
+        if ((size_t)e >= w.exp_seen.size() || w.exp_seen[e] != 7) return fail(HM_ERR_STATE, at + "mlp.e" + std::to_string(e));
+    return HM_OK;
+}
+
+// ---- scratch ---------------------------------------------------------------------------------------
+
+void Engine::free_gqa_scratch() {
+    auto fr = [](auto*& p) {
+        if (p) cudaFree(p);
+        p = nullptr;
+    };
+    fr(sub_); fr(v_first_); fr(rt_ids_); fr(rt_weights_); fr(rt_identity_); fr(rt_dense_); fr(rt_mask_); fr(exp_act_);
+}
+
+// A pass of a listed design has at most TC_ROWS rows.
+int Engine::alloc_gqa_scratch() {
+    if (!spec_.post_norm) return HM_OK;
+    size_t values = 1, top = 1, experts = 1, act = 1;
+    for (const LayerSpec& s : spec_.layers) {
+        if (s.v_mix) values = std::max(values, (size_t)s.kv_heads * s.vdim);
+        if (s.mlp != MLP_MOE) continue;
+        top = std::max(top, (size_t)s.top);
+        experts = std::max(experts, (size_t)s.experts);
+        act = std::max(act, (size_t)s.top * expert_blocks(s.ff) * 64);
+    }
+    auto get = [&](auto** p, size_t count) -> cudaError_t {
+        const cudaError_t e = cudaMalloc((void**)p, count * sizeof(**p));
+        return e == cudaSuccess ? cudaMemset(*p, 0, count * sizeof(**p)) : e;
+    };
+    HM_CUDA(get(&sub_, (size_t)TC_ROWS * H_));
+    HM_CUDA(get(&v_first_, TC_ROWS * values));
+    HM_CUDA(get(&rt_ids_, TC_ROWS * top));
+    HM_CUDA(get(&rt_weights_, TC_ROWS * top));
+    HM_CUDA(get(&rt_identity_, TC_ROWS));
+    HM_CUDA(get(&rt_dense_, TC_ROWS * experts));
+    HM_CUDA(get(&rt_mask_, TC_ROWS * ((experts + 31) / 32)));
+    HM_CUDA(get(&exp_act_, TC_ROWS * act));
+    return HM_OK;
+}
+
+GqaPool Engine::gqa_pool(int layer) const {
+    const LayerSpec& s = spec_.layers[layer];
+    return GqaPool{k_pool_[layer], v_pool_[layer], page_table_, max_pages_, s.kv_heads, s.dim, s.vdim, kv_bf16_ ? 1 : 0};
+}
+
+RouteOut Engine::route_out(const LayerSpec&) const { return RouteOut{rt_ids_, rt_weights_, rt_identity_, nullptr, rt_mask_}; }
+
+ExpertWeights Engine::expert_weights(int layer) const {
+    const LayerSpec& s = spec_.layers[layer];
+    return ExpertWeights{layers_[layer].exp_gu, layers_[layer].exp_down, H_, s.ff, s.top, s.limit};
+}
+
+// Bytes of expert weights that a step over so many rows reads, if its choices are spread evenly.
+uint64_t Engine::expert_bytes(int layer, int rows, bool gate_up) const {
+    if (!spec_.listed() || spec_.layers[layer].mlp != MLP_MOE) return 0;
+    const LayerSpec& s = spec_.layers[layer];
+    const double outs = s.experts + s.identity, used = s.experts * (1.0 - std::pow(1.0 - s.top / outs, rows));
+    return (uint64_t)(used * (gate_up ? 2.0 : 1.0) * s.ff * H_ * 2.0);
+}
+
+// ---- one layer ---------------------------------------------------------------------------------------
+
+int Engine::enqueue_gqa_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int next_lm_rows, int* launches) {
+    const LayerW& w = layers_[l];
+    const LayerSpec& s = spec_.layers[l];
+    const float eps = (float)cfg_.rms_norm_eps;
+    const bool tall = tall_rows(M);
+    auto want = [&](int cls) { return only_class_ < 0 || only_class_ == cls; };
+    auto prefetch = [&](const LinearW* n) {  // weights of the kernel two launches ahead (streaming passes)
+        pf_ptr_ = nullptr;
+        pf_bytes_ = 0;
+        if (!use_prefetch_ || tall || only_class_ >= 0 || !n || !n->slabs) return;
+        pf_ptr_ = n->slabs;
+        pf_bytes_ = std::min(n->bytes(), (size_t)24 << 20);
+    };
+    cudaError_t ce;
+    int rc = HM_OK;
+    if (want(PC_QKV)) {
+        if (tall) {
+            if (l == 0) {  // later layers find the residual's image where the norm in front left it
+                ce = launch_tc_pack_x(h_, H_, M, H_, nullptr, 0.f, xpack_, stream_, pdl_);
+                if (ce != cudaSuccess) return cuda_fail(ce, "activation pack launch");
+                ++*launches;
+            }
+            TcArgs a{};
+            rc = enqueue_tc(w.in, M, xpack_, EPI_STORE, mix_raw_, qkv_ld(s), a, launches);
+        } else {
+            prefetch(&w.o);
+            rc = enqueue_linear(w.in, M, h_, H_, PRO_PLAIN, nullptr, EPI_STORE, mix_raw_, qkv_ld(s), nullptr, nullptr, l, row_pos, row_seq, nullptr, nullptr, launches);
+        }
+        if (rc) return rc;
+    }
+    if (want(PC_KV_WRITE)) {
+        GqaPostArgs a{};
+        a.pool = gqa_pool(l);
+        a.raw = mix_raw_;
+        a.ld = qkv_ld(s);
+        a.M = M;
+        a.heads = s.heads;
+        a.qk_norm = s.qk_norm;
+        a.q_norm = w.q_norm;
+        a.k_norm = w.k_norm;
+        a.eps = eps;
+        a.q_scale = (float)(s.scale * 1.4426950408889634);
+        a.temp_coef = s.temp_coef;
+        a.temp_every = s.temp_every;
+        a.v_first = s.v_first >= 0 ? v_first_ : nullptr;
+        a.v_lambda = s.v_first >= 0 && s.v_first != l ? w.v_mix : nullptr;
+        a.row_pos = row_pos;
+        a.row_seq = row_seq;
+        a.q_out = q_;
+        ce = launch_gqa_post(a, stream_, pdl_);
+        if (ce != cudaSuccess) return cuda_fail(ce, "query / key norm launch");
+        ++*launches;
+    }
+    if (want(PC_ATTN)) {
+        GqaAttnArgs a{};
+        a.pool = gqa_pool(l);
+        a.q = q_;
+        a.M = M;
+        a.heads = s.heads;
+        a.row_pos = row_pos;
+        a.row_seq = row_seq;
+        a.bias = w.rel;
+        a.reach = w.reach;
+        a.longest_run = 1;
+        for (auto& r : pass_runs_) {
+            a.runs.row[a.runs.n++] = (uint8_t)r.first;
+            a.longest_run = std::max(a.longest_run, r.second);
+        }
+        a.runs.row[a.runs.n] = (uint8_t)M;
+        a.longest = pass_longest_;
+        a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
+        a.max_cluster = use_clusters_ ? std::min(max_cluster_, 16) : 1;
+        a.out = attn_;
+        if (tall) {
+            a.xp = xpack_attn_;
+            a.xp_mpad = tc_mpad(M);
+        }
+        a.err_flag = err_flag_;
+        ce = launch_gqa_attn(a, sm_count_, stream_, pdl_);
+        if (ce != cudaSuccess) return cuda_fail(ce, "attention launch");
+        ++*launches;
+    }
+    if (want(PC_O)) {
+        if (tall) {
+            TcArgs a{};
+            rc = enqueue_tc(w.o, M, xpack_attn_, EPI_STORE, sub_, H_, a, launches);
+        } else {
+            rc = enqueue_linear(w.o, M, attn_, s.heads * s.vdim, PRO_PLAIN, nullptr, EPI_STORE, sub_, H_, nullptr, nullptr, l, row_pos, row_seq, nullptr, nullptr, launches);
+        }
+        if (rc) return rc;
+    }
+    PostNormArgs pn{};
+    pn.y = sub_;
+    pn.x = h_;
+    pn.M = M;
+    pn.W = H_;
+    pn.mult = spec_.residual_mult;
+    pn.eps = eps;
+    if (tall) {
+        pn.xp = xpack_;
+        pn.xp_mpad = tc_mpad(M);
+    }
+    const bool moe = s.mlp == MLP_MOE;
+    if (want(moe ? PC_ROUTE : PC_NORM)) {
+        PostNormArgs a = pn;
+        a.w = w.in_ln;
+        if (moe) {
+            a.router = w.router;
+            a.correction = w.correction;
+            a.experts = s.experts;
+            a.n_out = s.experts + s.identity;
+            a.top = s.top;
+            a.out = route_out(s);
+        }
+        ce = launch_post_norm(a, sm_count_, stream_, pdl_);
+        if (ce != cudaSuccess) return cuda_fail(ce, "norm launch");
+        ++*launches;
+    }
+    if (!moe) return HM_OK;
+    if (want(PC_GATE_UP)) {
+        ce = launch_expert_gate_up(expert_weights(l), h_, M, route_out(s), exp_act_, stream_, pdl_);
+        if (ce != cudaSuccess) return cuda_fail(ce, "expert gate / up launch");
+        ++*launches;
+    }
+    if (want(PC_DOWN)) {
+        ce = launch_expert_down(expert_weights(l), exp_act_, M, route_out(s), sub_, stream_, pdl_);
+        if (ce != cudaSuccess) return cuda_fail(ce, "expert down launch");
+        ++*launches;
+    }
+    if (want(PC_NORM)) {
+        PostNormArgs a = pn;
+        a.w = w.post_ln;
+        a.identity = s.identity > 0 ? rt_identity_ : nullptr;
+        ce = launch_post_norm(a, sm_count_, stream_, pdl_);
+        if (ce != cudaSuccess) return cuda_fail(ce, "norm launch");
+        ++*launches;
+    }
+    return HM_OK;
+}
+
+}  // namespace hm

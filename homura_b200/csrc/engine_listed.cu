@@ -103,6 +103,7 @@ int Engine::load_listed_tensor(const std::string& name, int dtype, const int64_t
     const LayerSpec& s = spec_.layers[li];
     if (rest == "norm1") return vec(&w.in_ln, H_);
     if (rest == "norm2") return vec(&w.post_ln, H_);
+    if (s.mixer == MIX_GQA) return load_gqa_tensor(w, s, name, rest, dtype, shape, ndim, host, nbytes);
     if (rest == "shift") return vec(&w.shift, H_);
     if (rest == "ls1") return vec(&w.ls1, H_);
     if (rest == "ls2") return vec(&w.ls2, H_);
@@ -125,6 +126,11 @@ int Engine::finalize_listed() {
         const LayerSpec& s = spec_.layers[i];
         const std::string p = "missing weight in layer " + std::to_string(i) + ": ";
         if (!l.in_ln) return fail(HM_ERR_STATE, p + "norm1");
+        if (s.mixer == MIX_GQA) {
+            const int rc = finalize_gqa(l, s, p);
+            if (rc) return rc;
+            continue;
+        }
         if (spec_.token_shift && !l.shift) return fail(HM_ERR_STATE, p + "shift");
         if (spec_.layer_scale && !l.ls1) return fail(HM_ERR_STATE, p + "ls1");
         if (l.in.loaded_parts != (s.kv_from < 0 ? 3 : 2)) return fail(HM_ERR_STATE, p + "mix.q / mix.g / mix.dkv");
@@ -145,6 +151,7 @@ void Engine::free_listed() {
         if (p) cudaFree(p);
         p = nullptr;
     };
+    free_gqa_scratch();
     fr(mix_raw_); fr(qlat_); fr(ctx_); fr(xpack_q_); fr(xpack_ctx_); fr(lat_acc_); fr(lat_ml_);
 }
 
@@ -153,11 +160,16 @@ int Engine::alloc_listed_scratch(int cap) {
     size_t raw = 1, lat = 1, q_img = 1, ctx_img = 1, acc = 1, ml = 1;
     int kmax = H_;
     for (const LayerSpec& s : spec_.layers) {
+        kmax = std::max(kmax, std::max(s.heads * s.vdim, s.ff));
+        if (s.mixer != MIX_LATENT) {
+            raw = std::max(raw, (size_t)(s.heads * s.dim + s.kv_heads * (s.dim + s.vdim) + 3) / 4 * 4);
+            continue;
+        }
         raw = std::max(raw, (size_t)in_ld(s));
         lat = std::max(lat, (size_t)s.heads * s.kv_rank);
         q_img = std::max(q_img, s.heads * tc_xpack_bytes(TC_ROWS, s.dim));
         ctx_img = std::max(ctx_img, s.heads * tc_xpack_bytes(TC_ROWS, s.kv_rank));
-        kmax = std::max(kmax, std::max(std::max(s.heads * s.vdim, s.ff), std::max(s.dim, s.kv_rank)));
+        kmax = std::max(kmax, std::max(s.dim, s.kv_rank));
         // splits times rows never exceed the SMs times the rows that share a CTA (latent_pick_nsplit)
         for (int bf16 = 0; bf16 < 2; ++bf16) {
             const size_t rows = 2 * (size_t)sm_count_ * latent_rows_per_tile(TC_ROWS, 1 << 30, s.heads, s.kv_rank, bf16);
@@ -187,7 +199,7 @@ int Engine::alloc_listed_scratch(int cap) {
         HM_CUDA(get(&xpack_q_, q_img));
         HM_CUDA(get(&xpack_ctx_, ctx_img));
     }
-    return HM_OK;
+    return alloc_gqa_scratch();
 }
 
 void Engine::free_listed_cache() {
@@ -203,7 +215,15 @@ int Engine::alloc_listed_cache(int batch, size_t n_pages) {
     lat_pool_.assign(L_, nullptr);
     for (int l = 0; l < L_; ++l) {
         const LayerSpec& s = spec_.layers[l];
-        if (s.mixer != MIX_LATENT || s.kv_from >= 0) continue;
+        if (s.mixer == MIX_GQA) {
+            const size_t esz = kv_bf16_ ? 2 : 4, kb = n_pages * gqa_page_elems(s.kv_heads, s.dim) * esz, vb = n_pages * gqa_page_elems(s.kv_heads, s.vdim) * esz;
+            HM_CUDA(cudaMalloc(&k_pool_[l], kb));
+            HM_CUDA(cudaMalloc(&v_pool_[l], vb));
+            HM_CUDA(cudaMemset(k_pool_[l], 0, kb));
+            HM_CUDA(cudaMemset(v_pool_[l], 0, vb));
+            continue;
+        }
+        if (s.kv_from >= 0) continue;
         const size_t bytes = n_pages * latent_page_elems(s.kv_rank, kv_bf16_) * (kv_bf16_ ? 2 : 4);
         HM_CUDA(cudaMalloc(&lat_pool_[l], bytes));
         HM_CUDA(cudaMemset(lat_pool_[l], 0, bytes));
@@ -225,8 +245,8 @@ LatentPool Engine::latent_pool(int layer) const {
 int Engine::latent_view(int seq, int layer, float* out) {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (batch_ == 0) return fail(HM_ERR_STATE, "latent_view before kv_alloc");
-    if (!spec_.listed()) return fail(HM_ERR_UNSUPPORTED, "latent_view: this design caches keys and values (hm_kv_view)");
     if (seq < 0 || seq >= batch_ || layer < 0 || layer >= L_ || !out) return fail(HM_ERR_INVALID, "latent_view: bad arguments");
+    if (!spec_.listed() || spec_.layers[layer].mixer != MIX_LATENT) return fail(HM_ERR_UNSUPPORTED, "latent_view: this design caches keys and values (hm_kv_view)");
     const int len = len_[seq];
     if (len == 0) return HM_OK;
     const size_t bytes = (size_t)len * spec_.layers[layer].kv_rank * 4;

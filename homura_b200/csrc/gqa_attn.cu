@@ -1,0 +1,696 @@
+// Grouped-query attention for listed designs.
+//
+//   gqa_post_kernel        norms, temperature and blending of a projection's queries, keys and values; page slots
+//   gqa_attn_kernel        CUDA cores, f32 or bf16 pages, any head size
+//   gqa_attn_mma_kernel    bf16 pages on warp-level MMAs, prompts and decoding alike
+//
+// MMA kernel.  A CTA serves a tile of (row, query head) pairs of one key/value head: the heads of a decoded token, or the heads of
+// several rows of a prompt that follow one another, so that a page is read once for all of them.  Pages come through a ring of
+// bulk copies (one contiguous block of keys and one of values per page and head).  Every warp takes units of 16 tokens:
+//   scores^T [16 tokens x pairs] = K [16 x dim]      . Q^T        (K chunks through ldmatrix)
+//   out^T    [vdim x pairs]     += V^T [vdim x 16]   . P^T        (V chunks through ldmatrix, transposed)
+// Queries and weights are three bf16 terms each (exact to 2^-24), so that the products are f32 x bf16 ones.  The warps of a CTA and
+// then the CTAs of a cluster, which share the context of a tile, combine their results in shared memory.
+#include "gqa_attn.h"
+
+#include <algorithm>
+
+#include "launch_attrs.h"
+#include "mbarrier.cuh"
+#include "model_spec.h"
+
+namespace hm {
+namespace {
+
+constexpr int POST_WARPS = 8;
+constexpr int ATT_WARPS = 8;
+constexpr int A_THREADS = 256;
+constexpr int B_THREADS = ATT_WARPS * 32 + 32;
+constexpr int MAX_STAGES = 8;
+constexpr int MAX_CLUSTER = 16;
+
+// ---- after the projection ------------------------------------------------------------------------
+// One warp per head (queries, then keys, then values); with a norm over the whole projection every CTA sums the squares of the part
+// it needs.
+__global__ void __launch_bounds__(POST_WARPS * 32) gqa_post_kernel(const GqaPostArgs a) {
+    pdl_launch_dependents();
+    const int m = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
+    const int slot0 = blockIdx.y * POST_WARPS, slot = slot0 + warp;  // head slots: [heads] queries, [G] keys, [G] values
+    const int pos = a.row_pos[m], seq = a.row_seq[m];
+    const size_t page = (size_t)a.pool.page_table[(size_t)seq * a.pool.max_pages + pos / GQA_PAGE];
+    const int t = pos % GQA_PAGE;
+    __shared__ float s_part[2][POST_WARPS];
+    pdl_wait();
+    const float* raw = a.raw + (size_t)m * a.ld;
+    if (a.qk_norm == QKN_ALL) {
+        float sq = 0.f, sk = 0.f;
+        if (slot0 < a.heads)
+#pragma unroll 4
+            for (int i = tid; i < nq; i += POST_WARPS * 32) {
+                const float v = ld_cg_f32(raw + i);
+                sq = fmaf(v, v, sq);
+            }
+        if (slot0 < a.heads + G && slot0 + POST_WARPS > a.heads)
+#pragma unroll 4
+            for (int i = tid; i < nk; i += POST_WARPS * 32) {
+                const float v = ld_cg_f32(raw + nq + i);
+                sk = fmaf(v, v, sk);
+            }
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        if (lane == 0) {
+            s_part[0][warp] = sq;
+            s_part[1][warp] = sk;
+        }
+        __syncthreads();
+    }
+    if (slot >= a.heads + 2 * G) return;
+    if (slot < a.heads + G) {
+        const bool is_q = slot < a.heads;
+        const int h = is_q ? slot : slot - a.heads;
+        const float* x = raw + (is_q ? 0 : nq) + (size_t)h * dim;
+        float inv = 1.f;
+        if (a.qk_norm == QKN_ALL) {
+            float s = 0.f;
+#pragma unroll
+            for (int w = 0; w < POST_WARPS; ++w) s += s_part[is_q ? 0 : 1][w];
+            inv = 1.0f / sqrtf(s / (float)(is_q ? nq : nk) + a.eps);
+        } else if (a.qk_norm == QKN_HEAD) {
+            float s = 0.f;
+#pragma unroll 4
+            for (int d = lane; d < dim; d += 32) {
+                const float v = ld_cg_f32(x + d);
+                s = fmaf(v, v, s);
+            }
+            inv = 1.0f / sqrtf(warp_sum(s) / (float)dim + a.eps);
+        }
+        const float* w = a.qk_norm == QKN_NONE ? nullptr : (is_q ? a.q_norm : a.k_norm) + (a.qk_norm == QKN_ALL ? (size_t)h * dim : 0);
+        if (is_q) {
+            float f = 1.f;
+            if (a.temp_every > 0) f = 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
+            float* o = a.q_out + (size_t)m * nq + (size_t)h * dim;
+            for (int d = lane; d < dim; d += 32) {
+                const float v = w ? (ld_cg_f32(x + d) * inv) * __ldg(w + d) : ld_cg_f32(x + d);
+                o[d] = (v * f) * a.q_scale;
+            }
+        } else {
+            const size_t base = page * gqa_page_elems(G, dim) + (size_t)h * GQA_PAGE * gqa_pad(dim);
+            for (int d = lane; d < dim; d += 32) {
+                const float v = w ? (ld_cg_f32(x + d) * inv) * __ldg(w + d) : ld_cg_f32(x + d);
+                const size_t off = base + gqa_tile_off(t, d);
+                if (a.pool.bf16) reinterpret_cast<uint16_t*>(a.pool.k)[off] = f32_to_bf16_rne(v);
+                else reinterpret_cast<float*>(a.pool.k)[off] = v;
+            }
+        }
+    } else {
+        const int h = slot - a.heads - G;
+        const float* x = raw + nq + nk + (size_t)h * vdim;
+        float* first = a.v_first ? a.v_first + (size_t)m * G * vdim + (size_t)h * vdim : nullptr;
+        const float lam = first && a.v_lambda ? __ldg(a.v_lambda) : 0.f;
+        const size_t base = page * gqa_page_elems(G, vdim) + (size_t)h * GQA_PAGE * gqa_pad(vdim);
+        for (int d = lane; d < vdim; d += 32) {
+            float v = ld_cg_f32(x + d);
+            if (first) {
+                if (a.v_lambda) v = (1.0f - lam) * v + lam * ld_cg_f32(first + d);
+                else first[d] = v;
+            }
+            const size_t off = base + gqa_tile_off(t, d);
+            if (a.pool.bf16) reinterpret_cast<uint16_t*>(a.pool.v)[off] = f32_to_bf16_rne(v);
+            else reinterpret_cast<float*>(a.pool.v)[off] = v;
+        }
+    }
+}
+
+__global__ void gqa_read_kernel(const GqaPool pool, int seq, int len, float* __restrict__ k, float* __restrict__ v) {
+    const int D = pool.dim + pool.vdim;
+    const size_t total = (size_t)pool.kv_heads * len * D;
+    for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const int e = (int)(i % D), t = (int)(i / D % len), g = (int)(i / D / len);
+        const bool is_k = e < pool.dim;
+        const int d = is_k ? e : e - pool.dim, n = is_k ? pool.dim : pool.vdim;
+        const size_t off = (size_t)pool.page_table[(size_t)seq * pool.max_pages + t / GQA_PAGE] * gqa_page_elems(pool.kv_heads, n) + (size_t)g * GQA_PAGE * gqa_pad(n) + gqa_tile_off(t % GQA_PAGE, d);
+        const void* src = is_k ? pool.k : pool.v;
+        (is_k ? k : v)[((size_t)g * len + t) * n + d] = pool.bf16 ? bf16_bits_to_f32(reinterpret_cast<const uint16_t*>(src)[off]) : reinterpret_cast<const float*>(src)[off];
+    }
+}
+
+// ---- common to both attention kernels --------------------------------------------------------------
+__device__ __forceinline__ void store_piece(const GqaAttnArgs& a, int m, int head, int d0, const float (&v)[8]) {
+    const int vdim = a.pool.vdim, k0 = head * vdim + d0;
+    if (a.xp && (vdim & 7) == 0) {
+        tc_xpack_store8(a.xp, a.xp_mpad, m, k0, v);
+        return;
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        if (d0 + i >= vdim) break;
+        if (a.xp) tc_xpack_store(a.xp, a.xp_mpad, m, k0 + i, v[i]);
+        else a.out[(size_t)m * a.heads * vdim + k0 + i] = v[i];
+    }
+}
+
+// Results of a CTA's pairs in its shared memory: o [pairs][ldo] (not yet divided), ml [pairs][2] (maximum as a base-2 exponent, sum).
+// Splits are the CTAs of a cluster; every one of them combines and stores a share of the elements.  wts: [nsplit][pairs].
+template <typename RowHead>
+__device__ __forceinline__ void combine_and_store(const GqaAttnArgs& a, const float* o, int ldo, const float* ml, float* wts, int pairs, RowHead row_head) {
+    const int tid = threadIdx.x, nt = blockDim.x, ns = a.nsplit;
+    const int rank = ns > 1 ? (int)cluster_ctarank() : 0;
+    if (ns > 1) cluster_sync_all();
+    else __syncthreads();
+    for (int p = tid; p < pairs; p += nt) {
+        if (ns == 1) {
+            wts[p] = 1.0f / ml[2 * p + 1];
+            continue;
+        }
+        float mr[MAX_CLUSTER], lr[MAX_CLUSTER], mx = -INFINITY, l = 0.f;
+#pragma unroll
+        for (int r = 0; r < MAX_CLUSTER; ++r)
+            if (r < ns) {
+                mr[r] = ld_dsmem_f32(dsmem_addr(ml + 2 * p, (uint32_t)r));
+                lr[r] = ld_dsmem_f32(dsmem_addr(ml + 2 * p + 1, (uint32_t)r));
+            }
+#pragma unroll
+        for (int r = 0; r < MAX_CLUSTER; ++r)
+            if (r < ns) mx = fmaxf(mx, mr[r]);
+#pragma unroll
+        for (int r = 0; r < MAX_CLUSTER; ++r)
+            if (r < ns) {
+                mr[r] = mr[r] == -INFINITY ? 0.f : exp2f(mr[r] - mx);
+                l = fmaf(mr[r], lr[r], l);
+            }
+#pragma unroll
+        for (int r = 0; r < MAX_CLUSTER; ++r)
+            if (r < ns) wts[r * pairs + p] = mr[r] / l;
+    }
+    __syncthreads();
+    const int np = gqa_pad(a.pool.vdim) / 8;
+    for (int i = rank * nt + tid; i < pairs * np; i += ns * nt) {
+        const int p = i / np, d0 = (i - p * np) * 8;
+        float v[8];
+        if (ns == 1) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = o[p * ldo + d0 + e] * wts[p];
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = 0.f;
+#pragma unroll 4
+            for (int r = 0; r < ns; ++r) {
+                const float w = wts[r * pairs + p];
+                const float4 x = ld_dsmem_f32x4(dsmem_addr(o + p * ldo + d0, (uint32_t)r)), y = ld_dsmem_f32x4(dsmem_addr(o + p * ldo + d0 + 4, (uint32_t)r));
+                v[0] = fmaf(w, x.x, v[0]); v[1] = fmaf(w, x.y, v[1]); v[2] = fmaf(w, x.z, v[2]); v[3] = fmaf(w, x.w, v[3]);
+                v[4] = fmaf(w, y.x, v[4]); v[5] = fmaf(w, y.y, v[5]); v[6] = fmaf(w, y.z, v[6]); v[7] = fmaf(w, y.w, v[7]);
+            }
+        }
+        int m, head;
+        row_head(p, m, head);
+        if (d0 < a.pool.vdim) store_piece(a, m, head, d0, v);
+    }
+    if (ns > 1) cluster_sync_all();  // nobody leaves while a peer reads its shared memory
+}
+
+// ---- CUDA cores ------------------------------------------------------------------------------------
+// One CTA = one row, key/value head and split.
+template <bool BF16>
+__global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    const int g = a.heads / a.pool.kv_heads, kvh = blockIdx.y, m = blockIdx.z, split = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int dim = a.pool.dim, vdim = a.pool.vdim, dp = gqa_pad(dim), vp = gqa_pad(vdim), ldo = vp + 4;
+    float* q_s = sm;                  // [g][dp]
+    float* o_s = q_s + g * dp;        // [g][ldo]
+    float* p_s = o_s + g * ldo;       // [g][64]
+    float* ml = p_s + g * GQA_PAGE;   // [g][2]
+    float* corr = ml + 2 * g;         // [g]
+    float* wts = corr + g;            // [nsplit][g]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int pos = a.row_pos[m], len = pos + 1, npages = (len + GQA_PAGE - 1) / GQA_PAGE, pps = (npages + a.nsplit - 1) / a.nsplit;
+    const int p0 = split * pps, p1 = min(npages, p0 + pps);
+    const int32_t* pt = a.pool.page_table + (size_t)a.row_seq[m] * a.pool.max_pages;
+    for (int i = tid; i < g * dp; i += A_THREADS) {
+        const int j = i / dp, d = i - j * dp;
+        q_s[i] = d < dim ? ld_cg_f32(a.q + (size_t)m * a.heads * dim + (size_t)(kvh * g + j) * dim + d) : 0.f;
+    }
+    for (int i = tid; i < g * ldo; i += A_THREADS) o_s[i] = 0.f;
+    for (int i = tid; i < g; i += A_THREADS) {
+        ml[2 * i] = -INFINITY;
+        ml[2 * i + 1] = 0.f;
+    }
+    __syncthreads();
+    for (int p = p0; p < p1; ++p) {
+        const size_t kb = (size_t)pt[p] * gqa_page_elems(a.pool.kv_heads, dim) + (size_t)kvh * GQA_PAGE * dp;
+        const size_t vb = (size_t)pt[p] * gqa_page_elems(a.pool.kv_heads, vdim) + (size_t)kvh * GQA_PAGE * vp;
+        const int nt = min(GQA_PAGE, len - p * GQA_PAGE);
+        for (int i = tid; i < g * GQA_PAGE; i += A_THREADS) {
+            const int j = i / GQA_PAGE, t = i % GQA_PAGE;
+            float s = -INFINITY;
+            if (t < nt) {
+                const float* q = q_s + j * dp;
+                s = 0.f;
+                for (int c = 0; c < dp / 8; ++c) {
+                    float k[8];
+                    if (BF16) {
+                        const uint4 u = __ldcg(reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(a.pool.k) + kb + (size_t)(c * GQA_PAGE + t) * 8));
+                        k[0] = bf16_lo(u.x); k[1] = bf16_hi(u.x); k[2] = bf16_lo(u.y); k[3] = bf16_hi(u.y);
+                        k[4] = bf16_lo(u.z); k[5] = bf16_hi(u.z); k[6] = bf16_lo(u.w); k[7] = bf16_hi(u.w);
+                    } else {
+                        const float4* src = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(a.pool.k) + kb + (size_t)(c * GQA_PAGE + t) * 8);
+                        const float4 x = __ldcg(src), y = __ldcg(src + 1);
+                        k[0] = x.x; k[1] = x.y; k[2] = x.z; k[3] = x.w; k[4] = y.x; k[5] = y.y; k[6] = y.z; k[7] = y.w;
+                    }
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) s = fmaf(q[c * 8 + e], k[e], s);
+                }
+                if (a.bias) s += __ldg(a.bias + (size_t)(kvh * g + j) * (a.reach + 1) + min(pos - (p * GQA_PAGE + t), a.reach));
+            }
+            p_s[i] = s;
+        }
+        __syncthreads();
+        for (int j = warp; j < g; j += A_THREADS / 32) {
+            const float s0 = p_s[j * GQA_PAGE + lane], s1 = p_s[j * GQA_PAGE + 32 + lane];
+            const float old = ml[2 * j], mx = fmaxf(old, warp_max(fmaxf(s0, s1)));  // a page of a split has a token
+            const float e0 = exp2f(s0 - mx), e1 = exp2f(s1 - mx), f = exp2f(old - mx);
+            p_s[j * GQA_PAGE + lane] = e0;
+            p_s[j * GQA_PAGE + 32 + lane] = e1;
+            const float l = warp_sum(e0 + e1);
+            __syncwarp();
+            if (lane == 0) {
+                ml[2 * j] = mx;
+                ml[2 * j + 1] = fmaf(ml[2 * j + 1], f, l);
+                corr[j] = f;
+            }
+        }
+        __syncthreads();
+        for (int i = tid; i < g * vdim; i += A_THREADS) {
+            const int j = i / vdim, d = i - j * vdim;
+            float s = 0.f;
+#pragma unroll 4
+            for (int t = 0; t < nt; ++t) {
+                const size_t off = vb + gqa_tile_off(t, d);
+                s = fmaf(p_s[j * GQA_PAGE + t], BF16 ? bf16_bits_to_f32(__ldcg(reinterpret_cast<const uint16_t*>(a.pool.v) + off)) : __ldcg(reinterpret_cast<const float*>(a.pool.v) + off), s);
+            }
+            o_s[j * ldo + d] = fmaf(o_s[j * ldo + d], corr[j], s);
+        }
+        __syncthreads();
+    }
+    combine_and_store(a, o_s, ldo, ml, wts, g, [&](int p, int& row, int& head) {
+        row = m;
+        head = kvh * g + p;
+    });
+}
+
+// ---- warp-level MMAs on bf16 pages ---------------------------------------------------------------------
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ uint32_t transpose8x8(uint32_t v) {
+    uint32_t r;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+    return r;
+}
+
+__host__ __device__ inline size_t b_stage_bytes(int dp, int vp) { return (size_t)GQA_PAGE * (dp + vp) * 2; }
+__host__ __device__ inline size_t b_query_bytes(int nt, int dp) { return (size_t)nt * (dp / 16) * 3 * 32 * 8; }
+// the ring's memory serves the combination of the warps' results afterwards: maxima and sums of the warps, four partial results
+__host__ __device__ inline size_t b_merge_bytes(int nt, int vp) { return sizeof(float) * ((size_t)2 * ATT_WARPS * nt * 8 + (size_t)4 * nt * 8 * (vp + 4)); }
+
+// VT: tiles of 16 value elements (at most), NT: tiles of eight pairs.
+template <int VT, int NT>
+__global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_attn_mma_kernel(const GqaAttnArgs a, size_t ring_bytes) {
+    constexpr int P = NT * 8;
+    extern __shared__ __align__(128) unsigned char dyn[];
+    const int g = a.heads / a.pool.kv_heads, kvh = blockIdx.y, split = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int dim = a.pool.dim, vdim = a.pool.vdim, dp = gqa_pad(dim), vp = gqa_pad(vdim), kt_n = dp / 16, vt_n = vp / 16, ldo = vp + 4;
+    const int NST = a.stages;
+    const uint32_t k_bytes = (uint32_t)(GQA_PAGE * dp * 2), v_bytes = (uint32_t)(GQA_PAGE * vp * 2), stage = k_bytes + v_bytes;
+    unsigned char* ring = dyn;
+    uint2* qf = reinterpret_cast<uint2*>(dyn + ring_bytes);                                 // [NT][kt_n][3][32]
+    float* wts = reinterpret_cast<float*>(dyn + ring_bytes + b_query_bytes(NT, dp));        // [nsplit][pairs]
+    float* ml = wts + a.nsplit * P;                                                         // [P][2]
+    int32_t* pt_s = reinterpret_cast<int32_t*>(ml + 2 * P);                                 // this CTA's pages
+    __shared__ uint64_t full[MAX_STAGES], empty[MAX_STAGES];
+    __shared__ volatile int s_abort;
+    __shared__ int s_pos[P], s_bias[P];  // position of the pair's row (-1: no such pair), first element of its bias row
+
+    if (tid == 0) {
+        for (int s = 0; s < NST; ++s) {
+            mb_init(&full[s], 1);
+            mb_init(&empty[s], 4);
+        }
+        s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    pdl_launch_dependents();
+    if (!a.early) pdl_wait();
+    // this tile's pairs: run, first pair, rows
+    int row0, rows, pair0;
+    if (a.runs.n == 0) {
+        row0 = blockIdx.z / a.tiles_per_row;
+        rows = 1;
+        pair0 = (blockIdx.z - row0 * a.tiles_per_row) * P;
+    } else {
+        int r = 0;
+        while (r + 1 < a.runs.n && a.runs.tile[r + 1] <= blockIdx.z) ++r;
+        row0 = a.runs.row[r];
+        rows = a.runs.row[r + 1] - row0;
+        pair0 = (blockIdx.z - a.runs.tile[r]) * P;
+    }
+    const int pairs = min(P, rows * g - pair0);
+    const int row_hi = row0 + (pair0 + pairs - 1) / g;
+    const int seq = a.row_seq[row0], len = a.row_pos[row_hi] + 1;
+    const int npages = (len + GQA_PAGE - 1) / GQA_PAGE, pps = (npages + a.nsplit - 1) / a.nsplit;
+    const int p0 = split * pps, np = max(0, min(npages, p0 + pps) - p0);
+    const int32_t* pt = a.pool.page_table + (size_t)seq * a.pool.max_pages + p0;
+    for (int i = tid; i < np; i += B_THREADS) pt_s[i] = pt[i];
+    if (tid < P) {
+        const int pr = pair0 + tid;
+        s_pos[tid] = tid < pairs ? a.row_pos[row0 + pr / g] : -1;
+        s_bias[tid] = (kvh * g + (tid < pairs ? pr % g : 0)) * (a.reach + 1);
+    }
+    __syncthreads();
+    const unsigned char *kpool = reinterpret_cast<const unsigned char*>(a.pool.k), *vpool = reinterpret_cast<const unsigned char*>(a.pool.v);
+    auto fetch = [&](int i, int s) {
+        const size_t tile = (size_t)pt_s[i] * a.pool.kv_heads + kvh;
+        unsigned char* dst = ring + (size_t)s * stage;
+        mb_expect_tx(&full[s], stage);
+        bulk_copy(dst, kpool + tile * k_bytes, k_bytes, &full[s]);
+        bulk_copy(dst + k_bytes, vpool + tile * v_bytes, v_bytes, &full[s]);
+    };
+    int n_pre = 0;
+    if (a.early) {
+        if (tid == ATT_WARPS * 32)
+            for (; n_pre < np && n_pre < NST && p0 + n_pre < (len - 1) / GQA_PAGE; ++n_pre) fetch(n_pre, n_pre);
+        pdl_wait();
+    }
+    if (warp == ATT_WARPS) {
+        if (lane == 0)
+            for (int i = n_pre; i < np; ++i) {
+                const int s = i % NST;
+                if (i >= NST && !mb_wait(&empty[s], ((i / NST) & 1u) ^ 1u, a.err_flag, &s_abort)) break;
+                fetch(i, s);
+            }
+    } else {
+        // B fragments of the queries: lane (pair = lane / 4, i = lane % 4) holds elements 2i, 2i + 1 and 2i + 8, 2i + 9 of every 16
+        for (int i = tid; i < NT * kt_n * 32; i += ATT_WARPS * 32) {
+            const int ln = i & 31, kt = (i >> 5) % kt_n, nt = (i >> 5) / kt_n, p = nt * 8 + (ln >> 2), d0 = kt * 16 + (ln & 3) * 2;
+            uint32_t lo[3] = {0u, 0u, 0u}, hi[3] = {0u, 0u, 0u};
+            if (p < pairs) {
+                const int pr = pair0 + p;
+                const float* q = a.q + (size_t)(row0 + pr / g) * a.heads * dim + (size_t)(kvh * g + pr % g) * dim;
+                auto at = [&](int d) { return d < dim ? ld_cg_f32(q + d) : 0.f; };
+                bf16x2_split3(at(d0), at(d0 + 1), lo[0], lo[1], lo[2]);
+                bf16x2_split3(at(d0 + 8), at(d0 + 9), hi[0], hi[1], hi[2]);
+            }
+#pragma unroll
+            for (int t3 = 0; t3 < 3; ++t3) qf[((nt * kt_n + kt) * 3 + t3) * 32 + ln] = make_uint2(lo[t3], hi[t3]);
+        }
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+    }
+
+    const int gid = lane >> 2, tig = lane & 3;
+    float tm[NT][2], tl[NT][2], to[NT][VT][4];
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+        tm[nt][0] = tm[nt][1] = -INFINITY;
+        tl[nt][0] = tl[nt][1] = 0.f;
+#pragma unroll
+        for (int mt = 0; mt < VT; ++mt) to[nt][mt][0] = to[nt][mt][1] = to[nt][mt][2] = to[nt][mt][3] = 0.f;
+    }
+    if (warp < ATT_WARPS) {
+        const int u = warp & 3, mj = lane >> 3, mr = lane & 7;
+        int pos[NT][2], brow[NT][2];
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+            for (int hh = 0; hh < 2; ++hh) {
+                pos[nt][hh] = s_pos[nt * 8 + 2 * tig + hh];
+                brow[nt][hh] = s_bias[nt * 8 + 2 * tig + hh];
+            }
+        const uint32_t k_lane = (uint32_t)(((mj >> 1) * GQA_PAGE + u * 16 + (mj & 1) * 8 + mr) * 16), v_lane = (uint32_t)(((mj & 1) * GQA_PAGE + u * 16 + (mj >> 1) * 8 + mr) * 16);
+        // pages alternate between the two groups of four warps; the stage count is even, so a stage is always the same group's
+        for (int i = warp >> 2; i < np; i += 2) {
+            const int s = i % NST;
+            if (!__all_sync(0xffffffffu, mb_wait(&full[s], (i / NST) & 1u, a.err_flag, &s_abort))) break;
+            const int tok = (p0 + i) * GQA_PAGE + u * 16;
+            if (tok < len) {
+                const uint32_t kb = s32(ring + (size_t)s * stage) + k_lane, vb = s32(ring + (size_t)s * stage + k_bytes) + v_lane;
+                float sc[NT][4];
+#pragma unroll
+                for (int nt = 0; nt < NT; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
+#pragma unroll 2
+                for (int kt = 0; kt < kt_n; ++kt) {
+                    uint32_t ka[4];
+                    ldsm4(ka, kb + (uint32_t)kt * (2 * GQA_PAGE * 16));
+#pragma unroll
+                    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+                        for (int t3 = 0; t3 < 3; ++t3) {
+                            const uint2 b = qf[((nt * kt_n + kt) * 3 + t3) * 32 + lane];
+                            mma16816(sc[nt], ka, b.x, b.y);
+                        }
+                }
+                uint32_t pb[NT][3][2];
+                const int t0 = tok + gid, t1 = t0 + 8;
+#pragma unroll
+                for (int nt = 0; nt < NT; ++nt) {
+                    float pr[4], corr[2];
+#pragma unroll
+                    for (int hh = 0; hh < 2; ++hh) {
+                        const int n0 = pos[nt][hh] - t0, n1 = pos[nt][hh] - t1;
+                        float s0 = sc[nt][hh], s1 = sc[nt][2 + hh];
+                        if (a.bias) {
+                            s0 += __ldg(a.bias + brow[nt][hh] + min(max(n0, 0), a.reach));
+                            s1 += __ldg(a.bias + brow[nt][hh] + min(max(n1, 0), a.reach));
+                        }
+                        s0 = n0 >= 0 ? s0 : -INFINITY;
+                        s1 = n1 >= 0 ? s1 : -INFINITY;
+                        float mx = fmaxf(s0, s1);
+#pragma unroll
+                        for (int o = 4; o < 32; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+                        mx = fmaxf(tm[nt][hh], mx);
+                        const float ref = mx == -INFINITY ? 0.f : mx;  // no token of this pair yet
+                        const float e0 = exp2f(s0 - ref), e1 = exp2f(s1 - ref);
+                        float ps = e0 + e1;
+#pragma unroll
+                        for (int o = 4; o < 32; o <<= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
+                        corr[hh] = exp2f(tm[nt][hh] - ref);
+                        tl[nt][hh] = fmaf(tl[nt][hh], corr[hh], ps);
+                        tm[nt][hh] = mx;
+                        pr[hh] = e0;
+                        pr[2 + hh] = e1;
+                    }
+                    uint32_t lo[3], hi[3];
+                    bf16x2_split3(pr[0], pr[1], lo[0], lo[1], lo[2]);
+                    bf16x2_split3(pr[2], pr[3], hi[0], hi[1], hi[2]);
+#pragma unroll
+                    for (int t3 = 0; t3 < 3; ++t3) {
+                        pb[nt][t3][0] = transpose8x8(lo[t3]);
+                        pb[nt][t3][1] = transpose8x8(hi[t3]);
+                    }
+                    if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
+#pragma unroll
+                        for (int mt = 0; mt < VT; ++mt) {
+                            to[nt][mt][0] *= corr[0];
+                            to[nt][mt][1] *= corr[1];
+                            to[nt][mt][2] *= corr[0];
+                            to[nt][mt][3] *= corr[1];
+                        }
+                    }
+                }
+#pragma unroll
+                for (int mt = 0; mt < VT; ++mt) {
+                    if (mt < vt_n) {
+                        uint32_t va[4];
+                        ldsm4_trans(va, vb + (uint32_t)mt * (2 * GQA_PAGE * 16));
+#pragma unroll
+                        for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+                            for (int t3 = 0; t3 < 3; ++t3) mma16816(to[nt][mt], va, pb[nt][t3][0], pb[nt][t3][1]);
+                    }
+                }
+            }
+            __syncwarp();
+            if (lane == 0) mb_arrive(&empty[s]);
+        }
+    }
+    __syncthreads();  // every page consumed: the ring becomes scratch
+    float* wm = reinterpret_cast<float*>(ring);  // [ATT_WARPS][P]
+    float* wl = wm + ATT_WARPS * P;
+    float* buf = wl + ATT_WARPS * P;             // [4][P][ldo]
+    if (warp < ATT_WARPS && gid == 0) {
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+            for (int hh = 0; hh < 2; ++hh) {
+                wm[warp * P + nt * 8 + 2 * tig + hh] = tm[nt][hh];
+                wl[warp * P + nt * 8 + 2 * tig + hh] = tl[nt][hh];
+            }
+    }
+    __syncthreads();
+    if (tid < P) {
+        float mx = -INFINITY, l = 0.f;
+#pragma unroll
+        for (int w = 0; w < ATT_WARPS; ++w) mx = fmaxf(mx, wm[w * P + tid]);
+#pragma unroll
+        for (int w = 0; w < ATT_WARPS; ++w) l += wm[w * P + tid] == -INFINITY ? 0.f : exp2f(wm[w * P + tid] - mx) * wl[w * P + tid];
+        ml[2 * tid] = mx;
+        ml[2 * tid + 1] = l;
+    }
+    __syncthreads();
+    if (warp < ATT_WARPS) {
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+            float f[2];
+#pragma unroll
+            for (int hh = 0; hh < 2; ++hh) f[hh] = tm[nt][hh] == -INFINITY ? 0.f : exp2f(tm[nt][hh] - ml[2 * (nt * 8 + 2 * tig + hh)]);
+#pragma unroll
+            for (int mt = 0; mt < VT; ++mt) {
+                to[nt][mt][0] *= f[0];
+                to[nt][mt][1] *= f[1];
+                to[nt][mt][2] *= f[0];
+                to[nt][mt][3] *= f[1];
+            }
+        }
+    }
+    // halve the number of partial results until warp 0 holds the sum
+    for (int step = ATT_WARPS / 2; step >= 0; step >>= 1) {
+        const bool last = step == 0;
+        if (last ? warp == 0 : warp >= step && warp < 2 * step) {
+            float* b = buf + (size_t)(last ? 0 : warp - step) * P * ldo;
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+                for (int mt = 0; mt < VT; ++mt)
+                    if (mt < vt_n)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) b[(nt * 8 + 2 * tig + (e & 1)) * ldo + mt * 16 + gid + (e >> 1) * 8] = to[nt][mt][e];
+        }
+        if (last) break;
+        __syncthreads();
+        if (warp < step) {
+            const float* b = buf + (size_t)warp * P * ldo;
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+                for (int mt = 0; mt < VT; ++mt)
+                    if (mt < vt_n)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) to[nt][mt][e] += b[(nt * 8 + 2 * tig + (e & 1)) * ldo + mt * 16 + gid + (e >> 1) * 8];
+        }
+        __syncthreads();
+    }
+    combine_and_store(a, buf, ldo, ml, wts, pairs, [&](int p, int& row, int& head) {
+        row = row0 + (pair0 + p) / g;
+        head = kvh * g + (pair0 + p) % g;
+    });
+}
+
+template <typename... KArgs, typename... Args>
+cudaError_t launch_clustered(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, int cluster, cudaStream_t st, bool pdl, Args... args) {
+    cudaError_t e = ensure_dyn_smem(kern, smem);
+    if (e == cudaSuccess && cluster > 8) e = ensure_nonportable_clusters(kern);
+    if (e != cudaSuccess) return e;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute at[2];
+    int n = 0;
+    if (pdl) {
+        at[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        at[n].val.programmaticStreamSerializationAllowed = 1;
+        ++n;
+    }
+    if (cluster > 1) {
+        at[n].id = cudaLaunchAttributeClusterDimension;
+        at[n].val.clusterDim.x = (unsigned)cluster;
+        at[n].val.clusterDim.y = 1;
+        at[n].val.clusterDim.z = 1;
+        ++n;
+    }
+    cfg.attrs = at;
+    cfg.numAttrs = n;
+    return cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
+}
+
+template <int VT, int NT>
+cudaError_t launch_mma(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
+    constexpr int P = NT * 8;
+    const int g = a.heads / a.pool.kv_heads, dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
+    a.tiles_per_row = (g + P - 1) / P;
+    if (a.runs.n == 0) {
+        a.tiles = a.M * a.tiles_per_row;
+    } else {
+        a.tiles = 0;
+        for (int r = 0; r < a.runs.n; ++r) {
+            a.runs.tile[r] = (uint16_t)a.tiles;
+            a.tiles += ((a.runs.row[r + 1] - a.runs.row[r]) * g + P - 1) / P;
+        }
+        a.runs.tile[a.runs.n] = (uint16_t)a.tiles;
+    }
+    const int pages = (a.longest + GQA_PAGE - 1) / GQA_PAGE, pairs = a.tiles * a.pool.kv_heads;
+    constexpr int PER_SM = NT == 1 && VT <= 8 ? 2 : 1;
+    a.nsplit = std::max(1, std::min({PER_SM * sm_count / pairs, a.max_cluster, MAX_CLUSTER, pages}));
+    const size_t stage = b_stage_bytes(dp, vp);
+    const int ppc = (pages + a.nsplit - 1) / a.nsplit;
+    const size_t fixed = b_query_bytes(NT, dp) + sizeof(float) * ((size_t)a.nsplit * P + 2 * P) + 4 * (size_t)ppc + 128;
+    // CTAs that have an SM to themselves take a deep ring
+    const size_t budget = (PER_SM == 2 && (long)pairs * a.nsplit > sm_count ? 110 : 220) * 1024;
+    int stages = MAX_STAGES;
+    while (stages > 2 && (stages * stage + fixed > budget || stages - 2 >= ppc)) stages -= 2;
+    a.stages = stages;
+    const size_t ring = (std::max(stages * stage, b_merge_bytes(NT, vp)) + 127) / 128 * 128;
+    if (ring + fixed > 226 * 1024) return cudaErrorInvalidValue;
+    return launch_clustered(gqa_attn_mma_kernel<VT, NT>, dim3((unsigned)a.nsplit, (unsigned)a.pool.kv_heads, (unsigned)a.tiles), dim3(B_THREADS), ring + fixed, a.nsplit, st, pdl, a, ring);
+}
+
+template <int VT>
+cudaError_t launch_mma_n(const GqaAttnArgs& a, int sm_count, cudaStream_t st, bool pdl) {
+    const int pairs = a.longest_run * (a.heads / a.pool.kv_heads);
+    if (pairs <= 8) return launch_mma<VT, 1>(a, sm_count, st, pdl);
+    if (pairs <= 16 || VT > 8) return launch_mma<VT, 2>(a, sm_count, st, pdl);
+    return launch_mma<VT, VT <= 8 ? 4 : 2>(a, sm_count, st, pdl);
+}
+
+}  // namespace
+
+cudaError_t launch_gqa_post(const GqaPostArgs& a, cudaStream_t st, bool pdl) {
+    const int slots = a.heads + 2 * a.pool.kv_heads;
+    return launch_clustered(gqa_post_kernel, dim3((unsigned)a.M, (unsigned)((slots + POST_WARPS - 1) / POST_WARPS)), dim3(POST_WARPS * 32), 0, 1, st, pdl, a);
+}
+
+cudaError_t launch_gqa_attn(const GqaAttnArgs& a_in, int sm_count, cudaStream_t st, bool pdl) {
+    GqaAttnArgs a = a_in;
+    if (a.M < 1 || a.M > GQA_MAX_ROWS || a.heads % a.pool.kv_heads != 0) return cudaErrorInvalidValue;
+    if (!a.bias) a.reach = 0;
+    const int g = a.heads / a.pool.kv_heads, dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
+    if (a.runs.n == 0) a.longest_run = 1;
+    const long ppc_most = (a.longest + GQA_PAGE - 1) / GQA_PAGE;
+    if (a.pool.bf16 && vp <= 256 && dp <= 256 && ppc_most <= 8192) {
+        if (vp <= 64) return launch_mma_n<4>(a, sm_count, st, pdl);
+        if (vp <= 128) return launch_mma_n<8>(a, sm_count, st, pdl);
+        return launch_mma_n<16>(a, sm_count, st, pdl);
+    }
+    const int pages = (a.longest + GQA_PAGE - 1) / GQA_PAGE;
+    a.nsplit = std::max(1, std::min({4 * sm_count / (a.M * a.pool.kv_heads), a.max_cluster, MAX_CLUSTER, pages}));
+    const size_t smem = sizeof(float) * (size_t)g * (dp + vp + 4 + GQA_PAGE + 3 + a.nsplit);
+    const dim3 grid((unsigned)a.nsplit, (unsigned)a.pool.kv_heads, (unsigned)a.M);
+    return a.pool.bf16 ? launch_clustered(gqa_attn_kernel<true>, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a) : launch_clustered(gqa_attn_kernel<false>, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a);
+}
+
+cudaError_t launch_gqa_read(const GqaPool& pool, int seq, int len, float* k, float* v, cudaStream_t st) {
+    const size_t total = (size_t)pool.kv_heads * len * (pool.dim + pool.vdim);
+    gqa_read_kernel<<<(unsigned)std::min<size_t>((total + 255) / 256, 4096), 256, 0, st>>>(pool, seq, len, k, v);
+    return cudaGetLastError();
+}
+
+}  // namespace hm

@@ -1,0 +1,75 @@
+// Grouped-query attention over a paged cache for head sizes of any kind: `dim` elements per query and key, `vdim` per value,
+// an optional learned bias by distance, rows of several sequences in one launch (gqa_attn.cu).
+#pragma once
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "common.cuh"
+
+namespace hm {
+
+constexpr int GQA_PAGE = 64;       // tokens per page
+constexpr int GQA_MAX_ROWS = 64;   // rows of one launch
+
+// One layer's pools.  A page holds, per key/value head, its tokens in chunks of eight elements, [pad / 8][64 tokens][8] (pad = the
+// size rounded up to 16, the tail zero): one contiguous block per head, whose 8x8 matrices for ldmatrix are 128 contiguous bytes.
+struct GqaPool {
+    void *k, *v;
+    const int32_t* page_table;  // [sequences][max_pages]
+    int max_pages;
+    int kv_heads, dim, vdim;
+    int bf16;
+};
+__host__ __device__ __forceinline__ int gqa_pad(int d) { return (d + 15) & ~15; }
+__host__ __device__ __forceinline__ size_t gqa_page_elems(int kv_heads, int d) { return (size_t)kv_heads * GQA_PAGE * gqa_pad(d); }
+__host__ __device__ __forceinline__ int gqa_tile_off(int t, int d) { return ((d >> 3) * GQA_PAGE + t) * 8 + (d & 7); }
+
+// What happens to a projection's queries, keys and values before the attention: norms, temperature, blended values; keys and values
+// go to their page slots, queries to q_out.
+struct GqaPostArgs {
+    GqaPool pool;
+    const float* raw;        // [M][ld]: queries | keys | values
+    int ld, M, heads;
+    int qk_norm;             // QkNorm
+    const float *q_norm, *k_norm;
+    float eps;
+    float q_scale;           // times the score scale (and log2 e: weights are powers of two)
+    float temp_coef;
+    int temp_every;          // 0: no temperature
+    float* v_first;          // [M][kv_heads * vdim] or null: values of the layer that the others blend in
+    const float* v_lambda;   // null: this layer keeps its values in v_first
+    const int32_t *row_pos, *row_seq;
+    float* q_out;            // [M][heads * dim]
+};
+cudaError_t launch_gqa_post(const GqaPostArgs& a, cudaStream_t st, bool pdl);
+
+// Rows as runs: consecutive positions of one sequence, whose rows and heads share a CTA.
+struct GqaRuns {
+    int n = 0;                            // 0: every row is a run
+    uint8_t row[GQA_MAX_ROWS + 1];        // first row of every run; row[n] = rows of the pass
+    uint16_t tile[GQA_MAX_ROWS + 1];      // first tile of every run (filled in by the launcher)
+};
+
+struct GqaAttnArgs {
+    GqaPool pool;
+    const float* q;          // [M][heads * dim], scaled
+    int M, heads;
+    const int32_t *row_pos, *row_seq;  // a row sees the positions up to its own
+    const float* bias;       // [heads][reach + 1] by distance (the last one for all beyond), times log2 e; or null
+    int reach;
+    GqaRuns runs;
+    int longest_run, longest;  // rows of the longest run, tokens of the longest context
+    int early;               // every row is its own sequence and the pages in front of its newest token were complete before the launch in front began
+    int max_cluster;
+    float* out;              // [M][heads * vdim], or, when xp is given, the activation image of the next tensor-core projection
+    unsigned char* xp;
+    int xp_mpad;
+    int* err_flag;
+    // filled in by the launcher
+    int tiles, tiles_per_row, nsplit, stages;
+};
+cudaError_t launch_gqa_attn(const GqaAttnArgs& a, int sm_count, cudaStream_t st, bool pdl);
+// Positions [0, len) of a sequence as f32 [kv_heads][len][dim] and [kv_heads][len][vdim].
+cudaError_t launch_gqa_read(const GqaPool& pool, int seq, int len, float* k, float* v, cudaStream_t st);
+
+}  // namespace hm

@@ -46,7 +46,13 @@ __global__ void pack_from_kn_kernel(const uint16_t* __restrict__ src, int K, int
 }
 
 // ---- embedding gather (src/hf/emitter.rs:506-537): hidden[m] = f32(table[token[m]]) -------
-__global__ void embed_gather_kernel(const void* table, int dtype, const uint32_t* tokens, int H, int V, float* out, int* err_flag) {
+// Element i of the position vector: the fraction of a turn is taken in double precision, so that far positions keep their phase.
+__device__ __forceinline__ float position_element(const double* turns, int pos, int i) {
+    double f = turns[i >> 1] * (double)pos;
+    f -= rint(f);
+    return i & 1 ? cospif(2.0f * (float)f) : sinpif(2.0f * (float)f);
+}
+__global__ void embed_gather_kernel(const void* table, int dtype, const uint32_t* tokens, int H, int V, float* out, int* err_flag, const double* turns, const int32_t* row_pos) {
     pdl_launch_dependents();
     pdl_wait();
     const int m = blockIdx.x;
@@ -56,7 +62,13 @@ __global__ void embed_gather_kernel(const void* table, int dtype, const uint32_t
         for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)m * H + i] = 0.f;
         return;
     }
-    if (dtype == 1) {  // bf16 rows
+    if (turns) {
+        const int pos = row_pos[m];
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            const float e = dtype == 1 ? bf16_bits_to_f32(reinterpret_cast<const uint16_t*>(table)[(size_t)tok * H + i]) : reinterpret_cast<const float*>(table)[(size_t)tok * H + i];
+            out[(size_t)m * H + i] = e + position_element(turns, pos, i);
+        }
+    } else if (dtype == 1) {  // bf16 rows
         const uint16_t* row = reinterpret_cast<const uint16_t*>(table) + (size_t)tok * H;
         for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)m * H + i] = bf16_bits_to_f32(row[i]);
     } else {
@@ -414,8 +426,8 @@ cudaError_t launch_pack_slabs_from_kn(const uint16_t* src_kn, int K, int N, uint
     pack_from_kn_kernel<<<grid_for(total, 256), 256, 0, st>>>(src_kn, K, N, dst);
     return cudaGetLastError();
 }
-cudaError_t launch_embed_gather(const void* table, int table_dtype, const uint32_t* tokens, int M, int H, int V, float* out, int* err_flag, cudaStream_t st, bool pdl) {
-    return launch_pdl(embed_gather_kernel, dim3(M), dim3(256), st, pdl, table, table_dtype, tokens, H, V, out, err_flag);
+cudaError_t launch_embed_gather(const void* table, int table_dtype, const uint32_t* tokens, int M, int H, int V, float* out, int* err_flag, cudaStream_t st, bool pdl, const double* turns, const int32_t* row_pos) {
+    return launch_pdl(embed_gather_kernel, dim3(M), dim3(256), st, pdl, table, table_dtype, tokens, H, V, out, err_flag, turns, row_pos);
 }
 cudaError_t launch_gather_rows(const float* src, const int32_t* rows, int n, int W, float* dst, cudaStream_t st, bool pdl) {
     return launch_pdl(gather_rows_kernel, dim3(n), dim3(256), st, pdl, src, rows, W, dst);

@@ -22,6 +22,19 @@ bool get_int(const Json& o, const char* key, int* out) {
     return true;
 }
 bool is_null(const Json* v) { return !v || v->kind == Json::Null; }
+bool get_num(const Json& o, const char* key, double* out) {
+    const Json* v = o.get(key);
+    if (!v || v->kind != Json::Num) return false;
+    *out = v->num;
+    return true;
+}
+// A count that may be zero, absent or null.
+bool get_count(const Json& o, const char* key, int* out) {
+    const Json* v = o.get(key);
+    *out = 0;
+    if (is_null(v) || (v->kind == Json::Num && v->num == 0)) return true;
+    return get_int(o, key, out);
+}
 
 // Tunitar: latent attention without positions, squared-ReLU MLPs (or none), grouped norms, token shift, layer scales.
 bool read_tunitar(const Json& j, ModelSpec* s, std::string* err) {
@@ -73,11 +86,87 @@ bool read_tunitar(const Json& j, ModelSpec* s, std::string* err) {
     return true;
 }
 
+// Grouped-query attention of the layer lists: query and key norms per head or over the whole projection, query temperature,
+// distance bias, blended values.
+bool read_gqa_mixer(const Json& m, bool positional, LayerSpec* l, const std::string& at, std::string* err) {
+    double scale = 0;
+    l->mixer = MIX_GQA;
+    if (!get_int(m, "heads", &l->heads) || !get_int(m, "kv_heads", &l->kv_heads) || !get_int(m, "dim", &l->dim) || !get_int(m, "vdim", &l->vdim) || !get_num(m, "scale", &scale))
+        return fail(err, at + "the mixer needs heads, kv_heads, dim, vdim and scale");
+    if (l->heads % l->kv_heads != 0) return fail(err, at + "`kv_heads` does not divide `heads`");
+    l->scale = (float)scale;
+    l->qk_norm = positional ? QKN_ALL : QKN_HEAD;
+    const Json* mix = m.get("v_mix");
+    if (!is_null(mix) && mix->kind != Json::Bool) return fail(err, at + "`v_mix` must be true or false");
+    l->v_mix = !is_null(mix) && mix->b;
+    if (!positional) return true;
+    if (!get_num(m, "bias_max", &l->bias_reach) || l->bias_reach <= 0 || l->bias_reach > 1 << 20) return fail(err, at + "`bias_max` must be a positive number of tokens");
+    const Json* t = m.get("q_temp");
+    if (!is_null(t)) {
+        double coef = 0;
+        if (!get_num(*t, "coef", &coef) || !get_int(*t, "every", &l->temp_every)) return fail(err, at + "`q_temp` needs coef and every");
+        l->temp_coef = (float)coef;
+    }
+    return true;
+}
+
+bool read_moe(const Json& f, LayerSpec* l, const std::string& at, std::string* err) {
+    const Json *kind = f.get("kind"), *ex = f.get("expert"), *r = f.get("router");
+    double limit = 0;
+    if (!kind || kind->kind != Json::Str || kind->str != "moe") return fail(err, at + "unknown mlp");
+    if (!ex || !get_int(*ex, "ff", &l->ff) || !get_num(*ex, "limit", &limit)) return fail(err, at + "`mlp.expert` needs ff and limit");
+    if (!r || !get_int(*r, "experts", &l->experts) || !get_int(*r, "top", &l->top) || !get_count(*r, "identity", &l->identity)) return fail(err, at + "`mlp.router` needs experts and top");
+    if (l->top > l->experts + l->identity) return fail(err, at + "`mlp.router.top` is larger than the number of router outputs");
+    l->limit = (float)limit;
+    l->mlp = MLP_MOE;
+    return true;
+}
+
+// Dipisun: grouped-query attention in two kinds, norms on what the sublayers give back, mixtures of experts (or none).
+bool read_dipisun(const Json& j, ModelSpec* s, std::string* err) {
+    hm_config& c = s->cfg;
+    s->post_norm = s->sin_pos = true;
+    if (!get_int(j, "width", &c.hidden_size) || !get_int(j, "vocab", &c.vocab_size)) return fail(err, "missing `width` or `vocab`");
+    const Json* norm = j.get("norm");
+    double mult = 0;
+    if (!norm || !get_num(*norm, "eps", &c.rms_norm_eps)) return fail(err, "`norm` needs `eps`");
+    if (!get_num(j, "residual_mult", &mult)) return fail(err, "missing `residual_mult`");
+    s->residual_mult = (float)mult;
+    const Json* list = j.get("layers");
+    if (!list || list->kind != Json::Arr || list->arr.empty()) return fail(err, "missing `layers`");
+    int first = -1;
+    for (size_t i = 0; i < list->arr.size(); ++i) {
+        const Json& e = list->arr[i];
+        const std::string at = "layer " + std::to_string(i) + ": ";
+        LayerSpec l;
+        const Json *type = e.get("type"), *m = e.get("mixer"), *mlp = e.get("mlp");
+        const bool positional = type && type->kind == Json::Str && type->str == "attention";
+        if (!positional && !(type && type->kind == Json::Str && type->str == "attention_2")) return fail(err, at + "unknown mixer type");
+        if (!m) return fail(err, at + "missing `mixer`");
+        if (!read_gqa_mixer(*m, positional, &l, at, err)) return false;
+        if (l.v_mix) {
+            if (first < 0) first = (int)i;
+            l.v_first = first;
+            if (first < (int)i && s->layers[first].kv_heads * s->layers[first].vdim != l.kv_heads * l.vdim) return fail(err, at + "`v_mix` blends values of another size");
+        }
+        if (!is_null(mlp) && !read_moe(*mlp, &l, at, err)) return false;
+        c.num_attention_heads = std::max(c.num_attention_heads, l.heads);
+        c.num_key_value_heads = std::max(c.num_key_value_heads, l.kv_heads);
+        c.head_dim = std::max(c.head_dim, l.dim);
+        c.intermediate_size = std::max(c.intermediate_size, l.ff);
+        s->layers.push_back(l);
+    }
+    c.num_hidden_layers = (int)s->layers.size();
+    c.max_position_embeddings = 1 << 30;  // positions are computed: the cache is the only limit
+    c.intermediate_size = std::max(c.intermediate_size, 1);
+    return true;
+}
+
 struct Design {
     const char* name;
     bool (*read)(const Json&, ModelSpec*, std::string*);
 };
-const Design kDesigns[] = {{"Tunitar", read_tunitar}};
+const Design kDesigns[] = {{"Tunitar", read_tunitar}, {"Dipisun", read_dipisun}};
 
 }  // namespace
 
@@ -115,9 +204,18 @@ std::string layers_json(const ModelSpec& spec) {
     std::string o = "[";
     for (size_t i = 0; i < spec.layers.size(); ++i) {
         const LayerSpec& l = spec.layers[i];
-        char t[320];
-        std::snprintf(t, sizeof(t), "%s{\"type\":\"latent_attention\",\"heads\":%d,\"dim\":%d,\"vdim\":%d,\"kv_rank\":%d,\"kv_from\":%s,\"scale\":%.9g,\"ff\":%d}", i ? "," : "", l.heads, l.dim, l.vdim, l.kv_rank,
-                      l.kv_from < 0 ? "null" : std::to_string(l.kv_from).c_str(), l.scale, l.ff);
+        char t[512];
+        if (i) o += ",";
+        if (l.mixer == MIX_LATENT) {
+            std::snprintf(t, sizeof(t), "{\"type\":\"latent_attention\",\"heads\":%d,\"dim\":%d,\"vdim\":%d,\"kv_rank\":%d,\"kv_from\":%s,\"scale\":%.9g,\"ff\":%d}", l.heads, l.dim, l.vdim, l.kv_rank,
+                          l.kv_from < 0 ? "null" : std::to_string(l.kv_from).c_str(), l.scale, l.ff);
+            o += t;
+            continue;
+        }
+        std::snprintf(t, sizeof(t), "{\"type\":\"grouped_attention\",\"heads\":%d,\"kv_heads\":%d,\"dim\":%d,\"vdim\":%d,\"scale\":%.9g,\"qk_norm\":\"%s\",\"temp_coef\":%.9g,\"temp_every\":%d,\"bias_reach\":%.9g,\"v_first\":%s", l.heads,
+                      l.kv_heads, l.dim, l.vdim, l.scale, l.qk_norm == QKN_ALL ? "all" : l.qk_norm == QKN_HEAD ? "head" : "none", l.temp_coef, l.temp_every, l.bias_reach, l.v_first < 0 ? "null" : std::to_string(l.v_first).c_str());
+        o += t;
+        std::snprintf(t, sizeof(t), ",\"ff\":%d,\"experts\":%d,\"identity\":%d,\"top\":%d,\"limit\":%.9g}", l.ff, l.experts, l.identity, l.top, l.limit);
         o += t;
     }
     return o + "]";

@@ -13,7 +13,9 @@
 namespace hm {
 
 enum MixerKind { MIX_GQA = 0, MIX_LATENT = 1 };
-enum MlpKind { MLP_NONE = 0, MLP_SWIGLU = 1, MLP_SQRELU = 2 };
+enum MlpKind { MLP_NONE = 0, MLP_SWIGLU = 1, MLP_SQRELU = 2, MLP_MOE = 3 };
+// RMS norm of queries and keys: none, every head by itself (one weight vector of `dim`), the whole projection at once
+enum QkNorm { QKN_NONE = 0, QKN_HEAD = 1, QKN_ALL = 2 };
 
 struct LayerSpec {
     int mixer = MIX_GQA;
@@ -21,8 +23,19 @@ struct LayerSpec {
     int heads = 0, dim = 0, vdim = 0, kv_rank = 0;
     int kv_from = -1;  // layer whose cached latents this one reads (-1: its own)
     float scale = 1.f;
+    // MIX_GQA (listed): heads query heads of dim over kv_heads key heads of dim and value heads of vdim
+    int kv_heads = 0;
+    int qk_norm = QKN_NONE;
+    float temp_coef = 0.f;  // queries times 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1); temp_every 0: not
+    int temp_every = 0;
+    double bias_reach = 0;  // > 0: learned bias by distance, logarithmic steps up to this many tokens back
+    bool v_mix = false;     // values are blended with those of layer v_first (which keeps its own)
+    int v_first = -1;
     int mlp = MLP_NONE;
-    int ff = 0;
+    int ff = 0;             // of one expert with MLP_MOE
+    // MLP_MOE: `top` of experts + identity router outputs; the identity ones pass their input on
+    int experts = 0, identity = 0, top = 0;
+    float limit = 0.f;      // clamp of the experts' gate (above) and up (both sides)
 };
 
 struct ModelSpec {
@@ -32,6 +45,9 @@ struct ModelSpec {
     int norm_groups = 1;      // runs of the width that a norm divides by their own root mean square
     bool token_shift = false; // the mixer reads a blend of a token's normalised row and its predecessor's
     bool layer_scale = false; // mixer and MLP results are multiplied element by element before they join the residual
+    bool post_norm = false;   // mixer and MLP read the residual itself; their results are normalised, times residual_mult, before they join it
+    float residual_mult = 1.f;
+    bool sin_pos = false;     // sinusoidal position vectors are added to the embedding
     bool listed() const { return !layers.empty(); }
 };
 

@@ -1,0 +1,58 @@
+// Residual sums with normalised sublayer results, routers, and mixtures of experts (moe.cu).
+#pragma once
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "common.cuh"
+
+namespace hm {
+
+// Where a router puts its choice.
+struct RouteOut {
+    int32_t* ids;       // [M][top] chosen experts, -1 for identity ones
+    float* weights;     // [M][top]
+    float* identity;    // [M] sum of the weights of the chosen identity experts
+    float* dense;       // [M][experts] weight of every expert, 0 where it is not chosen; or null
+    uint32_t* mask;     // [M][ceil(experts / 32)] with dense: one bit per chosen expert
+};
+
+// x += mult * RMSnorm(y) * w, and then, optionally, the router over the new x.
+struct PostNormArgs {
+    const float* y;          // [M][W] what the sublayer gave back
+    const float* identity;   // [M] or null: y + identity * x instead of y
+    float* x;                // [M][W] residual
+    int M, W;
+    const float* w;
+    float mult, eps;
+    unsigned char* xp;       // optional: the new x as the activation image of the next tensor-core projection
+    int xp_mpad;
+    // router
+    const uint16_t* router;  // [n_out][W] bf16, or null
+    const float* correction; // [n_out]
+    int experts, n_out, top; // n_out = experts + identity ones (the last)
+    RouteOut out;
+};
+cudaError_t launch_post_norm(const PostNormArgs& a, int sm_count, cudaStream_t st, bool pdl);
+
+// Experts' weights as tensor-core tile images (gemm_tc.h), one after the other: gate and up interleaved 64 + 64 per block of 128
+// rows over W, down [W] over ff; ff padded to 64.
+struct ExpertWeights {
+    const uint16_t *gu, *down;
+    int W, ff, top;
+    float limit;
+};
+__host__ __device__ __forceinline__ int expert_blocks(int ff) { return (ff + 63) / 64; }
+size_t expert_gu_elems(int W, int ff);
+size_t expert_down_elems(int W, int ff);
+
+// Few rows: every (row, chosen expert) pair reads its own weights.  act: [M * top][ff padded], already times the routing weight.
+cudaError_t launch_expert_gate_up(const ExpertWeights& e, const float* x, int M, const RouteOut& r, float* act, cudaStream_t st, bool pdl);
+cudaError_t launch_expert_down(const ExpertWeights& e, const float* act, int M, const RouteOut& r, float* y, cudaStream_t st, bool pdl);
+
+// Gated activation of an expert: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1).
+__device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
+}  // namespace hm
