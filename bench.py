@@ -285,36 +285,64 @@ def run_c5(hm, synth, rank, world, local, barrier, vmax, K, W, peak):
     return out
 
 
-# --workload tunitar: (Tunitar stack, uniform stack of equal width, depth, heads and MLP parameters), and where each pair is timed:
-# (sequences, prompt tokens)
-TUNITAR_PAIRS = {
-    "0.5B": ("TUNITAR_05B", "QWEN25_05B", [(1, 128), (8, 1920)]),
-    "1.5B": ("TUNITAR_15B", "QWEN25_15B", [(1, 128), (64, 512), (8, 1920)]),
+# Workloads of the listed designs: (stack, uniform stack of equal width, depth, heads and MLP parameters per token), and where each
+# pair is timed: (sequences, prompt tokens)
+POINTS = {"0.5B": [(1, 128), (8, 1920)], "1.5B": [(1, 128), (64, 512), (8, 1920)]}
+DESIGNS = {
+    "tunitar": {"0.5B": ("TUNITAR_05B", "QWEN25_05B"), "1.5B": ("TUNITAR_15B", "QWEN25_15B")},
+    "dipisun": {"0.5B": ("DIPISUN_05B", "QWEN25_05B"), "1.5B": ("DIPISUN_15B", "QWEN25_15B")},
 }
 # kernel classes that do the same work in both designs
-TUNITAR_LIKE = {"in_proj": "qkv_rope_kvwrite", "key_up": "qkv_rope_kvwrite", "value_up_gate": "o_proj_residual", "attention": "attention", "o_proj_residual": "o_proj_residual", "up_sqrelu": "gate_up_swiglu",
-                "down_residual": "down_residual", "lm_head": "lm_head"}
+LIKE = {
+    "tunitar": {"in_proj": "qkv_rope_kvwrite", "key_up": "qkv_rope_kvwrite", "value_up_gate": "o_proj_residual", "attention": "attention", "o_proj_residual": "o_proj_residual", "up_sqrelu": "gate_up_swiglu",
+                "down_residual": "down_residual", "lm_head": "lm_head"},
+    "dipisun": {"qkv_proj": "qkv_rope_kvwrite", "attention": "attention", "o_proj": "o_proj_residual", "experts_gate_up": "gate_up_swiglu", "experts_down": "down_residual", "lm_head": "lm_head"},
+}
+WHAT = {"tunitar": "Tunitar stacks beside uniform GQA stacks of equal size", "dipisun": "Dipisun stacks beside uniform GQA stacks of equal width, depth, heads and MLP parameters per token"}
 
 
-def run_tunitar(args, hm, synth, K, W, peak, peak_kind):
-    """Prefill and decode throughput of the Tunitar design beside the uniform GQA / SwiGLU stack of equal size, bf16 pages."""
+def design_model(design, name, cfg, synth):
+    """Folder of a synthetic checkpoint of the design (written once)."""
+    d = os.path.join(tempfile.gettempdir(), f"homura_b200_bench_{name.lower()}_seed{SEED}")
+    if os.path.exists(os.path.join(d, ".complete")):
+        return d
+    if design == "tunitar":
+        synth.write_tunitar_model(d, cfg, SEED)
+    elif design == "dipisun":
+        # every layer's experts are drawn from one set; corrections of zero leave the choice to the router
+        specs = {s[0]: s for s in synth.dipisun_tensor_specs(cfg)}
+        experts = {}
+
+        class Weights:
+            def __getitem__(self, key):
+                name, shape, kind = specs[key]
+                if ".mlp.e" in name:
+                    name = "l0." + name.split(".", 1)[1]
+                    if name not in experts:
+                        experts[name] = synth.dipisun_tensor(SEED, (name, shape, kind))
+                    return experts[name]
+                w = synth.dipisun_tensor(SEED, (name, shape, kind))
+                return w * 0 if kind == "small" else w
+
+        synth.write_dipisun_model(d, cfg, SEED, Weights())
+    else:
+        synth.write_hf_model(d, cfg, SEED)
+    open(os.path.join(d, ".complete"), "w").write("ok")
+    return d
+
+
+def run_design(design, args, hm, synth, K, W, peak, peak_kind):
+    """Prefill and decode throughput of a listed design beside the uniform GQA / SwiGLU stack of equal size, bf16 pages."""
     K = min(K, 48)
     sampler = ClockSampler(0)
     sizes = {}
-    for size, (t_name, u_name, points) in TUNITAR_PAIRS.items():
+    for size, (t_name, u_name) in DESIGNS[design].items():
         rows = {}
-        for kind, name in (("tunitar", t_name), ("uniform", u_name)):
+        for kind, name in ((design, t_name), ("uniform", u_name)):
             cfg = getattr(synth, name)
-            d = os.path.join(tempfile.gettempdir(), f"homura_b200_bench_{name.lower()}_seed{SEED}")
-            if not os.path.exists(os.path.join(d, ".complete")):
-                if kind == "tunitar":
-                    synth.write_tunitar_model(d, cfg, SEED)
-                else:
-                    synth.write_hf_model(d, cfg, SEED)
-                open(os.path.join(d, ".complete"), "w").write("ok")
-            vocab = cfg["vocab"] if kind == "tunitar" else cfg.vocab_size
-            m = hm.HfModel.load_with_dtype(d, hm.DType.BF16)
-            for B, PL in points:
+            vocab = cfg.vocab_size if kind == "uniform" else cfg["vocab"]
+            m = hm.HfModel.load_with_dtype(design_model(kind, name, cfg, synth), hm.DType.BF16)
+            for B, PL in POINTS[size]:
                 m.init_kv_cache(PL + 2 * W + K + 16, batch=B, kv_dtype=hm.DType.BF16)
                 prompts = [synth.prompt_ids(SEED + b, PL, vocab) for b in range(B)]
                 m.prefill(prompts[0], seq=0)
@@ -324,7 +352,7 @@ def run_tunitar(args, hm, synth, K, W, peak, peak_kind):
                 pf_s = time.perf_counter() - t
                 m.decode_greedy_n(first, 0)
                 ms = m.time_decode(W, K)
-                prof = m.profile_decode(8)
+                prof = m.profile_decode(7)
                 rows.setdefault(f"{B}x{PL}", {})[kind] = {
                     "decode_tok_per_s": B * K / (ms / 1e3), "ms_per_step": ms / K, "prefill_tok_per_s": B * PL / pf_s, "launches_per_step": m.launches_per_step(), "weight_bytes": m.weight_bytes(),
                     "kernels": {p["name"]: {"launches": p["launches_per_step"], "us": round(1e3 * p["ms_per_step"], 2), "MB": round(p["bytes_per_step"] / 1e6, 3),
@@ -333,14 +361,14 @@ def run_tunitar(args, hm, synth, K, W, peak, peak_kind):
                 log(f"[bench] {size} {kind} {B}x{PL}: {rows[f'{B}x{PL}'][kind]['decode_tok_per_s']:.0f} tok/s decode, {rows[f'{B}x{PL}'][kind]['prefill_tok_per_s']:.0f} tok/s prefill")
             m.close()
         for r in rows.values():
-            tk, uk = r["tunitar"]["kernels"], r["uniform"]["kernels"]
-            r["fraction_relative_to_like_kernel"] = {a: round(tk[a]["frac"] / uk[b]["frac"], 3) for a, b in TUNITAR_LIKE.items() if tk[a]["frac"] and uk[b]["frac"]}
+            tk, uk = r[design]["kernels"], r["uniform"]["kernels"]
+            r["fraction_relative_to_like_kernel"] = {a: round(tk[a]["frac"] / uk[b]["frac"], 3) for a, b in LIKE[design].items() if tk[a]["frac"] and uk[b]["frac"]}
         sizes[size] = rows
-    head = sizes["1.5B"]["64x512"]["tunitar"]
+    head = sizes["1.5B"]["64x512"][design]
     return {
         "metric": "decode_tokens_per_s", "value": head["decode_tok_per_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W, "ms_per_step": head["ms_per_step"], "higher_is_better": True, "scaling": "weak",
         "vs_baseline": None, "dtype": "f32 accumulate over bf16 weights", "data": "synthetic",
-        "config": {"workload": "Tunitar stacks beside uniform GQA stacks of equal size, bf16 pages, greedy decode; value: 1.5B, 64 sequences, 512-token prompts", "l2": "weights and pages of a step exceed the L2", "seed": SEED,
+        "config": {"workload": f"{WHAT[design]}, bf16 pages, greedy decode; value: 1.5B, 64 sequences, 512-token prompts", "l2": "weights and pages of a step exceed the L2", "seed": SEED,
                    "peak_gbs": peak, "peak_source": f"{peak_kind} copy bandwidth"},
         "clocks": sampler.stop(), "gpu_launches": head["launches_per_step"] * K, "sizes": sizes,
     }
@@ -356,7 +384,7 @@ def main():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-c5", action="store_true", help="skip the batched Qwen2.5-1.5B x 64 block of the headline line")
     ap.add_argument("--prompt-len", type=int, default=None, help="prompt tokens before the timed decode steps (default: the workload's own, 128 for the headline)")
-    ap.add_argument("--workload", default=HEADLINE, choices=sorted(WORKLOADS) + ["tunitar"], help="default: the headline workload; the others are the remaining measured configurations")
+    ap.add_argument("--workload", default=HEADLINE, choices=sorted(WORKLOADS) + sorted(DESIGNS), help="default: the headline workload; the others are the remaining measured configurations")
     ap.add_argument("--device-only", action="store_true", help="only the device-timed region: skips the end-to-end loop, the per-kernel pass and the CPU baseline (for profiler runs)")
     args = ap.parse_args()
     claim_stdout()
@@ -368,9 +396,9 @@ def main():
 
     rank, world, local, barrier, vmax, close = dist_setup(args.gpus)
     K, W = args.steps, max(args.warmup, 3)
-    if args.workload == "tunitar":
+    if args.workload in DESIGNS:
         if rank == 0:
-            emit(run_tunitar(args, hm, synth, K, W, *measured_peak()))
+            emit(run_design(args.workload, args, hm, synth, K, W, *measured_peak()))
         close()
         return
     cfg_name, fmt, B, wl_desc = WORKLOADS[args.workload]

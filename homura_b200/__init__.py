@@ -19,7 +19,7 @@ import ctypes as C
 import enum
 import os
 from dataclasses import dataclass, field
-from typing import List, Optional, Sequence
+from typing import List, Optional, Sequence, Tuple
 
 import numpy as np
 
@@ -152,6 +152,10 @@ SIGNATURES = {
     "hm_latent_pool_bytes": (C.c_size_t, [_i32, _i32, _i32]),
     "hm_latent_write": (_i32, [_vp, _vp, C.c_float, _i32, _i32, _vp, _i32, _vp, _i32, _i32, _vp, _vp, _vp]),
     "hm_latent_attn_paged": (_i32, [_vp, _vp, _i32, _vp, _i32, _i32, _vp, _vp, _i32, _i32, _i32, C.c_float, _i32, _vp, _vp]),
+    "hm_gqa_pool_bytes": (C.c_size_t, [_i32, _i32, _i32, _i32]),
+    "hm_gqa_write": (_i32, [_vp, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _vp, C.c_float, C.c_float, C.c_float, _i32, _vp, _i32, C.c_float, _vp, _vp, _i32, _vp, _i32, _i32, _vp, _vp, _vp, _vp]),
+    "hm_gqa_attn_paged": (_i32, [_vp, _vp, _vp, _i32, _vp, _i32, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _vp, _i32, _i32, _vp, _vp]),
+    "hm_post_norm_route": (_i32, [_vp, _vp, _vp, _i32, _i32, _vp, C.c_float, C.c_float, _vp, _vp, _i32, _i32, _i32, _vp, _vp, _vp, _vp]),
     "hm_argmax": (_i32, [_vp, _i32, _i32, _vp, _vp]),
     "hm_dev_alloc": (_i32, [C.c_size_t, C.POINTER(_vp)]),
     "hm_dev_free": (_i32, [_vp]),
@@ -449,9 +453,14 @@ class HfModel:
     def kv_advance_by(self, n: int, seq: int = 0):
         _check(self._lib.hm_kv_append(self._h, seq, 0, None, None, n, 1), self._h)
 
-    def kv_view(self, layer: int, seq: int = 0):
+    def kv_view(self, layer: int, seq: int = 0, shape: Optional[Tuple[int, int, int]] = None):
+        """shape: (key/value heads, key size, value size) of the layer in designs whose layers differ."""
         c = self._config
         n = self.kv_cache_len(seq)
+        if shape is not None:
+            k, v = np.zeros((1, shape[0], n, shape[1]), np.float32), np.zeros((1, shape[0], n, shape[2]), np.float32)
+            _check(self._lib.hm_kv_view(self._h, seq, layer, _ptr(k), _ptr(v)), self._h)
+            return k, v
         k = np.zeros((1, c.kv_heads(), n, c.get_head_dim()), np.float32)
         v = np.zeros_like(k)
         _check(self._lib.hm_kv_view(self._h, seq, layer, _ptr(k), _ptr(v)), self._h)
@@ -766,6 +775,53 @@ class LatentCache:
         out = np.empty_like(q)
         _check(self._lib.hm_latent_attn_paged(_ptr(q), _ptr(self.pages.ptr), int(self.kv_dtype), _ptr(self.table), self.table.shape[0], self.table.shape[1], _ptr(s), _ptr(p), q.shape[0], q.shape[1], self.rank, scale, nsplit, _ptr(out), None))
         return out
+
+
+class GqaCache:
+    """A paged cache of one layer of grouped-query attention: kv_heads keys of dim and values of vdim elements per token."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, kv_dtype: DType, page_table):
+        self._lib = load_library()
+        self.heads, self.kv_heads, self.dim, self.vdim, self.kv_dtype = heads, kv_heads, dim, vdim, kv_dtype
+        self.table = np.ascontiguousarray(page_table, dtype=np.int32)
+        n = int(self.table.max()) + 1
+        sizes = [self._lib.hm_gqa_pool_bytes(kv_heads, d, int(kv_dtype), n) for d in (dim, vdim)]
+        self.k, self.v = DeviceBuffer(sizes[0]), DeviceBuffer(sizes[1])
+        for buf, size in zip((self.k, self.v), sizes):
+            buf.upload(np.zeros(size, np.uint8))
+
+    def write(self, raw, row_seq, row_pos, q_norm=None, k_norm=None, norm: int = 0, eps: float = 0.0, q_scale: float = 1.0, temperature=(0.0, 0), v_first=None, v_lambda: Optional[float] = None) -> np.ndarray:
+        """raw [rows, queries | keys | values]; keys and values go to their pages, returns the queries [rows, heads, dim].  norm: 0 none,
+        1 per head, 2 whole projection.  v_first without v_lambda receives the values, with it they are blended."""
+        f = lambda a: None if a is None else np.ascontiguousarray(a, dtype=np.float32)
+        raw, qn, kn = f(raw), f(q_norm), f(k_norm)
+        s, p = np.ascontiguousarray(row_seq, dtype=np.int32), np.ascontiguousarray(row_pos, dtype=np.int32)
+        q = np.empty((raw.shape[0], self.heads, self.dim), np.float32)
+        _check(self._lib.hm_gqa_write(_ptr(raw), raw.shape[0], self.heads, self.kv_heads, self.dim, self.vdim, norm, _ptr(qn), _ptr(kn), eps, q_scale, temperature[0], temperature[1], _ptr(v_first), int(v_lambda is None), v_lambda or 0.0,
+                                      _ptr(self.k.ptr), _ptr(self.v.ptr), int(self.kv_dtype), _ptr(self.table), self.table.shape[0], self.table.shape[1], _ptr(s), _ptr(p), _ptr(q), None))
+        return q
+
+    def attend(self, q, row_seq, row_pos, bias=None, nsplit: int = 0) -> np.ndarray:
+        """q [rows, heads, dim], bias [heads, reach + 1] by distance (both as base-2 exponents) -> [rows, heads, vdim]."""
+        q = np.ascontiguousarray(q, dtype=np.float32)
+        b = None if bias is None else np.ascontiguousarray(bias, dtype=np.float32)
+        s, p = np.ascontiguousarray(row_seq, dtype=np.int32), np.ascontiguousarray(row_pos, dtype=np.int32)
+        out = np.empty((q.shape[0], self.heads, self.vdim), np.float32)
+        _check(self._lib.hm_gqa_attn_paged(_ptr(q), _ptr(self.k.ptr), _ptr(self.v.ptr), int(self.kv_dtype), _ptr(self.table), self.table.shape[0], self.table.shape[1], _ptr(s), _ptr(p), q.shape[0], self.heads, self.kv_heads, self.dim,
+                                           self.vdim, _ptr(b), 0 if b is None else b.shape[1] - 1, nsplit, _ptr(out), None))
+        return out
+
+
+def post_norm_route(y, x, w, mult: float, eps: float, identity=None, router=None, correction=None, experts: int = 0, top: int = 0):
+    """x + mult * RMSnorm(y + identity * x) * w; with a router (bf16 bits [outputs, width]) also (ids, weights, identity weight)."""
+    lib = load_library()
+    f = lambda a: None if a is None else np.ascontiguousarray(a, dtype=np.float32)
+    y, x, w, ident, corr = f(y), f(x).copy(), f(w), f(identity), f(correction)
+    M, W = x.shape
+    ids, wts, idw = np.zeros((M, max(top, 1)), np.int32), np.zeros((M, max(top, 1)), np.float32), np.zeros(M, np.float32)
+    r = None if router is None else np.ascontiguousarray(router, dtype=np.uint16)
+    _check(lib.hm_post_norm_route(_ptr(y), _ptr(ident), _ptr(x), M, W, _ptr(w), mult, eps, _ptr(r), _ptr(corr), experts, 0 if r is None else r.shape[0] - experts, top, _ptr(ids), _ptr(wts), _ptr(idw), None))
+    return x if r is None else (x, ids, wts, idw)
 
 
 def dev_sync():

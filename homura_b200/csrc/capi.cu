@@ -11,6 +11,8 @@
 
 #include "engine.h"
 #include "gemm_tc.h"
+#include "gqa_attn.h"
+#include "moe.h"
 #include "kquant.h"
 #include "latent_attn.h"
 #include "sampler.h"
@@ -1057,6 +1059,109 @@ int hm_latent_attn_paged(const float* q, const void* pages, int kv_dtype, const 
     if (rc != HM_OK) return rc;
     if (take_wait_err()) return gfail(HM_ERR_TIMEOUT, "hm_latent_attn_paged: a bounded device-side wait ran out");
     return HM_OK;
+}
+
+size_t hm_gqa_pool_bytes(int kv_heads, int d, int kv_dtype, int n_pages) { return kv_heads < 1 || d < 1 || n_pages < 1 ? 0 : n_pages * gqa_page_elems(kv_heads, d) * (kv_dtype == HM_BF16 ? 2 : 4); }
+
+int hm_gqa_write(const float* raw, int M, int heads, int kv_heads, int dim, int vdim, int qk_norm, const float* q_norm, const float* k_norm, float eps, float q_scale, float temp_coef, int temp_every, float* v_first, int keep_first,
+                 float v_lambda, void* k_pages, void* v_pages, int kv_dtype, const int32_t* page_table, int n_seq, int max_pages, const int32_t* row_seq, const int32_t* row_pos, float* q_out, void* stream) {
+    if (!raw || !k_pages || !v_pages || !page_table || !row_seq || !row_pos || !q_out || M < 1 || heads < 1 || kv_heads < 1 || heads % kv_heads != 0 || dim < 1 || vdim < 1 || n_seq < 1 || max_pages < 1 || qk_norm < 0 || qk_norm > 2 ||
+        (qk_norm && (!q_norm || !k_norm)) || temp_every < 0)
+        return gfail(HM_ERR_INVALID, "hm_gqa_write: bad arguments");
+    if (kv_dtype != HM_F32 && kv_dtype != HM_BF16) return gfail(HM_ERR_UNSUPPORTED, "hm_gqa_write: cache dtype must be f32 or bf16");
+    NEED_DEVICE();
+    if (!is_device_ptr(k_pages) || !is_device_ptr(v_pages)) return gfail(HM_ERR_INVALID, "hm_gqa_write: the pages must live in device memory");
+    if (is_device_ptr(row_seq) || is_device_ptr(row_pos)) return gfail(HM_ERR_INVALID, "hm_gqa_write: row_seq and row_pos are host arrays");
+    if (const int rc = check_latent_rows(row_seq, row_pos, M, n_seq, max_pages)) return rc;
+    cudaStream_t st = (cudaStream_t)stream;
+    Staging sg(st);
+    GqaPostArgs a{};
+    a.pool = GqaPool{k_pages, v_pages, sg.in(page_table, (size_t)n_seq * max_pages), max_pages, kv_heads, dim, vdim, kv_dtype == HM_BF16};
+    a.ld = heads * dim + kv_heads * (dim + vdim);
+    a.raw = sg.in(raw, (size_t)M * a.ld);
+    a.M = M;
+    a.heads = heads;
+    a.qk_norm = qk_norm;
+    a.q_norm = sg.in(q_norm, (size_t)(qk_norm == QKN_ALL ? heads * dim : dim));
+    a.k_norm = sg.in(k_norm, (size_t)(qk_norm == QKN_ALL ? kv_heads * dim : dim));
+    a.eps = eps;
+    a.q_scale = q_scale;
+    a.temp_coef = temp_coef;
+    a.temp_every = temp_every;
+    a.v_first = sg.out(v_first, (size_t)M * kv_heads * vdim, true);
+    a.v_lambda = v_first && !keep_first ? sg.in(&v_lambda, 1) : nullptr;
+    a.row_seq = sg.in(row_seq, (size_t)M);
+    a.row_pos = sg.in(row_pos, (size_t)M);
+    a.q_out = sg.out(q_out, (size_t)M * heads * dim);
+    if (!a.pool.page_table || !a.raw || !a.row_seq || !a.row_pos || !a.q_out || (qk_norm && (!a.q_norm || !a.k_norm)) || (v_first && (!a.v_first || (!keep_first && !a.v_lambda)))) return sg.finish(cudaErrorMemoryAllocation);
+    return sg.finish(launch_gqa_post(a, st, false));
+}
+
+int hm_gqa_attn_paged(const float* q, const void* k_pages, const void* v_pages, int kv_dtype, const int32_t* page_table, int n_seq, int max_pages, const int32_t* row_seq, const int32_t* row_pos, int M, int heads, int kv_heads, int dim,
+                      int vdim, const float* bias, int reach, int nsplit, float* out, void* stream) {
+    if (!q || !k_pages || !v_pages || !page_table || !row_seq || !row_pos || !out || M < 1 || M > GQA_MAX_ROWS || heads < 1 || kv_heads < 1 || heads % kv_heads != 0 || dim < 1 || vdim < 1 || n_seq < 1 || max_pages < 1 || nsplit < 0 ||
+        nsplit > 8 || (bias && reach < 0))
+        return gfail(HM_ERR_INVALID, "hm_gqa_attn_paged: bad arguments (M <= 64, nsplit <= 8)");
+    if (kv_dtype != HM_F32 && kv_dtype != HM_BF16) return gfail(HM_ERR_UNSUPPORTED, "hm_gqa_attn_paged: cache dtype must be f32 or bf16");
+    NEED_DEVICE();
+    if (!is_device_ptr(k_pages) || !is_device_ptr(v_pages)) return gfail(HM_ERR_INVALID, "hm_gqa_attn_paged: the pages must live in device memory");
+    if (is_device_ptr(row_seq) || is_device_ptr(row_pos)) return gfail(HM_ERR_INVALID, "hm_gqa_attn_paged: row_seq and row_pos are host arrays");
+    if (const int rc = check_latent_rows(row_seq, row_pos, M, n_seq, max_pages)) return rc;
+    cudaStream_t st = (cudaStream_t)stream;
+    Staging sg(st);
+    GqaAttnArgs a{};
+    a.pool = GqaPool{const_cast<void*>(k_pages), const_cast<void*>(v_pages), sg.in(page_table, (size_t)n_seq * max_pages), max_pages, kv_heads, dim, vdim, kv_dtype == HM_BF16};
+    a.q = sg.in(q, (size_t)M * heads * dim);
+    a.M = M;
+    a.heads = heads;
+    a.row_seq = sg.in(row_seq, (size_t)M);
+    a.row_pos = sg.in(row_pos, (size_t)M);
+    a.bias = sg.in(bias, (size_t)heads * (reach + 1));
+    a.reach = reach;
+    for (int m = 0; m < M; ++m) {
+        a.longest = std::max(a.longest, row_pos[m] + 1);
+        if (m == 0 || row_seq[m - 1] != row_seq[m] || row_pos[m - 1] + 1 != row_pos[m]) a.runs.row[a.runs.n++] = (uint8_t)m;
+        a.longest_run = std::max(a.longest_run, m + 1 - a.runs.row[a.runs.n - 1]);
+    }
+    a.runs.row[a.runs.n] = (uint8_t)M;
+    a.max_cluster = 8;
+    a.nsplit = nsplit;
+    a.out = sg.out(out, (size_t)M * heads * vdim);
+    if (!a.pool.page_table || !a.q || !a.row_seq || !a.row_pos || !a.out || (bias && !a.bias)) return sg.finish(cudaErrorMemoryAllocation);
+    if (!sg.ok(get_wait_err(&a.err_flag))) return sg.finish(cudaSuccess);
+    const int rc = sg.finish(launch_gqa_attn(a, sm_count_of_current_device(), st, false));  // the row arrays are always staged, so this call synchronised
+    if (rc != HM_OK) return rc;
+    if (take_wait_err()) return gfail(HM_ERR_TIMEOUT, "hm_gqa_attn_paged: a bounded device-side wait ran out");
+    return HM_OK;
+}
+
+int hm_post_norm_route(const float* y, const float* identity, float* x, int M, int W, const float* w, float mult, float eps, const uint16_t* router, const float* correction, int experts, int identities, int top, int32_t* ids,
+                       float* weights, float* id_weight, void* stream) {
+    if (!y || !x || !w || M < 1 || W < 1 || (router && (!correction || experts < 1 || identities < 0 || top < 1 || top > experts + identities || !ids || !weights || !id_weight))) return gfail(HM_ERR_INVALID, "hm_post_norm_route: bad arguments");
+    NEED_DEVICE();
+    cudaStream_t st = (cudaStream_t)stream;
+    Staging sg(st);
+    PostNormArgs a{};
+    a.y = sg.in(y, (size_t)M * W);
+    a.identity = sg.in(identity, (size_t)M);
+    a.x = sg.out(x, (size_t)M * W, true);
+    a.M = M;
+    a.W = W;
+    a.w = sg.in(w, (size_t)W);
+    a.mult = mult;
+    a.eps = eps;
+    if (router) {
+        a.n_out = experts + identities;
+        a.experts = experts;
+        a.top = top;
+        a.router = sg.in(router, (size_t)a.n_out * W);
+        a.correction = sg.in(correction, (size_t)a.n_out);
+        a.out.ids = sg.out(ids, (size_t)M * top);
+        a.out.weights = sg.out(weights, (size_t)M * top);
+        a.out.identity = sg.out(id_weight, (size_t)M);
+    }
+    if (!a.y || !a.x || !a.w || (identity && !a.identity) || (router && (!a.router || !a.correction || !a.out.ids || !a.out.weights || !a.out.identity))) return sg.finish(cudaErrorMemoryAllocation);
+    return sg.finish(launch_post_norm(a, sm_count_of_current_device(), st, false));
 }
 
 int hm_argmax(const float* logits, int rows, int n, uint32_t* out, void* stream) {

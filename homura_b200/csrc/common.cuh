@@ -242,8 +242,8 @@ __device__ __forceinline__ float warp_max(float v) {
 // PRO_GNORM: RMSNorm in equal groups, optionally followed by the token shift (see RowNorm)
 // PRO_MERGE: the input rows are the splits of an attention over latents, still to be combined (SplitRows)
 enum Prologue { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_GNORM = 2, PRO_MERGE = 3 };
-// EPI_GATE: y = acc * sigmoid(gate); EPI_SQRELU: y = max(acc, 0)^2
-enum Epilogue { EPI_STORE = 0, EPI_QKV_ROPE = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3, EPI_GATE = 4, EPI_SQRELU = 5 };
+// EPI_GATE: y = acc * sigmoid(gate); EPI_SQRELU: y = max(acc, 0)^2; EPI_EXPERT: gated activation of a mixture's experts
+enum Epilogue { EPI_STORE = 0, EPI_QKV_ROPE = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3, EPI_GATE = 4, EPI_SQRELU = 5, EPI_EXPERT = 6 };
 
 // Normalisation of a projection's input rows in `groups` equal runs, each divided by its own root mean square, and the
 // token shift h + (h' - h) * shift, where h' is the normalised row of the sequence's previous token before its own shift

@@ -77,6 +77,7 @@ int Engine::create(const ModelSpec& spec, int device, bool strict_f32, Engine** 
         for (const LayerSpec& l : spec.layers) {
             e->qdim_ = std::max(e->qdim_, l.heads * std::max(l.vdim, l.mixer == MIX_GQA ? l.dim : 0));
             if (l.kv_rank > 1024) return bad("kv_rank must be at most 1024");
+            if (l.experts > 1024) return bad("a mixture has at most 1024 experts");
         }
     } else {
         if (e->hd_ != 64 && e->hd_ != 128) return bad("head_dim must be 64 or 128");
@@ -1635,8 +1636,8 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
     if (batch_ == 0) return fail(HM_ERR_STATE, "profile_decode before kv_alloc");
     if (steps < 1 || !out || !n_out || cap < (spec_.listed() ? PC_COUNT_LISTED : PC_COUNT)) return fail(HM_ERR_INVALID, "profile_decode: bad arguments (cap >= 8; 14 for listed designs)");
     for (int b = 0; b < batch_; ++b)
-        if (len_[b] + steps > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full: not enough room for the profiled steps");
-    if (const int prc = ensure_pages_all(steps)) return prc;
+        if (len_[b] + steps + (spec_.post_norm ? 1 : 0) > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full: not enough room for the profiled steps");
+    if (const int prc = ensure_pages_all(steps + (spec_.post_norm ? 1 : 0))) return prc;
     const int classes = spec_.listed() ? PC_COUNT_LISTED : PC_COUNT;
     pass_longest_ = max_seq_;
     HM_CUDA(cudaStreamSynchronize(stream_));
@@ -1682,6 +1683,20 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
     cudaEventDestroy(e0);
     cudaEventDestroy(e1);
     if (rc) return rc;
+    if (spec_.post_norm) {  // which experts such a step reads: one more pass, without logits, at the position it has reached
+        std::vector<int> seen;
+        int launches = 0;
+        experts_seen_ = &seen;
+        const int chunk = std::min(batch_, TC_ROWS);
+        rc = enqueue_pass(chunk, tokens_dev_, pos_dev_, seq_iota_, 0, 0, false, next_dev_, nullptr, nullptr, nullptr, &launches);
+        experts_seen_ = nullptr;
+        if (rc) return rc;
+        HM_CUDA(cudaStreamSynchronize(stream_));
+        experts_read_.assign(L_, 0);
+        size_t k = 0;
+        for (int l = 0; l < L_; ++l)
+            if (spec_.layers[l].mlp == MLP_MOE && k < seen.size()) experts_read_[l] = seen[k++] * ((batch_ + chunk - 1) / chunk);
+    }
     for (int b = 0; b < batch_; ++b) len_[b] += steps;
     uint64_t bytes[PC_COUNT_LISTED] = {0};
     bytes[PC_EMBED] = (uint64_t)batch_ * H_ * (embed_dtype_ == HM_BF16 ? 2 : 4);
@@ -1689,8 +1704,8 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
         bytes[PC_QKV] += l.qkv.bytes() + l.in.bytes();
         const int li = (int)(&l - layers_.data());
         bytes[PC_ROUTE] += l.router ? (uint64_t)(spec_.layers[li].experts + spec_.layers[li].identity) * H_ * 2 : 0;
-        bytes[PC_GATE_UP] += expert_bytes(li, batch_, true);
-        bytes[PC_DOWN] += expert_bytes(li, batch_, false);
+        bytes[PC_GATE_UP] += expert_bytes(li, true);
+        bytes[PC_DOWN] += expert_bytes(li, false);
         bytes[PC_KUP] += l.kup.bytes();
         bytes[PC_VUP] += l.vup.bytes();
         bytes[PC_O] += l.o.bytes();

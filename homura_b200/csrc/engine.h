@@ -156,9 +156,11 @@ class Engine {
     int alloc_gqa_scratch();
     void free_gqa_scratch();
     GqaPool gqa_pool(int layer) const;
-    RouteOut route_out(const LayerSpec& s) const;
+    RouteOut route_out(bool dense) const;
+    double experts_used(const LayerSpec& s, int rows) const;
     ExpertWeights expert_weights(int layer) const;
-    uint64_t expert_bytes(int layer, int rows, bool gate_up) const;
+    uint64_t expert_bytes(int layer, bool gate_up) const;
+    int count_experts(int M, const LayerSpec& s);
     int enqueue_gqa_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int next_lm_rows, int* launches);
     int enqueue_listed_logits(const float* x, int rows, float* dst, const struct ArgmaxFold& fold, int* launches);
     int enqueue_tc(const LinearW& L, int M, const unsigned char* xp, int epi, float* y, int ldy, TcArgs& a, int* launches);
@@ -255,7 +257,11 @@ class Engine {
     int32_t* rt_ids_ = nullptr;      // router's choice (RouteOut)
     float *rt_weights_ = nullptr, *rt_identity_ = nullptr, *rt_dense_ = nullptr;
     uint32_t* rt_mask_ = nullptr;
-    float* exp_act_ = nullptr;       // activations of the chosen experts
+    float* exp_act_ = nullptr;       // activations of the chosen experts: few rows,
+    unsigned char* exp_img_ = nullptr;  // or an image per expert
+    int sub_parts_ = 1;              // partial results sub_ has room for
+    std::vector<int>* experts_seen_ = nullptr;  // profile: experts used per layer of the pass being enqueued
+    std::vector<int> experts_read_;  // their counts of the last profiled step
     int32_t* seq_iota_ = nullptr;    // 0, 1, 2, ...: the sequence of every row of a decode step
     int pass_nsplit_ = 1;            // splits the attention of the layer being enqueued left for the next projection to combine
     int pass_longest_ = 0;           // longest context of the pass being enqueued (splits of the attention)

@@ -159,32 +159,35 @@ void Engine::free_gqa_scratch() {
         if (p) cudaFree(p);
         p = nullptr;
     };
-    fr(sub_); fr(v_first_); fr(rt_ids_); fr(rt_weights_); fr(rt_identity_); fr(rt_dense_); fr(rt_mask_); fr(exp_act_);
+    fr(sub_); fr(v_first_); fr(rt_ids_); fr(rt_weights_); fr(rt_identity_); fr(rt_dense_); fr(rt_mask_); fr(exp_act_); fr(exp_img_);
 }
 
 // A pass of a listed design has at most TC_ROWS rows.
 int Engine::alloc_gqa_scratch() {
     if (!spec_.post_norm) return HM_OK;
-    size_t values = 1, top = 1, experts = 1, act = 1;
+    size_t values = 1, top = 1, experts = 1, act = 1, img = 1;
     for (const LayerSpec& s : spec_.layers) {
         if (s.v_mix) values = std::max(values, (size_t)s.kv_heads * s.vdim);
         if (s.mlp != MLP_MOE) continue;
         top = std::max(top, (size_t)s.top);
         experts = std::max(experts, (size_t)s.experts);
         act = std::max(act, (size_t)s.top * expert_blocks(s.ff) * 64);
+        img = std::max(img, (size_t)s.experts * tc_xpack_bytes(TC_ROWS, s.ff));
     }
     auto get = [&](auto** p, size_t count) -> cudaError_t {
         const cudaError_t e = cudaMalloc((void**)p, count * sizeof(**p));
         return e == cudaSuccess ? cudaMemset(*p, 0, count * sizeof(**p)) : e;
     };
-    HM_CUDA(get(&sub_, (size_t)TC_ROWS * H_));
+    sub_parts_ = std::max(1, sm_count_ / ((H_ + SLAB - 1) / SLAB * 8));
+    HM_CUDA(get(&sub_, (size_t)TC_ROWS * H_ * sub_parts_));
     HM_CUDA(get(&v_first_, TC_ROWS * values));
     HM_CUDA(get(&rt_ids_, TC_ROWS * top));
     HM_CUDA(get(&rt_weights_, TC_ROWS * top));
     HM_CUDA(get(&rt_identity_, TC_ROWS));
     HM_CUDA(get(&rt_dense_, TC_ROWS * experts));
     HM_CUDA(get(&rt_mask_, TC_ROWS * ((experts + 31) / 32)));
-    HM_CUDA(get(&exp_act_, TC_ROWS * act));
+    HM_CUDA(get(&exp_act_, (use_tc_ ? MAX_M : TC_ROWS) * act));
+    if (use_tc_) HM_CUDA(get(&exp_img_, img));
     return HM_OK;
 }
 
@@ -193,19 +196,32 @@ GqaPool Engine::gqa_pool(int layer) const {
     return GqaPool{k_pool_[layer], v_pool_[layer], page_table_, max_pages_, s.kv_heads, s.dim, s.vdim, kv_bf16_ ? 1 : 0};
 }
 
-RouteOut Engine::route_out(const LayerSpec&) const { return RouteOut{rt_ids_, rt_weights_, rt_identity_, nullptr, rt_mask_}; }
+RouteOut Engine::route_out(bool dense) const { return RouteOut{rt_ids_, rt_weights_, rt_identity_, dense ? rt_dense_ : nullptr, rt_mask_}; }
+
+// Experts that so many rows use, if their choices are spread evenly.
+double Engine::experts_used(const LayerSpec& s, int rows) const { return s.experts * (1.0 - std::pow(1.0 - s.top / (double)(s.experts + s.identity), rows)); }
 
 ExpertWeights Engine::expert_weights(int layer) const {
     const LayerSpec& s = spec_.layers[layer];
     return ExpertWeights{layers_[layer].exp_gu, layers_[layer].exp_down, H_, s.ff, s.top, s.limit};
 }
 
-// Bytes of expert weights that a step over so many rows reads, if its choices are spread evenly.
-uint64_t Engine::expert_bytes(int layer, int rows, bool gate_up) const {
-    if (!spec_.listed() || spec_.layers[layer].mlp != MLP_MOE) return 0;
-    const LayerSpec& s = spec_.layers[layer];
-    const double outs = s.experts + s.identity, used = s.experts * (1.0 - std::pow(1.0 - s.top / outs, rows));
-    return (uint64_t)(used * (gate_up ? 2.0 : 1.0) * s.ff * H_ * 2.0);
+// Bytes of expert weights that the last profiled step read.
+uint64_t Engine::expert_bytes(int layer, bool gate_up) const {
+    if (!spec_.listed() || spec_.layers[layer].mlp != MLP_MOE || (int)experts_read_.size() <= layer) return 0;
+    return (uint64_t)experts_read_[layer] * (gate_up ? 2 : 1) * spec_.layers[layer].ff * H_ * 2;
+}
+
+// Experts that the rows of the pass being enqueued have chosen (waits for the router).
+int Engine::count_experts(int M, const LayerSpec& s) {
+    std::vector<int32_t> ids((size_t)M * s.top);
+    HM_CUDA(cudaMemcpyAsync(ids.data(), rt_ids_, ids.size() * 4, cudaMemcpyDeviceToHost, stream_));
+    HM_CUDA(cudaStreamSynchronize(stream_));
+    std::sort(ids.begin(), ids.end());
+    int n = 0;
+    for (size_t i = 0; i < ids.size(); ++i) n += ids[i] >= 0 && (i == 0 || ids[i] != ids[i - 1]);
+    experts_seen_->push_back(n);
+    return HM_OK;
 }
 
 // ---- one layer ---------------------------------------------------------------------------------------
@@ -322,26 +338,78 @@ int Engine::enqueue_gqa_layer(int l, int M, const int32_t* row_pos, const int32_
             a.experts = s.experts;
             a.n_out = s.experts + s.identity;
             a.top = s.top;
-            a.out = route_out(s);
+            a.out = route_out(tall);
         }
         ce = launch_post_norm(a, sm_count_, stream_, pdl_);
         if (ce != cudaSuccess) return cuda_fail(ce, "norm launch");
         ++*launches;
+        if (experts_seen_ && moe) {
+            rc = count_experts(M, s);
+            if (rc) return rc;
+        }
     }
     if (!moe) return HM_OK;
+    TcArgs ta{};
+    if (tall) {
+        ta.ex.n = s.experts;
+        ta.ex.blocks = expert_blocks(s.ff);
+        ta.ex.weight = rt_dense_;
+        ta.ex.mask = rt_mask_;
+        ta.ex.limit = s.limit;
+        ta.ex.img_bytes = tc_xpack_bytes(M, s.ff);
+        ta.ex.used = std::max(1, (int)experts_used(s, M));
+        ta.ex.parts = 1;
+        ta.ex.part_stride = (size_t)TC_ROWS * H_;
+        ta.M = M;
+        ta.xp_mpad = tc_mpad(M);
+        ta.err_flag = err_flag_;
+    }
     if (want(PC_GATE_UP)) {
-        ce = launch_expert_gate_up(expert_weights(l), h_, M, route_out(s), exp_act_, stream_, pdl_);
+        if (tall) {
+            TcArgs a = ta;
+            a.W = w.exp_gu;
+            a.K = H_;
+            a.Kp = tc_padded_k(H_);
+            a.N = s.experts * a.ex.blocks * SLAB;
+            a.ksplit = tc_pick_split(H_, a.ex.used * a.ex.blocks * SLAB, sm_count_);
+            a.xp = xpack_;
+            a.epi = EPI_EXPERT;
+            a.xp_out = exp_img_;
+            ce = launch_gemm_tc(a, stream_, pdl_);
+        } else {
+            ce = launch_expert_gate_up(expert_weights(l), h_, M, route_out(tall), exp_act_, stream_, pdl_);
+        }
         if (ce != cudaSuccess) return cuda_fail(ce, "expert gate / up launch");
         ++*launches;
     }
+    // the sum over the experts' activations is long: with few output blocks it is cut into parts, which the norm adds up
+    const int down_k = ta.ex.used * expert_blocks(s.ff) * 64, down_split = tc_pick_split(down_k, H_, sm_count_);
+    const int parts = !tall ? 1 : std::max(1, std::min({sub_parts_, sm_count_ / ((H_ + SLAB - 1) / SLAB * down_split), down_k / 64 / (4 * down_split)}));
     if (want(PC_DOWN)) {
-        ce = launch_expert_down(expert_weights(l), exp_act_, M, route_out(s), sub_, stream_, pdl_);
+        if (tall) {
+            TcArgs a = ta;
+            a.W = w.exp_down;
+            a.K = s.ff;
+            a.Kp = tc_padded_k(s.ff);
+            a.N = H_;
+            a.ksplit = down_split;
+            a.ex.parts = parts;
+            a.xp = exp_img_;
+            a.epi = EPI_STORE;
+            a.y = sub_;
+            a.ldy = H_;
+            ce = launch_gemm_tc(a, stream_, pdl_);
+        } else {
+            ce = launch_expert_down(expert_weights(l), exp_act_, M, route_out(tall), sub_, stream_, pdl_);
+        }
         if (ce != cudaSuccess) return cuda_fail(ce, "expert down launch");
         ++*launches;
     }
     if (want(PC_NORM)) {
         PostNormArgs a = pn;
         a.w = w.post_ln;
+        a.parts = parts;
+        a.part_stride = (size_t)TC_ROWS * H_;
         a.identity = s.identity > 0 ? rt_identity_ : nullptr;
         ce = launch_post_norm(a, sm_count_, stream_, pdl_);
         if (ce != cudaSuccess) return cuda_fail(ce, "norm launch");

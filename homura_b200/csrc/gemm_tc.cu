@@ -23,11 +23,13 @@
 // Roles: warp 0 = bulk-copy producer, warp 1 = TMEM owner + MMA issuer, warps 2-5 = activation
 // staging (f32 -> 3 x bf16, swizzled) and epilogue.  Every mbarrier wait is bounded.
 #include <cstdlib>
+#include <type_traits>
 
 #include "common.cuh"
 #include "gemm_tc.h"
 #include "launch_attrs.h"
 #include "mbarrier.cuh"
+#include "moe.h"
 
 namespace hm {
 namespace {
@@ -248,13 +250,28 @@ __global__ void __launch_bounds__(256) tc_pack_gnorm_kernel(const float* __restr
 // The same four epilogues as the streaming projection kernel (gemv_bf16.cu), for up to 64 rows.
 __device__ __forceinline__ bool tc_better(float v, int i, float bv, int bi) { return v > bv || (v == bv && i > bi); }
 
-// X: the extended variant (grouped weights, output scale, gate, squared ReLU, queries split into images), compiled apart so that the
-// plain projections carry none of it.
-template <bool X>
+// V: 1 is the extended variant (grouped weights, output scale, gate, squared ReLU, queries split into images), 2 that of mixtures of
+// experts, compiled apart so that the plain projections carry none of it.
+template <int V>
 __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, int nblk, int tid, const int* s_pos, const int* s_page) {
     // grouped projections: this block's output columns [n0, n_end)
+    constexpr bool X = V == 1;
     const int rows = m_hi - m_lo;
     int n0 = nblk * BM, n_end = a.N;
+    if constexpr (V == 2) {
+        if (a.epi == EPI_EXPERT) {
+            const int e = nblk / a.ex.blocks, k0 = (nblk - e * a.ex.blocks) * 64;
+            for (int idx = tid; idx < rows * 8; idx += TC_THREADS) {
+                const int m = m_lo + idx / 8, c = (idx % 8) * 8;
+                const float rw = ld_cg_f32(a.ex.weight + (size_t)m * a.ex.n + e);
+                float act[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) act[i] = rw == 0.f ? 0.f : clamped_glu(tile[m * BM + c + i], tile[m * BM + 64 + c + i], a.ex.limit) * rw;
+                tc_xpack_store8(a.xp_out + (size_t)e * a.ex.img_bytes, a.xp_mpad, m, k0 + c, act);
+            }
+            return;
+        }
+    }
     if constexpr (X) {
         if (a.group_blocks) {
             const int grp = nblk / a.group_blocks;
@@ -490,10 +507,18 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
 }
 
 // ---- the GEMM: warp 0 = bulk-copy producer, warp 1 = TMEM owner + MMA issuer, warps 2-5 = epilogue ----
-template <bool CL, bool X>
+struct ExpertList {
+    uint32_t mask[32];
+    uint16_t id[1024];
+    int n;
+};
+
+template <bool CL, int V>
 __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) {
+    constexpr bool X = V == 1;
     extern __shared__ __align__(1024) unsigned char dsm[];
     __shared__ TcShared sh;
+    __shared__ typename std::conditional<V == 2, ExpertList, int>::type xl;
     unsigned char* stage0 = dsm + ((1024u - (s32(dsm) & 1023u)) & 1023u);  // swizzle atoms need 1024-byte alignment
     const int mpad = a.mpad;
     const uint32_t x_tile = (uint32_t)(TERMS * mpad * 128);
@@ -507,12 +532,12 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) 
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int cs = CL ? a.ksplit : 1;
-    const int nblk = blockIdx.x / cs;
+    int nblk = blockIdx.x / cs, part = 0;
     const int split = blockIdx.x - nblk * cs;
-    const int kb_total = a.Kp / BK;
-    const int kb_per = (kb_total + cs - 1) / cs;
-    const int kb0 = split * kb_per, kb1 = min(kb_total, kb0 + kb_per);
-    const int nkb = max(0, kb1 - kb0);
+    int kb_total = a.Kp / BK;
+    int kb_per = (kb_total + cs - 1) / cs;
+    int kb0 = split * kb_per, kb1 = min(kb_total, kb0 + kb_per);
+    int nkb = max(0, kb1 - kb0);
     const int nst = a.nstage;
     HM_TRACE(const bool tr = a.trace != nullptr && blockIdx.x == 0;)
     HM_TRACE(if (tr && tid == 0) a.trace[0] = global_timer();)
@@ -539,6 +564,42 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) 
     }
     if (CL) cluster_sync_all(); else
     __syncthreads();
+    if constexpr (V == 2) {
+        // who chose what was stored by the launch in front of the gate / up projection
+        pdl_launch_dependents();
+        pdl_wait();
+        const int words = (a.ex.n + 31) / 32;
+        if (a.epi == EPI_EXPERT) {
+            const int e = nblk / a.ex.blocks;
+            const bool chosen = tid < a.M && (__ldcg(a.ex.mask + (size_t)tid * words + e / 32) >> (e & 31) & 1u);
+            if (!__syncthreads_or(chosen)) return;  // the same for every CTA of the cluster
+        } else {
+            part = nblk / ((a.N + BM - 1) / BM);
+            nblk -= part * ((a.N + BM - 1) / BM);
+            if (tid < words) xl.mask[tid] = 0u;
+            __syncthreads();
+            for (int i = tid; i < a.M * words; i += TC_THREADS) {
+                const uint32_t v = __ldcg(a.ex.mask + i);
+                if (v) atomicOr(&xl.mask[i % words], v);
+            }
+            __syncthreads();
+            if (warp == 0) {
+                int n = 0;
+                for (int w = 0; w < words; ++w) {
+                    const uint32_t v = xl.mask[w];
+                    if (v >> lane & 1u) xl.id[n + __popc(v & ((1u << lane) - 1u))] = (uint16_t)(w * 32 + lane);
+                    n += __popc(v);
+                }
+                if (lane == 0) xl.n = n;
+            }
+            __syncthreads();
+            kb_total = xl.n * a.ex.blocks;
+            kb_per = (kb_total + cs * a.ex.parts - 1) / (cs * a.ex.parts);
+            kb0 = (part * cs + split) * kb_per;
+            kb1 = min(kb_total, kb0 + kb_per);
+            nkb = max(0, kb1 - kb0);
+        }
+    }
     if (warp == 1) {  // TMEM: allocated and later freed by this warp
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(s32(&sh.tmem_base)), "r"(a.tmem_cols) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
@@ -551,7 +612,24 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) 
 
     pdl_launch_dependents();
 
-    if (warp == 0) {
+    bool produced = false;
+    if constexpr (V == 2) {
+        if (a.epi != EPI_EXPERT && warp == 0) {  // down: k-blocks of the chosen experts
+            if (lane == 0) {
+                const int nbs = (a.N + BM - 1) / BM;
+                for (int i = 0; i < nkb; ++i) {
+                    const int s = i % nst, slot = (kb0 + i) / a.ex.blocks, kb = kb0 + i - slot * a.ex.blocks, e = xl.id[slot];
+                    if (i >= nst && !mb_wait(&sh.empty[s], ((i / nst) & 1u) ^ 1u, a.err_flag, &sh.abort_flag)) break;
+                    mb_expect_tx(&sh.full[s], stage_bytes);
+                    bulk_copy(stage0 + (size_t)s * stage_bytes, reinterpret_cast<const unsigned char*>(a.W) + (((size_t)e * nbs + nblk) * a.ex.blocks + kb) * W_TILE, W_TILE, &sh.full[s]);
+                    bulk_copy(stage0 + (size_t)s * stage_bytes + W_TILE, a.xp + (size_t)e * a.ex.img_bytes + (size_t)kb * x_tile, x_tile, &sh.full[s]);
+                }
+            }
+            produced = true;
+        }
+    }
+    if (V == 2 && produced) {
+    } else if (warp == 0) {
         if (lane == 0) {
             const unsigned char* wsrc = reinterpret_cast<const unsigned char*>(a.W) + ((size_t)nblk * kb_total + kb0) * W_TILE;
             const unsigned char* xsrc = a.xp + (X && a.group_blocks ? (size_t)(nblk / a.group_blocks) * a.group_xp : 0) + (size_t)kb0 * x_tile;
@@ -688,7 +766,15 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) 
         __syncthreads();
     }
     HM_TRACE(if (tr && tid == 0) a.trace[8] = global_timer();)
-    tc_epilogue<X>(a, out_tile, m_lo, m_hi, nblk, tid, sh.pos, sh.page);
+    if constexpr (V == 2) {
+        if (part > 0) {
+            TcArgs b = a;
+            b.y += (size_t)part * a.ex.part_stride;
+            tc_epilogue<V>(b, out_tile, m_lo, m_hi, nblk, tid, sh.pos, sh.page);
+            return;
+        }
+    }
+    tc_epilogue<V>(a, out_tile, m_lo, m_hi, nblk, tid, sh.pos, sh.page);
     HM_TRACE(if (tr && tid == 0) a.trace[9] = global_timer();)
     HM_TRACE(if (tr && tid == 0) a.trace[10] = global_timer();)
     HM_TRACE(if (a.trace && tid == 0) atomicMax(a.trace + 12, global_timer());)
@@ -754,22 +840,31 @@ cudaError_t launch_tc_pack_gnorm(const float* x, int ldx, int M, int K, const fl
     return cudaLaunchKernelEx(&cfg, tc_pack_gnorm_kernel, x, ldx, M, tc_mpad(M), K, Kp, norm_w, eps, gn, (unsigned char*)xp);
 }
 
-template <bool X>
-static cudaError_t launch_gemm_tc_x(const TcArgs& a_in, cudaStream_t st, bool pdl) {
+template <int V>
+static cudaError_t launch_gemm_tc_v(const TcArgs& a_in, cudaStream_t st, bool pdl) {
     TcArgs a = a_in;
     if (a.M < 1 || a.M > MR || a.Kp % BK != 0 || !a.xp) return cudaErrorInvalidValue;
     a.mpad = tc_mpad(a.M);
     int dev = 0, sms = 148;
     if (cudaGetDevice(&dev) == cudaSuccess) cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    const int nblk = a.group_blocks ? a.N / a.group_n * a.group_blocks : (a.N + BM - 1) / BM;
-    const bool multi_wave = (long)nblk * (a.ksplit > 1 ? a.ksplit : 1) >= 2L * sms;
+    int nblk = a.group_blocks ? a.N / a.group_n * a.group_blocks : (a.N + BM - 1) / BM, busy = nblk;
+    if (V == 2) {
+        if (a.ex.n < 1 || a.ex.n > 1024 || a.ex.parts < 1) return cudaErrorInvalidValue;
+        if (a.epi == EPI_EXPERT) {
+            nblk = a.ex.n * a.ex.blocks;
+            busy = a.ex.used * a.ex.blocks;
+        } else {
+            busy = nblk *= a.ex.parts;
+        }
+    }
+    const bool multi_wave = (long)busy * (a.ksplit > 1 ? a.ksplit : 1) >= 2L * sms;
     a.nstage = tc_nstage(a.mpad, multi_wave);
     a.tmem_cols = a.mpad == 16 ? 64 : a.mpad == 32 ? 128 : 256;  // power of two >= 3 * mpad
     const bool cl = a.ksplit > 1;
     const size_t smem = tc_smem_for(a.mpad, multi_wave) + (cl ? tc_recv_bytes(a.M, a.ksplit) : 0);
     {
         const size_t mx = (tc_smem_for(64, false) > tc_smem_for(32, false) ? tc_smem_for(64, false) : tc_smem_for(32, false)) + (cl ? (size_t)(MR + 16) * BM * 4 : 0);
-        cudaError_t e = cl ? ensure_dyn_smem(gemm_tc_kernel<true, X>, mx) : ensure_dyn_smem(gemm_tc_kernel<false, X>, mx);
+        cudaError_t e = cl ? ensure_dyn_smem(gemm_tc_kernel<true, V>, mx) : ensure_dyn_smem(gemm_tc_kernel<false, V>, mx);
         if (e != cudaSuccess) return e;
     }
     cudaLaunchConfig_t cfg = {};
@@ -787,7 +882,7 @@ static cudaError_t launch_gemm_tc_x(const TcArgs& a_in, cudaStream_t st, bool pd
     if (cl) {
         if (a.ksplit > 16) return cudaErrorInvalidValue;
         if (a.ksplit > 8) {  // clusters of 9..16 CTAs are allowed on request
-            cudaError_t e = ensure_nonportable_clusters(gemm_tc_kernel<true, X>);
+            cudaError_t e = ensure_nonportable_clusters(gemm_tc_kernel<true, V>);
             if (e != cudaSuccess) return e;
         }
         at[n].id = cudaLaunchAttributeClusterDimension;
@@ -798,12 +893,13 @@ static cudaError_t launch_gemm_tc_x(const TcArgs& a_in, cudaStream_t st, bool pd
     }
     cfg.attrs = at;
     cfg.numAttrs = n;
-    return cl ? cudaLaunchKernelEx(&cfg, gemm_tc_kernel<true, X>, a) : cudaLaunchKernelEx(&cfg, gemm_tc_kernel<false, X>, a);
+    return cl ? cudaLaunchKernelEx(&cfg, gemm_tc_kernel<true, V>, a) : cudaLaunchKernelEx(&cfg, gemm_tc_kernel<false, V>, a);
 }
 
 cudaError_t launch_gemm_tc(const TcArgs& a, cudaStream_t st, bool pdl) {
     const bool x = a.group_blocks || a.out_scale || a.split_xp || a.epi == EPI_GATE || a.epi == EPI_SQRELU;
-    return x ? launch_gemm_tc_x<true>(a, st, pdl) : launch_gemm_tc_x<false>(a, st, pdl);
+    if (a.ex.n) return launch_gemm_tc_v<2>(a, st, pdl);
+    return x ? launch_gemm_tc_v<1>(a, st, pdl) : launch_gemm_tc_v<0>(a, st, pdl);
 }
 
 // ---- weight packing: [N][K] (HF [out,in]) or [K][N] bf16 -> swizzled K-major tiles ----------

@@ -9,6 +9,24 @@ namespace hm {
 
 constexpr int TC_ROWS = 64;  // activation rows one launch covers
 
+// Mixture of experts: every expert that some row of the pass chose is multiplied with all rows; a row's weight for an expert (0: not
+// chosen) scales its activations between the two projections, so that the second sums over the experts by itself.
+//   EPI_EXPERT  gate and up: W holds the blocks of all experts, blocks of experts nobody chose are skipped; the activations go to one
+//               image per expert (xp_out, img_bytes apart)
+//   EPI_STORE   down: the contraction runs over the k-blocks of the chosen experts; `parts` groups of CTAs take a share each and
+//               store to y + part * part_stride
+struct TcExperts {
+    int n;                  // experts, at most 1024; 0: not a mixture
+    int blocks;             // 64-element blocks of an expert's activations
+    const float* weight;    // [M][n]
+    const uint32_t* mask;   // [M][ceil(n / 32)] chosen experts
+    float limit;
+    size_t img_bytes;
+    int parts;
+    size_t part_stride;
+    int used;               // experts that are likely chosen by some row (launch shape)
+};
+
 struct TcArgs {
     const uint16_t* W;  // swizzled K-major tiles [n-block][k-block][128][64] bf16 (launch_pack_tc)
     int K, Kp, N;       // contraction length, K rounded up to 64, output features
@@ -33,7 +51,8 @@ struct TcArgs {
     unsigned char* split_xp;
     int split_n, split_k;
     size_t split_bytes;
-    unsigned char* xp_out;   // EPI_SWIGLU, EPI_GATE and EPI_SQRELU, optional: write the result as packed activations for the next GEMM instead of y
+    TcExperts ex;
+    unsigned char* xp_out;   // EPI_SWIGLU, EPI_GATE, EPI_EXPERT and EPI_SQRELU, optional: write the result as packed activations for the next GEMM instead of y
     int xp_mpad;
     // RMSNorm across two GEMMs without a packing launch in between.  Producer side (EPI_STORE): besides y, the
     // epilogue writes (y * next_norm_w) as the packed activations of the next GEMM and, per 128-feature block,

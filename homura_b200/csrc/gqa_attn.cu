@@ -639,7 +639,7 @@ cudaError_t launch_mma(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
     }
     const int pages = (a.longest + GQA_PAGE - 1) / GQA_PAGE, pairs = a.tiles * a.pool.kv_heads;
     constexpr int PER_SM = NT == 1 && VT <= 8 ? 2 : 1;
-    a.nsplit = std::max(1, std::min({PER_SM * sm_count / pairs, a.max_cluster, MAX_CLUSTER, pages}));
+    if (a.nsplit < 1) a.nsplit = std::max(1, std::min({PER_SM * sm_count / pairs, a.max_cluster, MAX_CLUSTER, pages}));
     const size_t stage = b_stage_bytes(dp, vp);
     const int ppc = (pages + a.nsplit - 1) / a.nsplit;
     const size_t fixed = b_query_bytes(NT, dp) + sizeof(float) * ((size_t)a.nsplit * P + 2 * P) + 4 * (size_t)ppc + 128;
@@ -670,7 +670,7 @@ cudaError_t launch_gqa_post(const GqaPostArgs& a, cudaStream_t st, bool pdl) {
 
 cudaError_t launch_gqa_attn(const GqaAttnArgs& a_in, int sm_count, cudaStream_t st, bool pdl) {
     GqaAttnArgs a = a_in;
-    if (a.M < 1 || a.M > GQA_MAX_ROWS || a.heads % a.pool.kv_heads != 0) return cudaErrorInvalidValue;
+    if (a.M < 1 || a.M > GQA_MAX_ROWS || a.nsplit > MAX_CLUSTER || a.heads % a.pool.kv_heads != 0) return cudaErrorInvalidValue;
     if (!a.bias) a.reach = 0;
     const int g = a.heads / a.pool.kv_heads, dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
     if (a.runs.n == 0) a.longest_run = 1;
@@ -681,7 +681,7 @@ cudaError_t launch_gqa_attn(const GqaAttnArgs& a_in, int sm_count, cudaStream_t 
         return launch_mma_n<16>(a, sm_count, st, pdl);
     }
     const int pages = (a.longest + GQA_PAGE - 1) / GQA_PAGE;
-    a.nsplit = std::max(1, std::min({4 * sm_count / (a.M * a.pool.kv_heads), a.max_cluster, MAX_CLUSTER, pages}));
+    if (a.nsplit < 1) a.nsplit = std::max(1, std::min({4 * sm_count / (a.M * a.pool.kv_heads), a.max_cluster, MAX_CLUSTER, pages}));
     const size_t smem = sizeof(float) * (size_t)g * (dp + vp + 4 + GQA_PAGE + 3 + a.nsplit);
     const dim3 grid((unsigned)a.nsplit, (unsigned)a.pool.kv_heads, (unsigned)a.M);
     return a.pool.bf16 ? launch_clustered(gqa_attn_kernel<true>, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a) : launch_clustered(gqa_attn_kernel<false>, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a);

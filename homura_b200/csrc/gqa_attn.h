@@ -65,8 +65,9 @@ struct GqaAttnArgs {
     unsigned char* xp;
     int xp_mpad;
     int* err_flag;
+    int nsplit;              // CTAs that share a tile's context; 0: as many as suit the launch
     // filled in by the launcher
-    int tiles, tiles_per_row, nsplit, stages;
+    int tiles, tiles_per_row, stages;
 };
 cudaError_t launch_gqa_attn(const GqaAttnArgs& a, int sm_count, cudaStream_t st, bool pdl);
 // Positions [0, len) of a sequence as f32 [kv_heads][len][dim] and [kv_heads][len][vdim].

@@ -113,6 +113,10 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PostNormArgs a
         for (int i = tid; i < a.W / 4; i += THREADS) {
             const float4 xv = ld_cg_f32x4(x + 4 * (size_t)i);
             float4 yv = ld_cg_f32x4(y + 4 * (size_t)i);
+            for (int p = 1; p < a.parts; ++p) {
+                const float4 t = ld_cg_f32x4(y + p * a.part_stride + 4 * (size_t)i);
+                yv = make_float4(yv.x + t.x, yv.y + t.y, yv.z + t.z, yv.w + t.w);
+            }
             yv = make_float4(fmaf(idw, xv.x, yv.x), fmaf(idw, xv.y, yv.y), fmaf(idw, xv.z, yv.z), fmaf(idw, xv.w, yv.w));
             reinterpret_cast<float4*>(xs)[i] = xv;
             reinterpret_cast<float4*>(ys)[i] = yv;
@@ -120,7 +124,10 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PostNormArgs a
         }
     } else {
         for (int i = tid; i < a.W; i += THREADS) {
-            const float xv = ld_cg_f32(x + i), yv = fmaf(idw, xv, ld_cg_f32(y + i));
+            const float xv = ld_cg_f32(x + i);
+            float yv = ld_cg_f32(y + i);
+            for (int p = 1; p < a.parts; ++p) yv += ld_cg_f32(y + p * a.part_stride + i);
+            yv = fmaf(idw, xv, yv);
             xs[i] = xv;
             ys[i] = yv;
             ss = fmaf(yv, yv, ss);

@@ -18,7 +18,9 @@ struct RouteOut {
 
 // x += mult * RMSnorm(y) * w, and then, optionally, the router over the new x.
 struct PostNormArgs {
-    const float* y;          // [M][W] what the sublayer gave back
+    const float* y;          // [M][W] what the sublayer gave back; with parts > 1 the sum of so many, part_stride apart
+    int parts;
+    size_t part_stride;
     const float* identity;   // [M] or null: y + identity * x instead of y
     float* x;                // [M][W] residual
     int M, W;

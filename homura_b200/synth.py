@@ -282,6 +282,84 @@ def write_tunitar_model(model_dir: str, cfg: dict, seed: int, weights: Optional[
     return _write_model(model_dir, cfg, tunitar_tensor_specs(cfg), lambda s: tunitar_tensor(seed, s) if weights is None else weights[s[0]])
 
 
+# ---- Dipisun ----------------------------------------------------------------------------------
+
+
+def dipisun_mixer(heads: int, kv_heads: int, dim: int, vdim: int, reach: Optional[float] = None, temp: Optional[Tuple[float, int]] = None, v_mix: bool = False, scale: Optional[float] = None) -> dict:
+    """(type, mixer).  With `reach` the kind of attention that knows distances (and may have a query temperature), else the other."""
+    m: dict = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim**-0.5 if scale is None else scale, "v_mix": v_mix}
+    if reach is not None:
+        m["bias_max"] = reach
+        if temp is not None:
+            m["q_temp"] = {"coef": temp[0], "every": temp[1]}
+    return {"type": "attention_2" if reach is None else "attention", "mixer": m}
+
+
+def dipisun_layer(mixer: dict, ff: Optional[int] = None, experts: int = 1, identity: int = 0, top: int = 1, limit: float = 2.0) -> dict:
+    """One entry of the layer list; ff None: without a mixture."""
+    mlp = None if ff is None else {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "identity": identity, "top": top}}
+    return {**mixer, "mlp": mlp}
+
+
+def dipisun_config(width: int, vocab: int, layers: List[dict], mult: float = 0.4, eps: float = 1e-6, **extra) -> dict:
+    return {"architecture": "Dipisun", "width": width, "vocab": vocab, "norm": {"eps": eps}, "residual_mult": mult, "layers": layers, **extra}
+
+
+def dipisun_uniform(width: int, vocab: int, n_layers: int, heads: int, kv_heads: int, dim: int, ff: int, experts: int, top: int, identity: int) -> dict:
+    """Every third layer knows distances, all blend their values, all have a mixture."""
+    mix = [dipisun_mixer(heads, kv_heads, dim, dim, 1024 if i % 3 == 1 else None, (0.1, 512) if i % 3 == 1 else None, True) for i in range(n_layers)]
+    return dipisun_config(width, vocab, [dipisun_layer(m, ff, experts, identity, top) for m in mix], 0.25)
+
+
+# Dipisun stacks with the width, depth, heads and head size of the Qwen2.5 architectures above; the chosen experts of a token have the
+# MLP parameters of theirs (4 x 1216 = 4864, 8 x 1120 = 8960).
+DIPISUN_05B = dipisun_uniform(896, 151936, 24, 14, 2, 64, 1216, 16, 4, 0)
+DIPISUN_15B = dipisun_uniform(1536, 151936, 28, 12, 2, 128, 1120, 32, 8, 2)
+
+
+def dipisun_tensor_specs(cfg: dict, buckets: int = 32) -> List[Tuple[str, Tuple[int, ...], str]]:
+    """(name, shape, kind); buckets: rows of the distance tables."""
+    W, V = cfg["width"], cfg["vocab"]
+    specs: List[Tuple[str, Tuple[int, ...], str]] = [("embed", (V, W), "embed")]
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        q, k, v, o = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], m["heads"] * m["vdim"]
+        whole = layer["type"] == "attention"
+        specs += [(p + "mix.q", (q, W), "w"), (p + "mix.k", (k, W), "w"), (p + "mix.v", (v, W), "w"), (p + "mix.o", (W, o), "w")]
+        specs += [(p + "mix.q.norm", (q if whole else m["dim"],), "one"), (p + "mix.k.norm", (k if whole else m["dim"],), "one"), (p + "norm1", (W,), "one")]
+        if whole:
+            specs.append((p + "mix.rel", (buckets, m["heads"]), "embed"))
+        if m.get("v_mix"):
+            specs.append((p + "mix.vmix", (), "share"))
+        if layer.get("mlp") is not None:
+            f, r = layer["mlp"]["expert"]["ff"], layer["mlp"]["router"]
+            n = r["experts"] + r["identity"]
+            specs += [(p + "norm2", (W,), "one"), (p + "mlp.router", (n, W), "w"), (p + "mlp.correction", (n,), "small")]
+            for e in range(r["experts"]):
+                specs += [(f"{p}mlp.e{e}.gate", (f, W), "w"), (f"{p}mlp.e{e}.up", (f, W), "w"), (f"{p}mlp.e{e}.down", (W, f), "w")]
+    return specs + [("final.norm", (W,), "one"), ("head", (V, W), "w")]
+
+
+def dipisun_tensor(seed: int, spec) -> np.ndarray:
+    """bf16 bits of one tensor: linears N(0, 1/in), vectors around 1, shares around one half, corrections around 0."""
+    name, shape, kind = spec
+    if kind in ("small", "share"):
+        g = _rng(seed, name)
+        v = 0.05 * g.standard_normal(shape, dtype=np.float32) if kind == "small" else 0.25 + 0.5 * g.random(shape, dtype=np.float32)
+        return f32_to_bf16_rne(np.asarray(v, np.float32))
+    return tunitar_tensor(seed, spec)
+
+
+def dipisun_weights(cfg: dict, seed: int, buckets: int = 32) -> Dict[str, np.ndarray]:
+    """name -> bf16 bits of every tensor."""
+    return {s[0]: dipisun_tensor(seed, s) for s in dipisun_tensor_specs(cfg, buckets)}
+
+
+def write_dipisun_model(model_dir: str, cfg: dict, seed: int, weights: Optional[Dict[str, np.ndarray]] = None, buckets: int = 32) -> str:
+    """config.json + model.safetensors of a Dipisun model (weights: bits to write instead of the seeded ones)."""
+    return _write_model(model_dir, cfg, dipisun_tensor_specs(cfg, buckets), lambda s: dipisun_tensor(seed, s) if weights is None else weights[s[0]])
+
+
 def shard_hf_model(src_dir: str, dst_dir: str, n_shards: int = 2) -> str:
     """Rewrite a single-file checkpoint as `n_shards` safetensors files plus model.safetensors.index.json,
     the layout HfModel::load_with_dtype falls back to (src/hf/model.rs:86-127).  Tensors are dealt out

@@ -307,6 +307,24 @@ HM_API int hm_latent_write(const float* c, const float* w, float eps, int M, int
  * sees positions 0 .. row_pos[m] of sequence row_seq[m] (M <= 64).  row_seq and row_pos are HOST arrays (range-checked);
  * nsplit CTAs share a context (0 = choose). */
 HM_API int hm_latent_attn_paged(const float* q, const void* pages, int kv_dtype, const int32_t* page_table, int n_seq, int max_pages, const int32_t* row_seq, const int32_t* row_pos, int M, int heads, int rank, float scale, int nsplit, float* out, void* stream);
+/* Grouped-query attention with head sizes of any kind over a paged cache of 64-token pages: keys of `dim` and values of `vdim` elements
+ * in pools of hm_gqa_pool_bytes each (device memory, zeroed by the caller before first use).  Rows are as in hm_latent_write.
+ * hm_gqa_write takes a projection's rows raw [M, heads*dim + kv_heads*(dim + vdim)] (queries, keys, values): RMS norm of queries and
+ * keys (qk_norm 0 none, 1 per head with weights [dim], 2 over the whole projection), queries times q_scale * (1 + temp_coef *
+ * ln(floor((position + 1) / temp_every) + 1)) (temp_every 0: without), values blended with v_first [M, kv_heads*vdim] as
+ * (1 - v_lambda) v + v_lambda v_first (NULL: not; keep_first: v_first receives the values instead); q_out [M, heads*dim]. */
+HM_API size_t hm_gqa_pool_bytes(int kv_heads, int d, int kv_dtype, int n_pages);
+HM_API int hm_gqa_write(const float* raw, int M, int heads, int kv_heads, int dim, int vdim, int qk_norm, const float* q_norm, const float* k_norm, float eps, float q_scale, float temp_coef, int temp_every, float* v_first, int keep_first,
+                        float v_lambda, void* k_pages, void* v_pages, int kv_dtype, const int32_t* page_table, int n_seq, int max_pages, const int32_t* row_seq, const int32_t* row_pos, float* q_out, void* stream);
+/* out [M, heads, vdim] = softmax over the positions up to each row's own of 2^(q . k + bias), i.e. scores are base-2 exponents; bias
+ * [heads, reach + 1] by distance, its last entry for every distance beyond, or NULL; nsplit 0: the library's own choice, else <= 8. */
+HM_API int hm_gqa_attn_paged(const float* q, const void* k_pages, const void* v_pages, int kv_dtype, const int32_t* page_table, int n_seq, int max_pages, const int32_t* row_seq, const int32_t* row_pos, int M, int heads, int kv_heads,
+                             int dim, int vdim, const float* bias, int reach, int nsplit, float* out, void* stream);
+/* x [M, W] += mult * RMSnorm(y + identity * x) * w (identity [M] or NULL); with a router [experts + identities, W] bf16, the softmax of
+ * its logits over the new x, `top` choices by score + correction: ids [M, top] (-1 for identity experts), weights [M, top] the scores,
+ * id_weight [M] the sum of the chosen identity experts' scores. */
+HM_API int hm_post_norm_route(const float* y, const float* identity, float* x, int M, int W, const float* w, float mult, float eps, const uint16_t* router, const float* correction, int experts, int identities, int top, int32_t* ids,
+                              float* weights, float* id_weight, void* stream);
 /* argmax with ties to the highest index (src/generate.rs:457-468): logits [rows, n]. */
 HM_API int hm_argmax(const float* logits, int rows, int n, uint32_t* out, void* stream);
 
