@@ -9,8 +9,9 @@
 // bulk copies (one contiguous block of keys and one of values per page and head).  Every warp takes units of 16 tokens:
 //   scores^T [16 tokens x pairs] = K [16 x dim]      . Q^T        (K chunks through ldmatrix)
 //   out^T    [vdim x pairs]     += V^T [vdim x 16]   . P^T        (V chunks through ldmatrix, transposed)
-// Queries and weights are three bf16 terms each (exact to 2^-24), so that the products are f32 x bf16 ones.  The warps of a CTA and
-// then the CTAs of a cluster, which share the context of a tile, combine their results in shared memory.
+// Queries and weights are three bf16 terms each (exact to 2^-24), so that the products are f32 x bf16 ones.  The warps of a CTA add
+// their results up in shared memory; the CTAs of a cluster share the context of a tile and send one another their pairs' results by
+// asynchronous stores.
 #include "gqa_attn.h"
 
 #include <algorithm>
@@ -319,8 +320,10 @@ __device__ __forceinline__ uint32_t transpose8x8(uint32_t v) {
 
 __host__ __device__ inline size_t b_stage_bytes(int dp, int vp) { return (size_t)GQA_PAGE * (dp + vp) * 2; }
 __host__ __device__ inline size_t b_query_bytes(int nt, int dp) { return (size_t)nt * (dp / 16) * 3 * 32 * 8; }
-// the ring's memory serves the combination of the warps' results afterwards: maxima and sums of the warps, four partial results
-__host__ __device__ inline size_t b_merge_bytes(int nt, int vp) { return sizeof(float) * ((size_t)2 * ATT_WARPS * nt * 8 + (size_t)4 * nt * 8 * (vp + 4)); }
+// the ring's memory takes the warps' results afterwards: maxima, sums and values
+__host__ __device__ inline size_t b_merge_bytes(int nt, int vp) { return sizeof(float) * ATT_WARPS * nt * 8 * ((size_t)2 + vp + 4); }
+// what a CTA receives: from every split, its share of the pairs (values, maximum, sum)
+__host__ __device__ inline size_t b_recv_bytes(int nt, int vp, int nsplit) { return sizeof(float) * (size_t)nsplit * ((nt * 8 + nsplit - 1) / nsplit) * (vp + 4); }
 
 // VT: tiles of 16 value elements (at most), NT: tiles of eight pairs.
 template <int VT, int NT>
@@ -333,23 +336,12 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
     const uint32_t k_bytes = (uint32_t)(GQA_PAGE * dp * 2), v_bytes = (uint32_t)(GQA_PAGE * vp * 2), stage = k_bytes + v_bytes;
     unsigned char* ring = dyn;
     uint2* qf = reinterpret_cast<uint2*>(dyn + ring_bytes);                                 // [NT][kt_n][3][32]
-    float* wts = reinterpret_cast<float*>(dyn + ring_bytes + b_query_bytes(NT, dp));        // [nsplit][pairs]
-    float* ml = wts + a.nsplit * P;                                                         // [P][2]
-    int32_t* pt_s = reinterpret_cast<int32_t*>(ml + 2 * P);                                 // this CTA's pages
-    __shared__ uint64_t full[MAX_STAGES], empty[MAX_STAGES];
+    float* recv = reinterpret_cast<float*>(dyn + ring_bytes + b_query_bytes(NT, dp));       // [nsplit][pairs of this CTA][vp + 4]
+    int32_t* pt_s = reinterpret_cast<int32_t*>(dyn + ring_bytes + b_query_bytes(NT, dp) + b_recv_bytes(NT, vp, a.nsplit));  // this CTA's pages
+    __shared__ uint64_t full[MAX_STAGES], empty[MAX_STAGES], s_rbar;
     __shared__ volatile int s_abort;
     __shared__ int s_pos[P], s_bias[P];  // position of the pair's row (-1: no such pair), first element of its bias row
 
-    if (tid == 0) {
-        for (int s = 0; s < NST; ++s) {
-            mb_init(&full[s], 1);
-            mb_init(&empty[s], 4);
-        }
-        s_abort = 0;
-        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-    }
-    pdl_launch_dependents();
-    if (!a.early) pdl_wait();
     // this tile's pairs: run, first pair, rows
     int row0, rows, pair0;
     if (a.runs.n == 0) {
@@ -364,6 +356,24 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
         pair0 = (blockIdx.z - a.runs.tile[r]) * P;
     }
     const int pairs = min(P, rows * g - pair0);
+    // the splits of a tile share its pairs: pair p is combined and stored by split p % ns
+    const int ns = a.nsplit, rank = ns > 1 ? (int)cluster_ctarank() : 0, own = pairs > rank ? (pairs - rank + ns - 1) / ns : 0, own_most = (P + ns - 1) / ns;
+    if (tid == 0) {
+        for (int s = 0; s < NST; ++s) {
+            mb_init(&full[s], 1);
+            mb_init(&empty[s], 4);
+        }
+        mb_init(&s_rbar, 1);
+        s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        if (ns > 1 && own > 0) mb_expect_tx(&s_rbar, (uint32_t)((ns - 1) * own * (vp + 2) * 4));
+    }
+    pdl_launch_dependents();
+    if (ns > 1) {
+        cluster_arrive_release();
+        cluster_wait_acquire();
+    }
+    if (!a.early) pdl_wait();
     const int row_hi = row0 + (pair0 + pairs - 1) / g;
     const int seq = a.row_seq[row0], len = a.row_pos[row_hi] + 1;
     const int npages = (len + GQA_PAGE - 1) / GQA_PAGE, pps = (npages + a.nsplit - 1) / a.nsplit;
@@ -442,9 +452,12 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
             const int tok = (p0 + i) * GQA_PAGE + u * 16;
             if (tok < len) {
                 const uint32_t kb = s32(ring + (size_t)s * stage) + k_lane, vb = s32(ring + (size_t)s * stage + k_bytes) + v_lane;
-                float sc[NT][4];
+                constexpr int CH = NT == 1 ? 3 : 1;  // a lone tile of pairs: one accumulator per term, or its MMAs would wait for one another
+                float sc[NT][CH][4];
 #pragma unroll
-                for (int nt = 0; nt < NT; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
+                for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+                    for (int c = 0; c < CH; ++c) sc[nt][c][0] = sc[nt][c][1] = sc[nt][c][2] = sc[nt][c][3] = 0.f;
 #pragma unroll 2
                 for (int kt = 0; kt < kt_n; ++kt) {
                     uint32_t ka[4];
@@ -454,7 +467,7 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
 #pragma unroll
                         for (int t3 = 0; t3 < 3; ++t3) {
                             const uint2 b = qf[((nt * kt_n + kt) * 3 + t3) * 32 + lane];
-                            mma16816(sc[nt], ka, b.x, b.y);
+                            mma16816(sc[nt][t3 % CH], ka, b.x, b.y);
                         }
                 }
                 uint32_t pb[NT][3][2];
@@ -463,9 +476,13 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
                 for (int nt = 0; nt < NT; ++nt) {
                     float pr[4], corr[2];
 #pragma unroll
+                    for (int c = CH - 1; c > 0; --c)  // small terms first
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) sc[nt][c - 1][e] += sc[nt][c][e];
+#pragma unroll
                     for (int hh = 0; hh < 2; ++hh) {
                         const int n0 = pos[nt][hh] - t0, n1 = pos[nt][hh] - t1;
-                        float s0 = sc[nt][hh], s1 = sc[nt][2 + hh];
+                        float s0 = sc[nt][0][hh], s1 = sc[nt][0][2 + hh];
                         if (a.bias) {
                             s0 += __ldg(a.bias + brow[nt][hh] + min(max(n0, 0), a.reach));
                             s1 += __ldg(a.bias + brow[nt][hh] + min(max(n1, 0), a.reach));
@@ -524,73 +541,80 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
     __syncthreads();  // every page consumed: the ring becomes scratch
     float* wm = reinterpret_cast<float*>(ring);  // [ATT_WARPS][P]
     float* wl = wm + ATT_WARPS * P;
-    float* buf = wl + ATT_WARPS * P;             // [4][P][ldo]
-    if (warp < ATT_WARPS && gid == 0) {
-#pragma unroll
-        for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-            for (int hh = 0; hh < 2; ++hh) {
-                wm[warp * P + nt * 8 + 2 * tig + hh] = tm[nt][hh];
-                wl[warp * P + nt * 8 + 2 * tig + hh] = tl[nt][hh];
-            }
-    }
-    __syncthreads();
-    if (tid < P) {
-        float mx = -INFINITY, l = 0.f;
-#pragma unroll
-        for (int w = 0; w < ATT_WARPS; ++w) mx = fmaxf(mx, wm[w * P + tid]);
-#pragma unroll
-        for (int w = 0; w < ATT_WARPS; ++w) l += wm[w * P + tid] == -INFINITY ? 0.f : exp2f(wm[w * P + tid] - mx) * wl[w * P + tid];
-        ml[2 * tid] = mx;
-        ml[2 * tid + 1] = l;
-    }
-    __syncthreads();
+    float* buf = wl + ATT_WARPS * P;             // [ATT_WARPS][P][ldo]
     if (warp < ATT_WARPS) {
+        float* b = buf + (size_t)warp * P * ldo;
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
-            float f[2];
+            if (gid == 0) {
 #pragma unroll
-            for (int hh = 0; hh < 2; ++hh) f[hh] = tm[nt][hh] == -INFINITY ? 0.f : exp2f(tm[nt][hh] - ml[2 * (nt * 8 + 2 * tig + hh)]);
-#pragma unroll
-            for (int mt = 0; mt < VT; ++mt) {
-                to[nt][mt][0] *= f[0];
-                to[nt][mt][1] *= f[1];
-                to[nt][mt][2] *= f[0];
-                to[nt][mt][3] *= f[1];
+                for (int hh = 0; hh < 2; ++hh) {
+                    wm[warp * P + nt * 8 + 2 * tig + hh] = tm[nt][hh];
+                    wl[warp * P + nt * 8 + 2 * tig + hh] = tl[nt][hh];
+                }
             }
+#pragma unroll
+            for (int mt = 0; mt < VT; ++mt)
+                if (mt < vt_n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) b[(nt * 8 + 2 * tig + (e & 1)) * ldo + mt * 16 + gid + (e >> 1) * 8] = to[nt][mt][e];
         }
     }
-    // halve the number of partial results until warp 0 holds the sum
-    for (int step = ATT_WARPS / 2; step >= 0; step >>= 1) {
-        const bool last = step == 0;
-        if (last ? warp == 0 : warp >= step && warp < 2 * step) {
-            float* b = buf + (size_t)(last ? 0 : warp - step) * P * ldo;
+    __syncthreads();
+    // the warps' results added up, four values a thread, and sent to the split that owns the pair
+    for (int i = tid; i < pairs * (vp / 4); i += B_THREADS) {
+        const int p = i / (vp / 4), d = (i - p * (vp / 4)) * 4;
+        float f[ATT_WARPS], mx = -INFINITY, l = 0.f;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-            for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-                for (int mt = 0; mt < VT; ++mt)
-                    if (mt < vt_n)
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) b[(nt * 8 + 2 * tig + (e & 1)) * ldo + mt * 16 + gid + (e >> 1) * 8] = to[nt][mt][e];
+        for (int w = 0; w < ATT_WARPS; ++w) {
+            f[w] = wm[w * P + p];
+            mx = fmaxf(mx, f[w]);
         }
-        if (last) break;
-        __syncthreads();
-        if (warp < step) {
-            const float* b = buf + (size_t)warp * P * ldo;
 #pragma unroll
-            for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-                for (int mt = 0; mt < VT; ++mt)
-                    if (mt < vt_n)
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) to[nt][mt][e] += b[(nt * 8 + 2 * tig + (e & 1)) * ldo + mt * 16 + gid + (e >> 1) * 8];
+        for (int w = 0; w < ATT_WARPS; ++w) {
+            f[w] = f[w] == -INFINITY ? 0.f : exp2f(f[w] - mx);
+            const float4 x = *reinterpret_cast<const float4*>(buf + (size_t)(w * P + p) * ldo + d);
+            v.x = fmaf(f[w], x.x, v.x); v.y = fmaf(f[w], x.y, v.y); v.z = fmaf(f[w], x.z, v.z); v.w = fmaf(f[w], x.w, v.w);
+            l = fmaf(f[w], wl[w * P + p], l);
         }
-        __syncthreads();
+        const uint32_t owner = (uint32_t)(p % ns);
+        float* slot = recv + (size_t)(rank * own_most + p / ns) * (vp + 4);
+        if ((int)owner == rank) {
+            *reinterpret_cast<float4*>(slot + d) = v;
+            if (d == 0) {
+                slot[vp] = mx;
+                slot[vp + 1] = l;
+            }
+        } else {
+            const uint32_t bar = dsmem_addr(&s_rbar, owner);
+            st_async_f32x4(dsmem_addr(slot + d, owner), v, bar);
+            if (d == 0) st_async_f32x2(dsmem_addr(slot + vp, owner), mx, l, bar);
+        }
     }
-    combine_and_store(a, buf, ldo, ml, wts, pairs, [&](int p, int& row, int& head) {
-        row = row0 + (pair0 + p) / g;
-        head = kvh * g + (pair0 + p) % g;
-    });
+    if (own == 0) return;
+    __syncthreads();
+    if (ns > 1 && !mb_wait_cluster(&s_rbar, 0, a.err_flag, &s_abort)) return;  // bounded
+    for (int i = tid; i < own * (vp / 8); i += B_THREADS) {
+        const int k = i / (vp / 8), d0 = (i - k * (vp / 8)) * 8, p = k * ns + rank;
+        float v[8], mx = -INFINITY, l = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = 0.f;
+        for (int r = 0; r < ns; ++r) mx = fmaxf(mx, recv[(size_t)(r * own_most + k) * (vp + 4) + vp]);
+#pragma unroll 4
+        for (int r = 0; r < ns; ++r) {
+            const float* slot = recv + (size_t)(r * own_most + k) * (vp + 4);
+            const float f = slot[vp] == -INFINITY ? 0.f : exp2f(slot[vp] - mx);
+            const float4 x = *reinterpret_cast<const float4*>(slot + d0), y = *reinterpret_cast<const float4*>(slot + d0 + 4);
+            l = fmaf(f, slot[vp + 1], l);
+            v[0] = fmaf(f, x.x, v[0]); v[1] = fmaf(f, x.y, v[1]); v[2] = fmaf(f, x.z, v[2]); v[3] = fmaf(f, x.w, v[3]);
+            v[4] = fmaf(f, y.x, v[4]); v[5] = fmaf(f, y.y, v[5]); v[6] = fmaf(f, y.z, v[6]); v[7] = fmaf(f, y.w, v[7]);
+        }
+        const float inv = 1.0f / l;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= inv;
+        if (d0 < vdim) store_piece(a, row0 + (pair0 + p) / g, kvh * g + (pair0 + p) % g, d0, v);
+    }
 }
 
 template <typename... KArgs, typename... Args>
@@ -639,10 +663,11 @@ cudaError_t launch_mma(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
     }
     const int pages = (a.longest + GQA_PAGE - 1) / GQA_PAGE, pairs = a.tiles * a.pool.kv_heads;
     constexpr int PER_SM = NT == 1 && VT <= 8 ? 2 : 1;
-    if (a.nsplit < 1) a.nsplit = std::max(1, std::min({PER_SM * sm_count / pairs, a.max_cluster, MAX_CLUSTER, pages}));
+    // clusters of more than eight CTAs are hard to place: only for long contexts
+    if (a.nsplit < 1) a.nsplit = std::max(1, std::min({PER_SM * sm_count / pairs, a.max_cluster, pages > 128 ? MAX_CLUSTER : 8, pages}));
     const size_t stage = b_stage_bytes(dp, vp);
     const int ppc = (pages + a.nsplit - 1) / a.nsplit;
-    const size_t fixed = b_query_bytes(NT, dp) + sizeof(float) * ((size_t)a.nsplit * P + 2 * P) + 4 * (size_t)ppc + 128;
+    const size_t fixed = b_query_bytes(NT, dp) + b_recv_bytes(NT, vp, a.nsplit) + 4 * (size_t)ppc + 128;
     // CTAs that have an SM to themselves take a deep ring
     const size_t budget = (PER_SM == 2 && (long)pairs * a.nsplit > sm_count ? 110 : 220) * 1024;
     int stages = MAX_STAGES;
