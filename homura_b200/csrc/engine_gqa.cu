@@ -203,7 +203,7 @@ double Engine::experts_used(const LayerSpec& s, int rows) const { return s.exper
 
 ExpertWeights Engine::expert_weights(int layer) const {
     const LayerSpec& s = spec_.layers[layer];
-    return ExpertWeights{layers_[layer].exp_gu, layers_[layer].exp_down, H_, s.ff, s.top, s.limit};
+    return ExpertWeights{layers_[layer].exp_gu, layers_[layer].exp_down, s.experts, H_, s.ff, s.top, s.limit};
 }
 
 // Bytes of expert weights that the last profiled step read.

@@ -586,7 +586,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) 
             if (warp == 0) {
                 int n = 0;
                 for (int w = 0; w < words; ++w) {
-                    const uint32_t v = xl.mask[w];
+                    const uint32_t v = xl.mask[w] & (a.ex.n - w * 32 < 32 ? (1u << (a.ex.n - w * 32)) - 1u : ~0u);
                     if (v >> lane & 1u) xl.id[n + __popc(v & ((1u << lane) - 1u))] = (uint16_t)(w * 32 + lane);
                     n += __popc(v);
                 }

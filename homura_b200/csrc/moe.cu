@@ -19,6 +19,7 @@ namespace {
 constexpr int THREADS = 256, WARPS = THREADS / 32;
 constexpr int TILE = 128 * 64;  // elements of a tile image: 128 rows of 64 k, 16-byte pieces XOR-ed by row & 7
 constexpr int GU_ROWS = 16, DOWN_ROWS = 8;
+constexpr int REG4 = 2;         // 16-byte pieces of a residual row that a thread of the post-norm keeps in registers
 
 __device__ __forceinline__ float block_sum(float v, float* part) {
     v = warp_sum(v);
@@ -52,33 +53,27 @@ __device__ __forceinline__ void choose(const PostNormArgs& a, int m, float* z, f
         l += e;
     }
     l = warp_sum(l);
+    uint32_t* key = reinterpret_cast<uint32_t*>(choice);  // unsigned integers in the order of the floats; 0: chosen already
     for (int r = lane; r < a.n_out; r += 32) {
         const float s = z[r] / l;
         z[r] = s;
-        choice[r] = s + __ldg(a.correction + r);
+        const uint32_t u = __float_as_uint(s + __ldg(a.correction + r));
+        key[r] = u >> 31 ? ~u : u | 0x80000000u;
     }
     __syncwarp();
     float ident = 0.f;
     for (int k = 0; k < a.top; ++k) {
-        float bv = -INFINITY;
-        int bi = a.n_out;
+        uint32_t best = 0u, at = lane < a.n_out ? lane : 0xffffffffu;
         for (int r = lane; r < a.n_out; r += 32)
-            if (choice[r] > bv || bi == a.n_out) {
-                bv = choice[r];
-                bi = r;
+            if (key[r] > best) {
+                best = key[r];
+                at = r;
             }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (oi < a.n_out && (bi == a.n_out || ov > bv || (ov == bv && oi < bi))) {
-                bv = ov;
-                bi = oi;
-            }
-        }
+        const uint32_t most = __reduce_max_sync(0xffffffffu, best);
+        const int bi = (int)__reduce_min_sync(0xffffffffu, best == most ? at : 0xffffffffu);
         const float s = z[bi];
         if (lane == 0) {
-            choice[bi] = -INFINITY;
+            key[bi] = 0u;
             const bool id = bi >= a.experts;
             a.out.ids[(size_t)m * a.top + k] = id ? -1 : bi;
             a.out.weights[(size_t)m * a.top + k] = s;
@@ -100,6 +95,21 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PostNormArgs a
     __shared__ float part[WARPS];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, m = blockIdx.x / cluster, rank = blockIdx.x - m * cluster;
     pdl_launch_dependents();
+    // weights do not depend on the launch in front: norm weights, and the first router row of the warp
+    const bool regs = (a.W & 7) == 0 && a.W <= 4 * REG4 * THREADS;
+    float4 w4[REG4];
+    uint4 r4[REG4 * 4];
+    const int first = rank * WARPS + warp;
+    if (regs) {
+#pragma unroll
+        for (int k = 0; k < REG4; ++k)
+            if (tid + k * THREADS < a.W / 4) w4[k] = __ldg(reinterpret_cast<const float4*>(a.w) + tid + k * THREADS);
+        if (a.router && first < a.n_out) {
+            const uint4* wr = reinterpret_cast<const uint4*>(a.router + (size_t)first * a.W);
+#pragma unroll
+            for (int k = 0; k < REG4 * 4; ++k) r4[k] = lane + k * 32 < a.W / 8 ? __ldg(wr + lane + k * 32) : make_uint4(0, 0, 0, 0);
+        }
+    }
     if (cluster > 1) {  // every CTA of the cluster has started before the first one stores into rank 0
         cluster_arrive_release();
         cluster_wait_acquire();
@@ -108,20 +118,35 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PostNormArgs a
     const float idw = a.identity ? ld_cg_f32(a.identity + m) : 0.f;
     const float *x = a.x + (size_t)m * a.W, *y = a.y + (size_t)m * a.W;
     float ss = 0.f;
-    if ((a.W & 3) == 0) {
-#pragma unroll 2
-        for (int i = tid; i < a.W / 4; i += THREADS) {
-            const float4 xv = ld_cg_f32x4(x + 4 * (size_t)i);
-            float4 yv = ld_cg_f32x4(y + 4 * (size_t)i);
-            for (int p = 1; p < a.parts; ++p) {
-                const float4 t = ld_cg_f32x4(y + p * a.part_stride + 4 * (size_t)i);
-                yv = make_float4(yv.x + t.x, yv.y + t.y, yv.z + t.z, yv.w + t.w);
+    if (regs) {
+        float4 x4[REG4], y4[REG4];
+#pragma unroll
+        for (int k = 0; k < REG4; ++k) {
+            const int i = tid + k * THREADS;
+            x4[k] = y4[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < a.W / 4) {
+                x4[k] = ld_cg_f32x4(x + 4 * (size_t)i);
+                y4[k] = ld_cg_f32x4(y + 4 * (size_t)i);
             }
-            yv = make_float4(fmaf(idw, xv.x, yv.x), fmaf(idw, xv.y, yv.y), fmaf(idw, xv.z, yv.z), fmaf(idw, xv.w, yv.w));
-            reinterpret_cast<float4*>(xs)[i] = xv;
-            reinterpret_cast<float4*>(ys)[i] = yv;
-            ss = fmaf(yv.x, yv.x, fmaf(yv.y, yv.y, fmaf(yv.z, yv.z, fmaf(yv.w, yv.w, ss))));
         }
+        for (int p = 1; p < a.parts; ++p)
+#pragma unroll
+            for (int k = 0; k < REG4; ++k)
+                if (tid + k * THREADS < a.W / 4) {
+                    const float4 t = ld_cg_f32x4(y + p * a.part_stride + 4 * (size_t)(tid + k * THREADS));
+                    y4[k] = make_float4(y4[k].x + t.x, y4[k].y + t.y, y4[k].z + t.z, y4[k].w + t.w);
+                }
+#pragma unroll
+        for (int k = 0; k < REG4; ++k) {
+            y4[k] = make_float4(fmaf(idw, x4[k].x, y4[k].x), fmaf(idw, x4[k].y, y4[k].y), fmaf(idw, x4[k].z, y4[k].z), fmaf(idw, x4[k].w, y4[k].w));
+            ss = fmaf(y4[k].x, y4[k].x, fmaf(y4[k].y, y4[k].y, fmaf(y4[k].z, y4[k].z, fmaf(y4[k].w, y4[k].w, ss))));
+        }
+        const float inv = 1.0f / sqrtf(block_sum(ss, part) / (float)a.W + a.eps);
+#pragma unroll
+        for (int k = 0; k < REG4; ++k)
+            if (tid + k * THREADS < a.W / 4)
+                reinterpret_cast<float4*>(xs)[tid + k * THREADS] = make_float4(fmaf(a.mult, (y4[k].x * inv) * w4[k].x, x4[k].x), fmaf(a.mult, (y4[k].y * inv) * w4[k].y, x4[k].y),
+                                                                              fmaf(a.mult, (y4[k].z * inv) * w4[k].z, x4[k].z), fmaf(a.mult, (y4[k].w * inv) * w4[k].w, x4[k].w));
     } else {
         for (int i = tid; i < a.W; i += THREADS) {
             const float xv = ld_cg_f32(x + i);
@@ -132,15 +157,19 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PostNormArgs a
             ys[i] = yv;
             ss = fmaf(yv, yv, ss);
         }
+        const float inv = 1.0f / sqrtf(block_sum(ss, part) / (float)a.W + a.eps);
+        for (int i = tid; i < Wp; i += THREADS) xs[i] = i < a.W ? fmaf(a.mult, (ys[i] * inv) * __ldg(a.w + i), xs[i]) : 0.f;
     }
-    const float inv = 1.0f / sqrtf(block_sum(ss, part) / (float)a.W + a.eps);
-    for (int i = tid; i < Wp; i += THREADS) xs[i] = i < a.W ? fmaf(a.mult, (ys[i] * inv) * __ldg(a.w + i), xs[i]) : 0.f;
     __syncthreads();
     if (a.router) {
-        for (int r = rank * WARPS + warp; r < a.n_out; r += cluster * WARPS) {
+        for (int r = first; r < a.n_out; r += cluster * WARPS) {
             const uint16_t* wr = a.router + (size_t)r * a.W;
             float s = 0.f;
-            if ((a.W & 7) == 0) {
+            if (regs && r == first) {
+#pragma unroll
+                for (int k = 0; k < REG4 * 4; ++k)
+                    if (lane + k * 32 < a.W / 8) s = dot8(r4[k], reinterpret_cast<const float4*>(xs)[2 * (lane + k * 32)], reinterpret_cast<const float4*>(xs)[2 * (lane + k * 32) + 1], s);
+            } else if ((a.W & 7) == 0) {
 #pragma unroll 4
                 for (int c = lane; c < a.W / 8; c += 32)
                     s = dot8(__ldg(reinterpret_cast<const uint4*>(wr) + c), reinterpret_cast<const float4*>(xs)[2 * c], reinterpret_cast<const float4*>(xs)[2 * c + 1], s);
@@ -190,14 +219,11 @@ __global__ void __launch_bounds__(THREADS) expert_gate_up_kernel(const ExpertWei
     __shared__ float red[WARPS][2 * GU_ROWS];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, pair = blockIdx.y, m = pair / w.top;
     const int blocks = expert_blocks(w.ff), blk = blockIdx.x / (64 / GU_ROWS), sub = blockIdx.x % (64 / GU_ROWS), kbs = (w.W + 63) / 64;
-    pdl_launch_dependents();
     pdl_wait();
+    pdl_launch_dependents();  // not earlier: the launch behind relies on the router's choice from its start
     const int e = __ldcg(ids + pair);
-    if (e < 0) return;
-    stage_row<THREADS, false>(x + (size_t)m * w.W, xs, w.W, tid);
-    for (int i = w.W + tid; i < kbs * 64; i += THREADS) xs[i] = 0.f;
+    if (e < 0 || e >= w.n) return;
     const float rw = ld_cg_f32(weights + pair);
-    __syncthreads();
     const uint16_t* base = w.gu + ((size_t)e * blocks + blk) * kbs * TILE;
     const int r8 = lane >> 3, p = lane & 7;
     float acc[8];
@@ -205,11 +231,19 @@ __global__ void __launch_bounds__(THREADS) expert_gate_up_kernel(const ExpertWei
     for (int j = 0; j < 8; ++j) acc[j] = 0.f;
     // loads j = 0..3: gate rows sub * 16 + 4 j + r8; j = 4..7: up rows
     const uint16_t* src[2] = {base + (size_t)(sub * GU_ROWS + r8) * 64 + p * 8, base + (size_t)(64 + sub * GU_ROWS + r8) * 64 + p * 8};
-#pragma unroll 2
-    for (int kb = warp; kb < kbs; kb += WARPS) {
-        uint4 v[8];
+    uint4 v[8], next[8];
+    auto fetch = [&](int kb, uint4 (&t)[8]) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) v[j] = ld_stream_u4(src[j >> 2] + (size_t)kb * TILE + (size_t)(j & 3) * 4 * 64);
+        for (int j = 0; j < 8; ++j) t[j] = ld_stream_u4(src[j >> 2] + (size_t)kb * TILE + (size_t)(j & 3) * 4 * 64);
+    };
+    if (warp < kbs) fetch(warp, next);
+    stage_row<THREADS, false>(x + (size_t)m * w.W, xs, w.W, tid);
+    for (int i = w.W + tid; i < kbs * 64; i += THREADS) xs[i] = 0.f;
+    __syncthreads();
+    for (int kb = warp; kb < kbs; kb += WARPS) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = next[j];
+        if (kb + WARPS < kbs) fetch(kb + WARPS, next);
         float4 xa[2], xb[2];
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
@@ -248,28 +282,46 @@ __global__ void __launch_bounds__(THREADS) expert_down_kernel(const ExpertWeight
     const float* row = act + (size_t)m * units * 64;
     int* s_id = reinterpret_cast<int*>(as + (staged ? units * 64 : 0));
     pdl_launch_dependents();
-    pdl_wait();
+    // the router's choice was complete before the gate / up projection let this launch start: weights are requested ahead of the wait,
+    // the first ones into registers, the others into the L2
     for (int i = tid; i < w.top; i += THREADS) s_id[i] = __ldcg(ids + m * w.top + i);
-    if (staged) stage_row<THREADS, false>(row, as, units * 64, tid);
     __syncthreads();
     const int r8 = lane >> 3, p = lane & 7;
     float acc[2] = {0.f, 0.f};
-    const size_t row_off = (size_t)(sub * DOWN_ROWS + r8) * 64 + p * 8;
-    for (int u0 = warp; u0 < units; u0 += 4 * WARPS) {
-        uint4 v[4][2];
-        bool on[4];
+    const size_t sub_off = (size_t)sub * DOWN_ROWS * 64, row_off = (size_t)r8 * 64 + p * 8;
+    auto tile = [&](int u) -> const uint16_t* {  // this CTA's rows of the u-th block of the chosen experts
+        const int slot = u / blocks, e = u < units ? s_id[slot] : -1;
+        return e < 0 || e >= w.n ? nullptr : w.down + (((size_t)e * nbs + nb) * blocks + (u - slot * blocks)) * TILE + sub_off;
+    };
+    constexpr int B = 4;  // blocks of a warp at a time
+    uint4 v[B][2], next[B][2];
+    const uint16_t *on[B], *next_on[B];
+    auto fetch = [&](int u0, uint4 (&t)[B][2], const uint16_t* (&o)[B]) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int u = u0 + i * WARPS, slot = u / blocks, e = u < units ? s_id[slot] : -1;
-            on[i] = e >= 0;
-            if (on[i]) {
-                const uint16_t* t = w.down + (((size_t)e * nbs + nb) * blocks + (u - slot * blocks)) * TILE + row_off;
-                v[i][0] = ld_stream_u4(t);
-                v[i][1] = ld_stream_u4(t + 4 * 64);
+        for (int i = 0; i < B; ++i) {
+            o[i] = tile(u0 + i * WARPS);
+            if (o[i]) {
+                t[i][0] = ld_stream_u4(o[i] + row_off);
+                t[i][1] = ld_stream_u4(o[i] + row_off + 4 * 64);
             }
         }
+    };
+    fetch(warp, next, next_on);
+    for (int u = B * WARPS + tid; u < units; u += THREADS)
+        if (const uint16_t* t = tile(u)) asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(t), "r"(DOWN_ROWS * 128) : "memory");
+    pdl_wait();
+    if (staged) stage_row<THREADS, false>(row, as, units * 64, tid);
+    __syncthreads();
+    for (int u0 = warp; u0 < units; u0 += B * WARPS) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
+        for (int i = 0; i < B; ++i) {
+            v[i][0] = next[i][0];
+            v[i][1] = next[i][1];
+            on[i] = next_on[i];
+        }
+        fetch(u0 + B * WARPS, next, next_on);
+#pragma unroll
+        for (int i = 0; i < B; ++i)
             if (on[i]) {
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {

@@ -40,7 +40,7 @@ cudaError_t launch_post_norm(const PostNormArgs& a, int sm_count, cudaStream_t s
 // rows over W, down [W] over ff; ff padded to 64.
 struct ExpertWeights {
     const uint16_t *gu, *down;
-    int W, ff, top;
+    int n, W, ff, top;       // n experts
     float limit;
 };
 __host__ __device__ __forceinline__ int expert_blocks(int ff) { return (ff + 63) / 64; }
