@@ -15,6 +15,9 @@
 #include "gqa_attn.h"
 
 #include <algorithm>
+#include <map>
+#include <mutex>
+#include <tuple>
 
 #include "launch_attrs.h"
 #include "mbarrier.cuh"
@@ -409,16 +412,23 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
             }
     } else {
         // B fragments of the queries: lane (pair = lane / 4, i = lane % 4) holds elements 2i, 2i + 1 and 2i + 8, 2i + 9 of every 16
+        const bool even = (dim & 1) == 0;  // rows of queries are then 8-byte aligned
+#pragma unroll 4
         for (int i = tid; i < NT * kt_n * 32; i += ATT_WARPS * 32) {
             const int ln = i & 31, kt = (i >> 5) % kt_n, nt = (i >> 5) / kt_n, p = nt * 8 + (ln >> 2), d0 = kt * 16 + (ln & 3) * 2;
-            uint32_t lo[3] = {0u, 0u, 0u}, hi[3] = {0u, 0u, 0u};
+            float2 x = make_float2(0.f, 0.f), y = x;
             if (p < pairs) {
-                const int pr = pair0 + p;
-                const float* q = a.q + (size_t)(row0 + pr / g) * a.heads * dim + (size_t)(kvh * g + pr % g) * dim;
-                auto at = [&](int d) { return d < dim ? ld_cg_f32(q + d) : 0.f; };
-                bf16x2_split3(at(d0), at(d0 + 1), lo[0], lo[1], lo[2]);
-                bf16x2_split3(at(d0 + 8), at(d0 + 9), hi[0], hi[1], hi[2]);
+                const float* q = a.q + (size_t)(s_pos[p] - s_pos[0] + row0 + pair0 / g) * a.heads * dim + (size_t)(kvh * g + (pair0 + p) % g) * dim;
+                auto at = [&](int d) {
+                    if (even) return d < dim ? __ldcg(reinterpret_cast<const float2*>(q + d)) : make_float2(0.f, 0.f);
+                    return make_float2(d < dim ? __ldcg(q + d) : 0.f, d + 1 < dim ? __ldcg(q + d + 1) : 0.f);
+                };
+                x = at(d0);
+                y = at(d0 + 8);
             }
+            uint32_t lo[3], hi[3];
+            bf16x2_split3(x.x, x.y, lo[0], lo[1], lo[2]);
+            bf16x2_split3(y.x, y.y, hi[0], hi[1], hi[2]);
 #pragma unroll
             for (int t3 = 0; t3 < 3; ++t3) qf[((nt * kt_n + kt) * 3 + t3) * 32 + ln] = make_uint2(lo[t3], hi[t3]);
         }
@@ -495,11 +505,8 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
                         mx = fmaxf(tm[nt][hh], mx);
                         const float ref = mx == -INFINITY ? 0.f : mx;  // no token of this pair yet
                         const float e0 = exp2f(s0 - ref), e1 = exp2f(s1 - ref);
-                        float ps = e0 + e1;
-#pragma unroll
-                        for (int o = 4; o < 32; o <<= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
                         corr[hh] = exp2f(tm[nt][hh] - ref);
-                        tl[nt][hh] = fmaf(tl[nt][hh], corr[hh], ps);
+                        tl[nt][hh] = fmaf(tl[nt][hh], corr[hh], e0 + e1);  // this lane's tokens
                         tm[nt][hh] = mx;
                         pr[hh] = e0;
                         pr[2 + hh] = e1;
@@ -546,6 +553,10 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
         float* b = buf + (size_t)warp * P * ldo;
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
+#pragma unroll
+            for (int hh = 0; hh < 2; ++hh)
+#pragma unroll
+                for (int o = 4; o < 32; o <<= 1) tl[nt][hh] += __shfl_xor_sync(0xffffffffu, tl[nt][hh], o);
             if (gid == 0) {
 #pragma unroll
                 for (int hh = 0; hh < 2; ++hh) {
@@ -646,6 +657,35 @@ cudaError_t launch_clustered(void (*kern)(KArgs...), dim3 grid, dim3 block, size
     return cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
 }
 
+// Clusters of a kernel that the current device holds at the same time (asked once per shape).
+template <typename... KArgs>
+int clusters_at_once(void (*kern)(KArgs...), int cluster, int threads, size_t smem) {
+    static std::mutex mu;
+    static std::map<std::tuple<const void*, int, int, size_t>, int> known;
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess) return 0;
+    const auto key = std::make_tuple(reinterpret_cast<const void*>(kern), dev, cluster, smem);
+    std::lock_guard<std::mutex> lk(mu);
+    const auto it = known.find(key);
+    if (it != known.end()) return it->second;
+    int n = 0;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3((unsigned)cluster);
+    cfg.blockDim = dim3((unsigned)threads);
+    cfg.dynamicSmemBytes = smem;
+    cudaLaunchAttribute at[1];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = (unsigned)cluster;
+    at[0].val.clusterDim.y = at[0].val.clusterDim.z = 1;
+    cfg.attrs = at;
+    cfg.numAttrs = 1;
+    if (ensure_dyn_smem(kern, smem) != cudaSuccess || (cluster > 8 && ensure_nonportable_clusters(kern) != cudaSuccess) || cudaOccupancyMaxActiveClusters(&n, kern, &cfg) != cudaSuccess) {
+        cudaGetLastError();
+        n = 0;
+    }
+    return known[key] = n;
+}
+
 template <int VT, int NT>
 cudaError_t launch_mma(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
     constexpr int P = NT * 8;
@@ -663,17 +703,27 @@ cudaError_t launch_mma(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
     }
     const int pages = (a.longest + GQA_PAGE - 1) / GQA_PAGE, pairs = a.tiles * a.pool.kv_heads;
     constexpr int PER_SM = NT == 1 && VT <= 8 ? 2 : 1;
-    // clusters of more than eight CTAs are hard to place: only for long contexts
-    if (a.nsplit < 1) a.nsplit = std::max(1, std::min({PER_SM * sm_count / pairs, a.max_cluster, pages > 128 ? MAX_CLUSTER : 8, pages}));
     const size_t stage = b_stage_bytes(dp, vp);
-    const int ppc = (pages + a.nsplit - 1) / a.nsplit;
-    const size_t fixed = b_query_bytes(NT, dp) + b_recv_bytes(NT, vp, a.nsplit) + 4 * (size_t)ppc + 128;
-    // CTAs that have an SM to themselves take a deep ring
-    const size_t budget = (PER_SM == 2 && (long)pairs * a.nsplit > sm_count ? 110 : 220) * 1024;
-    int stages = MAX_STAGES;
-    while (stages > 2 && (stages * stage + fixed > budget || stages - 2 >= ppc)) stages -= 2;
-    a.stages = stages;
-    const size_t ring = (std::max(stages * stage, b_merge_bytes(NT, vp)) + 127) / 128 * 128;
+    size_t ring = 0, fixed = 0;
+    auto shape = [&](int nsplit) {  // ring and shared memory of a launch with so many splits
+        const int ppc = (pages + nsplit - 1) / nsplit;
+        fixed = b_query_bytes(NT, dp) + b_recv_bytes(NT, vp, nsplit) + 4 * (size_t)ppc + 128;
+        // CTAs that have an SM to themselves take a deep ring
+        const size_t budget = (PER_SM == 2 && (long)pairs * nsplit > sm_count ? 110 : 220) * 1024;
+        int stages = MAX_STAGES;
+        while (stages > 2 && (stages * stage + fixed > budget || stages - 2 >= ppc)) stages -= 2;
+        a.stages = stages;
+        ring = (std::max(stages * stage, b_merge_bytes(NT, vp)) + 127) / 128 * 128;
+    };
+    if (a.nsplit < 1) {
+        // as many splits as run at once; clusters of more than eight CTAs are hard to place: only for long contexts
+        a.nsplit = std::max(1, std::min({PER_SM * sm_count / pairs, a.max_cluster, pages > 128 ? MAX_CLUSTER : 8, pages}));
+        for (; a.nsplit > 1; --a.nsplit) {
+            shape(a.nsplit);
+            if (ring + fixed <= 226 * 1024 && clusters_at_once(gqa_attn_mma_kernel<VT, NT>, a.nsplit, B_THREADS, ring + fixed) >= pairs) break;
+        }
+    }
+    shape(a.nsplit);
     if (ring + fixed > 226 * 1024) return cudaErrorInvalidValue;
     return launch_clustered(gqa_attn_mma_kernel<VT, NT>, dim3((unsigned)a.nsplit, (unsigned)a.pool.kv_heads, (unsigned)a.tiles), dim3(B_THREADS), ring + fixed, a.nsplit, st, pdl, a, ring);
 }
@@ -682,8 +732,8 @@ template <int VT>
 cudaError_t launch_mma_n(const GqaAttnArgs& a, int sm_count, cudaStream_t st, bool pdl) {
     const int pairs = a.longest_run * (a.heads / a.pool.kv_heads);
     if (pairs <= 8) return launch_mma<VT, 1>(a, sm_count, st, pdl);
-    if (pairs <= 16 || VT > 8) return launch_mma<VT, 2>(a, sm_count, st, pdl);
-    return launch_mma<VT, VT <= 8 ? 4 : 2>(a, sm_count, st, pdl);
+    if (pairs <= 16 || VT > 4) return launch_mma<VT, 2>(a, sm_count, st, pdl);  // four tiles of wide values do not fit the registers
+    return launch_mma<VT, VT <= 4 ? 4 : 2>(a, sm_count, st, pdl);
 }
 
 }  // namespace

@@ -72,18 +72,24 @@ __device__ __forceinline__ void choose(const PostNormArgs& a, int m, float* z, f
         const uint32_t most = __reduce_max_sync(0xffffffffu, best);
         const int bi = (int)__reduce_min_sync(0xffffffffu, best == most ? at : 0xffffffffu);
         const float s = z[bi];
+        __syncwarp();
         if (lane == 0) {
             key[bi] = 0u;
             const bool id = bi >= a.experts;
             a.out.ids[(size_t)m * a.top + k] = id ? -1 : bi;
             a.out.weights[(size_t)m * a.top + k] = s;
             if (id) ident += s;
-            else if (a.out.dense) {
-                a.out.dense[(size_t)m * a.experts + bi] = s;
-                a.out.mask[(size_t)m * ((a.experts + 31) / 32) + bi / 32] |= 1u << (bi & 31);
-            }
+            else if (a.out.dense) a.out.dense[(size_t)m * a.experts + bi] = s;
         }
         __syncwarp();
+    }
+    if (a.out.dense) {  // the chosen ones are those whose key is gone
+        const int words = (a.experts + 31) / 32;
+        for (int w = 0; w < words; ++w) {
+            const int r = w * 32 + lane;
+            const uint32_t bits = __ballot_sync(0xffffffffu, r < a.experts && key[r] == 0u);
+            if (lane == 0) a.out.mask[(size_t)m * words + w] = bits;
+        }
     }
     if (lane == 0) a.out.identity[m] = ident;
 }
@@ -182,11 +188,8 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PostNormArgs a
                 else st_dsmem_f32(dsmem_addr(z + r, 0u), s);
             }
         }
-        if (rank == 0 && a.out.dense) {
+        if (rank == 0 && a.out.dense)
             for (int i = tid; i < a.experts; i += THREADS) a.out.dense[(size_t)m * a.experts + i] = 0.f;
-            const int words = (a.experts + 31) / 32;
-            for (int i = tid; i < words; i += THREADS) a.out.mask[(size_t)m * words + i] = 0u;
-        }
     }
     // the residual is stored when every CTA of the row has read it
     if (cluster > 1) cluster_sync_all();
