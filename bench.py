@@ -291,14 +291,18 @@ POINTS = {"0.5B": [(1, 128), (8, 1920)], "1.5B": [(1, 128), (64, 512), (8, 1920)
 DESIGNS = {
     "tunitar": {"0.5B": ("TUNITAR_05B", "QWEN25_05B"), "1.5B": ("TUNITAR_15B", "QWEN25_15B")},
     "dipisun": {"0.5B": ("DIPISUN_05B", "QWEN25_05B"), "1.5B": ("DIPISUN_15B", "QWEN25_15B")},
+    "gebilorn": {"0.5B": ("GEBILORN_05B", "QWEN25_05B"), "1.5B": ("GEBILORN_15B", "QWEN25_15B")},
 }
 # kernel classes that do the same work in both designs
 LIKE = {
     "tunitar": {"in_proj": "qkv_rope_kvwrite", "key_up": "qkv_rope_kvwrite", "value_up_gate": "o_proj_residual", "attention": "attention", "o_proj_residual": "o_proj_residual", "up_sqrelu": "gate_up_swiglu",
                 "down_residual": "down_residual", "lm_head": "lm_head"},
     "dipisun": {"qkv_proj": "qkv_rope_kvwrite", "attention": "attention", "o_proj": "o_proj_residual", "experts_gate_up": "gate_up_swiglu", "experts_down": "down_residual", "lm_head": "lm_head"},
+    "gebilorn": {"in_proj": "qkv_rope_kvwrite", "attention": "attention", "query_up": "qkv_rope_kvwrite", "key_up": "qkv_rope_kvwrite", "value_up": "o_proj_residual", "out_proj": "o_proj_residual", "experts_gate_up": "gate_up_swiglu",
+                 "experts_down": "down_residual", "lm_head": "lm_head"},
 }
-WHAT = {"tunitar": "Tunitar stacks beside uniform GQA stacks of equal size", "dipisun": "Dipisun stacks beside uniform GQA stacks of equal width, depth, heads and MLP parameters per token"}
+WHAT = {"tunitar": "Tunitar stacks beside uniform GQA stacks of equal size", "dipisun": "Dipisun stacks beside uniform GQA stacks of equal width, depth, heads and MLP parameters per token",
+        "gebilorn": "Gebilorn stacks beside uniform GQA stacks of equal width, depth, heads and MLP parameters per token"}
 
 
 def design_model(design, name, cfg, synth):
@@ -308,9 +312,10 @@ def design_model(design, name, cfg, synth):
         return d
     if design == "tunitar":
         synth.write_tunitar_model(d, cfg, SEED)
-    elif design == "dipisun":
+    elif design in ("dipisun", "gebilorn"):
         # every layer's experts are drawn from one set; corrections of zero leave the choice to the router
-        specs = {s[0]: s for s in synth.dipisun_tensor_specs(cfg)}
+        all_specs, tensor, write = (synth.dipisun_tensor_specs, synth.dipisun_tensor, synth.write_dipisun_model) if design == "dipisun" else (synth.gebilorn_tensor_specs, synth.gebilorn_tensor, synth.write_gebilorn_model)
+        specs = {s[0]: s for s in all_specs(cfg)}
         experts = {}
 
         class Weights:
@@ -319,12 +324,12 @@ def design_model(design, name, cfg, synth):
                 if ".mlp.e" in name:
                     name = "l0." + name.split(".", 1)[1]
                     if name not in experts:
-                        experts[name] = synth.dipisun_tensor(SEED, (name, shape, kind))
+                        experts[name] = tensor(SEED, (name, shape, kind))
                     return experts[name]
-                w = synth.dipisun_tensor(SEED, (name, shape, kind))
+                w = tensor(SEED, (name, shape, kind))
                 return w * 0 if kind == "small" else w
 
-        synth.write_dipisun_model(d, cfg, SEED, Weights())
+        write(d, cfg, SEED, Weights())
     else:
         synth.write_hf_model(d, cfg, SEED)
     open(os.path.join(d, ".complete"), "w").write("ok")

@@ -354,6 +354,7 @@ int hm_weight_bytes(hm_engine* e, uint64_t* out) {
 // Vectors (norm weights, biases) first: whether a model has QK-norm is inferred from its tensors, and the layout of
 // a quantised QKV projection (rotation in its epilogue or not) is fixed when its first part is loaded.
 static int load_views(Engine* eng, const std::vector<TensorView>& views, std::string* err) {
+    for (const TensorView& t : views) eng->note_shape(t.name, t.shape);
     for (int pass = 0; pass < 2; ++pass) {
         for (const TensorView& t : views) {
             if (t.dtype < 0) {
@@ -425,6 +426,12 @@ int hm_model_load(const char* model_dir, int weight_dtype, int device, hm_engine
     Engine* eng = nullptr;
     int rc = Engine::create(spec, device, weight_dtype == HM_F32, &eng, &err);
     if (rc) return gfail(rc, err);
+    for (auto& f : files) {  // shapes of all shards first
+        MappedFile mf;
+        std::vector<TensorView> views;
+        if (files.size() > 1 && mf.open(f, &err) && parse_safetensors(mf, &views, &err))
+            for (const TensorView& t : views) eng->note_shape(t.name, t.shape);
+    }
     for (auto& f : files) {
         MappedFile mf;
         if (!mf.open(f, &err)) {

@@ -310,6 +310,32 @@ struct SplitRows {
     int n, groups;
 };
 
+// cos and sin of `turns` * pos full turns; the fraction of a turn is taken in double precision, so that far positions keep their phase.
+__device__ __forceinline__ void rotation_at(double turns, int pos, float& c, float& s) {
+    double f = turns * (double)pos;
+    f -= rint(f);
+    sincospif(2.0f * (float)f, &s, &c);
+}
+
+// Rotation in a projection's epilogue: outputs come in periods of `period` (even) columns, the first `dims` of which are pairs side by
+// side; pair i makes turns[i] turns per position.
+struct TurnedPairs {
+    const double* turns;     // null: none
+    int period, dims;
+    const int32_t* row_pos;
+};
+
+// Columns n (even) and n + 1 of row m.
+__device__ __forceinline__ void turn_pair(const TurnedPairs& t, int m, int n, float& u, float& v) {
+    const int d = n % t.period;
+    if (d >= t.dims) return;
+    float c, s;
+    rotation_at(__ldg(t.turns + d / 2), t.row_pos[m], c, s);
+    const float x = u, y = v;
+    u = fmaf(x, c, -y * s);
+    v = fmaf(y, c, x * s);
+}
+
 struct KvDesc {
     void* k_pool;            // this layer's K pages [n_pages][kv_heads][page_tokens][hd]
     void* v_pool;
@@ -445,7 +471,9 @@ struct GemvArgs : GemvBase {
     const float* out_scale;  // [N] or null (EPI_STORE: the result is multiplied element by element before the residual is added)
     const float* gate;   // EPI_GATE: [M][ld_gate]
     int ld_gate;
-    bool extended() const { return pro == PRO_GNORM || pro == PRO_MERGE || epi == EPI_GATE || epi == EPI_SQRELU || group_slabs != 0 || out_scale != nullptr; }
+    TurnedPairs turn;    // EPI_STORE: with turn.turns
+    float softcap;       // EPI_LOGITS: > 0: softcap * tanh(logit / softcap)
+    bool extended() const { return turn.turns != nullptr || softcap > 0.f || pro == PRO_GNORM || pro == PRO_MERGE || epi == EPI_GATE || epi == EPI_SQRELU || group_slabs != 0 || out_scale != nullptr; }
 };
 
 struct AttnArgs {
@@ -516,13 +544,26 @@ cudaError_t launch_attn_decode(const AttnArgs& a, int M, bool kv_bf16, cudaStrea
 int attn_pick_nsplit(int M, int kv_heads, int max_pages, int sm_count, bool bf16_pages);
 int attn_pick_cluster(int max_pages, int max_cluster);
 
-cudaError_t launch_pack_slabs_from_nk(const uint16_t* src_nk, int N, int K, uint16_t* dst, int n_off, int interleave_which, cudaStream_t st);
+// k_total > 0: the rows are inputs [k_off, k_off + K) of a projection over k_total inputs
+cudaError_t launch_pack_slabs_from_nk(const uint16_t* src_nk, int N, int K, uint16_t* dst, int n_off, int interleave_which, cudaStream_t st, int k_total = 0, int k_off = 0);
 cudaError_t launch_pack_slabs_from_kn(const uint16_t* src_kn, int K, int N, uint16_t* dst, cudaStream_t st);
 // dst[i] = src[rows[i]] for n rows of W floats
 cudaError_t launch_gather_rows(const float* src, const int32_t* rows, int n, int W, float* dst, cudaStream_t st, bool pdl);
-// turns (with row_pos): sinusoidal position vectors are added, sine in the even and cosine in the odd elements; pair i makes turns[i]
-// turns per position
-cudaError_t launch_embed_gather(const void* table, int table_dtype, const uint32_t* tokens, int M, int H, int V, float* out, int* err_flag, cudaStream_t st, bool pdl, const double* turns = nullptr, const int32_t* row_pos = nullptr);
+// What joins a token's embedding.
+struct EmbedExtra {
+    float scale = 1.f;                   // times the table's row
+    const int32_t *row_pos = nullptr, *row_seq = nullptr;
+    // sinusoidal position vectors, sine in the even and cosine in the odd elements; pair i makes turns[i] turns per position
+    const double* turns = nullptr;
+    // row (previous token * mul_prev + token * mul_cur) mod buckets of a second table, row `buckets` at position 0.  The tokens of every
+    // sequence are kept by position.
+    const uint16_t* bigram = nullptr;    // bf16 [buckets + 1][H]
+    unsigned long long buckets = 0, mul_prev = 0, mul_cur = 0;
+    uint32_t* kept = nullptr;            // [sequence][kept_stride]
+    int kept_stride = 0;
+};
+cudaError_t launch_embed_gather(const void* table, int table_dtype, const uint32_t* tokens, int M, int H, int V, float* out, int* err_flag, cudaStream_t st, bool pdl, const EmbedExtra& extra = EmbedExtra());
+cudaError_t launch_add_constant(float* x, size_t n, float c, cudaStream_t st);
 cudaError_t launch_argmax_finish(const float* amax_val, const int32_t* amax_idx, int nslabs, int M, uint32_t* next_tok, uint32_t* feed_tok, int32_t* pos, uint32_t* hist, int hist_stride, cudaStream_t st, bool pdl);
 cudaError_t launch_argmax_rows(const float* logits, int rows, int n, uint32_t* out, cudaStream_t st);
 cudaError_t launch_rms_norm(const float* x, const float* w, float eps, int rows, int n, float* out, cudaStream_t st);

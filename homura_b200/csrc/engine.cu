@@ -75,8 +75,10 @@ int Engine::create(const ModelSpec& spec, int device, bool strict_f32, Engine** 
         e->kvdim_ = 0;
         e->qdim_ = 0;
         for (const LayerSpec& l : spec.layers) {
-            e->qdim_ = std::max(e->qdim_, l.heads * std::max(l.vdim, l.mixer == MIX_GQA ? l.dim : 0));
-            if (l.kv_rank > 1024) return bad("kv_rank must be at most 1024");
+            e->qdim_ = std::max(e->qdim_, l.heads * std::max(l.vdim, l.paged_kv() ? l.dim : l.q_rank ? l.q_stride() : 0));
+            if (l.latent_rank() > 1024) return bad("kv_rank (with rot_dim) must be at most 1024");
+            GlaShape g;
+            if (l.mixer == MIX_PARALLEL && !gla_shape(l.lin_dim, l.lin_vdim, &g)) return bad("linear attention heads have at most 1024 key and 512 value elements");
             if (l.experts > 1024) return bad("a mixture has at most 1024 experts");
         }
     } else {
@@ -111,9 +113,9 @@ Engine::~Engine() {
     };
     fr(embed_); fr(final_norm_); fr(rope_cos_); fr(rope_sin_);
     for (auto& l : layers_)
-        for (float* p : {l.in_ln, l.post_ln, l.qkv_bias, l.q_norm, l.k_norm, l.shift, l.ls1, l.ls2, l.latent_norm, l.v_mix, l.rel, l.correction}) fr(p);
-    for (auto& l : layers_) { fr(l.router); fr(l.exp_gu); fr(l.exp_down); }
-    fr(turns_);
+        for (float* p : {l.in_ln, l.post_ln, l.qkv_bias, l.q_norm, l.k_norm, l.shift, l.ls1, l.ls2, l.latent_norm, l.v_mix, l.rel, l.correction, l.in_bias, l.sink, l.conv_w, l.lin_norm, l.lin_up, l.lin_bias}) fr(p);
+    for (auto& l : layers_) { fr(l.router); fr(l.exp_gu); fr(l.exp_down); fr(l.turns); }
+    fr(turns_); fr(bigram_);
     each_linear([&](LinearW& w) { fr(w.slabs); fr(w.tc); fr(w.scales); fr(w.codes); fr(w.kq_data); fr(w.kq_tile_type); });
     free_listed();
     free_listed_cache();
@@ -744,6 +746,7 @@ int Engine::kv_view(int seq, int layer, float* k_out, float* v_out) {
 static const char* kProfNames[PC_COUNT] = {"embed", "qkv_rope_kvwrite", "attention", "o_proj_residual", "gate_up_swiglu", "down_residual", "lm_head", "argmax"};
 static const char* kProfNamesListed[PC_COUNT_LISTED] = {"embed", "in_proj", "attention", "o_proj_residual", "up_sqrelu", "down_residual", "lm_head", "argmax", "latent_write", "key_up", "value_up_gate"};
 static const char* kProfNamesGqa[PC_COUNT_LISTED] = {"embed", "qkv_proj", "attention", "o_proj", "experts_gate_up", "experts_down", "lm_head", "argmax", nullptr, nullptr, nullptr, "qk_norm_kv_write", "post_norm_router", "post_norm"};
+static const char* kProfNamesParallel[PC_COUNT_LISTED] = {"embed", "in_proj", "attention", "out_proj", "experts_gate_up", "experts_down", "lm_head", "argmax", nullptr, "key_up", "value_up", "side", nullptr, "sum_norm", "query_up"};
 
 void Engine::prof_mark(int) {}
 
@@ -957,6 +960,9 @@ int Engine::enqueue_linear(const LinearW& L, int M, const float* x, int ldx, int
                     a.split.acc += (size_t)m0 * a.split.groups * a.split.n * L.K;
                     a.split.ml += (size_t)m0 * a.split.groups * a.split.n * 2;
                 }
+                a.turn = opt->turn;
+                if (a.turn.row_pos) a.turn.row_pos += m0;
+                a.softcap = opt->softcap;
                 a.out_scale = opt->out_scale;
                 a.gate = opt->gate ? opt->gate + (size_t)m0 * opt->ld_gate : nullptr;
                 a.ld_gate = opt->ld_gate;
@@ -1086,7 +1092,18 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
     }
     auto want = [&](int cls) { return only_class_ < 0 || only_class_ == cls; };
     if (want(PC_EMBED)) {
-        ce = launch_embed_gather(embed_, embed_dtype_ == HM_BF16 ? 1 : 0, tokens_dev, M, H_, V_, h_, err_flag_, stream_, pdl_, turns_, row_pos);
+        EmbedExtra x;
+        x.scale = spec_.embed_scale;
+        x.row_pos = row_pos;
+        x.row_seq = row_seq;
+        x.turns = turns_;
+        x.bigram = bigram_;
+        x.buckets = (unsigned long long)spec_.bigram_buckets;
+        x.mul_prev = (unsigned long long)spec_.bigram_prev;
+        x.mul_cur = (unsigned long long)spec_.bigram_cur;
+        x.kept = hist_dev_;
+        x.kept_stride = max_seq_ + 1;
+        ce = launch_embed_gather(embed_, embed_dtype_ == HM_BF16 ? 1 : 0, tokens_dev, M, H_, V_, h_, err_flag_, stream_, pdl_, x);
         if (ce != cudaSuccess) return cuda_fail(ce, "embed_gather");
         ++*launches;
     }
@@ -1114,7 +1131,7 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
     const bool fused = direct_pack && H_ % 128 == 0;
     for (int l = 0; l < L_; ++l) {
         if (spec_.listed()) {
-            rc = spec_.layers[l].mixer == MIX_GQA ? enqueue_gqa_layer(l, M, row_pos, row_seq, lm_rows, launches) : enqueue_listed_layer(l, M, row_pos, row_seq, lm_rows, launches);
+            rc = spec_.parallel ? enqueue_parallel_layer(l, M, row_pos, row_seq, lm_rows, launches) : spec_.layers[l].mixer == MIX_GQA ? enqueue_gqa_layer(l, M, row_pos, row_seq, lm_rows, launches) : enqueue_listed_layer(l, M, row_pos, row_seq, lm_rows, launches);
             if (rc) return rc;
             rc = tap(l, M);
             if (rc) return rc;
@@ -1634,10 +1651,11 @@ int Engine::time_decode(int warmup, int steps, float* ms_total) {
 int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (batch_ == 0) return fail(HM_ERR_STATE, "profile_decode before kv_alloc");
-    if (steps < 1 || !out || !n_out || cap < (spec_.listed() ? PC_COUNT_LISTED : PC_COUNT)) return fail(HM_ERR_INVALID, "profile_decode: bad arguments (cap >= 8; 14 for listed designs)");
+    if (steps < 1 || !out || !n_out || cap < (spec_.listed() ? PC_COUNT_LISTED : PC_COUNT)) return fail(HM_ERR_INVALID, "profile_decode: bad arguments (cap >= 8; 15 for listed designs)");
+    const bool moe = spec_.post_norm || spec_.parallel;
     for (int b = 0; b < batch_; ++b)
-        if (len_[b] + steps + (spec_.post_norm ? 1 : 0) > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full: not enough room for the profiled steps");
-    if (const int prc = ensure_pages_all(steps + (spec_.post_norm ? 1 : 0))) return prc;
+        if (len_[b] + steps + (moe ? 1 : 0) > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full: not enough room for the profiled steps");
+    if (const int prc = ensure_pages_all(steps + (moe ? 1 : 0))) return prc;
     const int classes = spec_.listed() ? PC_COUNT_LISTED : PC_COUNT;
     pass_longest_ = max_seq_;
     HM_CUDA(cudaStreamSynchronize(stream_));
@@ -1683,7 +1701,7 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
     cudaEventDestroy(e0);
     cudaEventDestroy(e1);
     if (rc) return rc;
-    if (spec_.post_norm) {  // which experts such a step reads: one more pass, without logits, at the position it has reached
+    if (moe) {  // which experts such a step reads: one more pass, without logits, at the position it has reached
         std::vector<int> seen;
         int launches = 0;
         experts_seen_ = &seen;
@@ -1708,17 +1726,26 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
         bytes[PC_DOWN] += expert_bytes(li, false);
         bytes[PC_KUP] += l.kup.bytes();
         bytes[PC_VUP] += l.vup.bytes();
+        bytes[PC_QUP] += l.uq.bytes();
+        if (spec_.parallel && spec_.layers[li].mixer == MIX_PARALLEL) bytes[PC_KV_WRITE] += 2ull * batch_ * spec_.layers[li].lin_heads * spec_.layers[li].lin_dim * spec_.layers[li].lin_vdim * 4;
         bytes[PC_O] += l.o.bytes();
         bytes[PC_GATE_UP] += l.gu.bytes();
         bytes[PC_DOWN] += l.down.bytes();
     }
     bytes[PC_LM_HEAD] = lm_head_.bytes();
     if (spec_.listed()) {
-        for (const LayerSpec& l : spec_.layers) bytes[PC_ATTN] += (uint64_t)(kv_tokens * (l.mixer == MIX_LATENT ? l.kv_rank : l.kv_heads * (l.dim + l.vdim)) * (kv_bf16_ ? 2 : 4));
+        for (const LayerSpec& l : spec_.layers) {
+            double tokens = kv_tokens;
+            if (l.window > 0) {
+                tokens = 0;
+                for (int b = 0; b < batch_; ++b) tokens += std::min(len_[b] - steps + 1, l.window + l.keep_first);
+            }
+            bytes[PC_ATTN] += (uint64_t)(tokens * (l.mixer == MIX_LATENT ? l.latent_rank() : l.kv_heads * (l.dim + l.vdim)) * (kv_bf16_ ? 2 : 4));
+        }
     } else {
         bytes[PC_ATTN] = (uint64_t)(kv_tokens * L_ * 2.0 * kvh_ * hd_ * (kv_bf16_ ? 2 : 4));
     }
-    const char* const* names = !spec_.listed() ? kProfNames : spec_.post_norm ? kProfNamesGqa : kProfNamesListed;
+    const char* const* names = !spec_.listed() ? kProfNames : spec_.parallel ? kProfNamesParallel : spec_.post_norm ? kProfNamesGqa : kProfNamesListed;
     int n = 0;
     for (int c = 0; c < classes; ++c) {
         if (!names[c]) continue;

@@ -12,11 +12,13 @@
 
 #include "../../include/homura_b200.h"
 #include "common.cuh"
+#include "gla.h"
 #include "gqa_attn.h"
 #include "latent_attn.h"
 #include "moe.h"
 #include "model_spec.h"
 #include "sampler.h"
+#include "side.h"
 
 namespace hm {
 
@@ -64,6 +66,17 @@ struct LayerW {
     float* correction = nullptr;
     uint16_t *exp_gu = nullptr, *exp_down = nullptr;  // all experts' tile images (moe.h)
     std::vector<uint8_t> exp_seen;       // per expert: bits of the parts loaded
+    // listed designs with parallel sublayers: `in` is everything that reads the norm, `o` everything that joins the residual (besides
+    // the chosen experts), see ParallelColumns
+    std::vector<std::string> seen;       // tensors loaded
+    float* in_bias = nullptr;            // [columns of `in`]
+    float* sink = nullptr;               // [heads]
+    float* conv_w = nullptr;             // [query, key and value channels][taps]
+    float *lin_norm = nullptr, *lin_up = nullptr, *lin_bias = nullptr;  // linear attention: result norm, decay up-projection [heads][rank][dim], its bias
+    LinearW uq;                          // queries out of their latent
+    double* turns = nullptr;             // rotation, turns per position of every pair
+    GlaShape gla{};
+    size_t conv_at = 0, gla_at = 0;      // this layer's part of a sequence's state, in floats
 };
 
 // What a projection launch needs beyond the common arguments (enqueue_linear)
@@ -74,6 +87,19 @@ struct LinOpt {
     const float* gate = nullptr;
     int ld_gate = 0;
     int group_x = 0;                     // grouped projections: inputs of one group to the next
+    TurnedPairs turn{};
+    float softcap = 0.f;
+};
+
+// Columns of a parallel layer's input projection (what reads the norm of the residual) and inputs of its output projection (what
+// joins the residual).  Parts start at multiples of 8 columns and of 64 inputs; queries, keys and values are contiguous.
+struct ParallelColumns {
+    int q = 0, k = 0, v = 0, gate = 0, gates = 0;          // attention, its output gates
+    int lq = 0, lk = 0, lv = 0, lg = 0, la = 0;            // linear attention, gate, decay latent
+    int dq = 0, dkv = 0;                                   // latents of queries; of keys and values with the rotated part behind
+    int router = 0, row_gate = 0, ff_gate = 0, ff_up = 0, ff = 0;  // dense or shared feed-forward
+    int n = 0, ld = 0;
+    int vals = 0, lin_in = 0, ff_in = 0, k_out = 0;
 };
 
 // final argmax folded into the LM-head launch (see GemvArgs::fin_ticket)
@@ -90,6 +116,8 @@ class Engine {
     static int create(const ModelSpec& spec, int device, bool strict_f32, Engine** out, std::string* err);
     ~Engine();
 
+    // Shape of a tensor that load_tensor will bring: sizes that only tensors tell must be known before their layer's projections.
+    void note_shape(const std::string& name, const std::vector<int64_t>& shape);
     int load_tensor(const char* name, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
     int finalize();
 
@@ -152,6 +180,7 @@ class Engine {
     int load_gqa_tensor(LayerW& w, const LayerSpec& s, const std::string& name, const std::string& rest, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
     int load_bias_table(LayerW& w, const LayerSpec& s, int dtype, const int64_t* shape, const void* host, size_t nbytes);
     int load_expert(LayerW& w, const LayerSpec& s, int expert, int part, int dtype, const void* host, size_t nbytes);
+    bool load_expert_tensor(LayerW& w, const LayerSpec& s, const std::string& name, const std::string& rest, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes, int* rc);
     int finalize_gqa(const LayerW& w, const LayerSpec& s, const std::string& at);
     int alloc_gqa_scratch();
     void free_gqa_scratch();
@@ -162,6 +191,22 @@ class Engine {
     uint64_t expert_bytes(int layer, bool gate_up) const;
     int count_experts(int M, const LayerSpec& s);
     int enqueue_gqa_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int next_lm_rows, int* launches);
+    // listed designs with parallel sublayers (engine_parallel.cu)
+    int load_parallel_tensor(int layer, const std::string& name, const std::string& rest, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
+    int load_inputs(LinearW& L, int k_total, int k_off, int k_part, int N, int dtype, const void* host, size_t nbytes);
+    int load_bigram(int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
+    int upload(float** dst, const std::vector<float>& v);
+    int finalize_parallel();
+    int alloc_parallel_scratch();
+    void free_parallel_scratch();
+    SideArgs side_args(int l, int M, bool tall, const ParallelColumns& c, const int32_t* row_pos, const int32_t* row_seq) const;
+    int enqueue_parallel_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int next_lm_rows, int* launches);
+    // shared by the listed designs
+    GqaRuns pass_runs(int M, int* longest) const;
+    GqaAttnArgs gqa_attn_args(int l, int M, bool tall, const int32_t* row_pos, const int32_t* row_seq) const;
+    int enqueue_latent_attn(int l, int M, bool tall, const int32_t* row_pos, const int32_t* row_seq, int* launches);
+    // x: the rows that the experts read (few rows); resid: added to the result (few rows) or null.  With many rows `parts` partial results in sub_.
+    int enqueue_experts(int l, int M, bool tall, const float* x, const float* resid, float* y, int* parts, int* launches);
     int enqueue_listed_logits(const float* x, int rows, float* dst, const struct ArgmaxFold& fold, int* launches);
     int enqueue_tc(const LinearW& L, int M, const unsigned char* xp, int epi, float* y, int ldy, TcArgs& a, int* launches);
     LatentPool latent_pool(int layer) const;
@@ -176,7 +221,7 @@ class Engine {
     template <typename F>
     void each_linear(F f) {
         for (auto& l : layers_)
-            for (LinearW* w : {&l.qkv, &l.o, &l.gu, &l.down, &l.in, &l.kup, &l.vup}) f(*w);
+            for (LinearW* w : {&l.qkv, &l.o, &l.gu, &l.down, &l.in, &l.kup, &l.vup, &l.uq}) f(*w);
         f(lm_head_);
     }
     // RMSNorm handed from one tensor-core GEMM to the next without a packing launch (see TcArgs)
@@ -251,6 +296,15 @@ class Engine {
     size_t lat_acc_floats_ = 0, lat_ml_floats_ = 0;
     std::vector<void*> lat_pool_;  // per layer, null for layers that read another's
     float *shift_state_ = nullptr, *shift_saved_ = nullptr;  // [layers][sequences][SHIFT_RING][H]; [layers][SHIFT_RING][H]
+    // State of a sequence that is not addressed by position: short convolutions and linear attention of all layers, one row per
+    // sequence; [state_floats_] for the copy that generation loops take
+    float *state_ = nullptr, *state_saved_ = nullptr;
+    size_t state_floats_ = 0;
+    uint16_t* bigram_ = nullptr;     // second embedding table
+    float* normed_ = nullptr;        // normalised input of a layer, for experts that read rows
+    float* cat_ = nullptr;           // inputs of a parallel layer's output projection,
+    unsigned char *xpack_cat_ = nullptr, *xpack_cq_ = nullptr;  // their image; that of the queries' latents
+    int cat_ld_ = 0;
     double* turns_ = nullptr;        // sinusoidal positions: turns per position of every pair of elements
     float* sub_ = nullptr;           // what a sublayer gave back, before its norm
     float* v_first_ = nullptr;       // values of the layer that the others blend in

@@ -87,6 +87,21 @@ int Engine::load_expert(LayerW& w, const LayerSpec& s, int expert, int part, int
     return HM_OK;
 }
 
+// mlp.e<index>.gate / up / down; false: another tensor
+bool Engine::load_expert_tensor(LayerW& w, const LayerSpec& s, const std::string& name, const std::string& rest, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes, int* rc) {
+    const size_t dot = rest.find('.', 5);
+    if (rest.compare(0, 5, "mlp.e") != 0 || dot == std::string::npos || dot <= 5 || rest.find_first_not_of("0123456789", 5) != dot) return false;
+    const long e = std::atol(rest.c_str() + 5);
+    const std::string what = rest.substr(dot + 1);
+    const int part = what == "gate" ? 0 : what == "up" ? 1 : what == "down" ? 2 : -1;
+    if (part < 0) return false;
+    if (e >= s.experts) *rc = fail(HM_ERR_INVALID, "expert index out of range in " + name);
+    else if (ndim != 2 || shape[0] != (part < 2 ? s.ff : H_) || shape[1] != (part < 2 ? H_ : s.ff)) *rc = fail(HM_ERR_INVALID, "unexpected shape for tensor " + name);
+    else if ((size_t)e < w.exp_seen.size() && (w.exp_seen[e] >> part & 1)) *rc = fail(HM_ERR_STATE, "tensor loaded twice: " + name);
+    else *rc = load_expert(w, s, (int)e, part, dtype, host, nbytes);
+    return true;
+}
+
 int Engine::load_gqa_tensor(LayerW& w, const LayerSpec& s, const std::string& name, const std::string& rest, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes) {
     size_t n = 1;
     for (int i = 0; i < ndim; ++i) n *= (size_t)shape[i];
@@ -122,18 +137,8 @@ int Engine::load_gqa_tensor(LayerW& w, const LayerSpec& s, const std::string& na
             HM_CUDA(cudaStreamSynchronize(stream_));
             return HM_OK;
         }
-        const size_t dot = rest.find('.', 5);
-        if (rest.compare(0, 5, "mlp.e") == 0 && dot != std::string::npos && dot > 5 && rest.find_first_not_of("0123456789", 5) == dot) {
-            const long e = std::atol(rest.c_str() + 5);
-            const std::string what = rest.substr(dot + 1);
-            const int part = what == "gate" ? 0 : what == "up" ? 1 : what == "down" ? 2 : -1;
-            if (part >= 0) {
-                if (e >= s.experts) return fail(HM_ERR_INVALID, "expert index out of range in " + name);
-                if (!(part < 2 ? is2(s.ff, H_) : is2(H_, s.ff))) return bad_shape();
-                if ((size_t)e < w.exp_seen.size() && (w.exp_seen[e] >> part & 1)) return twice();
-                return load_expert(w, s, (int)e, part, dtype, host, nbytes);
-            }
-        }
+        int rc = HM_OK;
+        if (load_expert_tensor(w, s, name, rest, dtype, shape, ndim, host, nbytes, &rc)) return rc;
     }
     return fail(HM_ERR_INVALID, "unknown tensor name: " + name);
 }
@@ -164,7 +169,7 @@ void Engine::free_gqa_scratch() {
 
 // A pass of a listed design has at most TC_ROWS rows.
 int Engine::alloc_gqa_scratch() {
-    if (!spec_.post_norm) return HM_OK;
+    if (!spec_.post_norm && !spec_.parallel) return HM_OK;
     size_t values = 1, top = 1, experts = 1, act = 1, img = 1;
     for (const LayerSpec& s : spec_.layers) {
         if (s.v_mix) values = std::max(values, (size_t)s.kv_heads * s.vdim);
@@ -203,7 +208,7 @@ double Engine::experts_used(const LayerSpec& s, int rows) const { return s.exper
 
 ExpertWeights Engine::expert_weights(int layer) const {
     const LayerSpec& s = spec_.layers[layer];
-    return ExpertWeights{layers_[layer].exp_gu, layers_[layer].exp_down, s.experts, H_, s.ff, s.top, s.limit};
+    return ExpertWeights{layers_[layer].exp_gu, layers_[layer].exp_down, s.experts, H_, s.ff, s.top, s.limit, s.act};
 }
 
 // Bytes of expert weights that the last profiled step read.
@@ -221,6 +226,102 @@ int Engine::count_experts(int M, const LayerSpec& s) {
     int n = 0;
     for (size_t i = 0; i < ids.size(); ++i) n += ids[i] >= 0 && (i == 0 || ids[i] != ids[i - 1]);
     experts_seen_->push_back(n);
+    return HM_OK;
+}
+
+// ---- shared pieces -----------------------------------------------------------------------------------
+
+GqaRuns Engine::pass_runs(int M, int* longest) const {
+    GqaRuns runs;
+    *longest = 1;
+    for (auto& r : pass_runs_) {
+        runs.row[runs.n++] = (uint8_t)r.first;
+        *longest = std::max(*longest, r.second);
+    }
+    runs.row[runs.n] = (uint8_t)M;
+    return runs;
+}
+
+// The attention of layer l over the queries in q_, without what only some designs have and where the results go.
+GqaAttnArgs Engine::gqa_attn_args(int l, int M, bool tall, const int32_t* row_pos, const int32_t* row_seq) const {
+    GqaAttnArgs a{};
+    a.pool = gqa_pool(l);
+    a.q = q_;
+    a.M = M;
+    a.heads = spec_.layers[l].heads;
+    a.row_pos = row_pos;
+    a.row_seq = row_seq;
+    a.runs = pass_runs(M, &a.longest_run);
+    a.longest = pass_longest_;
+    a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
+    a.max_cluster = use_clusters_ ? std::min(max_cluster_, 16) : 1;
+    a.xp_mpad = tall ? tc_mpad(M) : 0;
+    a.err_flag = err_flag_;
+    return a;
+}
+
+int Engine::enqueue_experts(int l, int M, bool tall, const float* x, const float* resid, float* y, int* parts, int* launches) {
+    const LayerW& w = layers_[l];
+    const LayerSpec& s = spec_.layers[l];
+    auto want = [&](int cls) { return only_class_ < 0 || only_class_ == cls; };
+    cudaError_t ce;
+    TcArgs ta{};
+    if (tall) {
+        ta.ex.n = s.experts;
+        ta.ex.blocks = expert_blocks(s.ff);
+        ta.ex.weight = rt_dense_;
+        ta.ex.mask = rt_mask_;
+        ta.ex.limit = s.limit;
+        ta.ex.act = s.act;
+        ta.ex.img_bytes = tc_xpack_bytes(M, s.ff);
+        ta.ex.used = std::max(1, (int)experts_used(s, M));
+        ta.ex.parts = 1;
+        ta.ex.part_stride = (size_t)TC_ROWS * H_;
+        ta.M = M;
+        ta.xp_mpad = tc_mpad(M);
+        ta.err_flag = err_flag_;
+    }
+    if (want(PC_GATE_UP)) {
+        if (tall) {
+            TcArgs a = ta;
+            a.W = w.exp_gu;
+            a.K = H_;
+            a.Kp = tc_padded_k(H_);
+            a.N = s.experts * a.ex.blocks * SLAB;
+            a.ksplit = tc_pick_split(H_, a.ex.used * a.ex.blocks * SLAB, sm_count_);
+            a.xp = xpack_;
+            a.epi = EPI_EXPERT;
+            a.xp_out = exp_img_;
+            ce = launch_gemm_tc(a, stream_, pdl_);
+        } else {
+            ce = launch_expert_gate_up(expert_weights(l), x, M, route_out(tall), exp_act_, stream_, pdl_);
+        }
+        if (ce != cudaSuccess) return cuda_fail(ce, "expert gate / up launch");
+        ++*launches;
+    }
+    // the sum over the experts' activations is long: with few output blocks it is cut into parts, which the norm adds up
+    const int down_k = ta.ex.used * expert_blocks(s.ff) * 64, down_split = tc_pick_split(down_k, H_, sm_count_);
+    *parts = !tall ? 1 : std::max(1, std::min({sub_parts_, sm_count_ / ((H_ + SLAB - 1) / SLAB * down_split), down_k / 64 / (4 * down_split)}));
+    if (want(PC_DOWN)) {
+        if (tall) {
+            TcArgs a = ta;
+            a.W = w.exp_down;
+            a.K = s.ff;
+            a.Kp = tc_padded_k(s.ff);
+            a.N = H_;
+            a.ksplit = down_split;
+            a.ex.parts = *parts;
+            a.xp = exp_img_;
+            a.epi = EPI_STORE;
+            a.y = sub_;
+            a.ldy = H_;
+            ce = launch_gemm_tc(a, stream_, pdl_);
+        } else {
+            ce = launch_expert_down(expert_weights(l), exp_act_, M, route_out(tall), resid, y, stream_, pdl_);
+        }
+        if (ce != cudaSuccess) return cuda_fail(ce, "expert down launch");
+        ++*launches;
+    }
     return HM_OK;
 }
 
@@ -280,30 +381,11 @@ int Engine::enqueue_gqa_layer(int l, int M, const int32_t* row_pos, const int32_
         ++*launches;
     }
     if (want(PC_ATTN)) {
-        GqaAttnArgs a{};
-        a.pool = gqa_pool(l);
-        a.q = q_;
-        a.M = M;
-        a.heads = s.heads;
-        a.row_pos = row_pos;
-        a.row_seq = row_seq;
+        GqaAttnArgs a = gqa_attn_args(l, M, tall, row_pos, row_seq);
         a.bias = w.rel;
         a.reach = w.reach;
-        a.longest_run = 1;
-        for (auto& r : pass_runs_) {
-            a.runs.row[a.runs.n++] = (uint8_t)r.first;
-            a.longest_run = std::max(a.longest_run, r.second);
-        }
-        a.runs.row[a.runs.n] = (uint8_t)M;
-        a.longest = pass_longest_;
-        a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
-        a.max_cluster = use_clusters_ ? std::min(max_cluster_, 16) : 1;
         a.out = attn_;
-        if (tall) {
-            a.xp = xpack_attn_;
-            a.xp_mpad = tc_mpad(M);
-        }
-        a.err_flag = err_flag_;
+        if (tall) a.xp = xpack_attn_;
         ce = launch_gqa_attn(a, sm_count_, stream_, pdl_);
         if (ce != cudaSuccess) return cuda_fail(ce, "attention launch");
         ++*launches;
@@ -349,62 +431,9 @@ int Engine::enqueue_gqa_layer(int l, int M, const int32_t* row_pos, const int32_
         }
     }
     if (!moe) return HM_OK;
-    TcArgs ta{};
-    if (tall) {
-        ta.ex.n = s.experts;
-        ta.ex.blocks = expert_blocks(s.ff);
-        ta.ex.weight = rt_dense_;
-        ta.ex.mask = rt_mask_;
-        ta.ex.limit = s.limit;
-        ta.ex.img_bytes = tc_xpack_bytes(M, s.ff);
-        ta.ex.used = std::max(1, (int)experts_used(s, M));
-        ta.ex.parts = 1;
-        ta.ex.part_stride = (size_t)TC_ROWS * H_;
-        ta.M = M;
-        ta.xp_mpad = tc_mpad(M);
-        ta.err_flag = err_flag_;
-    }
-    if (want(PC_GATE_UP)) {
-        if (tall) {
-            TcArgs a = ta;
-            a.W = w.exp_gu;
-            a.K = H_;
-            a.Kp = tc_padded_k(H_);
-            a.N = s.experts * a.ex.blocks * SLAB;
-            a.ksplit = tc_pick_split(H_, a.ex.used * a.ex.blocks * SLAB, sm_count_);
-            a.xp = xpack_;
-            a.epi = EPI_EXPERT;
-            a.xp_out = exp_img_;
-            ce = launch_gemm_tc(a, stream_, pdl_);
-        } else {
-            ce = launch_expert_gate_up(expert_weights(l), h_, M, route_out(tall), exp_act_, stream_, pdl_);
-        }
-        if (ce != cudaSuccess) return cuda_fail(ce, "expert gate / up launch");
-        ++*launches;
-    }
-    // the sum over the experts' activations is long: with few output blocks it is cut into parts, which the norm adds up
-    const int down_k = ta.ex.used * expert_blocks(s.ff) * 64, down_split = tc_pick_split(down_k, H_, sm_count_);
-    const int parts = !tall ? 1 : std::max(1, std::min({sub_parts_, sm_count_ / ((H_ + SLAB - 1) / SLAB * down_split), down_k / 64 / (4 * down_split)}));
-    if (want(PC_DOWN)) {
-        if (tall) {
-            TcArgs a = ta;
-            a.W = w.exp_down;
-            a.K = s.ff;
-            a.Kp = tc_padded_k(s.ff);
-            a.N = H_;
-            a.ksplit = down_split;
-            a.ex.parts = parts;
-            a.xp = exp_img_;
-            a.epi = EPI_STORE;
-            a.y = sub_;
-            a.ldy = H_;
-            ce = launch_gemm_tc(a, stream_, pdl_);
-        } else {
-            ce = launch_expert_down(expert_weights(l), exp_act_, M, route_out(tall), sub_, stream_, pdl_);
-        }
-        if (ce != cudaSuccess) return cuda_fail(ce, "expert down launch");
-        ++*launches;
-    }
+    int parts = 1;
+    rc = enqueue_experts(l, M, tall, h_, nullptr, sub_, &parts, launches);
+    if (rc) return rc;
     if (want(PC_NORM)) {
         PostNormArgs a = pn;
         a.w = w.post_ln;

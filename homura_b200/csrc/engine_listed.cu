@@ -15,6 +15,7 @@
 #include <algorithm>
 
 #include "engine.h"
+#include "engine_parallel.h"
 #include "engine_util.h"
 #include "gemm_tc.h"
 
@@ -90,9 +91,15 @@ int Engine::load_listed_tensor(const std::string& name, int dtype, const int64_t
         if (rc) return rc;
         HM_CUDA(cudaStreamSynchronize(stream_));
         embed_dtype_ = HM_BF16;
-        return HM_OK;
+        return cfg_.tie_word_embeddings ? lin(lm_head_, H_, V_, 0, V_) : HM_OK;
     }
-    if (name == "final.norm") return vec(&final_norm_, H_);
+    if (name == "final.norm") {
+        const int rc = vec(&final_norm_, H_);
+        if (rc == HM_OK && spec_.norm_offset) HM_CUDA(launch_add_constant(final_norm_, H_, 1.f, stream_));
+        return rc;
+    }
+    if (name == "bigram" && spec_.bigram_buckets > 0) return load_bigram(dtype, shape, ndim, host, nbytes);
+    if (name == "head" && cfg_.tie_word_embeddings) return fail(HM_ERR_INVALID, "unknown tensor name: " + name);
     if (name == "head") return lin(lm_head_, H_, V_, 0, V_);
     const size_t dot = name.find('.');
     if (name.size() < 3 || name[0] != 'l' || dot == std::string::npos || name.find_first_not_of("0123456789", 1) != dot) return fail(HM_ERR_INVALID, "unknown tensor name: " + name);
@@ -101,7 +108,12 @@ int Engine::load_listed_tensor(const std::string& name, int dtype, const int64_t
     const std::string rest = name.substr(dot + 1);
     LayerW& w = layers_[li];
     const LayerSpec& s = spec_.layers[li];
-    if (rest == "norm1") return vec(&w.in_ln, H_);
+    if (rest == "norm1") {
+        const int rc = vec(&w.in_ln, H_);
+        if (rc == HM_OK && spec_.norm_offset) HM_CUDA(launch_add_constant(w.in_ln, H_, 1.f, stream_));
+        return rc;
+    }
+    if (spec_.parallel) return load_parallel_tensor((int)li, name, rest, dtype, shape, ndim, host, nbytes);
     if (rest == "norm2") return vec(&w.post_ln, H_);
     if (s.mixer == MIX_GQA) return load_gqa_tensor(w, s, name, rest, dtype, shape, ndim, host, nbytes);
     if (rest == "shift") return vec(&w.shift, H_);
@@ -121,6 +133,7 @@ int Engine::load_listed_tensor(const std::string& name, int dtype, const int64_t
 }
 
 int Engine::finalize_listed() {
+    if (spec_.parallel) return finalize_parallel();
     for (int i = 0; i < L_; ++i) {
         const LayerW& l = layers_[i];
         const LayerSpec& s = spec_.layers[i];
@@ -152,6 +165,7 @@ void Engine::free_listed() {
         p = nullptr;
     };
     free_gqa_scratch();
+    free_parallel_scratch();
     fr(mix_raw_); fr(qlat_); fr(ctx_); fr(xpack_q_); fr(xpack_ctx_); fr(lat_acc_); fr(lat_ml_);
 }
 
@@ -161,19 +175,21 @@ int Engine::alloc_listed_scratch(int cap) {
     int kmax = H_;
     for (const LayerSpec& s : spec_.layers) {
         kmax = std::max(kmax, std::max(s.heads * s.vdim, s.ff));
+        if (spec_.parallel) raw = std::max(raw, (size_t)parallel_columns(s).ld);
         if (s.mixer != MIX_LATENT) {
             raw = std::max(raw, (size_t)(s.heads * s.dim + s.kv_heads * (s.dim + s.vdim) + 3) / 4 * 4);
             continue;
         }
         raw = std::max(raw, (size_t)in_ld(s));
-        lat = std::max(lat, (size_t)s.heads * s.kv_rank);
-        q_img = std::max(q_img, s.heads * tc_xpack_bytes(TC_ROWS, s.dim));
-        ctx_img = std::max(ctx_img, s.heads * tc_xpack_bytes(TC_ROWS, s.kv_rank));
-        kmax = std::max(kmax, std::max(s.dim, s.kv_rank));
+        const int rank = s.latent_rank();
+        lat = std::max(lat, (size_t)s.heads * rank);
+        q_img = std::max(q_img, s.heads * tc_xpack_bytes(TC_ROWS, s.q_rank ? s.q_stride() : s.dim));
+        ctx_img = std::max(ctx_img, s.heads * tc_xpack_bytes(TC_ROWS, rank));
+        kmax = std::max(kmax, std::max(s.dim, rank));
         // splits times rows never exceed the SMs times the rows that share a CTA (latent_pick_nsplit)
         for (int bf16 = 0; bf16 < 2; ++bf16) {
-            const size_t rows = 2 * (size_t)sm_count_ * latent_rows_per_tile(TC_ROWS, 1 << 30, s.heads, s.kv_rank, bf16);
-            acc = std::max(acc, rows * s.heads * s.kv_rank);
+            const size_t rows = 2 * (size_t)sm_count_ * latent_rows_per_tile(TC_ROWS, 1 << 30, s.heads, rank, bf16);
+            acc = std::max(acc, rows * s.heads * rank);
             ml = std::max(ml, rows * s.heads * 2);
         }
     }
@@ -199,7 +215,8 @@ int Engine::alloc_listed_scratch(int cap) {
         HM_CUDA(get(&xpack_q_, q_img));
         HM_CUDA(get(&xpack_ctx_, ctx_img));
     }
-    return alloc_gqa_scratch();
+    const int rc = alloc_gqa_scratch();
+    return rc ? rc : alloc_parallel_scratch();
 }
 
 void Engine::free_listed_cache() {
@@ -209,13 +226,16 @@ void Engine::free_listed_cache() {
     if (shift_state_) cudaFree(shift_state_);
     if (shift_saved_) cudaFree(shift_saved_);
     shift_state_ = shift_saved_ = nullptr;
+    if (state_) cudaFree(state_);
+    if (state_saved_) cudaFree(state_saved_);
+    state_ = state_saved_ = nullptr;
 }
 
 int Engine::alloc_listed_cache(int batch, size_t n_pages) {
     lat_pool_.assign(L_, nullptr);
     for (int l = 0; l < L_; ++l) {
         const LayerSpec& s = spec_.layers[l];
-        if (s.mixer == MIX_GQA) {
+        if (s.paged_kv()) {
             const size_t esz = kv_bf16_ ? 2 : 4, kb = n_pages * gqa_page_elems(s.kv_heads, s.dim) * esz, vb = n_pages * gqa_page_elems(s.kv_heads, s.vdim) * esz;
             HM_CUDA(cudaMalloc(&k_pool_[l], kb));
             HM_CUDA(cudaMalloc(&v_pool_[l], vb));
@@ -224,9 +244,23 @@ int Engine::alloc_listed_cache(int batch, size_t n_pages) {
             continue;
         }
         if (s.kv_from >= 0) continue;
-        const size_t bytes = n_pages * latent_page_elems(s.kv_rank, kv_bf16_) * (kv_bf16_ ? 2 : 4);
+        const size_t bytes = n_pages * latent_page_elems(s.latent_rank(), kv_bf16_) * (kv_bf16_ ? 2 : 4);
         HM_CUDA(cudaMalloc(&lat_pool_[l], bytes));
         HM_CUDA(cudaMemset(lat_pool_[l], 0, bytes));
+    }
+    state_floats_ = 0;
+    for (int l = 0; l < L_; ++l) {
+        const LayerSpec& s = spec_.layers[l];
+        LayerW& w = layers_[l];
+        w.conv_at = state_floats_;
+        if (s.conv > 1) state_floats_ += ((size_t)(s.conv - 1) * (s.heads * s.dim + s.kv_heads * (s.dim + s.vdim)) + 3) / 4 * 4;
+        w.gla_at = state_floats_;
+        if (s.mixer == MIX_PARALLEL) state_floats_ += s.lin_heads * w.gla.state_floats();
+    }
+    if (state_floats_) {
+        HM_CUDA(cudaMalloc(&state_, batch * state_floats_ * 4));
+        HM_CUDA(cudaMemset(state_, 0, batch * state_floats_ * 4));
+        HM_CUDA(cudaMalloc(&state_saved_, state_floats_ * 4));
     }
     if (spec_.token_shift) {
         const size_t row = (size_t)SHIFT_RING * H_ * 4;
@@ -239,7 +273,7 @@ int Engine::alloc_listed_cache(int batch, size_t n_pages) {
 
 LatentPool Engine::latent_pool(int layer) const {
     const LayerSpec& s = spec_.layers[layer];
-    return LatentPool{lat_pool_[s.kv_from >= 0 ? s.kv_from : layer], page_table_, max_pages_, s.kv_rank, kv_bf16_ ? 1 : 0};
+    return LatentPool{lat_pool_[s.kv_from >= 0 ? s.kv_from : layer], page_table_, max_pages_, s.latent_rank(), kv_bf16_ ? 1 : 0};
 }
 
 int Engine::latent_view(int seq, int layer, float* out) {
@@ -249,7 +283,7 @@ int Engine::latent_view(int seq, int layer, float* out) {
     if (!spec_.listed() || spec_.layers[layer].mixer != MIX_LATENT) return fail(HM_ERR_UNSUPPORTED, "latent_view: this design caches keys and values (hm_kv_view)");
     const int len = len_[seq];
     if (len == 0) return HM_OK;
-    const size_t bytes = (size_t)len * spec_.layers[layer].kv_rank * 4;
+    const size_t bytes = (size_t)len * spec_.layers[layer].latent_rank() * 4;
     float* d = nullptr;
     HM_CUDA(cudaMalloc(&d, bytes));
     cudaError_t ce = launch_latent_read(latent_pool(layer), seq, len, d, stream_);
@@ -261,6 +295,7 @@ int Engine::latent_view(int seq, int layer, float* out) {
 }
 
 int Engine::save_state(int seq) {
+    if (state_) HM_CUDA(cudaMemcpyAsync(state_saved_, state_ + seq * state_floats_, state_floats_ * 4, cudaMemcpyDeviceToDevice, stream_));
     if (!shift_state_) return HM_OK;
     const size_t row = (size_t)SHIFT_RING * H_ * 4;
     HM_CUDA(cudaMemcpy2DAsync(shift_saved_, row, reinterpret_cast<char*>(shift_state_) + seq * row, batch_ * row, row, L_, cudaMemcpyDeviceToDevice, stream_));
@@ -272,13 +307,14 @@ int Engine::save_state(int seq) {
 int Engine::rewind(int seq, int len, const std::vector<uint32_t>& fed) {
     const int target = len + (int)fed.size();
     if (len_[seq] == target) return HM_OK;
-    if (!shift_state_) {
+    if (!shift_state_ && !state_) {
         len_[seq] = target;
         HM_CUDA(cudaMemcpy(pos_dev_ + seq, &len_[seq], 4, cudaMemcpyHostToDevice));
         return HM_OK;
     }
     const size_t row = (size_t)SHIFT_RING * H_ * 4;
-    HM_CUDA(cudaMemcpy2DAsync(reinterpret_cast<char*>(shift_state_) + seq * row, batch_ * row, shift_saved_, row, row, L_, cudaMemcpyDeviceToDevice, stream_));
+    if (state_) HM_CUDA(cudaMemcpyAsync(state_ + seq * state_floats_, state_saved_, state_floats_ * 4, cudaMemcpyDeviceToDevice, stream_));
+    if (shift_state_) HM_CUDA(cudaMemcpy2DAsync(reinterpret_cast<char*>(shift_state_) + seq * row, batch_ * row, shift_saved_, row, row, L_, cudaMemcpyDeviceToDevice, stream_));
     HM_CUDA(cudaStreamSynchronize(stream_));
     HM_CUDA(cudaMemcpy(pos_dev_ + seq, &len, 4, cudaMemcpyHostToDevice));
     for (uint32_t t : fed) {
@@ -319,6 +355,47 @@ int Engine::enqueue_tc(const LinearW& L, int M, const unsigned char* xp, int epi
     const cudaError_t ce = launch_gemm_tc(a, stream_, pdl_);
     if (ce != cudaSuccess) return cuda_fail(ce, "tensor-core projection launch");
     ++*launches;
+    return HM_OK;
+}
+
+// Attention of layer l over the queries in latent space (qlat_) into ctx_ or, many rows, its images; pass_nsplit_ splits are left to the next projection.
+int Engine::enqueue_latent_attn(int l, int M, bool tall, const int32_t* row_pos, const int32_t* row_seq, int* launches) {
+    const LayerSpec& s = spec_.layers[l];
+    const int rank = s.latent_rank(), lat = s.heads * rank;
+    LatentAttnArgs a{};
+    a.pool = latent_pool(l);
+    a.q = qlat_;
+    a.ldq = lat;
+    a.M = M;
+    a.heads = s.heads;
+    a.row_pos = row_pos;
+    a.row_seq = row_seq;
+    a.scale = s.scale;
+    const size_t per = (size_t)M * s.heads;
+    const int most = (int)std::min<size_t>(std::min(lat_acc_floats_ / (per * rank), lat_ml_floats_ / (per * 2)), 256);
+    // tiles: every run is cut at the multiples of the rows that share a CTA
+    int longest_run = 1, tiles = 0;
+    for (auto& r : pass_runs_) longest_run = std::max(longest_run, r.second);
+    a.rows_per_tile = latent_rows_per_tile(longest_run, pass_longest_, s.heads, rank, kv_bf16_);
+    for (auto& r : pass_runs_) tiles += (r.first + r.second - 1) / a.rows_per_tile - r.first / a.rows_per_tile + 1;
+    if (a.rows_per_tile == 1) tiles = M;
+    a.tiles = tiles;
+    a.unmerged = !tall && rank % 4 == 0 ? 1 : 0;
+    a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
+    a.nsplit = latent_pick_nsplit(tiles, a.rows_per_tile, s.heads, rank, kv_bf16_, pass_longest_, sm_count_, most, a.unmerged != 0);
+    pass_nsplit_ = a.unmerged ? a.nsplit : 1;
+    a.part_acc = lat_acc_;
+    a.part_ml = lat_ml_;
+    a.out = ctx_;
+    a.ldo = lat;
+    if (tall) {
+        a.xp = xpack_ctx_;
+        a.xp_mpad = tc_mpad(M);
+        a.xp_bytes = tc_xpack_bytes(M, rank);
+    }
+    a.err_flag = err_flag_;
+    const cudaError_t ce = launch_latent_attn(a, stream_, pdl_, launches);
+    if (ce != cudaSuccess) return cuda_fail(ce, "latent attention launch");
     return HM_OK;
 }
 
@@ -397,40 +474,8 @@ int Engine::enqueue_listed_layer(int l, int M, const int32_t* row_pos, const int
         if (rc) return rc;
     }
     if (want(PC_ATTN)) {
-        LatentAttnArgs a{};
-        a.pool = latent_pool(l);
-        a.q = qlat_;
-        a.ldq = lat;
-        a.M = M;
-        a.heads = s.heads;
-        a.row_pos = row_pos;
-        a.row_seq = row_seq;
-        a.scale = s.scale;
-        const size_t per = (size_t)M * s.heads;
-        const int most = (int)std::min<size_t>(std::min(lat_acc_floats_ / (per * s.kv_rank), lat_ml_floats_ / (per * 2)), 256);
-        // tiles: every run is cut at the multiples of the rows that share a CTA
-        int longest_run = 1, tiles = 0;
-        for (auto& r : pass_runs_) longest_run = std::max(longest_run, r.second);
-        a.rows_per_tile = latent_rows_per_tile(longest_run, pass_longest_, s.heads, s.kv_rank, kv_bf16_);
-        for (auto& r : pass_runs_) tiles += (r.first + r.second - 1) / a.rows_per_tile - r.first / a.rows_per_tile + 1;
-        if (a.rows_per_tile == 1) tiles = M;
-        a.tiles = tiles;
-        a.unmerged = !tall && s.kv_rank % 4 == 0 ? 1 : 0;
-        a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
-        a.nsplit = latent_pick_nsplit(tiles, a.rows_per_tile, s.heads, s.kv_rank, kv_bf16_, pass_longest_, sm_count_, most, a.unmerged != 0);
-        pass_nsplit_ = a.unmerged ? a.nsplit : 1;
-        a.part_acc = lat_acc_;
-        a.part_ml = lat_ml_;
-        a.out = ctx_;
-        a.ldo = lat;
-        if (tall) {
-            a.xp = xpack_ctx_;
-            a.xp_mpad = tc_mpad(M);
-            a.xp_bytes = tc_xpack_bytes(M, s.kv_rank);
-        }
-        a.err_flag = err_flag_;
-        ce = launch_latent_attn(a, stream_, pdl_, launches);
-        if (ce != cudaSuccess) return cuda_fail(ce, "latent attention launch");
+        rc = enqueue_latent_attn(l, M, tall, row_pos, row_seq, launches);
+        if (rc) return rc;
     }
     if (want(PC_VUP)) {
         if (tall) {
@@ -512,10 +557,12 @@ int Engine::enqueue_listed_logits(const float* x, int rows, float* dst, const Ar
         TcArgs a{};
         a.amax_val = amax_val_;
         a.amax_idx = amax_idx_;
+        a.softcap = spec_.softcap;
         return enqueue_tc(lm_head_, rows, xpack_, EPI_LOGITS, dst, V_, a, launches);
     }
     LinOpt o;
     o.gn = gn;
+    o.softcap = spec_.softcap;
     return enqueue_linear(lm_head_, rows, x, H_, PRO_GNORM, final_norm_, EPI_LOGITS, dst, V_, nullptr, nullptr, -1, nullptr, nullptr, amax_val_, amax_idx_, launches, &fold, &o);
 }
 

@@ -266,7 +266,7 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                 const float rw = ld_cg_f32(a.ex.weight + (size_t)m * a.ex.n + e);
                 float act[8];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) act[i] = rw == 0.f ? 0.f : clamped_glu(tile[m * BM + c + i], tile[m * BM + 64 + c + i], a.ex.limit) * rw;
+                for (int i = 0; i < 8; ++i) act[i] = rw == 0.f ? 0.f : glu(a.ex.act, tile[m * BM + c + i], tile[m * BM + 64 + c + i], a.ex.limit) * rw;
                 tc_xpack_store8(a.xp_out + (size_t)e * a.ex.img_bytes, a.xp_mpad, m, k0 + c, act);
             }
             return;
@@ -282,7 +282,7 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
     const int lane = tid & 31, warp = tid >> 5;
     constexpr int NW = TC_THREADS / 32;
     if (a.epi == EPI_STORE) {
-        const bool vec = (a.ldy & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.resid) | reinterpret_cast<uintptr_t>(a.bias)) & 15) == 0 && n0 + BM <= n_end && (!X || ((n0 & 3) == 0 && (reinterpret_cast<uintptr_t>(a.out_scale) & 15) == 0));
+        const bool vec = (a.ldy & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.resid) | reinterpret_cast<uintptr_t>(a.bias)) & 15) == 0 && n0 + BM <= n_end && (!X || ((n0 & (a.split_xp ? 7 : 3)) == 0 && (reinterpret_cast<uintptr_t>(a.out_scale) & 15) == 0));
         if (vec) {
             // eight consecutive features per thread (one 16-byte chunk of the next GEMM's activation image); the 16
             // threads of a row are half a warp, which is where the row's sum of squares is reduced
@@ -301,6 +301,9 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                         const float4 s0 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c)), s1 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c + 4));
                         v[0] *= s0.x; v[1] *= s0.y; v[2] *= s0.z; v[3] *= s0.w; v[4] *= s1.x; v[5] *= s1.y; v[6] *= s1.z; v[7] *= s1.w;
                     }
+                    if (a.turn.turns && ok)
+#pragma unroll
+                        for (int e = 0; e < 8; e += 2) turn_pair(a.turn, m, n0 + c + e, v[e], v[e + 1]);
                     if (a.split_xp && n0 + c < a.split_n) {  // 8-element pieces never straddle split_n or an image: both are multiples of 8
                         if (ok) tc_xpack_store8(a.split_xp + (size_t)((n0 + c) / a.split_k) * a.split_bytes, a.xp_mpad, m, (n0 + c) % a.split_k, v);
                         continue;
@@ -342,6 +345,15 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                     if (a.bias) v += __ldg(a.bias + n);
                     if constexpr (X) {
                         if (a.out_scale) v *= __ldg(a.out_scale + n);
+                        if (a.turn.turns) {  // (columns are padded to whole periods, so a pair is in the same block)
+                            float o = tile[m * BM + (c ^ 1)], u = v;
+                            if (c & 1) {
+                                turn_pair(a.turn, m, n - 1, o, u);
+                            } else {
+                                turn_pair(a.turn, m, n, u, o);
+                            }
+                            v = u;
+                        }
                         if (a.split_xp && n < a.split_n) {
                             tc_xpack_store(a.split_xp + (size_t)(n / a.split_k) * a.split_bytes, a.xp_mpad, m, n % a.split_k, v);
                             continue;
@@ -409,6 +421,12 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
             }
         }
     } else if (a.epi == EPI_LOGITS) {
+        if constexpr (X) {
+            if (a.softcap > 0.f) {
+                for (int idx = tid; idx < rows * BM; idx += TC_THREADS) tile[m_lo * BM + idx] = a.softcap * tanhf(tile[m_lo * BM + idx] / a.softcap);
+                __syncthreads();
+            }
+        }
         for (int idx = tid; idx < rows * BM; idx += TC_THREADS) {
             const int m = m_lo + idx / BM, c = idx % BM, n = n0 + c;
             if (n < a.N) a.y[(size_t)m * a.ldy + n] = tile[m * BM + c];
@@ -897,37 +915,37 @@ static cudaError_t launch_gemm_tc_v(const TcArgs& a_in, cudaStream_t st, bool pd
 }
 
 cudaError_t launch_gemm_tc(const TcArgs& a, cudaStream_t st, bool pdl) {
-    const bool x = a.group_blocks || a.out_scale || a.split_xp || a.epi == EPI_GATE || a.epi == EPI_SQRELU;
+    const bool x = a.group_blocks || a.out_scale || a.split_xp || a.turn.turns || a.softcap > 0.f || a.epi == EPI_GATE || a.epi == EPI_SQRELU;
     if (a.ex.n) return launch_gemm_tc_v<2>(a, st, pdl);
     return x ? launch_gemm_tc_v<1>(a, st, pdl) : launch_gemm_tc_v<0>(a, st, pdl);
 }
 
 // ---- weight packing: [N][K] (HF [out,in]) or [K][N] bf16 -> swizzled K-major tiles ----------
 namespace {
-__global__ void pack_tc_kernel(const uint16_t* __restrict__ src, int N, int K, int src_is_kn, uint16_t* __restrict__ dst, int n_off, int interleave_which) {
-    const int kb_total = (K + BK - 1) / BK;
-    const size_t total = (size_t)N * kb_total * BK;
+__global__ void pack_tc_kernel(const uint16_t* __restrict__ src, int N, int K, int src_is_kn, uint16_t* __restrict__ dst, int n_off, int interleave_which, int k_total, int k_off) {
+    const int kb_n = (K + BK - 1) / BK, kb_total = (k_total + BK - 1) / BK;
+    const size_t total = (size_t)N * kb_n * BK;
     for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
         const int kk = (int)(i % BK);
-        const int kb = (int)((i / BK) % kb_total);
-        const int n = (int)(i / ((size_t)BK * kb_total));
+        const int kb = (int)((i / BK) % kb_n);
+        const int n = (int)(i / ((size_t)BK * kb_n));
         const int k = kb * BK + kk;
         const uint16_t v = k < K ? (src_is_kn ? src[(size_t)k * N + n] : src[(size_t)n * K + k]) : (uint16_t)0;
         const int no = interleave_which >= 0 ? (n / 64) * BM + interleave_which * 64 + (n % 64) : n + n_off;
         const int nb = no / BM, row = no % BM;
         const int chunk = kk >> 3, e = kk & 7;
-        const size_t tile = ((size_t)nb * kb_total + kb) * (BM * BK);
+        const size_t tile = ((size_t)nb * kb_total + k_off / BK + kb) * (BM * BK);
         dst[tile + (size_t)row * BK + (size_t)((chunk ^ (row & 7)) << 3) + e] = v;
     }
 }
 }  // namespace
 
-cudaError_t launch_pack_tc(const uint16_t* src, int N, int K, bool src_is_kn, uint16_t* dst, int n_off, int interleave_which, cudaStream_t st) {
+cudaError_t launch_pack_tc(const uint16_t* src, int N, int K, bool src_is_kn, uint16_t* dst, int n_off, int interleave_which, cudaStream_t st, int k_total, int k_off) {
     const size_t total = (size_t)N * ((K + BK - 1) / BK) * BK;
     size_t g = (total + 255) / 256;
     if (g > 148 * 32) g = 148 * 32;
     if (g < 1) g = 1;
-    pack_tc_kernel<<<(unsigned)g, 256, 0, st>>>(src, N, K, src_is_kn ? 1 : 0, dst, n_off, interleave_which);
+    pack_tc_kernel<<<(unsigned)g, 256, 0, st>>>(src, N, K, src_is_kn ? 1 : 0, dst, n_off, interleave_which, k_total > 0 ? k_total : K, k_off);
     return cudaGetLastError();
 }
 

@@ -21,6 +21,7 @@ struct TcExperts {
     const float* weight;    // [M][n]
     const uint32_t* mask;   // [M][ceil(n / 32)] chosen experts
     float limit;
+    int act;                // GluAct
     size_t img_bytes;
     int parts;
     size_t part_stride;
@@ -51,6 +52,8 @@ struct TcArgs {
     unsigned char* split_xp;
     int split_n, split_k;
     size_t split_bytes;
+    TurnedPairs turn;        // EPI_STORE: with turn.turns
+    float softcap;           // EPI_LOGITS: > 0: softcap * tanh(logit / softcap)
     TcExperts ex;
     unsigned char* xp_out;   // EPI_SWIGLU, EPI_GATE, EPI_EXPERT and EPI_SQRELU, optional: write the result as packed activations for the next GEMM instead of y
     int xp_mpad;
@@ -89,8 +92,9 @@ cudaError_t launch_tc_pack_x(const float* x, int ldx, int M, int K, const float*
 // The same image of rows normalised in groups and token-shifted (RowNorm; runs of any length up to M).
 cudaError_t launch_tc_pack_gnorm(const float* x, int ldx, int M, int K, const float* norm_w, float eps, const RowNorm& gn, void* xp, cudaStream_t st, bool pdl);
 cudaError_t launch_gemm_tc(const TcArgs& a, cudaStream_t st, bool pdl);
+// k_total > 0: the matrix covers inputs [k_off, k_off + K) of a projection over k_total inputs, k_off a multiple of 64.
 // src is [N][K] (src_is_kn = false) or [K][N]; rows land at n_off + n, or interleaved 64/64 per
 // 128-row block when interleave_which is 0 (gate) or 1 (up).
-cudaError_t launch_pack_tc(const uint16_t* src, int N, int K, bool src_is_kn, uint16_t* dst, int n_off, int interleave_which, cudaStream_t st);
+cudaError_t launch_pack_tc(const uint16_t* src, int N, int K, bool src_is_kn, uint16_t* dst, int n_off, int interleave_which, cudaStream_t st, int k_total = 0, int k_off = 0);
 
 }  // namespace hm

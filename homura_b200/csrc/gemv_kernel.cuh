@@ -573,6 +573,17 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
     // ---- epilogues on vals[M][128] (columns n0 .. n0+127 of the output) ----
     bool stored = false;
     if constexpr (X) {
+        if (a.epi == EPI_LOGITS && a.softcap > 0.f) {
+            for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) vals[idx] = a.softcap * tanhf(vals[idx] / a.softcap);
+            __syncthreads();
+        }
+        if (a.turn.turns) {  // pairs never straddle a slab
+            for (int idx = tid; idx < M * SLAB / 2; idx += GEMV_THREADS) {
+                const int m = idx / (SLAB / 2), c = idx % (SLAB / 2) * 2;
+                if (n0 + c < n_end && m < a.m_valid) turn_pair(a.turn, m, n0 + c, vals[m * SLAB + c], vals[m * SLAB + c + 1]);
+            }
+            __syncthreads();
+        }
         if (a.epi == EPI_GATE) {
             for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) {
                 const int m = idx / SLAB, n = n0 + (idx % SLAB);

@@ -19,6 +19,7 @@
 #include <mutex>
 #include <tuple>
 
+#include "gqa_post.cuh"
 #include "launch_attrs.h"
 #include "mbarrier.cuh"
 #include "model_spec.h"
@@ -26,7 +27,6 @@
 namespace hm {
 namespace {
 
-constexpr int POST_WARPS = 8;
 constexpr int ATT_WARPS = 8;
 constexpr int A_THREADS = 256;
 constexpr int B_THREADS = ATT_WARPS * 32 + 32;
@@ -34,96 +34,10 @@ constexpr int MAX_STAGES = 8;
 constexpr int MAX_CLUSTER = 16;
 
 // ---- after the projection ------------------------------------------------------------------------
-// One warp per head (queries, then keys, then values); with a norm over the whole projection every CTA sums the squares of the part
-// it needs.
 __global__ void __launch_bounds__(POST_WARPS * 32) gqa_post_kernel(const GqaPostArgs a) {
+    extern __shared__ __align__(16) float post_sm[];
     pdl_launch_dependents();
-    const int m = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
-    const int slot0 = blockIdx.y * POST_WARPS, slot = slot0 + warp;  // head slots: [heads] queries, [G] keys, [G] values
-    const int pos = a.row_pos[m], seq = a.row_seq[m];
-    const size_t page = (size_t)a.pool.page_table[(size_t)seq * a.pool.max_pages + pos / GQA_PAGE];
-    const int t = pos % GQA_PAGE;
-    __shared__ float s_part[2][POST_WARPS];
-    pdl_wait();
-    const float* raw = a.raw + (size_t)m * a.ld;
-    if (a.qk_norm == QKN_ALL) {
-        float sq = 0.f, sk = 0.f;
-        if (slot0 < a.heads)
-#pragma unroll 4
-            for (int i = tid; i < nq; i += POST_WARPS * 32) {
-                const float v = ld_cg_f32(raw + i);
-                sq = fmaf(v, v, sq);
-            }
-        if (slot0 < a.heads + G && slot0 + POST_WARPS > a.heads)
-#pragma unroll 4
-            for (int i = tid; i < nk; i += POST_WARPS * 32) {
-                const float v = ld_cg_f32(raw + nq + i);
-                sk = fmaf(v, v, sk);
-            }
-        sq = warp_sum(sq);
-        sk = warp_sum(sk);
-        if (lane == 0) {
-            s_part[0][warp] = sq;
-            s_part[1][warp] = sk;
-        }
-        __syncthreads();
-    }
-    if (slot >= a.heads + 2 * G) return;
-    if (slot < a.heads + G) {
-        const bool is_q = slot < a.heads;
-        const int h = is_q ? slot : slot - a.heads;
-        const float* x = raw + (is_q ? 0 : nq) + (size_t)h * dim;
-        float inv = 1.f;
-        if (a.qk_norm == QKN_ALL) {
-            float s = 0.f;
-#pragma unroll
-            for (int w = 0; w < POST_WARPS; ++w) s += s_part[is_q ? 0 : 1][w];
-            inv = 1.0f / sqrtf(s / (float)(is_q ? nq : nk) + a.eps);
-        } else if (a.qk_norm == QKN_HEAD) {
-            float s = 0.f;
-#pragma unroll 4
-            for (int d = lane; d < dim; d += 32) {
-                const float v = ld_cg_f32(x + d);
-                s = fmaf(v, v, s);
-            }
-            inv = 1.0f / sqrtf(warp_sum(s) / (float)dim + a.eps);
-        }
-        const float* w = a.qk_norm == QKN_NONE ? nullptr : (is_q ? a.q_norm : a.k_norm) + (a.qk_norm == QKN_ALL ? (size_t)h * dim : 0);
-        if (is_q) {
-            float f = 1.f;
-            if (a.temp_every > 0) f = 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
-            float* o = a.q_out + (size_t)m * nq + (size_t)h * dim;
-            for (int d = lane; d < dim; d += 32) {
-                const float v = w ? (ld_cg_f32(x + d) * inv) * __ldg(w + d) : ld_cg_f32(x + d);
-                o[d] = (v * f) * a.q_scale;
-            }
-        } else {
-            const size_t base = page * gqa_page_elems(G, dim) + (size_t)h * GQA_PAGE * gqa_pad(dim);
-            for (int d = lane; d < dim; d += 32) {
-                const float v = w ? (ld_cg_f32(x + d) * inv) * __ldg(w + d) : ld_cg_f32(x + d);
-                const size_t off = base + gqa_tile_off(t, d);
-                if (a.pool.bf16) reinterpret_cast<uint16_t*>(a.pool.k)[off] = f32_to_bf16_rne(v);
-                else reinterpret_cast<float*>(a.pool.k)[off] = v;
-            }
-        }
-    } else {
-        const int h = slot - a.heads - G;
-        const float* x = raw + nq + nk + (size_t)h * vdim;
-        float* first = a.v_first ? a.v_first + (size_t)m * G * vdim + (size_t)h * vdim : nullptr;
-        const float lam = first && a.v_lambda ? __ldg(a.v_lambda) : 0.f;
-        const size_t base = page * gqa_page_elems(G, vdim) + (size_t)h * GQA_PAGE * gqa_pad(vdim);
-        for (int d = lane; d < vdim; d += 32) {
-            float v = ld_cg_f32(x + d);
-            if (first) {
-                if (a.v_lambda) v = (1.0f - lam) * v + lam * ld_cg_f32(first + d);
-                else first[d] = v;
-            }
-            const size_t off = base + gqa_tile_off(t, d);
-            if (a.pool.bf16) reinterpret_cast<uint16_t*>(a.pool.v)[off] = f32_to_bf16_rne(v);
-            else reinterpret_cast<float*>(a.pool.v)[off] = v;
-        }
-    }
+    gqa_post_block(a, blockIdx.x, blockIdx.y, post_sm);
 }
 
 __global__ void gqa_read_kernel(const GqaPool pool, int seq, int len, float* __restrict__ k, float* __restrict__ v) {
@@ -140,9 +54,18 @@ __global__ void gqa_read_kernel(const GqaPool pool, int seq, int len, float* __r
 }
 
 // ---- common to both attention kernels --------------------------------------------------------------
-__device__ __forceinline__ void store_piece(const GqaAttnArgs& a, int m, int head, int d0, const float (&v)[8]) {
-    const int vdim = a.pool.vdim, k0 = head * vdim + d0;
-    if (a.xp && (vdim & 7) == 0) {
+__device__ __forceinline__ void store_piece(const GqaAttnArgs& a, int m, int head, int d0, float (&v)[8]) {
+    const int vdim = a.pool.vdim, e0 = head * vdim + d0, k0 = a.out_off + e0;
+    if (a.gate_kind != GATE_NONE) {
+        const float* g = a.gate + (size_t)m * a.ld_gate;
+        const float all = a.gate_kind == GATE_HEAD ? 1.0f / (1.0f + expf(-ld_cg_f32(g + head))) : 1.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] *= a.gate_kind == GATE_HEAD ? all : d0 + i < vdim ? 1.0f / (1.0f + expf(-ld_cg_f32(g + e0 + i))) : 0.f;
+    }
+    if (a.out_scale != 0.f)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] *= a.out_scale;
+    if (a.xp && ((vdim | a.out_off) & 7) == 0) {
         tc_xpack_store8(a.xp, a.xp_mpad, m, k0, v);
         return;
     }
@@ -150,8 +73,29 @@ __device__ __forceinline__ void store_piece(const GqaAttnArgs& a, int m, int hea
     for (int i = 0; i < 8; ++i) {
         if (d0 + i >= vdim) break;
         if (a.xp) tc_xpack_store(a.xp, a.xp_mpad, m, k0 + i, v[i]);
-        else a.out[(size_t)m * a.heads * vdim + k0 + i] = v[i];
+        else a.out[(size_t)m * a.ld_out + k0 + i] = v[i];
     }
+}
+
+// The sink's share of a denominator whose weights are relative to 2^mx.
+__device__ __forceinline__ float sink_weight(const GqaAttnArgs& a, int head, float mx) { return a.sink ? exp2f(fmaf(__ldg(a.sink + head), 1.4426950408889634f, -mx)) : 0.f; }
+
+// Pages that rows at positions [lo, hi] see: those of the first tokens, then those of the window.  Page number i of the list is
+// pages_skip(i): i itself in front of the gap, i + gap behind it.
+struct PageList {
+    int n, head, gap;
+    __device__ __forceinline__ int page(int i) const { return i < head ? i : i + gap; }
+};
+__device__ __forceinline__ PageList visible_pages(const GqaAttnArgs& a, int lo, int hi) {
+    const int all = hi / GQA_PAGE + 1;
+    PageList l{all, all, 0};
+    if (a.window > 0) {
+        const int from = max(0, lo - a.window + 1) / GQA_PAGE;  // first page of the window
+        l.head = min((a.keep_first + GQA_PAGE - 1) / GQA_PAGE, from);
+        l.gap = from - l.head;
+        l.n = all - l.gap;
+    }
+    return l;
 }
 
 // Results of a CTA's pairs in its shared memory: o [pairs][ldo] (not yet divided), ml [pairs][2] (maximum as a base-2 exponent, sum).
@@ -163,8 +107,10 @@ __device__ __forceinline__ void combine_and_store(const GqaAttnArgs& a, const fl
     if (ns > 1) cluster_sync_all();
     else __syncthreads();
     for (int p = tid; p < pairs; p += nt) {
+        int sm_row, sm_head;
+        row_head(p, sm_row, sm_head);
         if (ns == 1) {
-            wts[p] = 1.0f / ml[2 * p + 1];
+            wts[p] = 1.0f / (ml[2 * p + 1] + sink_weight(a, sm_head, ml[2 * p]));
             continue;
         }
         float mr[MAX_CLUSTER], lr[MAX_CLUSTER], mx = -INFINITY, l = 0.f;
@@ -183,6 +129,7 @@ __device__ __forceinline__ void combine_and_store(const GqaAttnArgs& a, const fl
                 mr[r] = mr[r] == -INFINITY ? 0.f : exp2f(mr[r] - mx);
                 l = fmaf(mr[r], lr[r], l);
             }
+        l += sink_weight(a, sm_head, mx);
 #pragma unroll
         for (int r = 0; r < MAX_CLUSTER; ++r)
             if (r < ns) wts[r * pairs + p] = mr[r] / l;
@@ -228,8 +175,9 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
     float* wts = corr + g;            // [nsplit][g]
     pdl_launch_dependents();
     pdl_wait();
-    const int pos = a.row_pos[m], len = pos + 1, npages = (len + GQA_PAGE - 1) / GQA_PAGE, pps = (npages + a.nsplit - 1) / a.nsplit;
-    const int p0 = split * pps, p1 = min(npages, p0 + pps);
+    const int pos = a.row_pos[m], len = pos + 1;
+    const PageList list = visible_pages(a, pos, pos);
+    const int pps = (list.n + a.nsplit - 1) / a.nsplit, p0 = split * pps, p1 = min(list.n, p0 + pps);
     const int32_t* pt = a.pool.page_table + (size_t)a.row_seq[m] * a.pool.max_pages;
     for (int i = tid; i < g * dp; i += A_THREADS) {
         const int j = i / dp, d = i - j * dp;
@@ -241,14 +189,15 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
         ml[2 * i + 1] = 0.f;
     }
     __syncthreads();
-    for (int p = p0; p < p1; ++p) {
+    for (int pi = p0; pi < p1; ++pi) {
+        const int p = list.page(pi);
         const size_t kb = (size_t)pt[p] * gqa_page_elems(a.pool.kv_heads, dim) + (size_t)kvh * GQA_PAGE * dp;
         const size_t vb = (size_t)pt[p] * gqa_page_elems(a.pool.kv_heads, vdim) + (size_t)kvh * GQA_PAGE * vp;
         const int nt = min(GQA_PAGE, len - p * GQA_PAGE);
         for (int i = tid; i < g * GQA_PAGE; i += A_THREADS) {
             const int j = i / GQA_PAGE, t = i % GQA_PAGE;
             float s = -INFINITY;
-            if (t < nt) {
+            if (t < nt && (a.window == 0 || pos - (p * GQA_PAGE + t) < a.window || p * GQA_PAGE + t < a.keep_first)) {
                 const float* q = q_s + j * dp;
                 s = 0.f;
                 for (int c = 0; c < dp / 8; ++c) {
@@ -272,7 +221,7 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
         __syncthreads();
         for (int j = warp; j < g; j += A_THREADS / 32) {
             const float s0 = p_s[j * GQA_PAGE + lane], s1 = p_s[j * GQA_PAGE + 32 + lane];
-            const float old = ml[2 * j], mx = fmaxf(old, warp_max(fmaxf(s0, s1)));  // a page of a split has a token
+            const float old = ml[2 * j], mx = fmaxf(old, warp_max(fmaxf(s0, s1)));  // a page of the list has a token that is seen
             const float e0 = exp2f(s0 - mx), e1 = exp2f(s1 - mx), f = exp2f(old - mx);
             p_s[j * GQA_PAGE + lane] = e0;
             p_s[j * GQA_PAGE + 32 + lane] = e1;
@@ -379,10 +328,12 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
     if (!a.early) pdl_wait();
     const int row_hi = row0 + (pair0 + pairs - 1) / g;
     const int seq = a.row_seq[row0], len = a.row_pos[row_hi] + 1;
-    const int npages = (len + GQA_PAGE - 1) / GQA_PAGE, pps = (npages + a.nsplit - 1) / a.nsplit;
-    const int p0 = split * pps, np = max(0, min(npages, p0 + pps) - p0);
-    const int32_t* pt = a.pool.page_table + (size_t)seq * a.pool.max_pages + p0;
-    for (int i = tid; i < np; i += B_THREADS) pt_s[i] = pt[i];
+    const PageList list = visible_pages(a, a.window > 0 ? a.row_pos[row0 + pair0 / g] : 0, len - 1);
+    const int pps = (list.n + a.nsplit - 1) / a.nsplit;
+    const int p0 = split * pps, np = max(0, min(list.n, p0 + pps) - p0);
+    const int32_t* pt = a.pool.page_table + (size_t)seq * a.pool.max_pages;
+    for (int i = tid; i < np; i += B_THREADS) pt_s[i] = pt[list.page(p0 + i)];
+    const int seen = a.window > 0 ? a.window : 0x7fffffff;
     if (tid < P) {
         const int pr = pair0 + tid;
         s_pos[tid] = tid < pairs ? a.row_pos[row0 + pr / g] : -1;
@@ -400,7 +351,7 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
     int n_pre = 0;
     if (a.early) {
         if (tid == ATT_WARPS * 32)
-            for (; n_pre < np && n_pre < NST && p0 + n_pre < (len - 1) / GQA_PAGE; ++n_pre) fetch(n_pre, n_pre);
+            for (; n_pre < np && n_pre < NST && list.page(p0 + n_pre) < (len - 1) / GQA_PAGE; ++n_pre) fetch(n_pre, n_pre);
         pdl_wait();
     }
     if (warp == ATT_WARPS) {
@@ -459,7 +410,7 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
         for (int i = warp >> 2; i < np; i += 2) {
             const int s = i % NST;
             if (!__all_sync(0xffffffffu, mb_wait(&full[s], (i / NST) & 1u, a.err_flag, &s_abort))) break;
-            const int tok = (p0 + i) * GQA_PAGE + u * 16;
+            const int tok = list.page(p0 + i) * GQA_PAGE + u * 16;
             if (tok < len) {
                 const uint32_t kb = s32(ring + (size_t)s * stage) + k_lane, vb = s32(ring + (size_t)s * stage + k_bytes) + v_lane;
                 constexpr int CH = NT == 1 ? 3 : 1;  // a lone tile of pairs: one accumulator per term, or its MMAs would wait for one another
@@ -497,8 +448,8 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
                             s0 += __ldg(a.bias + brow[nt][hh] + min(max(n0, 0), a.reach));
                             s1 += __ldg(a.bias + brow[nt][hh] + min(max(n1, 0), a.reach));
                         }
-                        s0 = n0 >= 0 ? s0 : -INFINITY;
-                        s1 = n1 >= 0 ? s1 : -INFINITY;
+                        s0 = n0 >= 0 && (n0 < seen || t0 < a.keep_first) ? s0 : -INFINITY;
+                        s1 = n1 >= 0 && (n1 < seen || t1 < a.keep_first) ? s1 : -INFINITY;
                         float mx = fmaxf(s0, s1);
 #pragma unroll
                         for (int o = 4; o < 32; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -621,7 +572,7 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
             v[0] = fmaf(f, x.x, v[0]); v[1] = fmaf(f, x.y, v[1]); v[2] = fmaf(f, x.z, v[2]); v[3] = fmaf(f, x.w, v[3]);
             v[4] = fmaf(f, y.x, v[4]); v[5] = fmaf(f, y.y, v[5]); v[6] = fmaf(f, y.z, v[6]); v[7] = fmaf(f, y.w, v[7]);
         }
-        const float inv = 1.0f / l;
+        const float inv = 1.0f / (l + sink_weight(a, kvh * g + (pair0 + p) % g, mx));
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[e] *= inv;
         if (d0 < vdim) store_piece(a, row0 + (pair0 + p) / g, kvh * g + (pair0 + p) % g, d0, v);
@@ -686,6 +637,15 @@ int clusters_at_once(void (*kern)(KArgs...), int cluster, int threads, size_t sm
     return known[key] = n;
 }
 
+// Pages that a tile of so many (row, head) pairs can see.
+int most_pages(const GqaAttnArgs& a, int pairs) {
+    const int all = (a.longest + GQA_PAGE - 1) / GQA_PAGE;
+    if (a.window == 0) return all;
+    const int rows = std::min(a.longest_run, (pairs + a.heads / a.pool.kv_heads - 1) / (a.heads / a.pool.kv_heads) + 1);
+    const long seen = (a.keep_first + GQA_PAGE - 1) / GQA_PAGE + ((long)a.window + rows - 2) / GQA_PAGE + 2;
+    return (int)std::min<long>(all, seen);
+}
+
 template <int VT, int NT>
 cudaError_t launch_mma(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
     constexpr int P = NT * 8;
@@ -701,7 +661,7 @@ cudaError_t launch_mma(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
         }
         a.runs.tile[a.runs.n] = (uint16_t)a.tiles;
     }
-    const int pages = (a.longest + GQA_PAGE - 1) / GQA_PAGE, pairs = a.tiles * a.pool.kv_heads;
+    const int pages = most_pages(a, P), pairs = a.tiles * a.pool.kv_heads;
     constexpr int PER_SM = NT == 1 && VT <= 8 ? 2 : 1;
     const size_t stage = b_stage_bytes(dp, vp);
     size_t ring = 0, fixed = 0;
@@ -739,23 +699,23 @@ cudaError_t launch_mma_n(const GqaAttnArgs& a, int sm_count, cudaStream_t st, bo
 }  // namespace
 
 cudaError_t launch_gqa_post(const GqaPostArgs& a, cudaStream_t st, bool pdl) {
-    const int slots = a.heads + 2 * a.pool.kv_heads;
-    return launch_clustered(gqa_post_kernel, dim3((unsigned)a.M, (unsigned)((slots + POST_WARPS - 1) / POST_WARPS)), dim3(POST_WARPS * 32), 0, 1, st, pdl, a);
+    return launch_clustered(gqa_post_kernel, dim3((unsigned)a.M, (unsigned)gqa_post_blocks(a)), dim3(POST_WARPS * 32), gqa_post_smem(a), 1, st, pdl, a);
 }
 
 cudaError_t launch_gqa_attn(const GqaAttnArgs& a_in, int sm_count, cudaStream_t st, bool pdl) {
     GqaAttnArgs a = a_in;
     if (a.M < 1 || a.M > GQA_MAX_ROWS || a.nsplit > MAX_CLUSTER || a.heads % a.pool.kv_heads != 0) return cudaErrorInvalidValue;
     if (!a.bias) a.reach = 0;
+    if (a.ld_out == 0) a.ld_out = a.heads * a.pool.vdim;
     const int g = a.heads / a.pool.kv_heads, dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
     if (a.runs.n == 0) a.longest_run = 1;
-    const long ppc_most = (a.longest + GQA_PAGE - 1) / GQA_PAGE;
+    const long ppc_most = most_pages(a, 32);
     if (a.pool.bf16 && vp <= 256 && dp <= 256 && ppc_most <= 8192) {
         if (vp <= 64) return launch_mma_n<4>(a, sm_count, st, pdl);
         if (vp <= 128) return launch_mma_n<8>(a, sm_count, st, pdl);
         return launch_mma_n<16>(a, sm_count, st, pdl);
     }
-    const int pages = (a.longest + GQA_PAGE - 1) / GQA_PAGE;
+    const int pages = most_pages(a, 1);
     if (a.nsplit < 1) a.nsplit = std::max(1, std::min({4 * sm_count / (a.M * a.pool.kv_heads), a.max_cluster, MAX_CLUSTER, pages}));
     const size_t smem = sizeof(float) * (size_t)g * (dp + vp + 4 + GQA_PAGE + 3 + a.nsplit);
     const dim3 grid((unsigned)a.nsplit, (unsigned)a.pool.kv_heads, (unsigned)a.M);

@@ -24,8 +24,31 @@ __host__ __device__ __forceinline__ int gqa_pad(int d) { return (d + 15) & ~15; 
 __host__ __device__ __forceinline__ size_t gqa_page_elems(int kv_heads, int d) { return (size_t)kv_heads * GQA_PAGE * gqa_pad(d); }
 __host__ __device__ __forceinline__ int gqa_tile_off(int t, int d) { return ((d >> 3) * GQA_PAGE + t) * 8 + (d & 7); }
 
-// What happens to a projection's queries, keys and values before the attention: norms, temperature, blended values; keys and values
-// go to their page slots, queries to q_out.
+// Rows as runs: consecutive positions of one sequence.
+struct GqaRuns {
+    int n = 0;                            // 0: every row is a run
+    uint8_t row[GQA_MAX_ROWS + 1];        // first row of every run; row[n] = rows of the pass
+    uint16_t tile[GQA_MAX_ROWS + 1];      // first tile of every run (filled in by the attention's launcher)
+    // The run of row m: [first, end).
+    __host__ __device__ __forceinline__ void find(int m, int& first, int& end) const {
+        if (n == 0) {
+            first = m;
+            end = m + 1;
+            return;
+        }
+        int lo = 0, hi = n;
+        while (hi - lo > 1) {
+            const int mid = (lo + hi) / 2;
+            if (row[mid] <= m) lo = mid;
+            else hi = mid;
+        }
+        first = row[lo];
+        end = row[lo + 1];
+    }
+};
+
+// What happens to a projection's queries, keys and values before the attention: a short convolution, norms, rotation, temperature,
+// blended values; keys and values go to their page slots, queries to q_out.
 struct GqaPostArgs {
     GqaPool pool;
     const float* raw;        // [M][ld]: queries | keys | values
@@ -40,15 +63,19 @@ struct GqaPostArgs {
     const float* v_lambda;   // null: this layer keeps its values in v_first
     const int32_t *row_pos, *row_seq;
     float* q_out;            // [M][heads * dim]
+    // Causal convolution over time of every channel (queries | keys | values), taps > 0: the inputs of the last taps - 1 tokens of a
+    // sequence are kept in conv_state, position p in slot p % (taps - 1).  The warp of a run's first row serves the first taps - 1 rows,
+    // so that nobody else reads what it replaces.
+    int taps;
+    const float* conv_w;     // [channels][taps], the last one meets the token itself
+    float* conv_state;       // [sequence][taps - 1][channels], sequences conv_stride floats apart
+    size_t conv_stride;
+    GqaRuns runs;            // with taps > 1
+    // rotation of the first rot_dims elements of queries and keys: pair (i, i + rot_dims / 2) makes turns[i] turns per position
+    int rot_dims;
+    const double* turns;
 };
 cudaError_t launch_gqa_post(const GqaPostArgs& a, cudaStream_t st, bool pdl);
-
-// Rows as runs: consecutive positions of one sequence, whose rows and heads share a CTA.
-struct GqaRuns {
-    int n = 0;                            // 0: every row is a run
-    uint8_t row[GQA_MAX_ROWS + 1];        // first row of every run; row[n] = rows of the pass
-    uint16_t tile[GQA_MAX_ROWS + 1];      // first tile of every run (filled in by the launcher)
-};
 
 struct GqaAttnArgs {
     GqaPool pool;
@@ -57,7 +84,13 @@ struct GqaAttnArgs {
     const int32_t *row_pos, *row_seq;  // a row sees the positions up to its own
     const float* bias;       // [heads][reach + 1] by distance (the last one for all beyond), times log2 e; or null
     int reach;
-    GqaRuns runs;
+    int window, keep_first;  // window > 0: a row at position p sees the positions above p - window and those below keep_first
+    const float* sink;       // [heads] or null: one more score in the denominator (not scaled, as it is in the softmax)
+    const float* gate;       // results are multiplied by the sigmoid of gate [M][ld_gate] (per element, or per head)
+    int ld_gate, gate_kind;  // OutGate
+    float out_scale;         // and by this (0: not)
+    int ld_out, out_off;     // row stride and first element of the results in `out` or the image (ld_out 0: heads * vdim)
+    GqaRuns runs;            // rows and heads of a run share a CTA
     int longest_run, longest;  // rows of the longest run, tokens of the longest context
     int early;               // every row is its own sequence and the pages in front of its newest token were complete before the launch in front began
     int max_cluster;

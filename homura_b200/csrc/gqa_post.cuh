@@ -1,0 +1,179 @@
+// What happens to the rows of a fused query / key / value projection before the attention (GqaPostArgs): one warp per row and head.
+#pragma once
+#include "gqa_attn.h"
+#include "model_spec.h"
+
+namespace hm {
+
+constexpr int POST_WARPS = 8;
+
+__host__ __device__ __forceinline__ int gqa_post_slots(const GqaPostArgs& a) { return a.heads + 2 * a.pool.kv_heads; }
+__host__ __device__ __forceinline__ int gqa_post_blocks(const GqaPostArgs& a) { return (gqa_post_slots(a) + POST_WARPS - 1) / POST_WARPS; }  // per row
+// a head's elements per warp, kept only where they are needed twice
+__host__ __device__ __forceinline__ int gqa_post_buf(const GqaPostArgs& a) { return a.taps > 0 || a.rot_dims > 0 || a.qk_norm == QKN_UNIT ? (a.pool.dim > a.pool.vdim ? a.pool.dim : a.pool.vdim) : 0; }
+__host__ __device__ __forceinline__ size_t gqa_post_smem(const GqaPostArgs& a) { return sizeof(float) * POST_WARPS * (size_t)gqa_post_buf(a); }
+
+// Rotates `half` pairs (buf[i], buf[i + half]) with the lanes of a warp.
+__device__ __forceinline__ void rotate_pairs(float* buf, int half, const double* turns, int pos, int lane) {
+    for (int i = lane; i < half; i += 32) {
+        float c, s;
+        rotation_at(__ldg(turns + i), pos, c, s);
+        const float u = buf[i], v = buf[i + half];
+        buf[i] = fmaf(u, c, -v * s);
+        buf[i + half] = fmaf(v, c, u * s);
+    }
+}
+
+// Row m of one head slot ([heads] queries, [kv_heads] keys, [kv_heads] values).  part_q / part_k: sums of squares of the whole
+// projections (QKN_ALL); first: the first row of m's run.
+__device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int slot, int first, float part_q, float part_k, float* buf) {
+    const int lane = threadIdx.x & 31;
+    const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
+    const int pos = a.row_pos[m], seq = a.row_seq[m], t = pos % GQA_PAGE;
+    const size_t page = (size_t)a.pool.page_table[(size_t)seq * a.pool.max_pages + pos / GQA_PAGE];
+    const bool is_v = slot >= a.heads + G, is_q = slot < a.heads;
+    const int h = is_v ? slot - a.heads - G : is_q ? slot : slot - a.heads, n = is_v ? vdim : dim;
+    const int ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n;  // first channel
+    const float* x = a.raw + (size_t)m * a.ld + ch0;
+    const bool buffered = gqa_post_buf(a) > 0;
+    if (buffered) {
+        const float* state = a.taps > 1 ? a.conv_state + (size_t)seq * a.conv_stride + ch0 : nullptr;
+        const int channels = nq + nk + G * vdim;
+        for (int d = lane; d < n; d += 32) {
+            float v = ld_cg_f32(x + d);
+            if (a.taps > 0) {
+                const float* w = a.conv_w + (size_t)(ch0 + d) * a.taps;
+                v *= __ldg(w + a.taps - 1);
+                for (int j = 1; j < a.taps; ++j) {
+                    if (j > pos) break;
+                    const float u = m - j >= first ? ld_cg_f32(x + d - (ptrdiff_t)j * a.ld) : ld_cg_f32(state + (size_t)((pos - j) % (a.taps - 1)) * channels + d);
+                    v = fmaf(u, __ldg(w + a.taps - 1 - j), v);
+                }
+            }
+            buf[d] = v;
+        }
+        __syncwarp();
+    }
+    auto at = [&](int d) { return buffered ? buf[d] : ld_cg_f32(x + d); };
+    if (!is_v) {
+        float inv = 1.f;
+        if (a.qk_norm == QKN_ALL) {
+            inv = 1.0f / sqrtf((is_q ? part_q : part_k) / (float)(is_q ? nq : nk) + a.eps);
+        } else if (a.qk_norm == QKN_HEAD) {
+            float s = 0.f;
+#pragma unroll 4
+            for (int d = lane; d < dim; d += 32) {
+                const float v = at(d);
+                s = fmaf(v, v, s);
+            }
+            inv = 1.0f / sqrtf(warp_sum(s) / (float)dim + a.eps);
+        }
+        const float* w = a.qk_norm == QKN_HEAD || a.qk_norm == QKN_ALL ? (is_q ? a.q_norm : a.k_norm) + (a.qk_norm == QKN_ALL ? (size_t)h * dim : 0) : nullptr;
+        auto normed = [&](int d) { return w ? (at(d) * inv) * __ldg(w + d) : at(d); };
+        float unit = 1.f;
+        const bool turned = a.rot_dims > 0;
+        if (turned || a.qk_norm == QKN_UNIT) {
+            if (w)
+                for (int d = lane; d < dim; d += 32) buf[d] = normed(d);
+            __syncwarp();
+            if (turned) rotate_pairs(buf, a.rot_dims / 2, a.turns, pos, lane);
+            __syncwarp();
+            if (a.qk_norm == QKN_UNIT) {
+                float s = 0.f;
+                for (int d = lane; d < dim; d += 32) s = fmaf(buf[d], buf[d], s);
+                unit = 1.0f / sqrtf(warp_sum(s) / (float)dim + a.eps);
+            }
+        }
+        auto value = [&](int d) { return turned || a.qk_norm == QKN_UNIT ? buf[d] * unit : normed(d); };
+        if (is_q) {
+            float f = 1.f;
+            if (a.temp_every > 0) f = 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
+            float* o = a.q_out + (size_t)m * nq + (size_t)h * dim;
+            for (int d = lane; d < dim; d += 32) o[d] = (value(d) * f) * a.q_scale;
+        } else {
+            const size_t base = page * gqa_page_elems(G, dim) + (size_t)h * GQA_PAGE * gqa_pad(dim);
+            for (int d = lane; d < dim; d += 32) {
+                const float v = value(d);
+                const size_t off = base + gqa_tile_off(t, d);
+                if (a.pool.bf16) reinterpret_cast<uint16_t*>(a.pool.k)[off] = f32_to_bf16_rne(v);
+                else reinterpret_cast<float*>(a.pool.k)[off] = v;
+            }
+        }
+    } else {
+        float* kept = a.v_first ? a.v_first + (size_t)m * G * vdim + (size_t)h * vdim : nullptr;
+        const float lam = kept && a.v_lambda ? __ldg(a.v_lambda) : 0.f;
+        const size_t base = page * gqa_page_elems(G, vdim) + (size_t)h * GQA_PAGE * gqa_pad(vdim);
+        for (int d = lane; d < vdim; d += 32) {
+            float v = at(d);
+            if (kept) {
+                if (a.v_lambda) v = (1.0f - lam) * v + lam * ld_cg_f32(kept + d);
+                else kept[d] = v;
+            }
+            const size_t off = base + gqa_tile_off(t, d);
+            if (a.pool.bf16) reinterpret_cast<uint16_t*>(a.pool.v)[off] = f32_to_bf16_rne(v);
+            else reinterpret_cast<float*>(a.pool.v)[off] = v;
+        }
+    }
+    __syncwarp();
+}
+
+// Row m and POST_WARPS head slots from blk * POST_WARPS on.
+__device__ __forceinline__ void gqa_post_block(const GqaPostArgs& a, int m, int blk, float* smem) {
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
+    const int slot0 = blk * POST_WARPS, slot = slot0 + warp;
+    __shared__ float s_part[2][POST_WARPS];
+    pdl_wait();
+    float sq = 0.f, sk = 0.f;
+    if (a.qk_norm == QKN_ALL) {  // every CTA sums the squares of the part it needs
+        const float* raw = a.raw + (size_t)m * a.ld;
+        if (slot0 < a.heads)
+#pragma unroll 4
+            for (int i = tid; i < nq; i += POST_WARPS * 32) {
+                const float v = ld_cg_f32(raw + i);
+                sq = fmaf(v, v, sq);
+            }
+        if (slot0 < a.heads + G && slot0 + POST_WARPS > a.heads)
+#pragma unroll 4
+            for (int i = tid; i < nk; i += POST_WARPS * 32) {
+                const float v = ld_cg_f32(raw + nq + i);
+                sk = fmaf(v, v, sk);
+            }
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        if (lane == 0) {
+            s_part[0][warp] = sq;
+            s_part[1][warp] = sk;
+        }
+        __syncthreads();
+        sq = sk = 0.f;
+#pragma unroll
+        for (int w = 0; w < POST_WARPS; ++w) {
+            sq += s_part[0][w];
+            sk += s_part[1][w];
+        }
+    }
+    if (slot >= gqa_post_slots(a)) return;
+    float* buf = smem + warp * gqa_post_buf(a);
+    if (a.taps <= 1) {
+        gqa_post_row(a, m, slot, m, sq, sk, buf);
+        return;
+    }
+    int first, end;
+    a.runs.find(m, first, end);
+    const int keep = a.taps - 1;
+    if (m > first && m < first + keep) return;  // served by the warp of the run's first row
+    gqa_post_row(a, m, slot, first, sq, sk, buf);
+    if (m > first) return;
+    for (int r = first + 1; r < min(end, first + keep); ++r) gqa_post_row(a, r, slot, first, 0.f, 0.f, buf);
+    // the run's last inputs replace the kept ones (a lane keeps the channels that it has read)
+    const bool is_v = slot >= a.heads + G, is_q = slot < a.heads;
+    const int h = is_v ? slot - a.heads - G : is_q ? slot : slot - a.heads, n = is_v ? vdim : dim, ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n, channels = nq + nk + G * vdim;
+    float* state = a.conv_state + (size_t)a.row_seq[m] * a.conv_stride + ch0;
+    for (int r = max(first, end - keep); r < end; ++r) {
+        const int p = a.row_pos[r];
+        for (int d = lane; d < n; d += 32) state[(size_t)(p % keep) * channels + d] = ld_cg_f32(a.raw + (size_t)r * a.ld + ch0 + d);
+    }
+}
+
+}  // namespace hm

@@ -17,6 +17,7 @@
 // accumulators are almost never rescaled.
 #include "latent_attn.h"
 
+#include "latent_post.cuh"
 #include "launch_attrs.h"
 #include "mbarrier.cuh"
 
@@ -30,28 +31,10 @@ __device__ __forceinline__ float latent_load(const void* page, size_t off, int b
 }
 
 __global__ void __launch_bounds__(128) latent_write_kernel(const LatentPool pool, const float* __restrict__ c, int ldc, const float* __restrict__ w, float eps, const int32_t* __restrict__ row_pos, const int32_t* __restrict__ row_seq) {
+    __shared__ float part[4];
     pdl_launch_dependents();
     pdl_wait();
-    const int m = blockIdx.x, tid = threadIdx.x, lane = tid & 31, R = pool.rank;
-    const float* x = c + (size_t)m * ldc;
-    float s = 0.f;
-    for (int i = tid; i < R; i += 128) {
-        const float v = ld_cg_f32(x + i);
-        s = fmaf(v, v, s);
-    }
-    __shared__ float sw[4];
-    s = warp_sum(s);
-    if (lane == 0) sw[tid >> 5] = s;
-    __syncthreads();
-    const float inv = 1.0f / sqrtf((sw[0] + sw[1] + sw[2] + sw[3]) / (float)R + eps);
-    const int pos = row_pos[m];
-    const size_t page = (size_t)pool.page_table[(size_t)row_seq[m] * pool.max_pages + pos / LATENT_PAGE] * latent_page_elems(R, pool.bf16);
-    for (int i = tid; i < R; i += 128) {
-        const float v = (ld_cg_f32(x + i) * inv) * __ldg(w + i);
-        const size_t off = page + latent_page_off(pos % LATENT_PAGE, i, R, pool.bf16);
-        if (pool.bf16) reinterpret_cast<uint16_t*>(pool.pages)[off] = f32_to_bf16_rne(v);
-        else reinterpret_cast<float*>(pool.pages)[off] = v;
-    }
+    latent_write_row(pool, c, ldc, blockIdx.x, w, eps, row_pos, row_seq, 0, nullptr, part);
 }
 
 __global__ void latent_read_kernel(const LatentPool pool, int seq, int len, float* out) {

@@ -15,7 +15,7 @@ namespace {
 // interleave_which >= 0 selects the gate/up interleave: output j of gate (which = 0) or up
 // (which = 1) lands in column (j/64)*128 + which*64 + j%64, so one slab holds 64 gate columns
 // followed by the 64 matching up columns and the SwiGLU epilogue finds both in one CTA.
-__global__ void pack_from_nk_kernel(const uint16_t* __restrict__ src, int N, int K, uint16_t* __restrict__ dst, int n_off, int interleave_which) {
+__global__ void pack_from_nk_kernel(const uint16_t* __restrict__ src, int N, int K, uint16_t* __restrict__ dst, int n_off, int interleave_which, int k_total, int k_off) {
     __shared__ uint16_t tile[32][33];
     const int n0 = blockIdx.y * 32, k0 = blockIdx.x * 32;
     for (int r = threadIdx.y; r < 32; r += blockDim.y) {
@@ -27,7 +27,7 @@ __global__ void pack_from_nk_kernel(const uint16_t* __restrict__ src, int N, int
         const int k = k0 + r, n = n0 + threadIdx.x;
         if (k < K && n < N) {
             const int no = interleave_which >= 0 ? (n / 64) * SLAB + interleave_which * 64 + (n % 64) : n + n_off;
-            dst[((size_t)(no / SLAB) * K + k) * SLAB + (no % SLAB)] = tile[threadIdx.x][r];
+            dst[((size_t)(no / SLAB) * k_total + k_off + k) * SLAB + (no % SLAB)] = tile[threadIdx.x][r];
         }
     }
 }
@@ -52,7 +52,7 @@ __device__ __forceinline__ float position_element(const double* turns, int pos, 
     f -= rint(f);
     return i & 1 ? cospif(2.0f * (float)f) : sinpif(2.0f * (float)f);
 }
-__global__ void embed_gather_kernel(const void* table, int dtype, const uint32_t* tokens, int H, int V, float* out, int* err_flag, const double* turns, const int32_t* row_pos) {
+__global__ void embed_gather_kernel(const void* table, int dtype, const uint32_t* tokens, int H, int V, float* out, int* err_flag, const EmbedExtra x) {
     pdl_launch_dependents();
     pdl_wait();
     const int m = blockIdx.x;
@@ -62,19 +62,30 @@ __global__ void embed_gather_kernel(const void* table, int dtype, const uint32_t
         for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)m * H + i] = 0.f;
         return;
     }
-    if (turns) {
-        const int pos = row_pos[m];
-        for (int i = threadIdx.x; i < H; i += blockDim.x) {
-            const float e = dtype == 1 ? bf16_bits_to_f32(reinterpret_cast<const uint16_t*>(table)[(size_t)tok * H + i]) : reinterpret_cast<const float*>(table)[(size_t)tok * H + i];
-            out[(size_t)m * H + i] = e + position_element(turns, pos, i);
+    auto row_of = [&](int i) { return dtype == 1 ? bf16_bits_to_f32(reinterpret_cast<const uint16_t*>(table)[(size_t)tok * H + i]) : reinterpret_cast<const float*>(table)[(size_t)tok * H + i]; };
+    if (x.bigram) {
+        const int pos = x.row_pos[m], seq = x.row_seq[m];
+        uint32_t* kept = x.kept + (size_t)seq * x.kept_stride;
+        unsigned long long b = x.buckets;
+        if (pos > 0) {
+            const bool follows = m > 0 && x.row_seq[m - 1] == seq && x.row_pos[m - 1] + 1 == pos;
+            const uint32_t prev = follows ? tokens[m - 1] : kept[pos - 1];
+            b = (prev * x.mul_prev + tok * x.mul_cur) % x.buckets;
         }
-    } else if (dtype == 1) {  // bf16 rows
-        const uint16_t* row = reinterpret_cast<const uint16_t*>(table) + (size_t)tok * H;
-        for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)m * H + i] = bf16_bits_to_f32(row[i]);
+        if (threadIdx.x == 0) kept[pos] = tok;
+        for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)m * H + i] = fmaf(row_of(i), x.scale, bf16_bits_to_f32(x.bigram[b * H + i]));
+    } else if (x.turns) {
+        const int pos = x.row_pos[m];
+        for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)m * H + i] = row_of(i) + position_element(x.turns, pos, i);
+    } else if (x.scale != 1.f) {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)m * H + i] = row_of(i) * x.scale;
     } else {
-        const float* row = reinterpret_cast<const float*>(table) + (size_t)tok * H;
-        for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)m * H + i] = row[i];
+        for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)m * H + i] = row_of(i);
     }
+}
+
+__global__ void add_constant_kernel(float* x, size_t n, float c) {
+    for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) x[i] += c;
 }
 
 // rows whose logits are wanted, out of a pass over portions of several sequences
@@ -416,9 +427,9 @@ cudaError_t launch_pdl(void (*kern)(KArgs...), dim3 grid, dim3 block, cudaStream
 
 }  // namespace
 
-cudaError_t launch_pack_slabs_from_nk(const uint16_t* src_nk, int N, int K, uint16_t* dst, int n_off, int interleave_which, cudaStream_t st) {
+cudaError_t launch_pack_slabs_from_nk(const uint16_t* src_nk, int N, int K, uint16_t* dst, int n_off, int interleave_which, cudaStream_t st, int k_total, int k_off) {
     dim3 grid((K + 31) / 32, (N + 31) / 32), block(32, 8);
-    pack_from_nk_kernel<<<grid, block, 0, st>>>(src_nk, N, K, dst, n_off, interleave_which);
+    pack_from_nk_kernel<<<grid, block, 0, st>>>(src_nk, N, K, dst, n_off, interleave_which, k_total > 0 ? k_total : K, k_off);
     return cudaGetLastError();
 }
 cudaError_t launch_pack_slabs_from_kn(const uint16_t* src_kn, int K, int N, uint16_t* dst, cudaStream_t st) {
@@ -426,8 +437,13 @@ cudaError_t launch_pack_slabs_from_kn(const uint16_t* src_kn, int K, int N, uint
     pack_from_kn_kernel<<<grid_for(total, 256), 256, 0, st>>>(src_kn, K, N, dst);
     return cudaGetLastError();
 }
-cudaError_t launch_embed_gather(const void* table, int table_dtype, const uint32_t* tokens, int M, int H, int V, float* out, int* err_flag, cudaStream_t st, bool pdl, const double* turns, const int32_t* row_pos) {
-    return launch_pdl(embed_gather_kernel, dim3(M), dim3(256), st, pdl, table, table_dtype, tokens, H, V, out, err_flag, turns, row_pos);
+cudaError_t launch_add_constant(float* x, size_t n, float c, cudaStream_t st) {
+    add_constant_kernel<<<(unsigned)((n + 255) / 256 < 1024 ? (n + 255) / 256 : 1024), 256, 0, st>>>(x, n, c);
+    return cudaGetLastError();
+}
+
+cudaError_t launch_embed_gather(const void* table, int table_dtype, const uint32_t* tokens, int M, int H, int V, float* out, int* err_flag, cudaStream_t st, bool pdl, const EmbedExtra& extra) {
+    return launch_pdl(embed_gather_kernel, dim3(M), dim3(256), st, pdl, table, table_dtype, tokens, H, V, out, err_flag, extra);
 }
 cudaError_t launch_gather_rows(const float* src, const int32_t* rows, int n, int W, float* dst, cudaStream_t st, bool pdl) {
     return launch_pdl(gather_rows_kernel, dim3(n), dim3(256), st, pdl, src, rows, W, dst);

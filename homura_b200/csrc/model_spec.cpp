@@ -162,13 +162,160 @@ bool read_dipisun(const Json& j, ModelSpec* s, std::string* err) {
     return true;
 }
 
+bool get_str(const Json& o, const char* key, std::string* out) {
+    const Json* v = o.get(key);
+    if (!v || v->kind != Json::Str) return false;
+    *out = v->str;
+    return true;
+}
+
+bool read_rotation(const Json& m, int dim, RotSpec* r, const std::string& at, std::string* err) {
+    const Json* j = m.get("rot");
+    if (is_null(j)) return fail(err, at + "the mixer needs `rot`");
+    if (!get_int(*j, "dims", &r->dims) || !get_num(*j, "base", &r->base) || r->base <= 0) return fail(err, at + "`rot` needs dims and base");
+    if (r->dims % 2 != 0 || r->dims > dim) return fail(err, at + "`rot.dims` must be even and at most the head size");
+    const Json* s = j->get("scaling");
+    if (is_null(s)) return true;
+    r->scaled = true;
+    if (!get_num(*s, "factor", &r->factor) || !get_num(*s, "low", &r->low) || !get_num(*s, "high", &r->high) || !get_num(*s, "original", &r->original)) return fail(err, at + "`rot.scaling` needs factor, low, high and original");
+    if (r->factor <= 0 || r->low <= 0 || r->high <= 0 || r->original <= 0) return fail(err, at + "`rot.scaling` must be positive");
+    return true;
+}
+
+// Sizes and scale of an attention, its window and the first tokens that stay visible behind it.
+bool read_windowed(const Json& m, LayerSpec* l, const std::string& at, std::string* err) {
+    double scale = 0;
+    if (!get_int(m, "heads", &l->heads) || !get_int(m, "kv_heads", &l->kv_heads) || !get_int(m, "dim", &l->dim) || !get_int(m, "vdim", &l->vdim) || !get_num(m, "scale", &scale))
+        return fail(err, at + "the mixer needs heads, kv_heads, dim, vdim and scale");
+    if (l->heads % l->kv_heads != 0) return fail(err, at + "`kv_heads` does not divide `heads`");
+    l->scale = (float)scale;
+    l->sink = true;
+    const Json* k = m.get("mask");
+    if (is_null(k) || !get_int(*k, "size", &l->window)) return fail(err, at + "`mask` needs size");
+    if (!get_count(*k, "keep_first", &l->keep_first)) return fail(err, at + "`mask.keep_first` must be a number of tokens");
+    return true;
+}
+
+// Gebilorn: three kinds of mixers (windowed attention with rotation, windowed attention beside gated linear attention, latent
+// attention), mixer and feed-forward in parallel, dense feed-forwards or mixtures with a shared expert, a bigram embedding.
+bool read_gebilorn(const Json& j, ModelSpec* s, std::string* err) {
+    hm_config& c = s->cfg;
+    s->parallel = s->norm_offset = true;
+    c.tie_word_embeddings = 1;
+    if (!get_int(j, "width", &c.hidden_size) || !get_int(j, "vocab", &c.vocab_size)) return fail(err, "missing `width` or `vocab`");
+    const Json *norm = j.get("norm"), *emb = j.get("embedding");
+    if (!norm || !get_num(*norm, "eps", &c.rms_norm_eps)) return fail(err, "`norm` needs `eps`");
+    double num = 0;
+    if (!emb || !get_num(*emb, "scale", &num)) return fail(err, "`embedding` needs `scale`");
+    s->embed_scale = (float)num;
+    if (const Json* b = emb->get("bigram"); !is_null(b)) {
+        double prev = 0, cur = 0;
+        int buckets = 0;
+        if (!get_int(*b, "buckets", &buckets) || !get_num(*b, "mul_prev", &prev) || !get_num(*b, "mul_cur", &cur) || prev < 0 || cur < 0 || prev > 2147483647.0 || cur > 2147483647.0)
+            return fail(err, "`embedding.bigram` needs buckets, mul_prev and mul_cur");
+        s->bigram_buckets = buckets;
+        s->bigram_prev = (long long)prev;
+        s->bigram_cur = (long long)cur;
+    }
+    const Json* cap = j.get("logit_softcap");
+    if (!is_null(cap)) {
+        if (!get_num(j, "logit_softcap", &num) || num <= 0) return fail(err, "`logit_softcap` must be positive");
+        s->softcap = (float)num;
+    }
+    const Json* list = j.get("layers");
+    if (!list || list->kind != Json::Arr || list->arr.empty()) return fail(err, "missing `layers`");
+    for (size_t i = 0; i < list->arr.size(); ++i) {
+        const Json& e = list->arr[i];
+        const std::string at = "layer " + std::to_string(i) + ": ";
+        LayerSpec l;
+        std::string type, kind;
+        const Json *m = e.get("mixer"), *mlp = e.get("mlp");
+        if (!get_str(e, "type", &type) || is_null(m)) return fail(err, at + "missing `type` or `mixer`");
+        if (type == "attention") {
+            l.mixer = MIX_GQA;
+            l.qk_norm = QKN_UNIT;
+            l.out_gate = GATE_ELEM;
+            if (!read_windowed(*m, &l, at, err) || !read_rotation(*m, l.dim, &l.rot, at, err)) return false;
+        } else if (type == "parallel") {
+            l.mixer = MIX_PARALLEL;
+            l.out_gate = GATE_HEAD;
+            l.qkv_bias = true;
+            const Json *left = m->get("left"), *right = m->get("right");
+            double ls = 0, rs = 0, tau = 0;
+            if (is_null(left) || is_null(right) || !get_num(*m, "left_scale", &ls) || !get_num(*m, "right_scale", &rs)) return fail(err, at + "the mixer needs left, right, left_scale and right_scale");
+            if (!read_windowed(*left, &l, at, err)) return false;
+            if (!get_count(*left, "conv", &l.conv)) return fail(err, at + "`left.conv` must be a number of taps");
+            if (!get_int(*right, "heads", &l.lin_heads) || !get_int(*right, "dim", &l.lin_dim) || !get_int(*right, "vdim", &l.lin_vdim) || !get_num(*right, "tau", &tau) || tau <= 0)
+                return fail(err, at + "`right` needs heads, dim, vdim and tau");
+            l.lin_tau = (float)tau;
+            l.left_scale = (float)ls;
+            l.right_scale = (float)rs;
+        } else if (type == "latent_attention") {
+            l.mixer = MIX_LATENT;
+            if (!get_int(*m, "heads", &l.heads) || !get_int(*m, "dim", &l.dim) || !get_int(*m, "vdim", &l.vdim) || !get_int(*m, "kv_rank", &l.kv_rank) || !get_int(*m, "q_rank", &l.q_rank) ||
+                !get_int(*m, "rot_dim", &l.rot_dim) || !get_num(*m, "scale", &num))
+                return fail(err, at + "the mixer needs heads, dim, rot_dim, vdim, q_rank, kv_rank and scale");
+            l.scale = (float)num;
+            if (!read_rotation(*m, l.rot_dim, &l.rot, at, err)) return false;
+            if (l.rot.dims != l.rot_dim) return fail(err, at + "`rot.dims` differs from `rot_dim`");
+        } else {
+            return fail(err, at + "unknown mixer type");
+        }
+        if (!is_null(mlp)) {
+            if (!get_str(*mlp, "kind", &kind)) return fail(err, at + "unknown mlp");
+            if (kind == "dense") {
+                l.mlp = MLP_GLU;
+                l.act = GLU_GELU;
+                if (!get_int(*mlp, "ff", &l.ff)) return fail(err, at + "`mlp` needs ff");
+            } else if (kind == "moe") {
+                const Json *ex = mlp->get("expert"), *r = mlp->get("router"), *sh = mlp->get("shared");
+                l.mlp = MLP_MOE;
+                l.act = GLU_SILU;
+                if (is_null(ex) || !get_int(*ex, "ff", &l.ff)) return fail(err, at + "`mlp.expert` needs ff");
+                if (is_null(r) || !get_int(*r, "experts", &l.experts) || !get_int(*r, "top", &l.top) || !get_num(*r, "scale", &num)) return fail(err, at + "`mlp.router` needs experts, top and scale");
+                if (l.top > l.experts) return fail(err, at + "`mlp.router.top` is larger than the number of experts");
+                l.router_scale = (float)num;
+                if (!is_null(sh) && !get_int(*sh, "ff", &l.shared_ff)) return fail(err, at + "`mlp.shared` needs ff");
+            } else {
+                return fail(err, at + "unknown mlp");
+            }
+        }
+        c.num_attention_heads = std::max(c.num_attention_heads, l.heads);
+        c.num_key_value_heads = std::max(c.num_key_value_heads, std::max(l.kv_heads, 1));
+        c.head_dim = std::max(c.head_dim, l.dim + l.rot_dim);
+        c.intermediate_size = std::max(c.intermediate_size, std::max(l.ff, l.shared_ff));
+        s->layers.push_back(l);
+    }
+    c.num_hidden_layers = (int)s->layers.size();
+    c.max_position_embeddings = 1 << 30;  // rotations are computed: the cache is the only limit
+    c.intermediate_size = std::max(c.intermediate_size, 1);
+    return true;
+}
+
 struct Design {
     const char* name;
     bool (*read)(const Json&, ModelSpec*, std::string*);
 };
-const Design kDesigns[] = {{"Tunitar", read_tunitar}, {"Dipisun", read_dipisun}};
+const Design kDesigns[] = {{"Tunitar", read_tunitar}, {"Dipisun", read_dipisun}, {"Gebilorn", read_gebilorn}};
 
 }  // namespace
+
+std::vector<double> rotation_turns(const RotSpec& r) {
+    const double full = 6.283185307179586;
+    std::vector<double> t(r.dims / 2);
+    for (size_t i = 0; i < t.size(); ++i) {
+        const double f = std::pow(r.base, -2.0 * (double)i / r.dims), wave = full / f;
+        double turned = f;
+        if (r.scaled && wave > r.original / r.low) {
+            turned = f / r.factor;
+        } else if (r.scaled && wave >= r.original / r.high) {
+            const double s = (r.original / wave - r.low) / (r.high - r.low);
+            turned = (1.0 - s) * f / r.factor + s * f;
+        }
+        t[i] = turned / full;
+    }
+    return t;
+}
 
 bool parse_model_spec(const char* text, size_t len, ModelSpec* out, std::string* err) {
     Json j;
@@ -200,12 +347,48 @@ bool parse_model_spec_file(const std::string& path, ModelSpec* out, std::string*
     return parse_model_spec(reinterpret_cast<const char*>(f.data()), f.size(), out, err);
 }
 
+namespace {
+std::string parallel_layer_json(const LayerSpec& l) {
+    std::string o;
+    char t[768];
+    auto rot = [&]() {
+        std::snprintf(t, sizeof(t), ",\"rot\":{\"dims\":%d,\"base\":%.9g", l.rot.dims, l.rot.base);
+        o += t;
+        if (l.rot.scaled) {
+            std::snprintf(t, sizeof(t), ",\"factor\":%.9g,\"low\":%.9g,\"high\":%.9g,\"original\":%.9g", l.rot.factor, l.rot.low, l.rot.high, l.rot.original);
+            o += t;
+        }
+        o += "}";
+    };
+    if (l.mixer == MIX_LATENT) {
+        std::snprintf(t, sizeof(t), "{\"type\":\"latent_attention\",\"heads\":%d,\"dim\":%d,\"rot_dim\":%d,\"vdim\":%d,\"q_rank\":%d,\"kv_rank\":%d,\"scale\":%.9g", l.heads, l.dim, l.rot_dim, l.vdim, l.q_rank, l.kv_rank, l.scale);
+        o += t;
+        rot();
+    } else {
+        std::snprintf(t, sizeof(t), "{\"type\":\"%s\",\"heads\":%d,\"kv_heads\":%d,\"dim\":%d,\"vdim\":%d,\"scale\":%.9g,\"window\":%d,\"keep_first\":%d,\"conv\":%d", l.mixer == MIX_GQA ? "windowed_attention" : "parallel", l.heads, l.kv_heads,
+                      l.dim, l.vdim, l.scale, l.window, l.keep_first, l.conv);
+        o += t;
+        if (l.rot.dims) rot();
+        if (l.mixer == MIX_PARALLEL) {
+            std::snprintf(t, sizeof(t), ",\"linear\":{\"heads\":%d,\"dim\":%d,\"vdim\":%d,\"tau\":%.9g},\"left_scale\":%.9g,\"right_scale\":%.9g", l.lin_heads, l.lin_dim, l.lin_vdim, l.lin_tau, l.left_scale, l.right_scale);
+            o += t;
+        }
+    }
+    std::snprintf(t, sizeof(t), ",\"ff\":%d,\"experts\":%d,\"top\":%d,\"router_scale\":%.9g,\"shared_ff\":%d}", l.ff, l.experts, l.top, l.router_scale, l.shared_ff);
+    return o + t;
+}
+}  // namespace
+
 std::string layers_json(const ModelSpec& spec) {
     std::string o = "[";
     for (size_t i = 0; i < spec.layers.size(); ++i) {
         const LayerSpec& l = spec.layers[i];
-        char t[512];
+        char t[768];
         if (i) o += ",";
+        if (spec.parallel) {
+            o += parallel_layer_json(l);
+            continue;
+        }
         if (l.mixer == MIX_LATENT) {
             std::snprintf(t, sizeof(t), "{\"type\":\"latent_attention\",\"heads\":%d,\"dim\":%d,\"vdim\":%d,\"kv_rank\":%d,\"kv_from\":%s,\"scale\":%.9g,\"ff\":%d}", l.heads, l.dim, l.vdim, l.kv_rank,
                           l.kv_from < 0 ? "null" : std::to_string(l.kv_from).c_str(), l.scale, l.ff);

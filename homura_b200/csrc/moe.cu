@@ -12,6 +12,7 @@
 
 #include "gemm_tc.h"
 #include "launch_attrs.h"
+#include "route.cuh"
 
 namespace hm {
 namespace {
@@ -39,59 +40,6 @@ __device__ __forceinline__ float dot8(const uint4& w, const float4& x, const flo
     s = fmaf(bf16_hi(w.z), y.y, s);
     s = fmaf(bf16_lo(w.w), y.z, s);
     return fmaf(bf16_hi(w.w), y.w, s);
-}
-
-// softmax over the router's outputs, choice by score + correction (ties to the lower index), weights without it: one warp
-__device__ __forceinline__ void choose(const PostNormArgs& a, int m, float* z, float* choice) {
-    const int lane = threadIdx.x & 31;
-    float mx = -INFINITY, l = 0.f;
-    for (int r = lane; r < a.n_out; r += 32) mx = fmaxf(mx, z[r]);
-    mx = warp_max(mx);
-    for (int r = lane; r < a.n_out; r += 32) {
-        const float e = expf(z[r] - mx);
-        z[r] = e;
-        l += e;
-    }
-    l = warp_sum(l);
-    uint32_t* key = reinterpret_cast<uint32_t*>(choice);  // unsigned integers in the order of the floats; 0: chosen already
-    for (int r = lane; r < a.n_out; r += 32) {
-        const float s = z[r] / l;
-        z[r] = s;
-        const uint32_t u = __float_as_uint(s + __ldg(a.correction + r));
-        key[r] = u >> 31 ? ~u : u | 0x80000000u;
-    }
-    __syncwarp();
-    float ident = 0.f;
-    for (int k = 0; k < a.top; ++k) {
-        uint32_t best = 0u, at = lane < a.n_out ? lane : 0xffffffffu;
-        for (int r = lane; r < a.n_out; r += 32)
-            if (key[r] > best) {
-                best = key[r];
-                at = r;
-            }
-        const uint32_t most = __reduce_max_sync(0xffffffffu, best);
-        const int bi = (int)__reduce_min_sync(0xffffffffu, best == most ? at : 0xffffffffu);
-        const float s = z[bi];
-        __syncwarp();
-        if (lane == 0) {
-            key[bi] = 0u;
-            const bool id = bi >= a.experts;
-            a.out.ids[(size_t)m * a.top + k] = id ? -1 : bi;
-            a.out.weights[(size_t)m * a.top + k] = s;
-            if (id) ident += s;
-            else if (a.out.dense) a.out.dense[(size_t)m * a.experts + bi] = s;
-        }
-        __syncwarp();
-    }
-    if (a.out.dense) {  // the chosen ones are those whose key is gone
-        const int words = (a.experts + 31) / 32;
-        for (int w = 0; w < words; ++w) {
-            const int r = w * 32 + lane;
-            const uint32_t bits = __ballot_sync(0xffffffffu, r < a.experts && key[r] == 0u);
-            if (lane == 0) a.out.mask[(size_t)m * words + w] = bits;
-        }
-    }
-    if (lane == 0) a.out.identity[m] = ident;
 }
 
 __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PostNormArgs a, int cluster) {
@@ -194,7 +142,7 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PostNormArgs a
     // the residual is stored when every CTA of the row has read it
     if (cluster > 1) cluster_sync_all();
     else __syncthreads();
-    if (a.router && rank == 0 && warp == 0) choose(a, m, z, choice);
+    if (a.router && rank == 0 && warp == 0) choose_experts(RouteSpec{a.correction, a.experts, a.n_out, a.top, 1.f, a.out}, m, z, choice);
     const int c_n = a.xp ? (a.W + 63) / 64 * 8 : Wp / 8;
     for (int c = rank * THREADS + tid; c < c_n; c += cluster * THREADS) {
         float v[8];
@@ -271,12 +219,12 @@ __global__ void __launch_bounds__(THREADS) expert_gate_up_kernel(const ExpertWei
             g += red[i][tid];
             u += red[i][GU_ROWS + tid];
         }
-        act[(size_t)pair * blocks * 64 + blk * 64 + sub * GU_ROWS + tid] = clamped_glu(g, u, w.limit) * rw;
+        act[(size_t)pair * blocks * 64 + blk * 64 + sub * GU_ROWS + tid] = glu(w.act, g, u, w.limit) * rw;
     }
 }
 
 // staged: the row's activations [top][ff padded] fit shared memory
-__global__ void __launch_bounds__(THREADS) expert_down_kernel(const ExpertWeights w, const float* __restrict__ act, const int32_t* __restrict__ ids, float* __restrict__ y, int staged) {
+__global__ void __launch_bounds__(THREADS) expert_down_kernel(const ExpertWeights w, const float* __restrict__ act, const int32_t* __restrict__ ids, const float* resid, float* y, int staged) {
     extern __shared__ __align__(16) float as[];
     __shared__ float red[WARPS][DOWN_ROWS];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, m = blockIdx.y;
@@ -346,7 +294,7 @@ __global__ void __launch_bounds__(THREADS) expert_down_kernel(const ExpertWeight
         float s = 0.f;
 #pragma unroll
         for (int i = 0; i < WARPS; ++i) s += red[i][tid];
-        y[(size_t)m * w.W + n] = s;
+        y[(size_t)m * w.W + n] = resid ? ld_cg_f32(resid + (size_t)m * w.W + n) + s : s;
     }
 }
 
@@ -398,11 +346,11 @@ cudaError_t launch_expert_gate_up(const ExpertWeights& e, const float* x, int M,
     return launch(expert_gate_up_kernel, dim3((unsigned)(expert_blocks(e.ff) * (64 / GU_ROWS)), (unsigned)(M * e.top)), smem, 1, st, pdl, e, x, r.ids, r.weights, act);
 }
 
-cudaError_t launch_expert_down(const ExpertWeights& e, const float* act, int M, const RouteOut& r, float* y, cudaStream_t st, bool pdl) {
+cudaError_t launch_expert_down(const ExpertWeights& e, const float* act, int M, const RouteOut& r, const float* resid, float* y, cudaStream_t st, bool pdl) {
     const size_t rows = sizeof(float) * (size_t)e.top * expert_blocks(e.ff) * 64;
     const int staged = rows <= 128 * 1024;
     const size_t smem = (staged ? rows : 0) + sizeof(int) * e.top;
-    return launch(expert_down_kernel, dim3((unsigned)((e.W + 127) / 128 * (128 / DOWN_ROWS)), (unsigned)M), smem, 1, st, pdl, e, act, r.ids, y, staged);
+    return launch(expert_down_kernel, dim3((unsigned)((e.W + 127) / 128 * (128 / DOWN_ROWS)), (unsigned)M), smem, 1, st, pdl, e, act, r.ids, resid, y, staged);
 }
 
 }  // namespace hm

@@ -4,6 +4,7 @@
 #include <stdint.h>
 
 #include "common.cuh"
+#include "model_spec.h"
 
 namespace hm {
 
@@ -14,6 +15,14 @@ struct RouteOut {
     float* identity;    // [M] sum of the weights of the chosen identity experts
     float* dense;       // [M][experts] weight of every expert, 0 where it is not chosen; or null
     uint32_t* mask;     // [M][ceil(experts / 32)] with dense: one bit per chosen expert
+};
+
+// How a router chooses: `top` of n_out = experts + identity ones (the last) by score + correction; weights are the scores times scale.
+struct RouteSpec {
+    const float* correction; // [n_out] or null
+    int experts, n_out, top;
+    float scale;
+    RouteOut out;
 };
 
 // x += mult * RMSnorm(y) * w, and then, optionally, the router over the new x.
@@ -42,6 +51,7 @@ struct ExpertWeights {
     const uint16_t *gu, *down;
     int n, W, ff, top;       // n experts
     float limit;
+    int act;                 // GluAct
 };
 __host__ __device__ __forceinline__ int expert_blocks(int ff) { return (ff + 63) / 64; }
 size_t expert_gu_elems(int W, int ff);
@@ -49,12 +59,20 @@ size_t expert_down_elems(int W, int ff);
 
 // Few rows: every (row, chosen expert) pair reads its own weights.  act: [M * top][ff padded], already times the routing weight.
 cudaError_t launch_expert_gate_up(const ExpertWeights& e, const float* x, int M, const RouteOut& r, float* act, cudaStream_t st, bool pdl);
-cudaError_t launch_expert_down(const ExpertWeights& e, const float* act, int M, const RouteOut& r, float* y, cudaStream_t st, bool pdl);
+// y = resid (or nothing) + the sum over the chosen experts; y may be resid.
+cudaError_t launch_expert_down(const ExpertWeights& e, const float* act, int M, const RouteOut& r, const float* resid, float* y, cudaStream_t st, bool pdl);
 
 // Gated activation of an expert: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1).
 __device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
     return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
+// act(gate) * up of the kinds of gated feed-forwards (GluAct).
+__device__ __forceinline__ float glu(int act, float gate, float up, float limit) {
+    if (act == GLU_SILU) return gate / (1.0f + expf(-gate)) * up;
+    if (act == GLU_GELU) return 0.5f * gate * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * gate * gate, gate, gate))) * up;
+    return clamped_glu(gate, up, limit);
 }
 
 }  // namespace hm

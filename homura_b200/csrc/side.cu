@@ -1,0 +1,257 @@
+// See side.h.  Blocks take their parts in order of weight: the recurrences first, then heads, latents, activations, routers.
+#include "side.h"
+
+#include <algorithm>
+
+#include "gemm_tc.h"
+#include "gla.cuh"
+#include "gqa_post.cuh"
+#include "latent_post.cuh"
+#include "launch_attrs.h"
+#include "route.cuh"
+
+namespace hm {
+namespace {
+
+constexpr int THREADS = 256, WARPS = THREADS / 32;
+static_assert(THREADS == GLA_THREADS && WARPS == POST_WARPS, "one block size for all parts");
+
+__device__ __forceinline__ float block_sum(float v, float* part) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < WARPS; ++i) s += part[i];
+    return s;
+}
+
+__device__ __forceinline__ int act_blocks(int ff) { return ((ff + 7) / 8 + THREADS - 1) / THREADS; }
+
+__device__ __forceinline__ void act_block(const SideArgs& a, int b) {
+    const MlpSide& f = a.mlp;
+    const int per = act_blocks(f.ff), m = b / per, c = ((b - m * per) * THREADS + threadIdx.x) * 8;
+    if (c >= f.ff) return;
+    const size_t row = (size_t)m * a.ld;
+    const float4 g0 = ld_cg_f32x4(f.gate + row + c), g1 = ld_cg_f32x4(f.gate + row + c + 4), u0 = ld_cg_f32x4(f.up + row + c), u1 = ld_cg_f32x4(f.up + row + c + 4);
+    const float rg = f.row_gate ? 1.0f / (1.0f + expf(-ld_cg_f32(f.row_gate + row))) : 1.f;
+    const float g[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w}, u[8] = {u0.x, u0.y, u0.z, u0.w, u1.x, u1.y, u1.z, u1.w};
+    float v[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = glu(f.act, g[e], u[e], 0.f) * rg;
+    if (f.xp) {
+        tc_xpack_store8(f.xp, a.xp_mpad, m, f.out_off + c, v);
+    } else {
+        float* o = f.out + (size_t)m * f.ld_out + f.out_off + c;
+        reinterpret_cast<float4*>(o)[0] = make_float4(v[0], v[1], v[2], v[3]);
+        reinterpret_cast<float4*>(o)[1] = make_float4(v[4], v[5], v[6], v[7]);
+    }
+}
+
+// One warp chooses, the others leave; z: 2 * n_out floats.
+__device__ __forceinline__ void route_block(const SideArgs& a, int m, float* z) {
+    const MlpSide& f = a.mlp;
+    if (f.route.out.dense)
+        for (int i = threadIdx.x; i < f.route.experts; i += THREADS) f.route.out.dense[(size_t)m * f.route.experts + i] = 0.f;
+    for (int i = threadIdx.x; i < f.route.n_out; i += THREADS) z[i] = ld_cg_f32(f.logits + (size_t)m * a.ld + i);
+    __syncthreads();
+    if (threadIdx.x < 32) choose_experts(f.route, m, z, z + f.route.n_out);
+}
+
+__device__ __forceinline__ void normed_block(const SideArgs& a, int m, float* part) {
+    const MlpSide& f = a.mlp;
+    const float* x = f.x + (size_t)m * f.W;
+    float s = 0.f;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < f.W; i += THREADS) {
+        const float v = ld_cg_f32(x + i);
+        s = fmaf(v, v, s);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(s, part) / (float)f.W + a.eps);
+#pragma unroll 4
+    for (int i = threadIdx.x; i < f.W; i += THREADS) f.normed[(size_t)m * f.W + i] = (ld_cg_f32(x + i) * inv) * __ldg(f.w + i);
+}
+
+// The queries' latent of row m, RMS-normed and packed.
+__device__ __forceinline__ void query_latent_block(const SideArgs& a, int m, float* part) {
+    const LatentSide& l = a.latent;
+    const float* x = l.cq + (size_t)m * a.ld;
+    float s = 0.f;
+    for (int i = threadIdx.x; i < l.q_rank; i += THREADS) {
+        const float v = ld_cg_f32(x + i);
+        s = fmaf(v, v, s);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(s, part) / (float)l.q_rank + a.eps);
+    for (int c = threadIdx.x * 8; c < (l.q_rank + 63) / 64 * 64; c += THREADS * 8) {
+        float v[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = c + e < l.q_rank ? (ld_cg_f32(x + c + e) * inv) * __ldg(l.q_w + c + e) : 0.f;
+        tc_xpack_store8(l.q_xp, a.xp_mpad, m, c, v);
+    }
+}
+
+// RD: state rows per thread of the linear attention, 0: there is none
+template <int RD>
+__global__ void __launch_bounds__(THREADS) side_kernel(const __grid_constant__ SideArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float part[WARPS];
+    pdl_launch_dependents();
+    int b = blockIdx.x;
+    if constexpr (RD > 0) {
+        if (b < a.n_gla) {
+            gla_block<RD>(a.gla, b % a.gla.heads, b / a.gla.heads, sm);
+            return;
+        }
+        b -= a.n_gla;
+    }
+    if (b < a.n_post) {
+        const int per = gqa_post_blocks(a.post);
+        gqa_post_block(a.post, b / per, b % per, sm);
+        return;
+    }
+    b -= a.n_post;
+    pdl_wait();
+    if (b < a.n_latent) {
+        if (b < a.M) latent_write_row(a.latent.pool, a.latent.c, a.ld, b, a.latent.w, a.eps, a.row_pos, a.row_seq, a.latent.rot_pairs, a.latent.turns, part);
+        else query_latent_block(a, b - a.M, part);
+        return;
+    }
+    b -= a.n_latent;
+    if (b < a.n_act) {
+        act_block(a, b);
+        return;
+    }
+    b -= a.n_act;
+    if (b < a.n_route) route_block(a, b, sm);
+    else normed_block(a, b - a.n_route, part);
+}
+
+__global__ void __launch_bounds__(THREADS) sum_norm_kernel(const SumNormArgs a) {
+    extern __shared__ __align__(16) float xs[];
+    __shared__ float part[WARPS];
+    const int m = blockIdx.x, tid = threadIdx.x, Wp = (a.W + 63) / 64 * 64;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (m >= a.M) {  // rows that pad the image
+        if (a.w)
+            for (int c = tid * 8; c < Wp; c += THREADS * 8) {
+                const float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+                tc_xpack_store8(a.xp, a.xp_mpad, m, c, v);
+            }
+        return;
+    }
+    float* x = a.x + (size_t)m * a.W;
+    const float* y = a.y + (size_t)m * a.W;
+    float s = 0.f;
+    if ((a.W & 3) == 0) {
+        for (int i = tid; i < a.W / 4; i += THREADS) {
+            float4 v = ld_cg_f32x4(x + 4 * (size_t)i);
+            for (int p = 0; p < a.parts; ++p) {
+                const float4 t = ld_cg_f32x4(y + p * a.part_stride + 4 * (size_t)i);
+                v = make_float4(v.x + t.x, v.y + t.y, v.z + t.z, v.w + t.w);
+            }
+            s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+            reinterpret_cast<float4*>(xs)[i] = v;
+            if (a.parts) reinterpret_cast<float4*>(x)[i] = v;
+        }
+    } else {
+        for (int i = tid; i < a.W; i += THREADS) {
+            float v = ld_cg_f32(x + i);
+            for (int p = 0; p < a.parts; ++p) v += ld_cg_f32(y + p * a.part_stride + i);
+            s = fmaf(v, v, s);
+            xs[i] = v;
+            if (a.parts) x[i] = v;
+        }
+    }
+    if (!a.w) return;
+    const float inv = 1.0f / sqrtf(block_sum(s, part) / (float)a.W + a.eps);  // (its barrier publishes the row as well)
+    for (int c = tid * 8; c < Wp; c += THREADS * 8) {
+        float v[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = c + e < a.W ? (xs[c + e] * inv) * __ldg(a.w + c + e) : 0.f;
+        tc_xpack_store8(a.xp, a.xp_mpad, m, c, v);
+    }
+}
+
+template <typename K, typename A>
+cudaError_t launch(K kern, unsigned blocks, size_t smem, cudaStream_t st, bool pdl, const A& args) {
+    const cudaError_t e = ensure_dyn_smem(kern, smem);
+    if (e != cudaSuccess) return e;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(blocks);
+    cfg.blockDim = dim3(THREADS);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute at[1];
+    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = at;
+    cfg.numAttrs = pdl ? 1 : 0;
+    return cudaLaunchKernelEx(&cfg, kern, args);
+}
+
+}  // namespace
+
+bool gla_shape(int dim, int vdim, GlaShape* out) {
+    if (dim < 1 || vdim < 1 || dim > 1024 || vdim > 512) return false;
+    GlaShape s;
+    s.cols = 8;
+    while (s.cols < vdim && s.cols < GLA_THREADS) s.cols *= 2;
+    for (; s.cols >= 8; s.cols /= 2) {
+        s.lanes = GLA_THREADS / s.cols;
+        if (s.lanes * 64 >= dim) break;
+    }
+    s.rows = 8;
+    while (s.rows * s.lanes < dim) s.rows *= 2;
+    s.slices = (vdim + s.cols - 1) / s.cols;
+    *out = s;
+    return true;
+}
+
+size_t gla_smem(GlaArgs* a) {
+    const size_t up = a->rank * a->dim <= GLA_UP_SMEM ? (size_t)(a->rank * a->dim + 3) / 4 * 4 : 0;
+    const int rows = a->runs.n ? a->longest_run : 1;
+    for (a->step = std::min(16, rows);; a->step /= 2) {
+        const size_t bytes = sizeof(float) * (up + (size_t)a->step * (3 * a->shape.padded_dim() + a->shape.cols + a->rank) + (size_t)(a->shape.slices > 1 ? rows : a->step) * a->vdim);
+        if (bytes <= 160 * 1024 || a->step == 1) return bytes;
+    }
+}
+
+cudaError_t launch_side(const SideArgs& a_in, cudaStream_t st, bool pdl) {
+    SideArgs a = a_in;
+    if (a.M < 1 || a.M > GQA_MAX_ROWS) return cudaErrorInvalidValue;
+    const int runs = a.gla.runs.n ? a.gla.runs.n : a.M;
+    size_t smem = 0;
+    a.n_gla = a.n_post = a.n_latent = a.n_act = a.n_route = a.n_normed = 0;
+    if (a.has_gla) {
+        a.n_gla = runs * a.gla.heads;
+        smem = std::max(smem, gla_smem(&a.gla));
+    }
+    if (a.has_post) {
+        a.n_post = a.M * gqa_post_blocks(a.post);
+        smem = std::max(smem, gqa_post_smem(a.post));
+    }
+    if (a.has_latent) a.n_latent = a.M * (a.latent.q_xp ? 2 : 1);
+    if (a.mlp.ff) a.n_act = a.M * (((a.mlp.ff + 7) / 8 + THREADS - 1) / THREADS);
+    if (a.mlp.logits) {
+        a.n_route = a.M;
+        smem = std::max(smem, 2 * sizeof(float) * (size_t)a.mlp.route.n_out);
+    }
+    if (a.mlp.normed) a.n_normed = a.M;
+    const unsigned blocks = (unsigned)(a.n_gla + a.n_post + a.n_latent + a.n_act + a.n_route + a.n_normed);
+    switch (a.has_gla ? a.gla.shape.rows : 0) {
+        case 0: return launch(side_kernel<0>, blocks, smem, st, pdl, a);
+        case 8: return launch(side_kernel<8>, blocks, smem, st, pdl, a);
+        case 16: return launch(side_kernel<16>, blocks, smem, st, pdl, a);
+        case 32: return launch(side_kernel<32>, blocks, smem, st, pdl, a);
+        case 64: return launch(side_kernel<64>, blocks, smem, st, pdl, a);
+        default: return cudaErrorInvalidValue;
+    }
+}
+
+cudaError_t launch_sum_norm(const SumNormArgs& a, cudaStream_t st, bool pdl) {
+    if (!a.w && !a.parts) return cudaSuccess;
+    return launch(sum_norm_kernel, (unsigned)(a.w ? tc_mpad(a.M) : a.M), sizeof(float) * (size_t)((a.W + 7) / 8 * 8), st, pdl, a);
+}
+
+}  // namespace hm

@@ -360,6 +360,128 @@ def write_dipisun_model(model_dir: str, cfg: dict, seed: int, weights: Optional[
     return _write_model(model_dir, cfg, dipisun_tensor_specs(cfg, buckets), lambda s: dipisun_tensor(seed, s) if weights is None else weights[s[0]])
 
 
+# ---- Gebilorn ---------------------------------------------------------------------------------
+
+
+def gebilorn_rot(dims: int, base: float = 10000.0, scaling: Optional[Tuple[float, float, float, float]] = None) -> dict:
+    """scaling: (factor, low, high, original)."""
+    r: dict = {"dims": dims, "base": base}
+    if scaling is not None:
+        r["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    return r
+
+
+def gebilorn_attention(heads: int, kv_heads: int, dim: int, vdim: int, window: int, rot: dict, keep_first: int = 0, scale: Optional[float] = None) -> dict:
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim**-0.5 if scale is None else scale, "mask": {"size": window, "keep_first": keep_first}, "rot": rot}
+    return {"type": "attention", "mixer": m}
+
+
+def gebilorn_parallel(left: Tuple[int, int, int, int], window: int, conv: int, right: Tuple[int, int, int], tau: float = 16.0, scales: Tuple[float, float] = (1.0, 1.0), scale: Optional[float] = None) -> dict:
+    """left: heads, kv_heads, dim, vdim of the windowed attention; right: heads, dim, vdim of the linear one."""
+    h, g, d, v = left
+    a = {"heads": h, "kv_heads": g, "dim": d, "vdim": v, "scale": d**-0.5 if scale is None else scale, "mask": {"size": window}, "conv": conv}
+    return {"type": "parallel", "mixer": {"left": a, "right": dict(zip(("heads", "dim", "vdim"), right), tau=tau), "left_scale": scales[0], "right_scale": scales[1]}}
+
+
+def gebilorn_latent(heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, rot: Optional[dict] = None, scale: Optional[float] = None) -> dict:
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "scale": (dim + rot_dim) ** -0.5 if scale is None else scale, "rot": rot or gebilorn_rot(rot_dim)}
+    return {"type": "latent_attention", "mixer": m}
+
+
+def gebilorn_dense(ff: int) -> dict:
+    return {"kind": "dense", "ff": ff}
+
+
+def gebilorn_moe(ff: int, experts: int, top: int, shared_ff: int, scale: float = 1.0) -> dict:
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "scale": scale}, "shared": {"ff": shared_ff}}
+
+
+def gebilorn_config(width: int, vocab: int, layers: List[Tuple[dict, Optional[dict]]], buckets: int = 61, muls: Tuple[int, int] = (31, 7), scale: float = 2.0, softcap: float = 50.0, eps: float = 1e-6, **extra) -> dict:
+    """layers: (mixer, mlp or None) pairs."""
+    emb = {"scale": scale, "bigram": {"buckets": buckets, "mul_prev": muls[0], "mul_cur": muls[1]}}
+    return {"architecture": "Gebilorn", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": emb, "logit_softcap": softcap, "layers": [{**m, "mlp": f} for m, f in layers], **extra}
+
+
+def gebilorn_uniform(width: int, vocab: int, n_layers: int, heads: int, kv_heads: int, dim: int, ff: int, experts: int, top: int, expert_ff: int, kv_rank: int) -> dict:
+    """Of every six layers four run windowed attention beside linear attention, one latent attention, one windowed attention with rotation;
+    every third feed-forward is dense, the others are mixtures whose chosen and shared experts have as many parameters."""
+    layers = []
+    for i in range(n_layers):
+        if i % 6 == 3:
+            m = gebilorn_attention(heads, kv_heads, dim, dim, 1024, gebilorn_rot(dim // 2, 500000.0, (8.0, 1.0, 4.0, 8192.0)), 64)
+        elif i % 6 == 5:
+            m = gebilorn_latent(heads, dim, 64, dim, width // 2, kv_rank)
+        else:
+            m = gebilorn_parallel((heads, kv_heads, dim, dim), 512, 4, (heads, dim, dim))
+        layers.append((m, gebilorn_dense(ff) if i % 3 == 0 else gebilorn_moe(expert_ff, experts, top, ff - top * expert_ff)))
+    return gebilorn_config(width, vocab, layers, 65521, (8191, 131))
+
+
+# Gebilorn stacks with the width, depth, heads and head size of the Qwen2.5 architectures above; dense feed-forwards, and chosen and shared
+# experts together, have the MLP parameters of theirs.
+GEBILORN_05B = gebilorn_uniform(896, 151936, 24, 14, 2, 64, 4864, 16, 4, 960, 256)
+GEBILORN_15B = gebilorn_uniform(1536, 151936, 28, 12, 2, 128, 8960, 32, 8, 960, 512)
+
+
+def gebilorn_tensor_specs(cfg: dict, decay_rank: int = 16) -> List[Tuple[str, Tuple[int, ...], str]]:
+    """(name, shape, kind); decay_rank: width of the decays' latents."""
+    W, V = cfg["width"], cfg["vocab"]
+    specs: List[Tuple[str, Tuple[int, ...], str]] = [("embed", (V, W), "embed"), ("bigram", (cfg["embedding"]["bigram"]["buckets"] + 1, W), "embed")]
+
+    def attention(p, m, gate):
+        q, k, v, o = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], m["heads"] * m["vdim"]
+        return [(p + "q", (q, W), "w"), (p + "k", (k, W), "w"), (p + "v", (v, W), "w"), (p + "sink", (m["heads"],), "embed"), (p + "g", (gate, W), "w"), (p + "o", (W, o), "w")]
+
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", layer["mixer"], layer.get("mlp")
+        specs.append((p + "norm1", (W,), "zero"))
+        if layer["type"] == "attention":
+            specs += attention(p + "mix.", m, m["heads"] * m["vdim"])
+        elif layer["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            specs += attention(p + "mix.left.", a, a["heads"])
+            for t, n in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])):
+                specs.append((f"{p}mix.left.{t}.b", (n,), "zero"))
+                if a.get("conv"):
+                    specs.append((f"{p}mix.left.{t}.conv", (n, a["conv"]), "w"))
+            k, v = r["heads"] * r["dim"], r["heads"] * r["vdim"]
+            for t, shape, kind in (("q", (k, W), "w"), ("k", (k, W), "w"), ("v", (v, W), "w"), ("g", (v, W), "w"), ("o", (W, v), "w"), ("norm", (r["vdim"],), "one"), ("a1", (decay_rank, W), "w"), ("a2", (k, decay_rank), "w"), ("a2.b", (k,), "embed")):
+                specs.append((f"{p}mix.right.{t}", shape, kind))
+        else:
+            h, d, r, rot = m["heads"], m["dim"], m["kv_rank"], m["rot_dim"]
+            specs += [(p + "mix.dq", (m["q_rank"], W), "w"), (p + "mix.dq.norm", (m["q_rank"],), "one"), (p + "mix.uq", (h * (d + rot), m["q_rank"]), "w"), (p + "mix.dkv", (r + rot, W), "w"), (p + "mix.dkv.norm", (r,), "one")]
+            specs += [(p + "mix.uk", (h * d, r), "w"), (p + "mix.uv", (h * m["vdim"], r), "w"), (p + "mix.o", (W, h * m["vdim"]), "w")]
+        mlp = lambda q, ff: [(q + "gate", (ff, W), "w"), (q + "up", (ff, W), "w"), (q + "down", (W, ff), "w")]
+        if f is None:
+            continue
+        if f["kind"] == "dense":
+            specs += mlp(p + "mlp.", f["ff"])
+        else:
+            specs.append((p + "mlp.router", (f["router"]["experts"], W), "w"))
+            for e in range(f["router"]["experts"]):
+                specs += mlp(f"{p}mlp.e{e}.", f["expert"]["ff"])
+            specs += mlp(p + "mlp.shared.", f["shared"]["ff"]) + [(p + "mlp.shared.sg", (1, W), "w")]
+    return specs + [("final.norm", (W,), "zero")]
+
+
+def gebilorn_tensor(seed: int, spec) -> np.ndarray:
+    """bf16 bits of one tensor: linears N(0, 1/in), offsets and biases around 0, other vectors around 1."""
+    name, shape, kind = spec
+    if kind == "zero":
+        return f32_to_bf16_rne(0.25 * _rng(seed, name).standard_normal(shape, dtype=np.float32))
+    return tunitar_tensor(seed, spec)
+
+
+def gebilorn_weights(cfg: dict, seed: int, decay_rank: int = 16) -> Dict[str, np.ndarray]:
+    """name -> bf16 bits of every tensor."""
+    return {s[0]: gebilorn_tensor(seed, s) for s in gebilorn_tensor_specs(cfg, decay_rank)}
+
+
+def write_gebilorn_model(model_dir: str, cfg: dict, seed: int, weights: Optional[Dict[str, np.ndarray]] = None, decay_rank: int = 16) -> str:
+    """config.json + model.safetensors of a Gebilorn model (weights: bits to write instead of the seeded ones)."""
+    return _write_model(model_dir, cfg, gebilorn_tensor_specs(cfg, decay_rank), lambda s: gebilorn_tensor(seed, s) if weights is None else weights[s[0]])
+
+
 def shard_hf_model(src_dir: str, dst_dir: str, n_shards: int = 2) -> str:
     """Rewrite a single-file checkpoint as `n_shards` safetensors files plus model.safetensors.index.json,
     the layout HfModel::load_with_dtype falls back to (src/hf/model.rs:86-127).  Tensors are dealt out
