@@ -18,7 +18,7 @@ def model(name):
             (LA(5, 24, 12, 20, 56, 72), M(40, 7, 3, 56, 1.7)),
             (A(4, 2, 28, 36, 50, R(20, 1000.0, (3.0, 1.0, 4.0, 60.0)), 9, 0.6), M(24, 5, 2, 72, 0.8)),
             (P((2, 1, 40, 16), 70, 4, (3, 32, 8), 3.0), M(48, 6, 4, 32)),
-            (LA(3, 16, 8, 48, 40, 40, R(8, 300.0)), None)]),
+            (LA(3, 16, 8, 48, 40, 40, R(8, 300.0)), None)], scale=0.2),
         # nothing is a multiple of four
         "odd": lambda: c(130, 77, [
             (P((5, 1, 11, 9), 13, 2, (3, 7, 5), 5.0, (0.7, 1.9)), D(33)),

@@ -145,8 +145,7 @@ def test_a_conspicuous_key_is_seen_exactly_inside_the_window(hm, tmp_path, name,
     """One token that every query looks for, at page borders and among the kept first tokens: its value comes back up to the window's
     last place and not one further, in prompts and in decoding."""
     cfg = model(name)
-    if layer > 0:
-        cfg["layers"] = [cfg["layers"][layer]]
+    cfg["layers"] = [cfg["layers"][layer]]
     w0 = {k.replace(f"l{layer}.", "l0."): v for k, v in weights(name).items() if k[0] != "l" or k.startswith(f"l{layer}.")}
     w = conspicuous(cfg, w0, 0, 7, part)
     o = Oracle(cfg, {k: synth.bf16_to_f32(v) for k, v in w.items()}, cache_round=bf16_round if dtype == "BF16" else None)
@@ -159,7 +158,9 @@ def test_a_conspicuous_key_is_seen_exactly_inside_the_window(hm, tmp_path, name,
         with_it = ids[:at] + [7] + ids[at + 1 :]
         want = o.forward(with_it)
         changed = np.abs(want - without).max(1) / np.abs(want).max()
-        assert changed[at + size - 1] > 1e-2 and (at < keep or part or changed[at + size] < 1e-6)  # (a linear state forgets slowly)
+        assert changed[at + size - 1] > 1e-2
+        if not part and at >= keep:  # (a linear state forgets slowly, and a convolution passes a key on)
+            assert changed[at + size] < 0.1 * changed[at + size - 1] and changed[at + size + 1] < 1e-6  # the next token's bigram has changed as well
         m.init_kv_cache(n + 20, batch=1, kv_dtype=hm.DType[dtype])
         cut = at + size - 6
         got = run_portions(m, with_it[:cut], [cut - 3, 3])
