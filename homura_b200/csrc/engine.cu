@@ -77,8 +77,7 @@ int Engine::create(const ModelSpec& spec, int device, bool strict_f32, Engine** 
         for (const LayerSpec& l : spec.layers) {
             e->qdim_ = std::max(e->qdim_, l.heads * std::max(l.vdim, l.paged_kv() ? l.dim : l.q_rank ? l.q_stride() : 0));
             if (l.latent_rank() > 1024) return bad("kv_rank (with rot_dim) must be at most 1024");
-            GlaShape g;
-            if (l.mixer == MIX_PARALLEL && !gla_shape(l.lin_dim, l.lin_vdim, &g)) return bad("linear attention heads have at most 1024 key and 512 value elements");
+            if (l.mixer == MIX_PARALLEL && (l.lin_dim > GLA_MAX_DIM || l.lin_vdim > GLA_MAX_VDIM)) return bad("linear attention heads have at most 1024 key and 512 value elements");
             if (l.experts > 1024) return bad("a mixture has at most 1024 experts");
         }
     } else {

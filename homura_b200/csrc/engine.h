@@ -75,7 +75,6 @@ struct LayerW {
     float *lin_norm = nullptr, *lin_up = nullptr, *lin_bias = nullptr;  // linear attention: result norm, decay up-projection [heads][rank][dim], its bias
     LinearW uq;                          // queries out of their latent
     double* turns = nullptr;             // rotation, turns per position of every pair
-    GlaShape gla{};
     size_t conv_at = 0, gla_at = 0;      // this layer's part of a sequence's state, in floats
 };
 

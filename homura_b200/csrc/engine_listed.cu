@@ -255,7 +255,7 @@ int Engine::alloc_listed_cache(int batch, size_t n_pages) {
         w.conv_at = state_floats_;
         if (s.conv > 1) state_floats_ += ((size_t)(s.conv - 1) * (s.heads * s.dim + s.kv_heads * (s.dim + s.vdim)) + 3) / 4 * 4;
         w.gla_at = state_floats_;
-        if (s.mixer == MIX_PARALLEL) state_floats_ += s.lin_heads * w.gla.state_floats();
+        if (s.mixer == MIX_PARALLEL) state_floats_ += s.lin_heads * gla_state_floats(s.lin_dim, s.lin_vdim);
     }
     if (state_floats_) {
         HM_CUDA(cudaMalloc(&state_, batch * state_floats_ * 4));

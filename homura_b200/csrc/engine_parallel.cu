@@ -290,7 +290,6 @@ int Engine::finalize_parallel() {
             HM_CUDA(cudaMalloc(&w.turns, t.size() * 8));
             HM_CUDA(cudaMemcpy(w.turns, t.data(), t.size() * 8, cudaMemcpyHostToDevice));
         }
-        if (s.mixer == MIX_PARALLEL) gla_shape(s.lin_dim, s.lin_vdim, &w.gla);
     }
     return HM_OK;
 }
@@ -377,7 +376,6 @@ SideArgs Engine::side_args(int l, int M, bool tall, const ParallelColumns& c, co
     if (s.mixer == MIX_PARALLEL) {
         a.has_gla = 1;
         GlaArgs& g = a.gla;
-        g.shape = w.gla;
         g.heads = s.lin_heads;
         g.dim = s.lin_dim;
         g.vdim = s.lin_vdim;
@@ -403,6 +401,7 @@ SideArgs Engine::side_args(int l, int M, bool tall, const ParallelColumns& c, co
         g.M = M;
         g.runs = runs;
         g.longest_run = longest;
+        g.err_flag = err_flag_;
         g.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
         g.out = cat_;
         g.ld_out = cat_ld_;
@@ -484,7 +483,7 @@ int Engine::enqueue_parallel_layer(int l, int M, const int32_t* row_pos, const i
         if (rc) return rc;
     }
     if (want(PC_KV_WRITE)) {
-        ce = launch_side(side_args(l, M, tall, c, row_pos, row_seq), stream_, pdl_);
+        ce = launch_side(side_args(l, M, tall, c, row_pos, row_seq), sm_count_, stream_, pdl_);
         if (ce != cudaSuccess) return cuda_fail(ce, "side launch");
         ++*launches;
         if (experts_seen_ && moe) {

@@ -1,6 +1,7 @@
 // Gated linear attention: per head a state S [dim x vdim] in f32 that every token of a sequence first shrinks, row by row, and then
-// joins,  S <- diag(alpha) S + k v^T,  o = S^T q.  A CTA of 256 threads keeps a head's state in registers while it walks through a
-// run's tokens (gla.cuh); between passes the state lives in the order of those registers.
+// joins,  S <- diag(alpha) S + k v^T,  o = S^T q.  In passes over runs of tokens the CTAs of a cluster share a head's columns and keep
+// them in registers while they walk through a run; in passes of single tokens a head's state goes through a CTA's shared memory
+// (gla.cuh).  Between passes the state lies column by column in memory, whatever the shape of the launches.
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -11,17 +12,23 @@ namespace hm {
 
 constexpr int GLA_THREADS = 256;
 
-// How a head's state is dealt out: `lanes` threads share a column, each with `rows` of its padded rows; a CTA holds `cols` columns at
-// a time and goes through `slices` of them.
+// How a launch deals out a head's state: `cluster` CTAs take `share` columns each and go through them in `slices` of `cols`; `lanes`
+// threads share a column, each with `rows` of its rows.
 struct GlaShape {
-    int rows = 0, lanes = 1, cols = 0, slices = 0;
-    __host__ __device__ int padded_dim() const { return rows * lanes; }
-    __host__ __device__ size_t state_floats() const { return (size_t)slices * rows * GLA_THREADS; }  // per head
+    int cluster, share, slices, cols, lanes, rows;
 };
-bool gla_shape(int dim, int vdim, GlaShape* out);  // false: the sizes are not covered
+constexpr int GLA_MAX_CLUSTER = 8;
+constexpr int GLA_UP_SMEM = 8192;        // floats of a head's decay projection that are staged ahead of the dependency
+constexpr int GLA_TOKEN_DIM = 256;       // single tokens: largest key size, and bytes of a head's state, that go through shared memory
+constexpr int GLA_TOKEN_BYTES = 96 * 1024;
+// heads: (run, head) pairs of the launch.
+GlaShape gla_shape(int dim, int vdim, int heads, int sm_count);
+__host__ __device__ __forceinline__ int gla_pad(int dim) { return (dim + 3) & ~3; }
+__host__ __device__ __forceinline__ size_t gla_state_floats(int dim, int vdim) { return (size_t)vdim * gla_pad(dim); }  // per head
+constexpr int GLA_MAX_DIM = 1024, GLA_MAX_VDIM = 512;
 
 struct GlaArgs {
-    GlaShape shape;
+    GlaShape shape;          // filled in by the launcher, like step
     int heads, dim, vdim, rank;
     // columns of the layer's input projection [M][ld]: queries, keys [heads * dim], values, output gate [heads * vdim], decay latent [rank]
     const float* raw;
@@ -32,7 +39,7 @@ struct GlaArgs {
     float inv_tau;
     const float* norm_w;     // [vdim]: every head's result is RMS-normed, times the silu of the gate
     float eps, out_scale;
-    float* state;            // [sequence][heads][state_floats], sequences seq_stride floats apart; position 0 starts from zero
+    float* state;            // [sequence][heads][vdim][gla_pad(dim)], sequences seq_stride floats apart; position 0 starts from zero
     size_t seq_stride;
     const int32_t *row_pos, *row_seq;
     int M;
@@ -43,8 +50,8 @@ struct GlaArgs {
     int ld_out, out_off;
     unsigned char* xp;
     int xp_mpad;
-    int step;                // tokens staged at a time (gla_smem fills it in)
+    int step;                // tokens staged at a time
+    int* err_flag;
 };
-size_t gla_smem(GlaArgs* a);  // dynamic shared memory of a CTA
 
 }  // namespace hm

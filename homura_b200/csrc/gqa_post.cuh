@@ -26,11 +26,10 @@ __device__ __forceinline__ void rotate_pairs(float* buf, int half, const double*
 
 // Row m of one head slot ([heads] queries, [kv_heads] keys, [kv_heads] values).  part_q / part_k: sums of squares of the whole
 // projections (QKN_ALL); first: the first row of m's run.
-__device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int slot, int first, float part_q, float part_k, float* buf) {
+__device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int slot, int first, int pos, int seq, size_t page, float part_q, float part_k, float* buf) {
     const int lane = threadIdx.x & 31;
     const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
-    const int pos = a.row_pos[m], seq = a.row_seq[m], t = pos % GQA_PAGE;
-    const size_t page = (size_t)a.pool.page_table[(size_t)seq * a.pool.max_pages + pos / GQA_PAGE];
+    const int t = pos % GQA_PAGE;
     const bool is_v = slot >= a.heads + G, is_q = slot < a.heads;
     const int h = is_v ? slot - a.heads - G : is_q ? slot : slot - a.heads, n = is_v ? vdim : dim;
     const int ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n;  // first channel
@@ -43,12 +42,17 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
             float v = ld_cg_f32(x + d);
             if (a.taps > 0) {
                 const float* w = a.conv_w + (size_t)(ch0 + d) * a.taps;
+                auto input = [&](int j) { return m - j >= first ? ld_cg_f32(x + d - (ptrdiff_t)j * a.ld) : ld_cg_f32(state + (size_t)((pos - j) % (a.taps - 1)) * channels + d); };
+                const int back = min(a.taps - 1, pos);
+                float u[3] = {0.f, 0.f, 0.f};  // requested together
+#pragma unroll
+                for (int j = 1; j <= 3; ++j)
+                    if (j <= back) u[j - 1] = input(j);
                 v *= __ldg(w + a.taps - 1);
-                for (int j = 1; j < a.taps; ++j) {
-                    if (j > pos) break;
-                    const float u = m - j >= first ? ld_cg_f32(x + d - (ptrdiff_t)j * a.ld) : ld_cg_f32(state + (size_t)((pos - j) % (a.taps - 1)) * channels + d);
-                    v = fmaf(u, __ldg(w + a.taps - 1 - j), v);
-                }
+#pragma unroll
+                for (int j = 1; j <= 3; ++j)
+                    if (j <= back) v = fmaf(u[j - 1], __ldg(w + a.taps - 1 - j), v);
+                for (int j = 4; j <= back; ++j) v = fmaf(input(j), __ldg(w + a.taps - 1 - j), v);
             }
             buf[d] = v;
         }
@@ -123,6 +127,10 @@ __device__ __forceinline__ void gqa_post_block(const GqaPostArgs& a, int m, int 
     const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
     const int slot0 = blk * POST_WARPS, slot = slot0 + warp;
     __shared__ float s_part[2][POST_WARPS];
+    // positions and pages do not depend on the launch in front
+    auto page_of = [&](int seq, int pos) { return (size_t)a.pool.page_table[(size_t)seq * a.pool.max_pages + pos / GQA_PAGE]; };
+    const int pos = a.row_pos[m], seq = a.row_seq[m];
+    const size_t page = page_of(seq, pos);
     pdl_wait();
     float sq = 0.f, sk = 0.f;
     if (a.qk_norm == QKN_ALL) {  // every CTA sums the squares of the part it needs
@@ -156,24 +164,23 @@ __device__ __forceinline__ void gqa_post_block(const GqaPostArgs& a, int m, int 
     if (slot >= gqa_post_slots(a)) return;
     float* buf = smem + warp * gqa_post_buf(a);
     if (a.taps <= 1) {
-        gqa_post_row(a, m, slot, m, sq, sk, buf);
+        gqa_post_row(a, m, slot, m, pos, seq, page, sq, sk, buf);
         return;
     }
     int first, end;
     a.runs.find(m, first, end);
     const int keep = a.taps - 1;
     if (m > first && m < first + keep) return;  // served by the warp of the run's first row
-    gqa_post_row(a, m, slot, first, sq, sk, buf);
+    gqa_post_row(a, m, slot, first, pos, seq, page, sq, sk, buf);
     if (m > first) return;
-    for (int r = first + 1; r < min(end, first + keep); ++r) gqa_post_row(a, r, slot, first, 0.f, 0.f, buf);
+    for (int r = first + 1; r < min(end, first + keep); ++r) gqa_post_row(a, r, slot, first, pos + r - first, seq, page_of(seq, pos + r - first), 0.f, 0.f, buf);
     // the run's last inputs replace the kept ones (a lane keeps the channels that it has read)
     const bool is_v = slot >= a.heads + G, is_q = slot < a.heads;
     const int h = is_v ? slot - a.heads - G : is_q ? slot : slot - a.heads, n = is_v ? vdim : dim, ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n, channels = nq + nk + G * vdim;
-    float* state = a.conv_state + (size_t)a.row_seq[m] * a.conv_stride + ch0;
-    for (int r = max(first, end - keep); r < end; ++r) {
-        const int p = a.row_pos[r];
-        for (int d = lane; d < n; d += 32) state[(size_t)(p % keep) * channels + d] = ld_cg_f32(a.raw + (size_t)r * a.ld + ch0 + d);
-    }
+    float* state = a.conv_state + (size_t)seq * a.conv_stride + ch0;
+    for (int r = max(first, end - keep); r < end; ++r)
+#pragma unroll 4
+        for (int d = lane; d < n; d += 32) state[(size_t)((pos + r - first) % keep) * channels + d] = ld_cg_f32(a.raw + (size_t)r * a.ld + ch0 + d);
 }
 
 }  // namespace hm

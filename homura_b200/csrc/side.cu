@@ -90,16 +90,17 @@ __device__ __forceinline__ void query_latent_block(const SideArgs& a, int m, flo
     }
 }
 
-// RD: state rows per thread of the linear attention, 0: there is none
+// RD: state rows per thread of the linear attention, 0: there is none, -1: single tokens, states in shared memory
 template <int RD>
-__global__ void __launch_bounds__(THREADS) side_kernel(const __grid_constant__ SideArgs a) {
+__global__ void __launch_bounds__(THREADS, RD > 32 ? 1 : RD > 0 ? 2 : 3) side_kernel(const __grid_constant__ SideArgs a) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float part[WARPS];
     pdl_launch_dependents();
     int b = blockIdx.x;
-    if constexpr (RD > 0) {
+    if constexpr (RD != 0) {
         if (b < a.n_gla) {
-            gla_block<RD>(a.gla, b % a.gla.heads, b / a.gla.heads, sm);
+            if constexpr (RD > 0) gla_block<RD>(a.gla, b, sm);
+            else gla_token_block(a.gla, b, sm, part);
             return;
         }
         b -= a.n_gla;
@@ -122,8 +123,12 @@ __global__ void __launch_bounds__(THREADS) side_kernel(const __grid_constant__ S
         return;
     }
     b -= a.n_act;
-    if (b < a.n_route) route_block(a, b, sm);
-    else normed_block(a, b - a.n_route, part);
+    if (b < a.n_route) {
+        route_block(a, b, sm);
+        return;
+    }
+    b -= a.n_route;
+    if (b < a.n_normed) normed_block(a, b, part);  // (the rest fills the last cluster)
 }
 
 __global__ void __launch_bounds__(THREADS) sum_norm_kernel(const SumNormArgs a) {
@@ -174,7 +179,7 @@ __global__ void __launch_bounds__(THREADS) sum_norm_kernel(const SumNormArgs a) 
 }
 
 template <typename K, typename A>
-cudaError_t launch(K kern, unsigned blocks, size_t smem, cudaStream_t st, bool pdl, const A& args) {
+cudaError_t launch(K kern, unsigned blocks, size_t smem, int cluster, cudaStream_t st, bool pdl, const A& args) {
     const cudaError_t e = ensure_dyn_smem(kern, smem);
     if (e != cudaSuccess) return e;
     cudaLaunchConfig_t cfg = {};
@@ -182,50 +187,71 @@ cudaError_t launch(K kern, unsigned blocks, size_t smem, cudaStream_t st, bool p
     cfg.blockDim = dim3(THREADS);
     cfg.dynamicSmemBytes = smem;
     cfg.stream = st;
-    cudaLaunchAttribute at[1];
-    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    at[0].val.programmaticStreamSerializationAllowed = 1;
+    cudaLaunchAttribute at[2];
+    int n = 0;
+    if (pdl) {
+        at[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        at[n].val.programmaticStreamSerializationAllowed = 1;
+        ++n;
+    }
+    if (cluster > 1) {
+        at[n].id = cudaLaunchAttributeClusterDimension;
+        at[n].val.clusterDim.x = (unsigned)cluster;
+        at[n].val.clusterDim.y = at[n].val.clusterDim.z = 1;
+        ++n;
+    }
     cfg.attrs = at;
-    cfg.numAttrs = pdl ? 1 : 0;
+    cfg.numAttrs = n;
     return cudaLaunchKernelEx(&cfg, kern, args);
 }
 
 }  // namespace
 
-bool gla_shape(int dim, int vdim, GlaShape* out) {
-    if (dim < 1 || vdim < 1 || dim > 1024 || vdim > 512) return false;
-    GlaShape s;
+GlaShape gla_shape(int dim, int vdim, int heads, int sm_count) {
+    GlaShape s{};
+    // a head's columns are spread over CTAs until they fill the SMs, as long as every thread has rows, and over enough of them that a
+    // thread holds at most 32 rows
+    s.cluster = 1;
+    auto share = [&](int cluster) { return ((vdim + cluster - 1) / cluster + 7) / 8 * 8; };
+    while (s.cluster < GLA_MAX_CLUSTER && vdim / (2 * s.cluster) >= 8 &&
+           ((2 * s.cluster * heads <= sm_count && GLA_THREADS / share(2 * s.cluster) * 4 <= gla_pad(dim)) || (size_t)gla_pad(dim) * vdim / s.cluster > 32 * GLA_THREADS))
+        s.cluster *= 2;
+    s.share = share(s.cluster);
     s.cols = 8;
-    while (s.cols < vdim && s.cols < GLA_THREADS) s.cols *= 2;
-    for (; s.cols >= 8; s.cols /= 2) {
-        s.lanes = GLA_THREADS / s.cols;
-        if (s.lanes * 64 >= dim) break;
-    }
-    s.rows = 8;
+    while (s.cols < s.share && s.cols < GLA_THREADS) s.cols *= 2;
+    for (; s.cols > 8; s.cols /= 2)
+        if (GLA_THREADS / s.cols * 64 >= dim) break;
+    s.lanes = GLA_THREADS / s.cols;
+    s.rows = 4;
     while (s.rows * s.lanes < dim) s.rows *= 2;
-    s.slices = (vdim + s.cols - 1) / s.cols;
-    *out = s;
-    return true;
+    s.slices = (s.share + s.cols - 1) / s.cols;
+    return s;
 }
 
-size_t gla_smem(GlaArgs* a) {
-    const size_t up = a->rank * a->dim <= GLA_UP_SMEM ? (size_t)(a->rank * a->dim + 3) / 4 * 4 : 0;
-    const int rows = a->runs.n ? a->longest_run : 1;
-    for (a->step = std::min(16, rows);; a->step /= 2) {
-        const size_t bytes = sizeof(float) * (up + (size_t)a->step * (3 * a->shape.padded_dim() + a->shape.cols + a->rank) + (size_t)(a->shape.slices > 1 ? rows : a->step) * a->vdim);
-        if (bytes <= 160 * 1024 || a->step == 1) return bytes;
-    }
-}
-
-cudaError_t launch_side(const SideArgs& a_in, cudaStream_t st, bool pdl) {
+cudaError_t launch_side(const SideArgs& a_in, int sm_count, cudaStream_t st, bool pdl) {
     SideArgs a = a_in;
     if (a.M < 1 || a.M > GQA_MAX_ROWS) return cudaErrorInvalidValue;
     const int runs = a.gla.runs.n ? a.gla.runs.n : a.M;
     size_t smem = 0;
     a.n_gla = a.n_post = a.n_latent = a.n_act = a.n_route = a.n_normed = 0;
+    int cluster = 1, kind = 0;
     if (a.has_gla) {
-        a.n_gla = runs * a.gla.heads;
-        smem = std::max(smem, gla_smem(&a.gla));
+        GlaArgs& g = a.gla;
+        if (g.dim > GLA_MAX_DIM || g.vdim > GLA_MAX_VDIM) return cudaErrorInvalidValue;
+        const int rows = g.runs.n ? g.longest_run : 1;
+        if (rows == 1 && g.dim <= GLA_TOKEN_DIM && gla_state_floats(g.dim, g.vdim) * 4 <= GLA_TOKEN_BYTES) {
+            kind = -1;
+            a.n_gla = a.M * g.heads;
+            smem = (size_t)gla_token_smem(g).total * 4;
+        } else {
+            g.shape = gla_shape(g.dim, g.vdim, runs * g.heads, sm_count);
+            kind = g.shape.rows;
+            cluster = g.shape.cluster;
+            a.n_gla = runs * g.heads * cluster;
+            for (g.step = rows; g.step > 1 && (size_t)gla_smem(g, rows).total * 4 > 110 * 1024; g.step = (g.step + 1) / 2) {
+            }
+            smem = (size_t)gla_smem(g, rows).total * 4;
+        }
     }
     if (a.has_post) {
         a.n_post = a.M * gqa_post_blocks(a.post);
@@ -238,20 +264,22 @@ cudaError_t launch_side(const SideArgs& a_in, cudaStream_t st, bool pdl) {
         smem = std::max(smem, 2 * sizeof(float) * (size_t)a.mlp.route.n_out);
     }
     if (a.mlp.normed) a.n_normed = a.M;
-    const unsigned blocks = (unsigned)(a.n_gla + a.n_post + a.n_latent + a.n_act + a.n_route + a.n_normed);
-    switch (a.has_gla ? a.gla.shape.rows : 0) {
-        case 0: return launch(side_kernel<0>, blocks, smem, st, pdl, a);
-        case 8: return launch(side_kernel<8>, blocks, smem, st, pdl, a);
-        case 16: return launch(side_kernel<16>, blocks, smem, st, pdl, a);
-        case 32: return launch(side_kernel<32>, blocks, smem, st, pdl, a);
-        case 64: return launch(side_kernel<64>, blocks, smem, st, pdl, a);
+    const unsigned blocks = (unsigned)((a.n_gla + a.n_post + a.n_latent + a.n_act + a.n_route + a.n_normed + cluster - 1) / cluster * cluster);
+    switch (kind) {
+        case -1: return launch(side_kernel<-1>, blocks, smem, cluster, st, pdl, a);
+        case 4: return launch(side_kernel<4>, blocks, smem, cluster, st, pdl, a);
+        case 0: return launch(side_kernel<0>, blocks, smem, cluster, st, pdl, a);
+        case 8: return launch(side_kernel<8>, blocks, smem, cluster, st, pdl, a);
+        case 16: return launch(side_kernel<16>, blocks, smem, cluster, st, pdl, a);
+        case 32: return launch(side_kernel<32>, blocks, smem, cluster, st, pdl, a);
+        case 64: return launch(side_kernel<64>, blocks, smem, cluster, st, pdl, a);
         default: return cudaErrorInvalidValue;
     }
 }
 
 cudaError_t launch_sum_norm(const SumNormArgs& a, cudaStream_t st, bool pdl) {
     if (!a.w && !a.parts) return cudaSuccess;
-    return launch(sum_norm_kernel, (unsigned)(a.w ? tc_mpad(a.M) : a.M), sizeof(float) * (size_t)((a.W + 7) / 8 * 8), st, pdl, a);
+    return launch(sum_norm_kernel, (unsigned)(a.w ? tc_mpad(a.M) : a.M), sizeof(float) * (size_t)((a.W + 7) / 8 * 8), 1, st, pdl, a);
 }
 
 }  // namespace hm

@@ -52,7 +52,7 @@ struct SideArgs {
     // blocks of the parts, in launch order (filled in by the launcher)
     int n_gla, n_post, n_latent, n_act, n_route, n_normed;
 };
-cudaError_t launch_side(const SideArgs& a, cudaStream_t st, bool pdl);
+cudaError_t launch_side(const SideArgs& a, int sm_count, cudaStream_t st, bool pdl);
 
 // Sums the parts of a sublayer's result into the residual and packs its RMS norm (weight w, null: nothing is packed) as the activation image of the next projection.
 struct SumNormArgs {

@@ -243,6 +243,24 @@ def test_mixed_batches_and_reused_pages(hm, engines, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["F32", "BF16"])
+@pytest.mark.parametrize("name", ["large", "parallel"])
+def test_many_sequences_in_a_pass(hm, engines, name, dtype):
+    """Forty sequences: a prompt each, then passes that mix single tokens with portions, then the captured step."""
+    m = engines(name, dtype)
+    m.init_kv_cache(64, batch=40, kv_dtype=hm.DType[dtype])
+    full = [expected(name, dtype, 100 + b % 4, 24) for b in range(40)]
+    m.step([(b, full[b][0][: 3 + b % 5], []) for b in range(40)], want_logits=False)
+    at = [3 + b % 5 for b in range(40)]
+    for wide in (0, 1):
+        n = [1 + (b % 3 if wide else 0) for b in range(40)]
+        got, _, _ = m.step([(b, full[b][0][at[b] : at[b] + n[b]], [n[b] - 1]) for b in range(40)])
+        at = [a + k for a, k in zip(at, n)]
+        close(got, np.stack([full[b][1][at[b] - 1] for b in range(40)]), dtype, "logits of many sequences")
+    lg, _ = m.decode_step([full[b][0][at[b]] for b in range(40)])
+    close(lg, np.stack([full[b][1][at[b]] for b in range(40)]), dtype, "logits of a captured step of many sequences")
+
+
+@pytest.mark.parametrize("dtype", ["F32", "BF16"])
 def test_a_slot_starts_from_nothing(hm, engines, dtype):
     """A request that takes over a slot sees neither the old keys nor the old states."""
     m = engines("mixed", dtype)
