@@ -801,7 +801,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) 
 }  // namespace
 
 int tc_mpad(int M) { return M <= 16 ? 16 : M <= 32 ? 32 : 64; }
-// Stages of the ring.  Launches of one wave (at most one CTA per SM: every layer projection of the 0.5-1.5 B
+// Stages of the ring.  Launches of one wave (at most one CTA per SM: most layer projections of the 0.5-1.5 B
 // models) take the deep ring, because the main loop of a lone CTA is bound by the bytes it keeps in flight
 // (measured on the 1.5 B x 64 step: 2.02 ms with 4 stages, 2.10 with 3, 2.30 with 2).  Launches of several
 // waves (the LM head: 1187 blocks) take two stages, which lets two CTAs share an SM (81 KB and 256 TMEM columns
@@ -875,7 +875,7 @@ static cudaError_t launch_gemm_tc_v(const TcArgs& a_in, cudaStream_t st, bool pd
             busy = nblk *= a.ex.parts;
         }
     }
-    const bool multi_wave = (long)busy * (a.ksplit > 1 ? a.ksplit : 1) >= 2L * sms;
+    const bool multi_wave = (long)busy * (a.ksplit > 1 ? a.ksplit : 1) > sms;
     a.nstage = tc_nstage(a.mpad, multi_wave);
     a.tmem_cols = a.mpad == 16 ? 64 : a.mpad == 32 ? 128 : 256;  // power of two >= 3 * mpad
     const bool cl = a.ksplit > 1;

@@ -249,34 +249,41 @@ __device__ __forceinline__ void gla_token_block(const GlaArgs& a, int block, flo
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int head = block % a.heads, m = block / a.heads, dim = a.dim, vdim = a.vdim, rank = a.rank, ldd = gla_pad(dim), ld4 = ldd / 4;
     const GlaTokenSmem lay = gla_token_smem(a);
-    __shared__ uint64_t landed;
+    constexpr uint32_t CHUNK = 16384;
+    __shared__ uint64_t landed[(GLA_TOKEN_BYTES + CHUNK - 1) / CHUNK], up_landed;  // a barrier per piece of the copy
     __shared__ volatile int s_abort;
+    const uint32_t bytes = (uint32_t)(vdim * ldd * 4);
+    const float* up = a.up + (size_t)head * rank * dim;
+    const bool up_staged = rank * dim <= GLA_UP_SMEM, up_bulk = up_staged && (rank * dim & 3) == 0;
+    if (tid == 0) {
+        for (uint32_t i = 0; i * CHUNK < bytes; ++i) mb_init(&landed[i], 1);
+        mb_init(&up_landed, 1);
+        s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        if (up_bulk) {
+            mb_expect_tx(&up_landed, (uint32_t)(rank * dim * 4));
+            bulk_copy(sm + lay.up, up, (uint32_t)(rank * dim * 4), &up_landed);
+        }
+    }
     const int seq = a.row_seq[m], pos = a.row_pos[m];
     float* const state = a.state + (size_t)seq * a.seq_stride + (size_t)head * vdim * ldd;
     auto fetch = [&]() {
-        const uint32_t bytes = (uint32_t)(vdim * ldd * 4);
-        mb_expect_tx(&landed, bytes);
-        for (uint32_t o = 0; o < bytes; o += 16384u) bulk_copy(reinterpret_cast<char*>(sm + lay.state) + o, reinterpret_cast<const char*>(state) + o, min(16384u, bytes - o), &landed);
-    };
-    if (tid == 0) {
-        mb_init(&landed, 1);
-        s_abort = 0;
-        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-        if (a.early && pos > 0) fetch();
-    }
-    const float* up = a.up + (size_t)head * rank * dim;
-    if (rank * dim <= GLA_UP_SMEM) {
-        if ((dim & 3) == 0) {
-#pragma unroll 4
-            for (int i = tid; i < rank * dim / 4; i += GLA_THREADS) reinterpret_cast<float4*>(sm + lay.up)[i] = __ldg(reinterpret_cast<const float4*>(up) + i);
-        } else {
-            for (int i = tid; i < rank * dim; i += GLA_THREADS) sm[lay.up + i] = __ldg(up + i);
+        for (uint32_t i = 0, o = 0; o < bytes; ++i, o += CHUNK) {
+            mb_expect_tx(&landed[i], min(CHUNK, bytes - o));
+            bulk_copy(reinterpret_cast<char*>(sm + lay.state) + o, reinterpret_cast<const char*>(state) + o, min(CHUNK, bytes - o), &landed[i]);
         }
-        up = sm + lay.up;
-    }
+    };
+    if (tid == 0 && a.early && pos > 0) fetch();
+    // weights of this thread's first decay and result
+    const float bias0 = tid < dim ? __ldg(a.bias + (size_t)head * dim + tid) : 0.f, norm0 = tid < vdim ? __ldg(a.norm_w + tid) : 0.f;
+    if (up_staged && !up_bulk)
+        for (int i = tid; i < rank * dim; i += GLA_THREADS) sm[lay.up + i] = __ldg(up + i);
+    if (up_staged) up = sm + lay.up;
     pdl_wait();
     if (tid == 0 && !a.early && pos > 0) fetch();
     const float* raw = a.raw + (size_t)m * a.ld;
+    // everything of the row is requested before the first use
+    const float lat0 = tid < rank ? ld_cg_f32(raw + a.a_off + tid) : 0.f, v0 = tid < vdim ? ld_cg_f32(raw + a.v_off + (size_t)head * vdim + tid) : 0.f, g0 = tid < vdim ? ld_cg_f32(raw + a.g_off + (size_t)head * vdim + tid) : 0.f;
     // lanes of a column: a power of two, so that several short columns share a warp
     const int LC = ld4 >= 32 ? 32 : 1 << (32 - __clz(ld4 - 1)), sub = lane / LC, piece = lane - sub * LC, CW = 32 / LC;
     float4 q[NJ], k[NJ], al[NJ];
@@ -293,32 +300,42 @@ __device__ __forceinline__ void gla_token_block(const GlaArgs& a, int block, flo
             q[j] = make_float4(ld_cg_f32(qr), d + 1 < dim ? ld_cg_f32(qr + 1) : 0.f, d + 2 < dim ? ld_cg_f32(qr + 2) : 0.f, d + 3 < dim ? ld_cg_f32(qr + 3) : 0.f);
             k[j] = make_float4(ld_cg_f32(kr), d + 1 < dim ? ld_cg_f32(kr + 1) : 0.f, d + 2 < dim ? ld_cg_f32(kr + 2) : 0.f, d + 3 < dim ? ld_cg_f32(kr + 3) : 0.f);
         }
-        q[j] = make_float4(q[j].x * a.q_scale, q[j].y * a.q_scale, q[j].z * a.q_scale, q[j].w * a.q_scale);
     }
-    for (int i = tid; i < rank; i += GLA_THREADS) sm[lay.lat + i] = ld_cg_f32(raw + a.a_off + i);
-    for (int i = tid; i < vdim; i += GLA_THREADS) {
+    if (tid < rank) sm[lay.lat + tid] = lat0;
+    if (tid < vdim) {
+        sm[lay.v + tid] = v0;
+        sm[lay.gate + tid] = g0;
+    }
+    for (int i = GLA_THREADS + tid; i < rank; i += GLA_THREADS) sm[lay.lat + i] = ld_cg_f32(raw + a.a_off + i);
+    for (int i = GLA_THREADS + tid; i < vdim; i += GLA_THREADS) {
         sm[lay.v + i] = ld_cg_f32(raw + a.v_off + (size_t)head * vdim + i);
         sm[lay.gate + i] = ld_cg_f32(raw + a.g_off + (size_t)head * vdim + i);
     }
     __syncthreads();
+    const bool up_ok = !up_bulk || mb_wait(&up_landed, 0, a.err_flag, &s_abort);  // bounded, like the waits below
     for (int d = tid; d < ldd; d += GLA_THREADS) {
         float v = 0.f;
-        if (d < dim) {
+        if (d < dim && up_ok) {
             float z = 0.f;
 #pragma unroll 8
             for (int r = 0; r < rank; ++r) z = fmaf(up[r * dim + d], sm[lay.lat + r], z);
-            v = gla_decay(z + __ldg(a.bias + (size_t)head * dim + d), a.inv_tau);
+            v = gla_decay(z + (d == tid ? bias0 : __ldg(a.bias + (size_t)head * dim + d)), a.inv_tau);
         }
         sm[lay.alpha + d] = v;
     }
     __syncthreads();
 #pragma unroll
-    for (int j = 0; j < NJ; ++j)
+    for (int j = 0; j < NJ; ++j) {
         if (j * 32 + piece < ld4) al[j] = reinterpret_cast<const float4*>(sm + lay.alpha)[j * 32 + piece];
-    const bool ok = pos == 0 || mb_wait(&landed, 0, a.err_flag, &s_abort);  // bounded
+        q[j] = make_float4(q[j].x * a.q_scale, q[j].y * a.q_scale, q[j].z * a.q_scale, q[j].w * a.q_scale);
+    }
+    bool ok = true;
+    uint32_t seen = 0;  // pieces that have landed
     const float4* tile = reinterpret_cast<const float4*>(sm + lay.state);
     constexpr int U = 4;  // columns whose sums go side by side
     for (int g = warp * U; g * CW < vdim; g += GLA_THREADS / 32 * U) {
+        if (pos > 0)  // every piece is waited for, so that none is on its way when the CTA ends; the waits are bounded
+            for (const uint32_t last = min(bytes, (uint32_t)((g + U) * CW * ldd * 4)); seen * CHUNK < last; ++seen) ok = mb_wait(&landed[seen], 0, a.err_flag, &s_abort) && ok;
         float o[U];
 #pragma unroll
         for (int u = 0; u < U; ++u) {
@@ -353,24 +370,26 @@ __device__ __forceinline__ void gla_token_block(const GlaArgs& a, int block, flo
     for (int c = tid; c < vdim; c += GLA_THREADS) s = fmaf(sm[lay.o + c], sm[lay.o + c], s);
     s = warp_sum(s);
     if (lane == 0) part[warp] = s;
+    for (int c = tid; c < vdim; c += GLA_THREADS) sm[lay.v + c] = c == tid ? norm0 : __ldg(a.norm_w + c);  // the values have been used
     __syncthreads();
     s = 0.f;
 #pragma unroll
     for (int w = 0; w < GLA_THREADS / 32; ++w) s += part[w];
     const float f = 1.0f / sqrtf(s / (float)vdim + a.eps);
     const int k0 = a.out_off + head * vdim;
-    auto value = [&](int c) { return ((sm[lay.o + c] * f) * __ldg(a.norm_w + c)) * gla_silu(sm[lay.gate + c]) * a.out_scale; };
+    auto value = [&](int c, float w) { return ((sm[lay.o + c] * f) * w) * gla_silu(sm[lay.gate + c]) * a.out_scale; };
     if (a.xp && ((vdim | a.out_off) & 7) == 0) {
         for (int c = tid * 8; c < vdim; c += GLA_THREADS * 8) {
             float v[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) v[e] = value(c + e);
+            for (int e = 0; e < 8; ++e) v[e] = value(c + e, sm[lay.v + c + e]);
             tc_xpack_store8(a.xp, a.xp_mpad, m, k0 + c, v);
         }
     } else {
         for (int c = tid; c < vdim; c += GLA_THREADS) {
-            if (a.xp) tc_xpack_store(a.xp, a.xp_mpad, m, k0 + c, value(c));
-            else a.out[(size_t)m * a.ld_out + k0 + c] = value(c);
+            const float v = value(c, sm[lay.v + c]);
+            if (a.xp) tc_xpack_store(a.xp, a.xp_mpad, m, k0 + c, v);
+            else a.out[(size_t)m * a.ld_out + k0 + c] = v;
         }
     }
 }
