@@ -55,6 +55,7 @@ void gemv_pick_cluster(int K, int N, int M, int sm_count, int max_cluster, int* 
     int cs = (2 * sm_count) / nslabs;  // two CTAs per SM resident at once (one per SM measured 1.5x slower on the widest projection)
     if (cs > max_cluster) cs = max_cluster;
     if (cs < 1) cs = 1;
+    if (cs == 1 && nslabs < 2 * sm_count && max_cluster > 1) cs = 2;  // between one and two CTAs per SM: halves even them out
     while (cs > 1 && K / cs < 32) --cs;
     int rps = ((K + cs - 1) / cs + ROWS_PER_PASS - 1) / ROWS_PER_PASS * ROWS_PER_PASS;
     const int max_rps = (12288 / M) / ROWS_PER_PASS * ROWS_PER_PASS;
