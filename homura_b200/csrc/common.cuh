@@ -462,7 +462,7 @@ struct GemvBase {
 
 // The arguments of the kernel's extended variant (gemv_ext.cu): what only some designs need is compiled apart, so that the
 // plain projections, which are latency chains, carry none of it.
-struct GemvArgs : GemvBase {
+struct GemvExt : GemvBase {
     RowNorm gn;          // PRO_GNORM
     SplitRows split;     // PRO_MERGE
     // Grouped projection (block-diagonal weights, e.g. one matrix per attention head): group g owns group_slabs slabs,
@@ -471,9 +471,13 @@ struct GemvArgs : GemvBase {
     const float* out_scale;  // [N] or null (EPI_STORE: the result is multiplied element by element before the residual is added)
     const float* gate;   // EPI_GATE: [M][ld_gate]
     int ld_gate;
+    bool extended() const { return pro == PRO_GNORM || pro == PRO_MERGE || epi == EPI_GATE || epi == EPI_SQRELU || group_slabs != 0 || out_scale != nullptr; }
+};
+// And of the variant behind that (gemv_turn.cu): rotation and capped logits in the epilogue.
+struct GemvArgs : GemvExt {
     TurnedPairs turn;    // EPI_STORE: with turn.turns
     float softcap;       // EPI_LOGITS: > 0: softcap * tanh(logit / softcap)
-    bool extended() const { return turn.turns != nullptr || softcap > 0.f || pro == PRO_GNORM || pro == PRO_MERGE || epi == EPI_GATE || epi == EPI_SQRELU || group_slabs != 0 || out_scale != nullptr; }
+    int variant() const { return turn.turns != nullptr || softcap > 0.f ? 2 : extended() ? 1 : 0; }
 };
 
 struct AttnArgs {
@@ -533,7 +537,8 @@ struct QuantArgs {
 
 // ---- launchers (defined in the .cu files) ----------------------------------------------
 cudaError_t launch_gemv_bf16(const GemvArgs& a, int M, cudaStream_t st, bool pdl);
-cudaError_t launch_gemv_bf16_ext(const GemvArgs& a, int M, cudaStream_t st, bool pdl);  // what launch_gemv_bf16 calls for extended() arguments
+cudaError_t launch_gemv_bf16_ext(const GemvArgs& a, int M, cudaStream_t st, bool pdl);  // what launch_gemv_bf16 calls for variant 1
+cudaError_t launch_gemv_bf16_turn(const GemvArgs& a, int M, cudaStream_t st, bool pdl);  // ... and 2
 
 size_t gemv_partial_floats(int N, int ksplit, int M);
 void gemv_pick_split(int K, int N, int M, int sm_count, int* ksplit, int* rows_per_split);

@@ -251,11 +251,11 @@ __global__ void __launch_bounds__(256) tc_pack_gnorm_kernel(const float* __restr
 __device__ __forceinline__ bool tc_better(float v, int i, float bv, int bi) { return v > bv || (v == bv && i > bi); }
 
 // V: 1 is the extended variant (grouped weights, output scale, gate, squared ReLU, queries split into images), 2 that of mixtures of
-// experts, compiled apart so that the plain projections carry none of it.
+// experts, 3 the extended one with rotation and capped logits, compiled apart so that the plain projections carry none of it.
 template <int V>
 __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, int nblk, int tid, const int* s_pos, const int* s_page) {
     // grouped projections: this block's output columns [n0, n_end)
-    constexpr bool X = V == 1;
+    constexpr bool X = V == 1 || V == 3;
     const int rows = m_hi - m_lo;
     int n0 = nblk * BM, n_end = a.N;
     if constexpr (V == 2) {
@@ -264,9 +264,15 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
             for (int idx = tid; idx < rows * 8; idx += TC_THREADS) {
                 const int m = m_lo + idx / 8, c = (idx % 8) * 8;
                 const float rw = ld_cg_f32(a.ex.weight + (size_t)m * a.ex.n + e);
+                const float *g = tile + m * BM + c, *u = g + 64;
                 float act[8];
+                if (a.ex.act == GLU_CLAMPED) {
 #pragma unroll
-                for (int i = 0; i < 8; ++i) act[i] = rw == 0.f ? 0.f : glu(a.ex.act, tile[m * BM + c + i], tile[m * BM + 64 + c + i], a.ex.limit) * rw;
+                    for (int i = 0; i < 8; ++i) act[i] = rw == 0.f ? 0.f : clamped_glu(g[i], u[i], a.ex.limit) * rw;
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) act[i] = rw == 0.f ? 0.f : glu(a.ex.act, g[i], u[i], a.ex.limit) * rw;
+                }
                 tc_xpack_store8(a.xp_out + (size_t)e * a.ex.img_bytes, a.xp_mpad, m, k0 + c, act);
             }
             return;
@@ -301,9 +307,11 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                         const float4 s0 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c)), s1 = __ldg(reinterpret_cast<const float4*>(a.out_scale + n0 + c + 4));
                         v[0] *= s0.x; v[1] *= s0.y; v[2] *= s0.z; v[3] *= s0.w; v[4] *= s1.x; v[5] *= s1.y; v[6] *= s1.z; v[7] *= s1.w;
                     }
-                    if (a.turn.turns && ok)
+                    if constexpr (V == 3) {
+                        if (a.turn.turns && ok)
 #pragma unroll
-                        for (int e = 0; e < 8; e += 2) turn_pair(a.turn, m, n0 + c + e, v[e], v[e + 1]);
+                            for (int e = 0; e < 8; e += 2) turn_pair(a.turn, m, n0 + c + e, v[e], v[e + 1]);
+                    }
                     if (a.split_xp && n0 + c < a.split_n) {  // 8-element pieces never straddle split_n or an image: both are multiples of 8
                         if (ok) tc_xpack_store8(a.split_xp + (size_t)((n0 + c) / a.split_k) * a.split_bytes, a.xp_mpad, m, (n0 + c) % a.split_k, v);
                         continue;
@@ -345,14 +353,12 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                     if (a.bias) v += __ldg(a.bias + n);
                     if constexpr (X) {
                         if (a.out_scale) v *= __ldg(a.out_scale + n);
-                        if (a.turn.turns) {  // (columns are padded to whole periods, so a pair is in the same block)
-                            float o = tile[m * BM + (c ^ 1)], u = v;
-                            if (c & 1) {
-                                turn_pair(a.turn, m, n - 1, o, u);
-                            } else {
-                                turn_pair(a.turn, m, n, u, o);
+                        if constexpr (V == 3) {
+                            if (a.turn.turns) {  // (columns are padded to whole periods, so a pair is in the same block)
+                                float o = tile[m * BM + (c ^ 1)];
+                                if (c & 1) turn_pair(a.turn, m, n - 1, o, v);
+                                else turn_pair(a.turn, m, n, v, o);
                             }
-                            v = u;
                         }
                         if (a.split_xp && n < a.split_n) {
                             tc_xpack_store(a.split_xp + (size_t)(n / a.split_k) * a.split_bytes, a.xp_mpad, m, n % a.split_k, v);
@@ -421,7 +427,7 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
             }
         }
     } else if (a.epi == EPI_LOGITS) {
-        if constexpr (X) {
+        if constexpr (V == 3) {
             if (a.softcap > 0.f) {
                 for (int idx = tid; idx < rows * BM; idx += TC_THREADS) tile[m_lo * BM + idx] = a.softcap * tanhf(tile[m_lo * BM + idx] / a.softcap);
                 __syncthreads();
@@ -533,7 +539,7 @@ struct ExpertList {
 
 template <bool CL, int V>
 __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const TcArgs a) {
-    constexpr bool X = V == 1;
+    constexpr bool X = V == 1 || V == 3;
     extern __shared__ __align__(1024) unsigned char dsm[];
     __shared__ TcShared sh;
     __shared__ typename std::conditional<V == 2, ExpertList, int>::type xl;
@@ -915,8 +921,9 @@ static cudaError_t launch_gemm_tc_v(const TcArgs& a_in, cudaStream_t st, bool pd
 }
 
 cudaError_t launch_gemm_tc(const TcArgs& a, cudaStream_t st, bool pdl) {
-    const bool x = a.group_blocks || a.out_scale || a.split_xp || a.turn.turns || a.softcap > 0.f || a.epi == EPI_GATE || a.epi == EPI_SQRELU;
+    const bool x = a.group_blocks || a.out_scale || a.split_xp || a.epi == EPI_GATE || a.epi == EPI_SQRELU;
     if (a.ex.n) return launch_gemm_tc_v<2>(a, st, pdl);
+    if (a.turn.turns || a.softcap > 0.f) return launch_gemm_tc_v<3>(a, st, pdl);
     return x ? launch_gemm_tc_v<1>(a, st, pdl) : launch_gemm_tc_v<0>(a, st, pdl);
 }
 

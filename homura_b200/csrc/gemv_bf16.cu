@@ -70,7 +70,7 @@ void gemv_pick_cluster(int K, int N, int M, int sm_count, int max_cluster, int* 
 // Asked of the current device every time (an occupancy query, no launch): engines on different GPUs of one
 // process each get their own answer.
 int gemv_max_cluster() {
-    if (ensure_nonportable_clusters(gemv_bf16_kernel<1, true, false, false>) != cudaSuccess) {
+    if (ensure_nonportable_clusters(gemv_bf16_kernel<1, true, false, 0>) != cudaSuccess) {
         cudaGetLastError();
         return 8;
     }
@@ -86,12 +86,15 @@ int gemv_max_cluster() {
     cfg.attrs = at;
     cfg.numAttrs = 1;
     int n = 0;
-    cudaError_t e = cudaOccupancyMaxActiveClusters(&n, gemv_bf16_kernel<1, true, false, false>, &cfg);
+    cudaError_t e = cudaOccupancyMaxActiveClusters(&n, gemv_bf16_kernel<1, true, false, 0>, &cfg);
     if (e != cudaSuccess) cudaGetLastError();
     return (e == cudaSuccess && n >= 4) ? 16 : 8;
 }
 
-cudaError_t launch_gemv_bf16(const GemvArgs& a, int M, cudaStream_t st, bool pdl) { return a.extended() ? launch_gemv_bf16_ext(a, M, st, pdl) : launch_rows<false>(a, M, st, pdl); }
+cudaError_t launch_gemv_bf16(const GemvArgs& a, int M, cudaStream_t st, bool pdl) {
+    const int v = a.variant();
+    return v == 2 ? launch_gemv_bf16_turn(a, M, st, pdl) : v == 1 ? launch_gemv_bf16_ext(a, M, st, pdl) : launch_rows<0>(a, M, st, pdl);
+}
 
 }  // namespace hm
 

@@ -3,6 +3,6 @@
 
 namespace hm {
 
-cudaError_t launch_gemv_bf16_ext(const GemvArgs& a, int M, cudaStream_t st, bool pdl) { return launch_rows<true>(a, M, st, pdl); }
+cudaError_t launch_gemv_bf16_ext(const GemvArgs& a, int M, cudaStream_t st, bool pdl) { return launch_rows<1>(a, M, st, pdl); }
 
 }  // namespace hm

@@ -1,5 +1,6 @@
-// The kernel of the weight-streaming bf16 projection and its launcher; instantiated by gemv_bf16.cu (X = false: the plain
-// projections) and gemv_ext.cu (X = true: grouped norm, split merge, grouped weights, gate, squared ReLU, output scale).
+// The kernel of the weight-streaming bf16 projection and its launcher; instantiated by gemv_bf16.cu (X = 0: the plain
+// projections), gemv_ext.cu (X = 1: grouped norm, split merge, grouped weights, gate, squared ReLU, output scale) and gemv_turn.cu
+// (X = 2: rotation and capped logits as well).
 #pragma once
 #include <type_traits>
 
@@ -77,7 +78,7 @@ __host__ __device__ __forceinline__ int gnorm_span(int K, int groups, int rps) {
 // everything that goes with it is requested before the factors are known.  The first slab's CTAs keep the last
 // row of every run in the state.
 template <int M>
-__device__ __forceinline__ void gnorm_stage(const GemvArgs& a, float* __restrict__ xs, float* __restrict__ gfac, const int* s_pos, const int* s_seq, int rps, int k0, int nrows, int slab, int tid) {
+__device__ __forceinline__ void gnorm_stage(const GemvExt& a, float* __restrict__ xs, float* __restrict__ gfac, const int* s_pos, const int* s_seq, int rps, int k0, int nrows, int slab, int tid) {
     if (nrows <= 0) return;  // uniform over the CTA
     const int lane = tid & 31, warp = tid >> 5;
     const int gs = a.K / a.gn.groups, g_lo = k0 / gs, ng = (k0 + nrows - 1) / gs - g_lo + 1;
@@ -163,7 +164,7 @@ __device__ __forceinline__ void gnorm_stage(const GemvArgs& a, float* __restrict
 // PRO_MERGE: elements [k0, k0 + nrows) of the combined rows of group `grp` into xs[M][rps]; wts holds M * n floats, part
 // M * 1024 (the slots of the reduction behind the multiply, not yet in use).
 template <int M>
-__device__ __forceinline__ void merge_stage(const GemvArgs& a, float* __restrict__ xs, float* __restrict__ wts, float* __restrict__ part, int rps, int k0, int nrows, int grp, int tid) {
+__device__ __forceinline__ void merge_stage(const GemvExt& a, float* __restrict__ xs, float* __restrict__ wts, float* __restrict__ part, int rps, int k0, int nrows, int grp, int tid) {
     const int lane = tid & 31, warp = tid >> 5, n = a.split.n;
     if (warp < M && warp < a.m_valid) {
         const float* ml = a.split.ml + ((size_t)warp * a.split.groups + grp) * n * 2;
@@ -223,10 +224,10 @@ __device__ __forceinline__ void merge_stage(const GemvArgs& a, float* __restrict
 // at most GEMV_STAGE_MAX bytes) is pulled into shared memory by bulk copies issued BEFORE the dependency
 // wait, so that by the time the predecessor has finished the multiply runs out of shared memory and HBM
 // latency is off the critical path of the dependent-kernel chain.
-template <bool X>
-using GemvArgsOf = typename std::conditional<X, GemvArgs, GemvBase>::type;
+template <int X>
+using GemvArgsOf = typename std::conditional<X == 2, GemvArgs, typename std::conditional<X == 1, GemvExt, GemvBase>::type>::type;
 
-template <int M, bool CL, bool ST, bool X>
+template <int M, bool CL, bool ST, int X>
 __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 ? 3 : (M <= 4 ? 2 : 1))) gemv_bf16_kernel(const GemvArgsOf<X> a) {
     extern __shared__ __align__(128) float smem_raw[];
     const int rps = a.rows_per_split;
@@ -572,7 +573,7 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
     HM_TRACE(if (tr) a.trace[5] = global_timer();)  // split-K reduced
     // ---- epilogues on vals[M][128] (columns n0 .. n0+127 of the output) ----
     bool stored = false;
-    if constexpr (X) {
+    if constexpr (X == 2) {
         if (a.epi == EPI_LOGITS && a.softcap > 0.f) {
             for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) vals[idx] = a.softcap * tanhf(vals[idx] / a.softcap);
             __syncthreads();
@@ -584,6 +585,8 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
             }
             __syncthreads();
         }
+    }
+    if constexpr (X) {
         if (a.epi == EPI_GATE) {
             for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) {
                 const int m = idx / SLAB, n = n0 + (idx % SLAB);
@@ -768,7 +771,7 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
 
 constexpr size_t GEMV_STAGE_MAX = 80 * 1024;  // largest weight slice staged in shared memory (two CTAs per SM stay resident)
 
-template <int M, bool CL, bool ST, bool X>
+template <int M, bool CL, bool ST, int X>
 cudaError_t launch_mcs(const GemvArgs& a, size_t smem, int nslabs, cudaStream_t st, bool pdl) {
     {
         cudaError_t e = ensure_dyn_smem(gemv_bf16_kernel<M, CL, ST, X>, smem);
@@ -799,7 +802,7 @@ cudaError_t launch_mcs(const GemvArgs& a, size_t smem, int nslabs, cudaStream_t 
     return cudaLaunchKernelEx(&cfg, gemv_bf16_kernel<M, CL, ST, X>, static_cast<const GemvArgsOf<X>&>(a));
 }
 
-template <int M, bool CL, bool X>
+template <int M, bool CL, int X>
 cudaError_t launch_mc(const GemvArgs& a_in, cudaStream_t st, bool pdl) {
     GemvArgs a = a_in;
     const int nslabs = a.group_slabs ? a.N / a.group_n * a.group_slabs : (a.N + SLAB - 1) / SLAB;
@@ -824,7 +827,7 @@ cudaError_t launch_mc(const GemvArgs& a_in, cudaStream_t st, bool pdl) {
     return launch_mcs<M, CL, false, X>(a, smem, nslabs, st, pdl);
 }
 
-template <int M, bool X>
+template <int M, int X>
 cudaError_t launch_m(const GemvArgs& a, cudaStream_t st, bool pdl) {
     if (a.cluster > 1) {
         if (a.cluster != a.ksplit || a.cluster > 16) return cudaErrorInvalidValue;
@@ -833,7 +836,7 @@ cudaError_t launch_m(const GemvArgs& a, cudaStream_t st, bool pdl) {
     return launch_mc<M, false, X>(a, st, pdl);
 }
 
-template <bool X>
+template <int X>
 cudaError_t launch_rows(const GemvArgs& a, int M, cudaStream_t st, bool pdl) {
     switch (M) {
         case 1: return launch_m<1, X>(a, st, pdl);

@@ -34,10 +34,11 @@ constexpr int MAX_STAGES = 8;
 constexpr int MAX_CLUSTER = 16;
 
 // ---- after the projection ------------------------------------------------------------------------
+template <bool X>
 __global__ void __launch_bounds__(POST_WARPS * 32) gqa_post_kernel(const GqaPostArgs a) {
     extern __shared__ __align__(16) float post_sm[];
     pdl_launch_dependents();
-    gqa_post_block(a, blockIdx.x, blockIdx.y, post_sm);
+    gqa_post_block<X>(a, blockIdx.x, blockIdx.y, post_sm);
 }
 
 __global__ void gqa_read_kernel(const GqaPool pool, int seq, int len, float* __restrict__ k, float* __restrict__ v) {
@@ -54,18 +55,20 @@ __global__ void gqa_read_kernel(const GqaPool pool, int seq, int len, float* __r
 }
 
 // ---- common to both attention kernels --------------------------------------------------------------
+// X: the variant with windows, sinks, gates and results that share their rows with others'.
+template <bool X>
 __device__ __forceinline__ void store_piece(const GqaAttnArgs& a, int m, int head, int d0, float (&v)[8]) {
-    const int vdim = a.pool.vdim, e0 = head * vdim + d0, k0 = a.out_off + e0;
-    if (a.gate_kind != GATE_NONE) {
+    const int vdim = a.pool.vdim, e0 = head * vdim + d0, off = X ? a.out_off : 0, k0 = off + e0, ld = X ? a.ld_out : a.heads * vdim;
+    if (X && a.gate_kind != GATE_NONE) {
         const float* g = a.gate + (size_t)m * a.ld_gate;
         const float all = a.gate_kind == GATE_HEAD ? 1.0f / (1.0f + expf(-ld_cg_f32(g + head))) : 1.f;
 #pragma unroll
         for (int i = 0; i < 8; ++i) v[i] *= a.gate_kind == GATE_HEAD ? all : d0 + i < vdim ? 1.0f / (1.0f + expf(-ld_cg_f32(g + e0 + i))) : 0.f;
     }
-    if (a.out_scale != 0.f)
+    if (X && a.out_scale != 0.f)
 #pragma unroll
         for (int i = 0; i < 8; ++i) v[i] *= a.out_scale;
-    if (a.xp && ((vdim | a.out_off) & 7) == 0) {
+    if (a.xp && ((vdim | off) & 7) == 0) {
         tc_xpack_store8(a.xp, a.xp_mpad, m, k0, v);
         return;
     }
@@ -73,12 +76,13 @@ __device__ __forceinline__ void store_piece(const GqaAttnArgs& a, int m, int hea
     for (int i = 0; i < 8; ++i) {
         if (d0 + i >= vdim) break;
         if (a.xp) tc_xpack_store(a.xp, a.xp_mpad, m, k0 + i, v[i]);
-        else a.out[(size_t)m * a.ld_out + k0 + i] = v[i];
+        else a.out[(size_t)m * ld + k0 + i] = v[i];
     }
 }
 
 // The sink's share of a denominator whose weights are relative to 2^mx.
-__device__ __forceinline__ float sink_weight(const GqaAttnArgs& a, int head, float mx) { return a.sink ? exp2f(fmaf(__ldg(a.sink + head), 1.4426950408889634f, -mx)) : 0.f; }
+template <bool X>
+__device__ __forceinline__ float sink_weight(const GqaAttnArgs& a, int head, float mx) { return X && a.sink ? exp2f(fmaf(__ldg(a.sink + head), 1.4426950408889634f, -mx)) : 0.f; }
 
 // Pages that rows at positions [lo, hi] see: those of the first tokens, then those of the window.  Page number i of the list is
 // pages_skip(i): i itself in front of the gap, i + gap behind it.
@@ -86,10 +90,11 @@ struct PageList {
     int n, head, gap;
     __device__ __forceinline__ int page(int i) const { return i < head ? i : i + gap; }
 };
+template <bool X>
 __device__ __forceinline__ PageList visible_pages(const GqaAttnArgs& a, int lo, int hi) {
     const int all = hi / GQA_PAGE + 1;
     PageList l{all, all, 0};
-    if (a.window > 0) {
+    if (X && a.window > 0) {
         const int from = max(0, lo - a.window + 1) / GQA_PAGE;  // first page of the window
         l.head = min((a.keep_first + GQA_PAGE - 1) / GQA_PAGE, from);
         l.gap = from - l.head;
@@ -100,17 +105,17 @@ __device__ __forceinline__ PageList visible_pages(const GqaAttnArgs& a, int lo, 
 
 // Results of a CTA's pairs in its shared memory: o [pairs][ldo] (not yet divided), ml [pairs][2] (maximum as a base-2 exponent, sum).
 // Splits are the CTAs of a cluster; every one of them combines and stores a share of the elements.  wts: [nsplit][pairs].
-template <typename RowHead>
+template <bool X, typename RowHead>
 __device__ __forceinline__ void combine_and_store(const GqaAttnArgs& a, const float* o, int ldo, const float* ml, float* wts, int pairs, RowHead row_head) {
     const int tid = threadIdx.x, nt = blockDim.x, ns = a.nsplit;
     const int rank = ns > 1 ? (int)cluster_ctarank() : 0;
     if (ns > 1) cluster_sync_all();
     else __syncthreads();
     for (int p = tid; p < pairs; p += nt) {
-        int sm_row, sm_head;
-        row_head(p, sm_row, sm_head);
+        int sm_row = 0, sm_head = 0;
+        if (X) row_head(p, sm_row, sm_head);
         if (ns == 1) {
-            wts[p] = 1.0f / (ml[2 * p + 1] + sink_weight(a, sm_head, ml[2 * p]));
+            wts[p] = 1.0f / (ml[2 * p + 1] + sink_weight<X>(a, sm_head, ml[2 * p]));
             continue;
         }
         float mr[MAX_CLUSTER], lr[MAX_CLUSTER], mx = -INFINITY, l = 0.f;
@@ -129,7 +134,7 @@ __device__ __forceinline__ void combine_and_store(const GqaAttnArgs& a, const fl
                 mr[r] = mr[r] == -INFINITY ? 0.f : exp2f(mr[r] - mx);
                 l = fmaf(mr[r], lr[r], l);
             }
-        l += sink_weight(a, sm_head, mx);
+        l += sink_weight<X>(a, sm_head, mx);
 #pragma unroll
         for (int r = 0; r < MAX_CLUSTER; ++r)
             if (r < ns) wts[r * pairs + p] = mr[r] / l;
@@ -155,14 +160,14 @@ __device__ __forceinline__ void combine_and_store(const GqaAttnArgs& a, const fl
         }
         int m, head;
         row_head(p, m, head);
-        if (d0 < a.pool.vdim) store_piece(a, m, head, d0, v);
+        if (d0 < a.pool.vdim) store_piece<X>(a, m, head, d0, v);
     }
     if (ns > 1) cluster_sync_all();  // nobody leaves while a peer reads its shared memory
 }
 
 // ---- CUDA cores ------------------------------------------------------------------------------------
 // One CTA = one row, key/value head and split.
-template <bool BF16>
+template <bool BF16, bool X>
 __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a) {
     extern __shared__ __align__(16) float sm[];
     const int g = a.heads / a.pool.kv_heads, kvh = blockIdx.y, m = blockIdx.z, split = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -176,7 +181,7 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
     pdl_launch_dependents();
     pdl_wait();
     const int pos = a.row_pos[m], len = pos + 1;
-    const PageList list = visible_pages(a, pos, pos);
+    const PageList list = visible_pages<X>(a, pos, pos);
     const int pps = (list.n + a.nsplit - 1) / a.nsplit, p0 = split * pps, p1 = min(list.n, p0 + pps);
     const int32_t* pt = a.pool.page_table + (size_t)a.row_seq[m] * a.pool.max_pages;
     for (int i = tid; i < g * dp; i += A_THREADS) {
@@ -197,7 +202,7 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
         for (int i = tid; i < g * GQA_PAGE; i += A_THREADS) {
             const int j = i / GQA_PAGE, t = i % GQA_PAGE;
             float s = -INFINITY;
-            if (t < nt && (a.window == 0 || pos - (p * GQA_PAGE + t) < a.window || p * GQA_PAGE + t < a.keep_first)) {
+            if (t < nt && (!X || a.window == 0 || pos - (p * GQA_PAGE + t) < a.window || p * GQA_PAGE + t < a.keep_first)) {
                 const float* q = q_s + j * dp;
                 s = 0.f;
                 for (int c = 0; c < dp / 8; ++c) {
@@ -246,7 +251,7 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
         }
         __syncthreads();
     }
-    combine_and_store(a, o_s, ldo, ml, wts, g, [&](int p, int& row, int& head) {
+    combine_and_store<X>(a, o_s, ldo, ml, wts, g, [&](int p, int& row, int& head) {
         row = m;
         head = kvh * g + p;
     });
@@ -278,7 +283,7 @@ __host__ __device__ inline size_t b_merge_bytes(int nt, int vp) { return sizeof(
 __host__ __device__ inline size_t b_recv_bytes(int nt, int vp, int nsplit) { return sizeof(float) * (size_t)nsplit * ((nt * 8 + nsplit - 1) / nsplit) * (vp + 4); }
 
 // VT: tiles of 16 value elements (at most), NT: tiles of eight pairs.
-template <int VT, int NT>
+template <int VT, int NT, bool X>
 __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_attn_mma_kernel(const GqaAttnArgs a, size_t ring_bytes) {
     constexpr int P = NT * 8;
     extern __shared__ __align__(128) unsigned char dyn[];
@@ -328,11 +333,12 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
     if (!a.early) pdl_wait();
     const int row_hi = row0 + (pair0 + pairs - 1) / g;
     const int seq = a.row_seq[row0], len = a.row_pos[row_hi] + 1;
-    const PageList list = visible_pages(a, a.window > 0 ? a.row_pos[row0 + pair0 / g] : 0, len - 1);
+    const PageList list = visible_pages<X>(a, X && a.window > 0 ? a.row_pos[row0 + pair0 / g] : 0, len - 1);
+    auto page_at = [&](int i) { return X ? list.page(i) : i; };
     const int pps = (list.n + a.nsplit - 1) / a.nsplit;
     const int p0 = split * pps, np = max(0, min(list.n, p0 + pps) - p0);
     const int32_t* pt = a.pool.page_table + (size_t)seq * a.pool.max_pages;
-    for (int i = tid; i < np; i += B_THREADS) pt_s[i] = pt[list.page(p0 + i)];
+    for (int i = tid; i < np; i += B_THREADS) pt_s[i] = pt[page_at(p0 + i)];
     const int seen = a.window > 0 ? a.window : 0x7fffffff;
     if (tid < P) {
         const int pr = pair0 + tid;
@@ -351,7 +357,7 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
     int n_pre = 0;
     if (a.early) {
         if (tid == ATT_WARPS * 32)
-            for (; n_pre < np && n_pre < NST && list.page(p0 + n_pre) < (len - 1) / GQA_PAGE; ++n_pre) fetch(n_pre, n_pre);
+            for (; n_pre < np && n_pre < NST && page_at(p0 + n_pre) < (len - 1) / GQA_PAGE; ++n_pre) fetch(n_pre, n_pre);
         pdl_wait();
     }
     if (warp == ATT_WARPS) {
@@ -410,7 +416,7 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
         for (int i = warp >> 2; i < np; i += 2) {
             const int s = i % NST;
             if (!__all_sync(0xffffffffu, mb_wait(&full[s], (i / NST) & 1u, a.err_flag, &s_abort))) break;
-            const int tok = list.page(p0 + i) * GQA_PAGE + u * 16;
+            const int tok = page_at(p0 + i) * GQA_PAGE + u * 16;
             if (tok < len) {
                 const uint32_t kb = s32(ring + (size_t)s * stage) + k_lane, vb = s32(ring + (size_t)s * stage + k_bytes) + v_lane;
                 constexpr int CH = NT == 1 ? 3 : 1;  // a lone tile of pairs: one accumulator per term, or its MMAs would wait for one another
@@ -448,8 +454,8 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
                             s0 += __ldg(a.bias + brow[nt][hh] + min(max(n0, 0), a.reach));
                             s1 += __ldg(a.bias + brow[nt][hh] + min(max(n1, 0), a.reach));
                         }
-                        s0 = n0 >= 0 && (n0 < seen || t0 < a.keep_first) ? s0 : -INFINITY;
-                        s1 = n1 >= 0 && (n1 < seen || t1 < a.keep_first) ? s1 : -INFINITY;
+                        s0 = n0 >= 0 && (!X || n0 < seen || t0 < a.keep_first) ? s0 : -INFINITY;
+                        s1 = n1 >= 0 && (!X || n1 < seen || t1 < a.keep_first) ? s1 : -INFINITY;
                         float mx = fmaxf(s0, s1);
 #pragma unroll
                         for (int o = 4; o < 32; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -572,10 +578,10 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
             v[0] = fmaf(f, x.x, v[0]); v[1] = fmaf(f, x.y, v[1]); v[2] = fmaf(f, x.z, v[2]); v[3] = fmaf(f, x.w, v[3]);
             v[4] = fmaf(f, y.x, v[4]); v[5] = fmaf(f, y.y, v[5]); v[6] = fmaf(f, y.z, v[6]); v[7] = fmaf(f, y.w, v[7]);
         }
-        const float inv = 1.0f / (l + sink_weight(a, kvh * g + (pair0 + p) % g, mx));
+        const float inv = 1.0f / (l + sink_weight<X>(a, kvh * g + (pair0 + p) % g, mx));
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[e] *= inv;
-        if (d0 < vdim) store_piece(a, row0 + (pair0 + p) / g, kvh * g + (pair0 + p) % g, d0, v);
+        if (d0 < vdim) store_piece<X>(a, row0 + (pair0 + p) / g, kvh * g + (pair0 + p) % g, d0, v);
     }
 }
 
@@ -646,7 +652,7 @@ int most_pages(const GqaAttnArgs& a, int pairs) {
     return (int)std::min<long>(all, seen);
 }
 
-template <int VT, int NT>
+template <int VT, int NT, bool X>
 cudaError_t launch_mma(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
     constexpr int P = NT * 8;
     const int g = a.heads / a.pool.kv_heads, dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
@@ -680,46 +686,50 @@ cudaError_t launch_mma(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
         a.nsplit = std::max(1, std::min({PER_SM * sm_count / pairs, a.max_cluster, pages > 128 ? MAX_CLUSTER : 8, pages}));
         for (; a.nsplit > 1; --a.nsplit) {
             shape(a.nsplit);
-            if (ring + fixed <= 226 * 1024 && clusters_at_once(gqa_attn_mma_kernel<VT, NT>, a.nsplit, B_THREADS, ring + fixed) >= pairs) break;
+            if (ring + fixed <= 226 * 1024 && clusters_at_once(gqa_attn_mma_kernel<VT, NT, X>, a.nsplit, B_THREADS, ring + fixed) >= pairs) break;
         }
     }
     shape(a.nsplit);
     if (ring + fixed > 226 * 1024) return cudaErrorInvalidValue;
-    return launch_clustered(gqa_attn_mma_kernel<VT, NT>, dim3((unsigned)a.nsplit, (unsigned)a.pool.kv_heads, (unsigned)a.tiles), dim3(B_THREADS), ring + fixed, a.nsplit, st, pdl, a, ring);
+    return launch_clustered(gqa_attn_mma_kernel<VT, NT, X>, dim3((unsigned)a.nsplit, (unsigned)a.pool.kv_heads, (unsigned)a.tiles), dim3(B_THREADS), ring + fixed, a.nsplit, st, pdl, a, ring);
 }
 
-template <int VT>
+template <int VT, bool X>
 cudaError_t launch_mma_n(const GqaAttnArgs& a, int sm_count, cudaStream_t st, bool pdl) {
     const int pairs = a.longest_run * (a.heads / a.pool.kv_heads);
-    if (pairs <= 8) return launch_mma<VT, 1>(a, sm_count, st, pdl);
-    if (pairs <= 16 || VT > 4) return launch_mma<VT, 2>(a, sm_count, st, pdl);  // four tiles of wide values do not fit the registers
-    return launch_mma<VT, VT <= 4 ? 4 : 2>(a, sm_count, st, pdl);
+    if (pairs <= 8) return launch_mma<VT, 1, X>(a, sm_count, st, pdl);
+    if (pairs <= 16 || VT > 4) return launch_mma<VT, 2, X>(a, sm_count, st, pdl);  // four tiles of wide values do not fit the registers
+    return launch_mma<VT, VT <= 4 ? 4 : 2, X>(a, sm_count, st, pdl);
 }
 
 }  // namespace
 
 cudaError_t launch_gqa_post(const GqaPostArgs& a, cudaStream_t st, bool pdl) {
-    return launch_clustered(gqa_post_kernel, dim3((unsigned)a.M, (unsigned)gqa_post_blocks(a)), dim3(POST_WARPS * 32), gqa_post_smem(a), 1, st, pdl, a);
+    const dim3 grid((unsigned)a.M, (unsigned)gqa_post_blocks(a)), block(POST_WARPS * 32);
+    return gqa_post_buf(a) > 0 ? launch_clustered(gqa_post_kernel<true>, grid, block, gqa_post_smem(a), 1, st, pdl, a) : launch_clustered(gqa_post_kernel<false>, grid, block, 0, 1, st, pdl, a);
 }
 
 cudaError_t launch_gqa_attn(const GqaAttnArgs& a_in, int sm_count, cudaStream_t st, bool pdl) {
     GqaAttnArgs a = a_in;
     if (a.M < 1 || a.M > GQA_MAX_ROWS || a.nsplit > MAX_CLUSTER || a.heads % a.pool.kv_heads != 0) return cudaErrorInvalidValue;
     if (!a.bias) a.reach = 0;
+    const bool x = a.window > 0 || a.sink || a.gate_kind != GATE_NONE || a.out_scale != 0.f || a.ld_out != 0;
     if (a.ld_out == 0) a.ld_out = a.heads * a.pool.vdim;
     const int g = a.heads / a.pool.kv_heads, dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
     if (a.runs.n == 0) a.longest_run = 1;
     const long ppc_most = most_pages(a, 32);
     if (a.pool.bf16 && vp <= 256 && dp <= 256 && ppc_most <= 8192) {
-        if (vp <= 64) return launch_mma_n<4>(a, sm_count, st, pdl);
-        if (vp <= 128) return launch_mma_n<8>(a, sm_count, st, pdl);
-        return launch_mma_n<16>(a, sm_count, st, pdl);
+        if (vp <= 64) return x ? launch_mma_n<4, true>(a, sm_count, st, pdl) : launch_mma_n<4, false>(a, sm_count, st, pdl);
+        if (vp <= 128) return x ? launch_mma_n<8, true>(a, sm_count, st, pdl) : launch_mma_n<8, false>(a, sm_count, st, pdl);
+        return x ? launch_mma_n<16, true>(a, sm_count, st, pdl) : launch_mma_n<16, false>(a, sm_count, st, pdl);
     }
     const int pages = most_pages(a, 1);
     if (a.nsplit < 1) a.nsplit = std::max(1, std::min({4 * sm_count / (a.M * a.pool.kv_heads), a.max_cluster, MAX_CLUSTER, pages}));
     const size_t smem = sizeof(float) * (size_t)g * (dp + vp + 4 + GQA_PAGE + 3 + a.nsplit);
     const dim3 grid((unsigned)a.nsplit, (unsigned)a.pool.kv_heads, (unsigned)a.M);
-    return a.pool.bf16 ? launch_clustered(gqa_attn_kernel<true>, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a) : launch_clustered(gqa_attn_kernel<false>, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a);
+    auto go = [&](auto kern) { return launch_clustered(kern, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a); };
+    if (x) return a.pool.bf16 ? go(gqa_attn_kernel<true, true>) : go(gqa_attn_kernel<false, true>);
+    return a.pool.bf16 ? go(gqa_attn_kernel<true, false>) : go(gqa_attn_kernel<false, false>);
 }
 
 cudaError_t launch_gqa_read(const GqaPool& pool, int seq, int len, float* k, float* v, cudaStream_t st) {

@@ -24,8 +24,9 @@ __device__ __forceinline__ void rotate_pairs(float* buf, int half, const double*
     }
 }
 
-// Row m of one head slot ([heads] queries, [kv_heads] keys, [kv_heads] values).  part_q / part_k: sums of squares of the whole
+// X: with convolution, rotation or norms behind it (the plain variant keeps no head in shared memory).  Row m of one head slot ([heads] queries, [kv_heads] keys, [kv_heads] values).  part_q / part_k: sums of squares of the whole
 // projections (QKN_ALL); first: the first row of m's run.
+template <bool X>
 __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int slot, int first, int pos, int seq, size_t page, float part_q, float part_k, float* buf) {
     const int lane = threadIdx.x & 31;
     const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
@@ -34,7 +35,7 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
     const int h = is_v ? slot - a.heads - G : is_q ? slot : slot - a.heads, n = is_v ? vdim : dim;
     const int ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n;  // first channel
     const float* x = a.raw + (size_t)m * a.ld + ch0;
-    const bool buffered = gqa_post_buf(a) > 0;
+    const bool buffered = X && gqa_post_buf(a) > 0;
     if (buffered) {
         const float* state = a.taps > 1 ? a.conv_state + (size_t)seq * a.conv_stride + ch0 : nullptr;
         const int channels = nq + nk + G * vdim;
@@ -75,8 +76,8 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
         const float* w = a.qk_norm == QKN_HEAD || a.qk_norm == QKN_ALL ? (is_q ? a.q_norm : a.k_norm) + (a.qk_norm == QKN_ALL ? (size_t)h * dim : 0) : nullptr;
         auto normed = [&](int d) { return w ? (at(d) * inv) * __ldg(w + d) : at(d); };
         float unit = 1.f;
-        const bool turned = a.rot_dims > 0;
-        if (turned || a.qk_norm == QKN_UNIT) {
+        const bool turned = X && a.rot_dims > 0, after = X && (turned || a.qk_norm == QKN_UNIT);
+        if (after) {
             if (w)
                 for (int d = lane; d < dim; d += 32) buf[d] = normed(d);
             __syncwarp();
@@ -88,7 +89,7 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
                 unit = 1.0f / sqrtf(warp_sum(s) / (float)dim + a.eps);
             }
         }
-        auto value = [&](int d) { return turned || a.qk_norm == QKN_UNIT ? buf[d] * unit : normed(d); };
+        auto value = [&](int d) { return after ? buf[d] * unit : normed(d); };
         if (is_q) {
             float f = 1.f;
             if (a.temp_every > 0) f = 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
@@ -122,6 +123,7 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
 }
 
 // Row m and POST_WARPS head slots from blk * POST_WARPS on.
+template <bool X>
 __device__ __forceinline__ void gqa_post_block(const GqaPostArgs& a, int m, int blk, float* smem) {
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
@@ -162,18 +164,18 @@ __device__ __forceinline__ void gqa_post_block(const GqaPostArgs& a, int m, int 
         }
     }
     if (slot >= gqa_post_slots(a)) return;
-    float* buf = smem + warp * gqa_post_buf(a);
-    if (a.taps <= 1) {
-        gqa_post_row(a, m, slot, m, pos, seq, page, sq, sk, buf);
+    float* buf = X ? smem + warp * gqa_post_buf(a) : nullptr;
+    if (!X || a.taps <= 1) {
+        gqa_post_row<X>(a, m, slot, m, pos, seq, page, sq, sk, buf);
         return;
     }
     int first, end;
     a.runs.find(m, first, end);
     const int keep = a.taps - 1;
     if (m > first && m < first + keep) return;  // served by the warp of the run's first row
-    gqa_post_row(a, m, slot, first, pos, seq, page, sq, sk, buf);
+    gqa_post_row<X>(a, m, slot, first, pos, seq, page, sq, sk, buf);
     if (m > first) return;
-    for (int r = first + 1; r < min(end, first + keep); ++r) gqa_post_row(a, r, slot, first, pos + r - first, seq, page_of(seq, pos + r - first), 0.f, 0.f, buf);
+    for (int r = first + 1; r < min(end, first + keep); ++r) gqa_post_row<X>(a, r, slot, first, pos + r - first, seq, page_of(seq, pos + r - first), 0.f, 0.f, buf);
     // the run's last inputs replace the kept ones (a lane keeps the channels that it has read)
     const bool is_v = slot >= a.heads + G, is_q = slot < a.heads;
     const int h = is_v ? slot - a.heads - G : is_q ? slot : slot - a.heads, n = is_v ? vdim : dim, ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n, channels = nq + nk + G * vdim;

@@ -34,7 +34,7 @@ __global__ void __launch_bounds__(128) latent_write_kernel(const LatentPool pool
     __shared__ float part[4];
     pdl_launch_dependents();
     pdl_wait();
-    latent_write_row(pool, c, ldc, blockIdx.x, w, eps, row_pos, row_seq, 0, nullptr, part);
+    latent_write_row<128, false>(pool, c, ldc, blockIdx.x, w, eps, row_pos, row_seq, 0, nullptr, part);
 }
 
 __global__ void latent_read_kernel(const LatentPool pool, int seq, int len, float* out) {

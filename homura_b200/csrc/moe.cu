@@ -219,7 +219,7 @@ __global__ void __launch_bounds__(THREADS) expert_gate_up_kernel(const ExpertWei
             g += red[i][tid];
             u += red[i][GU_ROWS + tid];
         }
-        act[(size_t)pair * blocks * 64 + blk * 64 + sub * GU_ROWS + tid] = glu(w.act, g, u, w.limit) * rw;
+        act[(size_t)pair * blocks * 64 + blk * 64 + sub * GU_ROWS + tid] = (w.act == GLU_CLAMPED ? clamped_glu(g, u, w.limit) : glu(w.act, g, u, w.limit)) * rw;
     }
 }
 

@@ -107,13 +107,13 @@ __global__ void __launch_bounds__(THREADS, RD > 32 ? 1 : RD > 0 ? 2 : 3) side_ke
     }
     if (b < a.n_post) {
         const int per = gqa_post_blocks(a.post);
-        gqa_post_block(a.post, b / per, b % per, sm);
+        gqa_post_block<true>(a.post, b / per, b % per, sm);
         return;
     }
     b -= a.n_post;
     pdl_wait();
     if (b < a.n_latent) {
-        if (b < a.M) latent_write_row(a.latent.pool, a.latent.c, a.ld, b, a.latent.w, a.eps, a.row_pos, a.row_seq, a.latent.rot_pairs, a.latent.turns, part);
+        if (b < a.M) latent_write_row<THREADS, true>(a.latent.pool, a.latent.c, a.ld, b, a.latent.w, a.eps, a.row_pos, a.row_seq, a.latent.rot_pairs, a.latent.turns, part);
         else query_latent_block(a, b - a.M, part);
         return;
     }
