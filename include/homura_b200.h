@@ -109,7 +109,8 @@ HM_API int hm_model_load_gguf(const char* gguf_path, int device, hm_engine** out
  * q_norm / k_norm weights before those projections (HM_ERR_STATE otherwise; hm_model_load* do so). */
 HM_API int hm_engine_create(const hm_config* cfg, int device, hm_engine** out);
 /* The same from the text of a config.json, for every design the library knows (its "architecture" key, e.g. "Tunitar", or
- * the Qwen2 / Qwen3 / Llama keys).  weight_dtype as in hm_model_load. */
+ * the Qwen2 / Qwen3 / Llama keys).  weight_dtype as in hm_model_load.  A tensor whose shape tells a size that the text does not
+ * ("Gebilorn": mix.right.a1) comes before the other tensors of its layer. */
 HM_API int hm_engine_create_json(const char* config_json, int weight_dtype, int device, hm_engine** out);
 /* Name of the design, "" for the uniform Qwen2 / Qwen3 / Llama stacks.  Valid until the engine is destroyed. */
 HM_API const char* hm_get_arch(hm_engine* e);
@@ -155,7 +156,8 @@ HM_API int hm_kv_append(hm_engine* e, int seq, int layer, const float* k_rows, c
 /* KvCache::view, src/runtime.rs:463-507: contiguous f32 [kv_heads, len, head_dim] copies. */
 HM_API int hm_kv_view(hm_engine* e, int seq, int layer, float* k_out, float* v_out);
 
-/* Latent caches: f32 [len, kv_rank] copies of the layer's latents (of the layer it shares them with). */
+/* Latent caches: f32 [len, kv_rank] copies of the layer's latents (of the layer it shares them with); with a rotated key part
+ * behind the latent [len, kv_rank + rot_dim], its pairs side by side. */
 HM_API int hm_latent_view(hm_engine* e, int seq, int layer, float* out);
 
 /* ---- one batch over several sequences --------------------------------------------------- */

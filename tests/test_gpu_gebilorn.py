@@ -394,6 +394,17 @@ def test_tensors_one_by_one_and_missing_ones(hm):
             hm.HfModel.from_config_json(json.dumps(cfg), [t for t in tensors if t[0] == "l0.mix.right.a1"] + [(name, hm.DType.BF16, shape, np.zeros(shape, np.uint16))])
 
 
+def test_a_sharded_checkpoint(hm, tmp_path):
+    """Shapes that tell sizes may lie in another shard than the tensors they size."""
+    d = synth.write_gebilorn_model(str(tmp_path / "one"), model("mixed"), 21, weights("mixed"), RANKS["mixed"])
+    ids, want, _ = expected("mixed", "F32", 1, 150)
+    for n in (2, 5):
+        m = hm.HfModel.load_with_dtype(synth.shard_hf_model(d, str(tmp_path / str(n)), n), hm.DType.F32)
+        m.init_kv_cache(256, batch=1, kv_dtype=hm.DType.F32)
+        close(run_portions(m, ids, [150]), want, "F32", "logits of a sharded checkpoint")
+        m.close()
+
+
 def test_step_refuses_bad_entries_and_keeps_its_state(hm, engines):
     ids, want, _ = expected("mixed", "F32", 1, 150)
     m = engines("mixed", "F32")
