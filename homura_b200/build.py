@@ -11,8 +11,8 @@ import sys
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libhomura_b200.so")
-SOURCES = ["gemv_bf16.cu", "gemv_ext.cu", "gemv_turn.cu", "gemm_tc.cu", "attention.cu", "quant.cu", "kquant.cu", "kquant_gemm.cu", "sampler.cu", "misc_kernels.cu", "latent_attn.cu", "gqa_attn.cu", "moe.cu", "side.cu", "engine.cu", "engine_listed.cu", "engine_gqa.cu", "engine_parallel.cu", "engine_step.cu", "capi.cu", "loaders.cpp", "model_spec.cpp", "launch_attrs.cpp"]
-HEADERS = ["common.cuh", "engine.h", "gemm_tc.h", "mbarrier.cuh", "gemv_kernel.cuh", "kquant.h", "sampler.h", "loaders.h", "launch_attrs.h", "latent_attn.h", "gqa_attn.h", "moe.h", "route.cuh", "gla.h", "gla.cuh", "gqa_post.cuh", "latent_post.cuh", "side.h", "engine_parallel.h", "model_spec.h", "engine_util.h", os.path.join("..", "..", "include", "homura_b200.h")]
+SOURCES = ["gemv_bf16.cu", "gemv_ext.cu", "gemv_turn.cu", "gemm_tc.cu", "attention.cu", "quant.cu", "kquant.cu", "kquant_gemm.cu", "sampler.cu", "misc_kernels.cu", "latent_attn.cu", "gqa_attn.cu", "moe.cu", "side.cu", "recur.cu", "sandwich.cu", "engine.cu", "engine_listed.cu", "engine_gqa.cu", "engine_parallel.cu", "engine_sandwich.cu", "engine_step.cu", "capi.cu", "loaders.cpp", "model_spec.cpp", "launch_attrs.cpp"]
+HEADERS = ["common.cuh", "engine.h", "gemm_tc.h", "mbarrier.cuh", "gemv_kernel.cuh", "kquant.h", "sampler.h", "loaders.h", "launch_attrs.h", "latent_attn.h", "gqa_attn.h", "moe.h", "route.cuh", "gla.h", "gla.cuh", "gqa_talk.cuh", "recur.h", "sandwich.h", "gqa_post.cuh", "latent_post.cuh", "side.h", "engine_parallel.h", "model_spec.h", "engine_util.h", os.path.join("..", "..", "include", "homura_b200.h")]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
     "-lineinfo", "-O3", "-std=c++17",

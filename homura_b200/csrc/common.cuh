@@ -242,8 +242,14 @@ __device__ __forceinline__ float warp_max(float v) {
 // PRO_GNORM: RMSNorm in equal groups, optionally followed by the token shift (see RowNorm)
 // PRO_MERGE: the input rows are the splits of an attention over latents, still to be combined (SplitRows)
 enum Prologue { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_GNORM = 2, PRO_MERGE = 3 };
-// EPI_GATE: y = acc * sigmoid(gate); EPI_SQRELU: y = max(acc, 0)^2; EPI_EXPERT: gated activation of a mixture's experts
-enum Epilogue { EPI_STORE = 0, EPI_QKV_ROPE = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3, EPI_GATE = 4, EPI_SQRELU = 5, EPI_EXPERT = 6 };
+// EPI_GATE: y = acc * sigmoid(gate); EPI_SQRELU: y = max(acc, 0)^2; EPI_EXPERT: gated activation of a mixture's experts; EPI_GLU: clamped
+// gated activation with biases, columns as for EPI_SWIGLU
+enum Epilogue { EPI_STORE = 0, EPI_QKV_ROPE = 1, EPI_SWIGLU = 2, EPI_LOGITS = 3, EPI_GATE = 4, EPI_SQRELU = 5, EPI_EXPERT = 6, EPI_GLU = 7 };
+// Gated activation: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1).
+__device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
 
 // Normalisation of a projection's input rows in `groups` equal runs, each divided by its own root mean square, and the
 // token shift h + (h' - h) * shift, where h' is the normalised row of the sequence's previous token before its own shift
@@ -323,12 +329,13 @@ struct TurnedPairs {
     const double* turns;     // null: none
     int period, dims;
     const int32_t* row_pos;
+    int columns;             // > 0: only the columns in front of this one
 };
 
 // Columns n (even) and n + 1 of row m.
 __device__ __forceinline__ void turn_pair(const TurnedPairs& t, int m, int n, float& u, float& v) {
     const int d = n % t.period;
-    if (d >= t.dims) return;
+    if (d >= t.dims || (t.columns > 0 && n >= t.columns)) return;
     float c, s;
     rotation_at(__ldg(t.turns + d / 2), t.row_pos[m], c, s);
     const float x = u, y = v;
@@ -471,7 +478,10 @@ struct GemvExt : GemvBase {
     const float* out_scale;  // [N] or null (EPI_STORE: the result is multiplied element by element before the residual is added)
     const float* gate;   // EPI_GATE: [M][ld_gate]
     int ld_gate;
-    bool extended() const { return pro == PRO_GNORM || pro == PRO_MERGE || epi == EPI_GATE || epi == EPI_SQRELU || group_slabs != 0 || out_scale != nullptr; }
+    int gate_per;        // EPI_GATE: > 1: so many columns share a gate
+    float limit;         // EPI_GLU
+    int glu_n;           // EPI_GLU: outputs (the last block may be padded)
+    bool extended() const { return pro == PRO_GNORM || pro == PRO_MERGE || epi == EPI_GATE || epi == EPI_SQRELU || epi == EPI_GLU || group_slabs != 0 || out_scale != nullptr; }
 };
 // And of the variant behind that (gemv_turn.cu): rotation and capped logits in the epilogue.
 struct GemvArgs : GemvExt {

@@ -1,5 +1,6 @@
 // Engine implementation.  See engine.h.
 #include "engine.h"
+#include "sandwich.h"
 #include "engine_util.h"
 #include "gemm_tc.h"
 #include "kquant.h"
@@ -76,8 +77,10 @@ int Engine::create(const ModelSpec& spec, int device, bool strict_f32, Engine** 
         e->qdim_ = 0;
         for (const LayerSpec& l : spec.layers) {
             e->qdim_ = std::max(e->qdim_, l.heads * std::max(l.vdim, l.paged_kv() ? l.dim : l.q_rank ? l.q_stride() : 0));
+            if (spec.sandwich && e->H_ > SANDWICH_MAX_WIDTH) return bad("width must be at most 16384");
+            if (l.talking && !gqa_talk_fits(l.heads, l.dim, l.vdim)) return bad("heads that mix their scores must fit one SM together (heads * (dim + vdim) up to about 40000)");
             if (l.latent_rank() > 1024) return bad("kv_rank (with rot_dim) must be at most 1024");
-            if (l.mixer == MIX_PARALLEL && (l.lin_dim > GLA_MAX_DIM || l.lin_vdim > GLA_MAX_VDIM)) return bad("linear attention heads have at most 1024 key and 512 value elements");
+            if (l.linear() && (l.lin_dim > GLA_MAX_DIM || l.lin_vdim > GLA_MAX_VDIM)) return bad("linear attention heads have at most 1024 key and 512 value elements");
             if (l.experts > 1024) return bad("a mixture has at most 1024 experts");
         }
     } else {
@@ -112,7 +115,7 @@ Engine::~Engine() {
     };
     fr(embed_); fr(final_norm_); fr(rope_cos_); fr(rope_sin_);
     for (auto& l : layers_)
-        for (float* p : {l.in_ln, l.post_ln, l.qkv_bias, l.q_norm, l.k_norm, l.shift, l.ls1, l.ls2, l.latent_norm, l.v_mix, l.rel, l.correction, l.in_bias, l.sink, l.conv_w, l.lin_norm, l.lin_up, l.lin_bias}) fr(p);
+        for (float* p : {l.in_ln, l.post_ln, l.qkv_bias, l.q_norm, l.k_norm, l.shift, l.ls1, l.ls2, l.latent_norm, l.v_mix, l.rel, l.correction, l.in_bias, l.sink, l.conv_w, l.lin_norm, l.lin_up, l.lin_bias, l.norm1b, l.norm2b, l.left_out, l.right_out, l.talk, l.temp, l.gu_bias, l.down_bias, l.lin_conv_w, l.lin_rate, l.lin_up_g, l.lin_decay}) fr(p);
     for (auto& l : layers_) { fr(l.router); fr(l.exp_gu); fr(l.exp_down); fr(l.turns); }
     fr(turns_); fr(bigram_);
     each_linear([&](LinearW& w) { fr(w.slabs); fr(w.tc); fr(w.scales); fr(w.codes); fr(w.kq_data); fr(w.kq_tile_type); });
@@ -723,6 +726,7 @@ int Engine::kv_view(int seq, int layer, float* k_out, float* v_out) {
     if (seq < 0 || seq >= batch_ || layer < 0 || layer >= L_ || !k_out || !v_out) return fail(HM_ERR_INVALID, "kv_view: bad arguments");
     const LayerSpec* ls = spec_.listed() ? &spec_.layers[layer] : nullptr;
     if (ls && ls->mixer == MIX_LATENT) return fail(HM_ERR_UNSUPPORTED, "kv_view: this design caches latents, not keys and values (hm_latent_view)");
+    if (ls && !ls->paged_kv()) return fail(HM_ERR_UNSUPPORTED, "kv_view: this layer keeps a state, not keys and values");
     const int len = len_[seq];
     if (len == 0) return HM_OK;
     const size_t k_bytes = (size_t)(ls ? ls->kv_heads * ls->dim : kvh_ * hd_) * len * 4, v_bytes = (size_t)(ls ? ls->kv_heads * ls->vdim : kvh_ * hd_) * len * 4;
@@ -745,6 +749,7 @@ int Engine::kv_view(int seq, int layer, float* k_out, float* v_out) {
 static const char* kProfNames[PC_COUNT] = {"embed", "qkv_rope_kvwrite", "attention", "o_proj_residual", "gate_up_swiglu", "down_residual", "lm_head", "argmax"};
 static const char* kProfNamesListed[PC_COUNT_LISTED] = {"embed", "in_proj", "attention", "o_proj_residual", "up_sqrelu", "down_residual", "lm_head", "argmax", "latent_write", "key_up", "value_up_gate"};
 static const char* kProfNamesGqa[PC_COUNT_LISTED] = {"embed", "qkv_proj", "attention", "o_proj", "experts_gate_up", "experts_down", "lm_head", "argmax", nullptr, nullptr, nullptr, "qk_norm_kv_write", "post_norm_router", "post_norm"};
+static const char* kProfNamesSandwich[PC_COUNT_LISTED] = {"embed", "in_proj", "attention", "out_proj", "gate_up", "down", "lm_head", "argmax", nullptr, "key_up", "value_up", "side", nullptr, "norm", nullptr, "recurrence"};
 static const char* kProfNamesParallel[PC_COUNT_LISTED] = {"embed", "in_proj", "attention", "out_proj", "experts_gate_up", "experts_down", "lm_head", "argmax", nullptr, "key_up", "value_up", "side", nullptr, "sum_norm", "query_up"};
 
 void Engine::prof_mark(int) {}
@@ -963,6 +968,9 @@ int Engine::enqueue_linear(const LinearW& L, int M, const float* x, int ldx, int
                 if (a.turn.row_pos) a.turn.row_pos += m0;
                 a.softcap = opt->softcap;
                 a.out_scale = opt->out_scale;
+                a.gate_per = opt->gate_per;
+                a.limit = opt->limit;
+                a.glu_n = opt->glu_n;
                 a.gate = opt->gate ? opt->gate + (size_t)m0 * opt->ld_gate : nullptr;
                 a.ld_gate = opt->ld_gate;
             }
@@ -1130,7 +1138,7 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
     const bool fused = direct_pack && H_ % 128 == 0;
     for (int l = 0; l < L_; ++l) {
         if (spec_.listed()) {
-            rc = spec_.parallel ? enqueue_parallel_layer(l, M, row_pos, row_seq, lm_rows, launches) : spec_.layers[l].mixer == MIX_GQA ? enqueue_gqa_layer(l, M, row_pos, row_seq, lm_rows, launches) : enqueue_listed_layer(l, M, row_pos, row_seq, lm_rows, launches);
+            rc = spec_.sandwich ? enqueue_sandwich_layer(l, M, row_pos, row_seq, lm_rows, launches) : spec_.parallel ? enqueue_parallel_layer(l, M, row_pos, row_seq, lm_rows, launches) : spec_.layers[l].mixer == MIX_GQA ? enqueue_gqa_layer(l, M, row_pos, row_seq, lm_rows, launches) : enqueue_listed_layer(l, M, row_pos, row_seq, lm_rows, launches);
             if (rc) return rc;
             rc = tap(l, M);
             if (rc) return rc;
@@ -1269,7 +1277,10 @@ int Engine::enqueue_pass(int M, const uint32_t* tokens_dev, const int32_t* row_p
         const bool fold_argmax = slab_argmax && !lm_tall;    // the streaming kernel's last epilogue also produces the greedy token
         lm_folds_argmax_ = fold_argmax;
         if (spec_.listed()) {
-            if (want(PC_LM_HEAD)) {
+            if (want(PC_LM_HEAD) && spec_.sandwich) {
+                rc = enqueue_sandwich_logits(x, lm_rows, final_norm_fits(M, lm_rows), (lm_out_ && fold_argmax) ? lm_out_ : lg, ArgmaxFold{next_dev, feed_dev, pos_dev, hist_dev, max_seq_ + 1}, launches);
+                if (rc) return rc;
+            } else if (want(PC_LM_HEAD)) {
                 rc = enqueue_listed_logits(x, lm_rows, (lm_out_ && fold_argmax) ? lm_out_ : lg, ArgmaxFold{next_dev, feed_dev, pos_dev, hist_dev, max_seq_ + 1}, launches);
                 if (rc) return rc;
             }
@@ -1650,7 +1661,7 @@ int Engine::time_decode(int warmup, int steps, float* ms_total) {
 int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) {
     if (!set_device()) return fail(HM_ERR_CUDA, "cudaSetDevice failed");
     if (batch_ == 0) return fail(HM_ERR_STATE, "profile_decode before kv_alloc");
-    if (steps < 1 || !out || !n_out || cap < (spec_.listed() ? PC_COUNT_LISTED : PC_COUNT)) return fail(HM_ERR_INVALID, "profile_decode: bad arguments (cap >= 8; 15 for listed designs)");
+    if (steps < 1 || !out || !n_out || cap < (spec_.listed() ? PC_COUNT_LISTED : PC_COUNT)) return fail(HM_ERR_INVALID, "profile_decode: bad arguments (cap >= 8; 16 for listed designs)");
     const bool moe = spec_.post_norm || spec_.parallel;
     for (int b = 0; b < batch_; ++b)
         if (len_[b] + steps + (moe ? 1 : 0) > max_seq_) return fail(HM_ERR_KV_FULL, "KV cache full: not enough room for the profiled steps");
@@ -1726,7 +1737,7 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
         bytes[PC_KUP] += l.kup.bytes();
         bytes[PC_VUP] += l.vup.bytes();
         bytes[PC_QUP] += l.uq.bytes();
-        if (spec_.parallel && spec_.layers[li].mixer == MIX_PARALLEL) bytes[PC_KV_WRITE] += 2ull * batch_ * spec_.layers[li].lin_heads * spec_.layers[li].lin_dim * spec_.layers[li].lin_vdim * 4;
+        if (spec_.listed() && spec_.layers[li].linear()) bytes[spec_.sandwich ? PC_RECUR : PC_KV_WRITE] += 2ull * batch_ * spec_.layers[li].lin_heads * spec_.layers[li].lin_dim * spec_.layers[li].lin_vdim * 4;
         bytes[PC_O] += l.o.bytes();
         bytes[PC_GATE_UP] += l.gu.bytes();
         bytes[PC_DOWN] += l.down.bytes();
@@ -1735,7 +1746,11 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
     if (spec_.listed()) {
         for (const LayerSpec& l : spec_.layers) {
             double tokens = kv_tokens;
-            if (l.window > 0) {
+            if (l.mixer == MIX_LINEAR) continue;
+            if (l.chunk > 0) {
+                tokens = 0;
+                for (int b = 0; b < batch_; ++b) tokens += (len_[b] - steps) % l.chunk + 1;
+            } else if (l.window > 0) {
                 tokens = 0;
                 for (int b = 0; b < batch_; ++b) tokens += std::min(len_[b] - steps + 1, l.window + l.keep_first);
             }
@@ -1744,7 +1759,7 @@ int Engine::profile_decode(int steps, hm_kernel_stat* out, int cap, int* n_out) 
     } else {
         bytes[PC_ATTN] = (uint64_t)(kv_tokens * L_ * 2.0 * kvh_ * hd_ * (kv_bf16_ ? 2 : 4));
     }
-    const char* const* names = !spec_.listed() ? kProfNames : spec_.parallel ? kProfNamesParallel : spec_.post_norm ? kProfNamesGqa : kProfNamesListed;
+    const char* const* names = !spec_.listed() ? kProfNames : spec_.sandwich ? kProfNamesSandwich : spec_.parallel ? kProfNamesParallel : spec_.post_norm ? kProfNamesGqa : kProfNamesListed;
     int n = 0;
     for (int c = 0; c < classes; ++c) {
         if (!names[c]) continue;

@@ -17,6 +17,7 @@
 #include "latent_attn.h"
 #include "moe.h"
 #include "model_spec.h"
+#include "recur.h"
 #include "sampler.h"
 #include "side.h"
 
@@ -74,6 +75,16 @@ struct LayerW {
     float* conv_w = nullptr;             // [query, key and value channels][taps]
     float *lin_norm = nullptr, *lin_up = nullptr, *lin_bias = nullptr;  // linear attention: result norm, decay up-projection [heads][rank][dim], its bias
     LinearW uq;                          // queries out of their latent
+    // listed designs with sublayers between two norms: `in` is everything that the mixer reads off its normed input
+    float *norm1b = nullptr, *norm2b = nullptr;  // norms behind mixer and MLP
+    float *left_out = nullptr, *right_out = nullptr;  // norms of a parallel mixer's two results
+    float *talk = nullptr, *temp = nullptr;  // mixing matrix of the heads' scores, temperatures
+    float *gu_bias = nullptr, *down_bias = nullptr;
+    std::vector<float> gu_bias_host;     // gate and up interleaved as their rows are
+    float *lin_conv_w = nullptr, *lin_rate = nullptr, *lin_up_g = nullptr, *lin_decay = nullptr;  // delta rule: convolution, -exp(A_log), gate up-projection; retention: decays
+    size_t lin_conv_at = 0;
+    struct Pending { std::string name, rest; int dtype; std::vector<int64_t> shape; std::vector<uint8_t> data; };
+    std::vector<Pending> pending;        // tensors that came before those that tell their layer's sizes
     double* turns = nullptr;             // rotation, turns per position of every pair
     size_t conv_at = 0, gla_at = 0;      // this layer's part of a sequence's state, in floats
 };
@@ -86,6 +97,9 @@ struct LinOpt {
     const float* gate = nullptr;
     int ld_gate = 0;
     int group_x = 0;                     // grouped projections: inputs of one group to the next
+    int gate_per = 0;                    // EPI_GATE: columns that share a gate
+    float limit = 0.f;                   // EPI_GLU
+    int glu_n = 0;
     TurnedPairs turn{};
     float softcap = 0.f;
 };
@@ -95,6 +109,7 @@ struct LinOpt {
 struct ParallelColumns {
     int q = 0, k = 0, v = 0, gate = 0, gates = 0;          // attention, its output gates
     int lq = 0, lk = 0, lv = 0, lg = 0, la = 0;            // linear attention, gate, decay latent
+    int lb = 0, lgl = 0;                                   // delta rule: step sizes, gate latent
     int dq = 0, dkv = 0;                                   // latents of queries; of keys and values with the rotated part behind
     int router = 0, row_gate = 0, ff_gate = 0, ff_up = 0, ff = 0;  // dense or shared feed-forward
     int n = 0, ld = 0;
@@ -200,7 +215,20 @@ class Engine {
     void free_parallel_scratch();
     SideArgs side_args(int l, int M, bool tall, const ParallelColumns& c, const int32_t* row_pos, const int32_t* row_seq) const;
     int enqueue_parallel_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int next_lm_rows, int* launches);
+    // listed designs with sublayers between two norms (engine_sandwich.cu)
+    int load_sandwich_tensor(int layer, const std::string& name, const std::string& rest, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
+    int load_group(LinearW& L, int groups, int g, int K, int k_part, int group_n, int dtype, const void* host, size_t nbytes);
+    int finalize_sandwich();
+    int alloc_sandwich_scratch();
+    int enqueue_sandwich(int M, bool tall, const LayerW* joined, const float* post_w, const float* next_w, int* launches);
+    SideArgs sandwich_side_args(int l, int M, const int32_t* row_pos, const int32_t* row_seq) const;
+    RecurArgs recur_args(int l, int M, bool tall, const int32_t* row_pos, const int32_t* row_seq) const;
+    int enqueue_sandwich_layer(int l, int M, const int32_t* row_pos, const int32_t* row_seq, int lm_rows, int* launches);
+    int enqueue_sandwich_logits(const float* x, int rows, bool normed, float* dst, const struct ArgmaxFold& fold, int* launches);
+    bool final_norm_fits(int M, int lm_rows) const { return lm_rows == M && !lm_pick_; }
     // shared by the listed designs
+    int load_key_up(LayerW& w, const LayerSpec& s, const std::string& name, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
+    int load_value_up(LayerW& w, const LayerSpec& s, const std::string& name, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes);
     GqaRuns pass_runs(int M, int* longest) const;
     GqaAttnArgs gqa_attn_args(int l, int M, bool tall, const int32_t* row_pos, const int32_t* row_seq) const;
     int enqueue_latent_attn(int l, int M, bool tall, const int32_t* row_pos, const int32_t* row_seq, int* launches);
@@ -304,6 +332,7 @@ class Engine {
     float* cat_ = nullptr;           // inputs of a parallel layer's output projection,
     unsigned char *xpack_cat_ = nullptr, *xpack_cq_ = nullptr;  // their image; that of the queries' latents
     int cat_ld_ = 0;
+    float* lin_rows_ = nullptr;      // rows of a pass that are prepared for a recurrence
     double* turns_ = nullptr;        // sinusoidal positions: turns per position of every pair of elements
     float* sub_ = nullptr;           // what a sublayer gave back, before its norm
     float* v_first_ = nullptr;       // values of the layer that the others blend in

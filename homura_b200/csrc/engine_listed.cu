@@ -113,6 +113,7 @@ int Engine::load_listed_tensor(const std::string& name, int dtype, const int64_t
         if (rc == HM_OK && spec_.norm_offset) HM_CUDA(launch_add_constant(w.in_ln, H_, 1.f, stream_));
         return rc;
     }
+    if (spec_.sandwich) return load_sandwich_tensor((int)li, name, rest, dtype, shape, ndim, host, nbytes);
     if (spec_.parallel) return load_parallel_tensor((int)li, name, rest, dtype, shape, ndim, host, nbytes);
     if (rest == "norm2") return vec(&w.post_ln, H_);
     if (s.mixer == MIX_GQA) return load_gqa_tensor(w, s, name, rest, dtype, shape, ndim, host, nbytes);
@@ -133,6 +134,7 @@ int Engine::load_listed_tensor(const std::string& name, int dtype, const int64_t
 }
 
 int Engine::finalize_listed() {
+    if (spec_.sandwich) return finalize_sandwich();
     if (spec_.parallel) return finalize_parallel();
     for (int i = 0; i < L_; ++i) {
         const LayerW& l = layers_[i];
@@ -176,6 +178,7 @@ int Engine::alloc_listed_scratch(int cap) {
     for (const LayerSpec& s : spec_.layers) {
         kmax = std::max(kmax, std::max(s.heads * s.vdim, s.ff));
         if (spec_.parallel) raw = std::max(raw, (size_t)parallel_columns(s).ld);
+        if (spec_.sandwich) raw = std::max(raw, (size_t)sandwich_columns(s).ld);
         if (s.mixer != MIX_LATENT) {
             raw = std::max(raw, (size_t)(s.heads * s.dim + s.kv_heads * (s.dim + s.vdim) + 3) / 4 * 4);
             continue;
@@ -183,7 +186,7 @@ int Engine::alloc_listed_scratch(int cap) {
         raw = std::max(raw, (size_t)in_ld(s));
         const int rank = s.latent_rank();
         lat = std::max(lat, (size_t)s.heads * rank);
-        q_img = std::max(q_img, s.heads * tc_xpack_bytes(TC_ROWS, s.q_rank ? s.q_stride() : s.dim));
+        q_img = std::max(q_img, s.heads * tc_xpack_bytes(TC_ROWS, s.rot_dim ? s.q_stride() : s.dim));
         ctx_img = std::max(ctx_img, s.heads * tc_xpack_bytes(TC_ROWS, rank));
         kmax = std::max(kmax, std::max(s.dim, rank));
         // splits times rows never exceed the SMs times the rows that share a CTA (latent_pick_nsplit)
@@ -215,8 +218,9 @@ int Engine::alloc_listed_scratch(int cap) {
         HM_CUDA(get(&xpack_q_, q_img));
         HM_CUDA(get(&xpack_ctx_, ctx_img));
     }
-    const int rc = alloc_gqa_scratch();
-    return rc ? rc : alloc_parallel_scratch();
+    int rc = alloc_gqa_scratch();
+    if (rc == HM_OK) rc = alloc_parallel_scratch();
+    return rc ? rc : alloc_sandwich_scratch();
 }
 
 void Engine::free_listed_cache() {
@@ -243,7 +247,7 @@ int Engine::alloc_listed_cache(int batch, size_t n_pages) {
             HM_CUDA(cudaMemset(v_pool_[l], 0, vb));
             continue;
         }
-        if (s.kv_from >= 0) continue;
+        if (s.mixer != MIX_LATENT || s.kv_from >= 0) continue;
         const size_t bytes = n_pages * latent_page_elems(s.latent_rank(), kv_bf16_) * (kv_bf16_ ? 2 : 4);
         HM_CUDA(cudaMalloc(&lat_pool_[l], bytes));
         HM_CUDA(cudaMemset(lat_pool_[l], 0, bytes));
@@ -253,9 +257,11 @@ int Engine::alloc_listed_cache(int batch, size_t n_pages) {
         const LayerSpec& s = spec_.layers[l];
         LayerW& w = layers_[l];
         w.conv_at = state_floats_;
-        if (s.conv > 1) state_floats_ += ((size_t)(s.conv - 1) * (s.heads * s.dim + s.kv_heads * (s.dim + s.vdim)) + 3) / 4 * 4;
+        if (s.conv > 1) state_floats_ += ((size_t)(s.conv - 1) * (s.heads * s.dim + s.kv_heads * (s.dim + (s.tied_values ? 0 : s.vdim))) + 3) / 4 * 4;
+        w.lin_conv_at = state_floats_;
+        if (s.lin_conv > 1) state_floats_ += ((size_t)(s.lin_conv - 1) * s.lin_channels() + 3) / 4 * 4;
         w.gla_at = state_floats_;
-        if (s.mixer == MIX_PARALLEL) state_floats_ += s.lin_heads * gla_state_floats(s.lin_dim, s.lin_vdim);
+        if (s.linear()) state_floats_ += s.lin_heads * gla_state_floats(s.lin_dim, s.lin_vdim);
     }
     if (state_floats_) {
         HM_CUDA(cudaMalloc(&state_, batch * state_floats_ * 4));
@@ -371,18 +377,20 @@ int Engine::enqueue_latent_attn(int l, int M, bool tall, const int32_t* row_pos,
     a.row_pos = row_pos;
     a.row_seq = row_seq;
     a.scale = s.scale;
+    a.window = s.window;
+    const int longest = s.window > 0 ? (int)std::min((long)pass_longest_, (long)s.window + TC_ROWS + 128) : pass_longest_;  // tokens that the tiles of a row range over
     const size_t per = (size_t)M * s.heads;
     const int most = (int)std::min<size_t>(std::min(lat_acc_floats_ / (per * rank), lat_ml_floats_ / (per * 2)), 256);
     // tiles: every run is cut at the multiples of the rows that share a CTA
     int longest_run = 1, tiles = 0;
     for (auto& r : pass_runs_) longest_run = std::max(longest_run, r.second);
-    a.rows_per_tile = latent_rows_per_tile(longest_run, pass_longest_, s.heads, rank, kv_bf16_);
+    a.rows_per_tile = latent_rows_per_tile(longest_run, longest, s.heads, rank, kv_bf16_);
     for (auto& r : pass_runs_) tiles += (r.first + r.second - 1) / a.rows_per_tile - r.first / a.rows_per_tile + 1;
     if (a.rows_per_tile == 1) tiles = M;
     a.tiles = tiles;
     a.unmerged = !tall && rank % 4 == 0 ? 1 : 0;
     a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
-    a.nsplit = latent_pick_nsplit(tiles, a.rows_per_tile, s.heads, rank, kv_bf16_, pass_longest_, sm_count_, most, a.unmerged != 0);
+    a.nsplit = latent_pick_nsplit(tiles, a.rows_per_tile, s.heads, rank, kv_bf16_, longest, sm_count_, most, a.unmerged != 0);
     pass_nsplit_ = a.unmerged ? a.nsplit : 1;
     a.part_acc = lat_acc_;
     a.part_ml = lat_ml_;

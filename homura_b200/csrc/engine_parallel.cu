@@ -68,11 +68,14 @@ ParallelColumns parallel_columns(const LayerSpec& s) {
 // ---- weights -------------------------------------------------------------------------------------
 
 void Engine::note_shape(const std::string& name, const std::vector<int64_t>& shape) {
-    if (!spec_.parallel || name.empty() || name[0] != 'l' || shape.size() != 2) return;
+    if (!(spec_.parallel || spec_.sandwich) || name.empty() || name[0] != 'l' || shape.size() != 2 || shape[0] < 1 || shape[0] > 1 << 16) return;
     const size_t dot = name.find('.');
-    if (dot == std::string::npos || name.substr(dot) != ".mix.right.a1" || name.find_first_not_of("0123456789", 1) != dot) return;
+    if (dot == std::string::npos || name.find_first_not_of("0123456789", 1) != dot) return;
     const long l = std::atol(name.c_str() + 1);
-    if (l >= 0 && l < L_ && shape[0] > 0 && shape[0] <= 1 << 16 && spec_.layers[l].decay_rank == 0) spec_.layers[l].decay_rank = (int)shape[0];
+    if (l < 0 || l >= L_) return;
+    LayerSpec& s = spec_.layers[l];
+    if (name.substr(dot) == ".mix.right.a1" && s.decay_rank == 0) s.decay_rank = (int)shape[0];
+    if (name.substr(dot) == ".mix.right.g1" && s.lin_kind == LIN_DELTA && s.gate_rank == 0) s.gate_rank = (int)shape[0];
 }
 
 int Engine::upload(float** dst, const std::vector<float>& v) {
@@ -118,6 +121,32 @@ int Engine::load_inputs(LinearW& L, int k_total, int k_off, int k_part, int N, i
     if (ce != cudaSuccess) return cuda_fail(ce, "load_inputs");
     L.loaded_parts++;
     return HM_OK;
+}
+
+// Keys are W_uk c, so a query meets the latents as W_uk^T q; its rotated part passes to the end of the cached row.
+int Engine::load_key_up(LayerW& w, const LayerSpec& s, const std::string& name, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes) {
+    const int R = s.latent_rank(), qs = s.q_stride();
+    const uint16_t* bits = static_cast<const uint16_t*>(host);
+    if (ndim != 2 || shape[0] != (int64_t)s.heads * s.dim || shape[1] != s.kv_rank) return fail(HM_ERR_INVALID, "unexpected shape for tensor " + name);
+    if (dtype != HM_BF16 || nbytes != (size_t)s.heads * s.dim * s.kv_rank * 2) return fail(HM_ERR_UNSUPPORTED, "projection weights of this design must be stored as bf16");
+    std::vector<uint16_t> m((size_t)s.heads * qs * R, 0);
+    for (int h = 0; h < s.heads; ++h) {
+        uint16_t* g = &m[(size_t)h * qs * R];
+        for (int e = 0; e < s.rot_dim; ++e) g[(size_t)e * R + s.kv_rank + e] = 0x3f80;  // 1
+        for (int d = 0; d < s.dim; ++d) std::memcpy(g + (size_t)(s.rot_dim + d) * R, bits + ((size_t)h * s.dim + d) * s.kv_rank, (size_t)s.kv_rank * 2);
+    }
+    return load_grouped(w.kup, s.heads, qs, R, true, dtype, m.data(), m.size() * 2);
+}
+
+// The rotated part of a cached row is no value.
+int Engine::load_value_up(LayerW& w, const LayerSpec& s, const std::string& name, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes) {
+    const int R = s.latent_rank();
+    const uint16_t* bits = static_cast<const uint16_t*>(host);
+    if (ndim != 2 || shape[0] != (int64_t)s.heads * s.vdim || shape[1] != s.kv_rank) return fail(HM_ERR_INVALID, "unexpected shape for tensor " + name);
+    if (dtype != HM_BF16 || nbytes != (size_t)s.heads * s.vdim * s.kv_rank * 2) return fail(HM_ERR_UNSUPPORTED, "projection weights of this design must be stored as bf16");
+    std::vector<uint16_t> m((size_t)s.heads * s.vdim * R, 0);
+    for (int i = 0; i < s.heads * s.vdim; ++i) std::memcpy(&m[(size_t)i * R], bits + (size_t)i * s.kv_rank, (size_t)s.kv_rank * 2);
+    return load_grouped(w.vup, s.heads, R, s.vdim, false, dtype, m.data(), m.size() * 2);
 }
 
 int Engine::load_parallel_tensor(int layer, const std::string& name, const std::string& rest, int dtype, const int64_t* shape, int ndim, const void* host, size_t nbytes) {
@@ -203,25 +232,9 @@ int Engine::load_parallel_tensor(int layer, const std::string& name, const std::
                 }
             return load_linear(w.uq, s.q_rank, s.heads * qs, 0, s.heads * qs, -1, dtype, m.data(), m.size() * 2);
         }
-        if (t == "uk") {
-            // keys are W_uk c, so a query meets the latents as W_uk^T q; its rotated part passes to the end of the cached row
-            if (!is2((int64_t)s.heads * s.dim, s.kv_rank)) return bad_shape();
-            if (!bf16()) return fail(HM_ERR_UNSUPPORTED, "projection weights of this design must be stored as bf16");
-            std::vector<uint16_t> m((size_t)s.heads * qs * R, 0);
-            for (int h = 0; h < s.heads; ++h) {
-                uint16_t* g = &m[(size_t)h * qs * R];
-                for (int e = 0; e < s.rot_dim; ++e) g[(size_t)e * R + s.kv_rank + e] = 0x3f80;  // 1
-                for (int d = 0; d < s.dim; ++d) std::memcpy(g + (size_t)(s.rot_dim + d) * R, bits + ((size_t)h * s.dim + d) * s.kv_rank, (size_t)s.kv_rank * 2);
-            }
-            return load_grouped(w.kup, s.heads, qs, R, true, dtype, m.data(), m.size() * 2);
-        }
-        if (t != "uv") return unknown();
-        // the rotated part of a cached row is no value
-        if (!is2((int64_t)s.heads * s.vdim, s.kv_rank)) return bad_shape();
-        if (!bf16()) return fail(HM_ERR_UNSUPPORTED, "projection weights of this design must be stored as bf16");
-        std::vector<uint16_t> m((size_t)s.heads * s.vdim * R, 0);
-        for (int i = 0; i < s.heads * s.vdim; ++i) std::memcpy(&m[(size_t)i * R], bits + (size_t)i * s.kv_rank, (size_t)s.kv_rank * 2);
-        return load_grouped(w.vup, s.heads, R, s.vdim, false, dtype, m.data(), m.size() * 2);
+        if (t == "uk") return load_key_up(w, s, name, dtype, shape, ndim, host, nbytes);
+        if (t == "uv") return load_value_up(w, s, name, dtype, shape, ndim, host, nbytes);
+        return unknown();
     };
     auto feed_forward = [&](const std::string& t) -> int {
         std::string part = t;
@@ -301,7 +314,7 @@ void Engine::free_parallel_scratch() {
         if (p) cudaFree(p);
         p = nullptr;
     };
-    fr(normed_); fr(cat_); fr(xpack_cat_); fr(xpack_cq_);
+    fr(normed_); fr(cat_); fr(xpack_cat_); fr(xpack_cq_); fr(lin_rows_);
 }
 
 int Engine::alloc_parallel_scratch() {

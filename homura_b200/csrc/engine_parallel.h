@@ -4,4 +4,5 @@
 
 namespace hm {
 ParallelColumns parallel_columns(const LayerSpec& s);
+ParallelColumns sandwich_columns(const LayerSpec& s);
 }  // namespace hm

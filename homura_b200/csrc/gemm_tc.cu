@@ -395,9 +395,31 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                 }
             }
         }
+    } else if (X && a.epi == EPI_GLU) {
+        // block = 64 gate features followed by the 64 matching up features; padding ones come out as zero
+        for (int idx = tid; idx < rows * 8; idx += TC_THREADS) {
+            const int m = m_lo + idx / 8, c = (idx % 8) * 8, j = nblk * 64 + c;
+            float v[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                float g = tile[m * BM + c + e], u = tile[m * BM + 64 + c + e];
+                if (a.bias) {
+                    g += __ldg(a.bias + n0 + c + e);
+                    u += __ldg(a.bias + n0 + 64 + c + e);
+                }
+                v[e] = j + e < a.glu_n ? clamped_glu(g, u, a.limit) : 0.f;
+            }
+            if (a.xp_out) {
+                tc_xpack_store8(a.xp_out, a.xp_mpad, m, j, v);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 8; ++e)
+                    if (j + e < a.glu_n) a.y[(size_t)m * a.ldy + j + e] = v[e];
+            }
+        }
     } else if (X && (a.epi == EPI_GATE || a.epi == EPI_SQRELU)) {
         auto act = [&](int m, int n, float v) {
-            if (a.epi == EPI_GATE) return v / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + n)));
+            if (a.epi == EPI_GATE) return v / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + (a.gate_per > 1 ? n / a.gate_per : n))));
             v = fmaxf(v, 0.f);
             return v * v;
         };
@@ -406,7 +428,7 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
             for (int idx = tid; idx < rows * nc; idx += TC_THREADS) {
                 const int m = m_lo + idx / nc, c = (idx % nc) * 8;
                 float v[8];
-                if (a.epi == EPI_GATE && (a.ld_gate & 3) == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 15) == 0) {
+                if (a.epi == EPI_GATE && a.gate_per <= 1 && (a.ld_gate & 3) == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 15) == 0) {
                     const float4 g0 = ld_cg_f32x4(a.gate + (size_t)m * a.ld_gate + n0 + c), g1 = ld_cg_f32x4(a.gate + (size_t)m * a.ld_gate + n0 + c + 4);
                     const float g[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
 #pragma unroll
@@ -921,7 +943,7 @@ static cudaError_t launch_gemm_tc_v(const TcArgs& a_in, cudaStream_t st, bool pd
 }
 
 cudaError_t launch_gemm_tc(const TcArgs& a, cudaStream_t st, bool pdl) {
-    const bool x = a.group_blocks || a.out_scale || a.split_xp || a.epi == EPI_GATE || a.epi == EPI_SQRELU;
+    const bool x = a.group_blocks || a.out_scale || a.split_xp || a.epi == EPI_GATE || a.epi == EPI_SQRELU || a.epi == EPI_GLU;
     if (a.ex.n) return launch_gemm_tc_v<2>(a, st, pdl);
     if (a.turn.turns || a.softcap > 0.f) return launch_gemm_tc_v<3>(a, st, pdl);
     return x ? launch_gemm_tc_v<1>(a, st, pdl) : launch_gemm_tc_v<0>(a, st, pdl);

@@ -43,6 +43,9 @@ struct TcArgs {
     const float* out_scale;  // EPI_STORE, optional [N]: y = resid + out_scale * (acc + bias)
     const float* gate;       // EPI_GATE: [M][ld_gate]
     int ld_gate;
+    int gate_per;            // EPI_GATE: > 1: so many columns share a gate
+    float limit;             // EPI_GLU
+    int glu_n;               // EPI_GLU: outputs (the last block may be padded)
     // Grouped projection (block-diagonal weights, e.g. one matrix per attention head): group g owns group_blocks blocks
     // of 128 features, reads the activation image at xp + g * group_xp and writes outputs [g * group_n, (g + 1) * group_n).
     int group_blocks, group_n;
@@ -55,7 +58,7 @@ struct TcArgs {
     TurnedPairs turn;        // EPI_STORE: with turn.turns
     float softcap;           // EPI_LOGITS: > 0: softcap * tanh(logit / softcap)
     TcExperts ex;
-    unsigned char* xp_out;   // EPI_SWIGLU, EPI_GATE, EPI_EXPERT and EPI_SQRELU, optional: write the result as packed activations for the next GEMM instead of y
+    unsigned char* xp_out;   // EPI_SWIGLU, EPI_GLU, EPI_GATE, EPI_EXPERT and EPI_SQRELU, optional: write the result as packed activations for the next GEMM instead of y
     int xp_mpad;
     // RMSNorm across two GEMMs without a packing launch in between.  Producer side (EPI_STORE): besides y, the
     // epilogue writes (y * next_norm_w) as the packed activations of the next GEMM and, per 128-feature block,

@@ -590,7 +590,7 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
         if (a.epi == EPI_GATE) {
             for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) {
                 const int m = idx / SLAB, n = n0 + (idx % SLAB);
-                if (n < n_end && m < a.m_valid) a.y[(size_t)m * a.ldy + n] = vals[idx] / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + n)));
+                if (n < n_end && m < a.m_valid) a.y[(size_t)m * a.ldy + n] = vals[idx] / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + (a.gate_per > 1 ? n / a.gate_per : n))));
             }
         } else if (a.epi == EPI_SQRELU) {
             for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) {
@@ -601,7 +601,20 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
                 }
             }
         }
-        stored = a.epi == EPI_GATE || a.epi == EPI_SQRELU;
+        if (a.epi == EPI_GLU) {
+            for (int idx = tid; idx < M * 64; idx += GEMV_THREADS) {
+                const int m = idx / 64, c = idx % 64, j = slab * 64 + c;
+                if (j < a.glu_n && m < a.m_valid) {
+                    float g = vals[m * SLAB + c], u = vals[m * SLAB + 64 + c];
+                    if (a.bias) {
+                        g += __ldg(a.bias + n0 + c);
+                        u += __ldg(a.bias + n0 + 64 + c);
+                    }
+                    a.y[(size_t)m * a.ldy + j] = clamped_glu(g, u, a.limit);
+                }
+            }
+        }
+        stored = a.epi == EPI_GATE || a.epi == EPI_SQRELU || a.epi == EPI_GLU;
     }
     if (stored) {
     } else if (a.epi == EPI_STORE) {

@@ -3,6 +3,7 @@
 //   gqa_post_kernel        norms, temperature and blending of a projection's queries, keys and values; page slots
 //   gqa_attn_kernel        CUDA cores, f32 or bf16 pages, any head size
 //   gqa_attn_mma_kernel    bf16 pages on warp-level MMAs, prompts and decoding alike
+//   talk_attn_mma_kernel   the same where the heads mix their scores (gqa_talk.cuh)
 //
 // MMA kernel.  A CTA serves a tile of (row, query head) pairs of one key/value head: the heads of a decoded token, or the heads of
 // several rows of a prompt that follow one another, so that a page is read once for all of them.  Pages come through a ring of
@@ -34,7 +35,7 @@ constexpr int MAX_STAGES = 8;
 constexpr int MAX_CLUSTER = 16;
 
 // ---- after the projection ------------------------------------------------------------------------
-template <bool X>
+template <int X>
 __global__ void __launch_bounds__(POST_WARPS * 32) gqa_post_kernel(const GqaPostArgs a) {
     extern __shared__ __align__(16) float post_sm[];
     pdl_launch_dependents();
@@ -90,12 +91,15 @@ struct PageList {
     int n, head, gap;
     __device__ __forceinline__ int page(int i) const { return i < head ? i : i + gap; }
 };
+// First position that a row at `pos` sees behind the kept ones.
+__device__ __forceinline__ int first_visible(const GqaAttnArgs& a, int pos) { return a.chunk > 0 ? pos - pos % a.chunk : a.window > 0 ? max(0, pos - a.window + 1) : 0; }
+
 template <bool X>
 __device__ __forceinline__ PageList visible_pages(const GqaAttnArgs& a, int lo, int hi) {
     const int all = hi / GQA_PAGE + 1;
     PageList l{all, all, 0};
-    if (X && a.window > 0) {
-        const int from = max(0, lo - a.window + 1) / GQA_PAGE;  // first page of the window
+    if (X && (a.window > 0 || a.chunk > 0)) {
+        const int from = first_visible(a, lo) / GQA_PAGE;  // first page of the window
         l.head = min((a.keep_first + GQA_PAGE - 1) / GQA_PAGE, from);
         l.gap = from - l.head;
         l.n = all - l.gap;
@@ -166,11 +170,11 @@ __device__ __forceinline__ void combine_and_store(const GqaAttnArgs& a, const fl
 }
 
 // ---- CUDA cores ------------------------------------------------------------------------------------
-// One CTA = one row, key/value head and split.
-template <bool BF16, bool X>
+// One CTA = one row, key/value head and split; TALK: all heads of a row and split.
+template <bool BF16, bool X, bool TALK>
 __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a) {
     extern __shared__ __align__(16) float sm[];
-    const int g = a.heads / a.pool.kv_heads, kvh = blockIdx.y, m = blockIdx.z, split = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int gq = a.heads / a.pool.kv_heads, g = TALK ? a.heads : gq, kvh = blockIdx.y, m = blockIdx.z, split = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int dim = a.pool.dim, vdim = a.pool.vdim, dp = gqa_pad(dim), vp = gqa_pad(vdim), ldo = vp + 4;
     float* q_s = sm;                  // [g][dp]
     float* o_s = q_s + g * dp;        // [g][ldo]
@@ -178,9 +182,11 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
     float* ml = p_s + g * GQA_PAGE;   // [g][2]
     float* corr = ml + 2 * g;         // [g]
     float* wts = corr + g;            // [nsplit][g]
+    float* raw = TALK ? wts + a.nsplit * g : nullptr;  // [g][64] scores before they are mixed
     pdl_launch_dependents();
     pdl_wait();
-    const int pos = a.row_pos[m], len = pos + 1;
+    const int pos = a.row_pos[m], len = pos + 1, from = X ? first_visible(a, pos) : 0;
+    auto seen = [&](int tok) { return !X || tok >= from || tok < a.keep_first; };
     const PageList list = visible_pages<X>(a, pos, pos);
     const int pps = (list.n + a.nsplit - 1) / a.nsplit, p0 = split * pps, p1 = min(list.n, p0 + pps);
     const int32_t* pt = a.pool.page_table + (size_t)a.row_seq[m] * a.pool.max_pages;
@@ -196,14 +202,15 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
     __syncthreads();
     for (int pi = p0; pi < p1; ++pi) {
         const int p = list.page(pi);
-        const size_t kb = (size_t)pt[p] * gqa_page_elems(a.pool.kv_heads, dim) + (size_t)kvh * GQA_PAGE * dp;
-        const size_t vb = (size_t)pt[p] * gqa_page_elems(a.pool.kv_heads, vdim) + (size_t)kvh * GQA_PAGE * vp;
+        const size_t kb0 = (size_t)pt[p] * gqa_page_elems(a.pool.kv_heads, dim) + (size_t)kvh * GQA_PAGE * dp;
+        const size_t vb0 = (size_t)pt[p] * gqa_page_elems(a.pool.kv_heads, vdim) + (size_t)kvh * GQA_PAGE * vp;
         const int nt = min(GQA_PAGE, len - p * GQA_PAGE);
         for (int i = tid; i < g * GQA_PAGE; i += A_THREADS) {
             const int j = i / GQA_PAGE, t = i % GQA_PAGE;
-            float s = -INFINITY;
-            if (t < nt && (!X || a.window == 0 || pos - (p * GQA_PAGE + t) < a.window || p * GQA_PAGE + t < a.keep_first)) {
+            float s = TALK ? 0.f : -INFINITY;
+            if (t < nt && seen(p * GQA_PAGE + t)) {
                 const float* q = q_s + j * dp;
+                const size_t kb = TALK ? kb0 + (size_t)(j / gq) * GQA_PAGE * dp : kb0;
                 s = 0.f;
                 for (int c = 0; c < dp / 8; ++c) {
                     float k[8];
@@ -221,9 +228,19 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
                 }
                 if (a.bias) s += __ldg(a.bias + (size_t)(kvh * g + j) * (a.reach + 1) + min(pos - (p * GQA_PAGE + t), a.reach));
             }
-            p_s[i] = s;
+            (TALK ? raw : p_s)[i] = s;
         }
         __syncthreads();
+        if constexpr (TALK) {
+            for (int i = tid; i < g * GQA_PAGE; i += A_THREADS) {
+                const int j = i / GQA_PAGE, t = i % GQA_PAGE;
+                const float* w = a.talk + (size_t)j * g;
+                float s = 0.f;
+                for (int e = 0; e < g; ++e) s = fmaf(__ldg(w + e), raw[e * GQA_PAGE + t], s);
+                p_s[i] = t < nt && seen(p * GQA_PAGE + t) ? s : -INFINITY;
+            }
+            __syncthreads();
+        }
         for (int j = warp; j < g; j += A_THREADS / 32) {
             const float s0 = p_s[j * GQA_PAGE + lane], s1 = p_s[j * GQA_PAGE + 32 + lane];
             const float old = ml[2 * j], mx = fmaxf(old, warp_max(fmaxf(s0, s1)));  // a page of the list has a token that is seen
@@ -241,6 +258,7 @@ __global__ void __launch_bounds__(A_THREADS) gqa_attn_kernel(const GqaAttnArgs a
         __syncthreads();
         for (int i = tid; i < g * vdim; i += A_THREADS) {
             const int j = i / vdim, d = i - j * vdim;
+            const size_t vb = TALK ? vb0 + (size_t)(j / gq) * GQA_PAGE * vp : vb0;
             float s = 0.f;
 #pragma unroll 4
             for (int t = 0; t < nt; ++t) {
@@ -297,7 +315,7 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
     int32_t* pt_s = reinterpret_cast<int32_t*>(dyn + ring_bytes + b_query_bytes(NT, dp) + b_recv_bytes(NT, vp, a.nsplit));  // this CTA's pages
     __shared__ uint64_t full[MAX_STAGES], empty[MAX_STAGES], s_rbar;
     __shared__ volatile int s_abort;
-    __shared__ int s_pos[P], s_bias[P];  // position of the pair's row (-1: no such pair), first element of its bias row
+    __shared__ int s_pos[P], s_bias[P], s_from[X ? P : 1];  // position of the pair's row (-1: no such pair), first element of its bias row, first position it sees
 
     // this tile's pairs: run, first pair, rows
     int row0, rows, pair0;
@@ -333,16 +351,16 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
     if (!a.early) pdl_wait();
     const int row_hi = row0 + (pair0 + pairs - 1) / g;
     const int seq = a.row_seq[row0], len = a.row_pos[row_hi] + 1;
-    const PageList list = visible_pages<X>(a, X && a.window > 0 ? a.row_pos[row0 + pair0 / g] : 0, len - 1);
+    const PageList list = visible_pages<X>(a, X && (a.window > 0 || a.chunk > 0) ? a.row_pos[row0 + pair0 / g] : 0, len - 1);
     auto page_at = [&](int i) { return X ? list.page(i) : i; };
     const int pps = (list.n + a.nsplit - 1) / a.nsplit;
     const int p0 = split * pps, np = max(0, min(list.n, p0 + pps) - p0);
     const int32_t* pt = a.pool.page_table + (size_t)seq * a.pool.max_pages;
     for (int i = tid; i < np; i += B_THREADS) pt_s[i] = pt[page_at(p0 + i)];
-    const int seen = a.window > 0 ? a.window : 0x7fffffff;
     if (tid < P) {
         const int pr = pair0 + tid;
         s_pos[tid] = tid < pairs ? a.row_pos[row0 + pr / g] : -1;
+        if (X) s_from[tid] = tid < pairs ? first_visible(a, s_pos[tid]) : 0;
         s_bias[tid] = (kvh * g + (tid < pairs ? pr % g : 0)) * (a.reach + 1);
     }
     __syncthreads();
@@ -403,13 +421,14 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
     }
     if (warp < ATT_WARPS) {
         const int u = warp & 3, mj = lane >> 3, mr = lane & 7;
-        int pos[NT][2], brow[NT][2];
+        int pos[NT][2], brow[NT][2], from[NT][2];
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
             for (int hh = 0; hh < 2; ++hh) {
                 pos[nt][hh] = s_pos[nt * 8 + 2 * tig + hh];
                 brow[nt][hh] = s_bias[nt * 8 + 2 * tig + hh];
+                from[nt][hh] = X ? s_from[nt * 8 + 2 * tig + hh] : 0;
             }
         const uint32_t k_lane = (uint32_t)(((mj >> 1) * GQA_PAGE + u * 16 + (mj & 1) * 8 + mr) * 16), v_lane = (uint32_t)(((mj & 1) * GQA_PAGE + u * 16 + (mj >> 1) * 8 + mr) * 16);
         // pages alternate between the two groups of four warps; the stage count is even, so a stage is always the same group's
@@ -454,8 +473,8 @@ __global__ void __launch_bounds__(B_THREADS, NT == 1 && VT <= 8 ? 2 : 1) gqa_att
                             s0 += __ldg(a.bias + brow[nt][hh] + min(max(n0, 0), a.reach));
                             s1 += __ldg(a.bias + brow[nt][hh] + min(max(n1, 0), a.reach));
                         }
-                        s0 = n0 >= 0 && (!X || n0 < seen || t0 < a.keep_first) ? s0 : -INFINITY;
-                        s1 = n1 >= 0 && (!X || n1 < seen || t1 < a.keep_first) ? s1 : -INFINITY;
+                        s0 = n0 >= 0 && (!X || t0 >= from[nt][hh] || t0 < a.keep_first) ? s0 : -INFINITY;
+                        s1 = n1 >= 0 && (!X || t1 >= from[nt][hh] || t1 < a.keep_first) ? s1 : -INFINITY;
                         float mx = fmaxf(s0, s1);
 #pragma unroll
                         for (int o = 4; o < 32; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -646,9 +665,9 @@ int clusters_at_once(void (*kern)(KArgs...), int cluster, int threads, size_t sm
 // Pages that a tile of so many (row, head) pairs can see.
 int most_pages(const GqaAttnArgs& a, int pairs) {
     const int all = (a.longest + GQA_PAGE - 1) / GQA_PAGE;
-    if (a.window == 0) return all;
+    if (a.window == 0 && a.chunk == 0) return all;
     const int rows = std::min(a.longest_run, (pairs + a.heads / a.pool.kv_heads - 1) / (a.heads / a.pool.kv_heads) + 1);
-    const long seen = (a.keep_first + GQA_PAGE - 1) / GQA_PAGE + ((long)a.window + rows - 2) / GQA_PAGE + 2;
+    const long seen = (a.keep_first + GQA_PAGE - 1) / GQA_PAGE + ((long)(a.chunk > 0 ? a.chunk : a.window) + rows - 2) / GQA_PAGE + 2;
     return (int)std::min<long>(all, seen);
 }
 
@@ -702,21 +721,28 @@ cudaError_t launch_mma_n(const GqaAttnArgs& a, int sm_count, cudaStream_t st, bo
     return launch_mma<VT, VT <= 4 ? 4 : 2, X>(a, sm_count, st, pdl);
 }
 
+#include "gqa_talk.cuh"
+
 }  // namespace
 
 cudaError_t launch_gqa_post(const GqaPostArgs& a, cudaStream_t st, bool pdl) {
     const dim3 grid((unsigned)a.M, (unsigned)gqa_post_blocks(a)), block(POST_WARPS * 32);
-    return gqa_post_buf(a) > 0 ? launch_clustered(gqa_post_kernel<true>, grid, block, gqa_post_smem(a), 1, st, pdl, a) : launch_clustered(gqa_post_kernel<false>, grid, block, 0, 1, st, pdl, a);
+    if (a.varied()) return launch_clustered(gqa_post_kernel<2>, grid, block, gqa_post_smem(a), 1, st, pdl, a);
+    return gqa_post_buf(a) > 0 ? launch_clustered(gqa_post_kernel<1>, grid, block, gqa_post_smem(a), 1, st, pdl, a) : launch_clustered(gqa_post_kernel<0>, grid, block, 0, 1, st, pdl, a);
 }
 
 cudaError_t launch_gqa_attn(const GqaAttnArgs& a_in, int sm_count, cudaStream_t st, bool pdl) {
     GqaAttnArgs a = a_in;
     if (a.M < 1 || a.M > GQA_MAX_ROWS || a.nsplit > MAX_CLUSTER || a.heads % a.pool.kv_heads != 0) return cudaErrorInvalidValue;
     if (!a.bias) a.reach = 0;
-    const bool x = a.window > 0 || a.sink || a.gate_kind != GATE_NONE || a.out_scale != 0.f || a.ld_out != 0;
+    const bool x = a.window > 0 || a.chunk > 0 || a.talk || a.sink || a.gate_kind != GATE_NONE || a.out_scale != 0.f || a.ld_out != 0;
     if (a.ld_out == 0) a.ld_out = a.heads * a.pool.vdim;
     const int g = a.heads / a.pool.kv_heads, dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
     if (a.runs.n == 0) a.longest_run = 1;
+    if (a.talk) {
+        if (a.bias) return cudaErrorInvalidValue;
+        return launch_talk(a, sm_count, st, pdl);
+    }
     const long ppc_most = most_pages(a, 32);
     if (a.pool.bf16 && vp <= 256 && dp <= 256 && ppc_most <= 8192) {
         if (vp <= 64) return x ? launch_mma_n<4, true>(a, sm_count, st, pdl) : launch_mma_n<4, false>(a, sm_count, st, pdl);
@@ -728,9 +754,11 @@ cudaError_t launch_gqa_attn(const GqaAttnArgs& a_in, int sm_count, cudaStream_t 
     const size_t smem = sizeof(float) * (size_t)g * (dp + vp + 4 + GQA_PAGE + 3 + a.nsplit);
     const dim3 grid((unsigned)a.nsplit, (unsigned)a.pool.kv_heads, (unsigned)a.M);
     auto go = [&](auto kern) { return launch_clustered(kern, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a); };
-    if (x) return a.pool.bf16 ? go(gqa_attn_kernel<true, true>) : go(gqa_attn_kernel<false, true>);
-    return a.pool.bf16 ? go(gqa_attn_kernel<true, false>) : go(gqa_attn_kernel<false, false>);
+    if (x) return a.pool.bf16 ? go(gqa_attn_kernel<true, true, false>) : go(gqa_attn_kernel<false, true, false>);
+    return a.pool.bf16 ? go(gqa_attn_kernel<true, false, false>) : go(gqa_attn_kernel<false, false, false>);
 }
+
+bool gqa_talk_fits(int heads, int dim, int vdim) { return talk_plain_smem(heads, gqa_pad(dim), gqa_pad(vdim), MAX_CLUSTER) <= 226 * 1024; }
 
 cudaError_t launch_gqa_read(const GqaPool& pool, int seq, int len, float* k, float* v, cudaStream_t st) {
     const size_t total = (size_t)pool.kv_heads * len * (pool.dim + pool.vdim);

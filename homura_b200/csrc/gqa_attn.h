@@ -74,6 +74,14 @@ struct GqaPostArgs {
     // rotation of the first rot_dims elements of queries and keys: pair (i, i + rot_dims / 2) makes turns[i] turns per position
     int rot_dims;
     const double* turns;
+    // what only some designs have (the post kernels' third variant)
+    int rot_neighbours;      // pairs are (2 i, 2 i + 1)
+    int conv_silu;           // convolved values pass through the silu
+    int tied_values;         // no values in `raw`: a key as it is before its rotation is its value
+    int v_heads;             // with k_out: heads of values
+    const float* head_scale; // [heads] or null: queries times this
+    float *k_out, *v_out;    // rows [M][kv_heads * dim] and [M][v_heads * vdim] instead of page slots
+    bool varied() const { return rot_neighbours || conv_silu || tied_values || head_scale || k_out; }
 };
 cudaError_t launch_gqa_post(const GqaPostArgs& a, cudaStream_t st, bool pdl);
 
@@ -85,6 +93,8 @@ struct GqaAttnArgs {
     const float* bias;       // [heads][reach + 1] by distance (the last one for all beyond), times log2 e; or null
     int reach;
     int window, keep_first;  // window > 0: a row at position p sees the positions above p - window and those below keep_first
+    int chunk;               // > 0: a row at position p sees the positions from p / chunk * chunk on
+    const float* talk;       // [heads][heads] or null: the scores that the softmax gets are this matrix times the heads' scores
     const float* sink;       // [heads] or null: one more score in the denominator (not scaled, as it is in the softmax)
     const float* gate;       // results are multiplied by the sigmoid of gate [M][ld_gate] (per element, or per head)
     int ld_gate, gate_kind;  // OutGate
@@ -103,6 +113,8 @@ struct GqaAttnArgs {
     int tiles, tiles_per_row, stages;
 };
 cudaError_t launch_gqa_attn(const GqaAttnArgs& a, int sm_count, cudaStream_t st, bool pdl);
+// Whether heads that mix their scores fit the kernels (all heads of a row share a CTA).
+bool gqa_talk_fits(int heads, int dim, int vdim);
 // Positions [0, len) of a sequence as f32 [kv_heads][len][dim] and [kv_heads][len][vdim].
 cudaError_t launch_gqa_read(const GqaPool& pool, int seq, int len, float* k, float* v, cudaStream_t st);
 

@@ -7,26 +7,29 @@ namespace hm {
 
 constexpr int POST_WARPS = 8;
 
-__host__ __device__ __forceinline__ int gqa_post_slots(const GqaPostArgs& a) { return a.heads + 2 * a.pool.kv_heads; }
+__host__ __device__ __forceinline__ int gqa_post_v_heads(const GqaPostArgs& a) { return a.tied_values ? 0 : a.k_out ? a.v_heads : a.pool.kv_heads; }
+__host__ __device__ __forceinline__ int gqa_post_slots(const GqaPostArgs& a) { return a.heads + a.pool.kv_heads + gqa_post_v_heads(a); }
 __host__ __device__ __forceinline__ int gqa_post_blocks(const GqaPostArgs& a) { return (gqa_post_slots(a) + POST_WARPS - 1) / POST_WARPS; }  // per row
 // a head's elements per warp, kept only where they are needed twice
-__host__ __device__ __forceinline__ int gqa_post_buf(const GqaPostArgs& a) { return a.taps > 0 || a.rot_dims > 0 || a.qk_norm == QKN_UNIT ? (a.pool.dim > a.pool.vdim ? a.pool.dim : a.pool.vdim) : 0; }
+__host__ __device__ __forceinline__ int gqa_post_buf(const GqaPostArgs& a) { return a.taps > 0 || a.rot_dims > 0 || a.qk_norm >= QKN_UNIT || a.conv_silu || a.tied_values ? (a.pool.dim > a.pool.vdim ? a.pool.dim : a.pool.vdim) : 0; }
 __host__ __device__ __forceinline__ size_t gqa_post_smem(const GqaPostArgs& a) { return sizeof(float) * POST_WARPS * (size_t)gqa_post_buf(a); }
 
-// Rotates `half` pairs (buf[i], buf[i + half]) with the lanes of a warp.
-__device__ __forceinline__ void rotate_pairs(float* buf, int half, const double* turns, int pos, int lane) {
+// Rotates `half` pairs (buf[i], buf[i + half]), or neighbours, with the lanes of a warp.
+__device__ __forceinline__ void rotate_pairs(float* buf, int half, const double* turns, int pos, int lane, bool neighbours = false) {
     for (int i = lane; i < half; i += 32) {
         float c, s;
         rotation_at(__ldg(turns + i), pos, c, s);
-        const float u = buf[i], v = buf[i + half];
-        buf[i] = fmaf(u, c, -v * s);
-        buf[i + half] = fmaf(v, c, u * s);
+        const int a = neighbours ? 2 * i : i, b = neighbours ? 2 * i + 1 : i + half;
+        const float u = buf[a], v = buf[b];
+        buf[a] = fmaf(u, c, -v * s);
+        buf[b] = fmaf(v, c, u * s);
     }
 }
 
-// X: with convolution, rotation or norms behind it (the plain variant keeps no head in shared memory).  Row m of one head slot ([heads] queries, [kv_heads] keys, [kv_heads] values).  part_q / part_k: sums of squares of the whole
+// X: 1 with convolution, rotation or norms behind it (the plain variant keeps no head in shared memory), 2 with everything that
+// GqaPostArgs::varied() names as well.  Row m of one head slot ([heads] queries, [kv_heads] keys, [kv_heads] values).  part_q / part_k: sums of squares of the whole
 // projections (QKN_ALL); first: the first row of m's run.
-template <bool X>
+template <int X>
 __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int slot, int first, int pos, int seq, size_t page, float part_q, float part_k, float* buf) {
     const int lane = threadIdx.x & 31;
     const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
@@ -36,9 +39,14 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
     const int ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n;  // first channel
     const float* x = a.raw + (size_t)m * a.ld + ch0;
     const bool buffered = X && gqa_post_buf(a) > 0;
+    const int VH = X == 2 ? gqa_post_v_heads(a) : G;
+    auto put_page = [&](void* pool, size_t off, float v) {
+        if (a.pool.bf16) reinterpret_cast<uint16_t*>(pool)[off] = f32_to_bf16_rne(v);
+        else reinterpret_cast<float*>(pool)[off] = v;
+    };
     if (buffered) {
         const float* state = a.taps > 1 ? a.conv_state + (size_t)seq * a.conv_stride + ch0 : nullptr;
-        const int channels = nq + nk + G * vdim;
+        const int channels = nq + nk + VH * vdim;
         for (int d = lane; d < n; d += 32) {
             float v = ld_cg_f32(x + d);
             if (a.taps > 0) {
@@ -55,7 +63,9 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
                     if (j <= back) v = fmaf(u[j - 1], __ldg(w + a.taps - 1 - j), v);
                 for (int j = 4; j <= back; ++j) v = fmaf(input(j), __ldg(w + a.taps - 1 - j), v);
             }
+            if (X == 2 && a.conv_silu) v = v / (1.0f + expf(-v));
             buf[d] = v;
+            if (X == 2 && a.tied_values && !is_q) put_page(a.pool.v, page * gqa_page_elems(G, dim) + (size_t)h * GQA_PAGE * gqa_pad(dim) + gqa_tile_off(t, d), v);
         }
         __syncwarp();
     }
@@ -76,34 +86,35 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
         const float* w = a.qk_norm == QKN_HEAD || a.qk_norm == QKN_ALL ? (is_q ? a.q_norm : a.k_norm) + (a.qk_norm == QKN_ALL ? (size_t)h * dim : 0) : nullptr;
         auto normed = [&](int d) { return w ? (at(d) * inv) * __ldg(w + d) : at(d); };
         float unit = 1.f;
-        const bool turned = X && a.rot_dims > 0, after = X && (turned || a.qk_norm == QKN_UNIT);
+        const bool turned = X && a.rot_dims > 0, after = X && (turned || a.qk_norm >= QKN_UNIT);
         if (after) {
             if (w)
                 for (int d = lane; d < dim; d += 32) buf[d] = normed(d);
             __syncwarp();
-            if (turned) rotate_pairs(buf, a.rot_dims / 2, a.turns, pos, lane);
+            if (turned) rotate_pairs(buf, a.rot_dims / 2, a.turns, pos, lane, X == 2 && a.rot_neighbours);
             __syncwarp();
-            if (a.qk_norm == QKN_UNIT) {
+            if (a.qk_norm >= QKN_UNIT) {
                 float s = 0.f;
                 for (int d = lane; d < dim; d += 32) s = fmaf(buf[d], buf[d], s);
-                unit = 1.0f / sqrtf(warp_sum(s) / (float)dim + a.eps);
+                s = warp_sum(s);
+                unit = 1.0f / sqrtf((X == 2 && a.qk_norm == QKN_SUM ? s : s / (float)dim) + a.eps);
             }
         }
         auto value = [&](int d) { return after ? buf[d] * unit : normed(d); };
         if (is_q) {
             float f = 1.f;
             if (a.temp_every > 0) f = 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
+            if (X == 2 && a.head_scale) f = __ldg(a.head_scale + h);
             float* o = a.q_out + (size_t)m * nq + (size_t)h * dim;
             for (int d = lane; d < dim; d += 32) o[d] = (value(d) * f) * a.q_scale;
+        } else if (X == 2 && a.k_out) {
+            for (int d = lane; d < dim; d += 32) a.k_out[(size_t)m * nk + (size_t)h * dim + d] = value(d);
         } else {
             const size_t base = page * gqa_page_elems(G, dim) + (size_t)h * GQA_PAGE * gqa_pad(dim);
-            for (int d = lane; d < dim; d += 32) {
-                const float v = value(d);
-                const size_t off = base + gqa_tile_off(t, d);
-                if (a.pool.bf16) reinterpret_cast<uint16_t*>(a.pool.k)[off] = f32_to_bf16_rne(v);
-                else reinterpret_cast<float*>(a.pool.k)[off] = v;
-            }
+            for (int d = lane; d < dim; d += 32) put_page(a.pool.k, base + gqa_tile_off(t, d), value(d));
         }
+    } else if (X == 2 && a.k_out) {
+        for (int d = lane; d < vdim; d += 32) a.v_out[(size_t)m * VH * vdim + (size_t)h * vdim + d] = at(d);
     } else {
         float* kept = a.v_first ? a.v_first + (size_t)m * G * vdim + (size_t)h * vdim : nullptr;
         const float lam = kept && a.v_lambda ? __ldg(a.v_lambda) : 0.f;
@@ -114,23 +125,21 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
                 if (a.v_lambda) v = (1.0f - lam) * v + lam * ld_cg_f32(kept + d);
                 else kept[d] = v;
             }
-            const size_t off = base + gqa_tile_off(t, d);
-            if (a.pool.bf16) reinterpret_cast<uint16_t*>(a.pool.v)[off] = f32_to_bf16_rne(v);
-            else reinterpret_cast<float*>(a.pool.v)[off] = v;
+            put_page(a.pool.v, base + gqa_tile_off(t, d), v);
         }
     }
     __syncwarp();
 }
 
 // Row m and POST_WARPS head slots from blk * POST_WARPS on.
-template <bool X>
+template <int X>
 __device__ __forceinline__ void gqa_post_block(const GqaPostArgs& a, int m, int blk, float* smem) {
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int G = a.pool.kv_heads, dim = a.pool.dim, vdim = a.pool.vdim, nq = a.heads * dim, nk = G * dim;
     const int slot0 = blk * POST_WARPS, slot = slot0 + warp;
     __shared__ float s_part[2][POST_WARPS];
     // positions and pages do not depend on the launch in front
-    auto page_of = [&](int seq, int pos) { return (size_t)a.pool.page_table[(size_t)seq * a.pool.max_pages + pos / GQA_PAGE]; };
+    auto page_of = [&](int seq, int pos) { return X == 2 && a.k_out ? (size_t)0 : (size_t)a.pool.page_table[(size_t)seq * a.pool.max_pages + pos / GQA_PAGE]; };
     const int pos = a.row_pos[m], seq = a.row_seq[m];
     const size_t page = page_of(seq, pos);
     pdl_wait();
@@ -178,7 +187,7 @@ __device__ __forceinline__ void gqa_post_block(const GqaPostArgs& a, int m, int 
     for (int r = first + 1; r < min(end, first + keep); ++r) gqa_post_row<X>(a, r, slot, first, pos + r - first, seq, page_of(seq, pos + r - first), 0.f, 0.f, buf);
     // the run's last inputs replace the kept ones (a lane keeps the channels that it has read)
     const bool is_v = slot >= a.heads + G, is_q = slot < a.heads;
-    const int h = is_v ? slot - a.heads - G : is_q ? slot : slot - a.heads, n = is_v ? vdim : dim, ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n, channels = nq + nk + G * vdim;
+    const int h = is_v ? slot - a.heads - G : is_q ? slot : slot - a.heads, n = is_v ? vdim : dim, ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n, channels = nq + nk + (X == 2 ? gqa_post_v_heads(a) : G) * vdim;
     float* state = a.conv_state + (size_t)seq * a.conv_stride + ch0;
     for (int r = max(first, end - keep); r < end; ++r)
 #pragma unroll 4

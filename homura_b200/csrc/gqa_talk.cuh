@@ -1,0 +1,335 @@
+// Attention whose heads mix their scores (GqaAttnArgs::talk): part of gqa_attn.cu.
+//
+// A CTA takes all heads of a tile of rows (rows of a run that follow one another; a decoded token is a tile of one) and a share of
+// their pages.  A page comes block by block through a ring of bulk copies: the keys of every key head, then the values of every one.
+//   scores^T [16 tokens x pairs] = K [16 x dim] . Q^T     per key head, into shared memory
+//   mix, mask, softmax                                    per (row, head): lanes along the tokens, f32
+//   out^T    [16 values x pairs] += V^T [16 x 64] . P^T   per key head, accumulators in shared memory
+// A pair is a (row, head); those of a key head are the MMAs' columns, eight at a time.  Queries and weights are three bf16 terms each.
+
+constexpr int TALK_MAX_STAGES = 16;
+constexpr int TALK_RAW_LD = GQA_PAGE + 4, TALK_P_LD = GQA_PAGE + 8;  // row strides of scores (floats) and weights (bf16): no bank conflicts
+
+struct TalkGeom {
+    int rows;       // of a tile
+    int per;        // pairs of a key head: rows * heads per key head
+    int ntile;      // tiles of eight of them
+    int cols2;      // pairs of columns that a tile uses (accumulators of the others are not kept)
+    int stages;
+    uint32_t block; // bytes of a ring stage
+    size_t front;   // bytes of the ring, which takes the results afterwards
+    size_t q, raw, p, corr, o, ml, talk, wts, pages, smem;  // offsets from the front's end, total
+};
+
+inline bool talk_geom(const GqaAttnArgs& a, int rows, int nsplit, int pages_per_cta, TalkGeom* g) {
+    const int H = a.heads, G = a.pool.kv_heads, gq = H / G, dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
+    const size_t pairs = (size_t)rows * H, padded = pairs + 8;
+    g->rows = rows;
+    g->per = rows * gq;
+    g->ntile = (g->per + 7) / 8;
+    g->cols2 = g->per >= 8 ? 4 : (g->per + 1) / 2;
+    g->block = (uint32_t)(GQA_PAGE * std::max(dp, vp) * 2);
+    size_t at = 0;
+    auto take = [&](size_t bytes) {
+        const size_t first = at;
+        at += (bytes + 15) / 16 * 16;
+        return first;
+    };
+    g->q = take(3 * padded * (dp + 8) * 2);
+    g->raw = take(pairs * TALK_RAW_LD * 4);
+    g->p = take(3 * padded * TALK_P_LD * 2);
+    g->corr = take(padded * 4);
+    g->o = take((size_t)G * (vp / 16) * g->ntile * g->cols2 * 8 * 16);
+    g->ml = take(pairs * 8);
+    g->talk = take((size_t)H * ((H + 3) / 4 * 4) * 4);
+    g->wts = take(pairs * nsplit * 4);
+    g->pages = take((size_t)pages_per_cta * 4);
+    const size_t result = pairs * (vp + 4) * 4, most = 226 * 1024;
+    if (at + std::max(result, 2 * (size_t)g->block) + 128 > most) return false;
+    g->stages = (int)std::min<size_t>({(most - at - 128) / g->block, (size_t)TALK_MAX_STAGES, (size_t)2 * G * std::max(1, pages_per_cta)});
+    g->front = (std::max(result, (size_t)g->stages * g->block) + 127) / 128 * 128;
+    g->smem = g->front + at;
+    return g->smem <= most;
+}
+
+__global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const GqaAttnArgs a, const TalkGeom geo) {
+    extern __shared__ __align__(128) unsigned char dyn[];
+    const int H = a.heads, G = a.pool.kv_heads, gq = H / G, dim = a.pool.dim, vdim = a.pool.vdim, dp = gqa_pad(dim), vp = gqa_pad(vdim), kt_n = dp / 16, vt_n = vp / 16, ldo = vp + 4;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, split = blockIdx.x, NST = geo.stages, HP = (H + 3) & ~3;
+    unsigned char *ring = dyn, *back = dyn + geo.front;
+    const int padded = geo.rows * H + 8, ldq = dp + 8;
+    uint16_t* qs = reinterpret_cast<uint16_t*>(back + geo.q);        // [3][padded][ldq], pairs by key head
+    float* raw = reinterpret_cast<float*>(back + geo.raw);           // [row][head][TALK_RAW_LD]
+    uint16_t* ps = reinterpret_cast<uint16_t*>(back + geo.p);        // [3][padded][TALK_P_LD], pairs by key head
+    float* corr = reinterpret_cast<float*>(back + geo.corr);         // [padded]
+    float4* os = reinterpret_cast<float4*>(back + geo.o);            // [key head][16 values][tile of pairs][two columns][8 lanes]
+    float* ml = reinterpret_cast<float*>(back + geo.ml);             // [row][head][2]
+    float* tk = reinterpret_cast<float*>(back + geo.talk);           // [head that is read][head, padded]
+    float* wts = reinterpret_cast<float*>(back + geo.wts);
+    int32_t* pt_s = reinterpret_cast<int32_t*>(back + geo.pages);
+    __shared__ uint64_t full[TALK_MAX_STAGES], empty[TALK_MAX_STAGES];
+    __shared__ volatile int s_abort;
+
+    int row0 = blockIdx.z, rows = 1;
+    if (a.runs.n > 0) {
+        int r = 0;
+        while (r + 1 < a.runs.n && a.runs.tile[r + 1] <= blockIdx.z) ++r;
+        row0 = a.runs.row[r] + (blockIdx.z - a.runs.tile[r]) * geo.rows;
+        rows = min(geo.rows, a.runs.row[r + 1] - row0);
+    }
+    const int pairs = rows * H;
+    if (tid == 0) {
+        for (int s = 0; s < NST; ++s) {
+            mb_init(&full[s], 1);
+            mb_init(&empty[s], ATT_WARPS);
+        }
+        s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    pdl_launch_dependents();
+    // positions, pages and the mixing matrix do not depend on the launch in front
+    const int seq = a.row_seq[row0], pos0 = a.row_pos[row0], len = pos0 + rows;
+    const PageList list = visible_pages<true>(a, pos0, len - 1);
+    const int pps = (list.n + a.nsplit - 1) / a.nsplit, p0 = split * pps, np = max(0, min(list.n, p0 + pps) - p0);
+    const int32_t* pt = a.pool.page_table + (size_t)seq * a.pool.max_pages;
+    for (int i = tid; i < np; i += B_THREADS) pt_s[i] = pt[list.page(p0 + i)];
+    for (int i = tid; i < H * HP; i += B_THREADS) {
+        const int e = i / HP, h = i - e * HP;
+        tk[i] = h < H ? __ldg(a.talk + (size_t)h * H + e) : 0.f;
+    }
+    for (int i = tid; i < pairs; i += B_THREADS) {
+        ml[2 * i] = -INFINITY;
+        ml[2 * i + 1] = 0.f;
+    }
+    const int o_tile = geo.cols2 * 8, o_n = G * vt_n * geo.ntile * o_tile;
+    for (int i = tid; i < o_n; i += B_THREADS) os[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    __syncthreads();
+    const unsigned char *kpool = reinterpret_cast<const unsigned char*>(a.pool.k), *vpool = reinterpret_cast<const unsigned char*>(a.pool.v);
+    const uint32_t k_bytes = (uint32_t)(GQA_PAGE * dp * 2), v_bytes = (uint32_t)(GQA_PAGE * vp * 2);
+    const int items = np * 2 * G;
+    if (warp == ATT_WARPS) {
+        if (lane == 0) {
+            int i = 0;
+            auto fetch = [&](int it) {
+                const int pg = it / (2 * G), b = it - pg * 2 * G, s = it % NST;
+                const bool is_v = b >= G;
+                const size_t tile = (size_t)pt_s[pg] * G + (is_v ? b - G : b);
+                mb_expect_tx(&full[s], is_v ? v_bytes : k_bytes);
+                bulk_copy(ring + (size_t)s * geo.block, is_v ? vpool + tile * v_bytes : kpool + tile * k_bytes, is_v ? v_bytes : k_bytes, &full[s]);
+            };
+            if (a.early)  // the captured decode step: pages in front of the newest token's are complete
+                for (; i < items && i < NST && list.page(p0 + i / (2 * G)) < (len - 1) / GQA_PAGE; ++i) fetch(i);
+            pdl_wait();
+            for (; i < items; ++i) {
+                if (i >= NST && !mb_wait(&empty[i % NST], ((i / NST) & 1u) ^ 1u, a.err_flag, &s_abort)) break;
+                fetch(i);
+            }
+        } else {
+            pdl_wait();
+        }
+    } else {
+        pdl_wait();
+        // queries: three bf16 terms, two elements a thread
+        const int d2 = dp / 2;
+#pragma unroll 4
+        for (int i = tid; i < pairs * d2; i += ATT_WARPS * 32) {
+            const int p = i / d2, d = (i - p * d2) * 2, r = p / H, h = p - r * H, qi = (h / gq) * geo.per + r * gq + h % gq;
+            const float* q = a.q + (size_t)(row0 + r) * H * dim + (size_t)h * dim + d;
+            const float x = d < dim ? ld_cg_f32(q) : 0.f, y = d + 1 < dim ? ld_cg_f32(q + 1) : 0.f;
+            uint32_t t[3];
+            bf16x2_split3(x, y, t[0], t[1], t[2]);
+#pragma unroll
+            for (int k = 0; k < 3; ++k) *reinterpret_cast<uint32_t*>(qs + (size_t)(k * padded + qi) * ldq + d) = t[k];
+        }
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        const int gid = lane >> 2, tig = lane & 3, mj = lane >> 3, mr = lane & 7;
+        for (int i = 0; i < np; ++i) {
+            const int tok0 = list.page(p0 + i) * GQA_PAGE;
+            // scores.  A wait that gives up leaves the work out; the barriers below are still met by every warp.
+            for (int g = 0; g < G; ++g) {
+                const int it = i * 2 * G + g, s = it % NST;
+                const bool ok = __all_sync(0xffffffffu, mb_wait(&full[s], (it / NST) & 1u, a.err_flag, &s_abort));
+                const uint32_t kb = s32(ring + (size_t)s * geo.block) + (uint32_t)(((mj >> 1) * GQA_PAGE + (mj & 1) * 8 + mr) * 16);
+                for (int j = (warp - g * 4 * geo.ntile) & 7; ok && j < 4 * geo.ntile; j += 8) {
+                    const int u = j & 3, nt = j >> 2;
+                    float sc[3][4];
+#pragma unroll
+                    for (int k = 0; k < 3; ++k) sc[k][0] = sc[k][1] = sc[k][2] = sc[k][3] = 0.f;
+                    const uint16_t* q = qs + (size_t)(g * geo.per + nt * 8 + gid) * ldq + 2 * tig;
+#pragma unroll 4
+                    for (int kt = 0; kt < kt_n; ++kt) {
+                        uint32_t ka[4];
+                        ldsm4(ka, kb + (uint32_t)(u * 256 + kt * (2 * GQA_PAGE * 16)));
+#pragma unroll
+                        for (int k = 0; k < 3; ++k) {
+                            const uint16_t* b = q + (size_t)k * padded * ldq + kt * 16;
+                            mma16816(sc[k], ka, *reinterpret_cast<const uint32_t*>(b), *reinterpret_cast<const uint32_t*>(b + 8));
+                        }
+                    }
+#pragma unroll
+                    for (int hh = 0; hh < 2; ++hh) {
+                        const int c = nt * 8 + 2 * tig + hh;
+                        if (c < rows * gq) {
+                            float* dst = raw + (size_t)((c / gq) * H + g * gq + c % gq) * TALK_RAW_LD + u * 16 + gid;
+                            dst[0] = (sc[2][hh] + sc[1][hh]) + sc[0][hh];
+                            dst[8] = (sc[2][2 + hh] + sc[1][2 + hh]) + sc[0][2 + hh];
+                        }
+                    }
+                }
+                __syncwarp();
+                if (lane == 0) mb_arrive(&empty[s]);
+            }
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            // four heads of a row at a time: their scores out of all heads', two tokens a lane
+            for (int w = warp; w < rows * (HP / 4); w += ATT_WARPS) {
+                const int r = w / (HP / 4), h0 = (w - r * (HP / 4)) * 4, pos = pos0 + r, from = first_visible(a, pos), ta = tok0 + 2 * lane;
+                float2 s[4];
+#pragma unroll
+                for (int k = 0; k < 4; ++k) s[k] = make_float2(0.f, 0.f);
+                const float* x = raw + (size_t)r * H * TALK_RAW_LD + 2 * lane;
+#pragma unroll 4
+                for (int e = 0; e < H; ++e) {
+                    const float2 v = *reinterpret_cast<const float2*>(x + (size_t)e * TALK_RAW_LD);
+                    const float4 t = *reinterpret_cast<const float4*>(tk + e * HP + h0);
+                    s[0].x = fmaf(t.x, v.x, s[0].x); s[0].y = fmaf(t.x, v.y, s[0].y);
+                    s[1].x = fmaf(t.y, v.x, s[1].x); s[1].y = fmaf(t.y, v.y, s[1].y);
+                    s[2].x = fmaf(t.z, v.x, s[2].x); s[2].y = fmaf(t.z, v.y, s[2].y);
+                    s[3].x = fmaf(t.w, v.x, s[3].x); s[3].y = fmaf(t.w, v.y, s[3].y);
+                }
+                const bool va = ta <= pos && (ta >= from || ta < a.keep_first), vb = ta + 1 <= pos && (ta + 1 >= from || ta + 1 < a.keep_first);
+                float mx[4], sum[4], f[4];
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    s[k].x = va ? s[k].x : -INFINITY;
+                    s[k].y = vb ? s[k].y : -INFINITY;
+                    mx[k] = fmaxf(s[k].x, s[k].y);
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], o));
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const int h = h0 + k;
+                    if (h >= H) break;
+                    const float old = ml[2 * (r * H + h)];
+                    mx[k] = fmaxf(old, mx[k]);
+                    const float ref = mx[k] == -INFINITY ? 0.f : mx[k];  // no token of this pair yet
+                    f[k] = exp2f(old - ref);
+                    s[k].x = exp2f(s[k].x - ref);
+                    s[k].y = exp2f(s[k].y - ref);
+                    uint32_t t[3];
+                    bf16x2_split3(s[k].x, s[k].y, t[0], t[1], t[2]);
+                    const int qi = (h / gq) * geo.per + r * gq + h % gq;
+#pragma unroll
+                    for (int e = 0; e < 3; ++e) *reinterpret_cast<uint32_t*>(ps + (size_t)(e * padded + qi) * TALK_P_LD + 2 * lane) = t[e];
+                }
+#pragma unroll
+                for (int k = 0; k < 4; ++k) sum[k] = s[k].x + s[k].y;
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) sum[k] += __shfl_xor_sync(0xffffffffu, sum[k], o);
+                __syncwarp();
+                if (lane == 0)
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        const int h = h0 + k;
+                        if (h >= H) break;
+                        float* m = ml + 2 * (r * H + h);
+                        m[0] = mx[k];
+                        m[1] = fmaf(m[1], f[k], sum[k]);
+                        corr[(h / gq) * geo.per + r * gq + h % gq] = f[k];
+                    }
+                __syncwarp();
+            }
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            for (int g = 0; g < G; ++g) {
+                const int it = i * 2 * G + G + g, s = it % NST, units = vt_n * geo.ntile;
+                const bool ok = __all_sync(0xffffffffu, mb_wait(&full[s], (it / NST) & 1u, a.err_flag, &s_abort));
+                const uint32_t vb = s32(ring + (size_t)s * geo.block) + (uint32_t)(((mj & 1) * GQA_PAGE + (mj >> 1) * 8 + mr) * 16);
+                for (int j = (warp - g * units) & 7; ok && j < units; j += 8) {
+                    const int nt = j / vt_n, mt = j - nt * vt_n, qi = g * geo.per + nt * 8;
+                    const bool kept = tig < geo.cols2;
+                    float4* o = os + (size_t)((g * vt_n + mt) * geo.ntile + nt) * o_tile + tig * 8 + gid;
+                    float4 c = kept ? *o : make_float4(0.f, 0.f, 0.f, 0.f);
+                    const float c0 = corr[qi + 2 * tig], c1 = corr[qi + 2 * tig + 1];
+                    float acc[3][4] = {{c.x * c0, c.y * c1, c.z * c0, c.w * c1}, {0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+                    const uint16_t* p = ps + (size_t)(qi + gid) * TALK_P_LD + 2 * tig;
+#pragma unroll
+                    for (int kt = 0; kt < 4; ++kt) {
+                        uint32_t va[4];
+                        ldsm4_trans(va, vb + (uint32_t)(mt * (2 * GQA_PAGE * 16) + kt * 256));
+#pragma unroll
+                        for (int k = 0; k < 3; ++k) {
+                            const uint16_t* b = p + (size_t)k * padded * TALK_P_LD + kt * 16;
+                            mma16816(acc[k], va, *reinterpret_cast<const uint32_t*>(b), *reinterpret_cast<const uint32_t*>(b + 8));
+                        }
+                    }
+                    if (kept) *o = make_float4((acc[2][0] + acc[1][0]) + acc[0][0], (acc[2][1] + acc[1][1]) + acc[0][1], (acc[2][2] + acc[1][2]) + acc[0][2], (acc[2][3] + acc[1][3]) + acc[0][3]);
+                }
+                __syncwarp();
+                if (lane == 0) mb_arrive(&empty[s]);
+            }
+        }
+    }
+    __syncthreads();  // every block consumed: the ring takes the results
+    float* res = reinterpret_cast<float*>(ring);  // [row][head][ldo]
+    for (int i = tid; i < o_n; i += B_THREADS) {
+        const int u = i / o_tile, e = i - u * o_tile, tig = e >> 3, gid = e & 7, nt = u % geo.ntile, gm = u / geo.ntile, g = gm / vt_n, mt = gm - g * vt_n;
+        const float4 v = os[i];
+        const float x[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int c = nt * 8 + 2 * tig + (k & 1);
+            if (c < rows * gq) res[(size_t)((c / gq) * H + g * gq + c % gq) * ldo + mt * 16 + gid + (k >> 1) * 8] = x[k];
+        }
+    }
+    combine_and_store<true>(a, res, ldo, ml, wts, pairs, [&](int p, int& row, int& head) {
+        row = row0 + p / H;
+        head = p % H;
+    });
+}
+
+inline size_t talk_plain_smem(int heads, int dp, int vp, int nsplit) { return sizeof(float) * (size_t)heads * (dp + vp + 4 + 2 * GQA_PAGE + 3 + nsplit); }
+
+inline cudaError_t launch_talk(GqaAttnArgs a, int sm_count, cudaStream_t st, bool pdl) {
+    const int dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
+    TalkGeom g{};
+    auto pages_of = [&](int rows) { return most_pages(a, rows * a.heads / a.pool.kv_heads); };
+    if (a.pool.bf16 && pages_of(1) <= 4096) {
+        const int gq = a.heads / a.pool.kv_heads;
+        const int asked = a.nsplit;
+        // rows of a run share a tile until the columns of an MMA are full
+        for (int rows = std::max(1, std::min(8 / gq, a.longest_run)); rows >= 1; rows /= 2) {
+            const int pages = pages_of(rows);
+            a.tiles = a.M;
+            if (a.runs.n > 0) {
+                a.tiles = 0;
+                for (int r = 0; r < a.runs.n; ++r) {
+                    a.runs.tile[r] = (uint16_t)a.tiles;
+                    a.tiles += (a.runs.row[r + 1] - a.runs.row[r] + rows - 1) / rows;
+                }
+                a.runs.tile[a.runs.n] = (uint16_t)a.tiles;
+            }
+            bool fits = false;
+            auto shape = [&]() { return fits = talk_geom(a, rows, a.nsplit, (pages + a.nsplit - 1) / a.nsplit, &g); };
+            if (asked > 0) {
+                a.nsplit = asked;
+                shape();
+            } else {
+                for (a.nsplit = std::max(1, std::min({sm_count / a.tiles, a.max_cluster, 8, pages})); a.nsplit >= 1; --a.nsplit)
+                    if (shape() && (a.nsplit == 1 || clusters_at_once(talk_attn_mma_kernel, a.nsplit, B_THREADS, g.smem) >= a.tiles)) break;
+            }
+            if (fits && a.nsplit >= 1) return launch_clustered(talk_attn_mma_kernel, dim3((unsigned)a.nsplit, 1, (unsigned)a.tiles), dim3(B_THREADS), g.smem, a.nsplit, st, pdl, a, g);
+        }
+        a.nsplit = asked;
+    }
+    const int pages = most_pages(a, 1);
+    if (a.nsplit < 1) a.nsplit = std::max(1, std::min({2 * sm_count / a.M, a.max_cluster, 8, pages}));
+    const size_t smem = talk_plain_smem(a.heads, dp, vp, a.nsplit);
+    if (smem > 226 * 1024) return cudaErrorInvalidValue;
+    const dim3 grid((unsigned)a.nsplit, 1, (unsigned)a.M);
+    return a.pool.bf16 ? launch_clustered(gqa_attn_kernel<true, true, true>, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a)
+                       : launch_clustered(gqa_attn_kernel<false, true, true>, grid, dim3(A_THREADS), smem, a.nsplit, st, pdl, a);
+}

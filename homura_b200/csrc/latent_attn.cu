@@ -68,8 +68,9 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const LatentAttnArgs a
     pdl_wait();
     const int m = blockIdx.x, h0 = blockIdx.y * CC_HEADS, split = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int nh = min(CC_HEADS, a.heads - h0);
-    const int len = a.row_pos[m] + 1, tiles = (len + CC_TOK - 1) / CC_TOK, per = (tiles + a.nsplit - 1) / a.nsplit;
-    const int t0 = split * per, t1 = min(tiles, t0 + per);
+    const int len = a.row_pos[m] + 1, from = a.window > 0 ? max(0, len - a.window) : 0, first = from / CC_TOK;
+    const int tiles = (len + CC_TOK - 1) / CC_TOK, per = (tiles - first + a.nsplit - 1) / a.nsplit;
+    const int t0 = first + split * per, t1 = min(tiles, t0 + per);
     for (int i = tid; i < CC_HEADS * LD; i += 256) {
         const int h = i / LD, r = i % LD;
         qs[i] = h < nh && r < R ? ld_cg_f32(a.q + (size_t)m * a.ldq + (size_t)(h0 + h) * R + r) : 0.f;
@@ -98,7 +99,7 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const LatentAttnArgs a
                 const float4 q = q4[i], c = c4[i];
                 s0 = fmaf(q.x, c.x, s0); s1 = fmaf(q.y, c.y, s1); s2 = fmaf(q.z, c.z, s2); s3 = fmaf(q.w, c.w, s3);
             }
-            const float s = tok0 + lane < len ? ((s0 + s1) + (s2 + s3)) * a.scale * LOG2E : -INFINITY;
+            const float s = tok0 + lane < len && tok0 + lane >= from ? ((s0 + s1) + (s2 + s3)) * a.scale * LOG2E : -INFINITY;
             const float nm = fmaxf(mx, warp_max(s));  // finite: a tile holds at least one visible token
             const float p = exp2f(s - nm), f = exp2f(mx - nm);
             l = l * f + warp_sum(p);
@@ -309,8 +310,9 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
     }
     const int seq = a.row_seq[m0], pos0 = a.row_pos[m0];
     const int pairs = rows * nh;  // pair p: row p / nh, head p % nh
-    const int len = pos0 + rows, tiles = (len + TOK - 1) / TOK, per = (tiles + a.nsplit - 1) / a.nsplit;
-    const int t0 = split * per, nt = min(tiles, t0 + per) - t0;
+    const int from = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;  // first position that the tile's first row sees
+    const int len = pos0 + rows, tiles = (len + TOK - 1) / TOK, per = (tiles - from / TOK + a.nsplit - 1) / a.nsplit;
+    const int t0 = from / TOK + split * per, nt = min(tiles, t0 + per) - t0;
     if (nt <= 0) {  // only with nsplit > 1
         pdl_launch_dependents();
         pdl_wait();  // the launch in front may still be reading this buffer
@@ -525,7 +527,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
             if (wbar_or(bad)) { bad = true; break; }
             unsigned char* pt = pb + (size_t)(t & 1) * (TOK / 64) * g.n * 128;
             const int tok = (t0 + t) * TOK + lane * TPL;
-            const bool whole = (t0 + t + 1) * TOK - 1 <= pos0;  // every row sees every token of the tile
+            const bool whole = (t0 + t + 1) * TOK - 1 <= pos0 && (a.window == 0 || (t0 + t) * TOK > len - 1 - a.window);  // every row sees every token of the tile
             bool moved = false;
             for (int c0 = 0; c0 < g.np; c0 += 16) {
                 // two pairs per warp side by side
@@ -543,10 +545,10 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                     }
                     ref[j] = sh.ref[p];
                     if (!whole) {
-                        const int last = sh.pos[p];
+                        const int last = sh.pos[p], before = a.window > 0 ? last - a.window : -1;
 #pragma unroll
                         for (int e = 0; e < TPL; ++e)
-                            if (tok + e > last) s[j][e] = -INFINITY;
+                            if (tok + e > last || tok + e <= before) s[j][e] = -INFINITY;
                     }
 #pragma unroll
                     for (int e = 0; e < TPL; ++e) grow |= s[j][e] > ref[j] + TCL_SLACK;

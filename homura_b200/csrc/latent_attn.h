@@ -35,6 +35,7 @@ struct LatentAttnArgs {
     const int32_t* row_pos;  // a row sees positions <= its own
     const int32_t* row_seq;
     float scale;
+    int window;              // > 0: a row at position p sees the positions above p - window only
     int rows_per_tile;       // latent_rows_per_tile: rows of one run (consecutive positions of a sequence) that may share a CTA
     int tiles;               // with rows_per_tile > 1 (at most 64 rows then): tiles the rows fall into, 0: not known
     int unmerged;            // leave the splits in part_acc / part_ml (the caller's next kernel combines them)

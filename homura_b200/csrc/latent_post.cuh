@@ -5,11 +5,11 @@
 
 namespace hm {
 
-// Row m of c [M][ldc]: rank - 2 * rot_pairs elements RMS-normed with weight w, then rot_pairs pairs (i, i + rot_pairs), rotated and
+// Row m of c [M][ldc]: rank - 2 * rot_pairs elements RMS-normed with weight w, then rot_pairs pairs (i, i + rot_pairs), or neighbours, rotated and
 // cached side by side.  All NT threads of the block; part: a float per warp.
 template <int NT, bool ROT>
 __device__ __forceinline__ void latent_write_row(const LatentPool& pool, const float* __restrict__ c, int ldc, int m, const float* __restrict__ w, float eps, const int32_t* __restrict__ row_pos, const int32_t* __restrict__ row_seq, int rot_pairs,
-                                                 const double* turns, float* part) {
+                                                 const double* turns, float* part, bool neighbours = false) {
     const int tid = threadIdx.x, lane = tid & 31, R = pool.rank, N = ROT ? R - 2 * rot_pairs : R;
     const float* x = c + (size_t)m * ldc;
     float s = 0.f;
@@ -36,7 +36,7 @@ __device__ __forceinline__ void latent_write_row(const LatentPool& pool, const f
         for (int i = NT - 1 - tid; i < rot_pairs; i += NT) {
             float cs, sn;
             rotation_at(__ldg(turns + i), pos, cs, sn);
-            const float u = ld_cg_f32(x + N + i), v = ld_cg_f32(x + N + rot_pairs + i);
+            const float u = ld_cg_f32(x + N + (neighbours ? 2 * i : i)), v = ld_cg_f32(x + N + (neighbours ? 2 * i + 1 : rot_pairs + i));
             put(N + 2 * i, fmaf(u, cs, -v * sn));
             put(N + 2 * i + 1, fmaf(v, cs, u * sn));
         }

@@ -292,11 +292,122 @@ bool read_gebilorn(const Json& j, ModelSpec* s, std::string* err) {
     return true;
 }
 
+// A number of tokens under `mask`, or none.
+bool read_mask(const Json& m, int* size, const std::string& at, std::string* err) {
+    const Json* k = m.get("mask");
+    return is_null(k) || get_int(*k, "size", size) || fail(err, at + "`mask` needs size");
+}
+
+// Retention: linear attention with a fixed decay per head.
+bool read_retention(const Json& m, LayerSpec* l, const std::string& at, std::string* err) {
+    l->mixer = MIX_LINEAR;
+    l->lin_kind = LIN_RETENTION;
+    if (!get_int(m, "heads", &l->lin_heads) || !get_int(m, "dim", &l->lin_dim) || !get_int(m, "vdim", &l->lin_vdim)) return fail(err, at + "the mixer needs heads, dim and vdim");
+    l->lin_kv_heads = l->lin_heads;
+    const Json* d = m.get("decay");
+    if (!d || d->kind != Json::Arr || (int)d->arr.size() != l->lin_heads) return fail(err, at + "`decay` needs a number per head");
+    for (const Json& v : d->arr) {
+        if (v.kind != Json::Num) return fail(err, at + "`decay` needs a number per head");
+        l->lin_decay.push_back((float)v.num);
+    }
+    return read_rotation(m, l->lin_dim, &l->rot, at, err);
+}
+
+// Attention inside chunks whose heads mix their scores, beside the gated delta rule.
+bool read_talking_delta(const Json& m, LayerSpec* l, const std::string& at, std::string* err) {
+    const Json *left = m.get("left"), *right = m.get("right");
+    double scale = 0;
+    l->mixer = MIX_PARALLEL;
+    l->lin_kind = LIN_DELTA;
+    l->tied_values = l->talking = l->sink = true;
+    l->out_gate = GATE_ELEM;
+    if (is_null(left) || is_null(right)) return fail(err, at + "the mixer needs left and right");
+    if (!get_int(*left, "heads", &l->heads) || !get_int(*left, "kv_heads", &l->kv_heads) || !get_int(*left, "dim", &l->dim) || !get_int(*left, "vdim", &l->vdim) || !get_num(*left, "scale", &scale))
+        return fail(err, at + "`left` needs heads, kv_heads, dim, vdim and scale");
+    if (l->heads % l->kv_heads != 0) return fail(err, at + "`left.kv_heads` does not divide `left.heads`");
+    if (l->vdim != l->dim) return fail(err, at + "`left.vdim` differs from `left.dim`: the values are the keys");
+    l->scale = (float)scale;
+    if (!get_count(*left, "conv", &l->conv)) return fail(err, at + "`left.conv` must be a number of taps");
+    if (!read_mask(*left, &l->chunk, at, err) || !read_rotation(*left, l->dim, &l->rot, at, err)) return false;
+    if (!get_int(*right, "heads", &l->lin_heads) || !get_int(*right, "kv_heads", &l->lin_kv_heads) || !get_int(*right, "dim", &l->lin_dim) || !get_int(*right, "vdim", &l->lin_vdim))
+        return fail(err, at + "`right` needs heads, kv_heads, dim and vdim");
+    if (l->lin_heads % l->lin_kv_heads != 0) return fail(err, at + "`right.kv_heads` does not divide `right.heads`");
+    return get_count(*right, "conv", &l->lin_conv) || fail(err, at + "`right.conv` must be a number of taps");
+}
+
+// Latent attention with a rotated part inside a window; a layer may read the latents of an earlier one.
+bool read_windowed_latent(const Json& m, const ModelSpec& s, LayerSpec* l, const std::string& at, std::string* err) {
+    double scale = 0;
+    l->mixer = MIX_LATENT;
+    l->out_gate = GATE_HEAD;
+    if (!get_int(m, "heads", &l->heads) || !get_int(m, "dim", &l->dim) || !get_int(m, "vdim", &l->vdim) || !get_int(m, "kv_rank", &l->kv_rank) || !get_int(m, "rot_dim", &l->rot_dim) || !get_num(m, "scale", &scale))
+        return fail(err, at + "the mixer needs heads, dim, rot_dim, vdim, kv_rank and scale");
+    l->scale = (float)scale;
+    if (!read_mask(m, &l->window, at, err) || !read_rotation(m, l->rot_dim, &l->rot, at, err)) return false;
+    if (l->rot.dims != l->rot_dim) return fail(err, at + "`rot.dims` differs from `rot_dim`");
+    const Json* from = m.get("kv_from");
+    if (is_null(from)) return true;
+    if (from->kind != Json::Num || from->num < 0 || from->num != std::floor(from->num) || from->num >= (double)s.layers.size()) return fail(err, at + "`kv_from` must name an earlier layer");
+    l->kv_from = (int)from->num;
+    const LayerSpec& o = s.layers[l->kv_from];
+    if (o.mixer != MIX_LATENT || o.kv_from >= 0) return fail(err, at + "`kv_from` names a layer without latents of its own");
+    if (o.kv_rank != l->kv_rank || o.rot_dim != l->rot_dim) return fail(err, at + "`kv_from` names a layer of another kv_rank or rot_dim");
+    return true;
+}
+
+// Pulenex: layer norms in front of and behind every sublayer; retention, chunked attention with talking heads beside the gated delta
+// rule, windowed latent attention; clamped gated feed-forwards with biases (or none).
+bool read_pulenex(const Json& j, ModelSpec* s, std::string* err) {
+    hm_config& c = s->cfg;
+    s->sandwich = true;
+    double num = 0;
+    if (!get_int(j, "width", &c.hidden_size) || !get_int(j, "vocab", &c.vocab_size)) return fail(err, "missing `width` or `vocab`");
+    const Json *norm = j.get("norm"), *list = j.get("layers");
+    if (!norm || !get_num(*norm, "eps", &c.rms_norm_eps)) return fail(err, "`norm` needs `eps`");
+    if (!get_num(j, "logit_scale", &num)) return fail(err, "missing `logit_scale`");
+    s->logit_scale = (float)num;
+    if (!list || list->kind != Json::Arr || list->arr.empty()) return fail(err, "missing `layers`");
+    for (size_t i = 0; i < list->arr.size(); ++i) {
+        const Json& e = list->arr[i];
+        const std::string at = "layer " + std::to_string(i) + ": ";
+        LayerSpec l;
+        std::string type, kind;
+        const Json *m = e.get("mixer"), *mlp = e.get("mlp");
+        if (!get_str(e, "type", &type) || is_null(m)) return fail(err, at + "missing `type` or `mixer`");
+        if (type == "retention") {
+            if (!read_retention(*m, &l, at, err)) return false;
+        } else if (type == "parallel") {
+            if (!read_talking_delta(*m, &l, at, err)) return false;
+        } else if (type == "latent_attention") {
+            if (!read_windowed_latent(*m, *s, &l, at, err)) return false;
+        } else {
+            return fail(err, at + "unknown mixer type");
+        }
+        if (!is_null(mlp)) {
+            if (!get_str(*mlp, "kind", &kind) || kind != "dense") return fail(err, at + "unknown mlp");
+            l.mlp = MLP_GLU;
+            l.act = GLU_CLAMPED;
+            l.mlp_bias = true;
+            if (!get_int(*mlp, "ff", &l.ff) || !get_num(*mlp, "limit", &num)) return fail(err, at + "`mlp` needs ff and limit");
+            l.limit = (float)num;
+        }
+        c.num_attention_heads = std::max(c.num_attention_heads, std::max(l.heads, l.lin_heads));
+        c.num_key_value_heads = std::max(c.num_key_value_heads, std::max(l.kv_heads, 1));
+        c.head_dim = std::max(c.head_dim, std::max(l.dim + l.rot_dim, l.lin_dim));
+        c.intermediate_size = std::max(c.intermediate_size, l.ff);
+        s->layers.push_back(l);
+    }
+    c.num_hidden_layers = (int)s->layers.size();
+    c.max_position_embeddings = 1 << 30;  // rotations are computed: the cache is the only limit
+    c.intermediate_size = std::max(c.intermediate_size, 1);
+    return true;
+}
+
 struct Design {
     const char* name;
     bool (*read)(const Json&, ModelSpec*, std::string*);
 };
-const Design kDesigns[] = {{"Tunitar", read_tunitar}, {"Dipisun", read_dipisun}, {"Gebilorn", read_gebilorn}};
+const Design kDesigns[] = {{"Tunitar", read_tunitar}, {"Dipisun", read_dipisun}, {"Gebilorn", read_gebilorn}, {"Pulenex", read_pulenex}};
 
 }  // namespace
 
@@ -377,6 +488,30 @@ std::string parallel_layer_json(const LayerSpec& l) {
     std::snprintf(t, sizeof(t), ",\"ff\":%d,\"experts\":%d,\"top\":%d,\"router_scale\":%.9g,\"shared_ff\":%d}", l.ff, l.experts, l.top, l.router_scale, l.shared_ff);
     return o + t;
 }
+std::string sandwich_layer_json(const LayerSpec& l) {
+    char t[768];
+    std::string o = "{\"type\":\"";
+    auto put = [&](const char* f, auto... v) {
+        std::snprintf(t, sizeof(t), f, v...);
+        o += t;
+    };
+    auto rot = [&]() { put(",\"rot\":{\"dims\":%d,\"base\":%.9g}", l.rot.dims, l.rot.base); };
+    if (l.mixer == MIX_LINEAR) {
+        put("retention\",\"heads\":%d,\"dim\":%d,\"vdim\":%d", l.lin_heads, l.lin_dim, l.lin_vdim);
+        o += ",\"decay\":[";
+        for (size_t i = 0; i < l.lin_decay.size(); ++i) put(i ? ",%.9g" : "%.9g", l.lin_decay[i]);
+        o += "]";
+    } else if (l.mixer == MIX_LATENT) {
+        put("latent_attention\",\"heads\":%d,\"dim\":%d,\"rot_dim\":%d,\"vdim\":%d,\"kv_rank\":%d,\"scale\":%.9g,\"window\":%d,\"kv_from\":%s", l.heads, l.dim, l.rot_dim, l.vdim, l.kv_rank, l.scale, l.window,
+            l.kv_from < 0 ? "null" : std::to_string(l.kv_from).c_str());
+    } else {
+        put("parallel\",\"heads\":%d,\"kv_heads\":%d,\"dim\":%d,\"vdim\":%d,\"scale\":%.9g,\"chunk\":%d,\"conv\":%d", l.heads, l.kv_heads, l.dim, l.vdim, l.scale, l.chunk, l.conv);
+        put(",\"linear\":{\"heads\":%d,\"kv_heads\":%d,\"dim\":%d,\"vdim\":%d,\"conv\":%d}", l.lin_heads, l.lin_kv_heads, l.lin_dim, l.lin_vdim, l.lin_conv);
+    }
+    rot();
+    put(",\"ff\":%d,\"limit\":%.9g}", l.ff, l.limit);
+    return o;
+}
 }  // namespace
 
 std::string layers_json(const ModelSpec& spec) {
@@ -385,8 +520,8 @@ std::string layers_json(const ModelSpec& spec) {
         const LayerSpec& l = spec.layers[i];
         char t[768];
         if (i) o += ",";
-        if (spec.parallel) {
-            o += parallel_layer_json(l);
+        if (spec.parallel || spec.sandwich) {
+            o += spec.parallel ? parallel_layer_json(l) : sandwich_layer_json(l);
             continue;
         }
         if (l.mixer == MIX_LATENT) {

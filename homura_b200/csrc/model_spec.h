@@ -12,12 +12,14 @@
 
 namespace hm {
 
-// MIX_PARALLEL: grouped-query attention and gated linear attention side by side
-enum MixerKind { MIX_GQA = 0, MIX_LATENT = 1, MIX_PARALLEL = 2 };
+// MIX_PARALLEL: grouped-query attention and linear attention side by side; MIX_LINEAR: linear attention alone
+enum MixerKind { MIX_GQA = 0, MIX_LATENT = 1, MIX_PARALLEL = 2, MIX_LINEAR = 3 };
+// Linear attention: a decay per key channel out of a latent; a fixed decay per head; a decay per key channel and the delta rule
+enum LinearKind { LIN_GATED = 0, LIN_RETENTION = 1, LIN_DELTA = 2 };
 enum MlpKind { MLP_NONE = 0, MLP_SWIGLU = 1, MLP_SQRELU = 2, MLP_MOE = 3, MLP_GLU = 4 };
 // RMS norm of queries and keys: none, every head by itself (one weight vector of `dim`), the whole projection at once, every head by
-// itself after its rotation and without a weight
-enum QkNorm { QKN_NONE = 0, QKN_HEAD = 1, QKN_ALL = 2, QKN_UNIT = 3 };
+// itself after its rotation and without a weight, the same by the sum of squares instead of their mean
+enum QkNorm { QKN_NONE = 0, QKN_HEAD = 1, QKN_ALL = 2, QKN_UNIT = 3, QKN_SUM = 4 };
 // Sigmoid gates on an attention's result: none, one per element, one per head
 enum OutGate { GATE_NONE = 0, GATE_ELEM = 1, GATE_HEAD = 2 };
 // Activations of gated feed-forwards: act(gate) * up
@@ -52,15 +54,23 @@ struct LayerSpec {
     int v_first = -1;
     int window = 0;         // > 0: a token sees itself and the window - 1 tokens in front of it,
     int keep_first = 0;     // and the first keep_first tokens
+    int chunk = 0;          // > 0: a token sees the tokens of its own chunk of so many, counted from the sequence's start
+    bool tied_values = false;  // values are the keys as they are before their rotation
+    bool talking = false;   // scores times a temperature per head, then mixed over the heads by a matrix
     bool sink = false;      // one more score per head in the softmax, without a value
     int out_gate = GATE_NONE;
     bool qkv_bias = false;
     int conv = 0;           // taps of a causal convolution per channel of queries, keys and values; 0: none
     RotSpec rot;            // also that of MIX_LATENT
     // MIX_PARALLEL: beside the attention above, gated linear attention with a decay per key channel
+    int lin_kind = LIN_GATED;
     int lin_heads = 0, lin_dim = 0, lin_vdim = 0;
+    int lin_kv_heads = 0;   // LIN_DELTA: heads of queries and keys
+    int lin_conv = 0;       // LIN_DELTA: taps of a causal convolution per channel of queries, keys and values
+    std::vector<float> lin_decay;  // LIN_RETENTION: per head
     float lin_tau = 1.f;
     int decay_rank = 0;     // from the tensors
+    int gate_rank = 0;      // LIN_DELTA: latent of the output gate, from the tensors
     float left_scale = 1.f, right_scale = 1.f;
     int mlp = MLP_NONE;
     int ff = 0;             // of one expert with MLP_MOE
@@ -69,8 +79,11 @@ struct LayerSpec {
     int shared_ff = 0;      // MLP_MOE: > 0: an expert that every token runs, times a sigmoid
     // MLP_MOE: `top` of experts + identity router outputs; the identity ones pass their input on
     int experts = 0, identity = 0, top = 0;
-    float limit = 0.f;      // clamp of the experts' gate (above) and up (both sides)
-    bool paged_kv() const { return mixer != MIX_LATENT; }      // caches keys and values
+    float limit = 0.f;      // GLU_CLAMPED: clamp of gate (above) and up (both sides)
+    bool mlp_bias = false;
+    bool linear() const { return mixer == MIX_PARALLEL || mixer == MIX_LINEAR; }
+    bool paged_kv() const { return mixer == MIX_GQA || mixer == MIX_PARALLEL; }  // caches keys and values
+    int lin_channels() const { return 2 * lin_kv_heads * lin_dim + lin_heads * lin_vdim; }  // LIN_DELTA: queries, keys and values
     int latent_rank() const { return kv_rank + rot_dim; }      // elements of a cached latent row
     int q_stride() const { return (dim + rot_dim + 7) / 8 * 8; }  // q_rank: a head's queries, rotated pairs first
 };
@@ -86,6 +99,8 @@ struct ModelSpec {
     float residual_mult = 1.f;
     bool sin_pos = false;     // sinusoidal position vectors are added to the embedding
     bool parallel = false;    // mixer and MLP read one norm of the residual and are added to it together
+    bool sandwich = false;    // mixer and MLP read a layer norm of the residual and give back through another one
+    float logit_scale = 1.f;
     bool norm_offset = false; // norm weights are stored as their distance from one
     float embed_scale = 1.f;
     // a second embedding by (previous token * mul_prev + token * mul_cur) mod buckets, row `buckets` for a sequence's first token

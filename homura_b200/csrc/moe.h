@@ -62,12 +62,6 @@ cudaError_t launch_expert_gate_up(const ExpertWeights& e, const float* x, int M,
 // y = resid (or nothing) + the sum over the chosen experts; y may be resid.
 cudaError_t launch_expert_down(const ExpertWeights& e, const float* act, int M, const RouteOut& r, const float* resid, float* y, cudaStream_t st, bool pdl);
 
-// Gated activation of an expert: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1).
-__device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
-    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
-    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
-}
-
 // act(gate) * up of the kinds of gated feed-forwards (GluAct).
 __device__ __forceinline__ float glu(int act, float gate, float up, float limit) {
     if (act == GLU_SILU) return gate / (1.0f + expf(-gate)) * up;

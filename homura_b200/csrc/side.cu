@@ -1,4 +1,5 @@
-// See side.h.  Blocks take their parts in order of weight: the recurrences first, then heads, latents, activations, routers.
+// See side.h.  Blocks take their parts in order of weight: the recurrences first, then heads, latents, activations, routers; the variant for
+// recurrences that are a launch of their own: factors, heads, latents.
 #include "side.h"
 
 #include <algorithm>
@@ -90,13 +91,96 @@ __device__ __forceinline__ void query_latent_block(const SideArgs& a, int m, flo
     }
 }
 
-// RD: state rows per thread of the linear attention, 0: there is none, -1: single tokens, states in shared memory
+// LR_ROWS rows and 32 columns of one of the two factors (LowRankSide); the warps share the rank.
+constexpr int LR_ROWS = 8, LR_AHEAD = 16;
+__device__ __forceinline__ int low_rank_blocks(const LowRankSide& l) { return (l.heads * l.dim + 31) / 32 + (l.heads * l.vdim + 31) / 32; }
+
+__device__ __forceinline__ void low_rank_block(const SideArgs& a, int b, float* sm) {
+    const LowRankSide& l = a.low;
+    const int per = low_rank_blocks(l), na = (l.heads * l.dim + 31) / 32, tile = b / per, cb = b - tile * per, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const bool is_a = cb < na;
+    const int N = l.heads * (is_a ? l.dim : l.vdim), col = (is_a ? cb : cb - na) * 32 + lane, rank = is_a ? l.rank_a : l.rank_g, m0 = tile * LR_ROWS, rows = min(LR_ROWS, a.M - m0);
+    const float* up = (is_a ? l.up_a : l.up_g) + col;
+    const float* lat = is_a ? l.a : l.g;
+    const bool on = col < N;
+    float w[LR_AHEAD];  // weights do not depend on the launch in front
+#pragma unroll
+    for (int i = 0; i < LR_AHEAD; ++i) {
+        const int r = warp + i * WARPS;
+        w[i] = on && r < rank ? __ldg(up + (size_t)r * N) : 0.f;
+    }
+    const float bias = is_a && on ? __ldg(l.bias + col) : 0.f, rate = is_a && on ? __ldg(l.neg_rate + col / l.dim) : 0.f;
+    pdl_wait();
+    float* red = sm + LR_ROWS * rank;  // [WARPS][LR_ROWS][32]
+    for (int i = threadIdx.x; i < rows * rank; i += THREADS) {
+        const int t = i / rank;
+        sm[i] = ld_cg_f32(lat + (size_t)(m0 + t) * a.ld + (i - t * rank));
+    }
+    __syncthreads();
+    float acc[LR_ROWS];
+#pragma unroll
+    for (int t = 0; t < LR_ROWS; ++t) acc[t] = 0.f;
+    for (int r0 = 0; r0 < rank; r0 += LR_AHEAD * WARPS) {
+#pragma unroll
+        for (int i = 0; i < LR_AHEAD; ++i) {
+            const int r = r0 + warp + i * WARPS;
+            if (r < rank) {
+#pragma unroll
+                for (int t = 0; t < LR_ROWS; ++t)
+                    if (t < rows) acc[t] = fmaf(w[i], sm[t * rank + r], acc[t]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < LR_AHEAD; ++i) {
+            const int r = r0 + (LR_AHEAD + i) * WARPS + warp;
+            w[i] = on && r < rank ? __ldg(up + (size_t)r * N) : 0.f;
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < LR_ROWS; ++t) red[(warp * LR_ROWS + t) * 32 + lane] = acc[t];
+    __syncthreads();
+    if (warp >= rows || !on) return;
+    float z = 0.f;
+#pragma unroll
+    for (int i = 0; i < WARPS; ++i) z += red[(i * LR_ROWS + warp) * 32 + lane];
+    if (is_a) {
+        z += bias;
+        l.alpha[(size_t)(m0 + warp) * N + col] = expf(rate * (fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)))));
+    } else {
+        l.gate[(size_t)(m0 + warp) * N + col] = z;
+    }
+}
+
+// RD: state rows per thread of the linear attention, 0: there is none, -1: single tokens, states in shared memory, -2: rows are
+// prepared for a recurrence, and whatever GqaPostArgs::varied() names
 template <int RD>
 __global__ void __launch_bounds__(THREADS, RD > 32 ? 1 : RD > 0 ? 2 : 3) side_kernel(const __grid_constant__ SideArgs a) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float part[WARPS];
     pdl_launch_dependents();
     int b = blockIdx.x;
+    if constexpr (RD == -2) {
+        if (b < a.n_low) {
+            low_rank_block(a, b, sm);
+            return;
+        }
+        b -= a.n_low;
+        if (b < a.n_post2) {
+            const int per = gqa_post_blocks(a.post2);
+            gqa_post_block<2>(a.post2, b / per, b % per, sm);
+            return;
+        }
+        b -= a.n_post2;
+        if (b < a.n_post) {
+            const int per = gqa_post_blocks(a.post);
+            gqa_post_block<2>(a.post, b / per, b % per, sm);
+            return;
+        }
+        b -= a.n_post;
+        pdl_wait();
+        if (b < a.n_latent) latent_write_row<THREADS, true>(a.latent.pool, a.latent.c, a.ld, b, a.latent.w, a.eps, a.row_pos, a.row_seq, a.latent.rot_pairs, a.latent.turns, part, a.latent.neighbours != 0);
+        return;
+    }
     if constexpr (RD != 0) {
         if (b < a.n_gla) {
             if constexpr (RD > 0) gla_block<RD>(a.gla, b, sm);
@@ -107,7 +191,7 @@ __global__ void __launch_bounds__(THREADS, RD > 32 ? 1 : RD > 0 ? 2 : 3) side_ke
     }
     if (b < a.n_post) {
         const int per = gqa_post_blocks(a.post);
-        gqa_post_block<true>(a.post, b / per, b % per, sm);
+        gqa_post_block<1>(a.post, b / per, b % per, sm);
         return;
     }
     b -= a.n_post;
@@ -233,7 +317,7 @@ cudaError_t launch_side(const SideArgs& a_in, int sm_count, cudaStream_t st, boo
     if (a.M < 1 || a.M > GQA_MAX_ROWS) return cudaErrorInvalidValue;
     const int runs = a.gla.runs.n ? a.gla.runs.n : a.M;
     size_t smem = 0;
-    a.n_gla = a.n_post = a.n_latent = a.n_act = a.n_route = a.n_normed = 0;
+    a.n_gla = a.n_post = a.n_latent = a.n_act = a.n_route = a.n_normed = a.n_post2 = a.n_low = 0;
     int cluster = 1, kind = 0;
     if (a.has_gla) {
         GlaArgs& g = a.gla;
@@ -257,6 +341,19 @@ cudaError_t launch_side(const SideArgs& a_in, int sm_count, cudaStream_t st, boo
         a.n_post = a.M * gqa_post_blocks(a.post);
         smem = std::max(smem, gqa_post_smem(a.post));
     }
+    if (a.has_post2 || a.has_low || (a.has_post && a.post.varied()) || (a.has_latent && a.latent.neighbours)) {
+        if (a.has_gla || a.mlp.ff || a.mlp.logits || a.mlp.normed || (a.has_latent && a.latent.q_xp)) return cudaErrorInvalidValue;
+        kind = -2;
+    }
+    if (a.has_post2) {
+        a.n_post2 = a.M * gqa_post_blocks(a.post2);
+        smem = std::max(smem, gqa_post_smem(a.post2));
+    }
+    if (a.has_low) {
+        const LowRankSide& l = a.low;
+        a.n_low = (a.M + LR_ROWS - 1) / LR_ROWS * ((l.heads * l.dim + 31) / 32 + (l.heads * l.vdim + 31) / 32);
+        smem = std::max(smem, sizeof(float) * LR_ROWS * ((size_t)std::max(l.rank_a, l.rank_g) + WARPS * 32));
+    }
     if (a.has_latent) a.n_latent = a.M * (a.latent.q_xp ? 2 : 1);
     if (a.mlp.ff) a.n_act = a.M * (((a.mlp.ff + 7) / 8 + THREADS - 1) / THREADS);
     if (a.mlp.logits) {
@@ -264,8 +361,9 @@ cudaError_t launch_side(const SideArgs& a_in, int sm_count, cudaStream_t st, boo
         smem = std::max(smem, 2 * sizeof(float) * (size_t)a.mlp.route.n_out);
     }
     if (a.mlp.normed) a.n_normed = a.M;
-    const unsigned blocks = (unsigned)((a.n_gla + a.n_post + a.n_latent + a.n_act + a.n_route + a.n_normed + cluster - 1) / cluster * cluster);
+    const unsigned blocks = (unsigned)((a.n_gla + a.n_post + a.n_latent + a.n_act + a.n_route + a.n_normed + a.n_post2 + a.n_low + cluster - 1) / cluster * cluster);
     switch (kind) {
+        case -2: return launch(side_kernel<-2>, blocks, smem, cluster, st, pdl, a);
         case -1: return launch(side_kernel<-1>, blocks, smem, cluster, st, pdl, a);
         case 4: return launch(side_kernel<4>, blocks, smem, cluster, st, pdl, a);
         case 0: return launch(side_kernel<0>, blocks, smem, cluster, st, pdl, a);

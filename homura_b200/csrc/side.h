@@ -14,6 +14,7 @@ struct LatentSide {
     const float* w;
     int rot_pairs;
     const double* turns;
+    int neighbours;          // rotated pairs are (2 i, 2 i + 1)
     // queries' latent, with q_xp: RMS-normed into the activation image of its up-projection
     const float* cq;
     int q_rank;
@@ -40,17 +41,30 @@ struct MlpSide {
     float* normed;           // or null
 };
 
+// What the gated delta rule reads besides queries, keys and values: factors out of two latents per row, [rank] x [rank][columns].
+//   alpha = exp(neg_rate[head] * softplus(up_a . a + bias))    per head and key channel
+//   gate  = up_g . g                                            per head and value channel (before its sigmoid)
+struct LowRankSide {
+    const float *a, *g;      // [M][ld] latents
+    int rank_a, rank_g;
+    const float *up_a, *bias, *neg_rate;
+    const float* up_g;
+    int heads, dim, vdim;
+    float *alpha, *gate;     // [M][heads * dim], [M][heads * vdim]
+};
+
 struct SideArgs {
     int M, ld, xp_mpad;
     float eps;
     const int32_t *row_pos, *row_seq;
-    int has_post, has_latent, has_gla;
-    GqaPostArgs post;
+    int has_post, has_latent, has_gla, has_post2, has_low;
+    GqaPostArgs post, post2;  // post2: rows for a recurrence (recur.h)
+    LowRankSide low;
     LatentSide latent;
     GlaArgs gla;
     MlpSide mlp;
     // blocks of the parts, in launch order (filled in by the launcher)
-    int n_gla, n_post, n_latent, n_act, n_route, n_normed;
+    int n_gla, n_post, n_latent, n_act, n_route, n_normed, n_post2, n_low;
 };
 cudaError_t launch_side(const SideArgs& a, int sm_count, cudaStream_t st, bool pdl);
 
