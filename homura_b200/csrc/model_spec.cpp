@@ -292,10 +292,9 @@ bool read_gebilorn(const Json& j, ModelSpec* s, std::string* err) {
     return true;
 }
 
-// A number of tokens under `mask`, or none.
 bool read_mask(const Json& m, int* size, const std::string& at, std::string* err) {
     const Json* k = m.get("mask");
-    return is_null(k) || get_int(*k, "size", size) || fail(err, at + "`mask` needs size");
+    return (!is_null(k) && get_int(*k, "size", size)) || fail(err, at + "`mask` needs size");
 }
 
 // Retention: linear attention with a fixed decay per head.
@@ -327,12 +326,12 @@ bool read_talking_delta(const Json& m, LayerSpec* l, const std::string& at, std:
     if (l->heads % l->kv_heads != 0) return fail(err, at + "`left.kv_heads` does not divide `left.heads`");
     if (l->vdim != l->dim) return fail(err, at + "`left.vdim` differs from `left.dim`: the values are the keys");
     l->scale = (float)scale;
-    if (!get_count(*left, "conv", &l->conv)) return fail(err, at + "`left.conv` must be a number of taps");
+    if (!get_int(*left, "conv", &l->conv)) return fail(err, at + "`left.conv` must be a number of taps");
     if (!read_mask(*left, &l->chunk, at, err) || !read_rotation(*left, l->dim, &l->rot, at, err)) return false;
     if (!get_int(*right, "heads", &l->lin_heads) || !get_int(*right, "kv_heads", &l->lin_kv_heads) || !get_int(*right, "dim", &l->lin_dim) || !get_int(*right, "vdim", &l->lin_vdim))
         return fail(err, at + "`right` needs heads, kv_heads, dim and vdim");
     if (l->lin_heads % l->lin_kv_heads != 0) return fail(err, at + "`right.kv_heads` does not divide `right.heads`");
-    return get_count(*right, "conv", &l->lin_conv) || fail(err, at + "`right.conv` must be a number of taps");
+    return get_int(*right, "conv", &l->lin_conv) || fail(err, at + "`right.conv` must be a number of taps");
 }
 
 // Latent attention with a rotated part inside a window; a layer may read the latents of an earlier one.

@@ -482,6 +482,117 @@ def write_gebilorn_model(model_dir: str, cfg: dict, seed: int, weights: Optional
     return _write_model(model_dir, cfg, gebilorn_tensor_specs(cfg, decay_rank), lambda s: gebilorn_tensor(seed, s) if weights is None else weights[s[0]])
 
 
+# ---- Pulenex ----------------------------------------------------------------------------------
+
+
+def pulenex_rot(dims: int, base: float = 10000.0) -> dict:
+    return {"dims": dims, "base": base}
+
+
+def pulenex_retention(heads: int, dim: int, vdim: int, rot: Optional[dict] = None, decay: Optional[List[float]] = None) -> dict:
+    """decay: per head; by default heads that forget within 4, 8, 16, ... tokens, up to 2048."""
+    decay = [1.0 - 2.0 ** -(2 + h % 10) for h in range(heads)] if decay is None else decay
+    return {"type": "retention", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "rot": rot or pulenex_rot(dim // 2 * 2), "decay": decay}}
+
+
+def pulenex_parallel(left: Tuple[int, int, int], chunk: int, conv: int, right: Tuple[int, int, int, int], right_conv: int, rot: Optional[dict] = None, scale: Optional[float] = None) -> dict:
+    """left: heads, kv_heads, dim of the chunked attention; right: heads, kv_heads, dim, vdim of the gated delta rule."""
+    h, g, d = left
+    a = {"heads": h, "kv_heads": g, "dim": d, "vdim": d, "scale": d**-0.5 if scale is None else scale, "mask": {"size": chunk}, "conv": conv, "rot": rot or pulenex_rot(d // 2 * 2)}
+    return {"type": "parallel", "mixer": {"left": a, "right": dict(zip(("heads", "kv_heads", "dim", "vdim"), right), conv=right_conv)}}
+
+
+def pulenex_latent(heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, window: int, kv_from: Optional[int] = None, base: float = 10000.0, scale: Optional[float] = None) -> dict:
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "scale": (dim + rot_dim) ** -0.5 if scale is None else scale, "mask": {"size": window}, "rot": pulenex_rot(rot_dim, base)}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": m}
+
+
+def pulenex_dense(ff: int, limit: float = 7.0) -> dict:
+    return {"kind": "dense", "ff": ff, "limit": limit}
+
+
+def pulenex_config(width: int, vocab: int, layers: List[Tuple[dict, Optional[dict]]], logit_scale: float = 1.0, eps: float = 1e-6, **extra) -> dict:
+    """layers: (mixer, mlp or None) pairs."""
+    return {"architecture": "Pulenex", "width": width, "vocab": vocab, "norm": {"eps": eps}, "logit_scale": logit_scale, "layers": [{**m, "mlp": f} for m, f in layers], **extra}
+
+
+def pulenex_uniform(width: int, vocab: int, n_layers: int, heads: int, kv_heads: int, dim: int, ff: int, kv_rank: int) -> dict:
+    """Of every four layers one runs retention, one chunked attention beside the gated delta rule, two latent attention in a window, the
+    second of which reads the first one's latents."""
+    layers = []
+    for i in range(n_layers):
+        if i % 4 == 0:
+            m = pulenex_retention(heads, dim, dim)
+        elif i % 4 == 1:
+            m = pulenex_parallel((heads, kv_heads, dim), 1024, 4, (heads, kv_heads, dim, dim), 4, pulenex_rot(dim, 500000.0))
+        else:
+            m = pulenex_latent(heads, dim, 64, dim, kv_rank, 1024, i - 1 if i % 4 == 3 else None)
+        layers.append((m, pulenex_dense(ff)))
+    return pulenex_config(width, vocab, layers)
+
+
+# Pulenex stacks with the width, depth, heads, head size and MLP parameters of the Qwen2.5 architectures above.
+PULENEX_05B = pulenex_uniform(896, 151936, 24, 14, 2, 64, 4864, 256)
+PULENEX_15B = pulenex_uniform(1536, 151936, 28, 12, 2, 128, 8960, 512)
+
+
+def pulenex_tensor_specs(cfg: dict, ranks: Tuple[int, int] = (64, 64)) -> List[Tuple[str, Tuple[int, ...], str]]:
+    """(name, shape, kind); ranks: widths of the latents of decays and of output gates."""
+    W, V = cfg["width"], cfg["vocab"]
+    specs: List[Tuple[str, Tuple[int, ...], str]] = [("embed", (V, W), "embed")]
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", layer["mixer"], layer.get("mlp")
+        specs += [(p + "norm1", (W,), "one"), (p + "norm1b", (W,), "one")]
+        if layer["type"] == "retention":
+            k, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            specs += [(p + "mix.q", (k, W), "w"), (p + "mix.k", (k, W), "w"), (p + "mix.v", (v, W), "w"), (p + "mix.g", (v, W), "w"), (p + "mix.o", (W, v), "w")]
+        elif layer["type"] == "parallel":
+            a, r, l, t = m["left"], m["right"], p + "mix.left.", p + "mix.right."
+            h, q, k = a["heads"], a["heads"] * a["dim"], a["kv_heads"] * a["dim"]
+            specs += [(l + "q", (q, W), "w"), (l + "k", (k, W), "w"), (l + "q.conv", (q, a["conv"]), "tap"), (l + "k.conv", (k, a["conv"]), "tap"), (l + "talk", (h, h), "mix"), (l + "temp", (h,), "one"), (l + "sink", (h,), "embed")]
+            specs += [(l + "g", (q, W), "w"), (l + "o", (W, q), "w"), (l + "out", (W,), "one")]
+            h, k, v = r["heads"], r["kv_heads"] * r["dim"], r["heads"] * r["vdim"]
+            specs += [(t + n, (c, W), "w") for n, c in (("q", k), ("k", k), ("v", v), ("b", h), ("a1", ranks[0]), ("g1", ranks[1]))] + [(t + n + ".conv", (c, r["conv"]), "tap") for n, c in (("q", k), ("k", k), ("v", v))]
+            specs += [(t + "A_log", (h,), "rate"), (t + "a2", (h * r["dim"], ranks[0]), "w"), (t + "dt_bias", (h * r["dim"],), "embed"), (t + "g2", (v, ranks[1]), "w"), (t + "norm", (r["vdim"],), "one"), (t + "o", (W, v), "w"), (t + "out", (W,), "one")]
+        else:
+            h, d, r, rot = m["heads"], m["dim"], m["kv_rank"], m["rot_dim"]
+            specs.append((p + "mix.q", (h * (d + rot), W), "w"))
+            if m.get("kv_from") is None:
+                specs += [(p + "mix.dkv", (r + rot, W), "w"), (p + "mix.dkv.norm", (r,), "one")]
+            specs += [(p + "mix.uk", (h * d, r), "w"), (p + "mix.uv", (h * m["vdim"], r), "w"), (p + "mix.g", (h, W), "w"), (p + "mix.o", (W, h * m["vdim"]), "w")]
+        if f is not None:
+            ff = f["ff"]
+            specs += [(p + "norm2", (W,), "one"), (p + "norm2b", (W,), "one"), (p + "mlp.gate", (ff, W), "w"), (p + "mlp.gate.b", (ff,), "zero"), (p + "mlp.up", (ff, W), "w"), (p + "mlp.up.b", (ff,), "zero")]
+            specs += [(p + "mlp.down", (W, ff), "w"), (p + "mlp.down.b", (W,), "zero")]
+    return specs + [("final.norm", (W,), "one"), ("head", (V, W), "w")]
+
+
+def pulenex_tensor(seed: int, spec) -> np.ndarray:
+    """bf16 bits of one tensor: linears N(0, 1/in), biases around 0, mixing matrices around the identity, decay rates from 1/16 to 1, other
+    vectors around 1."""
+    name, shape, kind = spec
+    g = _rng(seed, name)
+    if kind == "tap":
+        return f32_to_bf16_rne(float(shape[1]) ** -0.5 * g.standard_normal(shape, dtype=np.float32))
+    if kind == "mix":
+        return f32_to_bf16_rne((np.eye(shape[0]) + 0.3 * g.standard_normal(shape, dtype=np.float32)).astype(np.float32))
+    if kind == "rate":
+        return f32_to_bf16_rne(np.log(2.0 ** (-4.0 * g.random(shape, dtype=np.float32))).astype(np.float32))
+    return gebilorn_tensor(seed, spec)
+
+
+def pulenex_weights(cfg: dict, seed: int, ranks: Tuple[int, int] = (64, 64)) -> Dict[str, np.ndarray]:
+    """name -> bf16 bits of every tensor."""
+    return {s[0]: pulenex_tensor(seed, s) for s in pulenex_tensor_specs(cfg, ranks)}
+
+
+def write_pulenex_model(model_dir: str, cfg: dict, seed: int, weights: Optional[Dict[str, np.ndarray]] = None, ranks: Tuple[int, int] = (64, 64)) -> str:
+    """config.json + model.safetensors of a Pulenex model (weights: bits to write instead of the seeded ones)."""
+    return _write_model(model_dir, cfg, pulenex_tensor_specs(cfg, ranks), lambda s: pulenex_tensor(seed, s) if weights is None else weights[s[0]])
+
+
 def shard_hf_model(src_dir: str, dst_dir: str, n_shards: int = 2) -> str:
     """Rewrite a single-file checkpoint as `n_shards` safetensors files plus model.safetensors.index.json,
     the layout HfModel::load_with_dtype falls back to (src/hf/model.rs:86-127).  Tensors are dealt out
