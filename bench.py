@@ -285,13 +285,14 @@ def run_c5(hm, synth, rank, world, local, barrier, vmax, K, W, peak):
     return out
 
 
-# Workloads of the listed designs: (stack, uniform stack of equal width, depth, heads and MLP parameters per token), and where each
-# pair is timed: (sequences, prompt tokens)
+# Workloads of the listed designs: (stack, uniform stack of equal width, depth, heads and MLP parameters per token[, stack of a listed
+# design with like mechanisms]), and where they are timed: (sequences, prompt tokens)
 POINTS = {"0.5B": [(1, 128), (8, 1920)], "1.5B": [(1, 128), (64, 512), (8, 1920)]}
 DESIGNS = {
     "tunitar": {"0.5B": ("TUNITAR_05B", "QWEN25_05B"), "1.5B": ("TUNITAR_15B", "QWEN25_15B")},
     "dipisun": {"0.5B": ("DIPISUN_05B", "QWEN25_05B"), "1.5B": ("DIPISUN_15B", "QWEN25_15B")},
     "gebilorn": {"0.5B": ("GEBILORN_05B", "QWEN25_05B"), "1.5B": ("GEBILORN_15B", "QWEN25_15B")},
+    "pulenex": {"0.5B": ("PULENEX_05B", "QWEN25_05B", "GEBILORN_05B"), "1.5B": ("PULENEX_15B", "QWEN25_15B", "GEBILORN_15B")},
 }
 # kernel classes that do the same work in both designs
 LIKE = {
@@ -300,9 +301,13 @@ LIKE = {
     "dipisun": {"qkv_proj": "qkv_rope_kvwrite", "attention": "attention", "o_proj": "o_proj_residual", "experts_gate_up": "gate_up_swiglu", "experts_down": "down_residual", "lm_head": "lm_head"},
     "gebilorn": {"in_proj": "qkv_rope_kvwrite", "attention": "attention", "query_up": "qkv_rope_kvwrite", "key_up": "qkv_rope_kvwrite", "value_up": "o_proj_residual", "out_proj": "o_proj_residual", "experts_gate_up": "gate_up_swiglu",
                  "experts_down": "down_residual", "lm_head": "lm_head"},
+    "pulenex": {"in_proj": "qkv_rope_kvwrite", "attention": "attention", "key_up": "qkv_rope_kvwrite", "value_up": "o_proj_residual", "out_proj": "o_proj_residual", "gate_up": "gate_up_swiglu", "down": "down_residual", "lm_head": "lm_head"},
 }
+# the same against the third stack
+LIKE_LISTED = {"pulenex": ("gebilorn", {"in_proj": "in_proj", "attention": "attention", "key_up": "key_up", "value_up": "value_up", "out_proj": "out_proj", "recurrence": "side", "lm_head": "lm_head"})}
 WHAT = {"tunitar": "Tunitar stacks beside uniform GQA stacks of equal size", "dipisun": "Dipisun stacks beside uniform GQA stacks of equal width, depth, heads and MLP parameters per token",
-        "gebilorn": "Gebilorn stacks beside uniform GQA stacks of equal width, depth, heads and MLP parameters per token"}
+        "gebilorn": "Gebilorn stacks beside uniform GQA stacks of equal width, depth, heads and MLP parameters per token",
+        "pulenex": "Pulenex stacks beside uniform GQA stacks (and Gebilorn stacks) of equal width, depth, heads and MLP parameters per token"}
 
 
 def design_model(design, name, cfg, synth):
@@ -312,6 +317,8 @@ def design_model(design, name, cfg, synth):
         return d
     if design == "tunitar":
         synth.write_tunitar_model(d, cfg, SEED)
+    elif design == "pulenex":
+        synth.write_pulenex_model(d, cfg, SEED)
     elif design in ("dipisun", "gebilorn"):
         # every layer's experts are drawn from one set; corrections of zero leave the choice to the router
         all_specs, tensor, write = (synth.dipisun_tensor_specs, synth.dipisun_tensor, synth.write_dipisun_model) if design == "dipisun" else (synth.gebilorn_tensor_specs, synth.gebilorn_tensor, synth.write_gebilorn_model)
@@ -341,9 +348,10 @@ def run_design(design, args, hm, synth, K, W, peak, peak_kind):
     K = min(K, 48)
     sampler = ClockSampler(0)
     sizes = {}
-    for size, (t_name, u_name) in DESIGNS[design].items():
+    listed, like_listed = LIKE_LISTED.get(design, (None, {}))
+    for size, names in DESIGNS[design].items():
         rows = {}
-        for kind, name in ((design, t_name), ("uniform", u_name)):
+        for kind, name in zip((design, "uniform", listed), names):
             cfg = getattr(synth, name)
             vocab = cfg.vocab_size if kind == "uniform" else cfg["vocab"]
             m = hm.HfModel.load_with_dtype(design_model(kind, name, cfg, synth), hm.DType.BF16)
@@ -368,6 +376,9 @@ def run_design(design, args, hm, synth, K, W, peak, peak_kind):
         for r in rows.values():
             tk, uk = r[design]["kernels"], r["uniform"]["kernels"]
             r["fraction_relative_to_like_kernel"] = {a: round(tk[a]["frac"] / uk[b]["frac"], 3) for a, b in LIKE[design].items() if tk[a]["frac"] and uk[b]["frac"]}
+            if listed:
+                lk = r[listed]["kernels"]
+                r[f"fraction_relative_to_like_kernel_of_{listed}"] = {a: round(tk[a]["frac"] / lk[b]["frac"], 3) for a, b in like_listed.items() if tk[a]["frac"] and lk[b]["frac"]}
         sizes[size] = rows
     head = sizes["1.5B"]["64x512"][design]
     return {

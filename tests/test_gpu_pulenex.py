@@ -15,7 +15,7 @@ pytestmark = pytest.mark.gpu
 
 # relative to the largest reference value: f32 throughout; bf16 pages against an oracle that rounds its keys and values alike (one on
 # the edge of a rounding step may go the other way)
-TOL = {"F32": 3e-5, "BF16": 2e-3}
+TOL = {"F32": 3e-5, "BF16": 4e-3}
 
 
 def bf16_round(x):
