@@ -378,12 +378,12 @@ int Engine::enqueue_latent_attn(int l, int M, bool tall, const int32_t* row_pos,
     a.row_seq = row_seq;
     a.scale = s.scale;
     a.window = s.window;
-    const int longest = s.window > 0 ? (int)std::min((long)pass_longest_, (long)s.window + TC_ROWS + 128) : pass_longest_;  // tokens that the tiles of a row range over
     const size_t per = (size_t)M * s.heads;
     const int most = (int)std::min<size_t>(std::min(lat_acc_floats_ / (per * rank), lat_ml_floats_ / (per * 2)), 256);
     // tiles: every run is cut at the multiples of the rows that share a CTA
     int longest_run = 1, tiles = 0;
     for (auto& r : pass_runs_) longest_run = std::max(longest_run, r.second);
+    const int longest = s.window > 0 ? (int)std::min((long)pass_longest_, (long)s.window + longest_run + 62) : pass_longest_;  // tokens that a tile's pages range over
     a.rows_per_tile = latent_rows_per_tile(longest_run, longest, s.heads, rank, kv_bf16_);
     for (auto& r : pass_runs_) tiles += (r.first + r.second - 1) / a.rows_per_tile - r.first / a.rows_per_tile + 1;
     if (a.rows_per_tile == 1) tiles = M;

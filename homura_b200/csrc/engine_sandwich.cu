@@ -500,6 +500,7 @@ RecurArgs Engine::recur_args(int l, int M, bool tall, const int32_t* row_pos, co
     a.M = M;
     a.runs = pass_runs(M, &a.longest_run);
     a.early = pass_runs_.empty() ? 1 : 0;  // the captured decode step
+    a.err_flag = err_flag_;
     a.out = cat_;
     a.ld_out = cat_ld_;
     const bool second = s.mixer == MIX_PARALLEL;  // inputs of the second output projection

@@ -62,9 +62,16 @@ __device__ __forceinline__ void store_piece(const GqaAttnArgs& a, int m, int hea
     const int vdim = a.pool.vdim, e0 = head * vdim + d0, off = X ? a.out_off : 0, k0 = off + e0, ld = X ? a.ld_out : a.heads * vdim;
     if (X && a.gate_kind != GATE_NONE) {
         const float* g = a.gate + (size_t)m * a.ld_gate;
-        const float all = a.gate_kind == GATE_HEAD ? 1.0f / (1.0f + expf(-ld_cg_f32(g + head))) : 1.f;
+        if (a.gate_kind == GATE_ELEM && d0 + 8 <= vdim && (reinterpret_cast<uintptr_t>(g + e0) & 15) == 0) {
+            const float4 x = ld_cg_f32x4(g + e0), y = ld_cg_f32x4(g + e0 + 4);
+            const float z[8] = {x.x, x.y, x.z, x.w, y.x, y.y, y.z, y.w};
 #pragma unroll
-        for (int i = 0; i < 8; ++i) v[i] *= a.gate_kind == GATE_HEAD ? all : d0 + i < vdim ? 1.0f / (1.0f + expf(-ld_cg_f32(g + e0 + i))) : 0.f;
+            for (int i = 0; i < 8; ++i) v[i] *= 1.0f / (1.0f + expf(-z[i]));
+        } else {
+            const float all = a.gate_kind == GATE_HEAD ? 1.0f / (1.0f + expf(-ld_cg_f32(g + head))) : 1.f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] *= a.gate_kind == GATE_HEAD ? all : d0 + i < vdim ? 1.0f / (1.0f + expf(-ld_cg_f32(g + e0 + i))) : 0.f;
+        }
     }
     if (X && a.out_scale != 0.f)
 #pragma unroll

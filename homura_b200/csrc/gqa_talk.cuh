@@ -18,7 +18,7 @@ struct TalkGeom {
     int stages;
     uint32_t block; // bytes of a ring stage
     size_t front;   // bytes of the ring, which takes the results afterwards
-    size_t q, raw, p, corr, o, ml, talk, wts, pages, smem;  // offsets from the front's end, total
+    size_t q, raw, p, corr, o, ml, talk, wts, pages, qi, pair, smem;  // offsets from the front's end, total
 };
 
 inline bool talk_geom(const GqaAttnArgs& a, int rows, int nsplit, int pages_per_cta, TalkGeom* g) {
@@ -44,6 +44,8 @@ inline bool talk_geom(const GqaAttnArgs& a, int rows, int nsplit, int pages_per_
     g->talk = take((size_t)H * ((H + 3) / 4 * 4) * 4);
     g->wts = take(pairs * nsplit * 4);
     g->pages = take((size_t)pages_per_cta * 4);
+    g->qi = take(pairs * 2);
+    g->pair = take((size_t)g->per * 2);
     const size_t result = pairs * (vp + 4) * 4, most = 226 * 1024;
     if (at + std::max(result, 2 * (size_t)g->block) + 128 > most) return false;
     g->stages = (int)std::min<size_t>({(most - at - 128) / g->block, (size_t)TALK_MAX_STAGES, (size_t)2 * G * std::max(1, pages_per_cta)});
@@ -52,7 +54,86 @@ inline bool talk_geom(const GqaAttnArgs& a, int rows, int nsplit, int pages_per_
     return g->smem <= most;
 }
 
-__global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const GqaAttnArgs a, const TalkGeom geo) {
+// Scores of KH heads of a row out of all heads' (x: this lane's two tokens of the row's first head), mask, running softmax, weights.
+template <int KH>
+__device__ __forceinline__ void talk_mix(const GqaAttnArgs& a, int r, int h0, int pos, int from, int ta, const float* x, const float* tk, int HP, const uint16_t* qi, uint16_t* ps, int padded, float* ml, float* corr) {
+    const int H = a.heads, lane = threadIdx.x & 31;
+    float2 s[KH];
+    float old[KH];
+#pragma unroll
+    for (int k = 0; k < KH; ++k) {
+        s[k] = make_float2(0.f, 0.f);
+        old[k] = h0 + k < H ? ml[2 * (r * H + h0 + k)] : 0.f;
+    }
+#pragma unroll 4
+    for (int e = 0; e < H; ++e) {
+        const float2 v = *reinterpret_cast<const float2*>(x + e * TALK_RAW_LD);
+        float t[KH];
+        if constexpr (KH == 4) {
+            const float4 w = *reinterpret_cast<const float4*>(tk + e * HP + h0);
+            t[0] = w.x; t[1] = w.y; t[2] = w.z; t[3] = w.w;
+        } else if constexpr (KH == 2) {
+            const float2 w = *reinterpret_cast<const float2*>(tk + e * HP + h0);
+            t[0] = w.x; t[1] = w.y;
+        } else {
+            t[0] = tk[e * HP + h0];
+        }
+#pragma unroll
+        for (int k = 0; k < KH; ++k) {
+            s[k].x = fmaf(t[k], v.x, s[k].x);
+            s[k].y = fmaf(t[k], v.y, s[k].y);
+        }
+    }
+    const bool va = ta <= pos && (ta >= from || ta < a.keep_first), vb = ta + 1 <= pos && (ta + 1 >= from || ta + 1 < a.keep_first);
+    float mx[KH], sum[KH], f[KH];
+#pragma unroll
+    for (int k = 0; k < KH; ++k) {
+        s[k].x = va ? s[k].x : -INFINITY;
+        s[k].y = vb ? s[k].y : -INFINITY;
+        mx[k] = fmaxf(s[k].x, s[k].y);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int k = 0; k < KH; ++k) mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], o));
+#pragma unroll
+    for (int k = 0; k < KH; ++k) {
+        mx[k] = fmaxf(old[k], mx[k]);
+        const float ref = mx[k] == -INFINITY ? 0.f : mx[k];  // no token of this pair yet
+        f[k] = exp2f(old[k] - ref);
+        s[k].x = exp2f(s[k].x - ref);
+        s[k].y = exp2f(s[k].y - ref);
+        sum[k] = s[k].x + s[k].y;
+        if (h0 + k < H) {
+            uint32_t t[3];
+            bf16x2_split3(s[k].x, s[k].y, t[0], t[1], t[2]);
+            uint16_t* dst = ps + (size_t)qi[r * H + h0 + k] * TALK_P_LD + 2 * lane;
+#pragma unroll
+            for (int e = 0; e < 3; ++e) *reinterpret_cast<uint32_t*>(dst + (size_t)e * padded * TALK_P_LD) = t[e];
+        }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int k = 0; k < KH; ++k) sum[k] += __shfl_xor_sync(0xffffffffu, sum[k], o);
+    if (lane < KH && h0 + lane < H) {
+        float m = mx[0], c = f[0], l = sum[0];
+#pragma unroll
+        for (int k = 1; k < KH; ++k)
+            if (lane == k) {
+                m = mx[k];
+                c = f[k];
+                l = sum[k];
+            }
+        float* d = ml + 2 * (r * H + h0 + lane);
+        d[0] = m;
+        d[1] = fmaf(d[1], c, l);
+        corr[qi[r * H + h0 + lane]] = c;
+    }
+    __syncwarp();
+}
+
+__global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const __grid_constant__ GqaAttnArgs a, const __grid_constant__ TalkGeom geo) {
     extern __shared__ __align__(128) unsigned char dyn[];
     const int H = a.heads, G = a.pool.kv_heads, gq = H / G, dim = a.pool.dim, vdim = a.pool.vdim, dp = gqa_pad(dim), vp = gqa_pad(vdim), kt_n = dp / 16, vt_n = vp / 16, ldo = vp + 4;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, split = blockIdx.x, NST = geo.stages, HP = (H + 3) & ~3;
@@ -67,6 +148,8 @@ __global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const GqaAt
     float* tk = reinterpret_cast<float*>(back + geo.talk);           // [head that is read][head, padded]
     float* wts = reinterpret_cast<float*>(back + geo.wts);
     int32_t* pt_s = reinterpret_cast<int32_t*>(back + geo.pages);
+    uint16_t* qi = reinterpret_cast<uint16_t*>(back + geo.qi);       // [row][head] -> pair by key head
+    uint16_t* pair = reinterpret_cast<uint16_t*>(back + geo.pair);   // pair of the first key head -> [row][head]
     __shared__ uint64_t full[TALK_MAX_STAGES], empty[TALK_MAX_STAGES];
     __shared__ volatile int s_abort;
 
@@ -78,14 +161,12 @@ __global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const GqaAt
         rows = min(geo.rows, a.runs.row[r + 1] - row0);
     }
     const int pairs = rows * H;
-    if (tid == 0) {
-        for (int s = 0; s < NST; ++s) {
-            mb_init(&full[s], 1);
-            mb_init(&empty[s], ATT_WARPS);
-        }
-        s_abort = 0;
+    if (tid < NST) {
+        mb_init(&full[tid], 1);
+        mb_init(&empty[tid], ATT_WARPS);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
+    if (tid == 0) s_abort = 0;
     pdl_launch_dependents();
     // positions, pages and the mixing matrix do not depend on the launch in front
     const int seq = a.row_seq[row0], pos0 = a.row_pos[row0], len = pos0 + rows;
@@ -93,11 +174,12 @@ __global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const GqaAt
     const int pps = (list.n + a.nsplit - 1) / a.nsplit, p0 = split * pps, np = max(0, min(list.n, p0 + pps) - p0);
     const int32_t* pt = a.pool.page_table + (size_t)seq * a.pool.max_pages;
     for (int i = tid; i < np; i += B_THREADS) pt_s[i] = pt[list.page(p0 + i)];
-    for (int i = tid; i < H * HP; i += B_THREADS) {
-        const int e = i / HP, h = i - e * HP;
-        tk[i] = h < H ? __ldg(a.talk + (size_t)h * H + e) : 0.f;
-    }
+    for (int e = warp; e < H; e += B_THREADS / 32)
+        for (int h = lane; h < HP; h += 32) tk[e * HP + h] = h < H ? __ldg(a.talk + (size_t)h * H + e) : 0.f;
     for (int i = tid; i < pairs; i += B_THREADS) {
+        const int r = i / H, h = i - r * H, g = h / gq, q = r * gq + h - g * gq;
+        qi[i] = (uint16_t)(g * geo.per + q);
+        if (g == 0) pair[q] = (uint16_t)i;
         ml[2 * i] = -INFINITY;
         ml[2 * i + 1] = 0.f;
     }
@@ -106,60 +188,97 @@ __global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const GqaAt
     __syncthreads();
     const unsigned char *kpool = reinterpret_cast<const unsigned char*>(a.pool.k), *vpool = reinterpret_cast<const unsigned char*>(a.pool.v);
     const uint32_t k_bytes = (uint32_t)(GQA_PAGE * dp * 2), v_bytes = (uint32_t)(GQA_PAGE * vp * 2);
-    const int items = np * 2 * G;
     if (warp == ATT_WARPS) {
         if (lane == 0) {
-            int i = 0;
-            auto fetch = [&](int it) {
-                const int pg = it / (2 * G), b = it - pg * 2 * G, s = it % NST;
-                const bool is_v = b >= G;
-                const size_t tile = (size_t)pt_s[pg] * G + (is_v ? b - G : b);
-                mb_expect_tx(&full[s], is_v ? v_bytes : k_bytes);
-                bulk_copy(ring + (size_t)s * geo.block, is_v ? vpool + tile * v_bytes : kpool + tile * k_bytes, is_v ? v_bytes : k_bytes, &full[s]);
-            };
-            if (a.early)  // the captured decode step: pages in front of the newest token's are complete
-                for (; i < items && i < NST && list.page(p0 + i / (2 * G)) < (len - 1) / GQA_PAGE; ++i) fetch(i);
-            pdl_wait();
-            for (; i < items; ++i) {
-                if (i >= NST && !mb_wait(&empty[i % NST], ((i / NST) & 1u) ^ 1u, a.err_flag, &s_abort)) break;
-                fetch(i);
+            // blocks in order: a page's keys of every key head, then its values
+            int s = 0, filled = 0;
+            uint32_t phase = 1;  // of the stage's empty barrier; its first round needs no wait
+            bool ok = true, waited = false;
+            for (int i = 0; i < np && ok; ++i) {
+                const size_t tile = (size_t)pt_s[i] * G;
+                const bool settled = a.early && list.page(p0 + i) < (len - 1) / GQA_PAGE;  // complete before the launch in front began
+                for (int b = 0; b < 2 * G; ++b) {
+                    if (!waited && (!settled || filled == NST)) {
+                        pdl_wait();
+                        waited = true;
+                    }
+                    if (filled == NST && !mb_wait(&empty[s], phase, a.err_flag, &s_abort)) {
+                        ok = false;
+                        break;
+                    }
+                    const bool is_v = b >= G;
+                    mb_expect_tx(&full[s], is_v ? v_bytes : k_bytes);
+                    bulk_copy(ring + (size_t)s * geo.block, is_v ? vpool + (tile + b - G) * v_bytes : kpool + (tile + b) * k_bytes, is_v ? v_bytes : k_bytes, &full[s]);
+                    if (filled < NST) ++filled;
+                    if (++s == NST) {
+                        s = 0;
+                        phase ^= 1;
+                    }
+                }
             }
+            if (!waited) pdl_wait();
         } else {
             pdl_wait();
         }
     } else {
         pdl_wait();
-        // queries: three bf16 terms, two elements a thread
-        const int d2 = dp / 2;
-#pragma unroll 4
-        for (int i = tid; i < pairs * d2; i += ATT_WARPS * 32) {
-            const int p = i / d2, d = (i - p * d2) * 2, r = p / H, h = p - r * H, qi = (h / gq) * geo.per + r * gq + h % gq;
-            const float* q = a.q + (size_t)(row0 + r) * H * dim + (size_t)h * dim + d;
-            const float x = d < dim ? ld_cg_f32(q) : 0.f, y = d + 1 < dim ? ld_cg_f32(q + 1) : 0.f;
-            uint32_t t[3];
-            bf16x2_split3(x, y, t[0], t[1], t[2]);
+        // queries: three bf16 terms, a warp per (row, head)
+#pragma unroll 2
+        for (int p = warp; p < pairs; p += ATT_WARPS) {
+            const float* q = a.q + (size_t)row0 * H * dim + (size_t)p * dim;
+            uint16_t* dst = qs + (size_t)qi[p] * ldq;
+#pragma unroll 2
+            for (int d = 2 * lane; d < dp; d += 64) {
+                float x = 0.f, y = 0.f;
+                if ((dim & 1) == 0) {
+                    if (d < dim) {
+                        const float2 v = __ldcg(reinterpret_cast<const float2*>(q + d));
+                        x = v.x;
+                        y = v.y;
+                    }
+                } else {
+                    x = d < dim ? __ldcg(q + d) : 0.f;
+                    y = d + 1 < dim ? __ldcg(q + d + 1) : 0.f;
+                }
+                uint32_t t[3];
+                bf16x2_split3(x, y, t[0], t[1], t[2]);
 #pragma unroll
-            for (int k = 0; k < 3; ++k) *reinterpret_cast<uint32_t*>(qs + (size_t)(k * padded + qi) * ldq + d) = t[k];
+                for (int k = 0; k < 3; ++k) *reinterpret_cast<uint32_t*>(dst + (size_t)k * padded * ldq + d) = t[k];
+            }
         }
         asm volatile("bar.sync 1, 256;" ::: "memory");
-        const int gid = lane >> 2, tig = lane & 3, mj = lane >> 3, mr = lane & 7;
+        const int gid = lane >> 2, tig = lane & 3, mj = lane >> 3, mr = lane & 7, valid = rows * gq;
+        const uint32_t k_lane = (uint32_t)(((mj >> 1) * GQA_PAGE + (mj & 1) * 8 + mr) * 16), v_lane = (uint32_t)(((mj & 1) * GQA_PAGE + (mj >> 1) * 8 + mr) * 16);
+        const int kh = pairs > 16 ? 4 : pairs > 8 ? 2 : 1, hu = (H + kh - 1) / kh;  // heads of a unit of the mixing: few enough that every warp has one
+        const uint16_t *q_lane = qs + (size_t)gid * ldq + 2 * tig, *p_lane = ps + (size_t)gid * TALK_P_LD + 2 * tig;
+        const bool kept = tig < geo.cols2;
+        int s = 0;
+        uint32_t phase = 0;
+        auto next = [&]() {
+            __syncwarp();
+            if (lane == 0) mb_arrive(&empty[s]);
+            if (++s == NST) {
+                s = 0;
+                phase ^= 1;
+            }
+        };
         for (int i = 0; i < np; ++i) {
             const int tok0 = list.page(p0 + i) * GQA_PAGE;
             // scores.  A wait that gives up leaves the work out; the barriers below are still met by every warp.
             for (int g = 0; g < G; ++g) {
-                const int it = i * 2 * G + g, s = it % NST;
-                const bool ok = __all_sync(0xffffffffu, mb_wait(&full[s], (it / NST) & 1u, a.err_flag, &s_abort));
-                const uint32_t kb = s32(ring + (size_t)s * geo.block) + (uint32_t)(((mj >> 1) * GQA_PAGE + (mj & 1) * 8 + mr) * 16);
+                const bool ok = __all_sync(0xffffffffu, mb_wait(&full[s], phase, a.err_flag, &s_abort));
+                const uint32_t kb = s32(ring + (size_t)s * geo.block) + k_lane;
                 for (int j = (warp - g * 4 * geo.ntile) & 7; ok && j < 4 * geo.ntile; j += 8) {
                     const int u = j & 3, nt = j >> 2;
                     float sc[3][4];
 #pragma unroll
                     for (int k = 0; k < 3; ++k) sc[k][0] = sc[k][1] = sc[k][2] = sc[k][3] = 0.f;
-                    const uint16_t* q = qs + (size_t)(g * geo.per + nt * 8 + gid) * ldq + 2 * tig;
+                    const uint16_t* q = q_lane + (size_t)(g * geo.per + nt * 8) * ldq;
+                    const uint32_t ku = kb + (uint32_t)(u * 256);
 #pragma unroll 4
                     for (int kt = 0; kt < kt_n; ++kt) {
                         uint32_t ka[4];
-                        ldsm4(ka, kb + (uint32_t)(u * 256 + kt * (2 * GQA_PAGE * 16)));
+                        ldsm4(ka, ku + (uint32_t)(kt * (2 * GQA_PAGE * 16)));
 #pragma unroll
                         for (int k = 0; k < 3; ++k) {
                             const uint16_t* b = q + (size_t)k * padded * ldq + kt * 16;
@@ -169,93 +288,35 @@ __global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const GqaAt
 #pragma unroll
                     for (int hh = 0; hh < 2; ++hh) {
                         const int c = nt * 8 + 2 * tig + hh;
-                        if (c < rows * gq) {
-                            float* dst = raw + (size_t)((c / gq) * H + g * gq + c % gq) * TALK_RAW_LD + u * 16 + gid;
+                        if (c < valid) {
+                            float* dst = raw + (size_t)(pair[c] + g * gq) * TALK_RAW_LD + u * 16 + gid;
                             dst[0] = (sc[2][hh] + sc[1][hh]) + sc[0][hh];
                             dst[8] = (sc[2][2 + hh] + sc[1][2 + hh]) + sc[0][2 + hh];
                         }
                     }
                 }
-                __syncwarp();
-                if (lane == 0) mb_arrive(&empty[s]);
+                next();
             }
             asm volatile("bar.sync 1, 256;" ::: "memory");
-            // four heads of a row at a time: their scores out of all heads', two tokens a lane
-            for (int w = warp; w < rows * (HP / 4); w += ATT_WARPS) {
-                const int r = w / (HP / 4), h0 = (w - r * (HP / 4)) * 4, pos = pos0 + r, from = first_visible(a, pos), ta = tok0 + 2 * lane;
-                float2 s[4];
-#pragma unroll
-                for (int k = 0; k < 4; ++k) s[k] = make_float2(0.f, 0.f);
+            for (int w = warp; w < rows * hu; w += ATT_WARPS) {
+                const int r = rows == 1 ? 0 : w / hu, h0 = (w - r * hu) * kh, pos = pos0 + r, from = first_visible(a, pos), ta = tok0 + 2 * lane;
                 const float* x = raw + (size_t)r * H * TALK_RAW_LD + 2 * lane;
-#pragma unroll 4
-                for (int e = 0; e < H; ++e) {
-                    const float2 v = *reinterpret_cast<const float2*>(x + (size_t)e * TALK_RAW_LD);
-                    const float4 t = *reinterpret_cast<const float4*>(tk + e * HP + h0);
-                    s[0].x = fmaf(t.x, v.x, s[0].x); s[0].y = fmaf(t.x, v.y, s[0].y);
-                    s[1].x = fmaf(t.y, v.x, s[1].x); s[1].y = fmaf(t.y, v.y, s[1].y);
-                    s[2].x = fmaf(t.z, v.x, s[2].x); s[2].y = fmaf(t.z, v.y, s[2].y);
-                    s[3].x = fmaf(t.w, v.x, s[3].x); s[3].y = fmaf(t.w, v.y, s[3].y);
-                }
-                const bool va = ta <= pos && (ta >= from || ta < a.keep_first), vb = ta + 1 <= pos && (ta + 1 >= from || ta + 1 < a.keep_first);
-                float mx[4], sum[4], f[4];
-#pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    s[k].x = va ? s[k].x : -INFINITY;
-                    s[k].y = vb ? s[k].y : -INFINITY;
-                    mx[k] = fmaxf(s[k].x, s[k].y);
-                }
-#pragma unroll
-                for (int o = 16; o > 0; o >>= 1)
-#pragma unroll
-                    for (int k = 0; k < 4; ++k) mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], o));
-#pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    const int h = h0 + k;
-                    if (h >= H) break;
-                    const float old = ml[2 * (r * H + h)];
-                    mx[k] = fmaxf(old, mx[k]);
-                    const float ref = mx[k] == -INFINITY ? 0.f : mx[k];  // no token of this pair yet
-                    f[k] = exp2f(old - ref);
-                    s[k].x = exp2f(s[k].x - ref);
-                    s[k].y = exp2f(s[k].y - ref);
-                    uint32_t t[3];
-                    bf16x2_split3(s[k].x, s[k].y, t[0], t[1], t[2]);
-                    const int qi = (h / gq) * geo.per + r * gq + h % gq;
-#pragma unroll
-                    for (int e = 0; e < 3; ++e) *reinterpret_cast<uint32_t*>(ps + (size_t)(e * padded + qi) * TALK_P_LD + 2 * lane) = t[e];
-                }
-#pragma unroll
-                for (int k = 0; k < 4; ++k) sum[k] = s[k].x + s[k].y;
-#pragma unroll
-                for (int o = 16; o > 0; o >>= 1)
-#pragma unroll
-                    for (int k = 0; k < 4; ++k) sum[k] += __shfl_xor_sync(0xffffffffu, sum[k], o);
-                __syncwarp();
-                if (lane == 0)
-#pragma unroll
-                    for (int k = 0; k < 4; ++k) {
-                        const int h = h0 + k;
-                        if (h >= H) break;
-                        float* m = ml + 2 * (r * H + h);
-                        m[0] = mx[k];
-                        m[1] = fmaf(m[1], f[k], sum[k]);
-                        corr[(h / gq) * geo.per + r * gq + h % gq] = f[k];
-                    }
-                __syncwarp();
+                if (kh == 4) talk_mix<4>(a, r, h0, pos, from, ta, x, tk, HP, qi, ps, padded, ml, corr);
+                else if (kh == 2) talk_mix<2>(a, r, h0, pos, from, ta, x, tk, HP, qi, ps, padded, ml, corr);
+                else talk_mix<1>(a, r, h0, pos, from, ta, x, tk, HP, qi, ps, padded, ml, corr);
             }
             asm volatile("bar.sync 1, 256;" ::: "memory");
             for (int g = 0; g < G; ++g) {
-                const int it = i * 2 * G + G + g, s = it % NST, units = vt_n * geo.ntile;
-                const bool ok = __all_sync(0xffffffffu, mb_wait(&full[s], (it / NST) & 1u, a.err_flag, &s_abort));
-                const uint32_t vb = s32(ring + (size_t)s * geo.block) + (uint32_t)(((mj & 1) * GQA_PAGE + (mj >> 1) * 8 + mr) * 16);
+                const bool ok = __all_sync(0xffffffffu, mb_wait(&full[s], phase, a.err_flag, &s_abort));
+                const uint32_t vb = s32(ring + (size_t)s * geo.block) + v_lane;
+                const int units = vt_n * geo.ntile;
                 for (int j = (warp - g * units) & 7; ok && j < units; j += 8) {
-                    const int nt = j / vt_n, mt = j - nt * vt_n, qi = g * geo.per + nt * 8;
-                    const bool kept = tig < geo.cols2;
+                    const int nt = geo.ntile == 1 ? 0 : j / vt_n, mt = j - nt * vt_n, q0 = g * geo.per + nt * 8;
                     float4* o = os + (size_t)((g * vt_n + mt) * geo.ntile + nt) * o_tile + tig * 8 + gid;
-                    float4 c = kept ? *o : make_float4(0.f, 0.f, 0.f, 0.f);
-                    const float c0 = corr[qi + 2 * tig], c1 = corr[qi + 2 * tig + 1];
+                    const float4 c = kept ? *o : make_float4(0.f, 0.f, 0.f, 0.f);
+                    const float c0 = corr[q0 + 2 * tig], c1 = corr[q0 + 2 * tig + 1];
                     float acc[3][4] = {{c.x * c0, c.y * c1, c.z * c0, c.w * c1}, {0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-                    const uint16_t* p = ps + (size_t)(qi + gid) * TALK_P_LD + 2 * tig;
+                    const uint16_t* p = p_lane + (size_t)q0 * TALK_P_LD;
 #pragma unroll
                     for (int kt = 0; kt < 4; ++kt) {
                         uint32_t va[4];
@@ -268,26 +329,35 @@ __global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const GqaAt
                     }
                     if (kept) *o = make_float4((acc[2][0] + acc[1][0]) + acc[0][0], (acc[2][1] + acc[1][1]) + acc[0][1], (acc[2][2] + acc[1][2]) + acc[0][2], (acc[2][3] + acc[1][3]) + acc[0][3]);
                 }
-                __syncwarp();
-                if (lane == 0) mb_arrive(&empty[s]);
+                next();
             }
         }
     }
     __syncthreads();  // every block consumed: the ring takes the results
     float* res = reinterpret_cast<float*>(ring);  // [row][head][ldo]
-    for (int i = tid; i < o_n; i += B_THREADS) {
-        const int u = i / o_tile, e = i - u * o_tile, tig = e >> 3, gid = e & 7, nt = u % geo.ntile, gm = u / geo.ntile, g = gm / vt_n, mt = gm - g * vt_n;
-        const float4 v = os[i];
-        const float x[4] = {v.x, v.y, v.z, v.w};
+    {
+        const int gid = lane & 7, tig = lane >> 3;
+        for (int gm = warp; gm < G * vt_n; gm += B_THREADS / 32) {
+            const int g = gm / vt_n, mt = gm - g * vt_n;
+            for (int nt = 0; nt < geo.ntile; ++nt) {
+                if (tig >= geo.cols2) continue;
+                const float4 v = os[(size_t)(gm * geo.ntile + nt) * o_tile + lane];
+                const float x[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-            const int c = nt * 8 + 2 * tig + (k & 1);
-            if (c < rows * gq) res[(size_t)((c / gq) * H + g * gq + c % gq) * ldo + mt * 16 + gid + (k >> 1) * 8] = x[k];
+                for (int k = 0; k < 2; ++k) {
+                    const int c = nt * 8 + 2 * tig + k;
+                    if (c >= rows * gq) continue;
+                    float* d = res + (size_t)(pair[c] + g * gq) * ldo + mt * 16 + gid;
+                    d[0] = x[k];
+                    d[8] = x[2 + k];
+                }
+            }
         }
     }
     combine_and_store<true>(a, res, ldo, ml, wts, pairs, [&](int p, int& row, int& head) {
-        row = row0 + p / H;
-        head = p % H;
+        const int r = rows == 1 ? 0 : p / H;
+        row = row0 + r;
+        head = p - r * H;
     });
 }
 

@@ -2,6 +2,7 @@
 #include "recur.h"
 
 #include "launch_attrs.h"
+#include "mbarrier.cuh"
 
 namespace hm {
 namespace {
@@ -239,9 +240,177 @@ __global__ void __launch_bounds__(GLA_THREADS, RD > 32 ? 1 : 2) recur_kernel(con
     if (slices > 1) finish(0, n);
 }
 
-template <int RD, int KIND>
-cudaError_t launch(const RecurArgs& a, unsigned blocks, size_t smem, cudaStream_t st, bool pdl) {
-    const cudaError_t e = ensure_dyn_smem(recur_kernel<RD, KIND>, smem);
+// ---- single tokens ---------------------------------------------------------------------------------
+// A CTA per (sequence, head).  The state arrives in shared memory by bulk copies, in the captured decode step ahead of the dependency
+// wait; a warp takes whole columns, lanes along the key dimension, and stores them from registers as their piece has landed.
+struct RecurTokenSmem {
+    int state, v, gate, o, total;
+};
+__host__ __device__ __forceinline__ RecurTokenSmem recur_token_smem(const RecurArgs& a) {
+    const int vp = (a.vdim + 3) & ~3, st = (int)gla_state_floats(a.dim, a.vdim);
+    return RecurTokenSmem{0, st, st + vp, st + 2 * vp, st + 3 * vp};
+}
+
+template <int KIND>
+__global__ void __launch_bounds__(GLA_THREADS, 3) recur_token_kernel(const __grid_constant__ RecurArgs a) {
+    constexpr int NJ = GLA_TOKEN_DIM / 128, W = GLA_THREADS / 32;  // 16-byte pieces of a column per lane; warps
+    constexpr uint32_t CHUNK = 16384;
+    extern __shared__ __align__(16) float sm[];
+    __shared__ uint64_t landed[(GLA_TOKEN_BYTES + CHUNK - 1) / CHUNK];  // a barrier per piece of the copy
+    __shared__ volatile int s_abort;
+    __shared__ float part[W];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int head = blockIdx.x % a.heads, m = blockIdx.x / a.heads, kvh = head / (a.heads / a.kv_heads), dim = a.dim, vdim = a.vdim, ldd = gla_pad(dim), ld4 = ldd / 4;
+    const RecurTokenSmem lay = recur_token_smem(a);
+    float *vs = sm + lay.v, *gs = sm + lay.gate, *os = sm + lay.o;
+    const uint32_t bytes = (uint32_t)(vdim * ldd * 4);
+    if (tid == 0) {
+        for (uint32_t i = 0; i * CHUNK < bytes; ++i) mb_init(&landed[i], 1);
+        s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    pdl_launch_dependents();
+    const int seq = a.row_seq[m], pos = a.row_pos[m];
+    float* const state = a.state + (size_t)seq * a.seq_stride + (size_t)head * vdim * ldd;
+    auto fetch = [&]() {
+        for (uint32_t i = 0, o = 0; o < bytes; ++i, o += CHUNK) {
+            mb_expect_tx(&landed[i], min(CHUNK, bytes - o));
+            bulk_copy(reinterpret_cast<char*>(sm + lay.state) + o, reinterpret_cast<const char*>(state) + o, min(CHUNK, bytes - o), &landed[i]);
+        }
+    };
+    if (tid == 0 && a.early && pos > 0) fetch();
+    const float decay = KIND == LIN_RETENTION ? __ldg(a.decay + head) : 0.f, norm0 = a.norm_w && tid < vdim ? __ldg(a.norm_w + tid) : 1.f;
+    // lanes of a column: a power of two, so that several short columns share a warp
+    const int LC = ld4 >= 32 ? 32 : 1 << (32 - __clz(ld4 - 1)), sub = lane / LC, piece = lane - sub * LC, CW = 32 / LC;
+    pdl_wait();
+    if (tid == 0 && !a.early && pos > 0) fetch();
+    // everything of the row is requested before the first use
+    const float v0 = tid < vdim ? ld_cg_f32(a.v + (size_t)m * a.ldv + (size_t)head * vdim + tid) : 0.f, g0 = tid < vdim ? ld_cg_f32(a.gate + (size_t)m * a.ld_gate + (size_t)head * vdim + tid) : 0.f;
+    const float b0 = KIND == LIN_DELTA ? ld_cg_f32(a.beta + (size_t)m * a.ld_beta + head) : 0.f;
+    const float *qr = a.q + (size_t)m * a.ldq + (size_t)kvh * a.head_ld, *kr = a.k + (size_t)m * a.ldk + (size_t)kvh * a.head_ld, *ar = KIND == LIN_DELTA ? a.alpha + ((size_t)m * a.heads + head) * dim : nullptr;
+    auto load4 = [&](const float* row, int d) {
+        if ((reinterpret_cast<uintptr_t>(row) & 15) == 0 && d + 4 <= dim) return ld_cg_f32x4(row + d);
+        return make_float4(ld_cg_f32(row + d), d + 1 < dim ? ld_cg_f32(row + d + 1) : 0.f, d + 2 < dim ? ld_cg_f32(row + d + 2) : 0.f, d + 3 < dim ? ld_cg_f32(row + d + 3) : 0.f);
+    };
+    float4 q[NJ], k[NJ], al[NJ];
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        q[j] = k[j] = al[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        const int d = (j * 32 + piece) * 4;
+        if (d >= dim) continue;
+        q[j] = load4(qr, d);
+        k[j] = load4(kr, d);
+        if (KIND == LIN_DELTA) al[j] = load4(ar, d);
+    }
+    if (tid < vdim) {
+        vs[tid] = v0;
+        gs[tid] = g0;
+    }
+    for (int i = GLA_THREADS + tid; i < vdim; i += GLA_THREADS) {
+        vs[i] = ld_cg_f32(a.v + (size_t)m * a.ldv + (size_t)head * vdim + i);
+        gs[i] = ld_cg_f32(a.gate + (size_t)m * a.ld_gate + (size_t)head * vdim + i);
+    }
+    float kq = 0.f;  // what the token's own write adds to its result
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        q[j] = make_float4(q[j].x * a.q_scale, q[j].y * a.q_scale, q[j].z * a.q_scale, q[j].w * a.q_scale);
+        if (KIND == LIN_DELTA) kq += fmaf(q[j].x, k[j].x, q[j].y * k[j].y) + fmaf(q[j].z, k[j].z, q[j].w * k[j].w);
+    }
+    if (KIND == LIN_DELTA)
+        for (int s = 1; s < LC; s <<= 1) kq += __shfl_xor_sync(0xffffffffu, kq, s);
+    const float beta = KIND == LIN_DELTA ? sigmoid(b0) : 0.f;
+    __syncthreads();
+    bool ok = true;
+    uint32_t seen = 0;  // pieces that have landed
+    const float4* tile = reinterpret_cast<const float4*>(sm + lay.state);
+    constexpr int U = KIND == LIN_DELTA ? 2 : 4;  // columns whose sums go side by side
+    for (int g = warp * U; g * CW < vdim; g += W * U) {
+        if (pos > 0)  // every piece is waited for, so that none is on its way when the CTA ends; the waits are bounded
+            for (const uint32_t last = min(bytes, (uint32_t)((g + U) * CW * ldd * 4)); seen * CHUNK < last; ++seen) ok = mb_wait(&landed[seen], 0, a.err_flag, &s_abort) && ok;
+        float4 S[U][NJ];
+        float o[U], sk[U], v[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int c = (g + u) * CW + sub;
+            o[u] = sk[u] = 0.f;
+            v[u] = c < vdim ? vs[c] : 0.f;
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) {
+                const int p = j * 32 + piece;
+                S[u][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (c >= vdim || p >= ld4) continue;
+                if (pos > 0 && ok) S[u][j] = tile[c * ld4 + p];
+                float4& t = S[u][j];
+                if (KIND == LIN_DELTA) {
+                    t = make_float4(t.x * al[j].x, t.y * al[j].y, t.z * al[j].z, t.w * al[j].w);
+                    sk[u] += fmaf(t.x, k[j].x, t.y * k[j].y) + fmaf(t.z, k[j].z, t.w * k[j].w);
+                } else {
+                    t = make_float4(fmaf(t.x, decay, k[j].x * v[u]), fmaf(t.y, decay, k[j].y * v[u]), fmaf(t.z, decay, k[j].z * v[u]), fmaf(t.w, decay, k[j].w * v[u]));
+                    __stcg(reinterpret_cast<float4*>(state) + (size_t)c * ld4 + p, t);
+                }
+                o[u] += fmaf(t.x, q[j].x, t.y * q[j].y) + fmaf(t.z, q[j].z, t.w * q[j].w);
+            }
+        }
+        for (int s = 1; s < LC; s <<= 1)
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                o[u] += __shfl_xor_sync(0xffffffffu, o[u], s);
+                if (KIND == LIN_DELTA) sk[u] += __shfl_xor_sync(0xffffffffu, sk[u], s);
+            }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int c = (g + u) * CW + sub;
+            if (c >= vdim) continue;
+            if (KIND == LIN_DELTA) {
+                const float w = beta * (v[u] - sk[u]);
+#pragma unroll
+                for (int j = 0; j < NJ; ++j) {
+                    const int p = j * 32 + piece;
+                    if (p >= ld4) continue;
+                    const float4 t = S[u][j];
+                    __stcg(reinterpret_cast<float4*>(state) + (size_t)c * ld4 + p, make_float4(fmaf(k[j].x, w, t.x), fmaf(k[j].y, w, t.y), fmaf(k[j].z, w, t.z), fmaf(k[j].w, w, t.w)));
+                }
+                o[u] = fmaf(kq, w, o[u]);
+            }
+            if (piece == 0) os[c] = o[u];
+        }
+    }
+    if (pos > 0)  // (a warp whose columns end before the last piece)
+        for (; seen * CHUNK < bytes; ++seen) mb_wait(&landed[seen], 0, a.err_flag, &s_abort);
+    __syncthreads();
+    float s = 0.f;
+    for (int c = tid; c < vdim; c += GLA_THREADS) s = fmaf(os[c], os[c], s);
+    s = warp_sum(s);
+    if (lane == 0) part[warp] = s;
+    for (int c = tid; c < vdim; c += GLA_THREADS) vs[c] = c == tid ? norm0 : a.norm_w ? __ldg(a.norm_w + c) : 1.f;  // the values have been used
+    __syncthreads();
+    s = 0.f;
+#pragma unroll
+    for (int w = 0; w < W; ++w) s += part[w];
+    const float f = 1.0f / sqrtf(s / (float)vdim + a.eps);
+    const int k0 = a.out_off + head * vdim;
+    auto value = [&](int c) {
+        const float y = (os[c] * f) * vs[c], z = gs[c];
+        return KIND == LIN_RETENTION ? y * (z * sigmoid(z)) : y * sigmoid(z);
+    };
+    if (a.xp && ((vdim | a.out_off) & 7) == 0) {
+        for (int c = tid * 8; c < vdim; c += GLA_THREADS * 8) {
+            float v[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = value(c + e);
+            tc_xpack_store8(a.xp, a.xp_mpad, m, k0 + c, v);
+        }
+    } else {
+        for (int c = tid; c < vdim; c += GLA_THREADS) {
+            if (a.xp) tc_xpack_store(a.xp, a.xp_mpad, m, k0 + c, value(c));
+            else a.out[(size_t)m * a.ld_out + k0 + c] = value(c);
+        }
+    }
+}
+
+template <typename K>
+cudaError_t launch(K kern, const RecurArgs& a, unsigned blocks, size_t smem, int cluster, cudaStream_t st, bool pdl) {
+    const cudaError_t e = ensure_dyn_smem(kern, smem);
     if (e != cudaSuccess) return e;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(blocks);
@@ -255,25 +424,25 @@ cudaError_t launch(const RecurArgs& a, unsigned blocks, size_t smem, cudaStream_
         at[n].val.programmaticStreamSerializationAllowed = 1;
         ++n;
     }
-    if (a.shape.cluster > 1) {
+    if (cluster > 1) {
         at[n].id = cudaLaunchAttributeClusterDimension;
-        at[n].val.clusterDim.x = (unsigned)a.shape.cluster;
+        at[n].val.clusterDim.x = (unsigned)cluster;
         at[n].val.clusterDim.y = at[n].val.clusterDim.z = 1;
         ++n;
     }
     cfg.attrs = at;
     cfg.numAttrs = n;
-    return cudaLaunchKernelEx(&cfg, recur_kernel<RD, KIND>, a);
+    return cudaLaunchKernelEx(&cfg, kern, a);
 }
 
 template <int KIND>
 cudaError_t launch_kind(const RecurArgs& a, unsigned blocks, size_t smem, cudaStream_t st, bool pdl) {
     switch (a.shape.rows) {
-        case 4: return launch<4, KIND>(a, blocks, smem, st, pdl);
-        case 8: return launch<8, KIND>(a, blocks, smem, st, pdl);
-        case 16: return launch<16, KIND>(a, blocks, smem, st, pdl);
-        case 32: return launch<32, KIND>(a, blocks, smem, st, pdl);
-        case 64: return launch<64, KIND>(a, blocks, smem, st, pdl);
+        case 4: return launch(recur_kernel<4, KIND>, a, blocks, smem, a.shape.cluster, st, pdl);
+        case 8: return launch(recur_kernel<8, KIND>, a, blocks, smem, a.shape.cluster, st, pdl);
+        case 16: return launch(recur_kernel<16, KIND>, a, blocks, smem, a.shape.cluster, st, pdl);
+        case 32: return launch(recur_kernel<32, KIND>, a, blocks, smem, a.shape.cluster, st, pdl);
+        case 64: return launch(recur_kernel<64, KIND>, a, blocks, smem, a.shape.cluster, st, pdl);
         default: return cudaErrorInvalidValue;
     }
 }
@@ -284,6 +453,12 @@ cudaError_t launch_recur(const RecurArgs& a_in, int sm_count, cudaStream_t st, b
     RecurArgs a = a_in;
     if (a.M < 1 || a.M > GQA_MAX_ROWS || a.dim > GLA_MAX_DIM || a.vdim > GLA_MAX_VDIM || a.heads % a.kv_heads != 0 || (a.kind != LIN_RETENTION && a.kind != LIN_DELTA)) return cudaErrorInvalidValue;
     const int runs = a.runs.n ? a.runs.n : a.M, rows = a.runs.n ? a.longest_run : 1;
+    // (a few tokens: more CTAs per head are worth more than the earlier loads)
+    if (rows == 1 && a.M * a.heads > sm_count && a.dim <= GLA_TOKEN_DIM && gla_state_floats(a.dim, a.vdim) * 4 <= GLA_TOKEN_BYTES) {
+        const size_t smem = (size_t)recur_token_smem(a).total * 4;
+        const unsigned blocks = (unsigned)(a.M * a.heads);
+        return a.kind == LIN_DELTA ? launch(recur_token_kernel<LIN_DELTA>, a, blocks, smem, 1, st, pdl) : launch(recur_token_kernel<LIN_RETENTION>, a, blocks, smem, 1, st, pdl);
+    }
     a.shape = gla_shape(a.dim, a.vdim, runs * a.heads, sm_count);
     for (a.step = rows; a.step > 1 && (size_t)recur_smem(a, rows).total * 4 > 110 * 1024; a.step = (a.step + 1) / 2) {
     }

@@ -1,8 +1,9 @@
 // Recurrences of linear attention over prepared rows: per head a state S [dim x vdim] in f32, one token after the other,
 //   retention    S <- decay S + k v^T                                             (a fixed decay per head)
 //   delta rule   S <- diag(alpha) S;  S <- S + k (beta (v - S^T k))^T             (a decay per key channel)
-// and o = S^T q.  A cluster of CTAs shares a head's columns and keeps them in registers while it walks through a run of tokens; between
-// passes the state lies column by column in memory, as that of gla.h.
+// and o = S^T q.  In passes over runs of tokens a cluster of CTAs shares a head's columns and keeps them in registers while it walks through
+// a run; in passes of single tokens a head's state goes through a CTA's shared memory.  Between passes the state lies column by column
+// in memory, as that of gla.h.
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -40,6 +41,7 @@ struct RecurArgs {
     unsigned char* xp;
     int xp_mpad;
     int step;                // tokens staged at a time
+    int* err_flag;
 };
 cudaError_t launch_recur(const RecurArgs& a, int sm_count, cudaStream_t st, bool pdl);
 
