@@ -257,9 +257,9 @@ int Engine::alloc_listed_cache(int batch, size_t n_pages) {
         const LayerSpec& s = spec_.layers[l];
         LayerW& w = layers_[l];
         w.conv_at = state_floats_;
-        if (s.conv > 1) state_floats_ += ((size_t)(s.conv - 1) * (s.heads * s.dim + s.kv_heads * (s.dim + (s.tied_values ? 0 : s.vdim))) + 3) / 4 * 4;
+        if (s.conv > 1) state_floats_ += ((size_t)conv_slots(s.conv) * (s.heads * s.dim + s.kv_heads * (s.dim + (s.tied_values ? 0 : s.vdim))) + 3) / 4 * 4;
         w.lin_conv_at = state_floats_;
-        if (s.lin_conv > 1) state_floats_ += ((size_t)(s.lin_conv - 1) * s.lin_channels() + 3) / 4 * 4;
+        if (s.lin_conv > 1) state_floats_ += ((size_t)conv_slots(s.lin_conv) * s.lin_channels() + 3) / 4 * 4;
         w.gla_at = state_floats_;
         if (s.linear()) state_floats_ += s.lin_heads * gla_state_floats(s.lin_dim, s.lin_vdim);
     }

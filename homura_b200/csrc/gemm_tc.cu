@@ -433,6 +433,10 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                     const float g[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
 #pragma unroll
                     for (int e = 0; e < 8; ++e) v[e] = tile[m * BM + c + e] / (1.0f + expf(-g[e]));
+                } else if (a.epi == EPI_GATE && a.gate_per > 1 && (a.gate_per & 7) == 0) {  // a piece has one gate
+                    const float f = 1.0f / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + (n0 + c) / a.gate_per)));
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) v[e] = tile[m * BM + c + e] * f;
                 } else {
 #pragma unroll
                     for (int e = 0; e < 8; ++e) v[e] = act(m, n0 + c + e, tile[m * BM + c + e]);

@@ -47,6 +47,8 @@ struct GqaRuns {
     }
 };
 
+__host__ __device__ __forceinline__ int conv_slots(int taps) { return taps > 1 ? GQA_MAX_ROWS + taps - 1 : 0; }
+
 // What happens to a projection's queries, keys and values before the attention: a short convolution, norms, rotation, temperature,
 // blended values; keys and values go to their page slots, queries to q_out.
 struct GqaPostArgs {
@@ -64,11 +66,11 @@ struct GqaPostArgs {
     const int32_t *row_pos, *row_seq;
     float* q_out;            // [M][heads * dim]
     // Causal convolution over time of every channel (queries | keys | values), taps > 0: the inputs of the last taps - 1 tokens of a
-    // sequence are kept in conv_state, position p in slot p % (taps - 1).  The warp of a run's first row serves the first taps - 1 rows,
-    // so that nobody else reads what it replaces.
+    // sequence are kept in conv_state, position p in slot p % conv_slots(taps).  The ring is longer than a pass's rows, so that the slots
+    // in front of a run are never written by the launch that reads them.
     int taps;
     const float* conv_w;     // [channels][taps], the last one meets the token itself
-    float* conv_state;       // [sequence][taps - 1][channels], sequences conv_stride floats apart
+    float* conv_state;       // [sequence][conv_slots(taps)][channels], sequences conv_stride floats apart
     size_t conv_stride;
     GqaRuns runs;            // with taps > 1
     // rotation of the first rot_dims elements of queries and keys: pair (i, i + rot_dims / 2) makes turns[i] turns per position

@@ -46,12 +46,12 @@ __device__ __forceinline__ void gqa_post_row(const GqaPostArgs& a, int m, int sl
     };
     if (buffered) {
         const float* state = a.taps > 1 ? a.conv_state + (size_t)seq * a.conv_stride + ch0 : nullptr;
-        const int channels = nq + nk + VH * vdim;
+        const int channels = nq + nk + VH * vdim, slots = conv_slots(a.taps);
         for (int d = lane; d < n; d += 32) {
             float v = ld_cg_f32(x + d);
             if (a.taps > 0) {
                 const float* w = a.conv_w + (size_t)(ch0 + d) * a.taps;
-                auto input = [&](int j) { return m - j >= first ? ld_cg_f32(x + d - (ptrdiff_t)j * a.ld) : ld_cg_f32(state + (size_t)((pos - j) % (a.taps - 1)) * channels + d); };
+                auto input = [&](int j) { return m - j >= first ? ld_cg_f32(x + d - (ptrdiff_t)j * a.ld) : ld_cg_f32(state + (size_t)((pos - j) % slots) * channels + d); };
                 const int back = min(a.taps - 1, pos);
                 float u[3] = {0.f, 0.f, 0.f};  // requested together
 #pragma unroll
@@ -180,18 +180,14 @@ __device__ __forceinline__ void gqa_post_block(const GqaPostArgs& a, int m, int 
     }
     int first, end;
     a.runs.find(m, first, end);
-    const int keep = a.taps - 1;
-    if (m > first && m < first + keep) return;  // served by the warp of the run's first row
     gqa_post_row<X>(a, m, slot, first, pos, seq, page, sq, sk, buf);
-    if (m > first) return;
-    for (int r = first + 1; r < min(end, first + keep); ++r) gqa_post_row<X>(a, r, slot, first, pos + r - first, seq, page_of(seq, pos + r - first), 0.f, 0.f, buf);
-    // the run's last inputs replace the kept ones (a lane keeps the channels that it has read)
+    if (m < end - (a.taps - 1)) return;
+    // the inputs of a run's last rows are kept
     const bool is_v = slot >= a.heads + G, is_q = slot < a.heads;
     const int h = is_v ? slot - a.heads - G : is_q ? slot : slot - a.heads, n = is_v ? vdim : dim, ch0 = (is_v ? nq + nk : is_q ? 0 : nq) + h * n, channels = nq + nk + (X == 2 ? gqa_post_v_heads(a) : G) * vdim;
-    float* state = a.conv_state + (size_t)seq * a.conv_stride + ch0;
-    for (int r = max(first, end - keep); r < end; ++r)
+    float* kept = a.conv_state + (size_t)seq * a.conv_stride + (size_t)(pos % conv_slots(a.taps)) * channels + ch0;
 #pragma unroll 4
-        for (int d = lane; d < n; d += 32) state[(size_t)((pos + r - first) % keep) * channels + d] = ld_cg_f32(a.raw + (size_t)r * a.ld + ch0 + d);
+    for (int d = lane; d < n; d += 32) kept[d] = ld_cg_f32(a.raw + (size_t)m * a.ld + ch0 + d);
 }
 
 }  // namespace hm

@@ -18,10 +18,10 @@ struct TalkGeom {
     int stages;
     uint32_t block; // bytes of a ring stage
     size_t front;   // bytes of the ring, which takes the results afterwards
-    size_t q, raw, p, corr, o, ml, talk, wts, pages, qi, pair, smem;  // offsets from the front's end, total
+    size_t q, raw, p, corr, o, ml, talk, recv, pages, qi, pair, smem;  // offsets from the front's end, total
 };
 
-inline bool talk_geom(const GqaAttnArgs& a, int rows, int nsplit, int pages_per_cta, TalkGeom* g) {
+inline bool talk_geom(const GqaAttnArgs& a, int rows, int nsplit, int pages_per_cta, size_t most, TalkGeom* g) {
     const int H = a.heads, G = a.pool.kv_heads, gq = H / G, dp = gqa_pad(a.pool.dim), vp = gqa_pad(a.pool.vdim);
     const size_t pairs = (size_t)rows * H, padded = pairs + 8;
     g->rows = rows;
@@ -42,11 +42,12 @@ inline bool talk_geom(const GqaAttnArgs& a, int rows, int nsplit, int pages_per_
     g->o = take((size_t)G * (vp / 16) * g->ntile * g->cols2 * 8 * 16);
     g->ml = take(pairs * 8);
     g->talk = take((size_t)H * ((H + 3) / 4 * 4) * 4);
-    g->wts = take(pairs * nsplit * 4);
+    // what a CTA receives: from every split, its share of the pairs (values, maximum, sum)
+    g->recv = take(nsplit > 1 ? nsplit * ((pairs + nsplit - 1) / nsplit) * (vp + 4) * 4 : 0);
     g->pages = take((size_t)pages_per_cta * 4);
     g->qi = take(pairs * 2);
     g->pair = take((size_t)g->per * 2);
-    const size_t result = pairs * (vp + 4) * 4, most = 226 * 1024;
+    const size_t result = pairs * (vp + 4) * 4;
     if (at + std::max(result, 2 * (size_t)g->block) + 128 > most) return false;
     g->stages = (int)std::min<size_t>({(most - at - 128) / g->block, (size_t)TALK_MAX_STAGES, (size_t)2 * G * std::max(1, pages_per_cta)});
     g->front = (std::max(result, (size_t)g->stages * g->block) + 127) / 128 * 128;
@@ -133,7 +134,7 @@ __device__ __forceinline__ void talk_mix(const GqaAttnArgs& a, int r, int h0, in
     __syncwarp();
 }
 
-__global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const __grid_constant__ GqaAttnArgs a, const __grid_constant__ TalkGeom geo) {
+__global__ void __launch_bounds__(B_THREADS, 2) talk_attn_mma_kernel(const __grid_constant__ GqaAttnArgs a, const __grid_constant__ TalkGeom geo) {
     extern __shared__ __align__(128) unsigned char dyn[];
     const int H = a.heads, G = a.pool.kv_heads, gq = H / G, dim = a.pool.dim, vdim = a.pool.vdim, dp = gqa_pad(dim), vp = gqa_pad(vdim), kt_n = dp / 16, vt_n = vp / 16, ldo = vp + 4;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, split = blockIdx.x, NST = geo.stages, HP = (H + 3) & ~3;
@@ -146,11 +147,11 @@ __global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const __gri
     float4* os = reinterpret_cast<float4*>(back + geo.o);            // [key head][16 values][tile of pairs][two columns][8 lanes]
     float* ml = reinterpret_cast<float*>(back + geo.ml);             // [row][head][2]
     float* tk = reinterpret_cast<float*>(back + geo.talk);           // [head that is read][head, padded]
-    float* wts = reinterpret_cast<float*>(back + geo.wts);
+    float* recv = reinterpret_cast<float*>(back + geo.recv);         // [split][pairs of this CTA][vp + 4]
     int32_t* pt_s = reinterpret_cast<int32_t*>(back + geo.pages);
     uint16_t* qi = reinterpret_cast<uint16_t*>(back + geo.qi);       // [row][head] -> pair by key head
     uint16_t* pair = reinterpret_cast<uint16_t*>(back + geo.pair);   // pair of the first key head -> [row][head]
-    __shared__ uint64_t full[TALK_MAX_STAGES], empty[TALK_MAX_STAGES];
+    __shared__ uint64_t full[TALK_MAX_STAGES], empty[TALK_MAX_STAGES], s_rbar;
     __shared__ volatile int s_abort;
 
     int row0 = blockIdx.z, rows = 1;
@@ -161,13 +162,24 @@ __global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const __gri
         rows = min(geo.rows, a.runs.row[r + 1] - row0);
     }
     const int pairs = rows * H;
+    // the splits of a tile share its pairs: pair p is combined and stored by split p % ns
+    const int ns = a.nsplit, rank = ns > 1 ? (int)cluster_ctarank() : 0, own = pairs > rank ? (pairs - rank + ns - 1) / ns : 0, own_most = (geo.rows * H + ns - 1) / ns;
     if (tid < NST) {
         mb_init(&full[tid], 1);
         mb_init(&empty[tid], ATT_WARPS);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
-    if (tid == 0) s_abort = 0;
+    if (tid == 0) {
+        s_abort = 0;
+        mb_init(&s_rbar, 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        if (ns > 1 && own > 0) mb_expect_tx(&s_rbar, (uint32_t)((ns - 1) * own * (vp + 2) * 4));
+    }
     pdl_launch_dependents();
+    if (ns > 1) {
+        cluster_arrive_release();
+        cluster_wait_acquire();
+    }
     // positions, pages and the mixing matrix do not depend on the launch in front
     const int seq = a.row_seq[row0], pos0 = a.row_pos[row0], len = pos0 + rows;
     const PageList list = visible_pages<true>(a, pos0, len - 1);
@@ -354,11 +366,61 @@ __global__ void __launch_bounds__(B_THREADS, 1) talk_attn_mma_kernel(const __gri
             }
         }
     }
-    combine_and_store<true>(a, res, ldo, ml, wts, pairs, [&](int p, int& row, int& head) {
+    __syncthreads();
+    auto store = [&](int p, int d0, float (&v)[8]) {
         const int r = rows == 1 ? 0 : p / H;
-        row = row0 + r;
-        head = p - r * H;
-    });
+        store_piece<true>(a, row0 + r, p - r * H, d0, v);
+    };
+    const int np8 = vp / 8, np4 = vp / 4;
+    if (ns == 1) {
+        for (int i = tid; i < pairs * np8; i += B_THREADS) {
+            const int p = i / np8, d0 = (i - p * np8) * 8;
+            const float4 x = *reinterpret_cast<const float4*>(res + (size_t)p * ldo + d0), y = *reinterpret_cast<const float4*>(res + (size_t)p * ldo + d0 + 4);
+            const int h = rows == 1 ? p : p % H;
+            const float f = 1.0f / (ml[2 * p + 1] + sink_weight<true>(a, h, ml[2 * p]));
+            float v[8] = {x.x * f, x.y * f, x.z * f, x.w * f, y.x * f, y.y * f, y.z * f, y.w * f};
+            if (d0 < vdim) store(p, d0, v);
+        }
+        return;
+    }
+    for (int i = tid; i < pairs * np4; i += B_THREADS) {
+        const int p = i / np4, d = (i - p * np4) * 4, k = p / ns;
+        const uint32_t owner = (uint32_t)(p - k * ns);
+        const float4 v = *reinterpret_cast<const float4*>(res + (size_t)p * ldo + d);
+        float* slot = recv + (size_t)(rank * own_most + k) * (vp + 4);
+        if ((int)owner == rank) {
+            *reinterpret_cast<float4*>(slot + d) = v;
+            if (d == 0) {
+                slot[vp] = ml[2 * p];
+                slot[vp + 1] = ml[2 * p + 1];
+            }
+        } else {
+            const uint32_t bar = dsmem_addr(&s_rbar, owner);
+            st_async_f32x4(dsmem_addr(slot + d, owner), v, bar);
+            if (d == 0) st_async_f32x2(dsmem_addr(slot + vp, owner), ml[2 * p], ml[2 * p + 1], bar);
+        }
+    }
+    if (own == 0) return;
+    __syncthreads();
+    if (!mb_wait_cluster(&s_rbar, 0, a.err_flag, &s_abort)) return;  // bounded
+    for (int i = tid; i < own * np8; i += B_THREADS) {
+        const int k = i / np8, d0 = (i - k * np8) * 8, p = k * ns + rank;
+        float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, mx = -INFINITY, l = 0.f;
+        for (int r = 0; r < ns; ++r) mx = fmaxf(mx, recv[(size_t)(r * own_most + k) * (vp + 4) + vp]);
+#pragma unroll 4
+        for (int r = 0; r < ns; ++r) {
+            const float* slot = recv + (size_t)(r * own_most + k) * (vp + 4);
+            const float f = slot[vp] == -INFINITY ? 0.f : exp2f(slot[vp] - mx);
+            const float4 x = *reinterpret_cast<const float4*>(slot + d0), y = *reinterpret_cast<const float4*>(slot + d0 + 4);
+            l = fmaf(f, slot[vp + 1], l);
+            v[0] = fmaf(f, x.x, v[0]); v[1] = fmaf(f, x.y, v[1]); v[2] = fmaf(f, x.z, v[2]); v[3] = fmaf(f, x.w, v[3]);
+            v[4] = fmaf(f, y.x, v[4]); v[5] = fmaf(f, y.y, v[5]); v[6] = fmaf(f, y.z, v[6]); v[7] = fmaf(f, y.w, v[7]);
+        }
+        const float inv = 1.0f / (l + sink_weight<true>(a, rows == 1 ? p : p % H, mx));
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= inv;
+        if (d0 < vdim) store(p, d0, v);
+    }
 }
 
 inline size_t talk_plain_smem(int heads, int dp, int vp, int nsplit) { return sizeof(float) * (size_t)heads * (dp + vp + 4 + 2 * GQA_PAGE + 3 + nsplit); }
@@ -382,16 +444,22 @@ inline cudaError_t launch_talk(GqaAttnArgs a, int sm_count, cudaStream_t st, boo
                 }
                 a.runs.tile[a.runs.n] = (uint16_t)a.tiles;
             }
+            // first as many splits as keep two CTAs on every SM, which hide one another's barriers, then one with a deep ring
             bool fits = false;
-            auto shape = [&]() { return fits = talk_geom(a, rows, a.nsplit, (pages + a.nsplit - 1) / a.nsplit, &g); };
-            if (asked > 0) {
-                a.nsplit = asked;
-                shape();
-            } else {
-                for (a.nsplit = std::max(1, std::min({sm_count / a.tiles, a.max_cluster, 8, pages})); a.nsplit >= 1; --a.nsplit)
-                    if (shape() && (a.nsplit == 1 || clusters_at_once(talk_attn_mma_kernel, a.nsplit, B_THREADS, g.smem) >= a.tiles)) break;
+            for (int per_sm = pages > 2 ? 2 : 1; per_sm >= 1 && !fits; --per_sm) {
+                const size_t most = (per_sm == 2 ? 112 : 226) * 1024;
+                auto shape = [&](int n) {
+                    a.nsplit = n;
+                    return talk_geom(a, rows, n, (pages + n - 1) / n, most, &g) && (per_sm == 1 || g.stages >= 4);
+                };
+                if (asked > 0) {
+                    fits = shape(asked);
+                    continue;
+                }
+                for (int n = std::max(1, std::min({per_sm * sm_count / a.tiles, a.max_cluster, 8, pages})); n >= 1 && !fits; --n)
+                    fits = shape(n) && (n == 1 || clusters_at_once(talk_attn_mma_kernel, n, B_THREADS, g.smem) >= a.tiles);
             }
-            if (fits && a.nsplit >= 1) return launch_clustered(talk_attn_mma_kernel, dim3((unsigned)a.nsplit, 1, (unsigned)a.tiles), dim3(B_THREADS), g.smem, a.nsplit, st, pdl, a, g);
+            if (fits) return launch_clustered(talk_attn_mma_kernel, dim3((unsigned)a.nsplit, 1, (unsigned)a.tiles), dim3(B_THREADS), g.smem, a.nsplit, st, pdl, a, g);
         }
         a.nsplit = asked;
     }

@@ -234,6 +234,7 @@ struct TclGeom {
     int stages;
     int look;      // scores of the next tile are issued before the weights of this one are ready (two score accumulators)
     int cols;      // TMEM columns, a power of two
+    int pad;       // bytes by which the ring's second tile moves up to the end of the first, whose last slice is half full (rings of two tiles)
     int q_bytes, p_bytes, s_bytes;
     size_t smem;
     __host__ __device__ int slice() const { return 2 * tok * 128; }  // bytes of 128 elements of a tile's tokens: two K-major halves
@@ -252,6 +253,11 @@ bool tcl_geom_tok(int tok, int rank, int pairs, TclGeom* g) {
     const int fixed = g->q_bytes + g->p_bytes + g->s_bytes + 1024;
     g->stages = (222 * 1024 - fixed) / g->slice();
     if (g->stages > TCL_MAXSTG) g->stages = TCL_MAXSTG;
+    g->pad = 0;
+    if ((g->kbs & 1) && g->stages == 2 * g->nb - 1 && 2 * g->nb <= TCL_MAXSTG && g->kbs * g->slice() + fixed <= 222 * 1024) {
+        g->stages = 2 * g->nb;
+        g->pad = g->slice() / 2;
+    }
     if (g->stages < (g->nb > 2 ? g->nb : 2)) return false;  // the values of a tile are needed after its scores: the ring holds a whole tile
     g->look = g->stages >= 2 * g->nb && (g->nb + 2) * g->n <= 512 ? 1 : 0;
     const int need = (g->nb + 1 + g->look) * g->n;
@@ -260,8 +266,8 @@ bool tcl_geom_tok(int tok, int rank, int pairs, TclGeom* g) {
     while (g->cols < need) g->cols *= 2;
     // two CTAs per SM where their tensor memory and a ring of two tiles and a slice allow it
     const int pair = (TCL_PAIR_SMEM - fixed) / g->slice();
-    if (g->look && g->cols <= 256 && pair >= 2 * g->nb) g->stages = pair < TCL_MAXSTG ? pair : TCL_MAXSTG;
-    g->smem = (size_t)fixed + (size_t)g->stages * g->slice();
+    if (g->look && g->pad == 0 && g->cols <= 256 && pair >= 2 * g->nb) g->stages = pair < TCL_MAXSTG ? pair : TCL_MAXSTG;
+    g->smem = (size_t)fixed + (size_t)g->stages * g->slice() - g->pad;
     return true;
 }
 bool tcl_geom(int rank, int pairs, TclGeom* g) {
@@ -285,7 +291,8 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
     __shared__ TclShared sh;
     constexpr int SLICE = 2 * TOK * 128, PAGES = TOK / LATENT_PAGE, SLD = TOK, TPL = TOK / 32;  // bytes, pages per tile, score row, tokens per lane
     unsigned char* ring = tcl_smem + ((1024u - (s32(tcl_smem) & 1023u)) & 1023u);
-    unsigned char* qs = ring + (size_t)g.stages * SLICE;   // [kbs][n][128 B]
+    auto stage_at = [&](int s) { return (uint32_t)s * SLICE - (s >= g.nb ? (uint32_t)g.pad : 0u); };  // bytes from the ring's front
+    unsigned char* qs = ring + stage_at(g.stages);         // [kbs][n][128 B]
     unsigned char* pb = qs + g.q_bytes;                    // [2][TOK / 64][n][128 B]
     float* sc = reinterpret_cast<float*>(pb + g.p_bytes);  // [np][SLD]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -387,7 +394,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                     for (int hf = 0; hf < halves; ++hf)
 #pragma unroll
                         for (int i = 0; i < PAGES; ++i)
-                            bulk_copy(ring + (size_t)s * SLICE + hf * (SLICE / 2) + i * piece, pool + ((size_t)cur[i] * g.kbs + 2 * b + hf) * piece, piece, &sh.full[s]);
+                            bulk_copy(ring + stage_at(s) + hf * (SLICE / 2) + i * piece, pool + ((size_t)cur[i] * g.kbs + 2 * b + hf) * piece, piece, &sh.full[s]);
                     if (++s == g.stages) {
                         s = 0;
                         phase ^= 1;
@@ -420,7 +427,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                     uint32_t d = base_o;
                     const uint32_t p = plo + (uint32_t)(t & 1) * (TOK / 64) * row_block;
                     for (int b = 0; b < g.nb; ++b, d += g.n) {
-                        const uint32_t v = vlo + (uint32_t)pv_stage * (SLICE / 16);
+                        const uint32_t v = vlo + stage_at(pv_stage) / 16;
                         if (lead) {
 #pragma unroll
                             for (int ks = 0; ks < TOK / 16; ++ks) mma_bf16(d, v + ks * 128, p + (ks >> 2) * row_block + (ks & 3) * 2, id_o, t > 0 || ks > 0);
@@ -435,7 +442,7 @@ __global__ void __launch_bounds__(TCL_THREADS, 2) latent_attn_tc_kernel(const La
                 } else if (ks_tile < upto && ready(&sh.full[ks_stage], ks_phase)) {
                     // scores of one slice; the last slice of a tile publishes the tile's scores
                     tc_fence_after();
-                    const uint32_t d = base + (g.look ? (uint32_t)((ks_tile & 1) * g.n) : 0u), k = klo + (uint32_t)ks_stage * (SLICE / 16);
+                    const uint32_t d = base + (g.look ? (uint32_t)((ks_tile & 1) * g.n) : 0u), k = klo + stage_at(ks_stage) / 16;
                     const bool two = 2 * ks_slice + 1 < g.kbs;
                     if (lead) {
 #pragma unroll

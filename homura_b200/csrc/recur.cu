@@ -159,9 +159,13 @@ __global__ void __launch_bounds__(GLA_THREADS, RD > 32 ? 1 : 2) recur_kernel(con
             }
             __syncthreads();
             if constexpr (KIND == LIN_DELTA) {  // k . q: what a token's own write adds to its result
+#pragma unroll 4
                 for (int t = warp; t < tr; t += GLA_THREADS / 32) {
                     float s = 0.f;
-                    for (int d = lane; d < DP; d += 32) s = fmaf(ks[t * DP + d], qs[t * DP + d], s);
+                    for (int d = lane * 4; d < DP; d += 128) {
+                        const float4 x = *reinterpret_cast<const float4*>(ks + t * DP + d), y = *reinterpret_cast<const float4*>(qs + t * DP + d);
+                        s = fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, s))));
+                    }
                     s = warp_sum(s);
                     if (lane == 0) kq[t] = s;
                 }
@@ -204,31 +208,51 @@ __global__ void __launch_bounds__(GLA_THREADS, RD > 32 ? 1 : 2) recur_kernel(con
                     if (part == 0 && on) orow[t * share] = o;
                 }
             } else {
+                // with few rows a thread requests the next token's before this one's sums go through the lanes
+                constexpr bool AHEAD = RD <= 8;
+                float4 nq[AHEAD ? RD / 4 : 1], nk[AHEAD ? RD / 4 : 1], na[AHEAD ? RD / 4 : 1];
+                auto request = [&](int t) {
+                    if constexpr (AHEAD) {
+#pragma unroll
+                        for (int j = 0; j < RD / 4; ++j) {
+                            na[j] = (reinterpret_cast<const float4*>(as + t * DP) + part)[j * LP];
+                            nk[j] = (reinterpret_cast<const float4*>(ks + t * DP) + part)[j * LP];
+                            nq[j] = (reinterpret_cast<const float4*>(qs + t * DP) + part)[j * LP];
+                        }
+                    }
+                };
+                request(0);
                 for (int t = 0; t < tr; ++t) {
                     const float4 *q4 = reinterpret_cast<const float4*>(qs + t * DP) + part, *k4 = reinterpret_cast<const float4*>(ks + t * DP) + part, *a4 = reinterpret_cast<const float4*>(as + t * DP) + part;
+                    const float v = vs[t * CP + col], beta = bs[t], own = kq[t];
+                    float4 kt[AHEAD ? RD / 4 : 1];
                     // both sums over the shrunk state go through the lanes side by side: what it gives back for k, and for q
                     float sk0 = 0.f, sk1 = 0.f, sq0 = 0.f, sq1 = 0.f;
 #pragma unroll
                     for (int j = 0; j < RD / 4; ++j) {
-                        const float4 al = a4[j * LP], k = k4[j * LP], q = q4[j * LP];
+                        const float4 al = AHEAD ? na[AHEAD ? j : 0] : a4[j * LP], k = AHEAD ? nk[AHEAD ? j : 0] : k4[j * LP], q = AHEAD ? nq[AHEAD ? j : 0] : q4[j * LP];
+                        if (AHEAD) kt[AHEAD ? j : 0] = k;
                         S[j].x *= al.x; S[j].y *= al.y; S[j].z *= al.z; S[j].w *= al.w;
                         sk0 = fmaf(S[j].x, k.x, fmaf(S[j].y, k.y, sk0));
                         sk1 = fmaf(S[j].z, k.z, fmaf(S[j].w, k.w, sk1));
                         sq0 = fmaf(S[j].x, q.x, fmaf(S[j].y, q.y, sq0));
                         sq1 = fmaf(S[j].z, q.z, fmaf(S[j].w, q.w, sq1));
                     }
+                    request(min(t + 1, tr - 1));
                     float sk = sk0 + sk1, so = sq0 + sq1;
-                    for (int s = 1; s < LP; s <<= 1) {
-                        sk += __shfl_xor_sync(0xffffffffu, sk, s);
-                        so += __shfl_xor_sync(0xffffffffu, so, s);
-                    }
-                    const float u = bs[t] * (vs[t * CP + col] - sk);
+#pragma unroll
+                    for (int s = 1; s < 32; s <<= 1)
+                        if (s < LP) {
+                            sk += __shfl_xor_sync(0xffffffffu, sk, s);
+                            so += __shfl_xor_sync(0xffffffffu, so, s);
+                        }
+                    const float u = beta * (v - sk);
 #pragma unroll
                     for (int j = 0; j < RD / 4; ++j) {
-                        const float4 k = k4[j * LP];
+                        const float4 k = AHEAD ? kt[AHEAD ? j : 0] : k4[j * LP];
                         S[j].x = fmaf(k.x, u, S[j].x); S[j].y = fmaf(k.y, u, S[j].y); S[j].z = fmaf(k.z, u, S[j].z); S[j].w = fmaf(k.w, u, S[j].w);
                     }
-                    if (part == 0 && on) orow[t * share] = fmaf(kq[t], u, so);
+                    if (part == 0 && on) orow[t * share] = fmaf(own, u, so);
                 }
             }
             if (slices == 1) finish(t0, tr);
