@@ -478,16 +478,16 @@ struct GemvExt : GemvBase {
     const float* out_scale;  // [N] or null (EPI_STORE: the result is multiplied element by element before the residual is added)
     const float* gate;   // EPI_GATE: [M][ld_gate]
     int ld_gate;
-    int gate_per;        // EPI_GATE: > 1: so many columns share a gate
-    float limit;         // EPI_GLU
-    int glu_n;           // EPI_GLU: outputs (the last block may be padded)
-    bool extended() const { return pro == PRO_GNORM || pro == PRO_MERGE || epi == EPI_GATE || epi == EPI_SQRELU || epi == EPI_GLU || group_slabs != 0 || out_scale != nullptr; }
+    bool extended() const { return pro == PRO_GNORM || pro == PRO_MERGE || epi == EPI_GATE || epi == EPI_SQRELU || group_slabs != 0 || out_scale != nullptr; }
 };
-// And of the variant behind that (gemv_turn.cu): rotation and capped logits in the epilogue.
+// And of the variant behind that (gemv_turn.cu): rotation, capped logits, clamped gated activations and shared gates in the epilogue.
 struct GemvArgs : GemvExt {
     TurnedPairs turn;    // EPI_STORE: with turn.turns
     float softcap;       // EPI_LOGITS: > 0: softcap * tanh(logit / softcap)
-    int variant() const { return turn.turns != nullptr || softcap > 0.f ? 2 : extended() ? 1 : 0; }
+    int gate_per;        // EPI_GATE: > 1: so many columns share a gate
+    float limit;         // EPI_GLU
+    int glu_n;           // EPI_GLU: outputs (the last block may be padded)
+    int variant() const { return turn.turns != nullptr || softcap > 0.f || epi == EPI_GLU || gate_per > 1 ? 2 : extended() ? 1 : 0; }
 };
 
 struct AttnArgs {

@@ -251,7 +251,7 @@ __global__ void __launch_bounds__(256) tc_pack_gnorm_kernel(const float* __restr
 __device__ __forceinline__ bool tc_better(float v, int i, float bv, int bi) { return v > bv || (v == bv && i > bi); }
 
 // V: 1 is the extended variant (grouped weights, output scale, gate, squared ReLU, queries split into images), 2 that of mixtures of
-// experts, 3 the extended one with rotation and capped logits, compiled apart so that the plain projections carry none of it.
+// experts, 3 the extended one with rotation, capped logits, clamped gated activations and gates that columns share, compiled apart so that the plain projections carry none of it.
 template <int V>
 __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, int nblk, int tid, const int* s_pos, const int* s_page) {
     // grouped projections: this block's output columns [n0, n_end)
@@ -395,7 +395,7 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
                 }
             }
         }
-    } else if (X && a.epi == EPI_GLU) {
+    } else if (V == 3 && a.epi == EPI_GLU) {
         // block = 64 gate features followed by the 64 matching up features; padding ones come out as zero
         for (int idx = tid; idx < rows * 8; idx += TC_THREADS) {
             const int m = m_lo + idx / 8, c = (idx % 8) * 8, j = nblk * 64 + c;
@@ -419,7 +419,7 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
         }
     } else if (X && (a.epi == EPI_GATE || a.epi == EPI_SQRELU)) {
         auto act = [&](int m, int n, float v) {
-            if (a.epi == EPI_GATE) return v / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + (a.gate_per > 1 ? n / a.gate_per : n))));
+            if (a.epi == EPI_GATE) return v / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + (V == 3 && a.gate_per > 1 ? n / a.gate_per : n))));
             v = fmaxf(v, 0.f);
             return v * v;
         };
@@ -428,12 +428,12 @@ __device__ void tc_epilogue(const TcArgs& a, float* tile, int m_lo, int m_hi, in
             for (int idx = tid; idx < rows * nc; idx += TC_THREADS) {
                 const int m = m_lo + idx / nc, c = (idx % nc) * 8;
                 float v[8];
-                if (a.epi == EPI_GATE && a.gate_per <= 1 && (a.ld_gate & 3) == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 15) == 0) {
+                if (a.epi == EPI_GATE && (V != 3 || a.gate_per <= 1) && (a.ld_gate & 3) == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 15) == 0) {
                     const float4 g0 = ld_cg_f32x4(a.gate + (size_t)m * a.ld_gate + n0 + c), g1 = ld_cg_f32x4(a.gate + (size_t)m * a.ld_gate + n0 + c + 4);
                     const float g[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
 #pragma unroll
                     for (int e = 0; e < 8; ++e) v[e] = tile[m * BM + c + e] / (1.0f + expf(-g[e]));
-                } else if (a.epi == EPI_GATE && a.gate_per > 1 && (a.gate_per & 7) == 0) {  // a piece has one gate
+                } else if (V == 3 && a.epi == EPI_GATE && a.gate_per > 1 && (a.gate_per & 7) == 0) {  // a piece has one gate
                     const float f = 1.0f / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + (n0 + c) / a.gate_per)));
 #pragma unroll
                     for (int e = 0; e < 8; ++e) v[e] = tile[m * BM + c + e] * f;
@@ -947,9 +947,9 @@ static cudaError_t launch_gemm_tc_v(const TcArgs& a_in, cudaStream_t st, bool pd
 }
 
 cudaError_t launch_gemm_tc(const TcArgs& a, cudaStream_t st, bool pdl) {
-    const bool x = a.group_blocks || a.out_scale || a.split_xp || a.epi == EPI_GATE || a.epi == EPI_SQRELU || a.epi == EPI_GLU;
+    const bool x = a.group_blocks || a.out_scale || a.split_xp || a.epi == EPI_GATE || a.epi == EPI_SQRELU;
     if (a.ex.n) return launch_gemm_tc_v<2>(a, st, pdl);
-    if (a.turn.turns || a.softcap > 0.f) return launch_gemm_tc_v<3>(a, st, pdl);
+    if (a.turn.turns || a.softcap > 0.f || a.epi == EPI_GLU || (a.epi == EPI_GATE && a.gate_per > 1)) return launch_gemm_tc_v<3>(a, st, pdl);
     return x ? launch_gemm_tc_v<1>(a, st, pdl) : launch_gemm_tc_v<0>(a, st, pdl);
 }
 

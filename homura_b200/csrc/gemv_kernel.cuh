@@ -1,6 +1,6 @@
 // The kernel of the weight-streaming bf16 projection and its launcher; instantiated by gemv_bf16.cu (X = 0: the plain
 // projections), gemv_ext.cu (X = 1: grouped norm, split merge, grouped weights, gate, squared ReLU, output scale) and gemv_turn.cu
-// (X = 2: rotation and capped logits as well).
+// (X = 2: rotation, capped logits, clamped gated activations and gates shared by columns as well).
 #pragma once
 #include <type_traits>
 
@@ -590,7 +590,9 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
         if (a.epi == EPI_GATE) {
             for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) {
                 const int m = idx / SLAB, n = n0 + (idx % SLAB);
-                if (n < n_end && m < a.m_valid) a.y[(size_t)m * a.ldy + n] = vals[idx] / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + (a.gate_per > 1 ? n / a.gate_per : n))));
+                int gate = n;
+                if constexpr (X == 2) gate = a.gate_per > 1 ? n / a.gate_per : n;
+                if (n < n_end && m < a.m_valid) a.y[(size_t)m * a.ldy + n] = vals[idx] / (1.0f + expf(-ld_cg_f32(a.gate + (size_t)m * a.ld_gate + gate)));
             }
         } else if (a.epi == EPI_SQRELU) {
             for (int idx = tid; idx < M * SLAB; idx += GEMV_THREADS) {
@@ -601,6 +603,9 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
                 }
             }
         }
+        stored = a.epi == EPI_GATE || a.epi == EPI_SQRELU;
+    }
+    if constexpr (X == 2) {
         if (a.epi == EPI_GLU) {
             for (int idx = tid; idx < M * 64; idx += GEMV_THREADS) {
                 const int m = idx / 64, c = idx % 64, j = slab * 64 + c;
@@ -614,7 +619,7 @@ __global__ void __launch_bounds__(GEMV_THREADS, CL ? (M <= 4 ? 2 : 1) : (M == 1 
                 }
             }
         }
-        stored = a.epi == EPI_GATE || a.epi == EPI_SQRELU || a.epi == EPI_GLU;
+        stored = stored || a.epi == EPI_GLU;
     }
     if (stored) {
     } else if (a.epi == EPI_STORE) {

@@ -1,4 +1,4 @@
-// The variant of the weight-streaming projection with rotation and capped logits (see gemv_kernel.cuh).
+// The variant of the weight-streaming projection with rotation, capped logits, clamped gated activations and shared gates (see gemv_kernel.cuh).
 #include "gemv_kernel.cuh"
 
 namespace hm {

@@ -730,7 +730,7 @@ int latent_pick_nsplit(int tiles, int rows_per_tile, int heads, int rank, int bf
     const int hpc = mp ? tcl_heads(heads, mp) : CC_HEADS, ctas = tiles * ((heads + hpc - 1) / hpc);
     TclGeom g;
     const bool tc = mp > 0 && tcl_geom(rank, rows_per_tile * hpc, &g);
-    const int tok = tc ? (free_merge ? g.tok : 128) : CC_TOK, most = (longest + tok - 1) / tok;
+    const int tok = tc ? g.tok : CC_TOK, most = (longest + tok - 1) / tok;
     const int slots = tc && g.smem <= TCL_PAIR_SMEM && g.cols <= 256 ? 2 * sm_count : sm_count;  // CTAs resident at once
     int s = slots / (ctas > 0 ? ctas : 1);
     if (s > most) s = most;
