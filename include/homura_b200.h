@@ -110,7 +110,7 @@ HM_API int hm_model_load_gguf(const char* gguf_path, int device, hm_engine** out
 HM_API int hm_engine_create(const hm_config* cfg, int device, hm_engine** out);
 /* The same from the text of a config.json, for every design the library knows (its "architecture" key, e.g. "Tunitar", or
  * the Qwen2 / Qwen3 / Llama keys).  weight_dtype as in hm_model_load.  A tensor whose shape tells a size that the text does not
- * ("Gebilorn": mix.right.a1) comes before the other tensors of its layer. */
+ * ("Gebilorn": mix.right.a1) comes before the other tensors of its layer ("Pulenex": in any order). */
 HM_API int hm_engine_create_json(const char* config_json, int weight_dtype, int device, hm_engine** out);
 /* Name of the design, "" for the uniform Qwen2 / Qwen3 / Llama stacks.  Valid until the engine is destroyed. */
 HM_API const char* hm_get_arch(hm_engine* e);

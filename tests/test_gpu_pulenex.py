@@ -287,7 +287,7 @@ def test_mixed_batches_and_reused_pages(hm, engines, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["F32", "BF16"])
-@pytest.mark.parametrize("name", ["large", "parallel"])
+@pytest.mark.parametrize("name", ["large", "parallel", "retention", "odd", "mixed"])
 def test_many_sequences_in_a_pass(hm, engines, name, dtype):
     """Forty sequences: a prompt each, then passes that mix single tokens with portions, then the captured step."""
     m = engines(name, dtype)
