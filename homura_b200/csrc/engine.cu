@@ -78,7 +78,7 @@ int Engine::create(const ModelSpec& spec, int device, bool strict_f32, Engine** 
         for (const LayerSpec& l : spec.layers) {
             e->qdim_ = std::max(e->qdim_, l.heads * std::max(l.vdim, l.paged_kv() ? l.dim : l.q_rank ? l.q_stride() : 0));
             if (spec.sandwich && e->H_ > SANDWICH_MAX_WIDTH) return bad("width must be at most 16384");
-            if (l.talking && !gqa_talk_fits(l.heads, l.dim, l.vdim)) return bad("heads that mix their scores must fit one SM together (heads * (dim + vdim) up to about 40000)");
+            if (l.talking && !gqa_talk_fits(l.heads, l.dim, l.vdim)) return bad("heads that mix their scores must fit one SM together (heads * (dim + vdim + 151) up to 57856)");
             if (l.latent_rank() > 1024) return bad("kv_rank (with rot_dim) must be at most 1024");
             if (l.linear() && (l.lin_dim > GLA_MAX_DIM || l.lin_vdim > GLA_MAX_VDIM)) return bad("linear attention heads have at most 1024 key and 512 value elements");
             if (l.experts > 1024) return bad("a mixture has at most 1024 experts");
